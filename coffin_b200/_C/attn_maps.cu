@@ -1,0 +1,187 @@
+// Attention with several score maps per head over the same values: key/value append, the plain row kernel (any
+// sizes, fp32 or bf16 pages) and the kernel that merges key splits, combines the maps and finishes the head.
+// The tensor-core kernels for prompts and decoding are attn_maps_flash.cu.
+#include "attn_maps.cuh"
+
+namespace {
+
+template <typename TP, typename TA>
+__global__ void __launch_bounds__(256) maps_append_kernel(const AttnMapsArgs a) {
+  griddep_launch();
+  griddep_wait();
+  const int row = blockIdx.x, seg = a.row_seg ? a.row_seg[row] : row, pos = a.positions[row];
+  if (pos < 0) return;
+  const int64_t slot = (int64_t)a.tables[(int64_t)seg * a.ldbt + pos / kPage] * kPage + pos % kPage;
+  const TP* p = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
+  const int nk = a.G * a.maps * a.dim, nv = a.G * a.vdim;
+  TA* kp = reinterpret_cast<TA*>(a.kpool) + slot * nk;
+  TA* vp = reinterpret_cast<TA*>(a.vpool) + slot * nv;
+  for (int c = threadIdx.x; c < nk; c += 256) act_store(kp + c, act_load(p + a.k_col + c));
+  for (int c = threadIdx.x; c < nv; c += 256) act_store(vp + c, act_load(p + a.v_col + c));
+}
+
+// One CTA per (query row, head, map): 128 keys at a time, scores by thread, running softmax, values by column.
+constexpr int kRT = 128;
+template <typename TP, typename TA>
+__global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  float* q = sm;                 // [dim]
+  float* pr = q + a.dim;         // [kRT]
+  float* o = pr + kRT;           // [vdim]
+  const int tid = threadIdx.x, vh = blockIdx.x, row = blockIdx.y;
+  griddep_launch();
+  griddep_wait();
+  const int seg = a.row_seg ? a.row_seg[row] : row, pos = a.positions[row];
+  const int h = vh / a.maps, map = vh % a.maps, g = h / (a.H / a.G);
+  float* po = a.part_o + ((int64_t)row * a.H * a.maps + vh) * a.nsplit * a.vdim;
+  float* pm = a.part_ml + ((int64_t)row * a.H * a.maps + vh) * a.nsplit * 2;
+  if (pos < 0) return;
+  const float f = a.scale * query_temp(a, pos), inv_cap = a.cap > 0.f ? 1.f / a.cap : 0.f;
+  const TP* qr = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp + (int64_t)vh * a.dim;
+  for (int c = tid; c < a.dim; c += kRT) q[c] = act_round<TA>(act_load(qr + c)) * f;
+  for (int c = tid; c < a.vdim; c += kRT) o[c] = 0.f;
+  __syncthreads();
+  const int64_t ldk = (int64_t)a.G * a.maps * a.dim, ldv = (int64_t)a.G * a.vdim;
+  const TA* K = reinterpret_cast<const TA*>(a.kpool) + (int64_t)(g * a.maps + map) * a.dim;
+  const TA* V = reinterpret_cast<const TA*>(a.vpool) + (int64_t)g * a.vdim;
+  const int* bt = a.tables + (int64_t)seg * a.ldbt;
+  float m = -INFINITY, l = 0.f;
+  for (int k0 = 0; k0 <= pos; k0 += kRT) {
+    const int n = min(kRT, pos + 1 - k0), j = k0 + tid;
+    float s = -INFINITY;
+    if (tid < n) {
+      const TA* kr = K + ((int64_t)bt[j / kPage] * kPage + j % kPage) * ldk;
+      float d = 0.f;
+      for (int c = 0; c < a.dim; ++c) d = fmaf(q[c], act_load(kr + c), d);
+      s = a.cap > 0.f ? a.cap * tanhf(d * inv_cap) : d;
+    }
+    const float mn = fmaxf(m, block_max(s, red));
+    const float p = tid < n ? expf(s - mn) : 0.f, w = expf(m - mn);
+    pr[tid] = p;
+    l = l * w + block_sum(p, red);
+    m = mn;
+    __syncthreads();
+    for (int c = tid; c < a.vdim; c += kRT) {
+      float acc = o[c] * w;
+      for (int i = 0; i < n; ++i) {
+        const int jj = k0 + i;
+        acc = fmaf(pr[i], act_load(V + ((int64_t)bt[jj / kPage] * kPage + jj % kPage) * ldv + c), acc);
+      }
+      o[c] = acc;
+    }
+    __syncthreads();
+  }
+  for (int c = tid; c < a.vdim; c += kRT) po[c] = o[c];
+  for (int s = 1; s < a.nsplit; ++s)
+    for (int c = tid; c < a.vdim; c += kRT) po[(int64_t)s * a.vdim + c] = 0.f;
+  for (int s = tid; s < a.nsplit; s += kRT) { pm[2 * s] = s ? -INFINITY : m; pm[2 * s + 1] = s ? 0.f : l; }
+}
+
+// One warp per (row, head): merge the key splits of every map, o = a_0 - lambda a_1 (two maps), RMS norm over the
+// head's values without weight (two maps), times post_scale, times sigmoid(gate).
+constexpr int kVMax = 16;      // values per lane: vdim <= 512
+template <typename TA>
+__global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                          const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
+                                                          int64_t lda, const int* __restrict__ positions, int rows, int H,
+                                                          int maps, int vdim, int nsplit, float lambda, float post_scale, float eps) {
+  griddep_launch();
+  griddep_wait();
+  const int64_t w = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (w >= (int64_t)rows * H) return;
+  const int64_t row = w / H;
+  const int h = (int)(w % H);
+  if (positions[row] < 0) return;
+  float o[kVMax];
+#pragma unroll
+  for (int i = 0; i < kVMax; ++i) o[i] = 0.f;
+  for (int mp = 0; mp < maps; ++mp) {
+    const int64_t vh = (row * H + h) * maps + mp;
+    const float* ml = part_ml + vh * nsplit * 2;
+    const float* po = part_o + vh * nsplit * vdim;
+    float M = -INFINITY;
+    for (int s = lane; s < nsplit; s += 32) M = fmaxf(M, ml[2 * s]);
+    M = warp_max(M);
+    float den = 0.f;
+    for (int s = lane; s < nsplit; s += 32) den += ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - M) * ml[2 * s + 1];
+    den = warp_sum(den);
+    const float c = (mp == 0 ? 1.f : -lambda) / den;
+    for (int s = 0; s < nsplit; ++s) {
+      const float ms = ml[2 * s];
+      if (ms == -INFINITY) continue;
+      const float f = c * expf(ms - M);
+#pragma unroll
+      for (int i = 0; i < kVMax; ++i) {
+        const int v = lane + 32 * i;
+        if (v < vdim) o[i] = fmaf(f, po[(int64_t)s * vdim + v], o[i]);
+      }
+    }
+  }
+  float r = post_scale;
+  if (maps > 1) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kVMax; ++i) ss = fmaf(o[i], o[i], ss);
+    r *= 1.f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  }
+  if (gates) r *= sigmoid_x(gates[row * ldg + h]);
+  TA* out = act + row * lda + (int64_t)h * vdim;
+#pragma unroll
+  for (int i = 0; i < kVMax; ++i) {
+    const int v = lane + 32 * i;
+    if (v < vdim) act_store(out + v, o[i] * r);
+  }
+}
+
+bool maps_args_ok(const AttnMapsArgs& a) {
+  return a.proj && a.kpool && a.vpool && a.tables && a.positions && a.H > 0 && a.G > 0 && a.H % a.G == 0 && a.maps >= 1 && a.dim > 0 &&
+         a.vdim > 0;
+}
+
+}  // namespace
+
+CB_EXPORT int cb_attn_maps_args_size() { return (int)sizeof(AttnMapsArgs); }
+
+// Keys and values of `rows` projection rows into the pages.
+CB_EXPORT int cb_attn_maps_append(const void* args, int64_t rows, int64_t p_f32, int64_t f32, void* stream) {
+  if (!args || rows < 1) return CB_ERR_ARG;
+  const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
+  if (!maps_args_ok(a)) return CB_ERR_ARG;
+  cudaStream_t st = (cudaStream_t)stream;
+  const dim3 grid((unsigned)rows), block(256);
+  if (f32) return (int)cb_launch(maps_append_kernel<float, float>, grid, block, 0, st, a);
+  if (p_f32) return (int)cb_launch(maps_append_kernel<float, bf16>, grid, block, 0, st, a);
+  return (int)cb_launch(maps_append_kernel<bf16, bf16>, grid, block, 0, st, a);
+}
+
+// The plain kernel: every row against the pages (its own key included, so append first).
+CB_EXPORT int cb_attn_maps_rows(const void* args, int64_t rows, int64_t p_f32, int64_t f32, void* stream) {
+  if (!args || rows < 1 || rows > 65535) return CB_ERR_ARG;
+  const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
+  if (!maps_args_ok(a) || !a.part_o || !a.part_ml || a.nsplit < 1) return CB_ERR_ARG;
+  const size_t smem = sizeof(float) * (size_t)(a.dim + kRT + a.vdim);
+  if (smem > 40 * 1024) return CB_ERR_SHAPE;
+  cudaStream_t st = (cudaStream_t)stream;
+  const dim3 grid((unsigned)(a.H * a.maps), (unsigned)rows), block(kRT);
+  if (f32) return (int)cb_launch(maps_row_kernel<float, float>, grid, block, smem, st, a);
+  if (p_f32) return (int)cb_launch(maps_row_kernel<float, bf16>, grid, block, smem, st, a);
+  return (int)cb_launch(maps_row_kernel<bf16, bf16>, grid, block, smem, st, a);
+}
+
+CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const void* gates, int64_t ldg, void* act, int64_t lda,
+                                  const void* positions, int64_t rows, int64_t H, int64_t maps, int64_t vdim, int64_t nsplit,
+                                  float lambda, float post_scale, float eps, int64_t f32, void* stream) {
+  if (!part_o || !part_ml || !act || !positions || rows < 1 || maps < 1 || maps > 2 || nsplit < 1) return CB_ERR_ARG;
+  if (vdim > 32 * kVMax) return CB_ERR_SHAPE;
+  const dim3 grid((unsigned)((rows * H + 3) / 4)), block(128);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (f32)
+    return (int)cb_launch(maps_finish_kernel<float>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
+                          (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps,
+                          (int)vdim, (int)nsplit, lambda, post_scale, eps);
+  return (int)cb_launch(maps_finish_kernel<bf16>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
+                        (const float*)gates, ldg, (bf16*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps, (int)vdim,
+                        (int)nsplit, lambda, post_scale, eps);
+}

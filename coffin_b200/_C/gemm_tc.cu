@@ -43,6 +43,7 @@ struct GemmArgs {
   // multiplies a K slice and leaves an fp32 partial tile in `ws`; the last one to arrive (ticket)
   // adds the partials in slice order and writes the result, so the sum does not depend on timing.
   int splits; float* ws; unsigned* tickets;
+  int c_f32 = 0;                   // C is fp32 instead of bf16 (gate pre-activations, logits)
 };
 struct TileCoord { int m0, row_end, n0, brow; };
 template <int BN>
@@ -238,6 +239,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               f.x += __uint_as_float(rr.x << 16); f.y += __uint_as_float(rr.x & 0xffff0000u);
               f.z += __uint_as_float(rr.y << 16); f.w += __uint_as_float(rr.y & 0xffff0000u);
             }
+            if (a.c_f32) {
+              *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.C) + (int64_t)grow * a.ldc + gcol) = f;
+              continue;
+            }
             const __nv_bfloat162 lo = __floats2bfloat162_rn(f.x, f.y), hi = __floats2bfloat162_rn(f.z, f.w);
             uint2 o;
             o.x = *reinterpret_cast<const uint32_t*>(&lo);
@@ -278,7 +283,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
 #pragma unroll
               for (int i = 0; i < 8; ++i) f[i] += g[i];
             }
-            *reinterpret_cast<uint4*>(cp + v * 8) = float_to_bf16x8(f);
+            if (a.c_f32) {
+              float4* fp = reinterpret_cast<float4*>(reinterpret_cast<float*>(a.C) + (int64_t)row * a.ldc + col0 + v * 8);
+              fp[0] = make_float4(f[0], f[1], f[2], f[3]);
+              fp[1] = make_float4(f[4], f[5], f[6], f[7]);
+            } else {
+              *reinterpret_cast<uint4*>(cp + v * 8) = float_to_bf16x8(f);
+            }
           }
         }
       }
@@ -351,6 +362,38 @@ int pick_bn(int M, int N, int sms, bool allow64) {
 
 }  // namespace
 
+namespace {
+// Tile width and slice count for a product of at most 128 rows.  Every (tile, slice) gets its own CTA
+// in a single wave; the estimate is the bytes one CTA moves into shared memory (its slice of W and of
+// the valid rows of A) plus what the last slice re-reads to add the partial tiles.
+// K is counted in bytes of a row (a k-block is 128 bytes); n_cand = 2 leaves out the 64-wide tile.
+void plan_split(int64_t M, int64_t N, int64_t Kbytes, int* bn_out, int* s_out, int n_cand = 3) {
+  const int sms = sm_count();
+  const int64_t kb = (Kbytes + 127) / 128, K = Kbytes / 2;
+  const int cand[3] = {256, 128, 64};
+  double best = 1e300;
+  *bn_out = 256; *s_out = 1;
+  for (int i = 0; i < n_cand; ++i) {
+    const int bn = cand[i];
+    const int64_t tiles = (N + bn - 1) / bn;
+    int64_t s = sms / tiles;
+    if (s > kb / 4) s = kb / 4;          // at least four k-blocks per slice
+    if (s > 32) s = 32;
+    if (s < 1) s = 1;
+    for (;;) {                           // no slice may be empty: s = ceil(kb / ceil(kb / s))
+      const int64_t kper = (kb + s - 1) / s, s2 = (kb + kper - 1) / kper;
+      if (s2 == s) break;
+      s = s2;
+    }
+    const int64_t waves = (tiles * s + sms - 1) / sms;
+    const double stream = (double)waves * (bn + M) * ((double)K / s) * 2.0 / 130e3;        // us at ~130 GB/s per SM
+    const double reduce = s > 1 ? (double)s * M * bn * 4.0 / 100e3 + 2.0 : 0.0;
+    const double cost = stream + reduce;
+    if (cost < best) { best = cost; *bn_out = bn; *s_out = (int)s; }
+  }
+}
+}  // namespace
+
 // CTA-pair kernel (gemm_tc2.cu): tile width it would use for [M, N], or 0 for "not this product".
 int cb_gemm_pair_plan(int64_t M, int64_t N);
 int cb_gemm_pair_run(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, const void* residual,
@@ -390,6 +433,41 @@ CB_EXPORT int cb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ld
   if (bn == 128) return launch_gemm<128, 6, false>(tmA, tmB, a, sms, st);
   if (bn == 64) return launch_gemm<64, 8, false>(tmA, tmB, a, sms, st);
   return CB_ERR_ARG;
+}
+
+// C[M,N] (fp32) = A[M,K] (bf16) x W[N,K]^T (bf16): the accumulator leaves unrounded (gate pre-activations of the
+// recurrent mixers, logits of many rows).  K % 8 == 0, N % 8 == 0, ldc % 4 == 0.  ws / tickets: split-K scratch
+// for products of at most 128 rows (see cb_gemm_bf16_splitk); null = never split.
+CB_EXPORT int cb_gemm_bf16_f32out(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int64_t M,
+                                  int64_t N, int64_t K, void* ws, int64_t ws_bytes, void* tickets, int64_t n_tickets,
+                                  void* status, void* stream) {
+  if (M < 1 || N < 1 || K < 1 || K % 8 || N % 8 || ldc % 4 || !status) return CB_ERR_SHAPE;
+  const int sms = sm_count();
+  int bn = pick_bn((int)M, (int)N, sms, true), splits = 1;
+  if (ws && tickets && M <= BM) {
+    int b2, s2;
+    plan_split(M, N, K * 2, &b2, &s2);
+    const int64_t tiles = (N + b2 - 1) / b2;
+    if (s2 > 1 && ws_bytes >= tiles * s2 * BM * b2 * (int64_t)sizeof(float) && n_tickets >= tiles) { bn = b2; splits = s2; }
+  }
+  CUtensorMap tmA, tmB;
+  int rc = cb_make_tmap_2d(&tmA, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM, 64);
+  if (rc) return rc;
+  rc = cb_make_tmap_2d(&tmB, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, (uint32_t)bn, 64);
+  if (rc) return rc;
+  GemmArgs a;
+  a.C = C; a.ldc = ldc; a.residual = nullptr; a.ldr = 0; a.row_scale = nullptr; a.col_scale = nullptr;
+  a.M = (int)M; a.N = (int)N; a.K = (int)K; a.m_tiles = (int)((M + BM - 1) / BM); a.n_tiles = 0;
+  a.k_blocks = (int)((K + 63) / 64); a.status = (int*)status;
+  a.pf = nullptr; a.pf_seq = 0;
+  a.g_count = a.g_row0 = a.g_rows = a.g_expert = nullptr;
+  a.splits = splits; a.ws = (float*)ws; a.tickets = (unsigned*)tickets;
+  a.c_f32 = 1;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (bn == 256) return launch_gemm<256, 4, false>(tmA, tmB, a, sms, st);
+  if (bn == 160) return launch_gemm<160, 5, false>(tmA, tmB, a, sms, st);
+  if (bn == 128) return launch_gemm<128, 6, false>(tmA, tmB, a, sms, st);
+  return launch_gemm<64, 8, false>(tmA, tmB, a, sms, st);
 }
 
 // C[M,N] (bf16) = (A_q[M,K] int8 x W_q[N,K]^T int8) * row_scale[m] * col_scale[n] (+ residual). K % 16 == 0.
@@ -495,38 +573,6 @@ CB_EXPORT int cb_gemm_i8_grouped(const void* A, int64_t lda, const void* W, int6
 // few 256-wide tiles (N = 2560: 10 tiles x 14 slices).  ws holds the fp32 partial tiles
 // (cb_gemm_splitk_ws_bytes), tickets one zero-initialised counter per output tile; both may be
 // shared by all calls of a stream.  Falls back to the plain kernel when splitting does not pay.
-namespace {
-// Tile width and slice count for a product of at most 128 rows.  Every (tile, slice) gets its own CTA
-// in a single wave; the estimate is the bytes one CTA moves into shared memory (its slice of W and of
-// the valid rows of A) plus what the last slice re-reads to add the partial tiles.
-// K is counted in bytes of a row (a k-block is 128 bytes); n_cand = 2 leaves out the 64-wide tile.
-void plan_split(int64_t M, int64_t N, int64_t Kbytes, int* bn_out, int* s_out, int n_cand = 3) {
-  const int sms = sm_count();
-  const int64_t kb = (Kbytes + 127) / 128, K = Kbytes / 2;
-  const int cand[3] = {256, 128, 64};
-  double best = 1e300;
-  *bn_out = 256; *s_out = 1;
-  for (int i = 0; i < n_cand; ++i) {
-    const int bn = cand[i];
-    const int64_t tiles = (N + bn - 1) / bn;
-    int64_t s = sms / tiles;
-    if (s > kb / 4) s = kb / 4;          // at least four k-blocks per slice
-    if (s > 32) s = 32;
-    if (s < 1) s = 1;
-    for (;;) {                           // no slice may be empty: s = ceil(kb / ceil(kb / s))
-      const int64_t kper = (kb + s - 1) / s, s2 = (kb + kper - 1) / kper;
-      if (s2 == s) break;
-      s = s2;
-    }
-    const int64_t waves = (tiles * s + sms - 1) / sms;
-    const double stream = (double)waves * (bn + M) * ((double)K / s) * 2.0 / 130e3;        // us at ~130 GB/s per SM
-    const double reduce = s > 1 ? (double)s * M * bn * 4.0 / 100e3 + 2.0 : 0.0;
-    const double cost = stream + reduce;
-    if (cost < best) { best = cost; *bn_out = bn; *s_out = (int)s; }
-  }
-}
-}  // namespace
-
 // (slices, or 1 when the plain kernel is used) and the workspace a call needs
 CB_EXPORT int64_t cb_gemm_splitk_plan(int64_t M, int64_t N, int64_t K) {
   if (M > BM) return 1;

@@ -1,0 +1,33 @@
+// Arguments shared by the recurrent-state kernels (linrec.cu: token by token; linrec_chunk.cu: prompts in chunks).
+#pragma once
+#include "act_type.cuh"
+
+enum LinrecKind : int { LINREC_DELTA = 0, LINREC_MLSTM = 1 };
+
+// Column layout of a projection row: q | k | v | ... ; the first conv_width columns pass the short convolution
+// of the delta layers (channel index == column index).
+struct LinrecArgs {
+  // rows
+  const void* proj; int64_t ldp;        // q, k, v (and gate / low-rank) columns
+  const float* gates; int64_t ldg;      // fp32 gate pre-activations: delta b[H]; mLSTM i[H] | f[H]
+  const float* dec; int64_t ldd;        // delta, optional: decay pre-activations [H * dk] (before dt_bias)
+  const void* og; int64_t ldo;          // output-gate pre-activations [H * dv] (null: delta computes them from g1 / g2)
+  void* act; int64_t lda;               // result rows [H * dv]
+  // segments: rows [seg_row[s], seg_row[s + 1]) are consecutive tokens of one sequence from position seg_pos[s],
+  // whose state lives in slot seg_slot[s] (< 0: skip).  seg_row null: row s alone.
+  const int* seg_row; const int* seg_pos; const int* seg_slot;
+  // weights
+  const float* conv_w; int taps;        // [conv_width, taps]
+  const float* A_log; const float* dt_bias;
+  const void* a2; int64_t ra; int64_t a1_col;   // [H * dk, ra]
+  const void* g2; int64_t rg; int64_t g1_col;   // [H * dv, rg]
+  const float* norm_w;                  // delta [dv]; mLSTM [H * dv]
+  const float* gate_b;                  // mLSTM: i.b[H] | f.b[H]
+  // state of this layer
+  float* S; float* n; float* m;         // [slots, H, dk, dv], [slots, H, dk], [slots, H]
+  void* ring; int ring_mask; int64_t ring_w;    // [slots, ring, ring_w]
+  // sizes
+  int H, G, dk, dv, jc;
+  int64_t k_col, v_col;
+  float eps, cap;
+};

@@ -196,6 +196,9 @@ def preset(name: str) -> ModelConfig:
     if "qwen4" in name:
         from .models.qwen4exp.config import preset_qwen4
         return preset_qwen4(name)
+    if "zufilorn" in name:
+        from .models.zufilorn.config import preset_zufilorn
+        return preset_zufilorn(name)
     if name == "tiny-moe":
         return ModelConfig(name="tiny-moe", num_experts=8, num_experts_per_tok=2,
                            moe_intermediate_size=128, shared_expert_intermediate_size=128,
@@ -234,4 +237,7 @@ def load_config(model_dir: str | Path):
     if "qwen4" in kind.lower():
         from .models.qwen4exp.config import Qwen4Config
         return Qwen4Config.from_hf(raw, name=Path(model_dir).name)
+    if str(raw.get("architecture", "")).lower() == "zufilorn":
+        from .models.zufilorn.config import ZufilornConfig
+        return ZufilornConfig.from_hf(raw, name=Path(model_dir).name)
     return ModelConfig.from_hf(raw, name=Path(model_dir).name)

@@ -28,6 +28,7 @@ class EngineConfig:
                                        # as an option for parity with the reference, where it is also refused when
                                        # > 0 (no masked multi-query verify kernel, models/qwen35/model.py:1390-1401)
     group_prefill: bool = True         # chunks of several sequences share one forward (stacked rows)
+    mixed_batch: bool = True           # models that can: prompt chunks and decode rows share one forward
     chunk: int = 2048                  # largest prefill chunk handed to the model
     prefill_quantum: int = 2048        # tokens of one sequence prefilled per engine step
     max_num_seqs: int = 8              # concurrent sequences (= state slots = decode rows)

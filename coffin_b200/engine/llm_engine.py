@@ -1,7 +1,8 @@
 """``LLMEngine``: request lifecycle around the scheduler, the block manager and the runner.
 
 ``add_request`` queues a sequence; every ``step()`` runs exactly one forward (a decode step of
-all running rows, or one prefill quantum) and returns the tokens it produced.  Capacity is
+all running rows, one prefill quantum, or - for models that take both - the two together) and
+returns the tokens it produced.  Capacity is
 claimed lazily: before a decode step every row reserves room for one more token, and when the
 pool (after evicting cached blocks) cannot provide it the latest-arrived sequence is preempted
 and recomputed later.  A run of steps that makes no progress raises instead of spinning.
@@ -52,8 +53,8 @@ class LLMEngine:
             self.cfg = dataclasses.replace(self.cfg, max_num_seqs=limit)
         self.bm = bm or BlockManager(model, getattr(model, "num_blocks", None), self.cfg.block_size,
                                      self.cfg.snapshots, self.cfg.prefix_cache)
-        self.scheduler = Scheduler(self.cfg)
         self.runner = ModelRunner(model, self.bm, self.cfg)
+        self.scheduler = Scheduler(self.cfg, mixed=self.cfg.mixed_batch and self.runner.mixed_capable)
         self.runner.live_seqs = lambda: self.scheduler.prefilling + self.scheduler.running
         self.max_seq = min(self.cfg.max_seq, getattr(model, "max_seq", self.cfg.max_seq))
         self._stall = 0
@@ -145,6 +146,8 @@ class LLMEngine:
             progressed = self._run_prefill(batch, out)
         elif batch.kind == "decode":
             progressed = self._run_decode(batch.seqs, out)
+        elif batch.kind == "mixed":
+            progressed = self._run_mixed(batch, out)
         self._check_progress(progressed or bool(out), batch.kind)
         return out
 
@@ -194,7 +197,8 @@ class LLMEngine:
         return progressed
 
     # ------------------------------------------------------------------ decode
-    def _run_decode(self, seqs: list[Sequence], out: list[StepOutput]) -> bool:
+    def _reserve_decode(self, seqs: list[Sequence]) -> list[Sequence]:
+        """The rows of ``seqs`` that have room for one more token, preempting others where the pool is short."""
         ready = []
         for seq in list(seqs):
             if seq.finished or seq.status is not SequenceStatus.RUNNING:
@@ -208,7 +212,10 @@ class LLMEngine:
                     break
             if seq.status is SequenceStatus.RUNNING:
                 ready.append(seq)
-        ready = [s for s in ready if s.status is SequenceStatus.RUNNING]
+        return [s for s in ready if s.status is SequenceStatus.RUNNING]
+
+    def _run_decode(self, seqs: list[Sequence], out: list[StepOutput]) -> bool:
+        ready = self._reserve_decode(seqs)
         if not ready:
             return False
         tokens = [s.output[-1] for s in ready]
@@ -219,6 +226,32 @@ class LLMEngine:
         picked = self.runner.sample(ready, logits, greedy)
         for seq, tok in zip(ready, picked):
             self._commit(seq, tok, out)
+        return True
+
+    def _run_mixed(self, batch, out: list[StepOutput]) -> bool:
+        """All running rows and the scheduled prompt chunks in one forward.  A chunk without room is left out (its
+        turn comes again, or the step after the last running row preempts for it)."""
+        ready = self._reserve_decode(batch.decode)
+        chunks = []
+        for seq, n in zip(batch.seqs, batch.chunks):
+            if seq.finished or seq.status is not SequenceStatus.PREFILLING:
+                continue                                  # preempted to make room for a row
+            end = self.runner._chunk_end(seq, n)
+            if self.bm.ensure_blocks(seq.blocks, end - seq.num_computed):
+                chunks.append((seq, end))
+        if not chunks:
+            return self._run_decode(ready, out) if ready else False
+        logits = self.runner.mixed_step(ready, [s.output[-1] for s in ready], chunks)
+        done = [s for s, _e in chunks if s.remaining_prefill == 0]
+        for seq in done:
+            self.runner.finish_prefill(seq)
+            self.scheduler.prefill_done(seq)
+        rows = ready + done
+        if rows:
+            for seq, tok in zip(rows, self.runner.sample(rows, logits)):
+                if seq.first_token_time is None:
+                    seq.first_token_time = time.monotonic()
+                self._commit(seq, tok, out)
         return True
 
     def _run_spec(self, ready: list[Sequence], tokens: list[int], out: list[StepOutput]) -> bool:

@@ -35,6 +35,7 @@ class ModelRunner:
         self.n_cached_tokens = 0
         self.n_spec_steps = self.n_spec_drafted = self.n_spec_accepted = 0
         self.n_prefill_groups = 0
+        self.n_mixed_steps = 0
         # device status words (bounded waits that ran out): queued after every model call, looked at
         # after the next synchronisation (the token read-back in ``sample``)
         self._poll = getattr(model, "poll_status", None)
@@ -243,6 +244,68 @@ class ModelRunner:
         self._last_next = nxt
         return logits[:n]
 
+    # ------------------------------------------------------------------ mixed batches
+    @property
+    def mixed_capable(self) -> bool:
+        return bool(getattr(self.model, "mixed_batches", False))
+
+    def run_batch(self, entries: list[tuple[Sequence, list[int], list[int]]]) -> torch.Tensor | None:
+        """Run ``(sequence, its next tokens, wanted places among them)`` entries as one step from where the sequences
+        stand; room in their block tables has to be reserved.  Returns fp32 logits ``[wanted, vocab]`` in the order
+        of the entries, or None when nothing is wanted.
+
+        A step of single tokens is the decode step (CUDA graph).  Otherwise a model with mixed batches runs one
+        forward over portions and single tokens; any other model runs the entries one after the other, cut after
+        every wanted place (its prefill returns the logits of the last token)."""
+        if debug.KV_TRACE:
+            debug.check_block_alias(self.live() or [s for s, _t, _w in entries], self.block_size, "batch",
+                                    {s.seq_id: len(t) for s, t, _w in entries}, verbose=True)
+        n = len(entries)
+        if n <= BATCH_BUCKETS[-1] and all(len(t) == 1 for _s, t, _w in entries) and hasattr(self.model, "set_rows"):
+            logits = self.decode([s for s, _t, _w in entries], [t[0] for _s, t, _w in entries])
+            rows = [i for i, (_s, _t, w) in enumerate(entries) for _ in w]
+            return logits[rows] if rows else None
+        if self.mixed_capable:
+            out = self.model.forward_batch([(t, s.num_computed, s.slot, s.blocks.table) for s, t, _w in entries],
+                                           [w for _s, _t, w in entries])
+        else:
+            rows = []
+            cap = getattr(self.model, "max_chunk", self.cfg.chunk)
+            for s, toks, want in entries:
+                got, start = {}, 0
+                for end in sorted({*(w + 1 for w in want), *range(cap, len(toks), cap), len(toks)}):
+                    for a in range(start, end, cap):
+                        e = min(end, a + cap)
+                        lg = self.model.prefill(self._tokens(toks[a:e]), s.num_computed + a, s.slot, self._table(s),
+                                                want_logits=e == end and end - 1 in want)
+                    got[end - 1], start = lg, end
+                rows += [got[w] for w in want]
+            out = torch.stack(rows) if rows else None
+        if self._poll is not None:
+            self._poll()
+        for s, toks, _w in entries:
+            s.blocks.commit(len(toks))
+            s.num_computed += len(toks)
+        return out
+
+    def mixed_step(self, decode: list[Sequence], tokens: list[int], chunks: list[tuple[Sequence, int]]) -> torch.Tensor | None:
+        """One forward: ``decode[i]`` takes ``tokens[i]``, every ``(sequence, end)`` of ``chunks`` its prompt tokens up
+        to ``end``.  Returns the logits of the decode rows, then of the chunks that reach the end of their prompt."""
+        dec = [(s, [t], [0]) for s, t in zip(decode, tokens)]
+        pre = [(s, s.all_tokens[s.num_computed:e], [e - s.num_computed - 1] if e == s.num_tokens else []) for s, e in chunks]
+        out = self.model.forward_batch([(t, s.num_computed, s.slot, s.blocks.table) for s, t, _w in dec + pre],
+                                       [w for _s, _t, w in dec + pre])
+        if self._poll is not None:
+            self._poll()
+        for s in decode:
+            s.blocks.commit(1)
+            s.num_computed += 1
+        for s, e in chunks:
+            self._chunk_done(s, e, None)
+        self.n_decode_steps += bool(decode)
+        self.n_mixed_steps += 1
+        return out
+
     # ------------------------------------------------------------------ speculative decoding
     @property
     def spec_capable(self) -> bool:
@@ -360,5 +423,5 @@ class ModelRunner:
 
     def stats(self) -> dict:
         return {"prefill_tokens": self.n_prefill_tokens, "decode_steps": self.n_decode_steps,
-                "cached_tokens": self.n_cached_tokens, "prefill_groups": self.n_prefill_groups,
+                "cached_tokens": self.n_cached_tokens, "prefill_groups": self.n_prefill_groups, "mixed_steps": self.n_mixed_steps,
                 "spec": {"steps": self.n_spec_steps, "drafted": self.n_spec_drafted, "accepted": self.n_spec_accepted}}

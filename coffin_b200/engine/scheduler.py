@@ -2,9 +2,9 @@
 
 One engine step is either a *decode* step (every RUNNING sequence advances one token, rows
 padded to a bucket) or a *prefill* step (one quantum of prompt tokens of one or more admitted
-sequences).  The two never mix in one forward (the kernels for the two regimes differ), and
-they alternate while both kinds of work exist, so a long prompt cannot starve running
-streams and running streams cannot starve admission.  A sequence is admitted when a state
+sequences).  Where the model's forward takes both (``mixed``), a step carries all running rows and
+fills the rest of its token budget with prompt chunks; otherwise the two kinds alternate while both
+exist, so a long prompt cannot starve running streams and running streams cannot starve admission.  A sequence is admitted when a state
 slot is free; KV blocks are claimed chunk by chunk, so admission never over-commits the
 pool, and when the pool runs dry the most recently arrived running sequence is preempted
 and later recomputed.  Reference: ``engine/scheduler.py:144-427``.
@@ -23,14 +23,16 @@ PREEMPT_COOLDOWN = 1
 
 @dataclasses.dataclass
 class Batch:
-    kind: str                                   # "decode" | "prefill" | "idle"
+    kind: str                                   # "decode" | "prefill" | "mixed" | "idle"
     seqs: list[Sequence] = dataclasses.field(default_factory=list)
     chunks: list[int] = dataclasses.field(default_factory=list)   # prefill: tokens per sequence
+    decode: list[Sequence] = dataclasses.field(default_factory=list)   # mixed: the rows that advance one token
 
 
 class Scheduler:
-    def __init__(self, cfg: EngineConfig) -> None:
+    def __init__(self, cfg: EngineConfig, mixed: bool = False) -> None:
         self.cfg = cfg
+        self.mixed = mixed
         self.waiting: collections.deque[Sequence] = collections.deque()
         self.prefilling: list[Sequence] = []
         self.running: list[Sequence] = []
@@ -52,7 +54,10 @@ class Scheduler:
     def _admit(self) -> Sequence | None:
         if not self.waiting or not self._has_room():
             return None
-        seq = self.waiting.popleft()
+        return self.admit(self.waiting.popleft())
+
+    def admit(self, seq: Sequence) -> Sequence:
+        """Give ``seq`` a state slot now (the caller made sure there is one)."""
         seq.slot = self.free_slots.pop()
         seq.status = SequenceStatus.PREFILLING
         self.prefilling.append(seq)
@@ -70,7 +75,13 @@ class Scheduler:
         self.admitted = newly
         want_prefill = bool(self.prefilling)
         want_decode = bool(self.running)
-        if want_prefill and (not want_decode or self._last_kind == "decode"):
+        if want_prefill and want_decode and self.mixed:
+            batch = self._schedule_prefill(self.cfg.max_num_batched_tokens - len(self.running))
+            if batch.seqs:
+                for s in self.running:
+                    s.cooldown = max(0, s.cooldown - 1)
+                return dataclasses.replace(batch, kind="mixed", decode=list(self.running))
+        elif want_prefill and (not want_decode or self._last_kind == "decode"):
             return self._schedule_prefill()
         if want_decode:
             if self._hold_for_batch():
@@ -96,8 +107,8 @@ class Scheduler:
         self._hold_since = None
         return False
 
-    def _schedule_prefill(self) -> Batch:
-        budget = self.cfg.max_num_batched_tokens
+    def _schedule_prefill(self, budget: int | None = None) -> Batch:
+        budget = self.cfg.max_num_batched_tokens if budget is None else budget
         quantum = min(self.cfg.prefill_quantum, self.cfg.chunk)
         seqs, chunks = [], []
         for s in self.prefilling:

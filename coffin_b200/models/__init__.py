@@ -77,6 +77,28 @@ def _ensure_builtin() -> None:
     for n in ("qwen4_exp", "qwen4exp"):
         register(n, qwen4)
 
+    def zufilorn(cfg, sd, **kw):
+        from .zufilorn.model import ZufilornModel
+        if any(kw.pop(k + "_world", 1) > 1 for k in ("tp", "pp", "ep")):
+            raise NotImplementedError("the Zufilorn family runs on one GPU")
+        for k in ("tp_rank", "pp_rank", "ep_rank"):
+            kw.pop(k, None)
+        return ZufilornModel(cfg, sd, **kw)
+
+    register("zufilorn", zufilorn)
+
+
+#: kernel sources a family needs; families without an entry use the whole library
+_KERNELS: dict[str, tuple[str, ...]] = {
+    "zufilorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemv.cu", "gemv_stream.cu", "gemm_f32.cu", "streams.cu",
+                 "linrec.cu", "attn_maps.cu"),
+}
+
+
+def kernel_sources(arch: str) -> tuple[str, ...] | None:
+    """Kernel sources of a model family (None: all), for a process that serves that family only and has to compile first."""
+    return _KERNELS.get(arch)
+
 
 def detect_architecture(cfg: ModelConfig) -> str:
     """Registry key for a config; unknown names fall back on geometry (a config that has
@@ -84,7 +106,7 @@ def detect_architecture(cfg: ModelConfig) -> str:
     _ensure_builtin()
     if cfg.architecture in _REGISTRY:
         return cfg.architecture
-    if cfg.linear_num_value_heads > 0:
+    if getattr(cfg, "linear_num_value_heads", 0) > 0:
         return "qwen3_5"
     raise RuntimeError(f"no registered model family for architecture {cfg.architecture!r}")
 

@@ -30,16 +30,30 @@ def available() -> bool:
     return _LIB_PATH.exists()
 
 
+_only: tuple[str, ...] | None = None
+
+
+def use_sources(names: tuple[str, ...] | None) -> None:
+    """In a process that serves one model family: when the library has to be compiled first, compile just these
+    sources into a library of their own.  A complete up-to-date library is used as it is."""
+    global _only
+    assert _lib is None or names is None, "the kernel library is loaded already"
+    _only = tuple(names) if names is not None else None
+
+
 def lib() -> ctypes.CDLL:
     global _lib
     if _lib is None:
-        if not _LIB_PATH.exists():
-            if os.environ.get("COFFIN_B200_AUTOBUILD", "1") == "1":
-                from .._C.build import build
-                build()
-            else:
-                raise KernelError(f"{_LIB_PATH} is missing: run python -m coffin_b200._C.build")
-        _lib = ctypes.CDLL(str(_LIB_PATH))
+        path = _LIB_PATH
+        if os.environ.get("COFFIN_B200_AUTOBUILD", "1") == "1":
+            from .._C import build as B
+            if _only is not None and not B.up_to_date():
+                path = B.build(only=_only)
+            elif not path.exists():
+                B.build()
+        elif not path.exists():
+            raise KernelError(f"{path} is missing: run python -m coffin_b200._C.build")
+        _lib = ctypes.CDLL(str(path))
     return _lib
 
 

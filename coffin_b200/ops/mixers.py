@@ -1,0 +1,210 @@
+"""Entry points of the kernels behind hyper-connected streams, the recurrent mixers and multi-map attention.
+
+Like ``ops.kernels`` these are thin wrappers that launch on the current stream into caller-owned buffers.  Every
+constant of a mechanism (tap count, gate cap, number of maps, score cap, query temperature, number of streams) is
+an argument, so a model family picks what it needs:
+
+* ``streams_embed`` / ``streams_step``: a residual of several fp32 streams with static read / write / mixing weights;
+* ``Linrec``: recurrences with a matrix state - the per-channel gated delta rule and the mLSTM matrix memory;
+* ``AttnMaps``: paged attention with several score maps per head over the same values, capped scores and a
+  position-dependent query temperature;
+* ``gemm_f32out`` / ``gemm_f32``: projections whose result (or everything) stays fp32.
+"""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from . import _lib
+from . import kernels as K
+from ._lib import call
+
+DELTA, MLSTM = 0, 1
+RING = 16             # shallowest convolution ring
+_P, _I64, _I32, _F = ctypes.c_void_p, ctypes.c_int64, ctypes.c_int, ctypes.c_float
+
+
+def _ptr(t: torch.Tensor | None) -> int | None:
+    return None if t is None else t.data_ptr()
+
+
+def _is_f32(t: torch.Tensor) -> int:
+    return int(t.dtype == torch.float32)
+
+
+# ------------------------------------------------------------------ projections
+def gemm_f32out(A: torch.Tensor, W: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out[M, N] (fp32) = A[M, K] @ W[N, K]^T`` from bf16 operands on tcgen05, accumulator unrounded."""
+    M, Kd = A.shape
+    N = W.shape[0]
+    assert out.dtype == torch.float32 and out.stride(1) == 1 and A.stride(1) == 1 and W.stride(1) == 1
+    ws = tickets = None
+    if M <= 128 and K.SPLITK_GEMM:
+        ws, tickets = K._splitk_scratch(A.device)
+    call("gemm_bf16_f32out", A, A.stride(0), W, W.stride(0), out, out.stride(0), M, N, Kd, ws,
+         ws.numel() * 4 if ws is not None else 0, tickets, tickets.numel() if tickets is not None else 0, K.status_word(A.device))
+    K._count()
+    return out
+
+
+def gemm_f32(A: torch.Tensor, W: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """True fp32 product of any shape (the 32-bit mode of a model)."""
+    M, Kd = A.shape
+    N = W.shape[0]
+    assert A.dtype == W.dtype == out.dtype == torch.float32 and A.stride(1) == W.stride(1) == out.stride(1) == 1
+    call("gemm_f32", A, A.stride(0), W, W.stride(0), out, out.stride(0), M, N, Kd)
+    K._count()
+    return out
+
+
+def swiglu_f32(gu: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    M, two_i = gu.shape
+    call("swiglu_f32", gu, gu.stride(0), out, out.stride(0), M, two_i // 2)
+    K._count()
+    return out
+
+
+# ------------------------------------------------------------------ hyper-connected streams
+def streams_embed(embed: torch.Tensor, pos: torch.Tensor | None, tokens: torch.Tensor, positions: torch.Tensor,
+                  x: torch.Tensor) -> torch.Tensor:
+    """Every stream of row ``t`` of ``x [T, S, W]`` (fp32) starts as ``embed[token] + pos[position]``."""
+    T, S, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and tokens.dtype == torch.int64 and positions.dtype == torch.int32
+    call("streams_embed", embed, pos, tokens, positions, x, T, S, W, embed.shape[0], pos.shape[0] if pos is not None else 0, _is_f32(embed))
+    K._count()
+    return x
+
+
+def streams_step(x: torch.Tensor, h: torch.Tensor | None, *, gain: torch.Tensor | None = None, read: torch.Tensor | None = None,
+                 y: torch.Tensor | None = None, mix: torch.Tensor | None = None, write: torch.Tensor | None = None,
+                 rows: torch.Tensor | None = None, store: bool = True, eps: float = 1e-5) -> torch.Tensor | None:
+    """Boundary between two sublayers: write ``y`` back (``x_t <- sum_s mix[s, t] x_s + write[t] y``), then
+    ``h = rmsnorm(sum_s read[s] x_s) * gain`` (``read`` None: plain sum).  ``rows`` picks the stream rows behind the
+    rows of ``h`` (with ``store=False``)."""
+    T, S, W = x.shape
+    n = rows.numel() if rows is not None else (h.shape[0] if h is not None else T)
+    t = h if h is not None else y
+    call("streams_step", x, y, y.stride(0) if y is not None else 0, mix, write, read, gain, h, h.stride(0) if h is not None else 0,
+         rows, n, S, W, float(eps), int(store), _is_f32(t))
+    K._count()
+    return h
+
+
+# ------------------------------------------------------------------ recurrences with a matrix state
+class _LinrecStruct(ctypes.Structure):
+    _fields_ = [("proj", _P), ("ldp", _I64), ("gates", _P), ("ldg", _I64), ("dec", _P), ("ldd", _I64), ("og", _P), ("ldo", _I64),
+                ("act", _P), ("lda", _I64), ("seg_row", _P), ("seg_pos", _P), ("seg_slot", _P), ("conv_w", _P), ("taps", _I32),
+                ("A_log", _P), ("dt_bias", _P), ("a2", _P), ("ra", _I64), ("a1_col", _I64), ("g2", _P), ("rg", _I64), ("g1_col", _I64),
+                ("norm_w", _P), ("gate_b", _P), ("S", _P), ("n", _P), ("m", _P), ("ring", _P), ("ring_mask", _I32), ("ring_w", _I64),
+                ("H", _I32), ("G", _I32), ("dk", _I32), ("dv", _I32), ("jc", _I32), ("k_col", _I64), ("v_col", _I64),
+                ("eps", _F), ("cap", _F)]
+
+
+def linrec_supported(H: int, dk: int, dv: int) -> bool:
+    return bool(_lib.call_nostream("linrec_supported", H, dk, dv))
+
+
+class Linrec:
+    """One recurrent layer: fixed weights, state tensors and sizes; ``step`` / ``ring`` launch on a batch of rows.
+
+    ``state``: ``S [slots, H, dk, dv]`` and, by kind, ``ring [slots, depth, width]`` (delta: the last raw projection
+    rows, indexed by position modulo depth) or ``n [slots, H, dk]`` and ``m [slots, H]`` (mLSTM), all zero at the
+    start of a sequence."""
+
+    def __init__(self, kind: int, *, H: int, G: int, dk: int, dv: int, k_col: int, v_col: int, eps: float, state: dict,
+                 norm_w: torch.Tensor, conv_w: torch.Tensor | None = None, A_log=None, dt_bias=None, a2=None, a1_col: int = 0,
+                 g2=None, g1_col: int = 0, gate_b=None, cap: float = 0.0) -> None:
+        if not linrec_supported(H, dk, dv):
+            raise ValueError(f"recurrent head of {dk} x {dv} is outside the kernel's range")
+        a = self.a = _LinrecStruct()
+        size = _lib.call_nostream("linrec_args_size")
+        assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
+        self.kind, self.state, self.conv_w = kind, state, conv_w
+        self._keep = (norm_w, conv_w, A_log, dt_bias, a2, g2, gate_b, *state.values())
+        a.H, a.G, a.dk, a.dv, a.k_col, a.v_col, a.eps, a.cap = H, G, dk, dv, k_col, v_col, float(eps), float(cap)
+        a.norm_w, a.conv_w, a.A_log, a.dt_bias, a.gate_b = _ptr(norm_w), _ptr(conv_w), _ptr(A_log), _ptr(dt_bias), _ptr(gate_b)
+        a.taps = conv_w.shape[1] if conv_w is not None else 0
+        if a2 is not None:
+            a.a2, a.ra, a.a1_col, a.g2, a.rg, a.g1_col = _ptr(a2), a2.shape[1], a1_col, _ptr(g2), g2.shape[1], g1_col
+        a.S, a.n, a.m, a.ring = _ptr(state["S"]), _ptr(state.get("n")), _ptr(state.get("m")), _ptr(state.get("ring"))
+        ring = state.get("ring")
+        if ring is not None:
+            assert ring.shape[1] & (ring.shape[1] - 1) == 0, "ring depth must be a power of two"
+            a.ring_mask, a.ring_w = ring.shape[1] - 1, ring.shape[2]
+
+    def _fill(self, proj, gates, og, act, dec, seg_row, seg_pos, seg_slot) -> None:
+        a = self.a
+        a.proj, a.ldp, a.gates, a.ldg = proj.data_ptr(), proj.stride(0), gates.data_ptr(), gates.stride(0)
+        a.og, a.ldo = _ptr(og), og.stride(0) if og is not None else 0
+        a.dec, a.ldd = _ptr(dec), dec.stride(0) if dec is not None else 0
+        a.act, a.lda = act.data_ptr(), act.stride(0)
+        a.seg_row, a.seg_pos, a.seg_slot = _ptr(seg_row), _ptr(seg_pos), _ptr(seg_slot)
+
+    def step(self, proj, gates, og, act, seg_pos, seg_slot, *, segs: int, seg_row=None, dec=None) -> None:
+        """Token by token over ``segs`` segments (``seg_row`` None: one row each)."""
+        self._fill(proj, gates, og, act, dec, seg_row, seg_pos, seg_slot)
+        call("linrec_step", ctypes.byref(self.a), self.kind, segs, _is_f32(proj), _is_f32(act))
+        K._count()
+
+    def ring(self, proj, seg_row, seg_pos, seg_slot, segs: int) -> None:
+        """After the readers: the raw rows at the end of every segment of two or more tokens enter the ring."""
+        r = self.state.get("ring")
+        if r is None or segs < 1:
+            return
+        if proj.dtype != r.dtype:
+            proj = proj.to(r.dtype)
+        call("linrec_ring", proj, proj.stride(0), seg_row, seg_pos, seg_slot, segs, r, r.shape[1], r.shape[2], self.a.taps, _is_f32(r))
+        K._count()
+
+
+# ------------------------------------------------------------------ attention with several maps per head
+class _AttnStruct(ctypes.Structure):
+    _fields_ = [("proj", _P), ("ldp", _I64), ("k_col", _I64), ("v_col", _I64), ("kpool", _P), ("vpool", _P), ("tables", _P),
+                ("ldbt", _I64), ("row_seg", _P), ("positions", _P), ("seg_row", _P), ("seg_pos", _P), ("part_o", _P), ("part_ml", _P),
+                ("H", _I32), ("G", _I32), ("maps", _I32), ("dim", _I32), ("vdim", _I32), ("nsplit", _I32), ("scale", _F), ("cap", _F),
+                ("temp_coef", _F), ("temp_every", _I32)]
+
+
+MAX_VDIM = 512
+
+
+class AttnMaps:
+    """Attention layer constants plus its pages ``kpool [slots, G * maps, dim]``, ``vpool [slots, G, vdim]``."""
+
+    def __init__(self, *, H: int, G: int, maps: int, dim: int, vdim: int, k_col: int, v_col: int, scale: float, cap: float | None,
+                 temp: tuple[float, int] | None, kpool: torch.Tensor, vpool: torch.Tensor) -> None:
+        if vdim > MAX_VDIM or maps not in (1, 2):
+            raise ValueError(f"attention with {maps} maps and values of {vdim} is outside the kernels' range")
+        a = self.a = _AttnStruct()
+        size = _lib.call_nostream("attn_maps_args_size")
+        assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
+        self.kpool, self.vpool, self.H, self.G, self.maps, self.dim, self.vdim = kpool, vpool, H, G, maps, dim, vdim
+        a.H, a.G, a.maps, a.dim, a.vdim, a.k_col, a.v_col = H, G, maps, dim, vdim, k_col, v_col
+        a.kpool, a.vpool, a.scale, a.cap = _ptr(kpool), _ptr(vpool), float(scale), float(cap or 0.0)
+        if temp is not None:
+            a.temp_coef, a.temp_every = float(temp[0]), int(temp[1])
+
+    def _fill(self, proj, tables, positions, row_seg, part_o=None, part_ml=None, nsplit: int = 1, seg_row=None, seg_pos=None) -> None:
+        a = self.a
+        a.proj, a.ldp, a.tables, a.ldbt = proj.data_ptr(), proj.stride(0), tables.data_ptr(), tables.stride(0)
+        a.positions, a.row_seg, a.part_o, a.part_ml, a.nsplit = positions.data_ptr(), _ptr(row_seg), _ptr(part_o), _ptr(part_ml), nsplit
+        a.seg_row, a.seg_pos = _ptr(seg_row), _ptr(seg_pos)
+
+    def append(self, proj, tables, positions, row_seg=None) -> None:
+        self._fill(proj, tables, positions, row_seg)
+        call("attn_maps_append", ctypes.byref(self.a), positions.numel(), _is_f32(proj), _is_f32(self.kpool))
+        K._count()
+
+    def rows(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int = 1) -> None:
+        """The plain kernel: one query row at a time (keys of the rows themselves appended before)."""
+        self._fill(proj, tables, positions, row_seg, part_o, part_ml, nsplit)
+        call("attn_maps_rows", ctypes.byref(self.a), positions.numel(), _is_f32(proj), _is_f32(self.kpool))
+        K._count()
+
+    def finish(self, part_o, part_ml, gates, act, positions, *, nsplit: int = 1, lam: float = 0.0, post_scale: float = 1.0,
+               eps: float = 1e-5) -> None:
+        """Merge splits, ``o = a_0 - lam a_1`` + RMS norm (two maps), ``* post_scale * sigmoid(gate)`` per head."""
+        call("attn_maps_finish", part_o, part_ml, gates, gates.stride(0) if gates is not None else 0, act, act.stride(0), positions,
+             positions.numel(), self.H, self.maps, self.vdim, nsplit, float(lam), float(post_scale), float(eps), _is_f32(act))
+        K._count()

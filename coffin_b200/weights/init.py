@@ -104,6 +104,15 @@ def _draw(shape, kind: str, gen: torch.Generator, device, dtype, std: float) -> 
     if kind == "dt":
         return torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * 0.5
     t = torch.randn(shape, generator=gen, device=device, dtype=torch.float32)
+    if kind in ("hc_in", "hc_out", "hc_mix"):          # static hyper-connection: read about one stream's worth, keep the rest
+        if kind == "hc_mix":
+            return (torch.eye(shape[0], device=device) + 0.1 * torch.randn(shape, generator=gen, device=device)).to(dtype)
+        c = 1.0 / shape[0] if kind == "hc_in" else 1.0
+        return (c * (1.0 + 0.3 * torch.randn(shape, generator=gen, device=device))).to(dtype)
+    if kind == "gate_b":        # input / forget gate biases of a matrix memory
+        return torch.randn(shape, generator=gen, device=device, dtype=torch.float32).to(dtype)
+    if kind == "lam":
+        return (0.1 * torch.randn(shape, generator=gen, device=device)).to(dtype)
     if kind == "norm1":         # plain gain around one (gated norm of the delta-net output)
         return (1.0 + std * t).to(dtype)
     if kind == "conv":          # taps large enough that the conv output is not ~0
@@ -125,7 +134,8 @@ def random_state_dict(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = torc
         return qwen4_random(cfg, seed, dtype=dtype, device=device, std=std)
     sd: dict[str, torch.Tensor] = {}
     dev = torch.device(device)
-    for idx, (key, shape, kind) in enumerate(tensor_plan(cfg, mtp)):
+    plan = cfg.tensor_plan() if hasattr(cfg, "tensor_plan") else tensor_plan(cfg, mtp)      # a family may list its own tensors
+    for idx, (key, shape, kind) in enumerate(plan):
         gen = torch.Generator(device=dev)
         gen.manual_seed(seed * 1_000_003 + idx)
         sd[key] = _draw(shape, kind, gen, dev, dtype, std)
@@ -133,7 +143,7 @@ def random_state_dict(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = torc
 
 
 def param_count(cfg: ModelConfig) -> int:
-    return sum(math.prod(s) for _, s, _ in tensor_plan(cfg))
+    return sum(math.prod(s) for _, s, _ in (cfg.tensor_plan() if hasattr(cfg, "tensor_plan") else tensor_plan(cfg)))
 
 
 def save_checkpoint(cfg: ModelConfig, sd: dict[str, torch.Tensor], out_dir: str | Path,

@@ -14,6 +14,8 @@ from pathlib import Path
 import torch
 
 KEEP_PREFIXES = ("model.language_model.", "mtp.", "lm_head.", "model.visual.")
+# flat naming (Zufilorn): tables, ``l<layer>.<...>``, final norm and head at the top level
+FLAT_KEYS = re.compile(r"(embed|pos|head|final\.norm|l(\d+)\..+)")
 
 
 def shard_files(model_dir: Path) -> list[Path]:
@@ -82,6 +84,9 @@ def load_checkpoint(model_dir: str | Path, device: str = "cpu", vision: bool = T
         plan_of = lambda k: slice_plan(cfg, k, tp[0], tp[1])
 
     def wanted(k: str) -> bool:
+        flat = FLAT_KEYS.fullmatch(k)
+        if flat:
+            return layers is None or flat.group(2) is None or layers[0] <= int(flat.group(2)) < layers[1]
         if not k.startswith(KEEP_PREFIXES) or (not vision and k.startswith("model.visual.")):
             return False
         if layers is not None and k.startswith("model.language_model.layers."):

@@ -80,7 +80,7 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
 
 // One warp per (row, head): merge the key splits of every map, o = a_0 - lambda a_1 (two maps), RMS norm over the
 // head's values without weight (two maps), times post_scale, times sigmoid(gate).
-constexpr int kVMax = 16;      // values per lane: vdim <= 512
+constexpr int kVMax = 16;      // values per lane: vdim <= 512; at most 32 splits
 template <typename TA>
 __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                           const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
@@ -102,16 +102,17 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
     const float* ml = part_ml + vh * nsplit * 2;
     const float* po = part_o + vh * nsplit * vdim;
     float M = -INFINITY;
-    for (int s = lane; s < nsplit; s += 32) M = fmaxf(M, ml[2 * s]);
+    if (lane < nsplit) M = ml[2 * lane];
     M = warp_max(M);
-    float den = 0.f;
-    for (int s = lane; s < nsplit; s += 32) den += ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - M) * ml[2 * s + 1];
+    // splits are filled from the front: each lane weighs its own, the sums walk the filled ones
+    float fac = 0.f, den = 0.f;
+    if (lane < nsplit && ml[2 * lane] != -INFINITY) { fac = expf(ml[2 * lane] - M); den = fac * ml[2 * lane + 1]; }
     den = warp_sum(den);
-    const float c = (mp == 0 ? 1.f : -lambda) / den;
-    for (int s = 0; s < nsplit; ++s) {
-      const float ms = ml[2 * s];
-      if (ms == -INFINITY) continue;
-      const float f = c * expf(ms - M);
+    fac *= (mp == 0 ? 1.f : -lambda) / den;
+    const int used = __popc(__ballot_sync(0xffffffffu, lane < nsplit && ml[2 * lane] != -INFINITY));
+#pragma unroll 4
+    for (int s = 0; s < used; ++s) {
+      const float f = __shfl_sync(0xffffffffu, fac, s);
 #pragma unroll
       for (int i = 0; i < kVMax; ++i) {
         const int v = lane + 32 * i;
@@ -174,7 +175,7 @@ CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const
                                   const void* positions, int64_t rows, int64_t H, int64_t maps, int64_t vdim, int64_t nsplit,
                                   float lambda, float post_scale, float eps, int64_t f32, void* stream) {
   if (!part_o || !part_ml || !act || !positions || rows < 1 || maps < 1 || maps > 2 || nsplit < 1) return CB_ERR_ARG;
-  if (vdim > 32 * kVMax) return CB_ERR_SHAPE;
+  if (vdim > 32 * kVMax || nsplit > 32) return CB_ERR_SHAPE;
   const dim3 grid((unsigned)((rows * H + 3) / 4)), block(128);
   cudaStream_t st = (cudaStream_t)stream;
   if (f32)

@@ -1,0 +1,436 @@
+// Tensor-core prompt kernel and split-key decode kernel of the multi-map attention (attn_maps.cuh), bf16 pages.
+//
+// Prompt: one CTA per (128 consecutive query rows of a segment, head, map); keys and values come page by page through
+// a two-stage cp.async ring.  Scores, cap, query temperature and softmax are fp32.  The weights stay fp32 across the
+// second product: P is split into a bf16 head and a bf16 remainder (16 mantissa bits) and multiplied twice - with two
+// maps the result is a difference of two averages, which would amplify a rounded P.
+// Decode: one CTA per (key split, key/value head, row) walks its pages with every query head and map of the group, so
+// a page is read once; the CTA that owns the newest page appends the token's key and value first.
+// Both leave unnormalised sums and (max, denominator) for maps_finish_kernel.
+#include "attn_maps.cuh"
+
+namespace {
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void cp16(void* s, const void* g, bool ok) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(s);
+  const int n = ok ? 16 : 0;                                     // 0 source bytes: the destination is zero-filled
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(g), "r"(n) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t* r, const void* p) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t* r, const void* p) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// (x, y) -> packed bf16 head; the remainders replace x and y
+__device__ __forceinline__ uint32_t split_head(float& x, float& y) {
+  const uint32_t h = pack_bf162(x, y);
+  x -= __uint_as_float(h << 16);
+  y -= __uint_as_float(h & 0xffff0000u);
+  return h;
+}
+
+constexpr int kBM = 128, kBN = 64, kFT = 256;
+constexpr float kLog2e = 1.4426950408889634f;
+
+template <int DK, int DV>
+constexpr size_t flash_smem() { return sizeof(bf16) * ((size_t)kBM * (DK + 8) + 2 * (size_t)kBN * (DK + 8 + DV + 8)); }
+
+template <int DK, int DV, bool CAP>
+__global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a) {
+  constexpr int LK = DK + 8, LV = DV + 8, NK = DK / 16, NV = DV / 8;
+  constexpr bool QREG = DK <= 128;
+  extern __shared__ __align__(128) unsigned char smem[];
+  bf16* qs = reinterpret_cast<bf16*>(smem);            // [kBM][LK]
+  bf16* ks = qs + kBM * LK;                            // [2][kBN][LK]
+  bf16* vs = ks + 2 * kBN * LK;                        // [2][kBN][LV]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
+  const int vh = blockIdx.y, seg = blockIdx.z;
+  griddep_launch();
+  griddep_wait();
+  const int row0 = a.seg_row[seg], n = a.seg_row[seg + 1] - row0, pos0 = a.seg_pos[seg];
+  const int tile = (int)gridDim.x - 1 - (int)blockIdx.x;         // long tiles first
+  const int t0 = tile * kBM;
+  if (t0 >= n) return;
+  const int h = vh / a.maps, map = vh % a.maps, g = h / (a.H / a.G);
+  const int64_t ldk = (int64_t)a.G * a.maps * a.dim, ldv = (int64_t)a.G * a.vdim;
+  const bf16* K = reinterpret_cast<const bf16*>(a.kpool) + (int64_t)(g * a.maps + map) * a.dim;
+  const bf16* V = reinterpret_cast<const bf16*>(a.vpool) + (int64_t)g * a.vdim;
+  const int* bt = a.tables + (int64_t)seg * a.ldbt;
+  const bf16* Q = reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + t0) * a.ldp + (int64_t)vh * a.dim;
+  const int rows = min(kBM, n - t0);
+  for (int e = tid; e < kBM * (DK / 8); e += kFT) {
+    const int r = e / (DK / 8), c = (e % (DK / 8)) * 8;
+    const bool ok = r < rows && c < a.dim;
+    cp16(qs + r * LK + c, ok ? Q + (int64_t)r * a.ldp + c : Q, ok);
+  }
+  const int last = pos0 + t0 + rows - 1, pages = last / kPage + 1;
+  auto load = [&](int pg) {
+    const int64_t base = (int64_t)bt[pg] * kPage;
+    bf16* kd = ks + (pg & 1) * kBN * LK;
+    bf16* vd = vs + (pg & 1) * kBN * LV;
+    for (int e = tid; e < kBN * (DK / 8); e += kFT) {
+      const int r = e / (DK / 8), c = (e % (DK / 8)) * 8;
+      const bool ok = c < a.dim && pg * kPage + r <= last;
+      cp16(kd + r * LK + c, ok ? K + (base + r) * ldk + c : K, ok);
+    }
+    for (int e = tid; e < kBN * (DV / 8); e += kFT) {
+      const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+      const bool ok = c < a.vdim && pg * kPage + r <= last;
+      cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load(0);
+  float o[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float mx[2] = {-INFINITY, -INFINITY}, den[2] = {0.f, 0.f};
+  const int rlo = warp * 16 + g4;                                // tile rows of this lane: rlo, rlo + 8
+  const int plo = pos0 + t0 + rlo, phi = plo + 8;
+  const float inv_cap = CAP ? 1.f / a.cap : 0.f;
+  float f[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    f[i] = a.scale * query_temp(a, i ? phi : plo);
+    f[i] *= CAP ? 2.f * kLog2e * inv_cap : kLog2e;               // CAP: exponent of exp(2 s / cap); else log2 units
+  }
+  const float cap2 = a.cap * kLog2e;
+  uint32_t qf[QREG ? NK : 1][4];
+  const int warp_last = pos0 + t0 + warp * 16 + 15;
+  for (int pg = 0; pg < pages; ++pg) {
+    if (pg + 1 < pages) {
+      load(pg + 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    if (QREG && pg == 0) {
+#pragma unroll
+      for (int k = 0; k < NK; ++k) ldsm4(qf[QREG ? k : 0], qs + (warp * 16 + (lane & 15)) * LK + k * 16 + (lane >> 4) * 8);
+    }
+    if (pg * kPage <= warp_last) {
+      const bf16* kt = ks + (pg & 1) * kBN * LK;
+      const bf16* vt = vs + (pg & 1) * kBN * LV;
+      float s[8][4];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+#pragma unroll
+      for (int k = 0; k < NK; ++k) {
+        uint32_t qq[4];
+        if (!QREG) ldsm4(qq, qs + (warp * 16 + (lane & 15)) * LK + k * 16 + (lane >> 4) * 8);
+        const uint32_t* qa = QREG ? qf[QREG ? k : 0] : qq;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {                            // 16 keys per load: two n-tiles
+          uint32_t b[4];
+          ldsm4(b, kt + (j * 16 + (lane & 7) + ((lane >> 4) << 3)) * LK + k * 16 + ((lane >> 3) & 1) * 8);
+          mma(s[2 * j], qa, b[0], b[1]);
+          mma(s[2 * j + 1], qa, b[2], b[3]);
+        }
+      }
+      const bool edge = pg * kPage + kPage - 1 > pos0 + t0 + warp * 16;    // some key of the page is after some row
+      float nm[2] = {mx[0], mx[1]};
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float x = s[i][e] * f[e >> 1];
+          if (CAP) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);        // log2(e) * cap * tanh(score / cap)
+          if (edge && pg * kPage + i * 8 + t4 * 2 + (e & 1) > (e >> 1 ? phi : plo)) x = -INFINITY;
+          s[i][e] = x;
+          nm[e >> 1] = fmaxf(nm[e >> 1], x);
+        }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        nm[i] = fmaxf(nm[i], __shfl_xor_sync(0xffffffffu, nm[i], 1));
+        nm[i] = fmaxf(nm[i], __shfl_xor_sync(0xffffffffu, nm[i], 2));
+        // a tile's first page always holds a visible key (key 0), so nm is finite from then on
+        const float w = ex2(mx[i] - nm[i]);
+        if (nm[i] > mx[i]) {
+#pragma unroll
+          for (int v = 0; v < NV; ++v) { o[v][2 * i] *= w; o[v][2 * i + 1] *= w; }
+          den[i] *= w;
+        }
+        mx[i] = nm[i];
+      }
+      // P: bf16 head and remainder, already in A-fragment order
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {                            // a0: row lo, keys 2t..; a1: row hi; a2 / a3: keys + 8
+          const int i = 2 * k + (q >> 1), e = (q & 1) * 2;
+          float x = ex2(s[i][e] - nm[q & 1]), y = ex2(s[i][e + 1] - nm[q & 1]);
+          den[q & 1] += x + y;
+          ph[q] = split_head(x, y);
+          pl[q] = pack_bf162(x, y);
+        }
+#pragma unroll
+        for (int v = 0; v < NV; v += 2) {
+          uint32_t b[4];
+          ldsm4t(b, vt + (k * 16 + (lane & 15)) * LV + v * 8 + (lane >> 4) * 8);
+          mma(o[v], ph, b[0], b[1]);
+          mma(o[v + 1], ph, b[2], b[3]);
+          mma(o[v], pl, b[0], b[1]);
+          mma(o[v + 1], pl, b[2], b[3]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    den[i] += __shfl_xor_sync(0xffffffffu, den[i], 1);
+    den[i] += __shfl_xor_sync(0xffffffffu, den[i], 2);
+    const int r = rlo + 8 * i;
+    if (r >= rows) continue;
+    const int64_t idx = ((int64_t)(row0 + t0 + r) * a.H * a.maps + vh) * a.nsplit;
+    float* po = a.part_o + idx * a.vdim;
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int c = v * 8 + t4 * 2;
+      if (c < a.vdim) *reinterpret_cast<float2*>(po + c) = make_float2(o[v][2 * i], o[v][2 * i + 1]);
+    }
+    if (t4 == 0) {
+      a.part_ml[idx * 2] = mx[i] * (1.f / kLog2e);
+      a.part_ml[idx * 2 + 1] = den[i];
+      for (int sp = 1; sp < a.nsplit; ++sp) a.part_ml[(idx + sp) * 2] = -INFINITY;
+    }
+  }
+}
+
+template <int DK, int DV, bool CAP>
+int flash_launch(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
+  auto kern = maps_flash_kernel<DK, DV, CAP>;
+  constexpr size_t smem = flash_smem<DK, DV>();
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  return (int)cb_launch(kern, dim3((unsigned)tiles, (unsigned)(a.H * a.maps), (unsigned)segs), dim3(kFT), smem, st, a);
+}
+template <int DK>
+int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
+  const bool cap = a.cap > 0.f;
+#define CB_DV(N) \
+  if (a.vdim <= N) return cap ? flash_launch<DK, N, true>(a, tiles, segs, st) : flash_launch<DK, N, false>(a, tiles, segs, st)
+  CB_DV(32); CB_DV(64); CB_DV(128); CB_DV(256);
+#undef CB_DV
+  return CB_ERR_SHAPE;
+}
+
+// ---- decode -------------------------------------------------------------------------------------
+// NQ: query vectors (heads of the group x maps) of one CTA, padded.  256 threads: scores by (key, quarter of dim),
+// values by (8 columns, key group).
+constexpr int kDT = 256;
+template <int NQ, typename TP>
+__global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
+  extern __shared__ __align__(16) float sm[];
+  const int dimp = (a.dim + 31) & ~31;
+  float* q = sm;                           // [NQ][dimp], scaled (log2 units with or without the cap's factor)
+  float* p = q + NQ * dimp;                // [kPage][NQ]
+  float* red = p + kPage * NQ;             // [key groups][vdim]
+  __shared__ float m_s[NQ], l_s[NQ], w_s[NQ];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int split = blockIdx.x, row = blockIdx.z;
+  const int R = a.H / a.G, cpg = (R + hpc - 1) / hpc, g = blockIdx.y / cpg, r0 = (blockIdx.y % cpg) * hpc, nh = min(hpc, R - r0);
+  const int nq = nh * a.maps;
+  griddep_launch();
+  griddep_wait();
+  const int pos = a.positions[row], seg = a.row_seg ? a.row_seg[row] : row;
+  if (pos < 0) return;
+  const int64_t vh0 = (int64_t)row * a.H * a.maps + (int64_t)(g * R + r0) * a.maps;
+  const int pages = pos / kPage + 1, per = (pages + a.nsplit - 1) / a.nsplit;
+  const int pg0 = split * per, pg1 = min(pages, pg0 + per);
+  if (pg0 >= pages) {
+    if (tid < nq) a.part_ml[((vh0 + tid) * a.nsplit + split) * 2] = -INFINITY;
+    return;
+  }
+  const int* bt = a.tables + (int64_t)seg * a.ldbt;
+  const int64_t ldk = (int64_t)a.G * a.maps * a.dim, ldv = (int64_t)a.G * a.vdim;
+  bf16* K = reinterpret_cast<bf16*>(a.kpool) + (int64_t)g * a.maps * a.dim;
+  bf16* V = reinterpret_cast<bf16*>(a.vpool) + (int64_t)g * a.vdim;
+  const TP* pr = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
+  const bool cap = a.cap > 0.f;
+  const float f = a.scale * query_temp(a, pos) * (cap ? 2.f * kLog2e / a.cap : kLog2e), cap2 = a.cap * kLog2e;
+  for (int e = tid; e < NQ * dimp; e += kDT) {
+    const int i = e / dimp, c = e % dimp;
+    q[e] = i < nq && c < a.dim ? act_round<bf16>(act_load(pr + ((int64_t)(g * R + r0) * a.maps + i) * a.dim + c)) * f : 0.f;
+  }
+  if (pg1 == pages) {
+    // this CTA reads the token's own key and value: it stores them (CTAs of other heads of the group store the same)
+    const int64_t slot = (int64_t)bt[pages - 1] * kPage + pos % kPage;
+    for (int c = tid; c < a.maps * a.dim; c += kDT) act_store(K + slot * ldk + c, act_load(pr + a.k_col + (int64_t)g * a.maps * a.dim + c));
+    for (int c = tid; c < a.vdim; c += kDT) act_store(V + slot * ldv + c, act_load(pr + a.v_col + (int64_t)g * a.vdim + c));
+  }
+  if (tid < NQ) { m_s[tid] = -INFINITY; l_s[tid] = 0.f; }
+  const int co = a.vdim >> 3, KG = min(kPage, kDT / co), cg = tid % co, kg = tid / co;
+  float o[NQ][8];
+#pragma unroll
+  for (int i = 0; i < NQ; ++i)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
+  __syncthreads();
+  const int key = tid >> 2, part = tid & 3;
+  for (int pg = pg0; pg < pg1; ++pg) {
+    const int64_t base = (int64_t)bt[pg] * kPage;
+    const bool vis = pg * kPage + key <= pos;
+    // scores: lanes 4k .. 4k + 3 hold quarters of key k
+    for (int mp = 0; mp < a.maps; ++mp) {
+      float s[NQ];
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) s[i] = 0.f;
+      const bf16* kr = K + (base + key) * ldk + (int64_t)mp * a.dim;
+      for (int c = part * 8; c < a.dim; c += 32) {
+        float kf[8];
+        uint4 raw = make_uint4(0, 0, 0, 0);
+        if (vis) raw = *reinterpret_cast<const uint4*>(kr + c);
+        bf16x8_to_float(raw, kf);
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+          if (i * a.maps + mp < nq) {
+            const float4 q0 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c);
+            const float4 q1 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c + 4);
+            s[i] = fmaf(q0.x, kf[0], s[i]); s[i] = fmaf(q0.y, kf[1], s[i]); s[i] = fmaf(q0.z, kf[2], s[i]); s[i] = fmaf(q0.w, kf[3], s[i]);
+            s[i] = fmaf(q1.x, kf[4], s[i]); s[i] = fmaf(q1.y, kf[5], s[i]); s[i] = fmaf(q1.z, kf[6], s[i]); s[i] = fmaf(q1.w, kf[7], s[i]);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        if (i * a.maps + mp >= nq) continue;
+        float x = s[i];
+        x += __shfl_xor_sync(0xffffffffu, x, 1);
+        x += __shfl_xor_sync(0xffffffffu, x, 2);
+        if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
+        if (part == (i & 3)) p[key * NQ + i * a.maps + mp] = vis ? x : -INFINITY;
+      }
+    }
+    __syncthreads();
+    for (int i = warp; i < nq; i += kDT / 32) {
+      const float x0 = p[lane * NQ + i], x1 = p[(lane + 32) * NQ + i], mo = m_s[i];
+      const float mn = fmaxf(mo, warp_max(fmaxf(x0, x1)));       // finite: the first key of a walked page is visible
+      const float e0 = ex2(x0 - mn), e1 = ex2(x1 - mn), w = ex2(mo - mn);
+      const float sum = warp_sum(e0 + e1);
+      p[lane * NQ + i] = e0;
+      p[(lane + 32) * NQ + i] = e1;
+      if (lane == 0) { m_s[i] = mn; l_s[i] = l_s[i] * w + sum; w_s[i] = w; }
+    }
+    __syncthreads();
+    if (kg < KG) {
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        const float w = i < nq ? w_s[i] : 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[i][e] *= w;
+      }
+      const int nk = min(kPage, pos + 1 - pg * kPage);
+#pragma unroll 4
+      for (int k = kg; k < nk; k += KG) {
+        float vf[8];
+        bf16x8_to_float(*reinterpret_cast<const uint4*>(V + (base + k) * ldv + cg * 8), vf);
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+          const float w = p[k * NQ + i];
+          if (i < nq) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[i][e] = fmaf(w, vf[e], o[i][e]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    if (i < nq) {                                                // uniform over the CTA
+      if (kg < KG) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) red[kg * a.vdim + cg * 8 + e] = o[i][e];
+      }
+      __syncthreads();
+      float* po = a.part_o + ((vh0 + i) * a.nsplit + split) * a.vdim;
+      for (int c = tid; c < a.vdim; c += kDT) {
+        float x = 0.f;
+        for (int k = 0; k < KG; ++k) x += red[k * a.vdim + c];
+        po[c] = x;
+      }
+      __syncthreads();
+    }
+  }
+  if (tid < nq) {
+    float* ml = a.part_ml + ((vh0 + tid) * a.nsplit + split) * 2;
+    ml[0] = m_s[tid] * (1.f / kLog2e);
+    ml[1] = l_s[tid];
+  }
+}
+
+template <int NQ, typename TP>
+int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  const int dimp = (a.dim + 31) & ~31, co = a.vdim / 8, KG = kDT / co < kPage ? kDT / co : kPage;
+  const size_t smem = sizeof(float) * ((size_t)NQ * dimp + kPage * NQ + (size_t)KG * a.vdim);
+  auto kern = maps_decode_kernel<NQ, TP>;
+  if (smem > 40 * 1024) {
+    if (smem > 200 * 1024) return CB_ERR_SHAPE;
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  const int R = a.H / a.G;
+  return (int)cb_launch(kern, dim3((unsigned)a.nsplit, (unsigned)(a.G * ((R + hpc - 1) / hpc)), (unsigned)rows), dim3(kDT), smem, st, a, hpc);
+}
+
+}  // namespace
+
+// Whether the prompt / decode kernels of this file take a head of these sizes (16-byte rows; values in 8-column pieces).
+CB_EXPORT int cb_attn_maps_tc_ok(int64_t G, int64_t maps, int64_t dim, int64_t vdim) {
+  return dim % 8 == 0 && vdim % 8 == 0 && dim <= 256 && vdim <= 256 && dim >= 8 && vdim >= 8 && maps >= 1 && maps <= 2 && G >= 1;
+}
+
+// Prompt attention: `segs` segments (seg_row, seg_pos, one block table each) of at most `max_rows` rows; bf16 projection
+// rows, keys and values appended before.
+CB_EXPORT int cb_attn_maps_flash(const void* args, int64_t segs, int64_t max_rows, void* stream) {
+  if (!args || segs < 1 || segs > 65535 || max_rows < 1) return CB_ERR_ARG;
+  const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
+  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G)
+    return CB_ERR_ARG;
+  if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8) return CB_ERR_SHAPE;
+  const int tiles = (int)((max_rows + kBM - 1) / kBM);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (a.dim <= 32) return flash_dv<32>(a, tiles, (int)segs, st);
+  if (a.dim <= 64) return flash_dv<64>(a, tiles, (int)segs, st);
+  if (a.dim <= 128) return flash_dv<128>(a, tiles, (int)segs, st);
+  return flash_dv<256>(a, tiles, (int)segs, st);
+}
+
+// Decode attention of `rows` single tokens (appends their keys and values): splits of every row into part_o / part_ml.
+CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32, void* stream) {
+  if (!args || rows < 1 || rows > 65535) return CB_ERR_ARG;
+  const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
+  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
+      a.nsplit < 1 || a.nsplit > 32)
+    return CB_ERR_ARG;
+  if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim)) return CB_ERR_SHAPE;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int R = a.H / a.G;
+  int hpc = 8 / a.maps;                                  // heads per CTA: at most 8 query vectors
+  if (hpc > R) hpc = R;
+  const int nq = hpc * a.maps;
+  if (p_f32) {
+    if (nq <= 2) return decode_launch<2, float>(a, hpc, (int)rows, st);
+    if (nq <= 4) return decode_launch<4, float>(a, hpc, (int)rows, st);
+    return decode_launch<8, float>(a, hpc, (int)rows, st);
+  }
+  if (nq <= 2) return decode_launch<2, bf16>(a, hpc, (int)rows, st);
+  if (nq <= 4) return decode_launch<4, bf16>(a, hpc, (int)rows, st);
+  return decode_launch<8, bf16>(a, hpc, (int)rows, st);
+}

@@ -196,6 +196,13 @@ class ZufilornModel:
             t = self._bufs[key] = torch.zeros(cap, cols, dtype=dtype, device=self.device)
         return t[:rows]
 
+    def _scratch(self, floats: int) -> torch.Tensor:
+        """Untyped scratch of the chunked recurrences (grows; stream-ordered reuse)."""
+        t = self._bufs.get("scratch")
+        if t is None or t.numel() < floats:
+            t = self._bufs["scratch"] = torch.empty(floats, dtype=torch.float32, device=self.device)
+        return t
+
     def linear(self, W: torch.Tensor, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
         """``out = x @ W^T``; the result type is ``out``'s."""
         T, Kd = x.shape
@@ -237,17 +244,50 @@ class ZufilornModel:
 
     # ------------------------------------------------------------------ mixer cores
     def recur(self, core: X.Linrec, b: RowBatch, proj, gates, og, act, dec) -> None:
-        core.step(proj, gates, og, act, b.seg_pos, b.seg_slot, segs=b.n_seg, seg_row=b.seg_row, dec=dec)
+        n0 = 0
+        if b.n_pre and proj.dtype == torch.bfloat16 and core.chunked:
+            need = (core.chunk_scratch(b.pre_rows, b.n_pre) + 3) // 4
+            core.chunk(proj, gates, og, act, b.seg_row, b.seg_pos, b.seg_slot, self._scratch(need), segs=b.n_pre, max_rows=b.max_rows,
+                       rows=b.pre_rows, dec=dec)
+            n0 = b.n_pre
+        if n0 < b.n_seg:
+            core.step(proj, gates, og, act, b.seg_pos[n0:], b.seg_slot[n0:], segs=b.n_seg - n0,
+                      seg_row=b.seg_row[n0:] if b.seg_row is not None else None, dec=dec)
         if b.n_pre:
             core.ring(proj, b.seg_row, b.seg_pos, b.seg_slot, b.n_pre)
 
     def attend(self, core: X.AttnMaps, b: RowBatch, proj, gates, act, *, lam: float, post_scale: float) -> None:
-        vh = core.H * core.maps
-        part_o = self.buf("part_o", b.T, vh * core.vdim, torch.float32)
-        part_ml = self.buf("part_ml", b.T, vh * 2, torch.float32)
-        core.append(proj, b.tables, b.positions, b.row_seg)
-        core.rows(proj, b.tables, b.positions, b.row_seg, part_o, part_ml)
-        core.finish(part_o, part_ml, gates, act, b.positions, lam=lam, post_scale=post_scale, eps=self.eps)
+        vh, T, P = core.H * core.maps, b.T, b.pre_rows
+        fin = dict(lam=lam, post_scale=post_scale, eps=self.eps)
+
+        def parts(rows: int, nsplit: int):
+            return (self.buf("part_o", rows, vh * nsplit * core.vdim, torch.float32),
+                    self.buf("part_ml", rows, vh * nsplit * 2, torch.float32))
+
+        def sub(r0: int, r1: int):
+            return proj[r0:r1], b.positions[r0:r1], b.row_seg[r0:r1] if b.row_seg is not None else None
+
+        if not core.tc:                 # 32-bit mode, or head sizes outside the tensor-core kernels
+            po, pm = parts(T, 1)
+            core.append(proj, b.tables, b.positions, b.row_seg)
+            core.rows(proj, b.tables, b.positions, b.row_seg, po, pm)
+            core.finish(po, pm, gates, act, b.positions, **fin)
+            return
+        r0 = 0
+        if P:
+            pr, ps, rs = sub(0, P)
+            core.append(pr, b.tables, ps, rs)
+            if proj.dtype == self.dtype:
+                po, pm = parts(P, 1)
+                core.flash(pr, b.tables, b.seg_row, b.seg_pos, po, pm, segs=b.n_pre, max_rows=b.max_rows, positions=ps)
+                core.finish(po, pm, gates[:P], act[:P], ps, **fin)
+                r0 = P
+        if r0 < T:                      # single tokens; the rows of a few short portions are queries like any other
+            pr, ps, rs = sub(r0, T)
+            ns = core.decode_splits(T - r0)
+            po, pm = parts(T - r0, ns)
+            core.decode(pr, b.tables, ps, rs, po, pm, ns)
+            core.finish(po, pm, gates[r0:], act[r0:], ps, nsplit=ns, **fin)
 
     # ------------------------------------------------------------------ the stack
     def _stack(self, b: RowBatch) -> tuple[torch.Tensor, tuple]:

@@ -147,6 +147,24 @@ class Linrec:
         call("linrec_step", ctypes.byref(self.a), self.kind, segs, _is_f32(proj), _is_f32(act))
         K._count()
 
+    @property
+    def chunked(self) -> bool:
+        """Whether prompts of this head size run in chunks on the tensor cores (bf16 activations)."""
+        return bool(_lib.call_nostream("linrec_chunk_ok", self.a.dk, self.a.dv))
+
+    def chunk_scratch(self, rows: int, segs: int) -> int:
+        fn = _lib.lib().cb_linrec_chunk_scratch
+        fn.restype = ctypes.c_int64
+        a = self.a
+        return int(fn(*[ctypes.c_int64(v) for v in (self.kind, rows, segs, a.H, a.dk, a.dv)]))
+
+    def chunk(self, proj, gates, og, act, seg_row, seg_pos, seg_slot, scratch, *, segs: int, max_rows: int, rows: int, dec=None) -> None:
+        """The first ``segs`` segments (rows ``[0, rows)``, at most ``max_rows`` each) in chunks; ``scratch`` bytes as
+        ``chunk_scratch`` says.  The convolution ring is left as it was (``ring`` afterwards)."""
+        self._fill(proj, gates, og, act, dec, seg_row, seg_pos, seg_slot)
+        call("linrec_chunk", ctypes.byref(self.a), self.kind, segs, max_rows, rows, scratch, scratch.numel() * scratch.element_size())
+        K._count(4 if self.kind == MLSTM else 3)
+
     def ring(self, proj, seg_row, seg_pos, seg_slot, segs: int) -> None:
         """After the readers: the raw rows at the end of every segment of two or more tokens enter the ring."""
         r = self.state.get("ring")
@@ -200,6 +218,28 @@ class AttnMaps:
         """The plain kernel: one query row at a time (keys of the rows themselves appended before)."""
         self._fill(proj, tables, positions, row_seg, part_o, part_ml, nsplit)
         call("attn_maps_rows", ctypes.byref(self.a), positions.numel(), _is_f32(proj), _is_f32(self.kpool))
+        K._count()
+
+    @property
+    def tc(self) -> bool:
+        """Whether the tensor-core prompt kernel and the split decode kernel take this head."""
+        return self.kpool.dtype == torch.bfloat16 and bool(_lib.call_nostream("attn_maps_tc_ok", self.G, self.maps, self.dim, self.vdim))
+
+    def flash(self, proj, tables, seg_row, seg_pos, part_o, part_ml, *, segs: int, max_rows: int, positions) -> None:
+        """Portions of several tokens (bf16 projection rows; keys and values appended before)."""
+        self._fill(proj, tables, positions, None, part_o, part_ml, 1, seg_row, seg_pos)
+        call("attn_maps_flash", ctypes.byref(self.a), segs, max_rows)
+        K._count()
+
+    def decode_splits(self, rows: int) -> int:
+        R = self.H // self.G
+        hpc = min(R, 8 // self.maps)
+        return max(1, min(32, 296 // max(1, self.G * -(-R // hpc) * rows)))
+
+    def decode(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
+        """Single tokens (their keys and values are appended by the kernel): ``nsplit`` key splits per row."""
+        self._fill(proj, tables, positions, row_seg, part_o, part_ml, nsplit)
+        call("attn_maps_decode", ctypes.byref(self.a), positions.numel(), _is_f32(proj))
         K._count()
 
     def finish(self, part_o, part_ml, gates, act, positions, *, nsplit: int = 1, lam: float = 0.0, post_scale: float = 1.0,

@@ -134,7 +134,8 @@ def attention(h, W, m, eps):
     q = (h @ W["q"].T).view(T, H, 2, d)
     k = (h @ W["k"].T).view(T, G, 2, d)
     v = (h @ W["v"].T).view(T, G, e)
-    q = q * temperature(T, m["q_temp"]["coef"], m["q_temp"]["every"], h.dtype)[:, None, None, None]
+    if m.get("q_temp"):
+        q = q * temperature(T, m["q_temp"]["coef"], m["q_temp"]["every"], h.dtype)[:, None, None, None]
     lam = torch.exp((W["lq1"] * W["lk1"]).sum()) - torch.exp((W["lq2"] * W["lk2"]).sum()) + m["diff"]
     out = torch.zeros(T, H, e, dtype=h.dtype)
     for i in range(H):

@@ -27,3 +27,15 @@ __device__ __forceinline__ void act_store4(bf16* p, float4 v) {
 __device__ __forceinline__ float sigmoid_x(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_x(float x) { return x * sigmoid_x(x); }
 __device__ __forceinline__ float softplus_x(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+// log(1 + exp(x)) to fp32 relative accuracy everywhere (decays near one need small values right, not just absolutely):
+// log1p(e) = 2 atanh(e / (2 + e)) by the series of the inverse hyperbolic tangent, argument at most 1/3.
+__device__ __forceinline__ float softplus_s(float x) {
+  const float e = __expf(-fabsf(x)), s = __fdividef(e, 2.f + e), q = s * s;
+  float p = 1.f / 13.f;
+  p = fmaf(p, q, 1.f / 11.f); p = fmaf(p, q, 1.f / 9.f); p = fmaf(p, q, 1.f / 7.f);
+  p = fmaf(p, q, 0.2f); p = fmaf(p, q, 1.f / 3.f); p = fmaf(p, q, 1.f);
+  return fmaxf(x, 0.f) + 2.f * s * p;
+}
+__device__ __forceinline__ float sigmoid_s(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+__device__ __forceinline__ float silu_s(float x) { return x * sigmoid_s(x); }

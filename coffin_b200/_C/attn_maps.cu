@@ -94,6 +94,7 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
   const int64_t row = w / H;
   const int h = (int)(w % H);
   if (positions[row] < 0) return;
+  const bool v4 = vdim % 4 == 0;
   float o[kVMax];
 #pragma unroll
   for (int i = 0; i < kVMax; ++i) o[i] = 0.f;
@@ -110,13 +111,20 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
     den = warp_sum(den);
     fac *= (mp == 0 ? 1.f : -lambda) / den;
     const int used = __popc(__ballot_sync(0xffffffffu, lane < nsplit && ml[2 * lane] != -INFINITY));
-#pragma unroll 4
     for (int s = 0; s < used; ++s) {
       const float f = __shfl_sync(0xffffffffu, fac, s);
 #pragma unroll
-      for (int i = 0; i < kVMax; ++i) {
-        const int v = lane + 32 * i;
-        if (v < vdim) o[i] = fmaf(f, po[(int64_t)s * vdim + v], o[i]);
+      for (int i = 0; i < kVMax / 4; ++i) {                      // columns of a lane: 4 (lane + 32 i) .. + 3
+        const int v = 4 * (lane + 32 * i);
+        if (v + 3 < vdim && v4) {
+          const float4 p = *reinterpret_cast<const float4*>(po + (int64_t)s * vdim + v);
+          o[4 * i] = fmaf(f, p.x, o[4 * i]); o[4 * i + 1] = fmaf(f, p.y, o[4 * i + 1]);
+          o[4 * i + 2] = fmaf(f, p.z, o[4 * i + 2]); o[4 * i + 3] = fmaf(f, p.w, o[4 * i + 3]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (v + e < vdim) o[4 * i + e] = fmaf(f, po[(int64_t)s * vdim + v + e], o[4 * i + e]);
+        }
       }
     }
   }
@@ -130,10 +138,76 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
   if (gates) r *= sigmoid_x(gates[row * ldg + h]);
   TA* out = act + row * lda + (int64_t)h * vdim;
 #pragma unroll
-  for (int i = 0; i < kVMax; ++i) {
-    const int v = lane + 32 * i;
-    if (v < vdim) act_store(out + v, o[i] * r);
+  for (int i = 0; i < kVMax / 4; ++i) {
+    const int v = 4 * (lane + 32 * i);
+    if (v + 3 < vdim && v4 && lda % 4 == 0) {
+      act_store4(out + v, make_float4(o[4 * i] * r, o[4 * i + 1] * r, o[4 * i + 2] * r, o[4 * i + 3] * r));
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (v + e < vdim) act_store(out + v + e, o[4 * i + e] * r);
+    }
   }
+}
+
+// The same for rows with many key splits (decode): one CTA per (row, head), its warps share the (map, split) sums.
+constexpr int kWT = 256;
+template <typename TA>
+__global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                               const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
+                                                               int64_t lda, const int* __restrict__ positions, int H, int maps,
+                                                               int vdim, int nsplit, float lambda, float post_scale, float eps) {
+  extern __shared__ float sm[];                        // [warps][vdim]
+  __shared__ float red[32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int64_t row = blockIdx.y;
+  const int h = blockIdx.x;
+  griddep_launch();
+  griddep_wait();
+  if (positions[row] < 0) return;
+  float o[kVMax];
+#pragma unroll
+  for (int i = 0; i < kVMax; ++i) o[i] = 0.f;
+  for (int mp = 0; mp < maps; ++mp) {
+    const int64_t vh = (row * H + h) * maps + mp;
+    const float* ml = part_ml + vh * nsplit * 2;
+    const float* po = part_o + vh * nsplit * vdim;
+    float2 v = make_float2(-INFINITY, 0.f);
+    if (lane < nsplit) v = *reinterpret_cast<const float2*>(ml + 2 * lane);
+    const float M = warp_max(v.x);
+    float fac = v.x == -INFINITY ? 0.f : expf(v.x - M);
+    const float den = warp_sum(fac * v.y);
+    fac *= (mp == 0 ? 1.f : -lambda) / den;
+    const int used = __popc(__ballot_sync(0xffffffffu, v.x != -INFINITY));
+#pragma unroll 4
+    for (int s = warp; s < used; s += kWT / 32) {
+      const float f = __shfl_sync(0xffffffffu, fac, s);
+#pragma unroll
+      for (int i = 0; i < kVMax; ++i) {
+        const int c = lane + 32 * i;
+        if (c < vdim) o[i] = fmaf(f, po[(int64_t)s * vdim + c], o[i]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kVMax; ++i)
+    if (lane + 32 * i < vdim) sm[warp * vdim + lane + 32 * i] = o[i];
+  __syncthreads();
+  float x[2] = {0.f, 0.f}, ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int c = tid + kWT * k;
+    if (c < vdim)
+#pragma unroll
+      for (int w = 0; w < kWT / 32; ++w) x[k] += sm[w * vdim + c];
+    ss = fmaf(x[k], x[k], ss);
+  }
+  float r = post_scale;
+  if (maps > 1) r *= 1.f / sqrtf(block_sum(ss, red) / (float)vdim + eps);
+  if (gates) r *= sigmoid_x(gates[row * ldg + h]);
+#pragma unroll
+  for (int k = 0; k < 2; ++k)
+    if (tid + kWT * k < vdim) act_store(act + row * lda + (int64_t)h * vdim + tid + kWT * k, x[k] * r);
 }
 
 bool maps_args_ok(const AttnMapsArgs& a) {
@@ -176,8 +250,19 @@ CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const
                                   float lambda, float post_scale, float eps, int64_t f32, void* stream) {
   if (!part_o || !part_ml || !act || !positions || rows < 1 || maps < 1 || maps > 2 || nsplit < 1) return CB_ERR_ARG;
   if (vdim > 32 * kVMax || nsplit > 32) return CB_ERR_SHAPE;
-  const dim3 grid((unsigned)((rows * H + 3) / 4)), block(128);
   cudaStream_t st = (cudaStream_t)stream;
+  if (nsplit > 4 && rows <= 65535) {
+    const size_t smem = sizeof(float) * (size_t)(kWT / 32) * vdim;
+    const dim3 wide((unsigned)H, (unsigned)rows);
+    if (f32)
+      return (int)cb_launch(maps_finish_wide_kernel<float>, wide, dim3(kWT), smem, st, (const float*)part_o, (const float*)part_ml,
+                            (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)H, (int)maps, (int)vdim,
+                            (int)nsplit, lambda, post_scale, eps);
+    return (int)cb_launch(maps_finish_wide_kernel<bf16>, wide, dim3(kWT), smem, st, (const float*)part_o, (const float*)part_ml,
+                          (const float*)gates, ldg, (bf16*)act, lda, (const int*)positions, (int)H, (int)maps, (int)vdim, (int)nsplit,
+                          lambda, post_scale, eps);
+  }
+  const dim3 grid((unsigned)((rows * H + 3) / 4)), block(128);
   if (f32)
     return (int)cb_launch(maps_finish_kernel<float>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
                           (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps,

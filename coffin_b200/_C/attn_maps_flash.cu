@@ -233,13 +233,13 @@ int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
 // NQ: query vectors (heads of the group x maps) of one CTA, padded.  256 threads: scores by (key, quarter of dim),
 // values by (8 columns, key group).
 constexpr int kDT = 256;
-template <int NQ, typename TP>
+template <int NQ, int DC, typename TP>      // DC: 8-value pieces of a key per thread and map
 __global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
   extern __shared__ __align__(16) float sm[];
   const int dimp = (a.dim + 31) & ~31;
   float* q = sm;                           // [NQ][dimp], scaled (log2 units with or without the cap's factor)
   float* p = q + NQ * dimp;                // [kPage][NQ]
-  float* red = p + kPage * NQ;             // [key groups][vdim]
+  float* red = p + kPage * NQ;             // [NQ][key groups][vdim]
   __shared__ float m_s[NQ], l_s[NQ], w_s[NQ];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int split = blockIdx.x, row = blockIdx.z;
@@ -285,24 +285,43 @@ __global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, 
   for (int pg = pg0; pg < pg1; ++pg) {
     const int64_t base = (int64_t)bt[pg] * kPage;
     const bool vis = pg * kPage + key <= pos;
+    // everything this thread reads of the page, requested at once
+    uint4 kr[2][DC], vr[8];
+#pragma unroll
+    for (int mp = 0; mp < 2; ++mp)
+#pragma unroll
+      for (int j = 0; j < DC; ++j) {
+        const int c = part * 8 + 32 * j;
+        kr[mp][j] = mp < a.maps && c < a.dim && vis ? *reinterpret_cast<const uint4*>(K + (base + key) * ldk + (int64_t)mp * a.dim + c)
+                                                    : make_uint4(0, 0, 0, 0);
+      }
+    const int nk = min(kPage, pos + 1 - pg * kPage);
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      const int k = kg + u * KG;
+      vr[u] = kg < KG && k < nk ? *reinterpret_cast<const uint4*>(V + (base + k) * ldv + cg * 8) : make_uint4(0, 0, 0, 0);
+    }
     // scores: lanes 4k .. 4k + 3 hold quarters of key k
-    for (int mp = 0; mp < a.maps; ++mp) {
+#pragma unroll
+    for (int mp = 0; mp < 2; ++mp) {
+      if (mp >= a.maps) break;
       float s[NQ];
 #pragma unroll
       for (int i = 0; i < NQ; ++i) s[i] = 0.f;
-      const bf16* kr = K + (base + key) * ldk + (int64_t)mp * a.dim;
-      for (int c = part * 8; c < a.dim; c += 32) {
-        float kf[8];
-        uint4 raw = make_uint4(0, 0, 0, 0);
-        if (vis) raw = *reinterpret_cast<const uint4*>(kr + c);
-        bf16x8_to_float(raw, kf);
 #pragma unroll
-        for (int i = 0; i < NQ; ++i) {
-          if (i * a.maps + mp < nq) {
-            const float4 q0 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c);
-            const float4 q1 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c + 4);
-            s[i] = fmaf(q0.x, kf[0], s[i]); s[i] = fmaf(q0.y, kf[1], s[i]); s[i] = fmaf(q0.z, kf[2], s[i]); s[i] = fmaf(q0.w, kf[3], s[i]);
-            s[i] = fmaf(q1.x, kf[4], s[i]); s[i] = fmaf(q1.y, kf[5], s[i]); s[i] = fmaf(q1.z, kf[6], s[i]); s[i] = fmaf(q1.w, kf[7], s[i]);
+      for (int j = 0; j < DC; ++j) {
+        const int c = part * 8 + 32 * j;
+        float kf[8];
+        bf16x8_to_float(kr[mp][j], kf);
+        if (c < a.dim) {
+#pragma unroll
+          for (int i = 0; i < NQ; ++i) {
+            if (i * a.maps + mp < nq) {
+              const float4 q0 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c);
+              const float4 q1 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c + 4);
+              s[i] = fmaf(q0.x, kf[0], s[i]); s[i] = fmaf(q0.y, kf[1], s[i]); s[i] = fmaf(q0.z, kf[2], s[i]); s[i] = fmaf(q0.w, kf[3], s[i]);
+              s[i] = fmaf(q1.x, kf[4], s[i]); s[i] = fmaf(q1.y, kf[5], s[i]); s[i] = fmaf(q1.z, kf[6], s[i]); s[i] = fmaf(q1.w, kf[7], s[i]);
+            }
           }
         }
       }
@@ -334,39 +353,41 @@ __global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, 
 #pragma unroll
         for (int e = 0; e < 8; ++e) o[i][e] *= w;
       }
-      const int nk = min(kPage, pos + 1 - pg * kPage);
-#pragma unroll 4
-      for (int k = kg; k < nk; k += KG) {
-        float vf[8];
-        bf16x8_to_float(*reinterpret_cast<const uint4*>(V + (base + k) * ldv + cg * 8), vf);
 #pragma unroll
-        for (int i = 0; i < NQ; ++i) {
-          const float w = p[k * NQ + i];
-          if (i < nq) {
+      for (int u = 0; u < 8; ++u) {
+        const int k = kg + u * KG;
+        if (k < nk) {
+          float vf[8];
+          bf16x8_to_float(vr[u], vf);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) o[i][e] = fmaf(w, vf[e], o[i][e]);
+          for (int i = 0; i < NQ; ++i) {
+            if (i < nq) {
+              const float w = p[k * NQ + i];
+#pragma unroll
+              for (int e = 0; e < 8; ++e) o[i][e] = fmaf(w, vf[e], o[i][e]);
+            }
           }
         }
       }
     }
     __syncthreads();
   }
+  if (kg < KG) {
 #pragma unroll
-  for (int i = 0; i < NQ; ++i) {
-    if (i < nq) {                                                // uniform over the CTA
-      if (kg < KG) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) red[kg * a.vdim + cg * 8 + e] = o[i][e];
+    for (int i = 0; i < NQ; ++i)
+      if (i < nq) {
+        float4* d = reinterpret_cast<float4*>(red + ((int64_t)i * KG + kg) * a.vdim + cg * 8);
+        d[0] = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
+        d[1] = make_float4(o[i][4], o[i][5], o[i][6], o[i][7]);
       }
-      __syncthreads();
-      float* po = a.part_o + ((vh0 + i) * a.nsplit + split) * a.vdim;
-      for (int c = tid; c < a.vdim; c += kDT) {
-        float x = 0.f;
-        for (int k = 0; k < KG; ++k) x += red[k * a.vdim + c];
-        po[c] = x;
-      }
-      __syncthreads();
-    }
+  }
+  __syncthreads();
+  for (int e = tid; e < nq * a.vdim; e += kDT) {
+    const int i = e / a.vdim, c = e % a.vdim;
+    float x = 0.f;
+#pragma unroll 8
+    for (int k = 0; k < KG; ++k) x += red[(i * KG + k) * a.vdim + c];
+    a.part_o[((vh0 + i) * a.nsplit + split) * a.vdim + c] = x;
   }
   if (tid < nq) {
     float* ml = a.part_ml + ((vh0 + tid) * a.nsplit + split) * 2;
@@ -375,11 +396,11 @@ __global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, 
   }
 }
 
-template <int NQ, typename TP>
+template <int NQ, int DC, typename TP>
 int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
   const int dimp = (a.dim + 31) & ~31, co = a.vdim / 8, KG = kDT / co < kPage ? kDT / co : kPage;
-  const size_t smem = sizeof(float) * ((size_t)NQ * dimp + kPage * NQ + (size_t)KG * a.vdim);
-  auto kern = maps_decode_kernel<NQ, TP>;
+  const size_t smem = sizeof(float) * ((size_t)NQ * dimp + kPage * NQ + (size_t)NQ * KG * a.vdim);
+  auto kern = maps_decode_kernel<NQ, DC, TP>;
   if (smem > 40 * 1024) {
     if (smem > 200 * 1024) return CB_ERR_SHAPE;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -387,6 +408,13 @@ int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
   }
   const int R = a.H / a.G;
   return (int)cb_launch(kern, dim3((unsigned)a.nsplit, (unsigned)(a.G * ((R + hpc - 1) / hpc)), (unsigned)rows), dim3(kDT), smem, st, a, hpc);
+}
+template <int NQ, typename TP>
+int decode_dim(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  if (a.dim <= 32) return decode_launch<NQ, 1, TP>(a, hpc, rows, st);
+  if (a.dim <= 64) return decode_launch<NQ, 2, TP>(a, hpc, rows, st);
+  if (a.dim <= 128) return decode_launch<NQ, 4, TP>(a, hpc, rows, st);
+  return decode_launch<NQ, 8, TP>(a, hpc, rows, st);
 }
 
 }  // namespace
@@ -426,11 +454,11 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   if (hpc > R) hpc = R;
   const int nq = hpc * a.maps;
   if (p_f32) {
-    if (nq <= 2) return decode_launch<2, float>(a, hpc, (int)rows, st);
-    if (nq <= 4) return decode_launch<4, float>(a, hpc, (int)rows, st);
-    return decode_launch<8, float>(a, hpc, (int)rows, st);
+    if (nq <= 2) return decode_dim<2, float>(a, hpc, (int)rows, st);
+    if (nq <= 4) return decode_dim<4, float>(a, hpc, (int)rows, st);
+    return decode_dim<8, float>(a, hpc, (int)rows, st);
   }
-  if (nq <= 2) return decode_launch<2, bf16>(a, hpc, (int)rows, st);
-  if (nq <= 4) return decode_launch<4, bf16>(a, hpc, (int)rows, st);
-  return decode_launch<8, bf16>(a, hpc, (int)rows, st);
+  if (nq <= 2) return decode_dim<2, bf16>(a, hpc, (int)rows, st);
+  if (nq <= 4) return decode_dim<4, bf16>(a, hpc, (int)rows, st);
+  return decode_dim<8, bf16>(a, hpc, (int)rows, st);
 }

@@ -42,6 +42,45 @@ __device__ __forceinline__ float row_dot(const TW* __restrict__ w, const float* 
   return s0 + s1;
 }
 
+// Low-rank factor times a short vector, rows x rank spread over the block in 16-byte pieces (2^lsh lanes per row).  The
+// weights do not depend on the previous kernel, so the first PRE pieces of a thread are requested ahead of the
+// dependency wait and used once the vector is there.
+template <int PRE>
+struct LowRank {
+  uint4 w[PRE];
+  const bf16* W;
+  int rows, nch, lsh, iters;
+  __device__ __forceinline__ void init(const bf16* W_, int rows_, int rank) {
+    W = W_; rows = rows_; nch = rank >> 3;
+    lsh = nch <= 1 ? 0 : 32 - __clz(nch - 1);
+    iters = ((rows << lsh) + kT - 1) / kT;
+#pragma unroll
+    for (int i = 0; i < PRE; ++i) w[i] = i < iters ? piece(i) : make_uint4(0, 0, 0, 0);
+  }
+  __device__ __forceinline__ uint4 piece(int it) const {
+    const int i = it * kT + (int)threadIdx.x, r = i >> lsh, c = i & ((1 << lsh) - 1);
+    return r < rows && c < nch ? *reinterpret_cast<const uint4*>(W + ((int64_t)r * nch + c) * 8) : make_uint4(0, 0, 0, 0);
+  }
+  // out[r] = W[r, :] . x, by the first lane of a row
+  __device__ __forceinline__ void dot_piece(int it, const uint4& v, const float* x, float* out) const {
+    const int i = it * kT + (int)threadIdx.x, r = i >> lsh, c = i & ((1 << lsh) - 1);
+    float f[8], s = 0.f;
+    bf16x8_to_float(v, f);
+    if (c < nch) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s = fmaf(f[e], x[c * 8 + e], s);
+    }
+    for (int o = 1; o < (1 << lsh); o <<= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (c == 0 && r < rows) out[r] = s;
+  }
+  __device__ __forceinline__ void run(const float* x, float* out) const {
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+      if (i < iters) dot_piece(i, w[i], x, out);
+    for (int i = PRE; i < iters; ++i) dot_piece(i, piece(i), x, out);
+  }
+};
+
 // sums of three values over the block; every thread gets them
 __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* red) {
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
@@ -74,6 +113,12 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
   const int cq = jc >> 2, RG = kT / cq, q4 = tid % cq, rg = tid / cq;
   const bool act_thr = rg < RG;
   const int j0 = rank * jc, ncol = min(jc, dv - j0);   // ncol > 0 by construction of the grid
+  constexpr bool kLow = KIND == LINREC_DELTA && sizeof(TA) == 2;
+  const bool low_a = kLow && !a.dec && a.ra <= 256, low_g = kLow && !a.og && a.rg <= 256;
+  LowRank<kLow ? 8 : 1> lra;
+  LowRank<kLow ? 4 : 1> lrg;
+  if (low_a) lra.init(reinterpret_cast<const bf16*>(a.a2) + (int64_t)h * dk * a.ra, dk, (int)a.ra);
+  if (low_g) lrg.init(reinterpret_cast<const bf16*>(a.g2) + ((int64_t)h * dv + j0) * a.rg, ncol, (int)a.rg);
   griddep_launch();
   griddep_wait();
   const int row0 = a.seg_row ? a.seg_row[seg] : seg;
@@ -141,12 +186,15 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
       block_sum3(q2, k2, qk, red);
       const float rq = 1.f / (sqrtf(q2 + 1e-6f) * sqrtf((float)dk)), rk = 1.f / sqrtf(k2 + 1e-6f);
       kq = qk * rq * rk;
+      if (low_a) lra.run(low, sg);
+      if (low_g) lrg.run(low + (a.dec ? 0 : a.ra), sog);
+      if (low_a || low_g) __syncthreads();
       const float ea = expf(a.A_log[h]);
       const TA* a2 = reinterpret_cast<const TA*>(a.a2);
       for (int c = tid; c < dk; c += kT) {
         sq[c] *= rq; sk[c] *= rk;
         const int64_t ch = (int64_t)h * dk + c;
-        const float x = a.dec ? a.dec[row * a.ldd + ch] : row_dot(a2 + ch * a.ra, low, a.ra);
+        const float x = a.dec ? a.dec[row * a.ldd + ch] : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
         sg[c] = expf(-ea * softplus_x(x + a.dt_bias[ch]));
       }
       bb = sigmoid_x(a.gates[row * a.ldg + h]);            // beta
@@ -154,7 +202,7 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
       const float* lg = low + (a.dec ? 0 : a.ra);
       for (int c = tid; c < ncol; c += kT) {
         const int64_t ch = (int64_t)h * dv + j0 + c;
-        const float x = a.og ? act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch) : row_dot(g2 + ch * a.rg, lg, a.rg);
+        const float x = a.og ? act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
         sog[c] = sigmoid_x(x);
       }
     } else {

@@ -81,7 +81,7 @@ __device__ __forceinline__ int64_t block_index(int row0, int seg, int chunk) { r
 // ---- prep: delta -------------------------------------------------------------------------------
 constexpr int kPT = 128;
 template <int DK, int TAPS>
-__global__ void __launch_bounds__(kPT) chunk_prep_delta_kernel(const ChunkArgs ca) {
+__global__ void __launch_bounds__(kPT, 5) chunk_prep_delta_kernel(const ChunkArgs ca) {
   using I = Image<LINREC_DELTA, DK>;
   constexpr int LD = DK + 4;
   const LinrecArgs& a = ca.r;
@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(kPT) chunk_prep_delta_kernel(const ChunkArgs c
     const int c = 2 * (part == 0 ? e : (part == 1 ? e - kd : e - a.dk));
     const int64_t ch = part == 0 ? qb + c : (part == 1 ? a.k_col + qb + c : a.v_col + (int64_t)h * a.dv + c);
     auto emit = [&](int t, float x, float y) {
-      x = silu_x(x); y = silu_x(y);
+      x = silu_s(x); y = silu_s(y);
       if (t >= m) x = y = 0.f;
       if (part == 0) { sq[t * LD + c] = x; sq[t * LD + c + 1] = y; }
       else if (part == 1) { sk[t * LD + c] = x; sk[t * LD + c + 1] = y; }
@@ -162,7 +162,7 @@ __global__ void __launch_bounds__(kPT) chunk_prep_delta_kernel(const ChunkArgs c
     for (int t = 0; t < C; ++t) x[t] = ok && t < m ? a.dec[(int64_t)(row0 + c0 + t) * a.ldd + (int64_t)h * a.dk + c] : 0.f;
 #pragma unroll
     for (int t = 0; t < C; ++t) {
-      if (ok && t < m) L -= ea * softplus_x(x[t] + db);
+      if (ok && t < m) L -= ea * softplus_s(x[t] + db);
       sL[t * LD + c] = L;
     }
     if (!ok)
@@ -198,20 +198,32 @@ __global__ void __launch_bounds__(kPT) chunk_prep_delta_kernel(const ChunkArgs c
     float kt[DK / 32], qt[DK / 32], Lt[DK / 32];
 #pragma unroll
     for (int j = 0; j < DK / 32; ++j) { kt[j] = sk[t * LD + lane + 32 * j]; qt[j] = sq[t * LD + lane + 32 * j]; Lt[j] = sL[t * LD + lane + 32 * j]; }
-#pragma unroll 2
-    for (int s = 0; s <= t; ++s) {
-      float pa = 0.f, pb = 0.f;
+#pragma unroll 1
+    for (int s = 0; s <= t; s += 2) {                            // two tokens s: four sums share the reduction tree
+      float pa[2] = {0.f, 0.f}, pb[2] = {0.f, 0.f};
 #pragma unroll
-      for (int j = 0; j < DK / 32; ++j) {
-        const float x = sk[s * LD + lane + 32 * j] * ex2(Lt[j] - sL[s * LD + lane + 32 * j]);
-        pa = fmaf(kt[j], x, pa);
-        pb = fmaf(qt[j], x, pb);
+      for (int u = 0; u < 2; ++u) {                              // s + 1 may be t + 1 <= 15 (discarded; its factor is cut off at 1)
+#pragma unroll
+        for (int j = 0; j < DK / 32; ++j) {
+          const float x = sk[(s + u) * LD + lane + 32 * j] * ex2(fminf(Lt[j] - sL[(s + u) * LD + lane + 32 * j], 0.f));
+          pa[u] = fmaf(kt[j], x, pa[u]);
+          pb[u] = fmaf(qt[j], x, pb[u]);
+        }
       }
-      pa = warp_sum(pa);
-      pb = warp_sum(pb);
-      if (lane == 0) {
-        sA[t][s] = pa * beta[t];
-        put1(im + I::bh + t * 24 + s, im + I::bl + t * 24 + s, pb);
+      // halves of the warp keep s / s + 1, quarters keep A / B
+      const bool hi = lane & 16, hq = lane & 8;
+      float ka = hi ? pa[1] : pa[0], kb = hi ? pb[1] : pb[0];
+      ka += __shfl_xor_sync(0xffffffffu, hi ? pa[0] : pa[1], 16);
+      kb += __shfl_xor_sync(0xffffffffu, hi ? pb[0] : pb[1], 16);
+      float k = hq ? kb : ka;
+      k += __shfl_xor_sync(0xffffffffu, hq ? ka : kb, 8);
+      k += __shfl_xor_sync(0xffffffffu, k, 4);
+      k += __shfl_xor_sync(0xffffffffu, k, 2);
+      k += __shfl_xor_sync(0xffffffffu, k, 1);
+      const int su = s + (hi ? 1 : 0);
+      if ((lane & 7) == 0 && su <= t) {
+        if (hq) put1(im + I::bh + t * 24 + su, im + I::bl + t * 24 + su, k);
+        else sA[t][su] = k * beta[t];
       }
     }
     if (lane > t && lane < C) put1(im + I::bh + t * 24 + lane, im + I::bl + t * 24 + lane, 0.f);
@@ -232,40 +244,50 @@ __global__ void __launch_bounds__(kPT) chunk_prep_delta_kernel(const ChunkArgs c
 }
 
 // ---- prep: mLSTM -------------------------------------------------------------------------------
-// Log gates and the running maximum, one warp per (head, segment); the segment's last m becomes the slot's.
-__global__ void __launch_bounds__(32) chunk_gates_mlstm_kernel(const ChunkArgs ca) {
+// Log gates and the running maximum, one block per (head, segment): m_t = max(F_t + m_0, M_t) with (F, M) the prefix of
+// the pairs (f, i) under (F, M) o (f, i) = (F + f, max(M + f, i)); the segment's last m becomes the slot's.
+constexpr int kGT = 512;
+__global__ void __launch_bounds__(kGT) chunk_gates_mlstm_kernel(const ChunkArgs ca) {
   const LinrecArgs& a = ca.r;
-  const int lane = threadIdx.x, h = blockIdx.x, seg = blockIdx.y;
+  __shared__ float wF[kGT / 32], wM[kGT / 32], m_s;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, seg = blockIdx.y;
   griddep_launch();
   griddep_wait();
   const int row0 = a.seg_row[seg], n = a.seg_row[seg + 1] - row0, slot = a.seg_slot[seg];
   if (slot < 0 || n < 1) return;
   float m0 = a.m[(int64_t)slot * a.H + h];
   const float bi = a.gate_b[h], bf = a.gate_b[a.H + h];
-  for (int t0 = 0; t0 < n; t0 += 32) {
-    const int t = t0 + lane;
+  for (int t0 = 0; t0 < n; t0 += kGT) {
+    const int t = t0 + tid;
     const int64_t row = row0 + t;
     float ig = -INFINITY, fg = 0.f;
     if (t < n) {
       ig = a.cap * tanhf((a.gates[row * a.ldg + h] + bi) / a.cap);
       fg = -softplus_x(-a.cap * tanhf((a.gates[row * a.ldg + a.H + h] + bf) / a.cap));
     }
-    float F = fg, M = ig;                                       // m_t = max(F + m0, M) over the tokens so far
+    float F = fg, M = ig;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
       if (lane >= o) { M = fmaxf(Mp + F, M); F += Fp; }
     }
-    const float mt = fmaxf(F + m0, M);
+    if (lane == 31) { wF[warp] = F; wM[warp] = M; }
+    __syncthreads();
+    float mw = m0;                                               // m before this warp's tokens
+    for (int w = 0; w < warp; ++w) mw = fmaxf(wF[w] + mw, wM[w]);
+    const float mt = fmaxf(F + mw, M);
     float mb = __shfl_up_sync(0xffffffffu, mt, 1);
-    if (lane == 0) mb = m0;
+    if (lane == 0) mb = mw;
     if (t < n) {
       const int64_t i = row * a.H + h;
       ca.gi[i] = ig; ca.gf[i] = fg; ca.gm[i] = mt; ca.gb[i] = mb;
     }
-    m0 = __shfl_sync(0xffffffffu, mt, min(31, n - 1 - t0));
+    if (t == min(n, t0 + kGT) - 1) m_s = mt;
+    __syncthreads();
+    m0 = m_s;
+    __syncthreads();
   }
-  if (lane == 0) a.m[(int64_t)slot * a.H + h] = m0;
+  if (tid == 0) a.m[(int64_t)slot * a.H + h] = m0;
 }
 
 template <int DK>
@@ -380,18 +402,19 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
     for (int e = tid; e < (int)(I::bytes / 16); e += TH)
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + e * 16), "l"(src + (size_t)e * 16) : "memory");
   };
-  // values of the chunk in accumulator order: [token tile][row lo / hi, token 2t, 2t + 1]
-  auto values = [&](int ch, float (*v)[4]) {
+  // values of the chunk in accumulator order: [token tile][row lo / hi, token 2t, 2t + 1], as raw bits (nothing is computed
+  // on them here, so that the loads of the next chunk stay in flight)
+  auto values = [&](int ch, uint32_t (*v)[4]) {
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = ch * C + i * 8 + t4 * 2 + (e & 1), vv = e >> 1 ? vb : va;
-        float x = 0.f;
+        uint32_t x = 0;
         if (t < n && vv < vlim) {
-          if (nrm) x = 1.f;
-          else if (KIND == LINREC_DELTA) x = ca.v[(int64_t)(row0 + t) * a.H * a.dv + (int64_t)h * a.dv + vv];
-          else x = __bfloat162float(reinterpret_cast<const bf16*>(a.proj)[(int64_t)(row0 + t) * a.ldp + a.v_col + (int64_t)h * a.dv + vv]);
+          if (nrm) x = 0x3f80u;                                  // bf16 one
+          else if (KIND == LINREC_DELTA) x = __float_as_uint(ca.v[(int64_t)(row0 + t) * a.H * a.dv + (int64_t)h * a.dv + vv]);
+          else x = reinterpret_cast<const unsigned short*>(a.proj)[(int64_t)(row0 + t) * a.ldp + a.v_col + (int64_t)h * a.dv + vv];
         }
         v[i][e] = x;
       }
@@ -401,7 +424,7 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
     if (s < chunks) load(s);
     asm volatile("cp.async.commit_group;" ::: "memory");
   }
-  float vn[2][4];
+  uint32_t vn[2][4];
   values(0, vn);
   for (int ch = 0; ch < chunks; ++ch) {
     asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
@@ -412,7 +435,7 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[i][e] = vn[i][e];
+      for (int e = 0; e < 4; ++e) v[i][e] = __uint_as_float(KIND == LINREC_DELTA ? vn[i][e] : vn[i][e] << 16);
     if (ch + 1 < chunks) values(ch + 1, vn);
     const bf16* im = reinterpret_cast<const bf16*>(smem + (ch % STAGES) * I::bytes);
     const float* G = reinterpret_cast<const float*>(im + I::g);
@@ -536,23 +559,24 @@ __global__ void __launch_bounds__(128) chunk_finish_kernel(const ChunkArgs ca, i
   const float* nw = a.norm_w + (KIND == LINREC_MLSTM ? (int64_t)h * a.dv : 0);
   float inv = 1.f;
   if (KIND == LINREC_MLSTM) inv = 1.f / (fmaxf(fabsf(ca.nq[row * a.H + h]), expf(-ca.gm[row * a.H + h])) + 1e-6f);
-  float2 x[kVMax / 2];
+  float4 x[kVMax / 4];
   float ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < kVMax / 2; ++i) {
-    const int c = 2 * (lane + 32 * i);
-    x[i] = c < a.dv ? *reinterpret_cast<const float2*>(o + c) : make_float2(0.f, 0.f);
-    x[i].x *= inv; x[i].y *= inv;
-    ss = fmaf(x[i].x, x[i].x, fmaf(x[i].y, x[i].y, ss));
+  for (int i = 0; i < kVMax / 4; ++i) {
+    const int c = 4 * (lane + 32 * i);
+    x[i] = c < a.dv ? *reinterpret_cast<const float4*>(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    x[i].x *= inv; x[i].y *= inv; x[i].z *= inv; x[i].w *= inv;
+    ss = fmaf(x[i].x, x[i].x, fmaf(x[i].y, x[i].y, fmaf(x[i].z, x[i].z, fmaf(x[i].w, x[i].w, ss))));
   }
   const float r = 1.f / sqrtf(warp_sum(ss) / (float)a.dv + a.eps);
   bf16* out = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * a.dv;
 #pragma unroll
-  for (int i = 0; i < kVMax / 2; ++i) {
-    const int c = 2 * (lane + 32 * i);
+  for (int i = 0; i < kVMax / 4; ++i) {
+    const int c = 4 * (lane + 32 * i);
     if (c < a.dv) {
-      const float2 gt = ld2(og + c);
-      *reinterpret_cast<uint32_t*>(out + c) = pack_bf162(x[i].x * r * nw[c] * sigmoid_x(gt.x), x[i].y * r * nw[c + 1] * sigmoid_x(gt.y));
+      const float4 gt = act_load4(og + c), w4 = *reinterpret_cast<const float4*>(nw + c);
+      act_store4(out + c, make_float4(x[i].x * r * w4.x * sigmoid_s(gt.x), x[i].y * r * w4.y * sigmoid_s(gt.y),
+                                      x[i].z * r * w4.z * sigmoid_s(gt.z), x[i].w * r * w4.w * sigmoid_s(gt.w)));
     }
   }
 }
@@ -577,7 +601,7 @@ int run_chunks(const ChunkArgs& ca, int max_rows, int rows, cudaStream_t st) {
 #undef CB_PREP
     if (e != cudaSuccess) return (int)e;
   } else {
-    e = cb_launch(chunk_gates_mlstm_kernel, dim3((unsigned)a.H, (unsigned)ca.segs), dim3(32), 0, st, ca);
+    e = cb_launch(chunk_gates_mlstm_kernel, dim3((unsigned)a.H, (unsigned)ca.segs), dim3(kGT), 0, st, ca);
     if (e != cudaSuccess) return (int)e;
     const size_t smem = sizeof(bf16) * 2 * C * I::P;
     e = cb_launch(chunk_prep_mlstm_kernel<DK>, dim3((unsigned)chunks, (unsigned)a.H, (unsigned)ca.segs), dim3(64), smem, st, ca);
@@ -624,7 +648,7 @@ CB_EXPORT int cb_linrec_chunk(const void* args, int64_t kind, int64_t segs, int6
   const LinrecArgs& a = ca.r;
   if (!a.proj || !a.gates || !a.act || !a.og || !a.seg_row || !a.seg_pos || !a.seg_slot || !a.S || a.H < 1 || a.G < 1 || a.H % a.G)
     return CB_ERR_ARG;
-  if (!cb_linrec_chunk_ok(a.dk, a.dv) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || a.lda % 2 || a.ldo % 2) return CB_ERR_SHAPE;
+  if (!cb_linrec_chunk_ok(a.dk, a.dv) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || a.lda % 4 || a.ldo % 4) return CB_ERR_SHAPE;
   if (kind == LINREC_DELTA ? (!a.dec || !a.ring || a.taps < 1 || a.taps > a.ring_mask + 1) : (!a.n || !a.m || !(a.cap > 0.f))) return CB_ERR_ARG;
   if (scratch_bytes < cb_linrec_chunk_scratch(kind, rows, segs, a.H, a.dk, a.dv)) return CB_ERR_ARG;
   unsigned char* p = (unsigned char*)scratch;

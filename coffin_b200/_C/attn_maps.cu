@@ -80,7 +80,7 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
 
 // One warp per (row, head): merge the key splits of every map, o = a_0 - lambda a_1 (two maps), RMS norm over the
 // head's values without weight (two maps), times post_scale, times sigmoid(gate).
-constexpr int kVMax = 16;      // values per lane: vdim <= 512; at most 32 splits
+constexpr int kVMax = 16;      // values per lane: vdim <= 512; at most 64 splits (4 in the warp form)
 template <typename TA>
 __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                           const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
@@ -98,6 +98,24 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
   float o[kVMax];
 #pragma unroll
   for (int i = 0; i < kVMax; ++i) o[i] = 0.f;
+  if (nsplit == 1 && v4 && maps == 2) {                // prompts: everything a lane needs in one round of loads
+    const int64_t vh = (row * H + h) * 2;
+    const float d0 = part_ml[vh * 2 + 1], d1 = part_ml[vh * 2 + 3];
+    const float* po = part_o + vh * vdim;
+    float4 p0[kVMax / 4], p1[kVMax / 4];
+#pragma unroll
+    for (int i = 0; i < kVMax / 4; ++i) {
+      const int v = 4 * (lane + 32 * i);
+      p0[i] = v < vdim ? *reinterpret_cast<const float4*>(po + v) : make_float4(0.f, 0.f, 0.f, 0.f);
+      p1[i] = v < vdim ? *reinterpret_cast<const float4*>(po + vdim + v) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float f0 = 1.f / d0, f1 = -lambda / d1;
+#pragma unroll
+    for (int i = 0; i < kVMax / 4; ++i) {
+      o[4 * i] = fmaf(f1, p1[i].x, f0 * p0[i].x); o[4 * i + 1] = fmaf(f1, p1[i].y, f0 * p0[i].y);
+      o[4 * i + 2] = fmaf(f1, p1[i].z, f0 * p0[i].z); o[4 * i + 3] = fmaf(f1, p1[i].w, f0 * p0[i].w);
+    }
+  } else
   for (int mp = 0; mp < maps; ++mp) {
     const int64_t vh = (row * H + h) * maps + mp;
     const float* ml = part_ml + vh * nsplit * 2;
@@ -172,20 +190,23 @@ __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __re
     const int64_t vh = (row * H + h) * maps + mp;
     const float* ml = part_ml + vh * nsplit * 2;
     const float* po = part_o + vh * nsplit * vdim;
-    float2 v = make_float2(-INFINITY, 0.f);
-    if (lane < nsplit) v = *reinterpret_cast<const float2*>(ml + 2 * lane);
-    const float M = warp_max(v.x);
-    float fac = v.x == -INFINITY ? 0.f : expf(v.x - M);
-    const float den = warp_sum(fac * v.y);
-    fac *= (mp == 0 ? 1.f : -lambda) / den;
-    const int used = __popc(__ballot_sync(0xffffffffu, v.x != -INFINITY));
+    float2 v[2];                                       // splits lane and lane + 32
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      v[k] = lane + 32 * k < nsplit ? *reinterpret_cast<const float2*>(ml + 2 * (lane + 32 * k)) : make_float2(-INFINITY, 0.f);
+    const float M = warp_max(fmaxf(v[0].x, v[1].x));
+    float fac[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) fac[k] = v[k].x == -INFINITY ? 0.f : expf(v[k].x - M);
+    const float den = warp_sum(fac[0] * v[0].y + fac[1] * v[1].y), c = (mp == 0 ? 1.f : -lambda) / den;
+    const int used = __popc(__ballot_sync(0xffffffffu, v[0].x != -INFINITY)) + __popc(__ballot_sync(0xffffffffu, v[1].x != -INFINITY));
 #pragma unroll 4
     for (int s = warp; s < used; s += kWT / 32) {
-      const float f = __shfl_sync(0xffffffffu, fac, s);
+      const float f = c * __shfl_sync(0xffffffffu, s < 32 ? fac[0] : fac[1], s & 31);
 #pragma unroll
       for (int i = 0; i < kVMax; ++i) {
-        const int c = lane + 32 * i;
-        if (c < vdim) o[i] = fmaf(f, po[(int64_t)s * vdim + c], o[i]);
+        const int v_ = lane + 32 * i;
+        if (v_ < vdim) o[i] = fmaf(f, po[(int64_t)s * vdim + v_], o[i]);
       }
     }
   }
@@ -249,9 +270,10 @@ CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const
                                   const void* positions, int64_t rows, int64_t H, int64_t maps, int64_t vdim, int64_t nsplit,
                                   float lambda, float post_scale, float eps, int64_t f32, void* stream) {
   if (!part_o || !part_ml || !act || !positions || rows < 1 || maps < 1 || maps > 2 || nsplit < 1) return CB_ERR_ARG;
-  if (vdim > 32 * kVMax || nsplit > 32) return CB_ERR_SHAPE;
+  if (vdim > 32 * kVMax || nsplit > 64) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
-  if (nsplit > 4 && rows <= 65535) {
+  if (nsplit > 4) {
+    if (rows > 65535) return CB_ERR_SHAPE;
     const size_t smem = sizeof(float) * (size_t)(kWT / 32) * vdim;
     const dim3 wide((unsigned)H, (unsigned)rows);
     if (f32)

@@ -445,7 +445,7 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   if (!args || rows < 1 || rows > 65535) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
-      a.nsplit < 1 || a.nsplit > 32)
+      a.nsplit < 1 || a.nsplit > 64)
     return CB_ERR_ARG;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim)) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;

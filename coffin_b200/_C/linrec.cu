@@ -161,28 +161,50 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
     const TP* pr = prow0 + (int64_t)t * a.ldp;
     float aa = 1.f, bb = 1.f, kq = 0.f, den = 1.f;
     if (KIND == LINREC_DELTA) {
-      auto conv = [&](int64_t ch) {
-        float acc = 0.f;
-        for (int j = 0; j < a.taps; ++j) {
-          const int src = t - (a.taps - 1) + j, p = pos0 + src;
-          float x = 0.f;
-          if (src >= 0) x = act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
-          else if (p >= 0) x = act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch);
-          acc = fmaf(a.conv_w[ch * a.taps + j], x, acc);
-        }
-        return silu_x(acc);
+      // short convolution: channels q, k, v of this CTA spread over the block; up to four taps of two channels are
+      // requested together
+      const int nch = 2 * dk + ncol;
+      auto channel = [&](int e) { return e < dk ? (int64_t)qb + e : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk); };
+      auto tap = [&](int64_t ch, int j) {
+        const int src = t - (a.taps - 1) + j, p = pos0 + src;
+        if (src >= 0) return act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
+        return p >= 0 ? act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch) : 0.f;
       };
+      for (int e0 = tid; e0 < nch; e0 += 2 * kT) {
+        float acc[2] = {0.f, 0.f};
+        const int64_t ch[2] = {channel(e0), e0 + kT < nch ? channel(e0 + kT) : 0};
+        for (int j0_ = 0; j0_ < a.taps; j0_ += 4) {
+          float x[2][4], w[2][4];
+#pragma unroll
+          for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              const bool ok = j0_ + j < a.taps && (u == 0 || e0 + kT < nch);
+              x[u][j] = ok ? tap(ch[u], j0_ + j) : 0.f;
+              w[u][j] = ok ? a.conv_w[ch[u] * a.taps + j0_ + j] : 0.f;
+            }
+#pragma unroll
+          for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[u] = fmaf(w[u][j], x[u][j], acc[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const int e = e0 + u * kT;
+          if (e < nch) (e < 2 * dk ? sq : sv - 2 * dk)[e] = silu_x(acc[u]);     // sq and sk are adjacent
+        }
+      }
       for (int c = tid; c < lown; c += kT) {
         const int na = a.dec ? 0 : (int)a.ra;
         low[c] = act_round<TA>(act_load(pr + (c < na ? a.a1_col + c : a.g1_col + c - na)));
       }
+      bb = sigmoid_x(a.gates[row * a.ldg + h]);            // beta
+      __syncthreads();
       float q2 = 0.f, k2 = 0.f, qk = 0.f;
       for (int c = tid; c < dk; c += kT) {
-        const float qc = conv(qb + c), kc = conv(a.k_col + qb + c);
-        sq[c] = qc; sk[c] = kc;
+        const float qc = sq[c], kc = sk[c];
         q2 = fmaf(qc, qc, q2); k2 = fmaf(kc, kc, k2); qk = fmaf(qc, kc, qk);
       }
-      for (int c = tid; c < ncol; c += kT) sv[c] = conv(a.v_col + (int64_t)h * dv + j0 + c);
       block_sum3(q2, k2, qk, red);
       const float rq = 1.f / (sqrtf(q2 + 1e-6f) * sqrtf((float)dk)), rk = 1.f / sqrtf(k2 + 1e-6f);
       kq = qk * rq * rk;
@@ -197,7 +219,6 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
         const float x = a.dec ? a.dec[row * a.ldd + ch] : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
         sg[c] = expf(-ea * softplus_x(x + a.dt_bias[ch]));
       }
-      bb = sigmoid_x(a.gates[row * a.ldg + h]);            // beta
       const TA* g2 = reinterpret_cast<const TA*>(a.g2);
       const float* lg = low + (a.dec ? 0 : a.ra);
       for (int c = tid; c < ncol; c += kT) {
@@ -274,12 +295,17 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
       }
     }
     __syncthreads();
-    for (int c = tid; c < jc; c += kT) {
+    for (int c4 = tid; c4 < ((4 * jc + 31) & ~31); c4 += kT) {   // four lanes per column
+      const int c = c4 >> 2;
       float b = 0.f, d = 0.f;
-      for (int r = 0; r < RG; ++r) {
-        b += part[r * jc + c];
-        if (KIND == LINREC_DELTA) d += part[(RG + r) * jc + c];
-      }
+      if (c < jc)
+        for (int r = c4 & 3; r < RG; r += 4) {
+          b += part[r * jc + c];
+          if (KIND == LINREC_DELTA) d += part[(RG + r) * jc + c];
+        }
+      b += __shfl_xor_sync(0xffffffffu, b, 1); b += __shfl_xor_sync(0xffffffffu, b, 2);
+      d += __shfl_xor_sync(0xffffffffu, d, 1); d += __shfl_xor_sync(0xffffffffu, d, 2);
+      if ((c4 & 3) || c >= jc) continue;
       if (c >= ncol) b = 0.f;
       if (KIND == LINREC_DELTA) {
         const float u = c < ncol ? bb * (sv[c] - d) : 0.f;

@@ -9,8 +9,8 @@
 //   mLSTM :  u = v and the same with scalar decays under the running maximum; its normaliser n is one more value
 //            column, v = 1.
 //
-// `prep` (one CTA per chunk and head) computes those factors in fp32; `scan` (one warp per 16 value columns) walks the
-// chunks with S^T in accumulator registers.  The 32-bit quantities enter the products as a bf16 head plus a bf16
+// `prep` (one CTA per chunk and head) computes those factors in fp32; `scan` (two warps per 16 value columns) walks
+// the chunks with S^T in accumulator registers.  The 32-bit quantities enter the products as a bf16 head plus a bf16
 // remainder (three products, 16 mantissa bits), the sums and the state are fp32; `finish` applies the head norm and
 // the output gate.  A segment may start and end anywhere: its last chunk is padded with neutral tokens.
 #include "linrec.cuh"
@@ -366,14 +366,19 @@ __global__ void __launch_bounds__(64) chunk_prep_mlstm_kernel(const ChunkArgs ca
 }
 
 // ---- scan ---------------------------------------------------------------------------------------
-template <int KIND, int DK, int WARPS, int STAGES>
-__global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs ca) {
+// A CTA owns 32 value columns of a head: two column groups of 16, each shared by two warps that hold half of the key
+// channels.  The halves' partial read-outs meet in shared memory once per chunk; both then know u and update their half
+// of the state.
+constexpr int kST = 128;
+template <int KIND, int DK, int STAGES>
+__global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
   using I = Image<KIND, DK>;
-  constexpr int P = I::P, NT = DK / 8, NR = I::NX / 8, TH = WARPS * 32;
+  constexpr int P = I::P, NT = DK / 16, NR = I::NX / 8;         // NT: n-tiles (8 channels) of this warp's half
   const LinrecArgs& a = ca.r;
   extern __shared__ __align__(16) unsigned char smem[];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
-  const int h = blockIdx.y, seg = blockIdx.z;
+  __shared__ float xch[4][NR * 4][32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, cg = warp >> 1, half = warp & 1, g4 = lane >> 2, t4 = lane & 3;
+  const int h = blockIdx.y, seg = blockIdx.z, kc = half * (DK / 2);      // first channel of the half
   griddep_launch();
   griddep_wait();
   const int row0 = a.seg_row[seg], n = a.seg_row[seg + 1] - row0, slot = a.seg_slot[seg];
@@ -381,9 +386,10 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
   const int chunks = (n + C - 1) / C;
   // mLSTM: the slice after the value columns carries the normaliser as one column whose value is 1
   const bool nrm = KIND == LINREC_MLSTM && blockIdx.x == gridDim.x - 1;
-  const int v0 = nrm ? 0 : ((int)blockIdx.x * WARPS + warp) * 16;
-  const int vlim = nrm ? (warp == 0 ? 1 : 0) : a.dv;             // columns that exist
+  const int v0 = nrm ? 0 : ((int)blockIdx.x * 2 + cg) * 16;
+  const int vlim = nrm ? (cg == 0 ? 1 : 0) : a.dv;               // columns that exist
   const int va = v0 + g4, vb = va + 8;
+  const bool oka = va < vlim, okb = vb < vlim;
   const int64_t sstride = nrm ? 1 : a.dv;
   float* Sg = nrm ? a.n + ((int64_t)slot * a.H + h) * a.dk : a.S + ((int64_t)slot * a.H + h) * a.dk * a.dv;
   float S[NT][4];
@@ -391,45 +397,63 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
   for (int i = 0; i < NT; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int c = i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
+      const int c = kc + i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
       S[i][e] = c < a.dk && v < vlim ? Sg[(int64_t)c * sstride + v] : 0.f;
     }
-  const unsigned char* img = ca.image + (block_index(row0, seg, 0) * a.H + h) * I::bytes;
+  const unsigned char* img = ca.image + (block_index(row0, seg, 0) * a.H + h) * I::bytes + tid * 16;
   const size_t istep = (size_t)a.H * I::bytes;
-  auto load = [&](int ch) {
+  const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(smem) + tid * 16;
+  auto load = [&](int ch, int stage) {
     const unsigned char* src = img + (size_t)ch * istep;
-    const uint32_t dst = (uint32_t)__cvta_generic_to_shared(smem + (ch % STAGES) * I::bytes);
-    for (int e = tid; e < (int)(I::bytes / 16); e += TH)
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + e * 16), "l"(src + (size_t)e * 16) : "memory");
+    const uint32_t dst = sbase + stage * (uint32_t)I::bytes;
+    constexpr int full = (int)(I::bytes / 16) / kST, rest = (int)(I::bytes / 16) % kST;
+#pragma unroll
+    for (int i = 0; i < full; ++i)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * kST * 16), "l"(src + i * kST * 16) : "memory");
+    if (tid < rest)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + full * kST * 16), "l"(src + full * kST * 16) : "memory");
   };
-  // values of the chunk in accumulator order: [token tile][row lo / hi, token 2t, 2t + 1], as raw bits (nothing is computed
-  // on them here, so that the loads of the next chunk stay in flight)
+  // values of a chunk in accumulator order ([token tile][row lo / hi, token 2t, 2t + 1]) as raw bits: nothing is computed
+  // on them when they are requested, so that the next chunk's loads stay in flight
+  const int64_t ldv = KIND == LINREC_DELTA ? (int64_t)a.H * a.dv : a.ldp;
+  const char* vp = KIND == LINREC_DELTA
+                       ? reinterpret_cast<const char*>(ca.v + (int64_t)(row0 + t4 * 2) * ldv + (int64_t)h * a.dv + va)
+                       : reinterpret_cast<const char*>(reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + t4 * 2) * ldv + a.v_col +
+                                                       (int64_t)h * a.dv + va);
+  constexpr int VS = KIND == LINREC_DELTA ? 4 : 2;
+  const int64_t vstep = ldv * VS;
   auto values = [&](int ch, uint32_t (*v)[4]) {
+    const int left = n - ch * C - t4 * 2;                        // tokens from this lane's first on
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int t = ch * C + i * 8 + t4 * 2 + (e & 1), vv = e >> 1 ? vb : va;
+        const int dt = i * 8 + (e & 1);
         uint32_t x = 0;
-        if (t < n && vv < vlim) {
+        if (dt < left && (e >> 1 ? okb : oka)) {
+          const char* p = vp + dt * vstep + (e >> 1) * 8 * VS;
           if (nrm) x = 0x3f80u;                                  // bf16 one
-          else if (KIND == LINREC_DELTA) x = __float_as_uint(ca.v[(int64_t)(row0 + t) * a.H * a.dv + (int64_t)h * a.dv + vv]);
-          else x = reinterpret_cast<const unsigned short*>(a.proj)[(int64_t)(row0 + t) * a.ldp + a.v_col + (int64_t)h * a.dv + vv];
+          else if (VS == 4) x = *reinterpret_cast<const uint32_t*>(p);
+          else x = *reinterpret_cast<const unsigned short*>(p);
         }
         v[i][e] = x;
       }
+    vp += C * vstep;
   };
+  float* op = nrm ? ca.nq + (int64_t)(row0 + half * 8 + t4 * 2) * a.H + h : ca.o + (int64_t)(row0 + half * 8 + t4 * 2) * ca.ldo_ + (int64_t)h * a.dv + va;
+  const int64_t ostep = nrm ? a.H : ca.ldo_;
 #pragma unroll
   for (int s = 0; s < STAGES - 1; ++s) {
-    if (s < chunks) load(s);
+    if (s < chunks) load(s, s);
     asm volatile("cp.async.commit_group;" ::: "memory");
   }
   uint32_t vn[2][4];
   values(0, vn);
+  int stage = 0;
   for (int ch = 0; ch < chunks; ++ch) {
     asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
     __syncthreads();
-    if (ch + STAGES - 1 < chunks) load(ch + STAGES - 1);
+    if (ch + STAGES - 1 < chunks) load(ch + STAGES - 1, stage == 0 ? STAGES - 1 : stage - 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
     float v[2][4];
 #pragma unroll
@@ -437,13 +461,17 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
 #pragma unroll
       for (int e = 0; e < 4; ++e) v[i][e] = __uint_as_float(KIND == LINREC_DELTA ? vn[i][e] : vn[i][e] << 16);
     if (ch + 1 < chunks) values(ch + 1, vn);
-    const bf16* im = reinterpret_cast<const bf16*>(smem + (ch % STAGES) * I::bytes);
-    const float* G = reinterpret_cast<const float*>(im + I::g);
-    // R^T = S^T X^T
-    float R[NR][4];
+    const bf16* im = reinterpret_cast<const bf16*>(smem + stage * I::bytes);
+    const float* G = reinterpret_cast<const float*>(im + I::g) + kc;
+    stage = stage + 1 == STAGES ? 0 : stage + 1;
+    // R^T = S^T X^T over this half's channels; the cross terms have accumulators of their own (shorter chains)
+    float R[NR][4], R2[NR][4];
 #pragma unroll
-    for (int i = 0; i < NR; ++i) R[i][0] = R[i][1] = R[i][2] = R[i][3] = 0.f;
-    const int xr = ((lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
+    for (int i = 0; i < NR; ++i) {
+      R[i][0] = R[i][1] = R[i][2] = R[i][3] = 0.f;
+      R2[i][0] = R2[i][1] = R2[i][2] = R2[i][3] = 0.f;
+    }
+    const int xr = ((lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8 + kc;
 #pragma unroll
     for (int k = 0; k < NT / 2; ++k) {
       uint32_t ah[4], al[4];
@@ -460,32 +488,39 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
         ldsm4(bl, im + I::xl + j * 16 * P + xr + k * 16);
         mma(R[2 * j], ah, bh[0], bh[1]);
         mma(R[2 * j + 1], ah, bh[2], bh[3]);
-        mma(R[2 * j], al, bh[0], bh[1]);
-        mma(R[2 * j + 1], al, bh[2], bh[3]);
-        mma(R[2 * j], ah, bl[0], bl[1]);
-        mma(R[2 * j + 1], ah, bl[2], bl[3]);
+        mma(R2[2 * j], al, bh[0], bh[1]);
+        mma(R2[2 * j + 1], al, bh[2], bh[3]);
+        mma(R2[2 * j], ah, bl[0], bl[1]);
+        mma(R2[2 * j + 1], ah, bl[2], bl[3]);
       }
     }
+#pragma unroll
+    for (int i = 0; i < NR * 4; ++i) {
+      R[i >> 2][i & 3] += R2[i >> 2][i & 3];
+      xch[warp][i][lane] = R[i >> 2][i & 3];
+    }
+    asm volatile("bar.sync %0, 64;" ::"r"(1 + cg) : "memory");
+#pragma unroll
+    for (int i = 0; i < NR * 4; ++i) R[i >> 2][i & 3] += xch[warp ^ 1][i][lane];
     const int mr = ((lane & 7) + ((lane >> 4) << 3)) * 24 + ((lane >> 3) & 1) * 8;
-    float (*O)[4] = &R[NR - 2];
     uint32_t uh[4], ul[4];
     if (KIND == LINREC_DELTA) {
       uint32_t dh[4], dl[4], bh[4], bl[4];
+      ldsm4(bh, im + I::th + mr);
+      ldsm4(bl, im + I::tl + mr);
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
         float x = v[q >> 1][(q & 1) * 2] - R[q >> 1][(q & 1) * 2], y = v[q >> 1][(q & 1) * 2 + 1] - R[q >> 1][(q & 1) * 2 + 1];
         dh[q] = split_head(x, y);
         dl[q] = pack_bf162(x, y);
       }
-      float U[2][4] = {};
-      ldsm4(bh, im + I::th + mr);
-      ldsm4(bl, im + I::tl + mr);
+      float U[2][4] = {}, U2[2][4] = {};
       mma(U[0], dh, bh[0], bh[1]); mma(U[1], dh, bh[2], bh[3]);
-      mma(U[0], dl, bh[0], bh[1]); mma(U[1], dl, bh[2], bh[3]);
+      mma(U2[0], dl, bh[0], bh[1]); mma(U2[1], dl, bh[2], bh[3]);
       mma(U[0], dh, bl[0], bl[1]); mma(U[1], dh, bl[2], bl[3]);
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
-        float x = U[q >> 1][(q & 1) * 2], y = U[q >> 1][(q & 1) * 2 + 1];
+        float x = U[q >> 1][(q & 1) * 2] + U2[q >> 1][(q & 1) * 2], y = U[q >> 1][(q & 1) * 2 + 1] + U2[q >> 1][(q & 1) * 2 + 1];
         uh[q] = split_head(x, y);
         ul[q] = pack_bf162(x, y);
       }
@@ -496,19 +531,11 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
         ul[q] = 0;
       }
     }
-    {
-      uint32_t bh[4], bl[4];
-      ldsm4(bh, im + I::bh + mr);
-      ldsm4(bl, im + I::bl + mr);
-      mma(O[0], uh, bh[0], bh[1]); mma(O[1], uh, bh[2], bh[3]);
-      mma(O[0], uh, bl[0], bl[1]); mma(O[1], uh, bl[2], bl[3]);
-      if (KIND == LINREC_DELTA) { mma(O[0], ul, bh[0], bh[1]); mma(O[1], ul, bh[2], bh[3]); }
-    }
     // S^T <- G S^T + U^T K^
 #pragma unroll
     for (int k = 0; k < NT / 2; ++k) {
       uint32_t bh[4], bl[4];
-      const int off = (lane & 15) * P + k * 16 + (lane >> 4) * 8;
+      const int off = (lane & 15) * P + kc + k * 16 + (lane >> 4) * 8;
       ldsm4t(bh, im + I::kh + off);
       ldsm4t(bl, im + I::kl + off);
 #pragma unroll
@@ -521,23 +548,30 @@ __global__ void __launch_bounds__(WARPS * 32) chunk_scan_kernel(const ChunkArgs 
         if (KIND == LINREC_DELTA) mma(s, ul, bh[2 * i], bh[2 * i + 1]);
       }
     }
-    // read-outs
+    // read-outs of this half's eight tokens
+    {
+      uint32_t bh[4], bl[4];
+      ldsm4(bh, im + I::bh + mr);
+      ldsm4(bl, im + I::bl + mr);
+      const uint32_t b0 = half ? bh[2] : bh[0], b1 = half ? bh[3] : bh[1], l0 = half ? bl[2] : bl[0], l1 = half ? bl[3] : bl[1];
+      float O[4], O2[4] = {};
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+      for (int e = 0; e < 4; ++e) O[e] = half ? R[NR - 1][e] : R[NR - 2][e];
+      mma(O, uh, b0, b1);
+      mma(O2, uh, l0, l1);
+      if (KIND == LINREC_DELTA) mma(O2, ul, b0, b1);
+      const int left = n - ch * C - half * 8 - t4 * 2;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = ch * C + i * 8 + t4 * 2 + (e & 1), vv = e >> 1 ? vb : va;
-        if (t < n && vv < vlim) {
-          if (nrm) ca.nq[(int64_t)(row0 + t) * a.H + h] = O[i][e];
-          else ca.o[(int64_t)(row0 + t) * ca.ldo_ + (int64_t)h * a.dv + vv] = O[i][e];
-        }
-      }
+      for (int e = 0; e < 4; ++e)
+        if ((e & 1) < left && (e >> 1 ? okb : oka)) op[(e & 1) * ostep + (e >> 1) * 8] = O[e] + O2[e];
+      op += C * ostep;
+    }
   }
 #pragma unroll
   for (int i = 0; i < NT; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int c = i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
+      const int c = kc + i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
       if (c < a.dk && v < vlim) Sg[(int64_t)c * sstride + v] = S[i][e];
     }
 }
@@ -607,13 +641,13 @@ int run_chunks(const ChunkArgs& ca, int max_rows, int rows, cudaStream_t st) {
     e = cb_launch(chunk_prep_mlstm_kernel<DK>, dim3((unsigned)chunks, (unsigned)a.H, (unsigned)ca.segs), dim3(64), smem, st, ca);
     if (e != cudaSuccess) return (int)e;
   }
-  constexpr int WARPS = 2, STAGES = 3;
-  auto scan = chunk_scan_kernel<KIND, DK, WARPS, STAGES>;
+  constexpr int STAGES = 3;
+  auto scan = chunk_scan_kernel<KIND, DK, STAGES>;
   const size_t smem = STAGES * I::bytes;
   e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  const int slices = (a.dv + 16 * WARPS - 1) / (16 * WARPS) + (KIND == LINREC_MLSTM ? 1 : 0);
-  e = cb_launch(scan, dim3((unsigned)slices, (unsigned)a.H, (unsigned)ca.segs), dim3(WARPS * 32), smem, st, ca);
+  const int slices = (a.dv + 31) / 32 + (KIND == LINREC_MLSTM ? 1 : 0);
+  e = cb_launch(scan, dim3((unsigned)slices, (unsigned)a.H, (unsigned)ca.segs), dim3(kST), smem, st, ca);
   if (e != cudaSuccess) return (int)e;
   return (int)cb_launch(chunk_finish_kernel<KIND>, dim3((unsigned)(((int64_t)rows * a.H + 3) / 4)), dim3(128), 0, st, ca, rows);
 }

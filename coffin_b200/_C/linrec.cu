@@ -33,7 +33,7 @@ template <typename TW>
 __device__ __forceinline__ float row_dot(const TW* __restrict__ w, const float* x, int64_t n) {
   float s0 = 0.f, s1 = 0.f;
   int64_t i = 0;
-#pragma unroll 4
+#pragma unroll 1
   for (; i + 8 <= n; i += 8) {
     const float4 a = act_load4(w + i), b = act_load4(w + i + 4);
     s0 = fmaf(a.x, x[i], s0); s0 = fmaf(a.y, x[i + 1], s0); s0 = fmaf(a.z, x[i + 2], s0); s0 = fmaf(a.w, x[i + 3], s0);
@@ -77,6 +77,7 @@ struct LowRank {
 #pragma unroll
     for (int i = 0; i < PRE; ++i)
       if (i < iters) dot_piece(i, w[i], x, out);
+#pragma unroll 1
     for (int i = PRE; i < iters; ++i) dot_piece(i, piece(i), x, out);
   }
 };
@@ -94,7 +95,7 @@ __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* 
 }
 
 template <int KIND, typename TP, typename TA, int RMAX>
-__global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
+__global__ void __launch_bounds__(kT, RMAX <= 8 ? 2 : 1) linrec_step_kernel(const LinrecArgs a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
   __shared__ float cl_part;
@@ -161,39 +162,30 @@ __global__ void __launch_bounds__(kT) linrec_step_kernel(const LinrecArgs a) {
     const TP* pr = prow0 + (int64_t)t * a.ldp;
     float aa = 1.f, bb = 1.f, kq = 0.f, den = 1.f;
     if (KIND == LINREC_DELTA) {
-      // short convolution: channels q, k, v of this CTA spread over the block; up to four taps of two channels are
-      // requested together
+      // short convolution: channels q, k, v of this CTA spread over the block, four taps requested together (in a decode
+      // step all but the newest come from the ring)
       const int nch = 2 * dk + ncol;
-      auto channel = [&](int e) { return e < dk ? (int64_t)qb + e : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk); };
-      auto tap = [&](int64_t ch, int j) {
-        const int src = t - (a.taps - 1) + j, p = pos0 + src;
-        if (src >= 0) return act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
-        return p >= 0 ? act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch) : 0.f;
-      };
-      for (int e0 = tid; e0 < nch; e0 += 2 * kT) {
-        float acc[2] = {0.f, 0.f};
-        const int64_t ch[2] = {channel(e0), e0 + kT < nch ? channel(e0 + kT) : 0};
-        for (int j0_ = 0; j0_ < a.taps; j0_ += 4) {
-          float x[2][4], w[2][4];
+#pragma unroll 1
+      for (int e = tid; e < nch; e += kT) {
+        const int64_t ch = e < dk ? (int64_t)qb + e : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk);
+        float acc = 0.f;
+#pragma unroll 1
+        for (int b = 0; b < a.taps; b += 4) {
+          float x[4], w[4];
 #pragma unroll
-          for (int u = 0; u < 2; ++u)
+          for (int j = 0; j < 4; ++j) {
+            const int src = t - (a.taps - 1) + b + j, p = pos0 + src;
+            const bool ok = b + j < a.taps && p >= 0;
+            w[j] = ok ? a.conv_w[ch * a.taps + b + j] : 0.f;
+            x[j] = ok && src < 0 ? act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch) : 0.f;
+            if (ok && src >= 0) x[j] = act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
+          }
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const bool ok = j0_ + j < a.taps && (u == 0 || e0 + kT < nch);
-              x[u][j] = ok ? tap(ch[u], j0_ + j) : 0.f;
-              w[u][j] = ok ? a.conv_w[ch[u] * a.taps + j0_ + j] : 0.f;
-            }
-#pragma unroll
-          for (int u = 0; u < 2; ++u)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) acc[u] = fmaf(w[u][j], x[u][j], acc[u]);
+          for (int j = 0; j < 4; ++j) acc = fmaf(w[j], x[j], acc);
         }
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          const int e = e0 + u * kT;
-          if (e < nch) (e < 2 * dk ? sq : sv - 2 * dk)[e] = silu_x(acc[u]);     // sq and sk are adjacent
-        }
+        (e < 2 * dk ? sq : sv - 2 * dk)[e] = silu_x(acc);        // sq and sk are adjacent
       }
+#pragma unroll 1
       for (int c = tid; c < lown; c += kT) {
         const int na = a.dec ? 0 : (int)a.ra;
         low[c] = act_round<TA>(act_load(pr + (c < na ? a.a1_col + c : a.g1_col + c - na)));

@@ -413,54 +413,52 @@ __global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
     if (tid < rest)
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + full * kST * 16), "l"(src + full * kST * 16) : "memory");
   };
-  // values of a chunk in accumulator order ([token tile][row lo / hi, token 2t, 2t + 1]) as raw bits: nothing is computed
-  // on them when they are requested, so that the next chunk's loads stay in flight
+  // values of a chunk go through the same ring: [token][32 columns], pitch chosen against bank conflicts
+  constexpr int VE = KIND == LINREC_DELTA ? 4 : 2, VP = KIND == LINREC_DELTA ? 36 : 40, VB = C * VP * VE, VPER = 32 * VE / 16;   // 16-byte pieces a row
   const int64_t ldv = KIND == LINREC_DELTA ? (int64_t)a.H * a.dv : a.ldp;
-  const char* vp = KIND == LINREC_DELTA
-                       ? reinterpret_cast<const char*>(ca.v + (int64_t)(row0 + t4 * 2) * ldv + (int64_t)h * a.dv + va)
-                       : reinterpret_cast<const char*>(reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + t4 * 2) * ldv + a.v_col +
-                                                       (int64_t)h * a.dv + va);
-  constexpr int VS = KIND == LINREC_DELTA ? 4 : 2;
-  const int64_t vstep = ldv * VS;
-  auto values = [&](int ch, uint32_t (*v)[4]) {
-    const int left = n - ch * C - t4 * 2;                        // tokens from this lane's first on
-#pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int dt = i * 8 + (e & 1);
-        uint32_t x = 0;
-        if (dt < left && (e >> 1 ? okb : oka)) {
-          const char* p = vp + dt * vstep + (e >> 1) * 8 * VS;
-          if (nrm) x = 0x3f80u;                                  // bf16 one
-          else if (VS == 4) x = *reinterpret_cast<const uint32_t*>(p);
-          else x = *reinterpret_cast<const unsigned short*>(p);
-        }
-        v[i][e] = x;
-      }
-    vp += C * vstep;
+  const int vt = tid / VPER, vc = (int)blockIdx.x * 32 + (tid % VPER) * (16 / VE);          // token and first column this thread copies
+  const char* vsrc = KIND == LINREC_DELTA
+                         ? reinterpret_cast<const char*>(ca.v + (int64_t)(row0 + vt) * ldv + (int64_t)h * a.dv + vc)
+                         : reinterpret_cast<const char*>(reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + vt) * ldv + a.v_col +
+                                                         (int64_t)h * a.dv + vc);
+  const uint32_t vdst = (uint32_t)__cvta_generic_to_shared(smem) + STAGES * (uint32_t)I::bytes + vt * VP * VE + (tid % VPER) * 16;
+  auto load_v = [&](int ch, int stage) {
+    if (nrm || vt >= C) return;
+    const bool ok = ch * C + vt < n && vc < a.dv;                // 16-byte pieces never straddle dv (a multiple of 8)
+    const char* src = ok ? vsrc + (int64_t)ch * C * ldv * VE : reinterpret_cast<const char*>(a.proj);
+    const int bytes = ok ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vdst + stage * VB), "l"(src), "r"(bytes) : "memory");
   };
   float* op = nrm ? ca.nq + (int64_t)(row0 + half * 8 + t4 * 2) * a.H + h : ca.o + (int64_t)(row0 + half * 8 + t4 * 2) * ca.ldo_ + (int64_t)h * a.dv + va;
   const int64_t ostep = nrm ? a.H : ca.ldo_;
 #pragma unroll
   for (int s = 0; s < STAGES - 1; ++s) {
-    if (s < chunks) load(s, s);
+    if (s < chunks) { load(s, s); load_v(s, s); }
     asm volatile("cp.async.commit_group;" ::: "memory");
   }
-  uint32_t vn[2][4];
-  values(0, vn);
   int stage = 0;
   for (int ch = 0; ch < chunks; ++ch) {
     asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
     __syncthreads();
-    if (ch + STAGES - 1 < chunks) load(ch + STAGES - 1, stage == 0 ? STAGES - 1 : stage - 1);
+    if (ch + STAGES - 1 < chunks) {
+      const int fs = stage == 0 ? STAGES - 1 : stage - 1;
+      load(ch + STAGES - 1, fs);
+      load_v(ch + STAGES - 1, fs);
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
-    float v[2][4];
+    float v[2][4];                                               // [token tile][row lo / hi, token 2t, 2t + 1]
+    {
+      const unsigned char* vs = smem + STAGES * I::bytes + stage * VB;
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[i][e] = __uint_as_float(KIND == LINREC_DELTA ? vn[i][e] : vn[i][e] << 16);
-    if (ch + 1 < chunks) values(ch + 1, vn);
+        for (int e = 0; e < 4; ++e) {
+          const int idx = (i * 8 + t4 * 2 + (e & 1)) * VP + cg * 16 + g4 + (e >> 1) * 8;
+          if (nrm) v[i][e] = cg == 0 && g4 == 0 && e < 2 ? 1.f : 0.f;
+          else if (KIND == LINREC_DELTA) v[i][e] = reinterpret_cast<const float*>(vs)[idx];
+          else v[i][e] = __bfloat162float(reinterpret_cast<const bf16*>(vs)[idx]);
+        }
+    }
     const bf16* im = reinterpret_cast<const bf16*>(smem + stage * I::bytes);
     const float* G = reinterpret_cast<const float*>(im + I::g) + kc;
     stage = stage + 1 == STAGES ? 0 : stage + 1;
@@ -641,9 +639,9 @@ int run_chunks(const ChunkArgs& ca, int max_rows, int rows, cudaStream_t st) {
     e = cb_launch(chunk_prep_mlstm_kernel<DK>, dim3((unsigned)chunks, (unsigned)a.H, (unsigned)ca.segs), dim3(64), smem, st, ca);
     if (e != cudaSuccess) return (int)e;
   }
-  constexpr int STAGES = 3;
+  constexpr int STAGES = DK <= 128 ? 4 : 3;
   auto scan = chunk_scan_kernel<KIND, DK, STAGES>;
-  const size_t smem = STAGES * I::bytes;
+  const size_t smem = STAGES * (I::bytes + C * (KIND == LINREC_DELTA ? 36 * 4 : 40 * 2));
   e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const int slices = (a.dv + 31) / 32 + (KIND == LINREC_MLSTM ? 1 : 0);

@@ -1,0 +1,380 @@
+// Prompt attention with several score maps per head (attn_maps.cuh) on the 5th-generation tensor cores.
+//
+// One CTA owns 128 consecutive query rows of one (head, map) of a segment and walks the sequence's pages (64 keys) up
+// to the diagonal, with the division of labour of attn_tc.cu: a TMA warp fills rings of key and value pages, two
+// threads issue S_j = Q K_j^T (Q in tensor memory) and O += P_j V_j, eight warps do the softmax, two threads per row.
+// What differs: key and value sizes are independent; scores take a per-row query temperature and an optional cap
+// (cap * tanh(score / cap), evaluated through one exponential); the weights keep 32-bit meaning across the second
+// product, P = bf16 head + bf16 remainder, two products per page; the result leaves as unnormalised fp32 sums with
+// (reference maximum, denominator), which maps_finish_kernel combines across the maps.
+//
+// With a cap the scores are bounded, so the reference maximum is the cap itself (when 2^-2cap is far from underflow):
+// no row maximum, no exchange between the halves of a row, no rescale.  Otherwise the reference is raised lazily as in
+// attn_tc.cu.  Waits are bounded by 2 s and report through the status word; TMEM is freed on every path.
+#include "attn_maps.cuh"
+#include "sm100.cuh"
+
+namespace {
+using namespace sm100;
+
+constexpr int kBQ = 128, kBKV = 64, kThreads = 352;
+constexpr float kLog2e = 1.4426950408889634f;
+enum Mode : int { PLAIN = 0, CAP = 1, CAP_FIXED = 2 };
+
+__device__ __forceinline__ uint64_t now_ns() {
+  uint64_t t;
+  asm volatile("mov.u64 %0, %globaltimer;" : "=l"(t));
+  return t;
+}
+__device__ __forceinline__ bool wait_bar(uint64_t* bar, uint32_t parity, volatile int* abort_flag) {
+  if (mbar_try(bar, parity)) return true;
+  const uint64_t t0 = now_ns();
+  for (;;) {
+    for (int i = 0; i < 128; ++i)
+      if (mbar_try(bar, parity)) return true;
+    if (*abort_flag) return false;
+    if (now_ns() - t0 > 2000000000ull) return false;
+  }
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int DK, int DV, int MODE, int STAGES>
+__global__ void __launch_bounds__(kThreads, 1)
+maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnMapsArgs a, int* status) {
+  constexpr int NK = DK / 64, NV = DV / 64;           // 64-element (128-byte) chunks
+  constexpr int K_BYTES = kBKV * DK * 2, V_BYTES = kBKV * DV * 2, P_BYTES = kBQ * kBKV * 2;
+  constexpr int KC = kBKV * 128;                      // bytes of one chunk block of a page
+  constexpr uint32_t TMEM_COLS = 2 * kBKV + DV + DK / 2 <= 256 ? 256 : 512;
+  static_assert(2 * kBKV + DV + DK / 2 <= 512, "tensor memory");
+  constexpr uint32_t IDESC_S = umma_idesc(kBQ, kBKV, 1, 1);
+  constexpr uint32_t IDESC_O = umma_idesc(kBQ, DV, 1, 1) | (1u << 16);     // B operand MN-major
+  extern __shared__ __align__(1024) unsigned char smem_raw[];
+  unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  unsigned char* Ks = base;                           // [STAGES][K_BYTES]
+  unsigned char* Vs = Ks + STAGES * K_BYTES;          // [STAGES][V_BYTES]
+  unsigned char* Ps = Vs + STAGES * V_BYTES;          // [2][head | remainder]
+  __shared__ uint64_t q_full, k_full[STAGES], v_full[STAGES], k_free[STAGES], v_free[STAGES], s_full[2], s_free[2], p_full[2], p_free[2],
+      o_full, pair_bar[4];
+  __shared__ float xch[2][2][kBQ];                    // [tile parity][column half][row]: maxima of half rows
+  __shared__ uint32_t tmem_base_s;
+  __shared__ int abort_s;
+  volatile int* abort_flag = &abort_s;
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int qt = (int)gridDim.x - 1 - (int)blockIdx.x, vh = blockIdx.y, seg = blockIdx.z;    // long tiles first
+  const int h = vh / a.maps, kh = h / (a.H / a.G), kmap = kh * a.maps + vh % a.maps;
+  griddep_launch();
+  griddep_wait();
+  const int seg0 = a.seg_row[seg], n = a.seg_row[seg + 1] - seg0, pos0 = a.seg_pos[seg];
+  const int row0 = qt * kBQ;
+  if (row0 >= n) return;                              // the whole CTA, before anything is allocated
+  const int n_tiles = (pos0 + min(n, row0 + kBQ) - 1) / kBKV + 1;
+
+  if (threadIdx.x == 0) {
+    mbar_init(&q_full, 8);
+    mbar_init(&o_full, 1);
+    for (int i = 0; i < STAGES; ++i) {
+      mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&k_free[i], 1); mbar_init(&v_free[i], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_full[i], 1); mbar_init(&s_free[i], 8); mbar_init(&p_full[i], 8); mbar_init(&p_free[i], 1);
+    }
+    for (int i = 0; i < 4; ++i) mbar_init(&pair_bar[i], 64);
+    abort_s = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) {
+    tmem_alloc(&tmem_base_s, TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = tmem_base_s;
+  const uint32_t tmem_o = tmem_base + 2 * kBKV;       // S0 | S1 | O | Q
+  const uint32_t tmem_q = tmem_o + DV;
+
+  if (warp == 0) {
+    // ------------------------------------ TMA producer ------------------------------------------
+    if (lane == 0) {
+      const int* bt = a.tables + (int64_t)seg * a.ldbt;
+      for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
+        const int s = j % STAGES;
+        const uint32_t ph = (j / STAGES) & 1;
+        const int slot0 = bt[j] * kBKV;
+        if (!wait_bar(&k_free[s], ph ^ 1, abort_flag)) { atomicCAS(status, 0, 81); abort_s = 1; break; }
+        mbar_expect_tx(&k_full[s], K_BYTES);
+        for (int c = 0; c < NK; ++c) tma_load_2d(Ks + s * K_BYTES + c * KC, &tmK, &k_full[s], kmap * DK + c * 64, slot0);
+        if (!wait_bar(&v_free[s], ph ^ 1, abort_flag)) { atomicCAS(status, 0, 82); abort_s = 1; break; }
+        mbar_expect_tx(&v_full[s], V_BYTES);
+        for (int c = 0; c < NV; ++c) tma_load_2d(Vs + s * V_BYTES + c * KC, &tmV, &v_full[s], kh * DV + c * 64, slot0);
+      }
+    }
+  } else if (warp == 1) {
+    // ------------------------------------ MMA issuer: S_j = Q K_j^T -----------------------------
+    if (lane == 0) {
+      const bool ok = wait_bar(&q_full, 0, abort_flag);
+      if (!ok) { atomicCAS(status, 0, 83); abort_s = 1; }
+      tc_fence_after();
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        const int s = j % STAGES, sb = j & 1;
+        if (!wait_bar(&k_full[s], (j / STAGES) & 1, abort_flag)) { atomicCAS(status, 0, 84); abort_s = 1; break; }
+        if (!wait_bar(&s_free[sb], ((j >> 1) & 1) ^ 1, abort_flag)) { atomicCAS(status, 0, 85); abort_s = 1; break; }
+        tc_fence_after();
+#pragma unroll
+        for (int c = 0; c < NK; ++c) {
+          const uint64_t kd = umma_desc_sw128(Ks + s * K_BYTES + c * KC);
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            umma_f16_ta(tmem_base + sb * kBKV, tmem_q + c * 32 + k * 8, kd + 2 * k, IDESC_S, (c | k) != 0);
+        }
+        umma_commit(&k_free[s]);
+        umma_commit(&s_full[sb]);
+      }
+    }
+  } else if (warp == 10) {
+    // ------------------------------------ MMA issuer: O += P_j V_j ------------------------------
+    if (lane == 0) {
+      bool ok = true;
+      for (int j = 0; j < n_tiles; ++j) {
+        const int s = j % STAGES, sb = j & 1;
+        if (!wait_bar(&p_full[sb], (j >> 1) & 1, abort_flag)) { atomicCAS(status, 0, 86); abort_s = 1; ok = false; break; }
+        if (!wait_bar(&v_full[s], (j / STAGES) & 1, abort_flag)) { atomicCAS(status, 0, 87); abort_s = 1; ok = false; break; }
+        tc_fence_after();
+        const uint64_t pd = umma_desc_sw128(Ps + sb * 2 * P_BYTES), rd = umma_desc_sw128(Ps + sb * 2 * P_BYTES + P_BYTES);
+        const uint64_t vd = umma_desc_mn_sw128(Vs + s * V_BYTES, KC);
+#pragma unroll
+        for (int k = 0; k < 4; ++k)      // 16 keys per instruction: +32 bytes along P's rows, +16 rows of V
+          umma_f16(tmem_o, pd + 2 * k, vd + (uint64_t)(k * 16 * 128 >> 4), IDESC_O, (j | k) != 0);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) umma_f16(tmem_o, rd + 2 * k, vd + (uint64_t)(k * 16 * 128 >> 4), IDESC_O, 1);
+        umma_commit(&v_free[s]);
+        umma_commit(&p_free[sb]);
+      }
+      if (ok) umma_commit(&o_full);
+    }
+  } else {
+    // ------------------------------------ softmax + epilogue ------------------------------------
+    const int q = warp & 3, hf = (warp - 2) >> 2;      // TMEM lane quadrant, half of the row's columns
+    const int r = q * 32 + lane;
+    const int t = row0 + r, pos = pos0 + t;
+    const uint32_t lane_base = (uint32_t)(q * 32) << 16;
+    {
+      const bf16* qrow = reinterpret_cast<const bf16*>(a.proj) + (int64_t)(seg0 + min(t, n - 1)) * a.ldp + (int64_t)vh * DK;
+#pragma unroll 1
+      for (int i = hf; i < NK; i += 2) {
+        uint32_t w[32];
+#pragma unroll
+        for (int v = 0; v < 8; ++v) {
+          const uint4 x = *reinterpret_cast<const uint4*>(qrow + i * 64 + v * 8);
+          w[4 * v] = x.x; w[4 * v + 1] = x.y; w[4 * v + 2] = x.z; w[4 * v + 3] = x.w;
+        }
+        tmem_st32(tmem_q + lane_base + i * 32, w);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&q_full);
+    }
+    // score -> log2 units; with a cap first to the exponent of exp(2 score / cap)
+    const float f = a.scale * query_temp(a, min(pos, pos0 + n - 1)) * (MODE == PLAIN ? kLog2e : 2.f * kLog2e / a.cap);
+    const float cap2 = a.cap * kLog2e;
+    float m_ref = MODE == CAP_FIXED ? cap2 : -INFINITY, l = 0.f;
+    bool ok = true;
+    uint32_t xph = 0;
+    for (int j = 0; j < n_tiles; ++j) {
+      const int sb = j & 1;
+      if (!wait_bar(&s_full[sb], (j >> 1) & 1, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 88); abort_s = 1; } ok = false; break; }
+      tc_fence_after();
+      uint32_t sv[32];
+      tmem_ld32(tmem_base + lane_base + sb * kBKV + hf * 32, sv);
+      tmem_ld_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&s_free[sb]);
+      const int key0 = j * kBKV + hf * 32;
+      const bool edge = j * kBKV + kBKV - 1 > pos0 + row0;       // the page touches the diagonal
+      if (MODE == CAP_FIXED) {
+        // 2^(log2e (cap tanh - cap)) = 2^(-2 cap log2e / (exp(2 s / cap) + 1))
+#pragma unroll
+        for (int c = 0; c < 32; ++c) {
+          float p = ex2(-2.f * cap2 * rcp(ex2(__uint_as_float(sv[c]) * f) + 1.f));
+          if (edge && key0 + c > pos) p = 0.f;
+          sv[c] = __float_as_uint(p);
+        }
+      } else {
+        float mx = -INFINITY;
+#pragma unroll
+        for (int c = 0; c < 32; ++c) {
+          float x = __uint_as_float(sv[c]) * f;
+          if (MODE == CAP) x = cap2 - 2.f * cap2 * rcp(ex2(x) + 1.f);
+          if (edge && key0 + c > pos) x = -INFINITY;
+          sv[c] = __float_as_uint(x);
+          mx = fmaxf(mx, x);
+        }
+        xch[sb][hf][r] = mx;
+        mbar_arrive(&pair_bar[q]);
+        if (!wait_bar(&pair_bar[q], xph, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 92); abort_s = 1; } ok = false; break; }
+        xph ^= 1;
+        mx = fmaxf(xch[sb][0][r], xch[sb][1][r]);
+        if (j == 0) {
+          m_ref = mx;                                  // key 0 is visible to every row: finite
+        } else if (__any_sync(0xffffffffu, mx > m_ref + 8.f)) {
+          // every product that wrote O has to be complete before its rows are rescaled
+          if (!wait_bar(&p_free[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag)) {
+            if (lane == 0) { atomicCAS(status, 0, 89); abort_s = 1; }
+            ok = false;
+            break;
+          }
+          tc_fence_after();
+          const float m_new = fmaxf(m_ref, mx), w = ex2(m_ref - m_new);
+          m_ref = m_new;
+          l *= w;
+#pragma unroll 1
+          for (int c0 = hf * (DV / 2); c0 < (hf + 1) * (DV / 2); c0 += 32) {
+            uint32_t o[32];
+            tmem_ld32(tmem_o + lane_base + c0, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * w);
+            tmem_st32(tmem_o + lane_base + c0, o);
+          }
+          tmem_st_wait();
+          tc_fence_before();
+        }
+#pragma unroll
+        for (int c = 0; c < 32; ++c) sv[c] = __float_as_uint(ex2(__uint_as_float(sv[c]) - m_ref));
+      }
+      // head and remainder of the weights
+      uint32_t ph[16], pr[16];
+      float l0 = 0.f, l1 = 0.f;
+#pragma unroll
+      for (int c = 0; c < 16; ++c) {
+        float x = __uint_as_float(sv[2 * c]), y = __uint_as_float(sv[2 * c + 1]);
+        l0 += x; l1 += y;
+        ph[c] = pack_bf162(x, y);
+        x -= __uint_as_float(ph[c] << 16);
+        y -= __uint_as_float(ph[c] & 0xffff0000u);
+        pr[c] = pack_bf162(x, y);
+      }
+      l += l0 + l1;
+      if (j >= 2 && !wait_bar(&p_free[sb], ((j - 2) >> 1) & 1, abort_flag)) {   // the product of tile j - 2 has read this buffer
+        if (lane == 0) { atomicCAS(status, 0, 90); abort_s = 1; }
+        ok = false;
+        break;
+      }
+      unsigned char* prow = Ps + sb * 2 * P_BYTES + r * 128;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {                    // 16-byte chunk c of row r lives at chunk c ^ (r % 8)
+        const int at = ((hf * 4 + c) ^ (r & 7)) << 4;
+        *reinterpret_cast<uint4*>(prow + at) = make_uint4(ph[4 * c], ph[4 * c + 1], ph[4 * c + 2], ph[4 * c + 3]);
+        *reinterpret_cast<uint4*>(prow + P_BYTES + at) = make_uint4(pr[4 * c], pr[4 * c + 1], pr[4 * c + 2], pr[4 * c + 3]);
+      }
+      fence_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[sb]);
+    }
+    if (ok && !wait_bar(&o_full, 0, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 91); abort_s = 1; } ok = false; }
+    if (ok) {                                          // the halves of a row add their sums through the idle P buffer
+      float* lx = reinterpret_cast<float*>(Ps);
+      lx[hf * kBQ + r] = l;
+      mbar_arrive(&pair_bar[q]);
+      if (!wait_bar(&pair_bar[q], xph, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 93); abort_s = 1; } ok = false; }
+      else l = lx[r] + lx[kBQ + r];
+    }
+    if (ok) {
+      tc_fence_after();
+      const int64_t idx = ((int64_t)(seg0 + t) * a.H * a.maps + vh) * a.nsplit;
+      float* op = a.part_o + idx * DV;
+#pragma unroll 1
+      for (int c0 = hf * (DV / 2); c0 < (hf + 1) * (DV / 2); c0 += 32) {
+        uint32_t o[32];
+        tmem_ld32(tmem_o + lane_base + c0, o);         // warp-collective: rows beyond the segment load too
+        tmem_ld_wait();
+        if (t < n) {
+#pragma unroll
+          for (int v = 0; v < 8; ++v)
+            *reinterpret_cast<uint4*>(op + c0 + v * 4) = make_uint4(o[4 * v], o[4 * v + 1], o[4 * v + 2], o[4 * v + 3]);
+        }
+      }
+      if (t < n && hf == 0) {
+        a.part_ml[idx * 2] = m_ref * (1.f / kLog2e);
+        a.part_ml[idx * 2 + 1] = l;
+        for (int s = 1; s < a.nsplit; ++s) a.part_ml[(idx + s) * 2] = -INFINITY;
+      }
+    }
+  }
+  // ------------------------------------ teardown --------------------------------------------------
+  tc_fence_before();
+  __syncthreads();
+  if (abort_s) {  // give copies still in flight time to land before the shared memory is released
+    const uint64_t t0 = now_ns();
+    while (now_ns() - t0 < 2000000ull) __nanosleep(1000);
+  }
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, TMEM_COLS);
+  }
+}
+
+template <int DK, int DV, int MODE>
+int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
+  constexpr int STAGES = DK + DV > 384 ? 2 : 3;
+  const size_t smem = (size_t)STAGES * kBKV * (DK + DV) * 2 + 4 * (size_t)kBQ * kBKV * 2 + 1024;
+  auto kern = maps_tc_kernel<DK, DV, MODE, STAGES>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  const dim3 grid((unsigned)tiles, (unsigned)(a.H * a.maps), (unsigned)segs);
+  return (int)cb_launch(kern, grid, dim3(kThreads), smem, st, tmK, tmV, a, status);
+}
+template <int DK, int DV>
+int mode_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
+  if (!(a.cap > 0.f)) return launch_tc<DK, DV, PLAIN>(tmK, tmV, a, tiles, segs, status, st);
+  // 2^(-2 cap log2e) well inside the range of fp32 and of a bf16 remainder 2^-16 below it
+  if (a.cap <= 30.f) return launch_tc<DK, DV, CAP_FIXED>(tmK, tmV, a, tiles, segs, status, st);
+  return launch_tc<DK, DV, CAP>(tmK, tmV, a, tiles, segs, status, st);
+}
+
+}  // namespace
+
+// Whether cb_attn_maps_flash_tc takes these head sizes.
+CB_EXPORT int cb_attn_maps_flash_tc_ok(int64_t dim, int64_t vdim) {
+  return (dim == 64 || dim == 128 || dim == 256) && (vdim == 64 || vdim == 128 || vdim == 256);
+}
+
+// Prompt attention of `segs` segments of at most `max_rows` rows: the contract of cb_attn_maps_flash, on tcgen05.
+// `slots`: rows of the pools.
+CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_rows, int64_t slots, void* status, void* stream) {
+  if (!args || segs < 1 || segs > 65535 || max_rows < 1 || !status) return CB_ERR_ARG;
+  const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
+  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
+      a.maps < 1)
+    return CB_ERR_ARG;
+  if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || a.ldp % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
+  CUtensorMap tmK, tmV;
+  const uint64_t kw = (uint64_t)a.G * a.maps * a.dim, vw = (uint64_t)a.G * a.vdim;
+  int rc = cb_make_tmap_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kpool, (uint64_t)slots, kw, kw, kBKV, 64);
+  if (rc) return rc;
+  rc = cb_make_tmap_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.vpool, (uint64_t)slots, vw, vw, kBKV, 64);
+  if (rc) return rc;
+  const int tiles = (int)((max_rows + kBQ - 1) / kBQ);
+  int* st_word = (int*)status;
+  cudaStream_t st = (cudaStream_t)stream;
+#define CB_TC(K, V) \
+  if (a.dim == K && a.vdim == V) return mode_tc<K, V>(tmK, tmV, a, tiles, (int)segs, st_word, st)
+  CB_TC(64, 64); CB_TC(64, 128); CB_TC(64, 256); CB_TC(128, 64); CB_TC(128, 128); CB_TC(128, 256); CB_TC(256, 64); CB_TC(256, 128);
+  CB_TC(256, 256);
+#undef CB_TC
+  return CB_ERR_SHAPE;
+}

@@ -200,6 +200,7 @@ class AttnMaps:
         self.kpool, self.vpool, self.H, self.G, self.maps, self.dim, self.vdim = kpool, vpool, H, G, maps, dim, vdim
         a.H, a.G, a.maps, a.dim, a.vdim, a.k_col, a.v_col = H, G, maps, dim, vdim, k_col, v_col
         a.kpool, a.vpool, a.scale, a.cap = _ptr(kpool), _ptr(vpool), float(scale), float(cap or 0.0)
+        self._tcgen05 = bool(_lib.call_nostream("attn_maps_flash_tc_ok", dim, vdim))
         if temp is not None:
             a.temp_coef, a.temp_every = float(temp[0]), int(temp[1])
 
@@ -226,9 +227,13 @@ class AttnMaps:
         return self.kpool.dtype == torch.bfloat16 and bool(_lib.call_nostream("attn_maps_tc_ok", self.G, self.maps, self.dim, self.vdim))
 
     def flash(self, proj, tables, seg_row, seg_pos, part_o, part_ml, *, segs: int, max_rows: int, positions) -> None:
-        """Portions of several tokens (bf16 projection rows; keys and values appended before)."""
+        """Portions of several tokens (bf16 projection rows; keys and values appended before): tcgen05 for head sizes of
+        64 / 128 / 256 and portions worth a 128-row tile, ``mma.sync`` otherwise."""
         self._fill(proj, tables, positions, None, part_o, part_ml, 1, seg_row, seg_pos)
-        call("attn_maps_flash", ctypes.byref(self.a), segs, max_rows)
+        if K.ATTN_TC and max_rows >= K.ATTN_TC_MIN_T and self._tcgen05:
+            call("attn_maps_flash_tc", ctypes.byref(self.a), segs, max_rows, self.kpool.shape[0], K.status_word(proj.device))
+        else:
+            call("attn_maps_flash", ctypes.byref(self.a), segs, max_rows)
         K._count()
 
     def decode_splits(self, rows: int) -> int:

@@ -155,6 +155,26 @@ def test_mixer_in_portions(name, dtype, cuts):
     assert worst < 8 * TOL[dtype], worst
 
 
+@pytest.mark.parametrize("sizes", [(64, 64), (128, 256), (64, 128), (256, 64), (256, 256), (32, 64), (40, 96)])
+@pytest.mark.parametrize("cap", [None, 20.0, 60.0])
+def test_prompt_attention_kernels_agree(sizes, cap):
+    """tcgen05 (sizes of 64 / 128 / 256), mma.sync and the plain equations on prompts and long portions; peaky scores,
+    so that the uncapped form raises its reference maximum again and again."""
+    from coffin_b200.ops import kernels as K
+    d, e = sizes
+    layer = Z.attention(3, 1, d, e, scale=4.0 * d ** -0.5, softcap=cap, every=100)
+    for cuts in ([333], [130, 203]):
+        got, ref = mixer_pair(layer, BF16, 333, cuts, seed=d + e)
+        assert rel(got, ref) < TOL[BF16], (cuts, rel(got, ref))
+    K.check_status()
+    was, K.ATTN_TC = K.ATTN_TC, False
+    try:
+        other, _ = mixer_pair(layer, BF16, 333, [130, 203], seed=d + e)
+    finally:
+        K.ATTN_TC = was
+    assert rel(got, other) < 3e-3 and max(rel(got[i:i + 1], other[i:i + 1]) for i in range(0, 333, 7)) < 3e-2
+
+
 @pytest.mark.parametrize("bias", [-12.0, 12.0])
 def test_mlstm_running_maximum_starts_at_zero(bias):
     """With input gates far below (above) zero the denominator's exp(-m) decides the first tokens."""

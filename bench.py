@@ -117,6 +117,9 @@ def main() -> None:
     ap.add_argument("--mma-kcta", type=int, default=0, help="tuning: max CTAs sharing one 16-row GEMV block (1 = off)")
     ap.add_argument("--mma-prefetch", type=int, default=-1, help="tuning: GEMV sweep rounds prefetched into L2 before the dependency wait")
     ap.add_argument("--gemv-impl", default="", help="tuning: mma | scalar")
+    ap.add_argument("--beside", default="", choices=["", "zufilorn-1b", "zufilorn-4b"],
+                    help="instead of the headline workload: this model and the Qwen3.5 hybrid of the same width, heads, layers and "
+                         "vocabulary, prefill and decode throughput at a few sizes")
     ap.add_argument("--layers", type=int, default=0, help="Qwen4-exp: cut the geometry to its first N layers")
     ap.add_argument("--no-parity", action="store_true", help="multi-rank runs: skip the comparison with an unsharded copy on rank 0")
     ap.add_argument("--no-stream-gemv", action="store_true", help="tuning: register-staged GEMV for batch 1")
@@ -168,6 +171,8 @@ def main() -> None:
     if args.gemv_ctas or args.gemv_prefetch >= 0:
         from coffin_b200.ops import _lib
         _lib.call_nostream("set_gemv_opts", args.gemv_ctas or 2, 1 if args.gemv_prefetch != 0 else 0)
+    if args.beside:
+        return bench_beside(args, W)
     cfg = preset(args.model)
     if "qwen4" in args.model:
         return bench_qwen4(args, cfg, W)
@@ -417,6 +422,84 @@ def bench_qwen4(args, cfg, W: int) -> None:
                       "timing": "CUDA events; the decode loop reads every token back (eager step, host-staged rows)"},
             "clocks": clocks, "gpu_launches": launches, "impl": "ours"}
     print(json.dumps(line), flush=True)
+
+
+def bench_beside(args, W: int) -> None:
+    """Throughput of a Zufilorn shape beside the Qwen3.5 hybrid of equal size (both random-init bf16): prefill of one
+    prompt and CUDA-graph decode of 1, 8 and 32 sequences, device-timed with events over ``--steps`` repetitions after
+    ``--warmup`` untimed ones.  One JSON line."""
+    import dataclasses
+    import torch
+    from coffin_b200.config import _pattern, preset
+    from coffin_b200.engine.llm import LLM
+    from coffin_b200.ops import kernels as K
+    torch.cuda.set_device(0)
+    new = preset(args.beside)
+    old = preset("qwen35-4b")
+    if args.beside != "zufilorn-4b":                          # the same proportions at this width
+        f = 2560 // new.hidden_size
+        old = dataclasses.replace(old, name=f"qwen35 at width {new.hidden_size}", vocab_size=new.vocab_size, hidden_size=new.hidden_size,
+                                  num_hidden_layers=new.num_hidden_layers, layer_types=_pattern(new.num_hidden_layers),
+                                  num_attention_heads=16 // f, num_key_value_heads=4 // f, linear_num_key_heads=16 // f,
+                                  linear_num_value_heads=32 // f, intermediate_size=9216 // f)
+    prompts, rows, ctx, n_dec = (512, 2048, 8000), (1, 8, 32), 2048, 64
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+    out = {}
+    l0 = K.LAUNCHES
+    sampler = ClockSampler(0)
+    sampler.start()
+    for cfg in (new, old):
+        R = max(rows)
+        llm = LLM.from_random(cfg, seed=0, max_seq=8192, max_num_seqs=R, max_chunk=2048)
+        m = llm.model
+        g = torch.Generator().manual_seed(7)
+        res = {"weight_gb": round(m.weight_bytes() / 1e9, 2)}
+        with torch.no_grad():
+            for T in prompts:
+                toks = torch.randint(0, cfg.vocab_size, (T,), generator=g).cuda()
+                ms = 0.0
+                for it in range(W + args.steps):
+                    e0, e1 = ev(), ev()
+                    torch.cuda.synchronize()
+                    e0.record()
+                    llm.device_prefill(toks)
+                    e1.record()
+                    e1.synchronize()
+                    ms += e0.elapsed_time(e1) if it >= W else 0.0
+                res[f"prefill_{T}_tok_s"] = round(T * args.steps / (ms / 1e3))
+            pages = (ctx + n_dec + 63) // 64 + 1
+            tables = [list(range(1 + r * pages, 1 + (r + 1) * pages)) for r in range(R)]
+            for M in rows:
+                for r in range(M):
+                    m.zero_state(r)
+                # contents of the pages and states do not change the work of a step: decode from a synthetic context
+                fill = [int(v) for v in torch.randint(0, cfg.vocab_size, (M,), generator=g)]
+                m.capture(M, advance=True)
+                ms = 0.0
+                for it in range(W + args.steps):
+                    m.set_rows(M, fill, [ctx] * M, list(range(M)), tables[:M])
+                    e0, e1 = ev(), ev()
+                    torch.cuda.synchronize()
+                    e0.record()
+                    for _ in range(n_dec):
+                        m.decode(M, graph=True, advance=True)
+                    e1.record()
+                    e1.synchronize()
+                    ms += e0.elapsed_time(e1) if it >= W else 0.0
+                res[f"decode_{M}x{ctx}_tok_s"] = round(M * n_dec * args.steps / (ms / 1e3), 1)
+                res[f"launches_{M}_rows"] = m.launches_per_step(M)
+        out[cfg.name] = res
+        m._graphs.clear()
+        del llm, m
+        torch.cuda.empty_cache()
+    K.check_status()
+    a, b = out[new.name], out[old.name]
+    print(json.dumps({"metric": "tok_s_beside", "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": W, "higher_is_better": True,
+                      "dtype": "bf16", "data": "synthetic", "models": out,
+                      "ratio": {k: round(a[k] / b[k], 3) for k in a if k.endswith("tok_s")},
+                      "config": {"model": new.name, "beside": old.name, "decode_tokens": n_dec, "parallelism": "single",
+                                 "cache": "every step streams more weight bytes than the L2 holds"},
+                      "clocks": sampler.stop(), "gpu_launches": K.LAUNCHES - l0, "impl": "ours"}), flush=True)
 
 
 def bench_rows(args, cfg, W: int) -> None:

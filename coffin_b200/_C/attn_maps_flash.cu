@@ -230,26 +230,29 @@ int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
 }
 
 // ---- decode -------------------------------------------------------------------------------------
-// NQ: query vectors (heads of the group x maps) of one CTA, padded.  256 threads: scores by (key, quarter of dim),
-// values by (8 columns, key group).
+// One CTA per (key split, up to 8 / maps heads of a group, row).  Pages go through a two-stage cp.async ring; scores and
+// weighted sums are mma products with the query vectors as rows: eight of the sixteen rows are enough, so the second
+// product takes the bf16 heads of the weights in rows 0-7 and their remainders in rows 8-15.
 constexpr int kDT = 256;
-template <int NQ, int DC, typename TP>      // DC: 8-value pieces of a key per thread and map
-__global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
-  extern __shared__ __align__(16) float sm[];
-  const int dimp = (a.dim + 31) & ~31;
-  float* q = sm;                           // [NQ][dimp], scaled (log2 units with or without the cap's factor)
-  float* p = q + NQ * dimp;                // [kPage][NQ]
-  float* red = p + kPage * NQ;             // [NQ][key groups][vdim]
-  __shared__ float m_s[NQ], l_s[NQ], w_s[NQ];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+template <int DK, int DV, int MAPS, typename TP>
+__global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
+  constexpr int LK = DK + 8, LV = DV + 8, KPAGE = MAPS * kPage * LK, VPAGE = kPage * LV, NP = DV / 16, NPW = (NP + 7) / 8;
+  extern __shared__ __align__(128) unsigned char smem[];
+  bf16* ks = reinterpret_cast<bf16*>(smem);            // [2][MAPS][kPage][LK]
+  bf16* vs = ks + 2 * KPAGE;                           // [2][kPage][LV]
+  bf16* qs = vs + 2 * VPAGE;                           // [MAPS][8][LK]
+  bf16* pa = qs + MAPS * 8 * LK;                       // [16][kPage + 8]: heads, remainders
+  float* ps = reinterpret_cast<float*>(pa + 16 * (kPage + 8));   // [8][kPage] scores
+  __shared__ float w_s[8];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
   const int split = blockIdx.x, row = blockIdx.z;
   const int R = a.H / a.G, cpg = (R + hpc - 1) / hpc, g = blockIdx.y / cpg, r0 = (blockIdx.y % cpg) * hpc, nh = min(hpc, R - r0);
-  const int nq = nh * a.maps;
+  const int nq = nh * MAPS;                            // vector i: head i / MAPS of the CTA, map i % MAPS
   griddep_launch();
   griddep_wait();
   const int pos = a.positions[row], seg = a.row_seg ? a.row_seg[row] : row;
   if (pos < 0) return;
-  const int64_t vh0 = (int64_t)row * a.H * a.maps + (int64_t)(g * R + r0) * a.maps;
+  const int64_t vh0 = (int64_t)row * a.H * MAPS + (int64_t)(g * R + r0) * MAPS;
   const int pages = pos / kPage + 1, per = (pages + a.nsplit - 1) / a.nsplit;
   const int pg0 = split * per, pg1 = min(pages, pg0 + per);
   if (pg0 >= pages) {
@@ -257,164 +260,165 @@ __global__ void __launch_bounds__(kDT) maps_decode_kernel(const AttnMapsArgs a, 
     return;
   }
   const int* bt = a.tables + (int64_t)seg * a.ldbt;
-  const int64_t ldk = (int64_t)a.G * a.maps * a.dim, ldv = (int64_t)a.G * a.vdim;
-  bf16* K = reinterpret_cast<bf16*>(a.kpool) + (int64_t)g * a.maps * a.dim;
+  const int64_t ldk = (int64_t)a.G * MAPS * a.dim, ldv = (int64_t)a.G * a.vdim;
+  bf16* K = reinterpret_cast<bf16*>(a.kpool) + (int64_t)g * MAPS * a.dim;
   bf16* V = reinterpret_cast<bf16*>(a.vpool) + (int64_t)g * a.vdim;
   const TP* pr = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
+  auto load = [&](int pg) {
+    const int64_t base = (int64_t)bt[pg] * kPage;
+    const int n = pos + 1 - pg * kPage;                // keys of the page that exist
+    bf16* kd = ks + (pg & 1) * KPAGE;
+    bf16* vd = vs + (pg & 1) * VPAGE;
+    for (int e = tid; e < MAPS * kPage * (DK / 8); e += kDT) {
+      const int r = e / (MAPS * DK / 8), m = (e / (DK / 8)) % MAPS, c = (e % (DK / 8)) * 8;
+      const bool ok = r < n && c < a.dim;
+      cp16(kd + (m * kPage + r) * LK + c, ok ? K + (base + r) * ldk + m * a.dim + c : K, ok);
+    }
+    for (int e = tid; e < kPage * (DV / 8); e += kDT) {
+      const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+      const bool ok = r < n && c < a.vdim;
+      cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load(pg0);
   const bool cap = a.cap > 0.f;
   const float f = a.scale * query_temp(a, pos) * (cap ? 2.f * kLog2e / a.cap : kLog2e), cap2 = a.cap * kLog2e;
-  for (int e = tid; e < NQ * dimp; e += kDT) {
-    const int i = e / dimp, c = e % dimp;
-    q[e] = i < nq && c < a.dim ? act_round<bf16>(act_load(pr + ((int64_t)(g * R + r0) * a.maps + i) * a.dim + c)) * f : 0.f;
+  for (int e = tid; e < MAPS * 8 * LK; e += kDT) {
+    const int m = e / (8 * LK), i = (e / LK) % 8, c = e % LK;
+    const bool ok = i < nh && c < a.dim;
+    qs[e] = ok ? __float2bfloat16(act_load(pr + ((int64_t)(g * R + r0 + i) * MAPS + m) * a.dim + c)) : __float2bfloat16(0.f);
   }
-  if (pg1 == pages) {
-    // this CTA reads the token's own key and value: it stores them (CTAs of other heads of the group store the same)
-    const int64_t slot = (int64_t)bt[pages - 1] * kPage + pos % kPage;
-    for (int c = tid; c < a.maps * a.dim; c += kDT) act_store(K + slot * ldk + c, act_load(pr + a.k_col + (int64_t)g * a.maps * a.dim + c));
-    for (int c = tid; c < a.vdim; c += kDT) act_store(V + slot * ldv + c, act_load(pr + a.v_col + (int64_t)g * a.vdim + c));
-  }
-  if (tid < NQ) { m_s[tid] = -INFINITY; l_s[tid] = 0.f; }
-  const int co = a.vdim >> 3, KG = min(kPage, kDT / co), cg = tid % co, kg = tid / co;
-  float o[NQ][8];
+  for (int e = tid; e < 16 * (kPage + 8); e += kDT) pa[e] = __float2bfloat16(0.f);
+  float o[NPW][2][4];
 #pragma unroll
-  for (int i = 0; i < NQ; ++i)
+  for (int i = 0; i < NPW; ++i)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) o[i][e] = 0.f;
-  __syncthreads();
-  const int key = tid >> 2, part = tid & 3;
+    for (int j = 0; j < 2; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+  float m_run = -INFINITY, l_run = 0.f;                // of vector `warp`
   for (int pg = pg0; pg < pg1; ++pg) {
-    const int64_t base = (int64_t)bt[pg] * kPage;
-    const bool vis = pg * kPage + key <= pos;
-    // everything this thread reads of the page, requested at once
-    uint4 kr[2][DC], vr[8];
-#pragma unroll
-    for (int mp = 0; mp < 2; ++mp)
-#pragma unroll
-      for (int j = 0; j < DC; ++j) {
-        const int c = part * 8 + 32 * j;
-        kr[mp][j] = mp < a.maps && c < a.dim && vis ? *reinterpret_cast<const uint4*>(K + (base + key) * ldk + (int64_t)mp * a.dim + c)
-                                                    : make_uint4(0, 0, 0, 0);
-      }
-    const int nk = min(kPage, pos + 1 - pg * kPage);
-#pragma unroll
-    for (int u = 0; u < 8; ++u) {
-      const int k = kg + u * KG;
-      vr[u] = kg < KG && k < nk ? *reinterpret_cast<const uint4*>(V + (base + k) * ldv + cg * 8) : make_uint4(0, 0, 0, 0);
-    }
-    // scores: lanes 4k .. 4k + 3 hold quarters of key k
-#pragma unroll
-    for (int mp = 0; mp < 2; ++mp) {
-      if (mp >= a.maps) break;
-      float s[NQ];
-#pragma unroll
-      for (int i = 0; i < NQ; ++i) s[i] = 0.f;
-#pragma unroll
-      for (int j = 0; j < DC; ++j) {
-        const int c = part * 8 + 32 * j;
-        float kf[8];
-        bf16x8_to_float(kr[mp][j], kf);
-        if (c < a.dim) {
-#pragma unroll
-          for (int i = 0; i < NQ; ++i) {
-            if (i * a.maps + mp < nq) {
-              const float4 q0 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c);
-              const float4 q1 = *reinterpret_cast<const float4*>(q + (i * a.maps + mp) * dimp + c + 4);
-              s[i] = fmaf(q0.x, kf[0], s[i]); s[i] = fmaf(q0.y, kf[1], s[i]); s[i] = fmaf(q0.z, kf[2], s[i]); s[i] = fmaf(q0.w, kf[3], s[i]);
-              s[i] = fmaf(q1.x, kf[4], s[i]); s[i] = fmaf(q1.y, kf[5], s[i]); s[i] = fmaf(q1.z, kf[6], s[i]); s[i] = fmaf(q1.w, kf[7], s[i]);
-            }
-          }
-        }
-      }
-#pragma unroll
-      for (int i = 0; i < NQ; ++i) {
-        if (i * a.maps + mp >= nq) continue;
-        float x = s[i];
-        x += __shfl_xor_sync(0xffffffffu, x, 1);
-        x += __shfl_xor_sync(0xffffffffu, x, 2);
-        if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
-        if (part == (i & 3)) p[key * NQ + i * a.maps + mp] = vis ? x : -INFINITY;
-      }
+    if (pg + 1 < pg1) {
+      load(pg + 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    for (int i = warp; i < nq; i += kDT / 32) {
-      const float x0 = p[lane * NQ + i], x1 = p[(lane + 32) * NQ + i], mo = m_s[i];
-      const float mn = fmaxf(mo, warp_max(fmaxf(x0, x1)));       // finite: the first key of a walked page is visible
-      const float e0 = ex2(x0 - mn), e1 = ex2(x1 - mn), w = ex2(mo - mn);
-      const float sum = warp_sum(e0 + e1);
-      p[lane * NQ + i] = e0;
-      p[(lane + 32) * NQ + i] = e1;
-      if (lane == 0) { m_s[i] = mn; l_s[i] = l_s[i] * w + sum; w_s[i] = w; }
-    }
-    __syncthreads();
-    if (kg < KG) {
-#pragma unroll
-      for (int i = 0; i < NQ; ++i) {
-        const float w = i < nq ? w_s[i] : 0.f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[i][e] *= w;
+    bf16* kt = ks + (pg & 1) * KPAGE;
+    bf16* vt = vs + (pg & 1) * VPAGE;
+    if (pg == pages - 1) {
+      // the token's own key and value: into the staged page, and into the pool (CTAs of other heads of the group store
+      // the same values)
+      const int r = pos % kPage;
+      const int64_t slot = (int64_t)bt[pg] * kPage + r;
+      for (int c = tid; c < MAPS * a.dim; c += kDT) {
+        const bf16 x = __float2bfloat16(act_load(pr + a.k_col + (int64_t)g * MAPS * a.dim + c));
+        kt[((c / a.dim) * kPage + r) * LK + c % a.dim] = x;
+        K[slot * ldk + c] = x;
       }
+      for (int c = tid; c < a.vdim; c += kDT) {
+        const bf16 x = __float2bfloat16(act_load(pr + a.v_col + (int64_t)g * a.vdim + c));
+        vt[r * LV + c] = x;
+        V[slot * ldv + c] = x;
+      }
+      __syncthreads();
+    }
+    // scores of keys 8 warp .. 8 warp + 7
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const int k = kg + u * KG;
-        if (k < nk) {
-          float vf[8];
-          bf16x8_to_float(vr[u], vf);
+    for (int m = 0; m < MAPS; ++m) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+      const bf16* qr = qs + (m * 8 + g4) * LK + t4 * 2;
+      const bf16* kr = kt + (m * kPage + warp * 8 + (lane & 7)) * LK + (lane >> 3) * 8;
 #pragma unroll
-          for (int i = 0; i < NQ; ++i) {
-            if (i < nq) {
-              const float w = p[k * NQ + i];
+      for (int k = 0; k < DK / 32; ++k) {
+        uint32_t b[4];
+        ldsm4(b, kr + k * 32);
+        const uint32_t a0[4] = {*reinterpret_cast<const uint32_t*>(qr + k * 32), 0u, *reinterpret_cast<const uint32_t*>(qr + k * 32 + 8), 0u};
+        const uint32_t a1[4] = {*reinterpret_cast<const uint32_t*>(qr + k * 32 + 16), 0u, *reinterpret_cast<const uint32_t*>(qr + k * 32 + 24), 0u};
+        mma(s, a0, b[0], b[1]);
+        mma(s2, a1, b[2], b[3]);
+      }
+      if (g4 < nh) {
 #pragma unroll
-              for (int e = 0; e < 8; ++e) o[i][e] = fmaf(w, vf[e], o[i][e]);
-            }
-          }
+        for (int e = 0; e < 2; ++e) {
+          float x = (s[e] + s2[e]) * f;
+          if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
+          const int key = warp * 8 + t4 * 2 + e;
+          ps[(g4 * MAPS + m) * kPage + key] = pg * kPage + key <= pos ? x : -INFINITY;
         }
       }
     }
     __syncthreads();
-  }
-  if (kg < KG) {
+    if (warp < nq) {
+      const float2 x = *reinterpret_cast<const float2*>(ps + warp * kPage + 2 * lane);
+      const float mn = fmaxf(m_run, warp_max(fmaxf(x.x, x.y)));  // finite: the first key of a walked page is visible
+      float e0 = ex2(x.x - mn), e1 = ex2(x.y - mn);
+      const float w = ex2(m_run - mn);
+      l_run = l_run * w + warp_sum(e0 + e1);
+      m_run = mn;
+      *reinterpret_cast<uint32_t*>(pa + warp * (kPage + 8) + 2 * lane) = split_head(e0, e1);
+      *reinterpret_cast<uint32_t*>(pa + (8 + warp) * (kPage + 8) + 2 * lane) = pack_bf162(e0, e1);
+      if (lane == 0) w_s[warp] = w;
+    }
+    __syncthreads();
+    const float w = g4 < nq ? w_s[g4] : 0.f;
+    uint32_t pf[4][4];
 #pragma unroll
-    for (int i = 0; i < NQ; ++i)
-      if (i < nq) {
-        float4* d = reinterpret_cast<float4*>(red + ((int64_t)i * KG + kg) * a.vdim + cg * 8);
-        d[0] = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
-        d[1] = make_float4(o[i][4], o[i][5], o[i][6], o[i][7]);
+    for (int k = 0; k < 4; ++k) ldsm4(pf[k], pa + (lane & 15) * (kPage + 8) + k * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int i = 0; i < NPW; ++i) {
+      const int cp = warp + 8 * i;
+      if (cp >= NP) break;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) { o[i][j][0] *= w; o[i][j][1] *= w; o[i][j][2] *= w; o[i][j][3] *= w; }
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        uint32_t b[4];
+        ldsm4t(b, vt + (k * 16 + (lane & 15)) * LV + cp * 16 + (lane >> 4) * 8);
+        mma(o[i][0], pf[k], b[0], b[1]);
+        mma(o[i][1], pf[k], b[2], b[3]);
       }
+    }
+    __syncthreads();
   }
-  __syncthreads();
-  for (int e = tid; e < nq * a.vdim; e += kDT) {
-    const int i = e / a.vdim, c = e % a.vdim;
-    float x = 0.f;
-#pragma unroll 8
-    for (int k = 0; k < KG; ++k) x += red[(i * KG + k) * a.vdim + c];
-    a.part_o[((vh0 + i) * a.nsplit + split) * a.vdim + c] = x;
-  }
-  if (tid < nq) {
-    float* ml = a.part_ml + ((vh0 + tid) * a.nsplit + split) * 2;
-    ml[0] = m_s[tid] * (1.f / kLog2e);
-    ml[1] = l_s[tid];
+#pragma unroll
+  for (int i = 0; i < NPW; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int c = (warp + 8 * i) * 16 + j * 8 + t4 * 2;
+      if (warp + 8 * i < NP && g4 < nq && c < a.vdim)
+        *reinterpret_cast<float2*>(a.part_o + ((vh0 + g4) * a.nsplit + split) * a.vdim + c) =
+            make_float2(o[i][j][0] + o[i][j][2], o[i][j][1] + o[i][j][3]);
+    }
+  if (warp < nq && lane == 0) {
+    float* ml = a.part_ml + ((vh0 + warp) * a.nsplit + split) * 2;
+    ml[0] = m_run * (1.f / kLog2e);
+    ml[1] = l_run;
   }
 }
 
-template <int NQ, int DC, typename TP>
+template <int DK, int DV, int MAPS, typename TP>
 int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
-  const int dimp = (a.dim + 31) & ~31, co = a.vdim / 8, KG = kDT / co < kPage ? kDT / co : kPage;
-  const size_t smem = sizeof(float) * ((size_t)NQ * dimp + kPage * NQ + (size_t)NQ * KG * a.vdim);
-  auto kern = maps_decode_kernel<NQ, DC, TP>;
-  if (smem > 40 * 1024) {
-    if (smem > 200 * 1024) return CB_ERR_SHAPE;
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-  }
+  constexpr size_t smem = sizeof(bf16) * (2 * (size_t)kPage * (MAPS * (DK + 8) + DV + 8) + MAPS * 8 * (DK + 8) + 16 * (kPage + 8)) +
+                          sizeof(float) * 8 * kPage;
+  auto kern = maps_decode_kernel<DK, DV, MAPS, TP>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
   const int R = a.H / a.G;
   return (int)cb_launch(kern, dim3((unsigned)a.nsplit, (unsigned)(a.G * ((R + hpc - 1) / hpc)), (unsigned)rows), dim3(kDT), smem, st, a, hpc);
 }
-template <int NQ, typename TP>
-int decode_dim(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
-  if (a.dim <= 32) return decode_launch<NQ, 1, TP>(a, hpc, rows, st);
-  if (a.dim <= 64) return decode_launch<NQ, 2, TP>(a, hpc, rows, st);
-  if (a.dim <= 128) return decode_launch<NQ, 4, TP>(a, hpc, rows, st);
-  return decode_launch<NQ, 8, TP>(a, hpc, rows, st);
+template <int DK, int MAPS, typename TP>
+int decode_dv(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  if (a.vdim <= 64) return decode_launch<DK, 64, MAPS, TP>(a, hpc, rows, st);
+  if (a.vdim <= 128) return decode_launch<DK, 128, MAPS, TP>(a, hpc, rows, st);
+  return decode_launch<DK, 256, MAPS, TP>(a, hpc, rows, st);
+}
+template <int MAPS, typename TP>
+int decode_dk(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  if (a.dim <= 32) return decode_dv<32, MAPS, TP>(a, hpc, rows, st);
+  if (a.dim <= 64) return decode_dv<64, MAPS, TP>(a, hpc, rows, st);
+  if (a.dim <= 128) return decode_dv<128, MAPS, TP>(a, hpc, rows, st);
+  return decode_dv<256, MAPS, TP>(a, hpc, rows, st);
 }
 
 }  // namespace
@@ -452,13 +456,6 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   const int R = a.H / a.G;
   int hpc = 8 / a.maps;                                  // heads per CTA: at most 8 query vectors
   if (hpc > R) hpc = R;
-  const int nq = hpc * a.maps;
-  if (p_f32) {
-    if (nq <= 2) return decode_dim<2, float>(a, hpc, (int)rows, st);
-    if (nq <= 4) return decode_dim<4, float>(a, hpc, (int)rows, st);
-    return decode_dim<8, float>(a, hpc, (int)rows, st);
-  }
-  if (nq <= 2) return decode_dim<2, bf16>(a, hpc, (int)rows, st);
-  if (nq <= 4) return decode_dim<4, bf16>(a, hpc, (int)rows, st);
-  return decode_dim<8, bf16>(a, hpc, (int)rows, st);
+  if (a.maps == 1) return p_f32 ? decode_dk<1, float>(a, hpc, (int)rows, st) : decode_dk<1, bf16>(a, hpc, (int)rows, st);
+  return p_f32 ? decode_dk<2, float>(a, hpc, (int)rows, st) : decode_dk<2, bf16>(a, hpc, (int)rows, st);
 }

@@ -94,8 +94,9 @@ __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* 
   for (int i = 0; i < kT / 32; ++i) { a += red[i * 3]; b += red[i * 3 + 1]; c += red[i * 3 + 2]; }
 }
 
-template <int KIND, typename TP, typename TA, int RMAX>
-__global__ void __launch_bounds__(kT, RMAX <= 8 ? 2 : 1) linrec_step_kernel(const LinrecArgs a) {
+// LOW: the low-rank factors are multiplied here (few rows), else their results are given
+template <int KIND, typename TP, typename TA, int RMAX, bool LOW>
+__global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 1)) linrec_step_kernel(const LinrecArgs a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
   __shared__ float cl_part;
@@ -114,10 +115,10 @@ __global__ void __launch_bounds__(kT, RMAX <= 8 ? 2 : 1) linrec_step_kernel(cons
   const int cq = jc >> 2, RG = kT / cq, q4 = tid % cq, rg = tid / cq;
   const bool act_thr = rg < RG;
   const int j0 = rank * jc, ncol = min(jc, dv - j0);   // ncol > 0 by construction of the grid
-  constexpr bool kLow = KIND == LINREC_DELTA && sizeof(TA) == 2;
+  constexpr bool kLow = KIND == LINREC_DELTA && sizeof(TA) == 2 && LOW;
   const bool low_a = kLow && !a.dec && a.ra <= 256, low_g = kLow && !a.og && a.rg <= 256;
-  LowRank<kLow ? 8 : 1> lra;
-  LowRank<kLow ? 4 : 1> lrg;
+  LowRank<kLow ? (RMAX <= 8 ? 8 : 4) : 1> lra;
+  LowRank<kLow ? (RMAX <= 8 ? 4 : 2) : 1> lrg;
   if (low_a) lra.init(reinterpret_cast<const bf16*>(a.a2) + (int64_t)h * dk * a.ra, dk, (int)a.ra);
   if (low_g) lrg.init(reinterpret_cast<const bf16*>(a.g2) + ((int64_t)h * dv + j0) * a.rg, ncol, (int)a.rg);
   griddep_launch();
@@ -208,14 +209,14 @@ __global__ void __launch_bounds__(kT, RMAX <= 8 ? 2 : 1) linrec_step_kernel(cons
       for (int c = tid; c < dk; c += kT) {
         sq[c] *= rq; sk[c] *= rk;
         const int64_t ch = (int64_t)h * dk + c;
-        const float x = a.dec ? a.dec[row * a.ldd + ch] : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
+        const float x = !LOW || a.dec ? a.dec[row * a.ldd + ch] : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
         sg[c] = expf(-ea * softplus_x(x + a.dt_bias[ch]));
       }
       const TA* g2 = reinterpret_cast<const TA*>(a.g2);
       const float* lg = low + (a.dec ? 0 : a.ra);
       for (int c = tid; c < ncol; c += kT) {
         const int64_t ch = (int64_t)h * dv + j0 + c;
-        const float x = a.og ? act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
+        const float x = !LOW || a.og ? act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
         sog[c] = sigmoid_x(x);
       }
     } else {
@@ -389,9 +390,9 @@ __global__ void __launch_bounds__(256) linrec_ring_kernel(const TA* __restrict__
   }
 }
 
-template <int KIND, typename TP, typename TA, int RMAX>
+template <int KIND, typename TP, typename TA, int RMAX, bool LOW>
 int launch_step(const LinrecArgs& a, int ns, int segs, size_t smem, cudaStream_t st) {
-  auto kern = linrec_step_kernel<KIND, TP, TA, RMAX>;
+  auto kern = linrec_step_kernel<KIND, TP, TA, RMAX, LOW>;
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
@@ -417,19 +418,17 @@ int launch_step(const LinrecArgs& a, int ns, int segs, size_t smem, cudaStream_t
   return (int)cudaLaunchKernelEx(&cfg, kern, a);
 }
 
-// value columns per CTA: the head is cut into at most 8 slices; more slices while the grid is small, fewer rows per
-// thread than 32 always
+// value columns per CTA: a head is one CTA when 16 state rows per thread suffice, else the fewest slices that get there
+// (32 rows per thread if nothing does); more slices, down to 16 columns, while the machine has idle SMs
 int plan_cols(int64_t H, int64_t dk, int64_t dv, int64_t segs) {
-  int best = 0;
+  int best = 0, rows = 0;
   for (int ns = 1; ns <= 8; ++ns) {
     int jc = (int)((dv + ns - 1) / ns);
     jc = (jc + 3) & ~3;
     if ((dv + jc - 1) / jc != ns || jc > 4 * kT) continue;
-    const int RG = kT / (jc / 4);
-    if ((dk + RG - 1) / RG > 32) continue;
-    if (!best) best = jc;
-    // another slice as long as the machine has idle SMs and a slice keeps at least 16 columns
-    if (H * ns * segs <= 160 && jc >= 16) best = jc;
+    const int RG = kT / (jc / 4), r = (int)((dk + RG - 1) / RG);
+    if (r > 32) continue;
+    if (!best || rows > 16 || (H * ns * segs <= 160 && jc >= 16)) { best = jc; rows = r; }
   }
   return best;
 }
@@ -442,10 +441,14 @@ int dispatch_step(LinrecArgs& a, int segs, cudaStream_t st) {
   const int64_t lown = KIND == LINREC_DELTA ? (a.dec ? 0 : a.ra) + (a.og ? 0 : a.rg) : 0;
   const size_t smem = sizeof(float) * (size_t)(3 * a.dk + 4 * a.jc + ((lown + 3) & ~3) + 2 * RG * a.jc);
   if (smem > 200 * 1024) return CB_ERR_SHAPE;
-  if (rm <= 4) return launch_step<KIND, TP, TA, 4>(a, ns, segs, smem, st);
-  if (rm <= 8) return launch_step<KIND, TP, TA, 8>(a, ns, segs, smem, st);
-  if (rm <= 16) return launch_step<KIND, TP, TA, 16>(a, ns, segs, smem, st);
-  return launch_step<KIND, TP, TA, 32>(a, ns, segs, smem, st);
+#define CB_ROWS(R)                                                                        \
+  if (rm <= R) {                                                                          \
+    if (KIND == LINREC_DELTA && (!a.dec || !a.og)) return launch_step<KIND, TP, TA, R, KIND == LINREC_DELTA>(a, ns, segs, smem, st); \
+    return launch_step<KIND, TP, TA, R, false>(a, ns, segs, smem, st);                    \
+  }
+  CB_ROWS(4) CB_ROWS(8) CB_ROWS(16) CB_ROWS(32)
+#undef CB_ROWS
+  return CB_ERR_SHAPE;
 }
 
 }  // namespace

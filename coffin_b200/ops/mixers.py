@@ -239,7 +239,7 @@ class AttnMaps:
     def decode_splits(self, rows: int) -> int:
         R = self.H // self.G
         hpc = min(R, 8 // self.maps)
-        return max(1, min(64, 296 // max(1, self.G * -(-R // hpc) * rows)))
+        return max(1, min(64, 148 // max(1, self.G * -(-R // hpc) * rows)))
 
     def decode(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
         """Single tokens (their keys and values are appended by the kernel): ``nsplit`` key splits per row."""

@@ -30,7 +30,7 @@ __device__ __forceinline__ float ld_dsmem(const float* p, uint32_t rank) {
 
 // dot of a weight row (storage type) with fp32 values in shared memory; n is a multiple of 4
 template <typename TW>
-__device__ __forceinline__ float row_dot(const TW* __restrict__ w, const float* x, int64_t n) {
+__device__ __noinline__ float row_dot(const TW* __restrict__ w, const float* x, int64_t n) {
   float s0 = 0.f, s1 = 0.f;
   int64_t i = 0;
 #pragma unroll 1
@@ -61,24 +61,31 @@ struct LowRank {
     const int i = it * kT + (int)threadIdx.x, r = i >> lsh, c = i & ((1 << lsh) - 1);
     return r < rows && c < nch ? *reinterpret_cast<const uint4*>(W + ((int64_t)r * nch + c) * 8) : make_uint4(0, 0, 0, 0);
   }
-  // out[r] = W[r, :] . x, by the first lane of a row
-  __device__ __forceinline__ void dot_piece(int it, const uint4& v, const float* x, float* out) const {
+  // out[r] = W[r, :] . x, by the first lane of a row.  A thread's pieces all multiply the same eight values of x.
+  __device__ __forceinline__ void dot_piece(int it, const uint4& v, const float* xr, float* out) const {
     const int i = it * kT + (int)threadIdx.x, r = i >> lsh, c = i & ((1 << lsh) - 1);
     float f[8], s = 0.f;
     bf16x8_to_float(v, f);
-    if (c < nch) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) s = fmaf(f[e], x[c * 8 + e], s);
-    }
+    for (int e = 0; e < 8; ++e) s = fmaf(f[e], xr[e], s);
     for (int o = 1; o < (1 << lsh); o <<= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     if (c == 0 && r < rows) out[r] = s;
   }
-  __device__ __forceinline__ void run(const float* x, float* out) const {
+  __device__ __forceinline__ void run(const float* x, float* out) {
+    const int c = (int)threadIdx.x & ((1 << lsh) - 1);
+    float xr[8];
 #pragma unroll
-    for (int i = 0; i < PRE; ++i)
-      if (i < iters) dot_piece(i, w[i], x, out);
+    for (int e = 0; e < 8; ++e) xr[e] = c < nch ? x[c * 8 + e] : 0.f;
 #pragma unroll 1
-    for (int i = PRE; i < iters; ++i) dot_piece(i, piece(i), x, out);
+    for (int g = 0; g < iters; g += PRE) {
+      if (g > 0) {
+#pragma unroll
+        for (int i = 0; i < PRE; ++i) w[i] = g + i < iters ? piece(g + i) : make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+      for (int i = 0; i < PRE; ++i)
+        if (g + i < iters) dot_piece(g + i, w[i], xr, out);
+    }
   }
 };
 
@@ -118,35 +125,51 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
   constexpr bool kLow = KIND == LINREC_DELTA && sizeof(TA) == 2 && LOW;
   const bool low_a = kLow && !a.dec && a.ra <= 256, low_g = kLow && !a.og && a.rg <= 256;
   LowRank<kLow ? (RMAX <= 8 ? 8 : 4) : 1> lra;
-  LowRank<kLow ? (RMAX <= 8 ? 4 : 2) : 1> lrg;
+  LowRank<kLow ? 4 : 1> lrg;
   if (low_a) lra.init(reinterpret_cast<const bf16*>(a.a2) + (int64_t)h * dk * a.ra, dk, (int)a.ra);
   if (low_g) lrg.init(reinterpret_cast<const bf16*>(a.g2) + ((int64_t)h * dv + j0) * a.rg, ncol, (int)a.rg);
+  // parameters of this thread's channels, requested ahead of the dependency like the factors
+  float4 pcw[2];                                       // convolution taps of channels tid and tid + kT (four taps)
+  const int nch = 2 * dk + ncol;
+  const bool taps4 = a.taps == 4;
+  const int qb = h / (a.H / a.G) * dk;
+  auto channel = [&](int e) {
+    return e < dk ? (int64_t)(qb + e) : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk);
+  };
+  float p_dt = 0.f, p_ea = 0.f;
+  if (KIND == LINREC_DELTA) {
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+      pcw[u] = taps4 && tid + u * kT < nch ? *reinterpret_cast<const float4*>(a.conv_w + channel(tid + u * kT) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    p_ea = expf(a.A_log[h]);
+    if (tid < dk) p_dt = a.dt_bias[(int64_t)h * dk + tid];
+  }
+  const float* nw = a.norm_w + (KIND == LINREC_MLSTM ? (int64_t)h * dv : 0) + j0;
+  const float p_nw = tid < ncol ? nw[tid] : 0.f;
   griddep_launch();
   griddep_wait();
   const int row0 = a.seg_row ? a.seg_row[seg] : seg;
   const int nrow = a.seg_row ? a.seg_row[seg + 1] - row0 : 1;
   const int slot = a.seg_slot[seg], pos0 = a.seg_pos[seg];
   if (slot < 0 || nrow < 1 || pos0 < 0) return;        // the same for every CTA of the cluster
-  const int gk = h / (a.H / a.G);
-  const int qb = gk * dk;
   float* Sg = a.S + ((int64_t)slot * a.H + h) * dk * dv + j0;
   const bool vec = (dv & 3) == 0 && ncol == jc;
   float S[RMAX][4];
+  const int nr = act_thr && q4 * 4 < ncol ? (dk - rg + RG - 1) / RG : 0;      // state rows of this thread
+  float* const Sp = Sg + (int64_t)rg * dv + q4 * 4;
+  const int64_t sstep = (int64_t)RG * dv;
+  const int ne = min(4, ncol - q4 * 4);
+  if (vec) {
 #pragma unroll
-  for (int i = 0; i < RMAX; ++i) {
-    const int r = rg + i * RG;
-#pragma unroll
-    for (int e = 0; e < 4; ++e) S[i][e] = 0.f;
-    if (act_thr && r < dk) {
-      const float* p = Sg + (int64_t)r * dv + q4 * 4;
-      if (vec) {
-        const float4 f = *reinterpret_cast<const float4*>(p);
-        S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
-      } else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) if (q4 * 4 + e < ncol) S[i][e] = p[e];
-      }
+    for (int i = 0; i < RMAX; ++i) {
+      const float4 f = i < nr ? *reinterpret_cast<const float4*>(Sp + i * sstep) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
     }
+  } else {
+#pragma unroll
+    for (int i = 0; i < RMAX; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[i][e] = i < nr && e < ne ? Sp[i * sstep + e] : 0.f;
   }
   float mrun = 0.f;
   if (KIND == LINREC_MLSTM) {
@@ -165,33 +188,41 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     if (KIND == LINREC_DELTA) {
       // short convolution: channels q, k, v of this CTA spread over the block, four taps requested together (in a decode
       // step all but the newest come from the ring)
-      const int nch = 2 * dk + ncol;
+      auto tap = [&](int64_t ch, int j) {                // the row a tap reads is the same for every channel
+        const int src = t - (a.taps - 1) + j, p = pos0 + src;
+        float x = 0.f;
+        if (src >= 0) x = act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
+        else if (p >= 0) x = act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch);
+        return x;
+      };
+      auto put = [&](int e, float acc) { (e < 2 * dk ? sq : sv - 2 * dk)[e] = silu_s(acc); };       // sq and sk are adjacent
+      if (taps4) {
+        float x[2][4];
+        const int64_t ch0 = channel(tid < nch ? tid : 0), ch1 = channel(tid + kT < nch ? tid + kT : 0);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          x[0][j] = tid < nch ? tap(ch0, j) : 0.f;
+          x[1][j] = tid + kT < nch ? tap(ch1, j) : 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+          if (tid + u * kT < nch)
+            put(tid + u * kT, fmaf(pcw[u].w, x[u][3], fmaf(pcw[u].z, x[u][2], fmaf(pcw[u].y, x[u][1], pcw[u].x * x[u][0]))));
+      }
 #pragma unroll 1
-      for (int e = tid; e < nch; e += kT) {
-        const int64_t ch = e < dk ? (int64_t)qb + e : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk);
+      for (int e = tid + (taps4 ? 2 * kT : 0); e < nch; e += kT) {
+        const int64_t ch = channel(e);
         float acc = 0.f;
 #pragma unroll 1
-        for (int b = 0; b < a.taps; b += 4) {
-          float x[4], w[4];
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const int src = t - (a.taps - 1) + b + j, p = pos0 + src;
-            const bool ok = b + j < a.taps && p >= 0;
-            w[j] = ok ? a.conv_w[ch * a.taps + b + j] : 0.f;
-            x[j] = ok && src < 0 ? act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch) : 0.f;
-            if (ok && src >= 0) x[j] = act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
-          }
-#pragma unroll
-          for (int j = 0; j < 4; ++j) acc = fmaf(w[j], x[j], acc);
-        }
-        (e < 2 * dk ? sq : sv - 2 * dk)[e] = silu_x(acc);        // sq and sk are adjacent
+        for (int j = 0; j < a.taps; ++j) acc = fmaf(a.conv_w[ch * a.taps + j], tap(ch, j), acc);
+        put(e, acc);
       }
 #pragma unroll 1
       for (int c = tid; c < lown; c += kT) {
         const int na = a.dec ? 0 : (int)a.ra;
         low[c] = act_round<TA>(act_load(pr + (c < na ? a.a1_col + c : a.g1_col + c - na)));
       }
-      bb = sigmoid_x(a.gates[row * a.ldg + h]);            // beta
+      bb = sigmoid_s(a.gates[row * a.ldg + h]);            // beta
       __syncthreads();
       float q2 = 0.f, k2 = 0.f, qk = 0.f;
       for (int c = tid; c < dk; c += kT) {
@@ -204,20 +235,19 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
       if (low_a) lra.run(low, sg);
       if (low_g) lrg.run(low + (a.dec ? 0 : a.ra), sog);
       if (low_a || low_g) __syncthreads();
-      const float ea = expf(a.A_log[h]);
       const TA* a2 = reinterpret_cast<const TA*>(a.a2);
       for (int c = tid; c < dk; c += kT) {
         sq[c] *= rq; sk[c] *= rk;
         const int64_t ch = (int64_t)h * dk + c;
         const float x = !LOW || a.dec ? a.dec[row * a.ldd + ch] : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
-        sg[c] = expf(-ea * softplus_x(x + a.dt_bias[ch]));
+        sg[c] = __expf(-p_ea * softplus_s(x + (c == tid ? p_dt : a.dt_bias[ch])));
       }
       const TA* g2 = reinterpret_cast<const TA*>(a.g2);
       const float* lg = low + (a.dec ? 0 : a.ra);
       for (int c = tid; c < ncol; c += kT) {
         const int64_t ch = (int64_t)h * dv + j0 + c;
         const float x = !LOW || a.og ? act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
-        sog[c] = sigmoid_x(x);
+        sog[c] = sigmoid_s(x);
       }
     } else {
       const float rs = 1.f / sqrtf((float)dk);
@@ -241,7 +271,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
         const int64_t ch = (int64_t)h * dv + j0 + c;
         sv[c] = act_round<TA>(act_load(pr + a.v_col + ch));
         const float x = a.og ? act_load(reinterpret_cast<const TP*>(a.og) + row * a.ldo + ch) : 0.f;
-        sog[c] = sigmoid_x(x);
+        sog[c] = sigmoid_s(x);
       }
       block_sum3(nq, z1, z2, red);
       den = fmaxf(fabsf(nq), expf(-mn)) + 1e-6f;
@@ -256,7 +286,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
 #pragma unroll
       for (int i = 0; i < RMAX; ++i) {
         const int r = rg + i * RG;
-        if (act_thr && r < dk) {
+        if (i < nr) {
           const float k = sk[r], q = sq[r];
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
@@ -269,7 +299,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
 #pragma unroll
       for (int i = 0; i < RMAX; ++i) {
         const int r = rg + i * RG;
-        if (act_thr && r < dk) {
+        if (i < nr) {
           const float k = sk[r], q = sq[r], g = sg[r];
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
@@ -316,7 +346,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
 #pragma unroll
       for (int i = 0; i < RMAX; ++i) {
         const int r = rg + i * RG;
-        if (act_thr && r < dk) {
+        if (i < nr) {
           const float k = sk[r];
 #pragma unroll
           for (int e = 0; e < 4; ++e) S[i][e] = fmaf(k, u4[e], S[i][e]);
@@ -336,23 +366,20 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     }
     const float rstd = 1.f / sqrtf(ss / (float)dv + a.eps);
     TA* out = reinterpret_cast<TA*>(a.act) + row * a.lda + (int64_t)h * dv + j0;
-    const float* nw = a.norm_w + (KIND == LINREC_MLSTM ? (int64_t)h * dv : 0) + j0;
-    for (int c = tid; c < ncol; c += kT) act_store(out + c, so[c] * rstd * nw[c] * sog[c]);
+    for (int c = tid; c < ncol; c += kT) act_store(out + c, so[c] * rstd * (c == tid ? p_nw : nw[c]) * sog[c]);
     __syncthreads();
   }
   // ---- state back
+  if (vec) {
 #pragma unroll
-  for (int i = 0; i < RMAX; ++i) {
-    const int r = rg + i * RG;
-    if (act_thr && r < dk) {
-      float* p = Sg + (int64_t)r * dv + q4 * 4;
-      if (vec) {
-        *reinterpret_cast<float4*>(p) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-      } else {
+    for (int i = 0; i < RMAX; ++i)
+      if (i < nr) *reinterpret_cast<float4*>(Sp + i * sstep) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+  } else {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) if (q4 * 4 + e < ncol) p[e] = S[i][e];
-      }
-    }
+    for (int i = 0; i < RMAX; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (i < nr && e < ne) Sp[i * sstep + e] = S[i][e];
   }
   if (KIND == LINREC_MLSTM && rank == 0) {
     for (int c = tid; c < dk; c += kT) a.n[((int64_t)slot * a.H + h) * dk + c] = sg[c];
@@ -423,6 +450,7 @@ int launch_step(const LinrecArgs& a, int ns, int segs, size_t smem, cudaStream_t
 int plan_cols(int64_t H, int64_t dk, int64_t dv, int64_t segs) {
   int best = 0, rows = 0;
   for (int ns = 1; ns <= 8; ++ns) {
+    if (best && (ns & (ns - 1))) continue;             // slices by halving
     int jc = (int)((dv + ns - 1) / ns);
     jc = (jc + 3) & ~3;
     if ((dv + jc - 1) / jc != ns || jc > 4 * kT) continue;

@@ -136,7 +136,8 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
   auto channel = [&](int e) {
     return e < dk ? (int64_t)(qb + e) : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk);
   };
-  float p_dt = 0.f, p_ea = 0.f;
+  float p_dt = 0.f, p_ea = 0.f, p_bi = 0.f, p_bf = 0.f;
+  if (KIND == LINREC_MLSTM) { p_bi = a.gate_b[h]; p_bf = a.gate_b[a.H + h]; }
   if (KIND == LINREC_DELTA) {
 #pragma unroll
     for (int u = 0; u < 2; ++u)
@@ -185,6 +186,23 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     const int64_t row = row0 + t;
     const TP* pr = prow0 + (int64_t)t * a.ldp;
     float aa = 1.f, bb = 1.f, kq = 0.f, den = 1.f;
+    // what channel `tid` needs from this row, requested together
+    float x_a = 0.f, x_b = 0.f, x_v = 0.f, x_og = 0.f;
+    const int64_t vch = (int64_t)h * dv + j0 + tid;
+    const float gate0 = a.gates[row * a.ldg + h], gate1 = KIND == LINREC_MLSTM ? a.gates[row * a.ldg + a.H + h] : 0.f;
+    if (KIND == LINREC_DELTA) {
+      if (tid < dk && a.dec) x_a = a.dec[row * a.ldd + (int64_t)h * dk + tid];
+      if (tid < ncol && a.og) x_og = act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + vch);
+    } else {
+      if (tid < dk) {
+        x_a = act_load(pr + (int64_t)h * dk + tid);
+        x_b = act_load(pr + a.k_col + (int64_t)h * dk + tid);
+      }
+      if (tid < ncol) {
+        x_v = act_load(pr + a.v_col + vch);
+        x_og = act_load(reinterpret_cast<const TP*>(a.og) + row * a.ldo + vch);
+      }
+    }
     if (KIND == LINREC_DELTA) {
       // short convolution: channels q, k, v of this CTA spread over the block, four taps requested together (in a decode
       // step all but the newest come from the ring)
@@ -222,7 +240,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
         const int na = a.dec ? 0 : (int)a.ra;
         low[c] = act_round<TA>(act_load(pr + (c < na ? a.a1_col + c : a.g1_col + c - na)));
       }
-      bb = sigmoid_s(a.gates[row * a.ldg + h]);            // beta
+      bb = sigmoid_s(gate0);                                // beta
       __syncthreads();
       float q2 = 0.f, k2 = 0.f, qk = 0.f;
       for (int c = tid; c < dk; c += kT) {
@@ -239,19 +257,19 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
       for (int c = tid; c < dk; c += kT) {
         sq[c] *= rq; sk[c] *= rk;
         const int64_t ch = (int64_t)h * dk + c;
-        const float x = !LOW || a.dec ? a.dec[row * a.ldd + ch] : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
+        const float x = !LOW || a.dec ? (c == tid ? x_a : a.dec[row * a.ldd + ch]) : (low_a ? sg[c] : row_dot(a2 + ch * a.ra, low, a.ra));
         sg[c] = __expf(-p_ea * softplus_s(x + (c == tid ? p_dt : a.dt_bias[ch])));
       }
       const TA* g2 = reinterpret_cast<const TA*>(a.g2);
       const float* lg = low + (a.dec ? 0 : a.ra);
       for (int c = tid; c < ncol; c += kT) {
         const int64_t ch = (int64_t)h * dv + j0 + c;
-        const float x = !LOW || a.og ? act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
+        const float x = !LOW || a.og ? (c == tid ? x_og : act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch)) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
         sog[c] = sigmoid_s(x);
       }
     } else {
       const float rs = 1.f / sqrtf((float)dk);
-      const float zi = a.gates[row * a.ldg + h] + a.gate_b[h], zf = a.gates[row * a.ldg + a.H + h] + a.gate_b[a.H + h];
+      const float zi = gate0 + p_bi, zf = gate1 + p_bf;
       const float ig = a.cap * tanhf(zi / a.cap), fc = a.cap * tanhf(zf / a.cap);
       const float fg = -softplus_x(-fc);
       const float mn = fmaxf(fg + mrun, ig);
@@ -260,8 +278,8 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
       mrun = mn;
       float nq = 0.f, z1 = 0.f, z2 = 0.f;
       for (int c = tid; c < dk; c += kT) {
-        const float qc = act_round<TA>(act_load(pr + (int64_t)h * dk + c)) * rs;
-        const float kc = act_round<TA>(act_load(pr + a.k_col + (int64_t)h * dk + c)) * bb;
+        const float qc = act_round<TA>(c == tid ? x_a : act_load(pr + (int64_t)h * dk + c)) * rs;
+        const float kc = act_round<TA>(c == tid ? x_b : act_load(pr + a.k_col + (int64_t)h * dk + c)) * bb;
         sq[c] = qc; sk[c] = kc;
         const float nn = fmaf(aa, sg[c], kc);
         sg[c] = nn;
@@ -269,8 +287,8 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
       }
       for (int c = tid; c < ncol; c += kT) {
         const int64_t ch = (int64_t)h * dv + j0 + c;
-        sv[c] = act_round<TA>(act_load(pr + a.v_col + ch));
-        const float x = a.og ? act_load(reinterpret_cast<const TP*>(a.og) + row * a.ldo + ch) : 0.f;
+        sv[c] = act_round<TA>(c == tid ? x_v : act_load(pr + a.v_col + ch));
+        const float x = c == tid ? x_og : act_load(reinterpret_cast<const TP*>(a.og) + row * a.ldo + ch);
         sog[c] = sigmoid_s(x);
       }
       block_sum3(nq, z1, z2, red);

@@ -90,7 +90,7 @@ def _ensure_builtin() -> None:
 
 #: kernel sources a family needs; families without an entry use the whole library
 _KERNELS: dict[str, tuple[str, ...]] = {
-    "zufilorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemv.cu", "gemv_stream.cu", "gemm_f32.cu", "streams.cu",
+    "zufilorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "streams.cu",
                  "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
 }
 

@@ -428,3 +428,44 @@ def test_bad_batches_stop_on_the_host():
             m.forward_batch([item], [[]])
     with pytest.raises(ValueError):
         m.forward_batch([([1], 0, 0, [1]), ([2], 0, 0, [2])], [[], []])
+
+
+def test_serving_process_answers_with_the_plain_models_tokens(tmp_path):
+    """The resident engine process built from a checkpoint directory by the command line's own builder: greedy and
+    sampled requests, several at once."""
+    import threading
+    from coffin_b200.entrypoints.cli.runtime import build_server, parser
+    from coffin_b200.models.zufilorn.config import ZufilornConfig
+    from coffin_b200.serving.transport import call, serve
+    from coffin_b200.weights.init import save_checkpoint
+    cfg = Z.config([Z.mlstm(), Z.delta(), Z.attention()], vocab=300)
+    W = Z.weights(cfg, 19)
+    save_checkpoint(ZufilornConfig.from_hf(cfg), W, tmp_path / "model")
+    srv = build_server(parser().parse_args(["--serve", "--model", str(tmp_path / "model"), "--max-seq", "256", "--max-num-seqs", "4"]))
+    sock, ready = str(tmp_path / "s.sock"), threading.Event()
+    t = threading.Thread(target=serve, args=(srv, sock), kwargs={"ready": ready}, daemon=True)
+    t.start()
+    assert ready.wait(60)
+    try:
+        prompts = [toks(n, 256, n) for n in (20, 75, 3)]
+        reps = [None] * 3
+
+        def ask(i):
+            reps[i] = call(sock, {"op": "generate", "tokens": prompts[i], "max_new": 6, "ignore_eos": True})
+        threads = [threading.Thread(target=ask, args=(i,)) for i in range(3)]
+        for th in threads:
+            th.start()
+        for th in threads:
+            th.join(60)
+        for p, rep in zip(prompts, reps):
+            assert rep["ok"] and rep["n_new"] == 6
+            ids = list(p)
+            for tok in rep["tokens"]:                  # 16-bit: the token has to be among the plain model's near-best
+                lg = plain_logits(cfg, W, ids)[-1]
+                assert lg.max() - lg[tok] < 0.15 * lg.std(), rep["tokens"]
+                ids.append(tok)
+        warm = call(sock, {"op": "generate", "tokens": prompts[0], "max_new": 6, "temperature": 0.8, "seed": 3, "ignore_eos": True})
+        assert warm["ok"] and all(0 <= x < 300 for x in warm["tokens"])
+    finally:
+        call(sock, {"op": "stop"})
+        t.join(timeout=20)

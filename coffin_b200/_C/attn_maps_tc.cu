@@ -353,7 +353,7 @@ CB_EXPORT int cb_attn_maps_flash_tc_ok(int64_t dim, int64_t vdim) {
   return (dim == 64 || dim == 128 || dim == 256) && (vdim == 64 || vdim == 128 || vdim == 256);
 }
 
-// Prompt attention of `segs` segments of at most `max_rows` rows: the contract of cb_attn_maps_flash, on tcgen05.
+// Prompt attention of `segs` segments of at most `max_rows` rows on tcgen05; arguments as for cb_attn_maps_flash.
 // `slots`: rows of the pools.
 CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_rows, int64_t slots, void* status, void* stream) {
   if (!args || segs < 1 || segs > 65535 || max_rows < 1 || !status) return CB_ERR_ARG;

@@ -81,7 +81,7 @@ __device__ __forceinline__ int64_t block_index(int row0, int seg, int chunk) { r
 // ---- prep: delta -------------------------------------------------------------------------------
 constexpr int kPT = 128;
 template <int DK, int TAPS>
-__global__ void __launch_bounds__(kPT, 5) chunk_prep_delta_kernel(const ChunkArgs ca) {
+__global__ void __launch_bounds__(kPT, 7) chunk_prep_delta_kernel(const ChunkArgs ca) {
   using I = Image<LINREC_DELTA, DK>;
   constexpr int LD = DK + 4;
   const LinrecArgs& a = ca.r;

@@ -227,6 +227,13 @@ def preset(name: str) -> ModelConfig:
     raise KeyError(f"unknown preset {name!r}")
 
 
+def first_layers(cfg, n: int):
+    """``cfg`` cut to its first ``n`` layers (profiling workloads)."""
+    if hasattr(cfg, "first_layers"):
+        return cfg.first_layers(n)
+    return dataclasses.replace(cfg, num_hidden_layers=n, layer_types=cfg.layer_types[:n])
+
+
 PRESETS = ("tiny", "tiny-moe", "qwen35-4b", "qwen35-27b", "qwen35-35b-a3b")
 
 

@@ -109,6 +109,9 @@ class ZufilornConfig:
             if l.mixer.heads % kv:
                 raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
 
+    def first_layers(self, n: int) -> "ZufilornConfig":
+        return dataclasses.replace(self, layers=self.layers[:n])
+
     # ---- (de)serialisation
     @classmethod
     def from_hf(cls, raw: dict[str, Any], name: str = "checkpoint") -> "ZufilornConfig":
@@ -186,7 +189,7 @@ def preset_zufilorn(name: str) -> ZufilornConfig:
         big = name == "zufilorn-4b"
         W, H, A, ff, n, voc = (2560, 32, 16, 9216, 32, 151936) if big else (1280, 16, 8, 4608, 16, 65536)
         delta = (DELTA, DeltaMixer(H, H // 2, 128, 128, 4))
-        mem = (MLSTM, MLstmMixer(H // 2, 128, 256, 15.0))
-        att = (ATTENTION, AttentionMixer(A, A // 4, 128, 256, 128 ** -0.5, 20.0, 0.6, 0.1, 8192))
+        mem = (MLSTM, MLstmMixer(H // 2, 128, 256, 12.0))
+        att = (ATTENTION, AttentionMixer(A, A // 4, 128, 256, 128 ** -0.5, 30.0, 0.5, 0.1, 4096))
         return ZufilornConfig(voc, W, cycle(n, H, ff, (delta, mem, delta, att)), 2, 8192, name=name)
     raise KeyError(f"unknown preset {name!r}")

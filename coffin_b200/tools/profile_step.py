@@ -9,7 +9,6 @@ kernels have the full model's shapes while only ~2 GB is resident.
 from __future__ import annotations
 
 import argparse
-import dataclasses
 
 import torch
 
@@ -32,12 +31,12 @@ def main() -> None:
     import os
     if args.mega:
         os.environ["COFFIN_MEGA"] = "1"
-    from ..config import preset
+    from ..config import first_layers, preset
     from ..engine.llm import LLM
     from ..ops import kernels as K
     cfg = preset(args.model)
     if args.layers and args.layers < cfg.num_hidden_layers:
-        cfg = dataclasses.replace(cfg, num_hidden_layers=args.layers, layer_types=cfg.layer_types[:args.layers])
+        cfg = first_layers(cfg, args.layers)
     if args.tp_force or args.kv_dtype != "bf16":
         from ..models.qwen35.model import Qwen35Model
         from ..weights.init import random_state_dict

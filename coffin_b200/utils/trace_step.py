@@ -16,7 +16,6 @@ from __future__ import annotations
 import argparse
 import collections
 import ctypes
-import dataclasses
 import re
 
 import torch
@@ -136,7 +135,7 @@ def main() -> None:
     ap.add_argument("--mma-kcta", type=int, default=0, help="max CTAs sharing one 16-row GEMV block (1 = off)")
     ap.add_argument("--mma-prefetch", type=int, default=-1, help="GEMV sweep rounds prefetched into L2 before the wait")
     args = ap.parse_args()
-    from ..config import preset
+    from ..config import first_layers, preset
     from ..engine.llm import LLM
     from ..ops import _lib
     if args.mma_prefetch >= 0:
@@ -147,7 +146,7 @@ def main() -> None:
         _lib.call_nostream("set_mma_gemv_stage", args.mma_stage)
     cfg = preset(args.model)
     if args.layers and args.layers < cfg.num_hidden_layers:
-        cfg = dataclasses.replace(cfg, num_hidden_layers=args.layers, layer_types=cfg.layer_types[:args.layers])
+        cfg = first_layers(cfg, args.layers)
     import os
     world, rank = int(os.environ.get("WORLD_SIZE", "1")), int(os.environ.get("RANK", "0"))
     local = int(os.environ.get("LOCAL_RANK", "0"))

@@ -104,7 +104,7 @@ MIX = {
     "delta": Z.delta(), "delta_equal_heads": Z.delta(3, 3, 32, 32, 2), "delta_one_tap": Z.delta(2, 1, 8, 16, 1),
     "delta_wide": Z.delta(2, 1, 72, 64, 5), "delta_odd": Z.delta(2, 2, 10, 7, 3), "delta_128": Z.delta(2, 1, 128, 128, 4),
     "delta_256": Z.delta(1, 1, 256, 40, 4),
-    "mlstm": Z.mlstm(), "mlstm_wide": Z.mlstm(2, 64, 136, 15.0), "mlstm_odd": Z.mlstm(5, 9, 13, 3.0), "mlstm_one": Z.mlstm(1, 128, 256, 20.0),
+    "mlstm": Z.mlstm(), "mlstm_wide": Z.mlstm(2, 64, 136, 14.0), "mlstm_odd": Z.mlstm(5, 9, 13, 3.0), "mlstm_one": Z.mlstm(1, 128, 256, 20.0),
     "attn": Z.attention(), "attn_nocap": Z.attention(softcap=None, every=0), "attn_mqa": Z.attention(5, 1, 24, 16, every=7),
     "attn_equal": Z.attention(2, 2, 64, 128), "attn_wide": Z.attention(2, 1, 128, 256, scale=0.09), "attn_odd": Z.attention(3, 1, 6, 10),
     "attn_many": Z.attention(12, 1, 8, 8, scale=0.5),
@@ -156,7 +156,7 @@ def test_mixer_in_portions(name, dtype, cuts):
 
 
 @pytest.mark.parametrize("sizes", [(64, 64), (128, 256), (64, 128), (256, 64), (256, 256), (32, 64), (40, 96)])
-@pytest.mark.parametrize("cap", [None, 20.0, 60.0])
+@pytest.mark.parametrize("cap", [None, 18.0, 60.0])
 def test_prompt_attention_kernels_agree(sizes, cap):
     """tcgen05 (sizes of 64 / 128 / 256), mma.sync and the plain equations on prompts and long portions; peaky scores,
     so that the uncapped form raises its reference maximum again and again."""
@@ -178,7 +178,7 @@ def test_prompt_attention_kernels_agree(sizes, cap):
 @pytest.mark.parametrize("bias", [-12.0, 12.0])
 def test_mlstm_running_maximum_starts_at_zero(bias):
     """With input gates far below (above) zero the denominator's exp(-m) decides the first tokens."""
-    layer = Z.mlstm(2, 16, 24, 15.0)
+    layer = Z.mlstm(2, 16, 24, 13.0)
     cfg = Z.config([layer], width=64, ff=None)
     W = Z.weights(cfg, 5)
     W["l0.mix.i.b"] = torch.full_like(W["l0.mix.i.b"], bias)

@@ -9,55 +9,11 @@ from __future__ import annotations
 import torch
 
 from ...ops import mixers as X
+from ..rowmodel import Mixer, Projection, pad8, padded
 from .config import AttentionMixer, DeltaMixer, MLstmMixer
 
 
-def pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-class Projection:
-    """Row-concatenated projections of one input.  Sections start at multiples of 8 columns (16-byte tiles); ``main``
-    holds the activations, ``gate`` the columns whose result stays fp32 (gates of a recurrence, head gates)."""
-
-    def __init__(self, parts: dict[str, torch.Tensor], gates: dict[str, torch.Tensor], width: int, dtype, device) -> None:
-        self.col: dict[str, int] = {}
-        rows = []
-
-        def add(t: torch.Tensor) -> None:
-            w = torch.zeros(pad8(t.shape[0]), pad8(width), dtype=dtype, device=device)
-            w[:t.shape[0], :t.shape[1]] = t.to(device, dtype)
-            rows.append(w)
-
-        n = 0
-        for name, t in parts.items():
-            self.col[name] = n
-            add(t)
-            n += pad8(t.shape[0])
-        self.n_main = n
-        if gates:
-            add(torch.cat([t.to(device, dtype) for t in gates.values()]))
-        self.w = torch.cat(rows).contiguous()
-        self.n = self.w.shape[0]
-        self.main, self.gate = self.w[:self.n_main], self.w[self.n_main:]
-
-
-class _Mixer:
-    #: named state tensors ``[slots, ...]`` that travel with a sequence; paged pools are separate
-    state: dict[str, torch.Tensor]
-    pools: tuple[torch.Tensor, ...] = ()
-
-    def weights(self):
-        return [self.proj.w, self.w_out]
-
-
-def _padded(t: torch.Tensor, rows: int, cols: int, dtype, dev) -> torch.Tensor:
-    out = torch.zeros(rows, cols, dtype=dtype, device=dev)
-    out[:t.shape[0], :t.shape[1]] = t.to(dev, dtype)
-    return out
-
-
-class ChannelDelta(_Mixer):
+class ChannelDelta(Mixer):
     def __init__(self, m: DeltaMixer, W: dict[str, torch.Tensor], width: int, eps: float, slots: int, dtype, dev) -> None:
         self.m = m
         H, G, d, e = m.heads, m.kv_heads, m.dim, m.vdim
@@ -71,10 +27,10 @@ class ChannelDelta(_Mixer):
             t = W[n + ".conv"]
             conv[col[n]:col[n] + t.shape[0]] = f32(t)
         ra, rg = pad8(W["a1"].shape[0]), pad8(W["g1"].shape[0])
-        self.a2 = _padded(W["a2"], pad8(H * d), ra, dtype, dev)
-        self.g2 = _padded(W["g2"], pad8(H * e), rg, dtype, dev)
+        self.a2 = padded(W["a2"], pad8(H * d), ra, dtype, dev)
+        self.g2 = padded(W["g2"], pad8(H * e), rg, dtype, dev)
         self.ra, self.rg = ra, rg
-        self.w_out = _padded(W["o"], pad8(width), pad8(H * e), dtype, dev)
+        self.w_out = padded(W["o"], pad8(width), pad8(H * e), dtype, dev)
         depth = X.RING
         while depth < taps:
             depth *= 2
@@ -102,13 +58,13 @@ class ChannelDelta(_Mixer):
         return act
 
 
-class MLstm(_Mixer):
+class MLstm(Mixer):
     def __init__(self, m: MLstmMixer, W: dict[str, torch.Tensor], width: int, eps: float, slots: int, dtype, dev) -> None:
         self.m = m
         H, d, e = m.heads, m.dim, m.vdim
         self.proj = Projection({n: W[n] for n in ("q", "k", "v", "g")}, {"i": W["i"], "f": W["f"]}, width, dtype, dev)
         col = self.proj.col
-        self.w_out = _padded(W["o"], pad8(width), pad8(H * e), dtype, dev)
+        self.w_out = padded(W["o"], pad8(width), pad8(H * e), dtype, dev)
         self.state = {"S": torch.zeros(slots, H, d, e, dtype=torch.float32, device=dev),
                       "n": torch.zeros(slots, H, d, dtype=torch.float32, device=dev),
                       "m": torch.zeros(slots, H, dtype=torch.float32, device=dev)}
@@ -125,7 +81,7 @@ class MLstm(_Mixer):
         return act
 
 
-class DiffAttention(_Mixer):
+class DiffAttention(Mixer):
     MAPS = 2
 
     def __init__(self, m: AttentionMixer, W: dict[str, torch.Tensor], width: int, eps: float, num_blocks: int, page: int, dtype, dev) -> None:
@@ -133,7 +89,7 @@ class DiffAttention(_Mixer):
         H, G, d, e = m.heads, m.kv_heads, m.dim, m.vdim
         self.proj = Projection({n: W[n] for n in ("q", "k", "v")}, {"g": W["g"]}, width, dtype, dev)
         col = self.proj.col
-        self.w_out = _padded(W["o"], pad8(width), pad8(H * e), dtype, dev)
+        self.w_out = padded(W["o"], pad8(width), pad8(H * e), dtype, dev)
         lq1, lk1, lq2, lk2 = (W[n].float() for n in ("lq1", "lk1", "lq2", "lk2"))
         self.lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + m.diff
         kpool = torch.zeros(num_blocks * page, G * self.MAPS, d, dtype=dtype, device=dev)

@@ -24,29 +24,9 @@ import torch
 
 from ...ops import kernels as K
 from ...ops import mixers as X
+from ..rowmodel import RowBatch, RowModel, pad8, padded
 from .config import ATTENTION, DELTA, ZufilornConfig
-from .mixers import ChannelDelta, DiffAttention, MLstm, pad8, _padded
-
-BUCKETS = (1, 2, 4, 8, 16, 32, 64)
-
-
-@dataclasses.dataclass
-class RowBatch:
-    """Rows of one forward.  Segments ``0 .. n_pre - 1`` are portions of several tokens, the others one token each; the
-    rows of a segment are consecutive and segments are in row order."""
-    T: int
-    n_seg: int
-    n_pre: int                      # leading segments with more than one row
-    pre_rows: int                   # rows of those segments
-    tokens: torch.Tensor            # int64 [T]
-    positions: torch.Tensor         # int32 [T], -1: padding
-    row_seg: torch.Tensor | None    # int32 [T]; None: row r is segment r
-    seg_row: torch.Tensor | None    # int32 [n_seg + 1]
-    seg_pos: torch.Tensor           # int32 [n_seg]
-    seg_slot: torch.Tensor          # int32 [n_seg]
-    tables: torch.Tensor            # int32 [n_seg, pages]
-    max_rows: int = 1               # longest segment
-    max_len: int = 0                # largest position + 1 (0: unknown, inside a graph)
+from .mixers import ChannelDelta, DiffAttention, MLstm
 
 
 @dataclasses.dataclass
@@ -60,34 +40,19 @@ class _Layer:
     w_gu: torch.Tensor | None = None
     w_down: torch.Tensor | None = None
 
+    def ff_weights(self) -> list[torch.Tensor]:
+        return [self.w_gu, self.w_down] if self.w_gu is not None else []
 
-class ZufilornModel:
-    mixed_batches = True            # portions of prompts and single tokens share a forward
+
+class ZufilornModel(RowModel):
+    family = "Zufilorn"
 
     def __init__(self, cfg: ZufilornConfig, sd: dict[str, torch.Tensor], device: str | torch.device = "cuda", max_seq: int = 4096,
                  num_slots: int = 2, num_blocks: int | None = None, max_chunk: int = 2048, pdl: bool = True,
                  dtype: torch.dtype = torch.bfloat16, free_source: bool = False, quant: str = "none", kv_dtype: str = "bf16") -> None:
-        if quant != "none" or kv_dtype != "bf16":
-            raise NotImplementedError("the Zufilorn family has 16-bit (or fp32) weights and pages only")
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"dtype {dtype}: expected bfloat16 or float32")
-        self.cfg = c = cfg
-        self.dtype, self.f32 = dtype, dtype == torch.float32
-        self.device = dev = torch.device(device)
-        self.max_seq = min(int(max_seq), c.max_positions)
-        self.num_slots, self.max_chunk = int(num_slots), int(max_chunk)
-        self.max_blocks_per_seq = (self.max_seq + K.BLOCK - 1) // K.BLOCK
-        self.num_blocks = int(num_blocks) if num_blocks else self.max_blocks_per_seq * self.num_slots + 1
-        self.eps = c.rms_norm_eps
-        self.tp_world = 1
-        K.status_word(dev)
-        K._lib.set_pdl(pdl)
-        for name, shape, _ in c.tensor_plan():
-            if name not in sd:
-                raise KeyError(f"checkpoint lacks {name}")
-            # the rank of the low-rank projections is the tensors' own
-            if tuple(sd[name].shape) != shape and name.rpartition(".")[2] not in ("a1", "a2", "g1", "g2"):
-                raise ValueError(f"{name}: shape {tuple(sd[name].shape)}, config.json gives {shape}")
+        self._setup(cfg, sd, device, min(int(max_seq), cfg.max_positions), num_slots, num_blocks, max_chunk, pdl, dtype, quant, kv_dtype,
+                    free_shape=("a1", "a2", "g1", "g2"))   # the rank of the low-rank projections is the tensors' own
+        c, dev = self.cfg, self.device
 
         def take(name: str) -> torch.Tensor:
             return sd.pop(name) if free_source else sd[name]
@@ -97,7 +62,6 @@ class ZufilornModel:
         W = c.hidden_size
         self.embed = take("embed").to(dev, dtype).contiguous()
         self.pos = take("pos").to(dev, dtype).contiguous()
-        self.layers: list[_Layer] = []
         for i, spec in enumerate(c.layers):
             p = f"l{i}."
             mw = {k[len(p) + 4:]: take(k) for k in [k for k in sd if k.startswith(p + "mix.")]}
@@ -110,124 +74,13 @@ class ZufilornModel:
             if spec.ff is not None:
                 L.gain2, L.hc2 = gain(p + "norm2"), hc("hc2")
                 I, W8 = pad8(spec.ff), pad8(W)
-                L.w_gu = torch.cat([_padded(take(p + "mlp.gate"), I, W8, dtype, dev), _padded(take(p + "mlp.up"), I, W8, dtype, dev)])
-                L.w_down = _padded(take(p + "mlp.down"), W8, I, dtype, dev)
+                L.w_gu = torch.cat([padded(take(p + "mlp.gate"), I, W8, dtype, dev), padded(take(p + "mlp.up"), I, W8, dtype, dev)])
+                L.w_down = padded(take(p + "mlp.down"), W8, I, dtype, dev)
             self.layers.append(L)
         self.final_gain = gain("final.norm")
-        self.head = _padded(take("head"), pad8(c.vocab_size), pad8(W), dtype, dev)
-        self._bufs: dict = {}
-        self._rows: dict[int, dict] = {}
-        self._graphs: dict = {}
-        self._step_launches: dict[int, int] = {}
-        self.graph_pool = None
-        self._advance = False
-        self.layer_hook = None          # debugging: called as hook(layer index, sum of the streams [rows, W]) after every layer
+        self.head = padded(take("head"), pad8(c.vocab_size), pad8(W), dtype, dev)
 
-    # ------------------------------------------------------------------ bookkeeping
-    def weight_bytes(self) -> int:
-        """Bytes of weights one decode step streams."""
-        ts = [self.head]
-        for L in self.layers:
-            ts += L.mixer.weights() + ([L.w_gu, L.w_down] if L.w_gu is not None else [])
-        return sum(t.numel() * t.element_size() for t in ts)
-
-    def launches_per_step(self, M: int) -> int:
-        return self._step_launches.get(M, 0)
-
-    @staticmethod
-    def bucket_for(n: int) -> int:
-        for m in BUCKETS:
-            if n <= m:
-                return m
-        raise ValueError(f"{n} rows exceed the largest decode bucket {BUCKETS[-1]}")
-
-    @property
-    def max_decode_rows(self) -> int:
-        return BUCKETS[-1]
-
-    def poll_status(self) -> None:
-        K.poll_status()
-
-    def check_status(self) -> None:
-        K.raise_on_status()
-
-    def sample(self, logits: torch.Tensor, temps, us) -> torch.Tensor:
-        if temps is None:
-            return K.argmax(logits.contiguous())
-        t = torch.tensor(temps, dtype=torch.float32, device=self.device)
-        u = torch.tensor(us, dtype=torch.float32, device=self.device)
-        return K.sample(logits.contiguous(), t, u)
-
-    def embed_tokens(self, tokens: torch.Tensor) -> torch.Tensor:
-        return self.embed.index_select(0, tokens)
-
-    # ------------------------------------------------------------------ sequence state
-    def zero_state(self, slot: int) -> None:
-        for L in self.layers:
-            for t in L.mixer.state.values():
-                t[slot].zero_()
-
-    def snapshot_state(self, slot: int) -> list[torch.Tensor]:
-        return [t[slot].clone() for L in self.layers for t in L.mixer.state.values()]
-
-    def restore_state(self, slot: int, snap: list[torch.Tensor]) -> None:
-        it = iter(snap)
-        for L in self.layers:
-            for t in L.mixer.state.values():
-                t[slot].copy_(next(it))
-
-    def copy_block(self, src: int, dst: int) -> None:
-        s, d = src * K.BLOCK, dst * K.BLOCK
-        for L in self.layers:
-            for pool in L.mixer.pools:
-                pool[d:d + K.BLOCK].copy_(pool[s:s + K.BLOCK])
-
-    # ------------------------------------------------------------------ workspaces and products
-    def buf(self, name: str, rows: int, cols: int, dtype: torch.dtype | None = None) -> torch.Tensor:
-        """Scratch ``[rows, cols]``, contiguous.  Buffers of a name and width are zero when first handed out and padding
-        columns are never written, so a product over the padded width adds nothing.  Sizes of the decode buckets
-        have buffers of their own (fixed addresses inside CUDA graphs); larger batches share one that grows."""
-        dtype = dtype or self.dtype
-        small = rows if rows in BUCKETS else 0
-        key = (name, cols, dtype, small)
-        t = self._bufs.get(key)
-        if t is None or t.shape[0] < rows:
-            cap = small or max(rows, min(self.max_chunk, 256))
-            t = self._bufs[key] = torch.zeros(cap, cols, dtype=dtype, device=self.device)
-        return t[:rows]
-
-    def _scratch(self, floats: int) -> torch.Tensor:
-        """Untyped scratch of the chunked recurrences (grows; stream-ordered reuse)."""
-        t = self._bufs.get("scratch")
-        if t is None or t.numel() < floats:
-            t = self._bufs["scratch"] = torch.empty(floats, dtype=torch.float32, device=self.device)
-        return t
-
-    def linear(self, W: torch.Tensor, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-        """``out = x @ W^T``; the result type is ``out``'s."""
-        T, Kd = x.shape
-        if self.f32:
-            return X.gemm_f32(x, W, out)
-        if T <= 8 and T * Kd * 2 <= 160 * 1024:
-            return K.gemv(W, x.contiguous(), out)
-        if out.dtype == torch.float32:
-            return X.gemm_f32out(x, W, out)
-        return K.gemm(x, W, out=out)
-
-    def project(self, P, h: torch.Tensor, b: RowBatch) -> tuple[torch.Tensor, torch.Tensor]:
-        """``(main, gates)`` of an input projection: one fp32 product for few rows (and in 32-bit mode), else the main
-        columns in the activation type and the gate columns fp32."""
-        T = b.T
-        if self.f32 or T <= 8:
-            y = self.buf("proj32", T, P.n, torch.float32)
-            self.linear(P.w, h, y)
-            return y[:, :P.n_main], y[:, P.n_main:]
-        main = self.buf("proj", T, P.n_main)
-        self.linear(P.main, h, main)
-        gates = self.buf("gates", T, P.gate.shape[0], torch.float32)
-        self.linear(P.gate, h, gates)
-        return main, gates
-
+    # ------------------------------------------------------------------ sublayers
     def feed_forward(self, L: _Layer, h: torch.Tensor, T: int) -> torch.Tensor:
         I = L.w_down.shape[1]
         inter = self.buf("inter", T, I)
@@ -241,20 +94,6 @@ class ZufilornModel:
         else:
             K.swiglu(K.gemm(h, L.w_gu, out=self.buf("gu", T, 2 * I)), out=inter)
         return self.linear(L.w_down, inter, y)
-
-    # ------------------------------------------------------------------ mixer cores
-    def recur(self, core: X.Linrec, b: RowBatch, proj, gates, og, act, dec) -> None:
-        n0 = 0
-        if b.n_pre and proj.dtype == torch.bfloat16 and core.chunked:
-            need = (core.chunk_scratch(b.pre_rows, b.n_pre) + 3) // 4
-            core.chunk(proj, gates, og, act, b.seg_row, b.seg_pos, b.seg_slot, self._scratch(need), segs=b.n_pre, max_rows=b.max_rows,
-                       rows=b.pre_rows, dec=dec)
-            n0 = b.n_pre
-        if n0 < b.n_seg:
-            core.step(proj, gates, og, act, b.seg_pos[n0:], b.seg_slot[n0:], segs=b.n_seg - n0,
-                      seg_row=b.seg_row[n0:] if b.seg_row is not None else None, dec=dec)
-        if b.n_pre:
-            core.ring(proj, b.seg_row, b.seg_pos, b.seg_slot, b.n_pre)
 
     def attend(self, core: X.AttnMaps, b: RowBatch, proj, gates, act, *, lam: float, post_scale: float) -> None:
         vh, T, P = core.H * core.maps, b.T, b.pre_rows
@@ -312,195 +151,6 @@ class ZufilornModel:
                 self.layer_hook(li, x.sum(1))
         return x, pend
 
-    def _logits(self, x: torch.Tensor, pend: dict, rows: torch.Tensor | None, n: int, out: torch.Tensor) -> torch.Tensor:
-        """fp32 logits of ``n`` stream rows (``rows`` None: the first n) into ``out [n, padded vocab]``."""
-        h = self.buf("h_out", n, pad8(self.cfg.hidden_size))
+    def _out_rows(self, state, rows, n, h) -> None:
+        x, pend = state
         X.streams_step(x, h, gain=self.final_gain, rows=rows, store=False, eps=self.eps, **pend)
-        return self.linear(self.head, h, out)
-
-    # ------------------------------------------------------------------ batches of portions and tokens
-    def _check_row(self, pos0: int, n: int, table_len: int, slot: int) -> None:
-        """Everything a kernel indexes with a position or a slot is checked here, on the host."""
-        end = pos0 + n
-        if n < 1 or pos0 < 0 or end > self.max_seq or end > table_len * K.BLOCK or table_len > self.max_blocks_per_seq:
-            raise ValueError(f"positions {pos0}..{end - 1} outside the block table ({table_len} blocks) or the {self.max_seq}-token window")
-        if not 0 <= slot < self.num_slots:
-            raise ValueError(f"state slot {slot} outside 0..{self.num_slots - 1}")
-
-    def make_batch(self, items: list[tuple]) -> tuple[RowBatch, list[int], list[int]]:
-        """``items[i] = (tokens, pos0, slot, block_table)``.  Returns the batch, the segment order (item index per
-        segment: portions before single tokens) and the first row of every ITEM."""
-        toks = [t.tolist() if isinstance(t, torch.Tensor) else list(t) for t, *_ in items]
-        tabs = [t.tolist() if isinstance(t, torch.Tensor) else list(t) for *_, t in items]
-        for tk, (_, pos0, slot, _t), tb in zip(toks, items, tabs):
-            self._check_row(int(pos0), len(tk), len(tb), int(slot))
-            if any(not 0 <= b_ < self.num_blocks for b_ in tb):
-                raise ValueError("block table names a block outside the pool")
-        if len({int(it[2]) for it in items}) != len(items):
-            raise ValueError("two entries of a batch share a state slot")
-        order = sorted(range(len(items)), key=lambda i: len(toks[i]) == 1)
-        n_seg, T = len(items), sum(len(t) for t in toks)
-        n_pre = sum(len(t) > 1 for t in toks)
-        pages = max(len(t) for t in tabs)
-        host = torch.zeros(2 * T + (n_seg + 1) + 2 * n_seg + n_seg * pages, dtype=torch.int32)
-        if self.device.type == "cuda":
-            host = host.pin_memory()
-        positions, row_seg = host[:T], host[T:2 * T]
-        o = 2 * T
-        seg_row, seg_pos, seg_slot = host[o:o + n_seg + 1], host[o + n_seg + 1:o + 2 * n_seg + 1], host[o + 2 * n_seg + 1:o + 3 * n_seg + 1]
-        tables = host[o + 3 * n_seg + 1:].view(n_seg, pages)
-        first = [0] * len(items)
-        r, flat = 0, []
-        for s, i in enumerate(order):
-            n, pos0 = len(toks[i]), int(items[i][1])
-            first[i] = r
-            positions[r:r + n] = torch.arange(pos0, pos0 + n, dtype=torch.int32)
-            row_seg[r:r + n] = s
-            seg_row[s], seg_pos[s], seg_slot[s] = r, pos0, int(items[i][2])
-            tables[s, :len(tabs[i])] = torch.tensor(tabs[i], dtype=torch.int32)
-            flat += toks[i]
-            r += n
-        seg_row[n_seg] = r
-        tok = torch.tensor(flat, dtype=torch.int64)
-        if self.device.type == "cuda":
-            tok = tok.pin_memory()
-        dev = host.to(self.device, non_blocking=True)
-        b = RowBatch(T=T, n_seg=n_seg, n_pre=n_pre, pre_rows=T - (n_seg - n_pre), tokens=tok.to(self.device, non_blocking=True),
-                     positions=dev[:T], row_seg=dev[T:2 * T], seg_row=dev[o:o + n_seg + 1], seg_pos=dev[o + n_seg + 1:o + 2 * n_seg + 1],
-                     seg_slot=dev[o + 2 * n_seg + 1:o + 3 * n_seg + 1], tables=dev[o + 3 * n_seg + 1:].view(n_seg, pages),
-                     max_rows=max(len(t) for t in toks), max_len=max(int(it[1]) + len(t) for it, t in zip(items, toks)))
-        return b, order, first
-
-    @torch.no_grad()
-    def forward_batch(self, items: list[tuple], want: list[list[int]]) -> torch.Tensor | None:
-        """One forward over portions and single tokens of several sequences.  ``want[i]``: places among the tokens of
-        item ``i`` whose logits are wanted; returns fp32 ``[wanted, vocab]`` in the order of the items (None: none)."""
-        b, _order, first = self.make_batch(items)
-        x, pend = self._stack(b)
-        rows = [first[i] + int(p) for i, ps in enumerate(want) for p in ps]
-        if not rows:
-            return None                 # the last write-back feeds nothing
-        V8 = self.head.shape[0]
-        out = torch.empty(len(rows), V8, dtype=torch.float32, device=self.device)
-        idx = torch.tensor(rows, dtype=torch.int32).to(self.device)
-        self._logits(x, pend, idx, len(rows), out)
-        return out[:, :self.cfg.vocab_size]
-
-    @torch.no_grad()
-    def prefill_group(self, items: list[tuple], want_logits: list[bool] | None = None) -> list:
-        """Portions of several sequences in one forward; per item the logits ``[vocab]`` of its last token or None."""
-        want_logits = list(want_logits) if want_logits is not None else [True] * len(items)
-        out = self.forward_batch(items, [[int(len(it[0])) - 1] if w else [] for it, w in zip(items, want_logits)])
-        rows = iter(out if out is not None else ())
-        return [next(rows) if w else None for w in want_logits]
-
-    def prefill(self, tokens, pos0: int, slot: int, block_table, embeds=None, cos_sin=None, want_logits: bool = True):
-        if embeds is not None or cos_sin is not None:
-            raise ValueError("this family takes token ids only")
-        return self.prefill_group([(tokens, pos0, slot, block_table)], [want_logits])[0]
-
-    # ------------------------------------------------------------------ decode
-    def _row_buffers(self, M: int) -> dict:
-        b = self._rows.get(M)
-        if b is None:
-            dev = self.device
-            i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)
-            pin = (lambda t: t.pin_memory()) if dev.type == "cuda" else (lambda t: t)
-            b = self._rows[M] = {
-                "tokens": torch.zeros(M, dtype=torch.int64, device=dev), "positions": i32(M).fill_(-1), "rope_pos": i32(M),
-                "slots": i32(M).fill_(-1), "block_table": i32(M, self.max_blocks_per_seq),
-                "logits8": torch.zeros(M, self.head.shape[0], dtype=torch.float32, device=dev),
-                "next": torch.zeros(M, dtype=torch.int64, device=dev),
-                "h_tokens": pin(torch.zeros(M, dtype=torch.int64)), "h_meta": pin(torch.zeros(2, M, dtype=torch.int32)),
-                "h_bt": pin(torch.zeros(M, self.max_blocks_per_seq, dtype=torch.int32))}
-            b["logits"] = b["logits8"][:, :self.cfg.vocab_size]
-        return b
-
-    def set_rows(self, M: int, tokens, positions, slots, block_tables, rope_deltas=None) -> None:
-        """Stage up to ``M`` single tokens; missing rows are padding."""
-        b, n = self._row_buffers(M), len(tokens)
-        if n > M:
-            raise ValueError(f"{n} rows do not fit bucket {M}")
-        for r in range(n):
-            self._check_row(positions[r], 1, len(block_tables[r]), slots[r])
-        ev = b.get("h_event")
-        if ev is None:
-            ev = b["h_event"] = torch.cuda.Event()
-        else:
-            ev.synchronize()            # the pinned arrays are reused: the copies of the previous call have to have left them
-        ht, hm, hb = b["h_tokens"], b["h_meta"], b["h_bt"]
-        ht.zero_()
-        hm.fill_(-1)
-        for r in range(n):
-            ht[r], hm[0, r], hm[1, r] = int(tokens[r]), int(positions[r]), int(slots[r])
-            hb[r, :len(block_tables[r])] = torch.as_tensor(block_tables[r], dtype=torch.int32)
-        for dst, src in (("tokens", ht), ("positions", hm[0]), ("slots", hm[1]), ("block_table", hb)):
-            b[dst].copy_(src, non_blocking=True)
-        ev.record()
-
-    def _decode_body(self, M: int) -> None:
-        rb = self._row_buffers(M)
-        b = RowBatch(T=M, n_seg=M, n_pre=0, pre_rows=0, tokens=rb["tokens"], positions=rb["positions"], row_seg=None, seg_row=None,
-                     seg_pos=rb["positions"], seg_slot=rb["slots"], tables=rb["block_table"])
-        x, pend = self._stack(b)
-        self._logits(x, pend, None, M, rb["logits8"])
-        K.argmax(rb["logits"], rb["next"])
-        if self._advance:
-            self.advance_rows(M)
-
-    def advance_rows(self, M: int) -> None:
-        """Feed the sampled tokens back and advance the positions (no host synchronisation)."""
-        b = self._row_buffers(M)
-        K.call("advance_rows", b["tokens"], b["next"], b["positions"], b["rope_pos"], M)
-        K._count()
-
-    def _gkey(self, M: int, advance: bool):
-        return (M, bool(advance))
-
-    def capture(self, M: int, warmup: int = 2, advance: bool = False) -> None:
-        """Capture the step of bucket ``M`` into a CUDA graph; warm-up runs on padding rows and touches no state."""
-        key = self._gkey(M, advance)
-        if key in self._graphs:
-            return
-        b = self._row_buffers(M)
-        saved = {k: b[k].clone() for k in ("positions", "slots", "tokens")}
-        b["positions"].fill_(-1)
-        b["slots"].fill_(-1)
-        self._advance = bool(advance)
-        try:
-            s = torch.cuda.Stream(device=self.device)
-            s.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(s), torch.no_grad():
-                for _ in range(warmup):
-                    self._decode_body(M)
-            torch.cuda.current_stream().wait_stream(s)
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            if self.graph_pool is None:
-                self.graph_pool = torch.cuda.graph_pool_handle()
-            l0 = K.LAUNCHES
-            with K.capture_graph(g, pool=self.graph_pool), torch.no_grad():
-                self._decode_body(M)
-            self._step_launches[M] = K.LAUNCHES - l0
-            self._graphs[key] = g
-        finally:
-            self._advance = False
-        for k, v in saved.items():
-            b[k].copy_(v)
-
-    @torch.no_grad()
-    def decode(self, M: int, graph: bool = True, advance: bool = False) -> tuple[torch.Tensor, torch.Tensor]:
-        """One token for every staged row: ``(next_tokens [M], logits [M, vocab])``, overwritten by the next step."""
-        b = self._row_buffers(M)
-        if graph:
-            key = self._gkey(M, advance)
-            if key not in self._graphs:
-                self.capture(M, advance=advance)
-            self._graphs[key].replay()
-        else:
-            self._advance = bool(advance)
-            try:
-                self._decode_body(M)
-            finally:
-                self._advance = False
-        return b["next"], b["logits"]

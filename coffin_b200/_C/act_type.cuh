@@ -37,5 +37,12 @@ __device__ __forceinline__ float softplus_s(float x) {
   p = fmaf(p, q, 0.2f); p = fmaf(p, q, 1.f / 3.f); p = fmaf(p, q, 1.f);
   return fmaxf(x, 0.f) + 2.f * s * p;
 }
+// xIELU: a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise (_x: full precision)
+__device__ __forceinline__ float xielu_s(float z, float a, float b) {
+  return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (__expf(fminf(z, 0.f)) - 1.f - z));
+}
+__device__ __forceinline__ float xielu_x(float z, float a, float b) {
+  return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (expm1f(fminf(z, 0.f)) - z));
+}
 __device__ __forceinline__ float sigmoid_s(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 __device__ __forceinline__ float silu_s(float x) { return x * sigmoid_s(x); }

@@ -14,8 +14,8 @@ __global__ void __launch_bounds__(256) maps_append_kernel(const AttnMapsArgs a) 
   const int64_t slot = (int64_t)a.tables[(int64_t)seg * a.ldbt + pos / kPage] * kPage + pos % kPage;
   const TP* p = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
   const int nk = a.G * a.maps * a.dim, nv = a.G * a.vdim;
-  TA* kp = reinterpret_cast<TA*>(a.kpool) + slot * nk;
-  TA* vp = reinterpret_cast<TA*>(a.vpool) + slot * nv;
+  TA* kp = reinterpret_cast<TA*>(a.kpool) + slot * pool_ldk(a);
+  TA* vp = reinterpret_cast<TA*>(a.vpool) + slot * pool_ldv(a);
   for (int c = threadIdx.x; c < nk; c += 256) act_store(kp + c, act_load(p + a.k_col + c));
   for (int c = threadIdx.x; c < nv; c += 256) act_store(vp + c, act_load(p + a.v_col + c));
 }
@@ -42,7 +42,7 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
   for (int c = tid; c < a.dim; c += kRT) q[c] = act_round<TA>(act_load(qr + c)) * f;
   for (int c = tid; c < a.vdim; c += kRT) o[c] = 0.f;
   __syncthreads();
-  const int64_t ldk = (int64_t)a.G * a.maps * a.dim, ldv = (int64_t)a.G * a.vdim;
+  const int64_t ldk = pool_ldk(a), ldv = pool_ldv(a);
   const TA* K = reinterpret_cast<const TA*>(a.kpool) + (int64_t)(g * a.maps + map) * a.dim;
   const TA* V = reinterpret_cast<const TA*>(a.vpool) + (int64_t)g * a.vdim;
   const int* bt = a.tables + (int64_t)seg * a.ldbt;

@@ -19,9 +19,15 @@ struct AttnMapsArgs {
   int H, G, maps, dim, vdim, nsplit;
   float scale, cap;                      // cap <= 0: no cap
   float temp_coef; int temp_every;       // temp_every <= 0: no temperature
+  int64_t ldk, ldv;                      // row strides of the pools (0: dense, G * maps * dim and G * vdim)
+  // one map, prompt kernels: the finished head (divided by its denominator, times sigmoid(gate)) goes straight to
+  // bf16 rows instead of part_o / part_ml (null: no)
+  void* act; int64_t lda; const float* gates; int64_t ldg;
 };
 
 constexpr int kPage = 64;
+__host__ __device__ __forceinline__ int64_t pool_ldk(const AttnMapsArgs& a) { return a.ldk ? a.ldk : (int64_t)a.G * a.maps * a.dim; }
+__host__ __device__ __forceinline__ int64_t pool_ldv(const AttnMapsArgs& a) { return a.ldv ? a.ldv : (int64_t)a.G * a.vdim; }
 
 __device__ __forceinline__ float query_temp(const AttnMapsArgs& a, int pos) {
   return a.temp_every > 0 ? 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1)) : 1.f;

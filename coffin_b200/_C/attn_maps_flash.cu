@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
   const int t0 = tile * kBM;
   if (t0 >= n) return;
   const int h = vh / a.maps, map = vh % a.maps, g = h / (a.H / a.G);
-  const int64_t ldk = (int64_t)a.G * a.maps * a.dim, ldv = (int64_t)a.G * a.vdim;
+  const int64_t ldk = pool_ldk(a), ldv = pool_ldv(a);
   const bf16* K = reinterpret_cast<const bf16*>(a.kpool) + (int64_t)(g * a.maps + map) * a.dim;
   const bf16* V = reinterpret_cast<const bf16*>(a.vpool) + (int64_t)g * a.vdim;
   const int* bt = a.tables + (int64_t)seg * a.ldbt;
@@ -196,6 +196,17 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
     den[i] += __shfl_xor_sync(0xffffffffu, den[i], 2);
     const int r = rlo + 8 * i;
     if (r >= rows) continue;
+    if (a.act) {                                                 // one map: the head is finished here
+      const int64_t row = row0 + t0 + r;
+      const float s = (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / den[i];
+      bf16* out = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * a.vdim;
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int c = v * 8 + t4 * 2;
+        if (c < a.vdim) *reinterpret_cast<uint32_t*>(out + c) = pack_bf162(o[v][2 * i] * s, o[v][2 * i + 1] * s);
+      }
+      continue;
+    }
     const int64_t idx = ((int64_t)(row0 + t0 + r) * a.H * a.maps + vh) * a.nsplit;
     float* po = a.part_o + idx * a.vdim;
 #pragma unroll
@@ -260,7 +271,7 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
     return;
   }
   const int* bt = a.tables + (int64_t)seg * a.ldbt;
-  const int64_t ldk = (int64_t)a.G * MAPS * a.dim, ldv = (int64_t)a.G * a.vdim;
+  const int64_t ldk = pool_ldk(a), ldv = pool_ldv(a);
   bf16* K = reinterpret_cast<bf16*>(a.kpool) + (int64_t)g * MAPS * a.dim;
   bf16* V = reinterpret_cast<bf16*>(a.vpool) + (int64_t)g * a.vdim;
   const TP* pr = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
@@ -433,9 +444,9 @@ CB_EXPORT int cb_attn_maps_tc_ok(int64_t G, int64_t maps, int64_t dim, int64_t v
 CB_EXPORT int cb_attn_maps_flash(const void* args, int64_t segs, int64_t max_rows, void* stream) {
   if (!args || segs < 1 || segs > 65535 || max_rows < 1) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
-  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G)
-    return CB_ERR_ARG;
-  if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8) return CB_ERR_SHAPE;
+  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G) return CB_ERR_ARG;
+  if (a.act ? a.maps != 1 || a.lda % 2 : !a.part_o || !a.part_ml) return CB_ERR_ARG;
+  if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   const int tiles = (int)((max_rows + kBM - 1) / kBM);
   cudaStream_t st = (cudaStream_t)stream;
   if (a.dim <= 32) return flash_dv<32>(a, tiles, (int)segs, st);
@@ -451,7 +462,7 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
       a.nsplit < 1 || a.nsplit > 64)
     return CB_ERR_ARG;
-  if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim)) return CB_ERR_SHAPE;
+  if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
   const int R = a.H / a.G;
   int hpc = 8 / a.maps;                                  // heads per CTA: at most 8 query vectors

@@ -293,7 +293,27 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       if (!wait_bar(&pair_bar[q], xph, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 93); abort_s = 1; } ok = false; }
       else l = lx[r] + lx[kBQ + r];
     }
-    if (ok) {
+    if (ok && a.act) {                                 // one map: the head is finished here
+      tc_fence_after();
+      const int64_t row = seg0 + t;
+      const float s = t < n ? (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / l : 0.f;
+      bf16* op = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * DV;
+#pragma unroll 1
+      for (int c0 = hf * (DV / 2); c0 < (hf + 1) * (DV / 2); c0 += 32) {
+        uint32_t o[32];
+        tmem_ld32(tmem_o + lane_base + c0, o);         // warp-collective: rows beyond the segment load too
+        tmem_ld_wait();
+        if (t < n) {
+#pragma unroll
+          for (int v = 0; v < 4; ++v) {
+            float x[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[8 * v + e]) * s;
+            *reinterpret_cast<uint4*>(op + c0 + v * 8) = float_to_bf16x8(x);
+          }
+        }
+      }
+    } else if (ok) {
       tc_fence_after();
       const int64_t idx = ((int64_t)(seg0 + t) * a.H * a.maps + vh) * a.nsplit;
       float* op = a.part_o + idx * DV;
@@ -350,7 +370,7 @@ int mode_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& 
 
 // Whether cb_attn_maps_flash_tc takes these head sizes.
 CB_EXPORT int cb_attn_maps_flash_tc_ok(int64_t dim, int64_t vdim) {
-  return (dim == 64 || dim == 128 || dim == 256) && (vdim == 64 || vdim == 128 || vdim == 256);
+  return (dim == 64 || dim == 128 || dim == 192 || dim == 256) && (vdim == 64 || vdim == 128 || vdim == 256);
 }
 
 // Prompt attention of `segs` segments of at most `max_rows` rows on tcgen05; arguments as for cb_attn_maps_flash.
@@ -358,22 +378,21 @@ CB_EXPORT int cb_attn_maps_flash_tc_ok(int64_t dim, int64_t vdim) {
 CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_rows, int64_t slots, void* status, void* stream) {
   if (!args || segs < 1 || segs > 65535 || max_rows < 1 || !status) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
-  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
-      a.maps < 1)
-    return CB_ERR_ARG;
-  if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || a.ldp % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
+  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G || a.maps < 1) return CB_ERR_ARG;
+  if (a.act ? a.maps != 1 || a.lda % 8 || ((uintptr_t)a.act & 15) : !a.part_o || !a.part_ml) return CB_ERR_ARG;
+  if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || a.ldp % 8 || a.ldk % 8 || a.ldv % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
   CUtensorMap tmK, tmV;
   const uint64_t kw = (uint64_t)a.G * a.maps * a.dim, vw = (uint64_t)a.G * a.vdim;
-  int rc = cb_make_tmap_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kpool, (uint64_t)slots, kw, kw, kBKV, 64);
+  int rc = cb_make_tmap_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kpool, (uint64_t)slots, kw, (uint64_t)pool_ldk(a), kBKV, 64);
   if (rc) return rc;
-  rc = cb_make_tmap_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.vpool, (uint64_t)slots, vw, vw, kBKV, 64);
+  rc = cb_make_tmap_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.vpool, (uint64_t)slots, vw, (uint64_t)pool_ldv(a), kBKV, 64);
   if (rc) return rc;
   const int tiles = (int)((max_rows + kBQ - 1) / kBQ);
   int* st_word = (int*)status;
   cudaStream_t st = (cudaStream_t)stream;
 #define CB_TC(K, V) \
   if (a.dim == K && a.vdim == V) return mode_tc<K, V>(tmK, tmV, a, tiles, (int)segs, st_word, st)
-  CB_TC(64, 64); CB_TC(64, 128); CB_TC(64, 256); CB_TC(128, 64); CB_TC(128, 128); CB_TC(128, 256); CB_TC(256, 64); CB_TC(256, 128);
+  CB_TC(64, 64); CB_TC(64, 128); CB_TC(64, 256); CB_TC(128, 64); CB_TC(128, 128); CB_TC(128, 256); CB_TC(192, 64); CB_TC(192, 128); CB_TC(192, 256); CB_TC(256, 64); CB_TC(256, 128);
   CB_TC(256, 256);
 #undef CB_TC
   return CB_ERR_SHAPE;

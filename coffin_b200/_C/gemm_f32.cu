@@ -55,6 +55,15 @@ __global__ void __launch_bounds__(256) swiglu_f32_kernel(const float* __restrict
   for (int64_t i = threadIdx.x; i < I; i += 256) o[i] = silu_x(g[i]) * g[I + i];
 }
 
+__global__ void __launch_bounds__(256) xielu_f32_kernel(const float* __restrict__ x, int64_t ldx, float* __restrict__ out, int64_t ldo,
+                                                        int64_t I, float a, float b) {
+  griddep_launch();
+  griddep_wait();
+  const float* r = x + (int64_t)blockIdx.x * ldx;
+  float* o = out + (int64_t)blockIdx.x * ldo;
+  for (int64_t i = threadIdx.x; i < I; i += 256) o[i] = xielu_x(r[i], a, b);
+}
+
 }  // namespace
 
 CB_EXPORT int cb_gemm_f32(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int64_t M, int64_t N,
@@ -71,4 +80,11 @@ CB_EXPORT int cb_swiglu_f32(const void* gu, int64_t ldg, void* out, int64_t ldo,
   if (!gu || !out || M < 1 || I < 1) return CB_ERR_ARG;
   return (int)cb_launch(swiglu_f32_kernel, dim3((unsigned)M), dim3(256), 0, (cudaStream_t)stream, (const float*)gu, ldg,
                         (float*)out, ldo, I);
+}
+
+// out = xIELU(x) with the coefficients (a, b) of its two branches, fp32 (may be in place)
+CB_EXPORT int cb_xielu_f32(const void* x, int64_t ldx, void* out, int64_t ldo, int64_t M, int64_t I, float a, float b, void* stream) {
+  if (!x || !out || M < 1 || I < 1) return CB_ERR_ARG;
+  return (int)cb_launch(xielu_f32_kernel, dim3((unsigned)M), dim3(256), 0, (cudaStream_t)stream, (const float*)x, ldx, (float*)out,
+                        ldo, I, a, b);
 }

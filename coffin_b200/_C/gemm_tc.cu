@@ -14,6 +14,7 @@
 // Every CTA fetches its own tiles with plain (single-destination) TMA loads.
 // Replaces the reference's linear_prefill (torch matmul / cublasGemmEx + epilogue kernel,
 // backends/corex/__init__.py:1612-1701, kernels/w8a8.cu:196-366, w8a8_tcu.cu:327-776).
+#include "act_type.cuh"
 #include "sm100.cuh"
 #include "tp.cuh"
 
@@ -44,6 +45,7 @@ struct GemmArgs {
   // adds the partials in slice order and writes the result, so the sum does not depend on timing.
   int splits; float* ws; unsigned* tickets;
   int c_f32 = 0;                   // C is fp32 instead of bf16 (gate pre-activations, logits)
+  int act = 0; float act_a = 0.f, act_b = 0.f;   // 1: xIELU epilogue with these coefficients
 };
 struct TileCoord { int m0, row_end, n0, brow; };
 template <int BN>
@@ -234,6 +236,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               f.x *= rsr * a.col_scale[gcol]; f.y *= rsr * a.col_scale[gcol + 1];
               f.z *= rsr * a.col_scale[gcol + 2]; f.w *= rsr * a.col_scale[gcol + 3];
             }
+            if (a.act) {
+              f.x = xielu_s(f.x, a.act_a, a.act_b); f.y = xielu_s(f.y, a.act_a, a.act_b);
+              f.z = xielu_s(f.z, a.act_a, a.act_b); f.w = xielu_s(f.w, a.act_a, a.act_b);
+            }
             if (a.residual) {
               const uint2 rr = *reinterpret_cast<const uint2*>(a.residual + (int64_t)grow * a.ldr + gcol);
               f.x += __uint_as_float(rr.x << 16); f.y += __uint_as_float(rr.x & 0xffff0000u);
@@ -276,6 +282,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             for (int i = 0; i < 8; ++i) {
               if (I8) f[i] = (float)(int)r[v * 8 + i] * rs * cscale[col0 + v * 8 + i];
               else f[i] = __uint_as_float(r[v * 8 + i]);
+              if (a.act) f[i] = xielu_s(f[i], a.act_a, a.act_b);
             }
             if (rp) {
               float g[8];
@@ -399,6 +406,8 @@ int cb_gemm_pair_plan(int64_t M, int64_t N);
 int cb_gemm_pair_run(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, const void* residual,
                      int64_t ldr, const void* row_scale, const void* col_scale, int64_t M, int64_t N, int64_t K, int tile,
                      const void* pf, int64_t pf_seq, void* status, void* stream);
+int cb_gemm_pair_xielu(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int64_t M, int64_t N, int64_t K,
+                       int tile, float act_a, float act_b, void* status, void* stream);
 
 // C[M,N] (bf16) = A[M,K] (bf16) x W[N,K]^T (bf16) (+ residual[M,N]).  K % 8 == 0, N % 8 == 0.
 // bn_hint: 0 = choose (CTA pairs for more than 256 rows), 64/128/160/256 = one-CTA kernel with that tile
@@ -433,6 +442,42 @@ CB_EXPORT int cb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ld
   if (bn == 128) return launch_gemm<128, 6, false>(tmA, tmB, a, sms, st);
   if (bn == 64) return launch_gemm<64, 8, false>(tmA, tmB, a, sms, st);
   return CB_ERR_ARG;
+}
+
+// C[M,N] = xIELU(A[M,K] x W[N,K]^T), bf16, with the coefficients (act_a, act_b) of its two branches: the activation is taken
+// in the epilogue (CTA pairs above 256 rows, split K up to 128 rows when scratch is given).
+CB_EXPORT int cb_gemm_bf16_xielu(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int64_t M, int64_t N,
+                                 int64_t K, float act_a, float act_b, void* ws, int64_t ws_bytes, void* tickets, int64_t n_tickets,
+                                 void* status, void* stream) {
+  if (M < 1 || N < 1 || K < 1 || K % 8 || N % 8 || ldc % 8 || !status) return CB_ERR_SHAPE;
+  const int tile = cb_gemm_pair_plan(M, N);
+  if (tile) return cb_gemm_pair_xielu(A, lda, W, ldw, C, ldc, M, N, K, tile, act_a, act_b, status, stream);
+  const int sms = sm_count();
+  int bn = pick_bn((int)M, (int)N, sms, true), splits = 1;
+  if (ws && tickets && M <= BM) {
+    int b2, s2;
+    plan_split(M, N, K * 2, &b2, &s2);
+    const int64_t tiles = (N + b2 - 1) / b2;
+    if (s2 > 1 && ws_bytes >= tiles * s2 * BM * b2 * (int64_t)sizeof(float) && n_tickets >= tiles) { bn = b2; splits = s2; }
+  }
+  CUtensorMap tmA, tmB;
+  int rc = cb_make_tmap_2d(&tmA, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM, 64);
+  if (rc) return rc;
+  rc = cb_make_tmap_2d(&tmB, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, (uint32_t)bn, 64);
+  if (rc) return rc;
+  GemmArgs a;
+  a.C = C; a.ldc = ldc; a.residual = nullptr; a.ldr = 0; a.row_scale = nullptr; a.col_scale = nullptr;
+  a.M = (int)M; a.N = (int)N; a.K = (int)K; a.m_tiles = (int)((M + BM - 1) / BM); a.n_tiles = 0;
+  a.k_blocks = (int)((K + 63) / 64); a.status = (int*)status;
+  a.pf = nullptr; a.pf_seq = 0;
+  a.g_count = a.g_row0 = a.g_rows = a.g_expert = nullptr;
+  a.splits = splits; a.ws = (float*)ws; a.tickets = (unsigned*)tickets;
+  a.act = 1; a.act_a = act_a; a.act_b = act_b;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (bn == 256) return launch_gemm<256, 4, false>(tmA, tmB, a, sms, st);
+  if (bn == 160) return launch_gemm<160, 5, false>(tmA, tmB, a, sms, st);
+  if (bn == 128) return launch_gemm<128, 6, false>(tmA, tmB, a, sms, st);
+  return launch_gemm<64, 8, false>(tmA, tmB, a, sms, st);
 }
 
 // C[M,N] (fp32) = A[M,K] (bf16) x W[N,K]^T (bf16): the accumulator leaves unrounded (gate pre-activations of the

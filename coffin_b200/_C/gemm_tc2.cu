@@ -16,6 +16,7 @@
 // Every wait is bounded (2 s) and reports through the status word; an abort is forwarded to the
 // other CTA of the pair so that both unwind, meet at the cluster barrier and free tensor memory.
 // Replaces the reference's linear_prefill (backends/corex/__init__.py:1612-1701).
+#include "act_type.cuh"
 #include "sm100.cuh"
 #include "tp.cuh"
 
@@ -36,6 +37,7 @@ struct PairArgs {
   int* status;
   const TpPfDev* pf; unsigned pf_seq;   // tensor-parallel prefill: rows go to this rank's peer-visible buffer (tp.cuh)
   int up_off;                      // SwiGLU form: W is [gate rows | up rows], the up rows start here; N counts outputs
+  int act = 0; float act_a = 0.f, act_b = 0.f;   // 1: xIELU epilogue with these coefficients
 };
 
 __device__ __forceinline__ uint64_t now_ns() {
@@ -247,6 +249,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
               for (int i = 0; i < 8; ++i) {
                 if (I8) f[i] = (float)(int)r[v * 8 + i] * rs * a.col_scale[col0 + v * 8 + i];
                 else f[i] = __uint_as_float(r[v * 8 + i]);
+                if (a.act) f[i] = xielu_s(f[i], a.act_a, a.act_b);
               }
               if (rbase) {
                 float g[8];
@@ -361,6 +364,21 @@ int cb_gemm_pair_run(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     if (tile == 320) return launch_pair<160, 2, 6, true>(A, lda, W, ldw, a, st);
     return CB_ERR_ARG;
   }
+  if (tile == 256) return launch_pair<256, 1, 6, false>(A, lda, W, ldw, a, st);
+  if (tile == 288) return launch_pair<144, 2, 6, false>(A, lda, W, ldw, a, st);
+  if (tile == 320) return launch_pair<160, 2, 6, false>(A, lda, W, ldw, a, st);
+  return CB_ERR_ARG;
+}
+
+// C[M, N] = xIELU(A W^T), bf16, more than 256 rows; tile: 256, 288 or 320.
+int cb_gemm_pair_xielu(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int64_t M, int64_t N, int64_t K,
+                       int tile, float act_a, float act_b, void* status, void* stream) {
+  PairArgs a;
+  a.C = (bf16*)C; a.ldc = ldc; a.residual = nullptr; a.ldr = 0; a.row_scale = nullptr; a.col_scale = nullptr;
+  a.M = (int)M; a.N = (int)N; a.K = (int)K; a.m_tiles = (int)((M + 255) / 256); a.n_tiles = 0;
+  a.k_blocks = 0; a.status = (int*)status; a.pf = nullptr; a.pf_seq = 0; a.up_off = 0;
+  a.act = 1; a.act_a = act_a; a.act_b = act_b;
+  cudaStream_t st = (cudaStream_t)stream;
   if (tile == 256) return launch_pair<256, 1, 6, false>(A, lda, W, ldw, a, st);
   if (tile == 288) return launch_pair<144, 2, 6, false>(A, lda, W, ldw, a, st);
   if (tile == 320) return launch_pair<160, 2, 6, false>(A, lda, W, ldw, a, st);

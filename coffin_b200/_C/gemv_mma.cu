@@ -11,6 +11,7 @@
 // RMSNorm, or the tensor-parallel pull-sum) and epilogues (SwiGLU, fp32 logits, tensor-parallel
 // push) of gemv.cu, the K-split for narrow outputs and the grid-wide sweep order.
 #include <string.h>
+#include "act_type.cuh"
 #include "tp.cuh"
 
 namespace {
@@ -39,6 +40,7 @@ struct MmaArgs {
   // ranks' sums of push_site for every row, adds tail_res_in, stores the new residual in tail_res_out and
   // its RMSNorm (gain tail_gain) in tail_out - what a separate pull kernel would do one launch later
   const bf16* tail_res_in; const float* tail_gain; bf16* tail_res_out; bf16* tail_out; float tail_eps;
+  int act = 0; float act_a = 0.f, act_b = 0.f;         // 1: xIELU epilogue with these coefficients
   TpComm tp;
 };
 
@@ -305,6 +307,7 @@ __global__ void __launch_bounds__(kT, 3) gemv_mma_kernel(const MmaArgs a_in) {
           if (m < M && row < a.N) {
             float v = acc[0][e];
             if (SWIGLU) v = silu_f(v) * acc[PB - 1][e];
+            else if (a.act) v = xielu_s(v, a.act_a, a.act_b);
             if (a.push_site >= 0) tp_push_value(a.tp, a.push_site, (int64_t)m * a.N + row, v);
             else if (OUT_F32) reinterpret_cast<float*>(a.y)[(int64_t)m * a.ldy + row] = v;
             else reinterpret_cast<bf16*>(a.y)[(int64_t)m * a.ldy + row] = __float2bfloat16(v);
@@ -352,6 +355,7 @@ __global__ void __launch_bounds__(kT, 3) gemv_mma_kernel(const MmaArgs a_in) {
             if (SWIGLU) v2 += __ldcg(all + c * 256 + 128 + idx);
           }
           if (SWIGLU) v = silu_f(v) * v2;
+          else if (a.act) v = xielu_s(v, a.act_a, a.act_b);
           if (a.push_site >= 0) tp_push_value(a.tp, a.push_site, (int64_t)m * a.N + row, v);
           else if (OUT_F32) reinterpret_cast<float*>(a.y)[(int64_t)m * a.ldy + row] = v;
           else reinterpret_cast<bf16*>(a.y)[(int64_t)m * a.ldy + row] = __float2bfloat16(v);
@@ -372,6 +376,7 @@ __global__ void __launch_bounds__(kT, 3) gemv_mma_kernel(const MmaArgs a_in) {
         if (SWIGLU) v2 += pw[128 + r * 8 + m];
       }
       if (SWIGLU) v = silu_f(v) * v2;
+      else if (a.act) v = xielu_s(v, a.act_a, a.act_b);
       if (a.push_site >= 0) tp_push_value(a.tp, a.push_site, (int64_t)m * a.N + row, v);
       else if (OUT_F32) reinterpret_cast<float*>(a.y)[(int64_t)m * a.ldy + row] = v;
       else reinterpret_cast<bf16*>(a.y)[(int64_t)m * a.ldy + row] = __float2bfloat16(v);
@@ -581,6 +586,22 @@ static int gemv_mma_impl(const void* W, const void* x, void* y, int64_t M, int64
   }
   if (f32) return norm ? launch_mma<false, true, true>(a, st) : launch_mma<false, false, true>(a, st);
   return norm ? launch_mma<false, true, false>(a, st) : launch_mma<false, false, false>(a, st);
+}
+
+// y[M, N] = xIELU(x W^T) with the coefficients (act_a, act_b) of its two branches; M = 1..8, bf16.
+CB_EXPORT int cb_gemv_mma_bf16_xielu(const void* W, const void* x, void* y, int64_t M, int64_t N, int64_t K, int64_t ldy, float act_a,
+                                     float act_b, void* stream) {
+  if (!W || !x || !y) return CB_ERR_ARG;
+  if (K % 8 || M < 1 || M > 8 || N < 1) return CB_ERR_SHAPE;
+  MmaArgs a;
+  a.W = (const bf16*)W; a.x = (const bf16*)x; a.y = y; a.N = N; a.K = K; a.ldy = ldy; a.up_off = N;
+  a.res_in = nullptr; a.add = nullptr; a.gain = nullptr; a.res_out = nullptr; a.eps = 0.f; a.M = (int)M; a.ksplit = 1; a.rounds = 1;
+  a.pull_site = a.push_site = -1;
+  a.slot_expert = nullptr; a.slot_xrow = nullptr; a.expert_stride = 0;
+  a.tail_res_in = nullptr; a.tail_gain = nullptr; a.tail_res_out = nullptr; a.tail_out = nullptr; a.tail_eps = 0.f;
+  a.act = 1; a.act_a = act_a; a.act_b = act_b;
+  memset(&a.tp, 0, sizeof(a.tp));
+  return launch_mma<false, false, false>(a, (cudaStream_t)stream);
 }
 
 // Grouped expert projection for decode: for every slot s (a routed (token, expert) pair),

@@ -1,18 +1,18 @@
-// Arguments shared by the recurrent-state kernels (linrec.cu: token by token; linrec_chunk.cu: prompts in chunks).
+// Arguments shared by the recurrent-state kernels (linrec.cu: token by token; linrec_chunk.cu, ssd.cu: prompts in chunks).
 #pragma once
 #include "act_type.cuh"
 
-enum LinrecKind : int { LINREC_DELTA = 0, LINREC_MLSTM = 1 };
+enum LinrecKind : int { LINREC_DELTA = 0, LINREC_MLSTM = 1, LINREC_SSD = 2 };
 
-// Column layout of a projection row: q | k | v | ... ; the first conv_width columns pass the short convolution
-// of the delta layers (channel index == column index).
+// Column layout of a projection row: q | k | v | ... ; the first ring_w columns pass the short convolution of the delta
+// and state-space layers (channel index == column index).  State-space layers: q = C, k = B, v = x.
 struct LinrecArgs {
   // rows
   const void* proj; int64_t ldp;        // q, k, v (and gate / low-rank) columns
-  const float* gates; int64_t ldg;      // fp32 gate pre-activations: delta b[H]; mLSTM i[H] | f[H]
+  const float* gates; int64_t ldg;      // fp32 gate pre-activations: delta b[H]; mLSTM i[H] | f[H]; ssd dt[H]
   const float* dec; int64_t ldd;        // delta, optional: decay pre-activations [H * dk] (before dt_bias)
   const void* og; int64_t ldo;          // output-gate pre-activations [H * dv] (null: delta computes them from g1 / g2)
-  void* act; int64_t lda;               // result rows [H * dv]
+  void* act; int64_t lda;               // result rows [H * dv] (ssd: always fp32, before gate and norm)
   // segments: rows [seg_row[s], seg_row[s + 1]) are consecutive tokens of one sequence from position seg_pos[s],
   // whose state lives in slot seg_slot[s] (< 0: skip).  seg_row null: row s alone.
   const int* seg_row; const int* seg_pos; const int* seg_slot;
@@ -30,4 +30,6 @@ struct LinrecArgs {
   int H, G, dk, dv, jc;
   int64_t k_col, v_col;
   float eps, cap;
+  const float* conv_b;                  // ssd: convolution bias [conv_width]
+  const float* D;                       // ssd: [H], weight of the value itself in the read-out
 };

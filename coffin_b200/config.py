@@ -199,6 +199,9 @@ def preset(name: str) -> ModelConfig:
     if "zufilorn" in name:
         from .models.zufilorn.config import preset_zufilorn
         return preset_zufilorn(name)
+    if "sukisun" in name:
+        from .models.sukisun.config import preset_sukisun
+        return preset_sukisun(name)
     if name == "tiny-moe":
         return ModelConfig(name="tiny-moe", num_experts=8, num_experts_per_tok=2,
                            moe_intermediate_size=128, shared_expert_intermediate_size=128,
@@ -247,4 +250,7 @@ def load_config(model_dir: str | Path):
     if str(raw.get("architecture", "")).lower() == "zufilorn":
         from .models.zufilorn.config import ZufilornConfig
         return ZufilornConfig.from_hf(raw, name=Path(model_dir).name)
+    if str(raw.get("architecture", "")).lower() == "sukisun":
+        from .models.sukisun.config import SukisunConfig
+        return SukisunConfig.from_hf(raw, name=Path(model_dir).name)
     return ModelConfig.from_hf(raw, name=Path(model_dir).name)

@@ -30,12 +30,12 @@ def main(argv=None) -> int:
     import torch
     from ...config import load_config
     from ...engine.replay import TraceReplayer, pool_blocks
-    from ...models import build_model, detect_architecture, kernel_sources
+    from ...models import FLOAT32, build_model, detect_architecture, kernel_sources
     from ...ops import _lib
     from ...weights.loader import load_checkpoint
     cfg = load_config(args.model)
     arch = detect_architecture(cfg)
-    if args.dtype == "float32" and arch != "zufilorn":
+    if args.dtype == "float32" and arch not in FLOAT32:
         print(f"{arch}: this family computes in 16 bits only", file=sys.stderr)
         return 3
     _lib.use_sources(kernel_sources(arch))

@@ -87,12 +87,27 @@ def _ensure_builtin() -> None:
 
     register("zufilorn", zufilorn)
 
+    def sukisun(cfg, sd, **kw):
+        from .sukisun.model import SukisunModel
+        if any(kw.pop(k + "_world", 1) > 1 for k in ("tp", "pp", "ep")):
+            raise NotImplementedError("the Sukisun family runs on one GPU")
+        for k in ("tp_rank", "pp_rank", "ep_rank"):
+            kw.pop(k, None)
+        return SukisunModel(cfg, sd, **kw)
+
+    register("sukisun", sukisun)
+
 
 #: kernel sources a family needs; families without an entry use the whole library
 _KERNELS: dict[str, tuple[str, ...]] = {
     "zufilorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "streams.cu",
                  "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
+    "sukisun": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "depth.cu", "linrec.cu", "ssd.cu",
+                "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
 }
+
+#: families that also run in 32-bit (``dtype=torch.float32``)
+FLOAT32 = ("zufilorn", "sukisun")
 
 
 def kernel_sources(arch: str) -> tuple[str, ...] | None:

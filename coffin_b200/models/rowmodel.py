@@ -36,6 +36,26 @@ class RowBatch:
     tables: torch.Tensor            # int32 [n_seg, pages]
     max_rows: int = 1               # longest segment
     max_len: int = 0                # largest position + 1 (0: unknown, inside a graph)
+    pre_lens: tuple = ()            # tokens of every leading segment's sequence so far, its own rows included
+    cache: dict = dataclasses.field(default_factory=dict)     # what mixers of one forward share
+
+    def expansion(self):
+        """Whole-page rows of the leading segments side by side: ``(first row, length, tables of consecutive blocks)`` per
+        segment on the device, the total number of rows and the most pages of a segment."""
+        e = self.cache.get("expansion")
+        if e is None:
+            pages = [(n + K.BLOCK - 1) // K.BLOCK for n in self.pre_lens]
+            first = [sum(pages[:i]) for i in range(len(pages))]
+            host = torch.zeros(len(pages), 2 + max(pages), dtype=torch.int32)
+            for i, (p, f, n) in enumerate(zip(pages, first, self.pre_lens)):
+                host[i, 0], host[i, 1] = f * K.BLOCK, n
+                host[i, 2:2 + p] = torch.arange(f, f + p, dtype=torch.int32)
+            if self.positions.is_cuda:
+                host = host.pin_memory()
+            dev = host.to(self.positions.device, non_blocking=True)
+            base_len = dev[:, :2].t().contiguous()
+            e = self.cache["expansion"] = (base_len[0], base_len[1], dev[:, 2:], sum(pages) * K.BLOCK, max(pages))
+        return e
 
 
 def pad8(n: int) -> int:
@@ -304,6 +324,7 @@ class RowModel:
         b = RowBatch(T=T, n_seg=n_seg, n_pre=n_pre, pre_rows=T - (n_seg - n_pre), tokens=tok.to(self.device, non_blocking=True),
                      positions=dev[:T], row_seg=dev[T:2 * T], seg_row=dev[o:o + n_seg + 1], seg_pos=dev[o + n_seg + 1:o + 2 * n_seg + 1],
                      seg_slot=dev[o + 2 * n_seg + 1:o + 3 * n_seg + 1], tables=dev[o + 3 * n_seg + 1:].view(n_seg, pages),
+                     pre_lens=tuple(int(items[i][1]) + len(toks[i]) for i in order[:n_pre]),
                      max_rows=max(len(t) for t in toks), max_len=max(int(it[1]) + len(t) for it, t in zip(items, toks)))
         return b, order, first
 

@@ -1,14 +1,19 @@
-"""Entry points of the kernels behind hyper-connected streams, the recurrent mixers and multi-map attention.
+"""Entry points of the kernels behind fp32 residuals, the recurrent mixers, multi-map attention and latent attention.
 
 Like ``ops.kernels`` these are thin wrappers that launch on the current stream into caller-owned buffers.  Every
-constant of a mechanism (tap count, gate cap, number of maps, score cap, query temperature, number of streams) is
-an argument, so a model family picks what it needs:
+constant of a mechanism (tap count, gate cap, number of maps, score cap, query temperature, number of streams, rotary
+base) is an argument, so a model family picks what it needs:
 
 * ``streams_embed`` / ``streams_step``: a residual of several fp32 streams with static read / write / mixing weights;
-* ``Linrec``: recurrences with a matrix state - the per-channel gated delta rule and the mLSTM matrix memory;
+* ``depth_embed`` / ``depth_step``: a residual that becomes a weighted sum of all layer results after every layer;
+* ``Linrec``: recurrences with a matrix state - the per-channel gated delta rule, the mLSTM matrix memory and the
+  state space with scalar decays (Mamba-2); ``gated_norm``: its output gate and grouped RMS norm;
 * ``AttnMaps``: paged attention with several score maps per head over the same values, capped scores and a
   position-dependent query temperature;
-* ``gemm_f32out`` / ``gemm_f32``: projections whose result (or everything) stays fp32.
+* ``LatentAttn``: attention over cached low-rank latents with a rotated key part shared by all heads; ``rope_rows`` /
+  ``rope_heads``: rotary angles of a batch and interleaved rotation of head parts;
+* ``gemm_f32out`` / ``gemm_f32``: projections whose result (or everything) stays fp32; ``linear_xielu``: a projection
+  with xIELU in its epilogue.
 """
 from __future__ import annotations
 
@@ -20,7 +25,7 @@ from . import _lib
 from . import kernels as K
 from ._lib import call
 
-DELTA, MLSTM = 0, 1
+DELTA, MLSTM, SSD = 0, 1, 2
 RING = 16             # shallowest convolution ring
 _P, _I64, _I32, _F = ctypes.c_void_p, ctypes.c_int64, ctypes.c_int, ctypes.c_float
 
@@ -65,6 +70,24 @@ def swiglu_f32(gu: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def linear_xielu(W: torch.Tensor, x: torch.Tensor, out: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    """``out = xielu(x @ W^T)``, ``xielu(z) = z / 2 + (a z^2 if z > 0 else b (exp(z) - 1 - z))``."""
+    T, Kd = x.shape
+    if out.dtype == torch.float32:
+        gemm_f32(x, W, out)
+        call("xielu_f32", out, out.stride(0), out, out.stride(0), T, W.shape[0], float(a), float(b))
+    elif T <= 8 and T * Kd * 2 <= 160 * 1024:
+        call("gemv_mma_bf16_xielu", W, x.contiguous(), out, T, W.shape[0], Kd, out.stride(0), float(a), float(b))
+    else:
+        ws = tickets = None
+        if T <= 128 and K.SPLITK_GEMM:
+            ws, tickets = K._splitk_scratch(x.device)
+        call("gemm_bf16_xielu", x, x.stride(0), W, W.stride(0), out, out.stride(0), T, W.shape[0], Kd, float(a), float(b), ws,
+             ws.numel() * 4 if ws is not None else 0, tickets, tickets.numel() if tickets is not None else 0, K.status_word(x.device))
+    K._count(2 if out.dtype == torch.float32 else 1)
+    return out
+
+
 # ------------------------------------------------------------------ hyper-connected streams
 def streams_embed(embed: torch.Tensor, pos: torch.Tensor | None, tokens: torch.Tensor, positions: torch.Tensor,
                   x: torch.Tensor) -> torch.Tensor:
@@ -91,6 +114,32 @@ def streams_step(x: torch.Tensor, h: torch.Tensor | None, *, gain: torch.Tensor 
     return h
 
 
+# ------------------------------------------------------------------ depth-averaged residual
+def depth_embed(embed: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, scale: float) -> torch.Tensor:
+    """Planes 0 (the embedding output) and 1 (the running residual of the first layer) of ``x [T, planes, W]`` (fp32)."""
+    T, planes, W = x.shape
+    assert x.dtype == torch.float32 and x.stride(2) == 1 and x.stride(1) == W and planes >= 2 and tokens.dtype == torch.int64
+    call("depth_embed", embed, tokens, x, x.stride(0), T, W, embed.shape[0], float(scale), _is_f32(embed))
+    K._count()
+    return x
+
+
+def depth_step(x: torch.Tensor, plane: int, h: torch.Tensor | None, *, gain: torch.Tensor | None = None, y: torch.Tensor | None = None,
+               weights: torch.Tensor | None = None, rows: torch.Tensor | None = None, store: bool = True, eps: float = 1e-5,
+               center: bool = True) -> torch.Tensor | None:
+    """Boundary between two sublayers: plane ``plane`` of ``x [T, planes, W]`` += ``y``; with ``weights`` (a layer's end) the
+    weighted sum of planes ``0 .. plane`` becomes plane ``plane + 1``; then ``h = norm(result) * gain``, layer norm
+    (``center``) or RMS norm.  ``rows`` picks the rows behind the rows of ``h`` (with ``store=False``)."""
+    T, planes, W = x.shape
+    n = rows.numel() if rows is not None else (h.shape[0] if h is not None else T)
+    t = h if h is not None else y
+    assert weights is None or (weights.numel() == plane + 1 and (not store or plane + 2 <= planes))
+    call("depth_step", x, x.stride(0), plane, y, y.stride(0) if y is not None else 0, weights, gain, h, h.stride(0) if h is not None else 0,
+         rows, n, W, float(eps), int(center), int(store), _is_f32(t) if t is not None else 0)
+    K._count()
+    return h
+
+
 # ------------------------------------------------------------------ recurrences with a matrix state
 class _LinrecStruct(ctypes.Structure):
     _fields_ = [("proj", _P), ("ldp", _I64), ("gates", _P), ("ldg", _I64), ("dec", _P), ("ldd", _I64), ("og", _P), ("ldo", _I64),
@@ -98,7 +147,7 @@ class _LinrecStruct(ctypes.Structure):
                 ("A_log", _P), ("dt_bias", _P), ("a2", _P), ("ra", _I64), ("a1_col", _I64), ("g2", _P), ("rg", _I64), ("g1_col", _I64),
                 ("norm_w", _P), ("gate_b", _P), ("S", _P), ("n", _P), ("m", _P), ("ring", _P), ("ring_mask", _I32), ("ring_w", _I64),
                 ("H", _I32), ("G", _I32), ("dk", _I32), ("dv", _I32), ("jc", _I32), ("k_col", _I64), ("v_col", _I64),
-                ("eps", _F), ("cap", _F)]
+                ("eps", _F), ("cap", _F), ("conv_b", _P), ("D", _P)]
 
 
 def linrec_supported(H: int, dk: int, dv: int) -> bool:
@@ -110,18 +159,20 @@ class Linrec:
 
     ``state``: ``S [slots, H, dk, dv]`` and, by kind, ``ring [slots, depth, width]`` (delta: the last raw projection
     rows, indexed by position modulo depth) or ``n [slots, H, dk]`` and ``m [slots, H]`` (mLSTM), all zero at the
-    start of a sequence."""
+    start of a sequence.  State space: keys, queries and values are B, C and x, the ring is the delta's, and the rows
+    that leave are fp32 and unnormed (``gated_norm`` follows)."""
 
     def __init__(self, kind: int, *, H: int, G: int, dk: int, dv: int, k_col: int, v_col: int, eps: float, state: dict,
-                 norm_w: torch.Tensor, conv_w: torch.Tensor | None = None, A_log=None, dt_bias=None, a2=None, a1_col: int = 0,
-                 g2=None, g1_col: int = 0, gate_b=None, cap: float = 0.0) -> None:
+                 norm_w: torch.Tensor | None = None, conv_w: torch.Tensor | None = None, A_log=None, dt_bias=None, a2=None,
+                 a1_col: int = 0, g2=None, g1_col: int = 0, gate_b=None, cap: float = 0.0, conv_b=None, D=None) -> None:
         if not linrec_supported(H, dk, dv):
             raise ValueError(f"recurrent head of {dk} x {dv} is outside the kernel's range")
         a = self.a = _LinrecStruct()
         size = _lib.call_nostream("linrec_args_size")
         assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
         self.kind, self.state, self.conv_w = kind, state, conv_w
-        self._keep = (norm_w, conv_w, A_log, dt_bias, a2, g2, gate_b, *state.values())
+        self._keep = (norm_w, conv_w, A_log, dt_bias, a2, g2, gate_b, conv_b, D, *state.values())
+        a.conv_b, a.D = _ptr(conv_b), _ptr(D)
         a.H, a.G, a.dk, a.dv, a.k_col, a.v_col, a.eps, a.cap = H, G, dk, dv, k_col, v_col, float(eps), float(cap)
         a.norm_w, a.conv_w, a.A_log, a.dt_bias, a.gate_b = _ptr(norm_w), _ptr(conv_w), _ptr(A_log), _ptr(dt_bias), _ptr(gate_b)
         a.taps = conv_w.shape[1] if conv_w is not None else 0
@@ -144,15 +195,19 @@ class Linrec:
     def step(self, proj, gates, og, act, seg_pos, seg_slot, *, segs: int, seg_row=None, dec=None) -> None:
         """Token by token over ``segs`` segments (``seg_row`` None: one row each)."""
         self._fill(proj, gates, og, act, dec, seg_row, seg_pos, seg_slot)
-        call("linrec_step", ctypes.byref(self.a), self.kind, segs, _is_f32(proj), _is_f32(act))
+        call("linrec_step", ctypes.byref(self.a), self.kind, segs, _is_f32(proj), _is_f32(self.state.get("ring", act)))
         K._count()
 
     @property
     def chunked(self) -> bool:
         """Whether prompts of this head size run in chunks on the tensor cores (bf16 activations)."""
-        return bool(_lib.call_nostream("linrec_chunk_ok", self.a.dk, self.a.dv))
+        return bool(_lib.call_nostream("ssd_chunk_ok" if self.kind == SSD else "linrec_chunk_ok", self.a.dk, self.a.dv))
 
     def chunk_scratch(self, rows: int, segs: int) -> int:
+        if self.kind == SSD:
+            fn = _lib.lib().cb_ssd_chunk_scratch
+            fn.restype = ctypes.c_int64
+            return int(fn(*[ctypes.c_int64(v) for v in (rows, self.a.H, self.a.ring_w)]))
         fn = _lib.lib().cb_linrec_chunk_scratch
         fn.restype = ctypes.c_int64
         a = self.a
@@ -162,6 +217,10 @@ class Linrec:
         """The first ``segs`` segments (rows ``[0, rows)``, at most ``max_rows`` each) in chunks; ``scratch`` bytes as
         ``chunk_scratch`` says.  The convolution ring is left as it was (``ring`` afterwards)."""
         self._fill(proj, gates, og, act, dec, seg_row, seg_pos, seg_slot)
+        if self.kind == SSD:
+            call("ssd_chunk", ctypes.byref(self.a), segs, max_rows, rows, scratch, scratch.numel() * scratch.element_size())
+            K._count(2)
+            return
         call("linrec_chunk", ctypes.byref(self.a), self.kind, segs, max_rows, rows, scratch, scratch.numel() * scratch.element_size())
         K._count(4 if self.kind == MLSTM else 3)
 
@@ -176,12 +235,19 @@ class Linrec:
         K._count()
 
 
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, act: torch.Tensor, *, groups: int, n: int, eps: float) -> torch.Tensor:
+    """``act = rmsnorm(y * silu(z)) * weight``, each row in ``groups`` parts of ``n`` columns with a root mean square of their own."""
+    call("gated_norm", y, y.stride(0), z, z.stride(0), weight, act, act.stride(0), y.shape[0], groups, n, float(eps), _is_f32(z), _is_f32(act))
+    K._count()
+    return act
+
+
 # ------------------------------------------------------------------ attention with several maps per head
 class _AttnStruct(ctypes.Structure):
     _fields_ = [("proj", _P), ("ldp", _I64), ("k_col", _I64), ("v_col", _I64), ("kpool", _P), ("vpool", _P), ("tables", _P),
                 ("ldbt", _I64), ("row_seg", _P), ("positions", _P), ("seg_row", _P), ("seg_pos", _P), ("part_o", _P), ("part_ml", _P),
                 ("H", _I32), ("G", _I32), ("maps", _I32), ("dim", _I32), ("vdim", _I32), ("nsplit", _I32), ("scale", _F), ("cap", _F),
-                ("temp_coef", _F), ("temp_every", _I32)]
+                ("temp_coef", _F), ("temp_every", _I32), ("ldk", _I64), ("ldv", _I64), ("act", _P), ("lda", _I64), ("gates", _P), ("ldg", _I64)]
 
 
 MAX_VDIM = 512
@@ -197,12 +263,19 @@ class AttnMaps:
         a = self.a = _AttnStruct()
         size = _lib.call_nostream("attn_maps_args_size")
         assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
-        self.kpool, self.vpool, self.H, self.G, self.maps, self.dim, self.vdim = kpool, vpool, H, G, maps, dim, vdim
+        self.H, self.G, self.maps, self.dim, self.vdim = H, G, maps, dim, vdim
         a.H, a.G, a.maps, a.dim, a.vdim, a.k_col, a.v_col = H, G, maps, dim, vdim, k_col, v_col
-        a.kpool, a.vpool, a.scale, a.cap = _ptr(kpool), _ptr(vpool), float(scale), float(cap or 0.0)
+        a.scale, a.cap = float(scale), float(cap or 0.0)
+        self.set_pools(kpool, vpool)
         self._tcgen05 = bool(_lib.call_nostream("attn_maps_flash_tc_ok", dim, vdim))
         if temp is not None:
             a.temp_coef, a.temp_every = float(temp[0]), int(temp[1])
+
+    def set_pools(self, kpool: torch.Tensor, vpool: torch.Tensor) -> None:
+        """Rows of keys and values; they may be column ranges of wider rows."""
+        a = self.a
+        self.kpool, self.vpool = kpool, vpool
+        a.kpool, a.vpool, a.ldk, a.ldv = _ptr(kpool), _ptr(vpool), kpool.stride(0), vpool.stride(0)
 
     def _fill(self, proj, tables, positions, row_seg, part_o=None, part_ml=None, nsplit: int = 1, seg_row=None, seg_pos=None) -> None:
         a = self.a
@@ -226,10 +299,14 @@ class AttnMaps:
         """Whether the tensor-core prompt kernel and the split decode kernel take this head."""
         return self.kpool.dtype == torch.bfloat16 and bool(_lib.call_nostream("attn_maps_tc_ok", self.G, self.maps, self.dim, self.vdim))
 
-    def flash(self, proj, tables, seg_row, seg_pos, part_o, part_ml, *, segs: int, max_rows: int, positions) -> None:
+    def flash(self, proj, tables, seg_row, seg_pos, part_o, part_ml, *, segs: int, max_rows: int, positions, act=None, gates=None) -> None:
         """Portions of several tokens (bf16 projection rows; keys and values appended before): tcgen05 for head sizes of
-        64 / 128 / 256 and portions worth a 128-row tile, ``mma.sync`` otherwise."""
+        64 / 128 / 192 / 256 (values 64 / 128 / 256) and portions worth a 128-row tile, ``mma.sync`` otherwise.  With one map
+        ``act`` takes the finished heads, times ``sigmoid(gates)`` if given, and there are no parts."""
         self._fill(proj, tables, positions, None, part_o, part_ml, 1, seg_row, seg_pos)
+        a = self.a
+        a.act, a.lda = _ptr(act), act.stride(0) if act is not None else 0
+        a.gates, a.ldg = _ptr(gates), gates.stride(0) if gates is not None else 0
         if K.ATTN_TC and max_rows >= K.ATTN_TC_MIN_T and self._tcgen05:
             call("attn_maps_flash_tc", ctypes.byref(self.a), segs, max_rows, self.kpool.shape[0], K.status_word(proj.device))
         else:
@@ -253,3 +330,90 @@ class AttnMaps:
         call("attn_maps_finish", part_o, part_ml, gates, gates.stride(0) if gates is not None else 0, act, act.stride(0), positions,
              positions.numel(), self.H, self.maps, self.vdim, nsplit, float(lam), float(post_scale), float(eps), _is_f32(act))
         K._count()
+
+
+# ------------------------------------------------------------------ rotary angles
+def rope_turns(base: float, dims: int, device) -> torch.Tensor:
+    """fp64 ``[dims / 2]``: turns per position of pair ``i``, ``base^(-2 i / dims) / (2 pi)``."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    return (torch.tensor(float(base), dtype=torch.float64) ** (-2.0 * i / dims) / (2.0 * torch.pi)).to(device)
+
+
+def rope_rows(positions: torch.Tensor, turns: torch.Tensor, cs: torch.Tensor) -> torch.Tensor:
+    """``cs [rows, pairs * 2]`` (fp32) = (cos, sin) of every pair at the rows' positions."""
+    call("rope_rows", positions, turns, cs, positions.numel(), turns.numel())
+    K._count()
+    return cs
+
+
+def rope_heads(src: torch.Tensor, hs: int, dst: torch.Tensor, hd: int, cs: torch.Tensor, *, half: int, rot: int, H: int) -> None:
+    """Rotate ``rot`` columns of ``H`` heads, pairs ``(2i, 2i + 1)`` for the first ``half`` pairs; ``src`` / ``dst`` start at the
+    first head's rotated column, heads are ``hs`` / ``hd`` columns apart; may be in place."""
+    assert src.dtype == dst.dtype
+    call("rope_heads", src, src.stride(0), hs, dst, dst.stride(0), hd, cs, half, rot, H, src.shape[0], _is_f32(dst))
+    K._count()
+
+
+# ------------------------------------------------------------------ latent attention
+class _LatentStruct(ctypes.Structure):
+    _fields_ = [("proj", _P), ("ldp", _I64), ("c_col", _I64), ("r_col", _I64), ("norm_q", _P), ("norm_c", _P), ("cq", _P), ("ldq", _I64),
+                ("pool", _P), ("ldk", _I64), ("tables", _P), ("ldbt", _I64), ("row_seg", _P), ("positions", _P), ("cs", _P), ("half", _I32),
+                ("q_rank", _I32), ("kv_rank", _I32), ("rot", _I32), ("cp", _I32), ("eps", _F)]
+
+
+def head_linear(w: torch.Tensor, x: torch.Tensor, hx: int, y: torch.Tensor, hy: int, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """``y[t, h hy : h hy + N] = w[h] @ x[t, h hx : h hx + K]`` for ``w [H, N, K]``, times ``sigmoid(gate[t, h])`` if given."""
+    H, N, Kd = w.shape
+    call("head_linear", w, x, x.stride(0), hx, y, y.stride(0), hy, gate, gate.stride(0) if gate is not None else 0, x.shape[0], H, N, Kd,
+         _is_f32(w))
+    K._count()
+    return y
+
+
+class LatentAttn:
+    """Latent attention of one layer: pages ``pool [slots, ldk]`` hold ``[c | rotated key part]`` (the part at column ``cp``),
+    its own or those of the layer it borrows them from."""
+
+    def __init__(self, *, H: int, q_rank: int, kv_rank: int, rot: int, rot_dims: int, cp: int, scale: float, eps: float, pool: torch.Tensor,
+                 norm_q: torch.Tensor, norm_c: torch.Tensor | None, c_col: int = 0, r_col: int = 0) -> None:
+        a = self.a = _LatentStruct()
+        size = _lib.call_nostream("latent_args_size")
+        assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
+        self.H, self.cp, self.scale, self.pool, self.own, self.ldk = H, cp, float(scale), pool, norm_c is not None, pool.shape[1]
+        self._keep = (norm_q, norm_c)
+        a.q_rank, a.kv_rank, a.rot, a.cp, a.eps, a.half, a.c_col, a.r_col = q_rank, kv_rank, rot, cp, float(eps), rot_dims // 2, c_col, r_col
+        a.norm_q, a.norm_c, a.pool, a.ldk = _ptr(norm_q), _ptr(norm_c), _ptr(pool), pool.stride(0)
+        # the plain kernel and the merge of key splits see one key / value head whose values are the head of the key row
+        self._plain = AttnMaps(H=H, G=1, maps=1, dim=self.ldk, vdim=cp, k_col=0, v_col=0, scale=scale, cap=None, temp=None, kpool=pool,
+                               vpool=pool)
+        self.tc = pool.dtype == torch.bfloat16 and bool(_lib.call_nostream("latent_decode_ok", self.ldk, cp))
+
+    def rows(self, proj, cq, tables, positions, row_seg, cs) -> None:
+        """Norm the query latents into ``cq``; an owner also norms, rotates and appends what it caches."""
+        a = self.a
+        a.proj, a.ldp, a.cq, a.ldq = proj.data_ptr(), proj.stride(0), cq.data_ptr(), cq.stride(0)
+        a.tables, a.ldbt, a.row_seg, a.positions, a.cs = tables.data_ptr(), tables.stride(0), _ptr(row_seg), positions.data_ptr(), _ptr(cs)
+        call("latent_rows", ctypes.byref(a), positions.numel(), int(self.own), _is_f32(proj), _is_f32(cq))
+        K._count()
+
+    def gather(self, tables, base, lens, out, *, segs: int, max_pages: int) -> None:
+        """Page rows of ``segs`` sequences side by side in ``out`` (segment ``s`` from row ``base[s]``)."""
+        call("latent_gather", self.pool, self.pool.stride(0) * self.pool.element_size(), tables, tables.stride(0), base, lens, out, segs, max_pages)
+        K._count()
+
+    def decode_splits(self, rows: int) -> int:
+        groups = -(-self.H // (16 if self.H <= 16 else 32))
+        return max(1, min(64, 148 // max(1, groups * rows)))
+
+    def absorbed(self, q, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
+        """Queries ``q [rows, H * ldk]`` against the pages: key splits for ``merge`` (one split without the tensor-core kernel)."""
+        if self.tc:
+            call("latent_decode", q, q.stride(0), self.pool, self.pool.stride(0), tables, tables.stride(0), row_seg, positions, part_o, part_ml,
+                 positions.numel(), self.H, self.cp, nsplit, self.scale)
+            K._count()
+        else:
+            self._plain.rows(q, tables, positions, row_seg, part_o, part_ml, nsplit)
+
+    def merge(self, part_o, part_ml, out, positions, nsplit: int) -> None:
+        """Weighted averages of the latents, ``out [rows, H * cp]``."""
+        self._plain.finish(part_o, part_ml, None, out, positions, nsplit=nsplit)

@@ -109,6 +109,10 @@ def _draw(shape, kind: str, gen: torch.Generator, device, dtype, std: float) -> 
             return (torch.eye(shape[0], device=device) + 0.1 * torch.randn(shape, generator=gen, device=device)).to(dtype)
         c = 1.0 / shape[0] if kind == "hc_in" else 1.0
         return (c * (1.0 + 0.3 * torch.randn(shape, generator=gen, device=device))).to(dtype)
+    if kind == "dwa":           # depth average: mostly the newest result
+        w = 0.1 * torch.randn(shape, generator=gen, device=device) / shape[0]
+        w[-1] += 1.0
+        return w.to(dtype)
     if kind == "gate_b":        # input / forget gate biases of a matrix memory
         return torch.randn(shape, generator=gen, device=device, dtype=torch.float32).to(dtype)
     if kind == "lam":

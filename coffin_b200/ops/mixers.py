@@ -201,7 +201,9 @@ class Linrec:
     @property
     def chunked(self) -> bool:
         """Whether prompts of this head size run in chunks on the tensor cores (bf16 activations)."""
-        return bool(_lib.call_nostream("ssd_chunk_ok" if self.kind == SSD else "linrec_chunk_ok", self.a.dk, self.a.dv))
+        if self.kind == SSD:
+            return bool(_lib.call_nostream("ssd_chunk_ok", self.a.dk, self.a.dv))
+        return bool(_lib.call_nostream("linrec_chunk_ok", self.a.dk, self.a.dv))
 
     def chunk_scratch(self, rows: int, segs: int) -> int:
         if self.kind == SSD:

@@ -23,8 +23,8 @@ class Twin:
     model run over all of them.  Positions and tables are checked, so a batch the engine builds wrongly fails."""
     mixed_batches = True
 
-    def __init__(self, cfg, W, slots, blocks, max_seq=256):
-        self.cfg_raw, self.W, self.device = cfg, W, torch.device("cpu")
+    def __init__(self, cfg, W, slots, blocks, max_seq=256, forward=P.forward):
+        self.cfg_raw, self.W, self.device, self.forward = cfg, W, torch.device("cpu"), forward
         self.num_slots, self.num_blocks, self.max_seq, self.max_chunk = slots, blocks, max_seq, 2048
         self.fed = [[] for _ in range(slots)]
         self.batches = []
@@ -53,7 +53,7 @@ class Twin:
             assert pos0 == len(self.fed[slot]) and len(table) * 64 >= pos0 + len(toks) and 0 not in table
             self.fed[slot] += toks
             if w:
-                lg = P.forward(self.cfg_raw, self.W, self.fed[slot])
+                lg = self.forward(self.cfg_raw, self.W, self.fed[slot])
                 rows += [lg[pos0 + i] for i in w]
         return torch.stack(rows) if rows else None
 

@@ -93,6 +93,27 @@ static inline cudaError_t cb_launch(void (*kernel)(KArgs...), dim3 grid, dim3 bl
   return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
 }
 
+// The same with a preferred split of the SM's memory between L1 and shared memory: `carve` percent shared.  Loads in flight
+// need room in L1.  A kernel with little shared memory that runs after one with a lot otherwise inherits its split.
+template <typename... KArgs, typename... Args>
+static inline cudaError_t cb_launch_carve(int carve, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                          Args... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributePreferredSharedMemoryCarveout;
+  attr[0].val.sharedMemCarveout = (unsigned)carve;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = g_cb_use_pdl ? 2 : 1;
+  if (g_cb_trace_names) cb_trace_name((const void*)kernel);
+  return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
+}
+
 // ---- small math ---------------------------------------------------------------------------
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -12,7 +12,7 @@
 
 namespace {
 
-constexpr int kT = 256;
+constexpr int kT = 256, kMaxPlanes = 1024;
 
 __device__ __forceinline__ float ld_dsmem(const float* p, uint32_t rank) {
   const uint32_t a = sm100::map_to_cta((uint32_t)__cvta_generic_to_shared(p), rank);
@@ -33,14 +33,49 @@ struct DepthArgs {
   int center, store;
 };
 
-template <typename TA, int V>
-__global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a) {
-  extern __shared__ float v_s[];       // this CTA's columns of the (averaged) residual
-  __shared__ float red[32], w_s[256];
+// acc += sum over planes j0, j0 + step, ... < n of w[j] * x[j][i .. i + V)
+template <int V>
+__device__ __forceinline__ void plane_sum(float* acc, const float* __restrict__ xi, int64_t W, const float* w, int j0, int step, int n) {
+  constexpr int U = 8;                           // planes requested together
+  for (int j = j0; j < n; j += U * step) {
+    float f[U][V];
+#pragma unroll
+    for (int k = 0; k < U; ++k) {
+      const bool ok = j + k * step < n;
+      const float* p = xi + (int64_t)(j + k * step) * W;
+      if (V == 4) {
+        const float4 q = ok ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+        f[k][0] = q.x; f[k][1 % V] = q.y; f[k][2 % V] = q.z; f[k][3 % V] = q.w;
+      } else {
+        f[k][0] = ok ? *p : 0.f;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < U; ++k) {
+      const float c = j + k * step < n ? w[j + k * step] : 0.f;
+#pragma unroll
+      for (int v = 0; v < V; ++v) acc[v] = fmaf(c, f[k][v], acc[v]);
+    }
+  }
+}
+template <int V> __device__ __forceinline__ void ld_f32(float* d, const float* p) {
+  if (V == 4) { const float4 q = *reinterpret_cast<const float4*>(p); d[0] = q.x; d[1 % V] = q.y; d[2 % V] = q.z; d[3 % V] = q.w; }
+  else d[0] = *p;
+}
+template <int V> __device__ __forceinline__ void st_f32(float* p, const float* d) {
+  if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(d[0], d[1 % V], d[2 % V], d[3 % V]);
+  else *p = d[0];
+}
+
+// PG: groups of threads that share a row's planes (few rows); 1: every thread takes whole columns
+template <typename TA, int V, bool GROUPS>
+__global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a, int pg_n) {
+  extern __shared__ float v_s[];       // this CTA's columns of the (averaged) residual; then partial sums of the other groups
+  __shared__ float red[32], w_s[kMaxPlanes];
   __shared__ float cl[2];
-  const int ns = gridDim.x, c0 = blockIdx.x * a.cols, c1 = min(a.W, c0 + a.cols);
+  const int ns = gridDim.x, c0 = blockIdx.x * a.cols, c1 = min(a.W, c0 + a.cols), nc = c1 - c0;
   if (a.dwa)
-    for (int j = threadIdx.x; j <= a.plane && j < 256; j += kT) w_s[j] = a.dwa[j];
+    for (int j = threadIdx.x; j <= a.plane; j += kT) w_s[j] = a.dwa[j];
   griddep_launch();
   griddep_wait();
   const int64_t r = a.rows ? a.rows[blockIdx.y] : (int64_t)blockIdx.y;
@@ -50,95 +85,89 @@ __global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a) {
   float* cur = xr + (int64_t)a.plane * a.W;
   const TA* yr = a.y ? reinterpret_cast<const TA*>(a.y) + r * a.ldy : nullptr;
   float s = 0.f;
-  for (int i = c0 + threadIdx.x * V; i < c1; i += kT * V) {
-    float u[V];
+  auto own = [&](float* u, int i) {    // the running residual with the sublayer's output
+    ld_f32<V>(u, cur + i);
+    if (!yr) return;
     if (V == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(cur + i);
-      u[0] = f.x; u[1 % V] = f.y; u[2 % V] = f.z; u[3 % V] = f.w;
+      const float4 f = act_load4(yr + i);
+      u[0] += f.x; u[1 % V] += f.y; u[2 % V] += f.z; u[3 % V] += f.w;
     } else {
-      u[0] = cur[i];
+      u[0] += act_load(yr + i);
     }
-    if (yr) {
-      if (V == 4) {
-        const float4 f = act_load4(yr + i);
-        u[0] += f.x; u[1 % V] += f.y; u[2 % V] += f.z; u[3 % V] += f.w;
-      } else {
-        u[0] += act_load(yr + i);
+    if (a.store) st_f32<V>(cur + i, u);
+  };
+  auto keep = [&](const float* u, int i) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) { v_s[i + v] = u[v]; s += a.center ? u[v] : u[v] * u[v]; }
+  };
+  if (GROUPS) {
+    const int units = (nc + V - 1) / V, unit = threadIdx.x % units, pg = threadIdx.x / units, i = c0 + unit * V;
+    float acc[V] = {};
+    if (pg < pg_n) {
+      if (pg == 0) {
+        float u[V];
+        own(u, i);
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[v] = w_s[a.plane] * u[v];
       }
-      if (a.store) {
-        if (V == 4) *reinterpret_cast<float4*>(cur + i) = make_float4(u[0], u[1 % V], u[2 % V], u[3 % V]);
-        else cur[i] = u[0];
-      }
+      plane_sum<V>(acc, xr + i, a.W, w_s, pg, pg_n, a.plane);
+      if (pg) st_f32<V>(v_s + pg * a.cols + unit * V, acc);
     }
-    if (a.dwa) {
-      float acc[V];
-      const float wl = a.plane < 256 ? w_s[a.plane] : a.dwa[a.plane];
+    __syncthreads();
+    if (pg == 0) {
+      for (int g = 1; g < pg_n; ++g)
 #pragma unroll
-      for (int v = 0; v < V; ++v) acc[v] = wl * u[v];
-      const float* p = xr + i;
-      int j = 0;
-      for (; j + 8 <= a.plane; j += 8) {                         // eight planes requested together
-        float f[8][V];
-#pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          if (V == 4) {
-            const float4 q = *reinterpret_cast<const float4*>(p + (int64_t)(j + k) * a.W);
-            f[k][0] = q.x; f[k][1 % V] = q.y; f[k][2 % V] = q.z; f[k][3 % V] = q.w;
-          } else {
-            f[k][0] = p[(int64_t)(j + k) * a.W];
-          }
-        }
-#pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          const float w = j + k < 256 ? w_s[j + k] : a.dwa[j + k];
-#pragma unroll
-          for (int v = 0; v < V; ++v) acc[v] = fmaf(w, f[k][v], acc[v]);
-        }
-      }
-#pragma unroll 1
-      for (; j < a.plane; ++j) {
-        const float w = j < 256 ? w_s[j] : a.dwa[j];
-        if (V == 4) {
-          const float4 q = *reinterpret_cast<const float4*>(p + (int64_t)j * a.W);
-          acc[0] = fmaf(w, q.x, acc[0]); acc[1 % V] = fmaf(w, q.y, acc[1 % V]);
-          acc[2 % V] = fmaf(w, q.z, acc[2 % V]); acc[3 % V] = fmaf(w, q.w, acc[3 % V]);
-        } else {
-          acc[0] = fmaf(w, p[(int64_t)j * a.W], acc[0]);
-        }
-      }
-#pragma unroll
-      for (int v = 0; v < V; ++v) u[v] = acc[v];
-      if (a.store) {
-        if (V == 4) *reinterpret_cast<float4*>(cur + a.W + i) = make_float4(u[0], u[1 % V], u[2 % V], u[3 % V]);
-        else cur[a.W + i] = u[0];
-      }
+        for (int v = 0; v < V; ++v) acc[v] += v_s[g * a.cols + unit * V + v];
+      if (a.store) st_f32<V>(cur + a.W + i, acc);
+      keep(acc, unit * V);
     }
+  } else {
+    for (int i = c0 + threadIdx.x * V; i < c1; i += kT * V) {
+      float u[V];
+      own(u, i);
+      if (a.dwa) {
+        float acc[V];
 #pragma unroll
-    for (int v = 0; v < V; ++v) { v_s[i - c0 + v] = u[v]; s += a.center ? u[v] : u[v] * u[v]; }
+        for (int v = 0; v < V; ++v) acc[v] = w_s[a.plane] * u[v];
+        plane_sum<V>(acc, xr + i, a.W, w_s, 0, 1, a.plane);
+#pragma unroll
+        for (int v = 0; v < V; ++v) u[v] = acc[v];
+        if (a.store) st_f32<V>(cur + a.W + i, u);
+      }
+      keep(u, i - c0);
+    }
   }
   if (!a.h) return;
-  // first sum: the mean (layer norm) or the mean square; second: squared deviations
-  auto row_sum = [&](float v, int k) {
-    v = block_sum(v, red);
-    if (ns == 1) return v;
-    if (threadIdx.x == 0) cl[k] = v;
-    sm100::cluster_sync_all();
-    float t = 0.f;
-    for (int q = 0; q < ns; ++q) t += ld_dsmem(&cl[k], q);
-    return t;
-  };
-  float m = row_sum(s, 0) / (float)a.W, mean = 0.f, rstd;
+  // mean and squared deviations of this CTA's columns, then of the row (RMS norm: plain squares about zero)
+  s = block_sum(s, red);
+  float mean = 0.f, m2 = s;
   if (a.center) {
-    mean = m;
+    mean = s / (float)nc;
     float d2 = 0.f;
-    for (int i = threadIdx.x * V; i < c1 - c0; i += kT * V)      // each thread re-reads what it wrote
-#pragma unroll
-      for (int v = 0; v < V; ++v) { const float d = v_s[i + v] - mean; d2 = fmaf(d, d, d2); }
-    m = row_sum(d2, 1) / (float)a.W;
+    for (int i = threadIdx.x; i < nc; i += kT) { const float d = v_s[i] - mean; d2 = fmaf(d, d, d2); }
+    m2 = block_sum(d2, red);
   }
-  rstd = 1.f / sqrtf(m + a.eps);
+  if (ns > 1) {
+    if (threadIdx.x == 0) { cl[0] = mean; cl[1] = m2; }
+    sm100::cluster_sync_all();
+    float mq[8], vq[8], tot = 0.f;
+    for (int q = 0; q < ns; ++q) {
+      mq[q & 7] = ld_dsmem(&cl[0], q);
+      vq[q & 7] = ld_dsmem(&cl[1], q);
+      tot += mq[q & 7] * (float)(min(a.W, (q + 1) * a.cols) - q * a.cols);
+    }
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");    // this CTA has read what it needs
+    mean = tot / (float)a.W;
+    m2 = 0.f;
+    for (int q = 0; q < ns; ++q) {
+      const float d = mq[q & 7] - mean;
+      m2 += vq[q & 7] + (a.center ? d * d * (float)(min(a.W, (q + 1) * a.cols) - q * a.cols) : 0.f);
+    }
+    if (!a.center) mean = 0.f;
+  }
+  const float rstd = 1.f / sqrtf(m2 / (float)a.W + a.eps);
   TA* hr = reinterpret_cast<TA*>(a.h) + (int64_t)blockIdx.y * a.ldh;
-  for (int i = threadIdx.x * V; i < c1 - c0; i += kT * V) {
+  for (int i = threadIdx.x * V; i < nc; i += kT * V) {
     if (V == 4) {
       const float4 g = *reinterpret_cast<const float4*>(a.gain + c0 + i);
       act_store4(hr + c0 + i, make_float4((v_s[i] - mean) * rstd * g.x, (v_s[i + 1 % V] - mean) * rstd * g.y,
@@ -147,7 +176,7 @@ __global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a) {
       act_store(hr + c0 + i, (v_s[i] - mean) * rstd * a.gain[c0 + i]);
     }
   }
-  if (ns > 1) sm100::cluster_sync_all();         // nobody leaves while its sums may still be read
+  if (ns > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");     // nobody leaves while its sums may still be read
 }
 
 // planes 0 and 1 of row t = embed[token[t]] * scale
@@ -173,8 +202,13 @@ int launch_depth(DepthArgs a, int64_t n, cudaStream_t st) {
   while (ns < 8 && n * ns * 2 <= 148 && a.W / (ns * 2) >= 256) ns <<= 1;
   a.cols = ((a.W + ns - 1) / ns + 3) & ~3;
   ns = (a.W + a.cols - 1) / a.cols;
-  auto kern = v4 ? depth_step_kernel<TA, 4> : depth_step_kernel<TA, 1>;
-  const size_t smem = (size_t)a.cols * sizeof(float);
+  const int units = v4 ? (a.cols + 3) / 4 : a.cols;
+  int pg = a.dwa && a.plane > 8 && n <= 64 ? kT / units : 1;     // few rows: groups of threads share the planes
+  if (pg > 8) pg = 8;
+  auto kern = pg > 1 ? (v4 ? depth_step_kernel<TA, 4, true> : depth_step_kernel<TA, 1, true>)
+                     : (v4 ? depth_step_kernel<TA, 4, false> : depth_step_kernel<TA, 1, false>);
+  if (pg < 1) pg = 1;
+  const size_t smem = (size_t)a.cols * pg * sizeof(float);
   if (smem > 200 * 1024) return CB_ERR_SHAPE;
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -200,7 +234,7 @@ int launch_depth(DepthArgs a, int64_t n, cudaStream_t st) {
   cfg.attrs = attr;
   cfg.numAttrs = na;
   if (g_cb_trace_names) cb_trace_name((const void*)kern);
-  return (int)cudaLaunchKernelEx(&cfg, kern, a);
+  return (int)cudaLaunchKernelEx(&cfg, kern, a, pg);
 }
 
 }  // namespace
@@ -211,7 +245,7 @@ int launch_depth(DepthArgs a, int64_t n, cudaStream_t st) {
 CB_EXPORT int cb_depth_step(void* x, int64_t ldx, int64_t plane, const void* y, int64_t ldy, const void* dwa, const void* gain,
                             void* h, int64_t ldh, const void* rows, int64_t n, int64_t W, float eps, int64_t center, int64_t store,
                             int64_t f32, void* stream) {
-  if (!x || n < 1 || n > 65535 || W < 1 || plane < 0 || (h && !gain) || (rows && store)) return CB_ERR_ARG;
+  if (!x || n < 1 || n > 65535 || W < 1 || plane < 0 || plane >= kMaxPlanes || (h && !gain) || (rows && store)) return CB_ERR_ARG;
   if (ldx < (plane + (dwa && store ? 2 : 1)) * W) return CB_ERR_ARG;
   DepthArgs a;
   a.x = (float*)x; a.ldx = ldx; a.plane = (int)plane; a.y = y; a.ldy = ldy; a.dwa = (const float*)dwa; a.gain = (const float*)gain;

@@ -45,6 +45,7 @@ struct GemmArgs {
   // adds the partials in slice order and writes the result, so the sum does not depend on timing.
   int splits; float* ws; unsigned* tickets;
   int c_f32 = 0;                   // C is fp32 instead of bf16 (gate pre-activations, logits)
+  float* C2 = nullptr; int64_t ldc2 = 0; int n_main = 0;   // columns from n_main on leave as fp32 in C2 (null: none)
   int act = 0; float act_a = 0.f, act_b = 0.f;   // 1: xIELU epilogue with these coefficients
 };
 struct TileCoord { int m0, row_end, n0, brow; };
@@ -249,6 +250,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.C) + (int64_t)grow * a.ldc + gcol) = f;
               continue;
             }
+            if (a.C2 && gcol >= a.n_main) {
+              *reinterpret_cast<float4*>(a.C2 + (int64_t)grow * a.ldc2 + gcol - a.n_main) = f;
+              continue;
+            }
             const __nv_bfloat162 lo = __floats2bfloat162_rn(f.x, f.y), hi = __floats2bfloat162_rn(f.z, f.w);
             uint2 o;
             o.x = *reinterpret_cast<const uint32_t*>(&lo);
@@ -290,8 +295,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
 #pragma unroll
               for (int i = 0; i < 8; ++i) f[i] += g[i];
             }
-            if (a.c_f32) {
-              float4* fp = reinterpret_cast<float4*>(reinterpret_cast<float*>(a.C) + (int64_t)row * a.ldc + col0 + v * 8);
+            if (a.c_f32 || (a.C2 && col0 + v * 8 >= a.n_main)) {
+              float4* fp = a.c_f32 ? reinterpret_cast<float4*>(reinterpret_cast<float*>(a.C) + (int64_t)row * a.ldc + col0 + v * 8)
+                                   : reinterpret_cast<float4*>(a.C2 + (int64_t)row * a.ldc2 + col0 + v * 8 - a.n_main);
               fp[0] = make_float4(f[0], f[1], f[2], f[3]);
               fp[1] = make_float4(f[4], f[5], f[6], f[7]);
             } else {
@@ -408,6 +414,8 @@ int cb_gemm_pair_run(const void* A, int64_t lda, const void* W, int64_t ldw, voi
                      const void* pf, int64_t pf_seq, void* status, void* stream);
 int cb_gemm_pair_xielu(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int64_t M, int64_t N, int64_t K,
                        int tile, float act_a, float act_b, void* status, void* stream);
+int cb_gemm_pair_mixed(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, void* C2, int64_t ldc2, int64_t n_main,
+                       int64_t M, int64_t N, int64_t K, int tile, void* status, void* stream);
 
 // C[M,N] (bf16) = A[M,K] (bf16) x W[N,K]^T (bf16) (+ residual[M,N]).  K % 8 == 0, N % 8 == 0.
 // bn_hint: 0 = choose (CTA pairs for more than 256 rows), 64/128/160/256 = one-CTA kernel with that tile
@@ -473,6 +481,42 @@ CB_EXPORT int cb_gemm_bf16_xielu(const void* A, int64_t lda, const void* W, int6
   a.g_count = a.g_row0 = a.g_rows = a.g_expert = nullptr;
   a.splits = splits; a.ws = (float*)ws; a.tickets = (unsigned*)tickets;
   a.act = 1; a.act_a = act_a; a.act_b = act_b;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (bn == 256) return launch_gemm<256, 4, false>(tmA, tmB, a, sms, st);
+  if (bn == 160) return launch_gemm<160, 5, false>(tmA, tmB, a, sms, st);
+  if (bn == 128) return launch_gemm<128, 6, false>(tmA, tmB, a, sms, st);
+  return launch_gemm<64, 8, false>(tmA, tmB, a, sms, st);
+}
+
+// One product, two results: columns [0, n_main) of A[M,K] x W[N,K]^T as bf16 in C, the others (gate pre-activations) as
+// fp32 in C2.  n_main % 8 == 0; ws / tickets as above.
+CB_EXPORT int cb_gemm_bf16_mixed(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, void* C2, int64_t ldc2,
+                                 int64_t n_main, int64_t M, int64_t N, int64_t K, void* ws, int64_t ws_bytes, void* tickets, int64_t n_tickets,
+                                 void* status, void* stream) {
+  if (M < 1 || N < 1 || K < 1 || K % 8 || N % 8 || ldc % 8 || ldc2 % 4 || n_main % 8 || n_main < 0 || n_main > N || !C2 || !status) return CB_ERR_SHAPE;
+  const int tile = cb_gemm_pair_plan(M, N);
+  if (tile) return cb_gemm_pair_mixed(A, lda, W, ldw, C, ldc, C2, ldc2, n_main, M, N, K, tile, status, stream);
+  const int sms = sm_count();
+  int bn = pick_bn((int)M, (int)N, sms, true), splits = 1;
+  if (ws && tickets && M <= BM) {
+    int b2, s2;
+    plan_split(M, N, K * 2, &b2, &s2);
+    const int64_t tiles = (N + b2 - 1) / b2;
+    if (s2 > 1 && ws_bytes >= tiles * s2 * BM * b2 * (int64_t)sizeof(float) && n_tickets >= tiles) { bn = b2; splits = s2; }
+  }
+  CUtensorMap tmA, tmB;
+  int rc = cb_make_tmap_2d(&tmA, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, A, (uint64_t)M, (uint64_t)K, (uint64_t)lda, BM, 64);
+  if (rc) return rc;
+  rc = cb_make_tmap_2d(&tmB, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, W, (uint64_t)N, (uint64_t)K, (uint64_t)ldw, (uint32_t)bn, 64);
+  if (rc) return rc;
+  GemmArgs a;
+  a.C = C; a.ldc = ldc; a.residual = nullptr; a.ldr = 0; a.row_scale = nullptr; a.col_scale = nullptr;
+  a.M = (int)M; a.N = (int)N; a.K = (int)K; a.m_tiles = (int)((M + BM - 1) / BM); a.n_tiles = 0;
+  a.k_blocks = (int)((K + 63) / 64); a.status = (int*)status;
+  a.pf = nullptr; a.pf_seq = 0;
+  a.g_count = a.g_row0 = a.g_rows = a.g_expert = nullptr;
+  a.splits = splits; a.ws = (float*)ws; a.tickets = (unsigned*)tickets;
+  a.C2 = (float*)C2; a.ldc2 = ldc2; a.n_main = (int)n_main;
   cudaStream_t st = (cudaStream_t)stream;
   if (bn == 256) return launch_gemm<256, 4, false>(tmA, tmB, a, sms, st);
   if (bn == 160) return launch_gemm<160, 5, false>(tmA, tmB, a, sms, st);

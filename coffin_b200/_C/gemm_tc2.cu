@@ -37,6 +37,7 @@ struct PairArgs {
   int* status;
   const TpPfDev* pf; unsigned pf_seq;   // tensor-parallel prefill: rows go to this rank's peer-visible buffer (tp.cuh)
   int up_off;                      // SwiGLU form: W is [gate rows | up rows], the up rows start here; N counts outputs
+  float* C2 = nullptr; int64_t ldc2 = 0; int n_main = 0;   // columns from n_main on leave as fp32 in C2 (null: none)
   int act = 0; float act_a = 0.f, act_b = 0.f;   // 1: xIELU epilogue with these coefficients
 };
 
@@ -257,6 +258,12 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 #pragma unroll
                 for (int i = 0; i < 8; ++i) f[i] += g[i];
               }
+              if (a.C2 && col0 + v * 8 >= a.n_main) {
+                float4* fp = reinterpret_cast<float4*>(a.C2 + (int64_t)row * a.ldc2 + col0 + v * 8 - a.n_main);
+                fp[0] = make_float4(f[0], f[1], f[2], f[3]);
+                fp[1] = make_float4(f[4], f[5], f[6], f[7]);
+                continue;
+              }
               *reinterpret_cast<uint4*>(cp + v * 8) = float_to_bf16x8(f);
             }
           }
@@ -364,6 +371,21 @@ int cb_gemm_pair_run(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     if (tile == 320) return launch_pair<160, 2, 6, true>(A, lda, W, ldw, a, st);
     return CB_ERR_ARG;
   }
+  if (tile == 256) return launch_pair<256, 1, 6, false>(A, lda, W, ldw, a, st);
+  if (tile == 288) return launch_pair<144, 2, 6, false>(A, lda, W, ldw, a, st);
+  if (tile == 320) return launch_pair<160, 2, 6, false>(A, lda, W, ldw, a, st);
+  return CB_ERR_ARG;
+}
+
+// C[M, n_main] bf16 and C2[M, N - n_main] fp32 from one product, more than 256 rows; tile: 256, 288 or 320.
+int cb_gemm_pair_mixed(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, void* C2, int64_t ldc2, int64_t n_main,
+                       int64_t M, int64_t N, int64_t K, int tile, void* status, void* stream) {
+  PairArgs a;
+  a.C = (bf16*)C; a.ldc = ldc; a.residual = nullptr; a.ldr = 0; a.row_scale = nullptr; a.col_scale = nullptr;
+  a.M = (int)M; a.N = (int)N; a.K = (int)K; a.m_tiles = (int)((M + 255) / 256); a.n_tiles = 0;
+  a.k_blocks = 0; a.status = (int*)status; a.pf = nullptr; a.pf_seq = 0; a.up_off = 0;
+  a.C2 = (float*)C2; a.ldc2 = ldc2; a.n_main = (int)n_main;
+  cudaStream_t st = (cudaStream_t)stream;
   if (tile == 256) return launch_pair<256, 1, 6, false>(A, lda, W, ldw, a, st);
   if (tile == 288) return launch_pair<144, 2, 6, false>(A, lda, W, ldw, a, st);
   if (tile == 320) return launch_pair<160, 2, 6, false>(A, lda, W, ldw, a, st);

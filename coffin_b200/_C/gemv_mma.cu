@@ -423,6 +423,7 @@ __global__ void __launch_bounds__(kT, 3) gemv_mma_kernel(const MmaArgs a_in) {
   }
 }
 
+int g_mma_carve = 1;   // 0: leave the L1 / shared memory split to the driver
 int g_mma_sms = 0;
 int g_mma_ctas = 3;
 int g_mma_pf_rounds = 0;
@@ -522,7 +523,14 @@ int launch_mma(MmaArgs a, cudaStream_t st, int n_slots = 1) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return (int)cb_launch(kern, dim3((unsigned)grid_x, (unsigned)n_slots), dim3((unsigned)warps * 32), smem, st, a);
+  // shared memory for the CTAs that can be resident, the rest of the SM's memory for loads in flight
+  int64_t per_sm = warps_sm / warps;
+  const int64_t need_sm = (grid_x * n_slots + g_mma_sms - 1) / g_mma_sms;
+  if (per_sm > need_sm) per_sm = need_sm;
+  int64_t carve = (per_sm * (int64_t)(smem + 2048) * 100 + 228 * 1024 - 1) / (228 * 1024);
+  carve = carve < 1 ? 1 : (carve > 100 ? 100 : carve);
+  const dim3 grid((unsigned)grid_x, (unsigned)n_slots), block((unsigned)warps * 32);
+  return (int)(g_mma_carve ? cb_launch_carve((int)carve, kern, grid, block, smem, st, a) : cb_launch(kern, grid, block, smem, st, a));
 }
 
 }  // namespace
@@ -532,6 +540,8 @@ CB_EXPORT int cb_set_mma_gemv_opts(int64_t ctas_per_sm) { g_mma_ctas = ctas_per_
 CB_EXPORT int cb_set_mma_gemv_kcta(int64_t n) { g_mma_kcta_max = n < 1 ? 1 : (n > 4 ? 4 : (int)n); return 0; }
 // Weight batches (4 KB per warp each) staged in shared memory ahead of the dependency wait.
 CB_EXPORT int cb_set_mma_gemv_stage(int64_t n) { g_mma_stage = n < 0 ? 0 : (n > 4 ? 4 : (int)n); return 0; }
+// 0: the driver chooses the L1 / shared memory split of the GEMVs.
+CB_EXPORT int cb_set_mma_gemv_carve(int64_t on) { g_mma_carve = on ? 1 : 0; return 0; }
 // Sweep rounds prefetched into L2 ahead of the dependency wait (0 = none).
 CB_EXPORT int cb_set_mma_gemv_prefetch(int64_t rounds) { g_mma_pf_rounds = rounds < 0 ? 0 : (int)rounds; return 0; }
 

@@ -73,7 +73,7 @@ struct LatentArgs {
   float eps;
 };
 
-constexpr int kPT = 128;
+constexpr int kPT = 256, kPV = 8;        // values a thread keeps in registers
 template <typename TP, typename TA>
 __global__ void __launch_bounds__(kPT) latent_rows_kernel(const LatentArgs a) {
   __shared__ float red[32];
@@ -90,10 +90,22 @@ __global__ void __launch_bounds__(kPT) latent_rows_kernel(const LatentArgs a) {
     const int seg = a.row_seg ? a.row_seg[row] : row;
     out += ((int64_t)a.tables[(int64_t)seg * a.ldbt + pos / kPage] * kPage + pos % kPage) * a.ldk;
   }
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < n; c += kPT) { const float v = act_load(p + c); ss = fmaf(v, v, ss); }
+  float ss = 0.f, v[kPV];
+#pragma unroll
+  for (int i = 0; i < kPV; ++i) {
+    const int c = threadIdx.x + i * kPT;
+    v[i] = c < n ? act_load(p + c) : 0.f;
+  }
+#pragma unroll
+  for (int i = 0; i < kPV; ++i) ss = fmaf(v[i], v[i], ss);
+  for (int c = threadIdx.x + kPV * kPT; c < n; c += kPT) { const float x = act_load(p + c); ss = fmaf(x, x, ss); }
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)n + a.eps);
-  for (int c = threadIdx.x; c < n; c += kPT) act_store(out + c, act_load(p + c) * r * w[c]);
+#pragma unroll
+  for (int i = 0; i < kPV; ++i) {
+    const int c = threadIdx.x + i * kPT;
+    if (c < n) act_store(out + c, v[i] * r * w[c]);
+  }
+  for (int c = threadIdx.x + kPV * kPT; c < n; c += kPT) act_store(out + c, act_load(p + c) * r * w[c]);
   if (part) {
     const TP* q = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp + a.r_col;
     for (int i = threadIdx.x; 2 * i < a.rot; i += kPT) {
@@ -246,9 +258,9 @@ __global__ void __launch_bounds__(256) head_linear_f32_kernel(const HeadArgs a) 
 }
 
 // ---- decode ------------------------------------------------------------------------------------
-// One CTA per (key split, group of 16 MT heads, row): the pages of the split go through a two-stage cp.async ring and
+// One CTA per (key split, group of 16 MT heads, row), sixteen warps: the pages of the split go through a two-stage cp.async ring and
 // serve every head of the group - scores over the whole page row, weighted sums over its first cp columns.  Leaves
-// unnormalised sums and (max, denominator) for cb_attn_maps_finish.
+// unnormalised sums and (max, denominator) for latent_merge_kernel.
 struct LatentDecodeArgs {
   const void* q; int64_t ldq;            // absorbed queries [rows, H, ldk]
   const void* pool; int64_t ldk;         // page rows
@@ -257,19 +269,19 @@ struct LatentDecodeArgs {
   int H, cp, nsplit;
   float scale;
 };
-constexpr int kDT = 256;
-template <int MT, int NP2>               // NP2: 16-column pairs of the values per warp (cp <= 128 NP2)
+constexpr int kDT = 512, kPS = kPage + 4;
+template <int MT, int NP2>               // NP2: 16-column pairs of the values per warp (cp <= 256 NP2)
 __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecodeArgs a) {
-  constexpr int PP = kPage + 8;
+  constexpr int PP = kPage + 8, NH = 16 * MT, KS = 4 / MT;      // KS: slices of the page row that share a score
   extern __shared__ __align__(128) unsigned char smem[];
   const int LW = (int)a.ldk, LK = LW + 8, KPAGE = kPage * LK;
   bf16* ks = reinterpret_cast<bf16*>(smem);            // [2][kPage][LK]
-  bf16* qs = ks + 2 * KPAGE;                           // [16 MT][LK]
-  bf16* pa = qs + 16 * MT * LK;                        // [2][16 MT][PP]: heads, remainders
-  float* ps = reinterpret_cast<float*>(pa + 2 * 16 * MT * PP);   // [16 MT][kPage + 4] scores
-  __shared__ float w_s[16 * MT];
+  bf16* qs = ks + 2 * KPAGE;                           // [NH][LK]
+  bf16* pa = qs + NH * LK;                             // [2][NH][PP]: heads, remainders
+  float* ps = reinterpret_cast<float*>(pa + 2 * NH * PP);        // [KS][NH][kPS] partial scores
+  __shared__ float w_s[NH];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
-  const int split = blockIdx.x, row = blockIdx.z, h0 = blockIdx.y * 16 * MT, nh = min(16 * MT, a.H - h0);
+  const int split = blockIdx.x, row = blockIdx.z, h0 = blockIdx.y * NH, nh = min(NH, a.H - h0);
   griddep_launch();
   griddep_wait();
   const int pos = a.positions[row], seg = a.row_seg ? a.row_seg[row] : row;
@@ -294,7 +306,7 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
   };
   load(pg0);
   const bf16* q = reinterpret_cast<const bf16*>(a.q) + (int64_t)row * a.ldq + (int64_t)h0 * LW;
-  for (int r = warp; r < 16 * MT; r += kDT / 32)
+  for (int r = warp; r < NH; r += kDT / 32)
     for (int c = lane; c < pieces; c += 32)
       *reinterpret_cast<uint4*>(qs + r * LK + c * 8) = r < nh ? *reinterpret_cast<const uint4*>(q + (int64_t)r * LW + c * 8) : make_uint4(0, 0, 0, 0);
   float o[MT][NP2][2][4];
@@ -304,11 +316,14 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
     for (int i = 0; i < NP2; ++i)
 #pragma unroll
       for (int j = 0; j < 2; ++j) o[m][i][j][0] = o[m][i][j][1] = o[m][i][j][2] = o[m][i][j][3] = 0.f;
-  float m_run[2 * MT], l_run[2 * MT];                  // of heads warp + 8 i
+  float m_run[MT], l_run[MT];                          // of heads warp + 16 i
 #pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+  for (int i = 0; i < MT; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
   const float f = a.scale * kLog2e;
   const int ksteps = LW / 16, np = a.cp / 16;
+  // scores: a warp takes 16 keys, one head tile and one slice of the page row
+  const int kg = warp & 3, mt = (warp >> 2) % MT, sl = (warp >> 2) / MT;
+  const int kper = (ksteps + KS - 1) / KS, k0 = sl * kper, k1 = min(ksteps, k0 + kper);
   for (int pg = pg0; pg < pg1; ++pg) {
     if (pg + 1 < pg1) {
       load(pg + 1);
@@ -318,59 +333,60 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
     }
     __syncthreads();
     const bf16* kt = ks + (pg & 1) * KPAGE;
-    // scores of keys 8 warp .. 8 warp + 7; two chains of k-steps
     {
-      float s[MT][2][4];
+      float s[2][2][4];                                // [chain][key half]
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+      for (int c = 0; c < 2; ++c)
 #pragma unroll
-        for (int j = 0; j < 2; ++j) s[m][j][0] = s[m][j][1] = s[m][j][2] = s[m][j][3] = 0.f;
-      const bf16* kr = kt + (warp * 8 + (lane & 7)) * LK + (lane >> 3) * 8;
-      const bf16* qr = qs + (lane & 15) * LK + (lane >> 4) * 8;
-      int k = 0;
-#pragma unroll 2
-      for (; k + 2 <= ksteps; k += 2) {
-        uint32_t b[4];
-        ldsm4(b, kr + k * 16);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a0[4], a1[4];
-          ldsm4(a0, qr + m * 16 * LK + k * 16);
-          ldsm4(a1, qr + m * 16 * LK + k * 16 + 16);
-          mma(s[m][0], a0, b[0], b[1]);
-          mma(s[m][1], a1, b[2], b[3]);
-        }
+        for (int j = 0; j < 2; ++j) s[c][j][0] = s[c][j][1] = s[c][j][2] = s[c][j][3] = 0.f;
+      const bf16* kr = kt + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * LK + ((lane >> 3) & 1) * 8;
+      const bf16* qr = qs + (mt * 16 + (lane & 15)) * LK + (lane >> 4) * 8;
+      int k = k0;
+#pragma unroll 3
+      for (; k + 2 <= k1; k += 2) {
+        uint32_t a0[4], a1[4], b0[4], b1[4];
+        ldsm4(a0, qr + k * 16);
+        ldsm4(b0, kr + k * 16);
+        ldsm4(a1, qr + k * 16 + 16);
+        ldsm4(b1, kr + k * 16 + 16);
+        mma(s[0][0], a0, b0[0], b0[1]);
+        mma(s[0][1], a0, b0[2], b0[3]);
+        mma(s[1][0], a1, b1[0], b1[1]);
+        mma(s[1][1], a1, b1[2], b1[3]);
       }
-      if (k < ksteps) {                                // odd number of k-steps: the lanes of the second half re-read the first
-        uint32_t b[4];
-        ldsm4(b, kt + (warp * 8 + (lane & 7)) * LK + ((lane >> 3) & 1) * 8 + k * 16);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a0[4];
-          ldsm4(a0, qr + m * 16 * LK + k * 16);
-          mma(s[m][0], a0, b[0], b[1]);
-        }
+      if (k < k1) {
+        uint32_t a0[4], b0[4];
+        ldsm4(a0, qr + k * 16);
+        ldsm4(b0, kr + k * 16);
+        mma(s[0][0], a0, b0[0], b0[1]);
+        mma(s[0][1], a0, b0[2], b0[3]);
       }
+      float* pd = ps + (sl * NH + mt * 16 + g4) * kPS + kg * 16 + t4 * 2;
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int key = warp * 8 + t4 * 2 + (e & 1), hd = m * 16 + g4 + (e >> 1) * 8;
-          ps[hd * (kPage + 4) + key] = pg * kPage + key <= pos ? (s[m][0][e] + s[m][1][e]) * f : -INFINITY;
-        }
+      for (int j = 0; j < 2; ++j) {
+        *reinterpret_cast<float2*>(pd + j * 8) = make_float2(s[0][j][0] + s[1][j][0], s[0][j][1] + s[1][j][1]);
+        *reinterpret_cast<float2*>(pd + 8 * kPS + j * 8) = make_float2(s[0][j][2] + s[1][j][2], s[0][j][3] + s[1][j][3]);
+      }
     }
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < 2 * MT; ++i) {
-      const int hd = warp + 8 * i;
-      const float2 x = *reinterpret_cast<const float2*>(ps + hd * (kPage + 4) + 2 * lane);
+    for (int i = 0; i < MT; ++i) {
+      const int hd = warp + 16 * i, key = pg * kPage + 2 * lane;
+      float2 x = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int c = 0; c < KS; ++c) {
+        const float2 p = *reinterpret_cast<const float2*>(ps + (c * NH + hd) * kPS + 2 * lane);
+        x.x += p.x; x.y += p.y;
+      }
+      x.x = key <= pos ? x.x * f : -INFINITY;
+      x.y = key + 1 <= pos ? x.y * f : -INFINITY;
       const float mn = fmaxf(m_run[i], warp_max(fmaxf(x.x, x.y)));     // finite: the first key of a walked page is visible
       float e0 = ex2(x.x - mn), e1 = ex2(x.y - mn);
       const float w = ex2(m_run[i] - mn);
-      l_run[i] = l_run[i] * w + warp_sum(e0 + e1);
+      l_run[i] = l_run[i] * w + e0 + e1;               // this lane's share
       m_run[i] = mn;
       *reinterpret_cast<uint32_t*>(pa + hd * PP + 2 * lane) = split_head(e0, e1);
-      *reinterpret_cast<uint32_t*>(pa + (16 * MT + hd) * PP + 2 * lane) = pack_bf162(e0, e1);
+      *reinterpret_cast<uint32_t*>(pa + (NH + hd) * PP + 2 * lane) = pack_bf162(e0, e1);
       if (lane == 0) w_s[hd] = w;
     }
     __syncthreads();
@@ -392,7 +408,7 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
       }
 #pragma unroll
       for (int i = 0; i < NP2; ++i) {
-        const int cp = warp + 8 * i;
+        const int cp = warp + 16 * i;
         if (cp < np) {
           uint32_t b[4];
           ldsm4t(b, kt + (k * 16 + (lane & 15)) * LK + cp * 16 + (lane >> 4) * 8);
@@ -400,6 +416,9 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
           for (int m = 0; m < MT; ++m) {
             mma(o[m][i][0], ph[m], b[0], b[1]);
             mma(o[m][i][1], ph[m], b[2], b[3]);
+          }
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
             mma(o[m][i][0], pl[m], b[0], b[1]);
             mma(o[m][i][1], pl[m], b[2], b[3]);
           }
@@ -412,29 +431,63 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
   for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int i = 0; i < NP2; ++i) {
-      if (warp + 8 * i >= np) continue;
+      if (warp + 16 * i >= np) continue;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int hd = m * 16 + g4 + 8 * e, c = (warp + 8 * i) * 16 + j * 8 + t4 * 2;
+          const int hd = m * 16 + g4 + 8 * e, c = (warp + 16 * i) * 16 + j * 8 + t4 * 2;
           if (hd < nh)
             *reinterpret_cast<float2*>(a.part_o + ((vh0 + hd) * a.nsplit + split) * a.cp + c) = make_float2(o[m][i][j][2 * e], o[m][i][j][2 * e + 1]);
         }
     }
 #pragma unroll
-  for (int i = 0; i < 2 * MT; ++i) {
-    const int hd = warp + 8 * i;
+  for (int i = 0; i < MT; ++i) {
+    const int hd = warp + 16 * i;
+    const float l = warp_sum(l_run[i]);
     if (hd < nh && lane == 0) {
       float* ml = a.part_ml + ((vh0 + hd) * a.nsplit + split) * 2;
       ml[0] = m_run[i] * (1.f / kLog2e);
-      ml[1] = l_run[i];
+      ml[1] = l;
     }
   }
 }
 
+// merge of the key splits: 128 columns of one (row, head) per CTA, two groups of threads share the splits
+template <typename TA>
+__global__ void __launch_bounds__(256) latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                           const int* __restrict__ positions, TA* __restrict__ out, int64_t ldo, int H,
+                                                           int cp, int nsplit) {
+  __shared__ float sum_s[128];
+  const int tid = threadIdx.x, lane = tid & 31, h = blockIdx.y, c = blockIdx.x * 128 + (tid & 127), sg = tid >> 7;
+  const int64_t row = blockIdx.z;
+  griddep_launch();
+  griddep_wait();
+  if (positions[row] < 0) return;
+  const int64_t vh = row * H + h;
+  const float* ml = part_ml + vh * nsplit * 2;
+  float2 v[2];                                         // splits lane and lane + 32
+#pragma unroll
+  for (int k = 0; k < 2; ++k)
+    v[k] = lane + 32 * k < nsplit ? *reinterpret_cast<const float2*>(ml + 2 * (lane + 32 * k)) : make_float2(-INFINITY, 0.f);
+  // splits are filled from the front
+  const int used = __popc(__ballot_sync(0xffffffffu, v[0].x != -INFINITY)) + __popc(__ballot_sync(0xffffffffu, v[1].x != -INFINITY));
+  const float M = warp_max(fmaxf(v[0].x, v[1].x));
+  float fac[2];
+#pragma unroll
+  for (int k = 0; k < 2; ++k) fac[k] = v[k].x == -INFINITY ? 0.f : expf(v[k].x - M);
+  const float inv = 1.f / warp_sum(fac[0] * v[0].y + fac[1] * v[1].y);
+  const float* po = part_o + vh * nsplit * cp + min(c, cp - 1);
+  float acc = 0.f;
+#pragma unroll 8
+  for (int s = sg; s < used; s += 2) acc = fmaf(__shfl_sync(0xffffffffu, s < 32 ? fac[0] : fac[1], s & 31), po[(int64_t)s * cp], acc);
+  if (sg) sum_s[tid & 127] = acc;
+  __syncthreads();
+  if (!sg && c < cp) act_store(out + row * ldo + (int64_t)h * cp + c, (acc + sum_s[tid]) * inv);
+}
+
 size_t decode_smem(int mt, int64_t lw) {
-  return sizeof(bf16) * (size_t)(2 * kPage * (lw + 8) + 16 * mt * (lw + 8) + 2 * 16 * mt * (kPage + 8)) + sizeof(float) * 16 * mt * (kPage + 4);
+  return sizeof(bf16) * (size_t)(2 * kPage * (lw + 8) + 16 * mt * (lw + 8) + 2 * 16 * mt * (kPage + 8)) + sizeof(float) * 64 * kPS;
 }
 template <int MT, int NP2>
 int launch_decode(const LatentDecodeArgs& a, int rows, cudaStream_t st) {
@@ -524,10 +577,11 @@ CB_EXPORT int cb_latent_decode_ok(int64_t ldk, int64_t cp) {
 }
 
 // Absorbed attention of `rows` queries [rows, H, ldk] against the pages (their own rows appended before): key splits into
-// part_o [rows, H, nsplit, cp] / part_ml.
+// part_o [rows, H, nsplit, cp] / part_ml.  tiles: groups of 16 heads a CTA serves (1 or 2).
 CB_EXPORT int cb_latent_decode(const void* q, int64_t ldq, const void* pool, int64_t ldk, const void* tables, int64_t ldbt,
                                const void* row_seg, const void* positions, void* part_o, void* part_ml, int64_t rows, int64_t H, int64_t cp,
-                               int64_t nsplit, float scale, void* stream) {
+                               int64_t nsplit, int64_t tiles, float scale, void* stream) {
+  if (tiles < 1 || tiles > 2) return CB_ERR_ARG;
   if (!q || !pool || !tables || !positions || !part_o || !part_ml || rows < 1 || rows > 65535 || H < 1 || nsplit < 1 || nsplit > 64)
     return CB_ERR_ARG;
   if (!cb_latent_decode_ok(ldk, cp) || ldq % 8 || ((uintptr_t)q & 15) || ((uintptr_t)pool & 15)) return CB_ERR_SHAPE;
@@ -537,12 +591,19 @@ CB_EXPORT int cb_latent_decode(const void* q, int64_t ldq, const void* pool, int
   a.nsplit = (int)nsplit; a.scale = scale;
   cudaStream_t st = (cudaStream_t)stream;
   const int r = (int)rows;
-  if (H <= 16) {
-    if (cp <= 128) return launch_decode<1, 1>(a, r, st);
-    if (cp <= 256) return launch_decode<1, 2>(a, r, st);
-    return launch_decode<1, 4>(a, r, st);
-  }
-  if (cp <= 128) return launch_decode<2, 1>(a, r, st);
-  if (cp <= 256) return launch_decode<2, 2>(a, r, st);
-  return launch_decode<2, 4>(a, r, st);
+  if (tiles == 1) return cp <= 256 ? launch_decode<1, 1>(a, r, st) : launch_decode<1, 2>(a, r, st);
+  return cp <= 256 ? launch_decode<2, 1>(a, r, st) : launch_decode<2, 2>(a, r, st);
+}
+
+// out[row, h, :cp] = average of the key splits left by cb_latent_decode.  f32: out is fp32 instead of bf16.
+CB_EXPORT int cb_latent_merge(const void* part_o, const void* part_ml, const void* positions, void* out, int64_t ldo, int64_t rows, int64_t H,
+                              int64_t cp, int64_t nsplit, int64_t f32, void* stream) {
+  if (!part_o || !part_ml || !positions || !out || rows < 1 || rows > 65535 || H < 1 || H > 65535 || cp < 1 || nsplit < 1 || nsplit > 64) return CB_ERR_ARG;
+  const dim3 grid((unsigned)((cp + 127) / 128), (unsigned)H, (unsigned)rows), block(256);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (f32)
+    return (int)cb_launch(latent_merge_kernel<float>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml, (const int*)positions,
+                          (float*)out, ldo, (int)H, (int)cp, (int)nsplit);
+  return (int)cb_launch(latent_merge_kernel<bf16>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml, (const int*)positions,
+                        (bf16*)out, ldo, (int)H, (int)cp, (int)nsplit);
 }

@@ -8,9 +8,6 @@
 //              S <- exp(f + m' - m) S + exp(i - m) k v^T;  n likewise with k;
 //              o = S^T q / (max(|n.q|, exp(-m)) + 1e-6)
 //            o is RMS-normed per head, weighted and multiplied by a sigmoid gate.
-//   ssd    : state space with a scalar decay per head (Mamba-2),
-//              S <- exp(-exp(A_log) dt) S + dt B x^T;  y = S^T C + D x       (k = B, q = C shared by a group of heads, v = x)
-//            behind a short causal convolution with bias + SiLU; y leaves in fp32, gate and norm follow (ssd.cu).
 //
 // One cluster of CTAs per (head, sequence): every CTA owns `jc` value columns of the head's state in registers
 // (the columns of S never interact), computes the head's q / k / decays itself, and only the RMS norm over the
@@ -125,7 +122,6 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
   const int cq = jc >> 2, RG = kT / cq, q4 = tid % cq, rg = tid / cq;
   const bool act_thr = rg < RG;
   const int j0 = rank * jc, ncol = min(jc, dv - j0);   // ncol > 0 by construction of the grid
-  constexpr bool kConv = KIND != LINREC_MLSTM;          // short convolution ahead of the recurrence
   constexpr bool kLow = KIND == LINREC_DELTA && sizeof(TA) == 2 && LOW;
   const bool low_a = kLow && !a.dec && a.ra <= 256, low_g = kLow && !a.og && a.rg <= 256;
   LowRank<kLow ? (RMAX <= 8 ? 8 : 4) : 1> lra;
@@ -140,24 +136,17 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
   auto channel = [&](int e) {
     return e < dk ? (int64_t)(qb + e) : (e < 2 * dk ? a.k_col + qb + e - dk : a.v_col + (int64_t)h * dv + j0 + e - 2 * dk);
   };
-  float p_dt = 0.f, p_ea = 0.f, p_bi = 0.f, p_bf = 0.f, p_cb[2] = {0.f, 0.f};
-  if (KIND == LINREC_SSD) {
-    p_dt = a.dt_bias[h];
-    p_bi = a.D[h];
-#pragma unroll
-    for (int u = 0; u < 2; ++u)
-      if (tid + u * kT < nch) p_cb[u] = a.conv_b[channel(tid + u * kT)];
-  }
+  float p_dt = 0.f, p_ea = 0.f, p_bi = 0.f, p_bf = 0.f;
   if (KIND == LINREC_MLSTM) { p_bi = a.gate_b[h]; p_bf = a.gate_b[a.H + h]; }
-  if (kConv) {
+  if (KIND == LINREC_DELTA) {
 #pragma unroll
     for (int u = 0; u < 2; ++u)
       pcw[u] = taps4 && tid + u * kT < nch ? *reinterpret_cast<const float4*>(a.conv_w + channel(tid + u * kT) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     p_ea = expf(a.A_log[h]);
-    if (KIND == LINREC_DELTA && tid < dk) p_dt = a.dt_bias[(int64_t)h * dk + tid];
+    if (tid < dk) p_dt = a.dt_bias[(int64_t)h * dk + tid];
   }
   const float* nw = a.norm_w + (KIND == LINREC_MLSTM ? (int64_t)h * dv : 0) + j0;
-  const float p_nw = KIND != LINREC_SSD && tid < ncol ? nw[tid] : 0.f;
+  const float p_nw = tid < ncol ? nw[tid] : 0.f;
   griddep_launch();
   griddep_wait();
   const int row0 = a.seg_row ? a.seg_row[seg] : seg;
@@ -204,7 +193,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     if (KIND == LINREC_DELTA) {
       if (tid < dk && a.dec) x_a = a.dec[row * a.ldd + (int64_t)h * dk + tid];
       if (tid < ncol && a.og) x_og = act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + vch);
-    } else if (KIND == LINREC_MLSTM) {
+    } else {
       if (tid < dk) {
         x_a = act_load(pr + (int64_t)h * dk + tid);
         x_b = act_load(pr + a.k_col + (int64_t)h * dk + tid);
@@ -214,7 +203,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
         x_og = act_load(reinterpret_cast<const TP*>(a.og) + row * a.ldo + vch);
       }
     }
-    if (kConv) {
+    if (KIND == LINREC_DELTA) {
       // short convolution: channels q, k, v of this CTA spread over the block, four taps requested together (in a decode
       // step all but the newest come from the ring)
       auto tap = [&](int64_t ch, int j) {                // the row a tap reads is the same for every channel
@@ -236,22 +225,16 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
 #pragma unroll
         for (int u = 0; u < 2; ++u)
           if (tid + u * kT < nch)
-            put(tid + u * kT, fmaf(pcw[u].w, x[u][3], fmaf(pcw[u].z, x[u][2], fmaf(pcw[u].y, x[u][1], fmaf(pcw[u].x, x[u][0], p_cb[u])))));
+            put(tid + u * kT, fmaf(pcw[u].w, x[u][3], fmaf(pcw[u].z, x[u][2], fmaf(pcw[u].y, x[u][1], pcw[u].x * x[u][0]))));
       }
 #pragma unroll 1
       for (int e = tid + (taps4 ? 2 * kT : 0); e < nch; e += kT) {
         const int64_t ch = channel(e);
-        float acc = KIND == LINREC_SSD ? a.conv_b[ch] : 0.f;
+        float acc = 0.f;
 #pragma unroll 1
         for (int j = 0; j < a.taps; ++j) acc = fmaf(a.conv_w[ch * a.taps + j], tap(ch, j), acc);
         put(e, acc);
       }
-    }
-    if (KIND == LINREC_SSD) {
-      const float dt = softplus_s(gate0 + p_dt);
-      aa = __expf(-p_ea * dt);
-      bb = dt;
-    } else if (KIND == LINREC_DELTA) {
 #pragma unroll 1
       for (int c = tid; c < lown; c += kT) {
         const int na = a.dec ? 0 : (int)a.ra;
@@ -314,10 +297,10 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     __syncthreads();
     // ---- state pass: partial sums of the read-outs over this thread's rows
     float pa[4] = {}, pb[4] = {};
-    if (KIND != LINREC_DELTA) {
+    if (KIND == LINREC_MLSTM) {
       float v4[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v4[e] = q4 * 4 + e < ncol ? (KIND == LINREC_SSD ? bb : 1.f) * sv[q4 * 4 + e] : 0.f;
+      for (int e = 0; e < 4; ++e) v4[e] = q4 * 4 + e < ncol ? sv[q4 * 4 + e] : 0.f;
 #pragma unroll
       for (int i = 0; i < RMAX; ++i) {
         const int r = rg + i * RG;
@@ -369,8 +352,6 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
         const float u = c < ncol ? bb * (sv[c] - d) : 0.f;
         su[c] = u;
         so[c] = fmaf(u, kq, b);
-      } else if (KIND == LINREC_SSD) {
-        so[c] = c < ncol ? fmaf(p_bi, sv[c], b) : 0.f;
       } else {
         so[c] = b / den;
       }
@@ -389,12 +370,6 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
           for (int e = 0; e < 4; ++e) S[i][e] = fmaf(k, u4[e], S[i][e]);
         }
       }
-    }
-    if (KIND == LINREC_SSD) {
-      float* out = reinterpret_cast<float*>(a.act) + row * a.lda + (int64_t)h * dv + j0;
-      for (int c = tid; c < ncol; c += kT) out[c] = so[c];
-      __syncthreads();
-      continue;
     }
     // ---- head norm and output gate
     float ss = 0.f;
@@ -428,7 +403,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     for (int c = tid; c < dk; c += kT) a.n[((int64_t)slot * a.H + h) * dk + c] = sg[c];
     if (tid == 0) a.m[(int64_t)slot * a.H + h] = mrun;
   }
-  if (kConv && nrow == 1) {
+  if (KIND == LINREC_DELTA && nrow == 1) {
     // one token: its raw rows enter the ring here (no reader of this step looks at that entry); longer segments
     // leave it to linrec_ring_kernel, which runs after every reader
     TA* w = reinterpret_cast<TA*>(a.ring) + ((int64_t)slot * (a.ring_mask + 1) + (pos0 & a.ring_mask)) * a.ring_w;
@@ -539,11 +514,6 @@ CB_EXPORT int cb_linrec_step(const void* args, int64_t kind, int64_t segs, int64
     if (!a.ring || a.taps < 1 || a.taps > a.ring_mask + 1 || a.ra % 8 || a.rg % 8) return CB_ERR_ARG;
     if (f32) return dispatch_step<LINREC_DELTA, float, float>(a, (int)segs, st);
     return p_f32 ? dispatch_step<LINREC_DELTA, float, bf16>(a, (int)segs, st) : dispatch_step<LINREC_DELTA, bf16, bf16>(a, (int)segs, st);
-  }
-  if (kind == LINREC_SSD) {
-    if (!a.ring || a.taps < 1 || a.taps > a.ring_mask + 1 || !a.A_log || !a.dt_bias || !a.D || !a.conv_b || !a.conv_w) return CB_ERR_ARG;
-    if (f32) return dispatch_step<LINREC_SSD, float, float>(a, (int)segs, st);
-    return p_f32 ? dispatch_step<LINREC_SSD, float, bf16>(a, (int)segs, st) : dispatch_step<LINREC_SSD, bf16, bf16>(a, (int)segs, st);
   }
   if (kind == LINREC_MLSTM) {
     if (!a.n || !a.m || !a.og || !(a.cap > 0.f)) return CB_ERR_ARG;

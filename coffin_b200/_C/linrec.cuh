@@ -1,8 +1,8 @@
-// Arguments shared by the recurrent-state kernels (linrec.cu: token by token; linrec_chunk.cu, ssd.cu: prompts in chunks).
+// Arguments shared by the recurrent-state kernels (linrec.cu: token by token; linrec_chunk.cu: prompts in chunks; ssd.cu: both for state-space layers).
 #pragma once
 #include "act_type.cuh"
 
-enum LinrecKind : int { LINREC_DELTA = 0, LINREC_MLSTM = 1, LINREC_SSD = 2 };
+enum LinrecKind : int { LINREC_DELTA = 0, LINREC_MLSTM = 1 };      // state-space layers (ssd.cu) have entry points of their own
 
 // Column layout of a projection row: q | k | v | ... ; the first ring_w columns pass the short convolution of the delta
 // and state-space layers (channel index == column index).  State-space layers: q = C, k = B, v = x.

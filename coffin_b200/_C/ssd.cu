@@ -11,7 +11,8 @@
 //
 // a is the cumulated log decay, only differences that are <= 0 are exponentiated.  The 32-bit factors (the state, the
 // decayed scores, the weighted values) enter the products as bf16 head + remainder, sums and state are fp32.
-// Token by token (decoding, 32-bit mode, odd sizes): linrec.cu.
+// `step` goes token by token (decoding, 32-bit mode, odd sizes): one CTA per sequence and up to four heads of a group, which
+// convolves their channels and streams their state through registers once per token.
 #include "linrec.cuh"
 
 namespace {
@@ -138,6 +139,175 @@ __global__ void __launch_bounds__(kCT) ssd_conv_kernel(const SsdArgs s, int cblo
   }
 }
 
+// ---- step --------------------------------------------------------------------------------------
+constexpr int kNT = 256, kHPC = 4, kRB = 8;
+// V: state columns per thread (4: dv is a multiple of 4)
+template <typename TP, typename TA, int V>
+__global__ void __launch_bounds__(kNT, 2) ssd_step_kernel(const SsdArgs s, int hpc) {
+  const LinrecArgs& a = s.r;
+  extern __shared__ __align__(16) float sm[];
+  const int tid = threadIdx.x, seg = blockIdx.y, dk = a.dk, dv = a.dv;
+  const int hpg = a.H / a.G, cpg = (hpg + hpc - 1) / hpc, g = blockIdx.x / cpg, h0 = g * hpg + (blockIdx.x % cpg) * hpc;
+  const int nh = min(hpc, (g + 1) * hpg - h0);
+  const int CQ = min(dv / V, kNT), RG = kNT / CQ, q = tid % CQ, rg = tid / CQ;         // column unit and row group of this thread
+  float* sc = sm;                                      // [dk]
+  float* sb = sc + dk;                                 // [dk]
+  float* sx = sb + dk;                                 // [hpc][dv]
+  float* part = sx + hpc * dv;                         // [hpc][RG][dv]
+  __shared__ float dt_s[kHPC], de_s[kHPC];
+  const int nch = 2 * dk + nh * dv;
+  auto channel = [&](int e) {                          // C, B, then the values of the heads
+    return e < dk ? (int64_t)g * dk + e : (e < 2 * dk ? a.k_col + (int64_t)g * dk + e - dk : a.v_col + (int64_t)h0 * dv + e - 2 * dk);
+  };
+  const bool taps4 = a.taps == 4;
+  float4 pw[2];
+  float pb[2];
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const bool ok = tid + u * kNT < nch;
+    pw[u] = ok && taps4 ? *reinterpret_cast<const float4*>(a.conv_w + channel(tid + u * kNT) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    pb[u] = ok && a.conv_b ? a.conv_b[channel(tid + u * kNT)] : 0.f;
+  }
+  const float p_dt = tid < nh ? a.dt_bias[h0 + tid] : 0.f, p_ea = tid < nh ? expf(a.A_log[h0 + tid]) : 0.f;
+  griddep_launch();
+  griddep_wait();
+  const int row0 = a.seg_row ? a.seg_row[seg] : seg;
+  const int nrow = a.seg_row ? a.seg_row[seg + 1] - row0 : 1;
+  const int slot = a.seg_slot[seg], pos0 = a.seg_pos[seg];
+  if (slot < 0 || nrow < 1 || pos0 < 0) return;
+  float* Sg = a.S + ((int64_t)slot * a.H + h0) * dk * dv;
+  const TA* ring = reinterpret_cast<const TA*>(a.ring) + (int64_t)slot * (a.ring_mask + 1) * a.ring_w;
+  const TP* prow0 = reinterpret_cast<const TP*>(a.proj) + (int64_t)row0 * a.ldp;
+  const int per = (dk + RG - 1) / RG, nb = (per + kRB - 1) / kRB, items = nh * nb;      // blocks of kRB rows per head and thread
+  for (int cb = 0; cb * CQ * V < dv; ++cb) {           // more than kNT column units: one round after the other
+    const int c = (cb * CQ + q) * V;
+    const bool act = rg < RG && c < dv;
+    auto load = [&](int it, float (*f)[V]) {
+      const float* p = Sg + (int64_t)(it / nb) * dk * dv + c;
+#pragma unroll
+      for (int i = 0; i < kRB; ++i) {
+        const int r = rg + ((it % nb) * kRB + i) * RG;
+        if (V == 4) {
+          const float4 x = act && r < dk ? *reinterpret_cast<const float4*>(p + (int64_t)r * dv) : make_float4(0.f, 0.f, 0.f, 0.f);
+          f[i][0] = x.x; f[i][1 % V] = x.y; f[i][2 % V] = x.z; f[i][3 % V] = x.w;
+        } else {
+          f[i][0] = act && r < dk ? p[(int64_t)r * dv] : 0.f;
+        }
+      }
+    };
+    for (int t = 0; t < nrow; ++t) {
+      const int64_t row = row0 + t;
+      float nx[kRB][V];
+      load(0, nx);                                     // in flight during the convolution
+      const float gate = tid < nh ? a.gates[row * a.ldg + h0 + tid] : 0.f;
+      auto tap = [&](int64_t ch, int j) {
+        const int src = t - (a.taps - 1) + j, p = pos0 + src;
+        float x = 0.f;
+        if (src >= 0) x = act_round<TA>(act_load(prow0 + (int64_t)src * a.ldp + ch));
+        else if (p >= 0) x = act_load(ring + (int64_t)(p & a.ring_mask) * a.ring_w + ch);
+        return x;
+      };
+      if (taps4) {
+        float x[2][4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) x[u][j] = tid + u * kNT < nch ? tap(channel(tid + u * kNT), j) : 0.f;
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+          if (tid + u * kNT < nch)                     // sc, sb and sx are adjacent
+            sm[tid + u * kNT] = silu_s(fmaf(pw[u].w, x[u][3], fmaf(pw[u].z, x[u][2], fmaf(pw[u].y, x[u][1], fmaf(pw[u].x, x[u][0], pb[u])))));
+      }
+#pragma unroll 1
+      for (int e = tid + (taps4 ? 2 * kNT : 0); e < nch; e += kNT) {
+        const int64_t ch = channel(e);
+        float acc = a.conv_b ? a.conv_b[ch] : 0.f;
+#pragma unroll 1
+        for (int j = 0; j < a.taps; ++j) acc = fmaf(a.conv_w[ch * a.taps + j], tap(ch, j), acc);
+        sm[e] = silu_s(acc);
+      }
+      if (tid < nh) {
+        const float dt = softplus_s(gate + p_dt);
+        dt_s[tid] = dt;
+        de_s[tid] = __expf(-p_ea * dt);
+      }
+      __syncthreads();
+      float acc[V];
+#pragma unroll 1
+      for (int it = 0; it < items; ++it) {
+        float cur[kRB][V];
+#pragma unroll
+        for (int i = 0; i < kRB; ++i)
+#pragma unroll
+          for (int v = 0; v < V; ++v) cur[i][v] = nx[i][v];
+        if (it + 1 < items) load(it + 1, nx);
+        const int hi = it / nb, b = it % nb;
+        const float de = de_s[hi], dt = dt_s[hi];
+        float xv[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+          xv[v] = act ? dt * sx[hi * dv + c + v] : 0.f;
+          if (b == 0) acc[v] = 0.f;
+        }
+        float* p = Sg + (int64_t)hi * dk * dv + c;
+#pragma unroll
+        for (int i = 0; i < kRB; ++i) {
+          const int r = rg + (b * kRB + i) * RG;
+          if (act && r < dk) {
+            const float k = sb[r], cc = sc[r];
+#pragma unroll
+            for (int v = 0; v < V; ++v) {
+              cur[i][v] = fmaf(de, cur[i][v], k * xv[v]);
+              acc[v] = fmaf(cc, cur[i][v], acc[v]);
+            }
+            if (V == 4) *reinterpret_cast<float4*>(p + (int64_t)r * dv) = make_float4(cur[i][0], cur[i][1 % V], cur[i][2 % V], cur[i][3 % V]);
+            else p[(int64_t)r * dv] = cur[i][0];
+          }
+        }
+        if (act && b == nb - 1)
+#pragma unroll
+          for (int v = 0; v < V; ++v) part[(hi * RG + rg) * dv + c + v] = acc[v];
+      }
+      __syncthreads();
+      for (int e = tid; e < nh * CQ * V; e += kNT) {
+        const int hi = e / (CQ * V), col = cb * CQ * V + e % (CQ * V);
+        if (col >= dv) continue;
+        float y = a.D[h0 + hi] * sx[hi * dv + col];
+        for (int r = 0; r < RG; ++r) y += part[(hi * RG + r) * dv + col];
+        s.y[row * a.lda + (int64_t)(h0 + hi) * dv + col] = y;
+      }
+      __syncthreads();
+    }
+  }
+  if (nrow == 1) {
+    // one token: its raw rows enter the ring here (no reader of this step looks at that entry); longer segments
+    // leave it to cb_linrec_ring, which runs after every reader
+    TA* w = reinterpret_cast<TA*>(a.ring) + ((int64_t)slot * (a.ring_mask + 1) + (pos0 & a.ring_mask)) * a.ring_w;
+    for (int e = tid + (h0 == g * hpg ? 0 : 2 * dk); e < nch; e += kNT) {
+      const int64_t ch = channel(e);
+      act_store(w + ch, act_load(prow0 + ch));
+    }
+  }
+}
+
+template <typename TP, typename TA>
+int launch_step(const SsdArgs& s, int segs, cudaStream_t st) {
+  const LinrecArgs& a = s.r;
+  const int hpg = a.H / a.G;
+  int hpc = kHPC;
+  while (hpc > 1 && (int64_t)a.G * ((hpg + hpc - 1) / hpc) * segs < 200) hpc >>= 1;      // few sequences: one head per CTA
+  const bool v4 = a.dv % 4 == 0;
+  const int V = v4 ? 4 : 1, CQ = a.dv / V < kNT ? a.dv / V : kNT, RG = kNT / CQ;
+  const size_t smem = sizeof(float) * ((size_t)2 * a.dk + (size_t)hpc * a.dv * (1 + RG));
+  if (smem > 200 * 1024) return CB_ERR_SHAPE;
+  auto kern = v4 ? ssd_step_kernel<TP, TA, 4> : ssd_step_kernel<TP, TA, 1>;
+  if (smem > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)cb_launch(kern, dim3((unsigned)(a.G * ((hpg + hpc - 1) / hpc)), (unsigned)segs), dim3(kNT), smem, st, s, hpc);
+}
+
 // ---- scan --------------------------------------------------------------------------------------
 template <int NP>
 struct Plan {
@@ -149,8 +319,89 @@ struct Plan {
   static constexpr size_t bytes = sizeof(bf16) * (2 * TILE + 2 * Q * VP + 2 * NP * VP) + sizeof(float) * 4 * Q;
 };
 
+// read-outs of token rows 16 RG .. 16 RG + 15, columns 16 half .. + 15: scores against tokens 0 .. 16 RG + 15 and the
+// read-out of the old state share the C fragments
+template <int NP, int RG>
+__device__ __forceinline__ void read_out(const bf16* ct, const bf16* bt, const bf16* xt, const bf16* st, const float* av, const float* dtv,
+                                         int half, int lane, int m, int nv, float Dh, float* y, int64_t ldy) {
+  constexpr int P = NP + 8;
+  const int g4 = lane >> 2, t4 = lane & 3;
+  float G[2 * RG + 2][4], Y[2][4], Y2[2][4];
+#pragma unroll
+  for (int i = 0; i < 2 * RG + 2; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = 0.f;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
+    Y2[i][0] = Y2[i][1] = Y2[i][2] = Y2[i][3] = 0.f;
+  }
+  const bf16* cr = ct + (RG * 16 + (lane & 15)) * P + (lane >> 4) * 8;
+  const bf16* sr = st + (lane & 15) * VP + half * 16 + (lane >> 4) * 8;
+  const bf16* br = bt + ((lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
+#pragma unroll
+  for (int k = 0; k < NP / 16; ++k) {
+    uint32_t ca[4], sh[4], sl[4], b[RG + 1][4];
+    ldsm4(ca, cr + k * 16);
+    ldsm4t(sh, sr + k * 16 * VP);
+    ldsm4t(sl, sr + (NP + k * 16) * VP);
+#pragma unroll
+    for (int j = 0; j <= RG; ++j) ldsm4(b[j], br + j * 16 * P + k * 16);
+    mma(Y[0], ca, sh[0], sh[1]);
+    mma(Y[1], ca, sh[2], sh[3]);
+    mma(Y2[0], ca, sl[0], sl[1]);
+    mma(Y2[1], ca, sl[2], sl[3]);
+#pragma unroll
+    for (int j = 0; j <= RG; ++j) {
+      mma(G[2 * j], ca, b[j][0], b[j][1]);
+      mma(G[2 * j + 1], ca, b[j][2], b[j][3]);
+    }
+  }
+  const int tl = RG * 16 + g4, th = tl + 8;
+  const float al = av[tl], ah = av[th], el = ex2(al), eh = ex2(ah);
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    Y[i][0] = (Y[i][0] + Y2[i][0]) * el; Y[i][1] = (Y[i][1] + Y2[i][1]) * el;
+    Y[i][2] = (Y[i][2] + Y2[i][2]) * eh; Y[i][3] = (Y[i][3] + Y2[i][3]) * eh;
+    Y2[i][0] = Y2[i][1] = Y2[i][2] = Y2[i][3] = 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j <= RG; ++j) {
+    uint32_t mh[4], ml[4], b[4];
+    ldsm4t(b, xt + (j * 16 + (lane & 15)) * VP + half * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int p = 0; p < 2; ++p) {                                // tokens u, u + 1 of rows lo, then hi
+      const int u = j * 16 + p * 8 + t4 * 2;
+      const float2 au = *reinterpret_cast<const float2*>(av + u), du = *reinterpret_cast<const float2*>(dtv + u);
+      const float* gg = G[2 * j + p];
+      float x = gg[0] * (du.x * ex2(fminf(al - au.x, 0.f))), y = gg[1] * (du.y * ex2(fminf(al - au.y, 0.f)));
+      float z = gg[2] * (du.x * ex2(fminf(ah - au.x, 0.f))), w = gg[3] * (du.y * ex2(fminf(ah - au.y, 0.f)));
+      if (j == RG) {
+        if (u > tl) x = 0.f;
+        if (u + 1 > tl) y = 0.f;
+        if (u > th) z = 0.f;
+        if (u + 1 > th) w = 0.f;
+      }
+      mh[2 * p] = split_head(x, y); ml[2 * p] = pack_bf162(x, y);          // a0 / a2: row lo; a1 / a3: row hi
+      mh[2 * p + 1] = split_head(z, w); ml[2 * p + 1] = pack_bf162(z, w);
+    }
+    mma(Y[0], mh, b[0], b[1]);
+    mma(Y[1], mh, b[2], b[3]);
+    mma(Y2[0], ml, b[0], b[1]);
+    mma(Y2[1], ml, b[2], b[3]);
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = e ? th : tl, c = half * 16 + i * 8 + t4 * 2;
+      if (t < m && c < nv) {
+        const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(xt + t * VP + c));
+        *reinterpret_cast<float2*>(y + t * ldy + c) = make_float2(fmaf(Dh, x.x, Y[i][2 * e] + Y2[i][2 * e]), fmaf(Dh, x.y, Y[i][2 * e + 1] + Y2[i][2 * e + 1]));
+      }
+    }
+}
+
 template <int NP>
-__global__ void __launch_bounds__(kST) ssd_scan_kernel(const SsdArgs s) {
+__global__ void __launch_bounds__(kST, NP <= 128 ? 2 : 1) ssd_scan_kernel(const SsdArgs s) {
   using L = Plan<NP>;
   constexpr int P = L::P, MPW = L::MPW, NTW = L::NTW;
   const LinrecArgs& a = s.r;
@@ -250,83 +501,21 @@ __global__ void __launch_bounds__(kST) ssd_scan_kernel(const SsdArgs s) {
       *reinterpret_cast<uint4*>(xw + Q * VP + t * VP + c) = make_uint4(rm[0], rm[1], rm[2], rm[3]);
     }
     if (rg * 16 < m) {
-      // scores against tokens 0 .. 16 rg + 15 and the read-out of the old state share the C fragments
-      float G[8][4], Y[2][4], Y2[2][4];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = 0.f;
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
-        Y2[i][0] = Y2[i][1] = Y2[i][2] = Y2[i][3] = 0.f;
-      }
-#pragma unroll
-      for (int k = 0; k < NP / 16; ++k) {
-        if (k * 16 >= N) break;
-        uint32_t ca[4], b[4];
-        ldsm4(ca, ct + (rg * 16 + (lane & 15)) * P + k * 16 + (lane >> 4) * 8);
-        ldsm4t(b, st + (k * 16 + (lane & 15)) * VP + half * 16 + (lane >> 4) * 8);
-        mma(Y[0], ca, b[0], b[1]);
-        mma(Y[1], ca, b[2], b[3]);
-        ldsm4t(b, st + (NP + k * 16 + (lane & 15)) * VP + half * 16 + (lane >> 4) * 8);
-        mma(Y2[0], ca, b[0], b[1]);
-        mma(Y2[1], ca, b[2], b[3]);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          if (j > rg) break;
-          ldsm4(b, bt + (j * 16 + (lane & 7) + ((lane >> 4) << 3)) * P + k * 16 + ((lane >> 3) & 1) * 8);
-          mma(G[2 * j], ca, b[0], b[1]);
-          mma(G[2 * j + 1], ca, b[2], b[3]);
-        }
-      }
-      const int tl = rg * 16 + g4, th = tl + 8;
-      const float al = av[tl], ah = av[th], el = ex2(al), eh = ex2(ah);
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        Y[i][0] = (Y[i][0] + Y2[i][0]) * el; Y[i][1] = (Y[i][1] + Y2[i][1]) * el;
-        Y[i][2] = (Y[i][2] + Y2[i][2]) * eh; Y[i][3] = (Y[i][3] + Y2[i][3]) * eh;
-      }
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        if (j > rg) break;
-        uint32_t mh[4], ml[4], b[4];
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {                            // a0: row lo, tokens 2t..; a1: row hi; a2 / a3: tokens + 8
-          const int u = j * 16 + (q >> 1) * 8 + t4 * 2, t = q & 1 ? th : tl;
-          const float at = q & 1 ? ah : al;
-          float x = u <= t ? G[2 * j + (q >> 1)][(q & 1) * 2] * (dtv[u] * ex2(fminf(at - av[u], 0.f))) : 0.f;
-          float y = u + 1 <= t ? G[2 * j + (q >> 1)][(q & 1) * 2 + 1] * (dtv[u + 1] * ex2(fminf(at - av[u + 1], 0.f))) : 0.f;
-          mh[q] = split_head(x, y);
-          ml[q] = pack_bf162(x, y);
-        }
-        ldsm4t(b, xt + (j * 16 + (lane & 15)) * VP + half * 16 + (lane >> 4) * 8);
-        mma(Y[0], mh, b[0], b[1]);
-        mma(Y[1], mh, b[2], b[3]);
-        mma(Y[0], ml, b[0], b[1]);
-        mma(Y[1], ml, b[2], b[3]);
-      }
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int t = e ? th : tl, c = half * 16 + i * 8 + t4 * 2;
-          if (t < m && c < nv) {
-            const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(xt + t * VP + c));
-            *reinterpret_cast<float2*>(s.y + (int64_t)(row0 + ch * Q + t) * a.lda + (int64_t)h * a.dv + v0 + c) =
-                make_float2(fmaf(Dh, x.x, Y[i][2 * e]), fmaf(Dh, x.y, Y[i][2 * e + 1]));
-          }
-        }
+      float* y = s.y + (int64_t)(row0 + ch * Q) * a.lda + (int64_t)h * a.dv + v0;
+      if (rg == 0) read_out<NP, 0>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
+      else if (rg == 1) read_out<NP, 1>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
+      else if (rg == 2) read_out<NP, 2>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
+      else read_out<NP, 3>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
     }
     __syncthreads();                                             // weighted values in place, the old state has been read
     const float ge = ex2(aq);
 #pragma unroll
     for (int i = 0; i < MPW; ++i) {
-      if ((rt0 + i) * 16 >= N) break;
 #pragma unroll
       for (int j = 0; j < NTW; ++j) { S[i][j][0] *= ge; S[i][j][1] *= ge; S[i][j][2] *= ge; S[i][j][3] *= ge; }
 #pragma unroll
-      for (int k = 0; k < Q / 16; ++k) {
-        if (k * 16 >= m) break;
-        uint32_t ba[4], b[4];
+      for (int k = 0; k < Q / 16; ++k) {                         // padding tokens weigh nothing
+        uint32_t ba[4];
         ldsm4t(ba, bt + (k * 16 + (lane & 7) + ((lane >> 4) << 3)) * P + (rt0 + i) * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
         for (int rem = 0; rem < 2; ++rem) {
@@ -334,11 +523,13 @@ __global__ void __launch_bounds__(kST) ssd_scan_kernel(const SsdArgs s) {
           if (NTW >= 2) {
 #pragma unroll
             for (int j = 0; j < NTW / 2; ++j) {
+              uint32_t b[4];
               ldsm4t(b, w + (ct0 + 2 * j) * 8 + (lane >> 4) * 8);
               mma(S[i][(2 * j) % NTW], ba, b[0], b[1]);
               mma(S[i][(2 * j + 1) % NTW], ba, b[2], b[3]);
             }
           } else {
+            uint32_t b[4];
             ldsm4t(b, w + (ct0 & ~1) * 8 + (lane >> 4) * 8);
             mma(S[i][0], ba, ct0 & 1 ? b[2] : b[0], ct0 & 1 ? b[3] : b[1]);
           }
@@ -459,6 +650,21 @@ CB_EXPORT int cb_ssd_chunk(const void* args, int64_t segs, int64_t max_rows, int
   if (a.dk <= 64) return launch_scan<64>(s, (int)segs, st);
   if (a.dk <= 128) return launch_scan<128>(s, (int)segs, st);
   return launch_scan<256>(s, (int)segs, st);
+}
+
+// `segs` segments token by token (seg_row null: one row each); p_f32: projection rows are fp32, f32: the ring is fp32 (else bf16).
+CB_EXPORT int cb_ssd_step(const void* args, int64_t segs, int64_t p_f32, int64_t f32, void* stream) {
+  if (!args || segs < 1 || segs > 65535) return CB_ERR_ARG;
+  SsdArgs s;
+  s.r = *(const LinrecArgs*)args;
+  s.xc = nullptr; s.a = s.dt = nullptr; s.y = (float*)s.r.act;
+  const LinrecArgs& a = s.r;
+  if (!a.proj || !a.gates || !a.act || !a.seg_pos || !a.seg_slot || !a.S || !a.ring || !a.conv_w || !a.A_log || !a.dt_bias || !a.D || a.H < 1 ||
+      a.G < 1 || a.H % a.G || a.dk < 1 || a.dv < 1 || a.taps < 1 || a.taps > a.ring_mask + 1)
+    return CB_ERR_ARG;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (f32) return launch_step<float, float>(s, (int)segs, st);
+  return p_f32 ? launch_step<float, bf16>(s, (int)segs, st) : launch_step<bf16, bf16>(s, (int)segs, st);
 }
 
 // act[r, c] = y[r, c] silu(z[r, c]) / rms(its part of the row) * w[c]; `groups` equal parts of n columns.  y fp32; z_f32 / f32: type

@@ -241,17 +241,16 @@ class RowModel:
         return K.gemm(x, W, out=out)
 
     def project(self, P, h: torch.Tensor, b: RowBatch) -> tuple[torch.Tensor, torch.Tensor]:
-        """``(main, gates)`` of an input projection: one fp32 product for few rows (and in 32-bit mode), else the main
-        columns in the activation type and the gate columns fp32."""
+        """``(main, gates)`` of an input projection, one product: fp32 for few rows (and in 32-bit mode), else the main columns
+        in the activation type and the gate columns fp32."""
         T = b.T
         if self.f32 or T <= 8:
             y = self.buf("proj32", T, P.n, torch.float32)
             self.linear(P.w, h, y)
             return y[:, :P.n_main], y[:, P.n_main:]
         main = self.buf("proj", T, P.n_main)
-        self.linear(P.main, h, main)
         gates = self.buf("gates", T, P.gate.shape[0], torch.float32)
-        self.linear(P.gate, h, gates)
+        X.gemm_mixed(h, P.w, main, gates)
         return main, gates
 
     # ------------------------------------------------------------------ mixer cores

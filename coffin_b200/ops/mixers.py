@@ -53,6 +53,19 @@ def gemm_f32out(A: torch.Tensor, W: torch.Tensor, out: torch.Tensor) -> torch.Te
     return out
 
 
+def gemm_mixed(A: torch.Tensor, W: torch.Tensor, main: torch.Tensor, gates: torch.Tensor) -> None:
+    """One product ``A @ W^T``: its first columns rounded to bf16 in ``main``, the others unrounded in ``gates`` (fp32)."""
+    M, Kd = A.shape
+    N, n_main = W.shape[0], main.shape[1]
+    assert gates.dtype == torch.float32 and gates.shape[1] == N - n_main and main.stride(1) == gates.stride(1) == A.stride(1) == 1
+    ws = tickets = None
+    if M <= 128 and K.SPLITK_GEMM:
+        ws, tickets = K._splitk_scratch(A.device)
+    call("gemm_bf16_mixed", A, A.stride(0), W, W.stride(0), main, main.stride(0), gates, gates.stride(0), n_main, M, N, Kd, ws,
+         ws.numel() * 4 if ws is not None else 0, tickets, tickets.numel() if tickets is not None else 0, K.status_word(A.device))
+    K._count()
+
+
 def gemm_f32(A: torch.Tensor, W: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """True fp32 product of any shape (the 32-bit mode of a model)."""
     M, Kd = A.shape
@@ -165,7 +178,7 @@ class Linrec:
     def __init__(self, kind: int, *, H: int, G: int, dk: int, dv: int, k_col: int, v_col: int, eps: float, state: dict,
                  norm_w: torch.Tensor | None = None, conv_w: torch.Tensor | None = None, A_log=None, dt_bias=None, a2=None,
                  a1_col: int = 0, g2=None, g1_col: int = 0, gate_b=None, cap: float = 0.0, conv_b=None, D=None) -> None:
-        if not linrec_supported(H, dk, dv):
+        if kind != SSD and not linrec_supported(H, dk, dv):
             raise ValueError(f"recurrent head of {dk} x {dv} is outside the kernel's range")
         a = self.a = _LinrecStruct()
         size = _lib.call_nostream("linrec_args_size")
@@ -195,7 +208,10 @@ class Linrec:
     def step(self, proj, gates, og, act, seg_pos, seg_slot, *, segs: int, seg_row=None, dec=None) -> None:
         """Token by token over ``segs`` segments (``seg_row`` None: one row each)."""
         self._fill(proj, gates, og, act, dec, seg_row, seg_pos, seg_slot)
-        call("linrec_step", ctypes.byref(self.a), self.kind, segs, _is_f32(proj), _is_f32(self.state.get("ring", act)))
+        if self.kind == SSD:
+            call("ssd_step", ctypes.byref(self.a), segs, _is_f32(proj), _is_f32(self.state["ring"]))
+        else:
+            call("linrec_step", ctypes.byref(self.a), self.kind, segs, _is_f32(proj), _is_f32(act))
         K._count()
 
     @property
@@ -403,19 +419,24 @@ class LatentAttn:
         call("latent_gather", self.pool, self.pool.stride(0) * self.pool.element_size(), tables, tables.stride(0), base, lens, out, segs, max_pages)
         K._count()
 
+    def _tiles(self, rows: int) -> int:
+        """Groups of 16 heads per CTA of the decode kernel: two share the staged pages unless few rows leave SMs idle."""
+        return 1 if self.H <= 16 or rows <= 2 else 2
+
     def decode_splits(self, rows: int) -> int:
-        groups = -(-self.H // (16 if self.H <= 16 else 32))
+        groups = -(-self.H // (16 * self._tiles(rows)))
         return max(1, min(64, 148 // max(1, groups * rows)))
 
     def absorbed(self, q, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
         """Queries ``q [rows, H * ldk]`` against the pages: key splits for ``merge`` (one split without the tensor-core kernel)."""
         if self.tc:
             call("latent_decode", q, q.stride(0), self.pool, self.pool.stride(0), tables, tables.stride(0), row_seg, positions, part_o, part_ml,
-                 positions.numel(), self.H, self.cp, nsplit, self.scale)
+                 positions.numel(), self.H, self.cp, nsplit, self._tiles(positions.numel()), self.scale)
             K._count()
         else:
             self._plain.rows(q, tables, positions, row_seg, part_o, part_ml, nsplit)
 
     def merge(self, part_o, part_ml, out, positions, nsplit: int) -> None:
         """Weighted averages of the latents, ``out [rows, H * cp]``."""
-        self._plain.finish(part_o, part_ml, None, out, positions, nsplit=nsplit)
+        call("latent_merge", part_o, part_ml, positions, out, out.stride(0), positions.numel(), self.H, self.cp, nsplit, _is_f32(out))
+        K._count()

@@ -133,11 +133,15 @@ def main() -> None:
     ap.add_argument("--prefill", action="store_true", help="trace the prefill pass of the prompt instead of a decode step")
     ap.add_argument("--mma-stage", type=int, default=-1, help="tuning: GEMV weight batches per warp staged in shared memory before the wait")
     ap.add_argument("--mma-kcta", type=int, default=0, help="max CTAs sharing one 16-row GEMV block (1 = off)")
+    ap.add_argument("--mma-carve", type=int, default=1, help="0: leave the L1 / shared memory split of the GEMVs to the driver")
     ap.add_argument("--mma-prefetch", type=int, default=-1, help="GEMV sweep rounds prefetched into L2 before the wait")
     args = ap.parse_args()
     from ..config import first_layers, preset
     from ..engine.llm import LLM
     from ..ops import _lib
+    if not args.mma_carve:
+        from ..ops import _lib
+        _lib.call_nostream("set_mma_gemv_carve", 0)
     if args.mma_prefetch >= 0:
         _lib.call_nostream("set_mma_gemv_prefetch", args.mma_prefetch)
     if args.mma_kcta:

@@ -3,7 +3,9 @@
 //
 // A row keeps its results side by side, x [rows, planes, W] fp32: plane 0 is the embedding output, plane i + 1 the
 // result of layer i.  The running residual of layer i lives in plane i + 1 from the start (its sublayers add to it in
-// place), so a result is never copied.  One kernel per sublayer boundary: add the sublayer's output, at a layer's end take
+// place), so a result is never copied.  The averages are taken in blocks: the last layer of a block reads all planes once and
+// leaves, for every layer of the next block, the sum of what exists by then in the plane where that layer's average will go;
+// inside a block only the partial sum and the few newer planes are read.  One kernel per sublayer boundary: add the sublayer's output, at a layer's end take
 // the weighted sum over the planes into the next one, and normalise for the next projection - layer norm (weight, no
 // bias) or RMS norm.  Sums and norms are fp32.  Few rows: a cluster of CTAs shares a row's columns and exchanges
 // the two sums of the norm through distributed shared memory.
@@ -12,7 +14,7 @@
 
 namespace {
 
-constexpr int kT = 256, kMaxPlanes = 1024;
+constexpr int kT = 256, kWide = 640, kMaxPlanes = 1024, kPrep = 8;
 
 __device__ __forceinline__ float ld_dsmem(const float* p, uint32_t rank) {
   const uint32_t a = sm100::map_to_cta((uint32_t)__cvta_generic_to_shared(p), rank);
@@ -25,7 +27,9 @@ struct DepthArgs {
   float* x; int64_t ldx;               // row stride (planes * W)
   int plane;                           // the running residual
   const void* y; int64_t ldy;          // sublayer output to add (null: none)
-  const float* dwa;                    // weights of planes 0 .. plane (null: not a layer's end)
+  const float* dwa; int64_t ldw;       // weights of planes 0 .. plane, rows of the following layers behind (null: not a layer's end)
+  int first;                           // planes < first are summed up in plane + 1 already (0: nothing is there)
+  int prep;                            // following layers whose sums over planes 0 .. plane go to planes plane + 2 ..
   const float* gain; void* h; int64_t ldh;     // normalised rows (h null: none)
   const int* rows;                     // which row feeds output row i (null: row i)
   int W, cols;                         // columns per CTA
@@ -67,15 +71,18 @@ template <int V> __device__ __forceinline__ void st_f32(float* p, const float* d
   else *p = d[0];
 }
 
-// PG: groups of threads that share a row's planes (few rows); 1: every thread takes whole columns
-template <typename TA, int V, bool GROUPS>
-__global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a, int pg_n) {
-  extern __shared__ float v_s[];       // this CTA's columns of the (averaged) residual; then partial sums of the other groups
-  __shared__ float red[32], w_s[kMaxPlanes];
+// PREP: the sums for the next block of layers as well
+template <typename TA, int V, bool PREP>
+__global__ void __launch_bounds__(PREP ? kT : kWide, PREP ? 3 : 1) depth_step_kernel(const DepthArgs a) {
+  extern __shared__ float v_s[];       // this CTA's columns of the (averaged) residual, then the weights
+  __shared__ float red[32];
   __shared__ float cl[2];
+  float* w_s = v_s + a.cols;           // [1 + prep][plane + 1]
+  const int np1 = a.plane + 1, nT = blockDim.x;
   const int ns = gridDim.x, c0 = blockIdx.x * a.cols, c1 = min(a.W, c0 + a.cols), nc = c1 - c0;
   if (a.dwa)
-    for (int j = threadIdx.x; j <= a.plane; j += kT) w_s[j] = a.dwa[j];
+    for (int k = 0; k <= (PREP ? a.prep : 0); ++k)
+      for (int j = threadIdx.x; j <= a.plane; j += nT) w_s[k * np1 + j] = a.dwa[k * a.ldw + j];
   griddep_launch();
   griddep_wait();
   const int64_t r = a.rows ? a.rows[blockIdx.y] : (int64_t)blockIdx.y;
@@ -100,42 +107,57 @@ __global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a, int p
 #pragma unroll
     for (int v = 0; v < V; ++v) { v_s[i + v] = u[v]; s += a.center ? u[v] : u[v] * u[v]; }
   };
-  if (GROUPS) {
-    const int units = (nc + V - 1) / V, unit = threadIdx.x % units, pg = threadIdx.x / units, i = c0 + unit * V;
-    float acc[V] = {};
-    if (pg < pg_n) {
-      if (pg == 0) {
-        float u[V];
-        own(u, i);
+  for (int i = c0 + threadIdx.x * V; i < c1; i += nT * V) {
+    float u[V];
+    own(u, i);
+    if (a.dwa) {
+      float acc[V];
 #pragma unroll
-        for (int v = 0; v < V; ++v) acc[v] = w_s[a.plane] * u[v];
+      for (int v = 0; v < V; ++v) acc[v] = w_s[a.plane] * u[v];
+      if (PREP) {
+        float pre[kPrep][V];
+#pragma unroll
+        for (int k = 0; k < kPrep; ++k)
+#pragma unroll
+          for (int v = 0; v < V; ++v) pre[k][v] = k < a.prep ? w_s[(1 + k) * np1 + a.plane] * u[v] : 0.f;
+        constexpr int U = 4;
+        for (int j = 0; j < a.plane; j += U) {
+          float f[U][V];
+#pragma unroll
+          for (int q = 0; q < U; ++q) {
+#pragma unroll
+            for (int v = 0; v < V; ++v) f[q][v] = 0.f;
+            if (j + q < a.plane) ld_f32<V>(f[q], xr + (int64_t)(j + q) * a.W + i);
+          }
+#pragma unroll
+          for (int q = 0; q < U; ++q) {
+            const int jj = min(j + q, a.plane);                // past the end: the values are zero
+#pragma unroll
+            for (int v = 0; v < V; ++v) acc[v] = fmaf(w_s[jj], f[q][v], acc[v]);
+#pragma unroll
+            for (int k = 0; k < kPrep; ++k) {
+              const float w = k < a.prep ? w_s[(1 + k) * np1 + jj] : 0.f;
+#pragma unroll
+              for (int v = 0; v < V; ++v) pre[k][v] = fmaf(w, f[q][v], pre[k][v]);
+            }
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < kPrep; ++k)
+          if (k < a.prep && a.store) st_f32<V>(cur + (int64_t)(2 + k) * a.W + i, pre[k]);
+      } else {
+        if (a.first) {
+          ld_f32<V>(u, cur + a.W + i);
+#pragma unroll
+          for (int v = 0; v < V; ++v) acc[v] += u[v];
+        }
+        plane_sum<V>(acc, xr + i, a.W, w_s, a.first, 1, a.plane);
       }
-      plane_sum<V>(acc, xr + i, a.W, w_s, pg, pg_n, a.plane);
-      if (pg) st_f32<V>(v_s + pg * a.cols + unit * V, acc);
-    }
-    __syncthreads();
-    if (pg == 0) {
-      for (int g = 1; g < pg_n; ++g)
 #pragma unroll
-        for (int v = 0; v < V; ++v) acc[v] += v_s[g * a.cols + unit * V + v];
-      if (a.store) st_f32<V>(cur + a.W + i, acc);
-      keep(acc, unit * V);
+      for (int v = 0; v < V; ++v) u[v] = acc[v];
+      if (a.store) st_f32<V>(cur + a.W + i, u);
     }
-  } else {
-    for (int i = c0 + threadIdx.x * V; i < c1; i += kT * V) {
-      float u[V];
-      own(u, i);
-      if (a.dwa) {
-        float acc[V];
-#pragma unroll
-        for (int v = 0; v < V; ++v) acc[v] = w_s[a.plane] * u[v];
-        plane_sum<V>(acc, xr + i, a.W, w_s, 0, 1, a.plane);
-#pragma unroll
-        for (int v = 0; v < V; ++v) u[v] = acc[v];
-        if (a.store) st_f32<V>(cur + a.W + i, u);
-      }
-      keep(u, i - c0);
-    }
+    keep(u, i - c0);
   }
   if (!a.h) return;
   // mean and squared deviations of this CTA's columns, then of the row (RMS norm: plain squares about zero)
@@ -144,30 +166,32 @@ __global__ void __launch_bounds__(kT) depth_step_kernel(const DepthArgs a, int p
   if (a.center) {
     mean = s / (float)nc;
     float d2 = 0.f;
-    for (int i = threadIdx.x; i < nc; i += kT) { const float d = v_s[i] - mean; d2 = fmaf(d, d, d2); }
+    for (int i = threadIdx.x; i < nc; i += nT) { const float d = v_s[i] - mean; d2 = fmaf(d, d, d2); }
     m2 = block_sum(d2, red);
   }
   if (ns > 1) {
     if (threadIdx.x == 0) { cl[0] = mean; cl[1] = m2; }
     sm100::cluster_sync_all();
     float mq[8], vq[8], tot = 0.f;
-    for (int q = 0; q < ns; ++q) {
-      mq[q & 7] = ld_dsmem(&cl[0], q);
-      vq[q & 7] = ld_dsmem(&cl[1], q);
-      tot += mq[q & 7] * (float)(min(a.W, (q + 1) * a.cols) - q * a.cols);
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      mq[q] = q < ns ? ld_dsmem(&cl[0], q) : 0.f;
+      vq[q] = q < ns ? ld_dsmem(&cl[1], q) : 0.f;
+      tot += mq[q] * (float)max(0, min(a.W, (q + 1) * a.cols) - q * a.cols);
     }
     asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");    // this CTA has read what it needs
     mean = tot / (float)a.W;
     m2 = 0.f;
-    for (int q = 0; q < ns; ++q) {
-      const float d = mq[q & 7] - mean;
-      m2 += vq[q & 7] + (a.center ? d * d * (float)(min(a.W, (q + 1) * a.cols) - q * a.cols) : 0.f);
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const float d = mq[q] - mean;
+      m2 += vq[q] + (a.center ? d * d * (float)max(0, min(a.W, (q + 1) * a.cols) - q * a.cols) : 0.f);
     }
     if (!a.center) mean = 0.f;
   }
   const float rstd = 1.f / sqrtf(m2 / (float)a.W + a.eps);
   TA* hr = reinterpret_cast<TA*>(a.h) + (int64_t)blockIdx.y * a.ldh;
-  for (int i = threadIdx.x * V; i < nc; i += kT * V) {
+  for (int i = threadIdx.x * V; i < nc; i += nT * V) {
     if (V == 4) {
       const float4 g = *reinterpret_cast<const float4*>(a.gain + c0 + i);
       act_store4(hr + c0 + i, make_float4((v_s[i] - mean) * rstd * g.x, (v_s[i + 1 % V] - mean) * rstd * g.y,
@@ -188,27 +212,38 @@ __global__ void __launch_bounds__(kT) depth_embed_kernel(const TA* __restrict__ 
   const int64_t r = blockIdx.x;
   int64_t tok = tokens[r];
   tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
-  for (int i = threadIdx.x; i < W; i += kT) {
-    const float v = act_load(embed + tok * W + i) * scale;
-    x[r * ldx + i] = v;
-    x[r * ldx + W + i] = v;
+  const TA* e = embed + tok * W;
+  float* xr = x + r * ldx;
+  if (W % 4 == 0 && ldx % 4 == 0) {
+    for (int i = threadIdx.x * 4; i < W; i += kT * 4) {
+      float4 v = act_load4(e + i);
+      v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
+      *reinterpret_cast<float4*>(xr + i) = v;
+      *reinterpret_cast<float4*>(xr + W + i) = v;
+    }
+    return;
   }
+  for (int i = threadIdx.x; i < W; i += kT) xr[i] = xr[W + i] = act_load(e + i) * scale;
 }
 
 template <typename TA>
 int launch_depth(DepthArgs a, int64_t n, cudaStream_t st) {
   const bool v4 = a.W % 4 == 0 && a.ldx % 4 == 0 && a.ldh % 4 == 0 && a.ldy % 4 == 0;
+  // a row with many planes to read is shared by a cluster of CTAs while SMs are idle; otherwise few rows get wide blocks
   int ns = 1;
-  while (ns < 8 && n * ns * 2 <= 148 && a.W / (ns * 2) >= 256) ns <<= 1;
+  if (a.dwa && a.plane - a.first > 12)
+    while (ns < 8 && n * ns * 2 <= 148 && a.W / (ns * 2) >= 256) ns <<= 1;
   a.cols = ((a.W + ns - 1) / ns + 3) & ~3;
   ns = (a.W + a.cols - 1) / a.cols;
   const int units = v4 ? (a.cols + 3) / 4 : a.cols;
-  int pg = a.dwa && a.plane > 8 && n <= 64 ? kT / units : 1;     // few rows: groups of threads share the planes
-  if (pg > 8) pg = 8;
-  auto kern = pg > 1 ? (v4 ? depth_step_kernel<TA, 4, true> : depth_step_kernel<TA, 1, true>)
+  int threads = kT;
+  if (!a.prep && n <= 148) {
+    threads = (units + 31) & ~31;
+    threads = threads < kT ? kT : (threads > kWide ? kWide : threads);
+  }
+  auto kern = a.prep ? (v4 ? depth_step_kernel<TA, 4, true> : depth_step_kernel<TA, 1, true>)
                      : (v4 ? depth_step_kernel<TA, 4, false> : depth_step_kernel<TA, 1, false>);
-  if (pg < 1) pg = 1;
-  const size_t smem = (size_t)a.cols * pg * sizeof(float);
+  const size_t smem = ((size_t)a.cols + (a.dwa ? (size_t)(1 + a.prep) * (a.plane + 1) : 0)) * sizeof(float);
   if (smem > 200 * 1024) return CB_ERR_SHAPE;
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -216,7 +251,7 @@ int launch_depth(DepthArgs a, int64_t n, cudaStream_t st) {
   }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3((unsigned)ns, (unsigned)n);
-  cfg.blockDim = dim3(kT);
+  cfg.blockDim = dim3((unsigned)threads);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
   cudaLaunchAttribute attr[2];
@@ -234,21 +269,25 @@ int launch_depth(DepthArgs a, int64_t n, cudaStream_t st) {
   cfg.attrs = attr;
   cfg.numAttrs = na;
   if (g_cb_trace_names) cb_trace_name((const void*)kern);
-  return (int)cudaLaunchKernelEx(&cfg, kern, a, pg);
+  return (int)cudaLaunchKernelEx(&cfg, kern, a);
 }
 
 }  // namespace
 
 // One sublayer boundary over `n` rows of x [*, ldx]: plane `plane` += y (y null: nothing), with dwa the weighted sum of
-// planes 0 .. plane goes to plane + 1, and h = norm(the result) * gain (center: layer norm, else RMS norm).  `rows`
+// planes 0 .. plane goes to plane + 1 (first > 0: planes < first are summed up there already), the sums of the next `prep`
+// layers over these planes to the planes behind (their weights in the rows of dwa, ldw apart), and h = norm(the result) * gain
+// (center: layer norm, else RMS norm).  `rows`
 // (int32 [n]): which row feeds output row i; `store` 0: x is left as it is.  f32: y and h are fp32 instead of bf16.
-CB_EXPORT int cb_depth_step(void* x, int64_t ldx, int64_t plane, const void* y, int64_t ldy, const void* dwa, const void* gain,
-                            void* h, int64_t ldh, const void* rows, int64_t n, int64_t W, float eps, int64_t center, int64_t store,
+CB_EXPORT int cb_depth_step(void* x, int64_t ldx, int64_t plane, const void* y, int64_t ldy, const void* dwa, int64_t ldw,
+                            int64_t first, int64_t prep, const void* gain, void* h, int64_t ldh, const void* rows, int64_t n, int64_t W, float eps, int64_t center, int64_t store,
                             int64_t f32, void* stream) {
   if (!x || n < 1 || n > 65535 || W < 1 || plane < 0 || plane >= kMaxPlanes || (h && !gain) || (rows && store)) return CB_ERR_ARG;
-  if (ldx < (plane + (dwa && store ? 2 : 1)) * W) return CB_ERR_ARG;
+  if (prep < 0 || prep > kPrep || first < 0 || first > plane || ((prep || first) && !dwa) || (prep && first)) return CB_ERR_ARG;
+  if (ldx < (plane + (dwa && store ? 2 + prep : (first ? 2 : 1))) * W) return CB_ERR_ARG;
   DepthArgs a;
-  a.x = (float*)x; a.ldx = ldx; a.plane = (int)plane; a.y = y; a.ldy = ldy; a.dwa = (const float*)dwa; a.gain = (const float*)gain;
+  a.x = (float*)x; a.ldx = ldx; a.plane = (int)plane; a.y = y; a.ldy = ldy; a.dwa = (const float*)dwa; a.ldw = ldw;
+  a.first = (int)first; a.prep = (int)prep; a.gain = (const float*)gain;
   a.h = h; a.ldh = ldh; a.rows = (const int*)rows; a.W = (int)W; a.cols = 0; a.eps = eps; a.center = (int)center; a.store = (int)store;
   return f32 ? launch_depth<float>(a, n, (cudaStream_t)stream) : launch_depth<bf16>(a, n, (cudaStream_t)stream);
 }

@@ -316,88 +316,102 @@ struct Plan {
   static constexpr int SH = MTN < 8 ? 8 / MTN : 1;               // warps that share a row tile
   static constexpr int NTW = 4 / SH;                             // column tiles (8) per warp
   static constexpr int TILE = 2 * Q * P + Q * VP;                // one stage: C, B, x (bf16)
-  static constexpr size_t bytes = sizeof(bf16) * (2 * TILE + 2 * Q * VP + 2 * NP * VP) + sizeof(float) * 4 * Q;
+  static constexpr bool XOWN = 16 * P * 2 < 2048;                // sixteen C rows do not hold a pair's exchange
+  static constexpr size_t bytes = sizeof(bf16) * (2 * TILE + 2 * Q * VP + 2 * NP * VP) + sizeof(float) * 4 * Q + (XOWN ? 4 * 2048 : 0);
 };
 
-// read-outs of token rows 16 RG .. 16 RG + 15, columns 16 half .. + 15: scores against tokens 0 .. 16 RG + 15 and the
-// read-out of the old state share the C fragments
-template <int NP, int RG>
-__device__ __forceinline__ void read_out(const bf16* ct, const bf16* bt, const bf16* xt, const bf16* st, const float* av, const float* dtv,
-                                         int half, int lane, int m, int nv, float Dh, float* y, int64_t ldy) {
-  constexpr int P = NP + 8;
+// Read-outs of token rows 16 RG .. 16 RG + 15 by two warps: each takes half of the earlier tokens (scores, decays, values)
+// and half of the old state's channels over all columns; the partial sums meet in `xch` (the pair's own rows of the C tile,
+// which nobody else reads, where those are large enough), and each warp finishes 16 columns.
+template <int NP, int RG, int HALF>
+__device__ __forceinline__ void read_out(const bf16* ct, float4* xch, const bf16* bt, const bf16* xt, const bf16* st, const float* av, const float* dtv,
+                                         int lane, int m, int nv, float Dh, float* y, int64_t ldy) {
+  constexpr int P = NP + 8, J0 = HALF ? (RG + 2) / 2 : 0, J1 = HALF ? RG + 1 : (RG + 2) / 2, NJ = J1 - J0, KH = NP / 32;
   const int g4 = lane >> 2, t4 = lane & 3;
-  float G[2 * RG + 2][4], Y[2][4], Y2[2][4];
+  float G[NJ > 0 ? 2 * NJ : 1][4], Y[4][4];
 #pragma unroll
-  for (int i = 0; i < 2 * RG + 2; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = 0.f;
+  for (int i = 0; i < 2 * NJ; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = 0.f;
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
-    Y2[i][0] = Y2[i][1] = Y2[i][2] = Y2[i][3] = 0.f;
-  }
+  for (int i = 0; i < 4; ++i) Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
   const bf16* cr = ct + (RG * 16 + (lane & 15)) * P + (lane >> 4) * 8;
-  const bf16* sr = st + (lane & 15) * VP + half * 16 + (lane >> 4) * 8;
-  const bf16* br = bt + ((lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
+  const bf16* sr = st + (lane & 15) * VP + (lane >> 4) * 8;
+  const bf16* br = bt + (J0 * 16 + (lane & 7) + ((lane >> 4) << 3)) * P + ((lane >> 3) & 1) * 8;
 #pragma unroll
   for (int k = 0; k < NP / 16; ++k) {
-    uint32_t ca[4], sh[4], sl[4], b[RG + 1][4];
+    const bool mine = k / KH == HALF;                            // compile time
+    if (NJ == 0 && !mine) continue;
+    uint32_t ca[4];
     ldsm4(ca, cr + k * 16);
-    ldsm4t(sh, sr + k * 16 * VP);
-    ldsm4t(sl, sr + (NP + k * 16) * VP);
+    if (mine) {
+      uint32_t s0[4], s1[4];
+      ldsm4t(s0, sr + k * 16 * VP);
+      ldsm4t(s1, sr + k * 16 * VP + 16);
+      mma(Y[0], ca, s0[0], s0[1]); mma(Y[1], ca, s0[2], s0[3]);
+      mma(Y[2], ca, s1[0], s1[1]); mma(Y[3], ca, s1[2], s1[3]);
+      ldsm4t(s0, sr + (NP + k * 16) * VP);
+      ldsm4t(s1, sr + (NP + k * 16) * VP + 16);
+      mma(Y[0], ca, s0[0], s0[1]); mma(Y[1], ca, s0[2], s0[3]);
+      mma(Y[2], ca, s1[0], s1[1]); mma(Y[3], ca, s1[2], s1[3]);
+    }
 #pragma unroll
-    for (int j = 0; j <= RG; ++j) ldsm4(b[j], br + j * 16 * P + k * 16);
-    mma(Y[0], ca, sh[0], sh[1]);
-    mma(Y[1], ca, sh[2], sh[3]);
-    mma(Y2[0], ca, sl[0], sl[1]);
-    mma(Y2[1], ca, sl[2], sl[3]);
-#pragma unroll
-    for (int j = 0; j <= RG; ++j) {
-      mma(G[2 * j], ca, b[j][0], b[j][1]);
-      mma(G[2 * j + 1], ca, b[j][2], b[j][3]);
+    for (int j = 0; j < NJ; ++j) {
+      uint32_t b[4];
+      ldsm4(b, br + j * 16 * P + k * 16);
+      mma(G[2 * j], ca, b[0], b[1]);
+      mma(G[2 * j + 1], ca, b[2], b[3]);
     }
   }
   const int tl = RG * 16 + g4, th = tl + 8;
   const float al = av[tl], ah = av[th], el = ex2(al), eh = ex2(ah);
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    Y[i][0] = (Y[i][0] + Y2[i][0]) * el; Y[i][1] = (Y[i][1] + Y2[i][1]) * el;
-    Y[i][2] = (Y[i][2] + Y2[i][2]) * eh; Y[i][3] = (Y[i][3] + Y2[i][3]) * eh;
-    Y2[i][0] = Y2[i][1] = Y2[i][2] = Y2[i][3] = 0.f;
-  }
+  for (int i = 0; i < 4; ++i) { Y[i][0] *= el; Y[i][1] *= el; Y[i][2] *= eh; Y[i][3] *= eh; }
 #pragma unroll
-  for (int j = 0; j <= RG; ++j) {
-    uint32_t mh[4], ml[4], b[4];
-    ldsm4t(b, xt + (j * 16 + (lane & 15)) * VP + half * 16 + (lane >> 4) * 8);
+  for (int j = 0; j < NJ; ++j) {
+    uint32_t mh[4], ml[4], b0[4], b1[4];
+    ldsm4t(b0, xt + ((J0 + j) * 16 + (lane & 15)) * VP + (lane >> 4) * 8);
+    ldsm4t(b1, xt + ((J0 + j) * 16 + (lane & 15)) * VP + 16 + (lane >> 4) * 8);
 #pragma unroll
     for (int p = 0; p < 2; ++p) {                                // tokens u, u + 1 of rows lo, then hi
-      const int u = j * 16 + p * 8 + t4 * 2;
+      const int u = (J0 + j) * 16 + p * 8 + t4 * 2;
       const float2 au = *reinterpret_cast<const float2*>(av + u), du = *reinterpret_cast<const float2*>(dtv + u);
       const float* gg = G[2 * j + p];
-      float x = gg[0] * (du.x * ex2(fminf(al - au.x, 0.f))), y = gg[1] * (du.y * ex2(fminf(al - au.y, 0.f)));
-      float z = gg[2] * (du.x * ex2(fminf(ah - au.x, 0.f))), w = gg[3] * (du.y * ex2(fminf(ah - au.y, 0.f)));
-      if (j == RG) {
+      float x = gg[0] * (du.x * ex2(fminf(al - au.x, 0.f))), z = gg[1] * (du.y * ex2(fminf(al - au.y, 0.f)));
+      float v = gg[2] * (du.x * ex2(fminf(ah - au.x, 0.f))), w = gg[3] * (du.y * ex2(fminf(ah - au.y, 0.f)));
+      if (J0 + j == RG) {
         if (u > tl) x = 0.f;
-        if (u + 1 > tl) y = 0.f;
-        if (u > th) z = 0.f;
+        if (u + 1 > tl) z = 0.f;
+        if (u > th) v = 0.f;
         if (u + 1 > th) w = 0.f;
       }
-      mh[2 * p] = split_head(x, y); ml[2 * p] = pack_bf162(x, y);          // a0 / a2: row lo; a1 / a3: row hi
-      mh[2 * p + 1] = split_head(z, w); ml[2 * p + 1] = pack_bf162(z, w);
+      mh[2 * p] = split_head(x, z); ml[2 * p] = pack_bf162(x, z);          // a0 / a2: row lo; a1 / a3: row hi
+      mh[2 * p + 1] = split_head(v, w); ml[2 * p + 1] = pack_bf162(v, w);
     }
-    mma(Y[0], mh, b[0], b[1]);
-    mma(Y[1], mh, b[2], b[3]);
-    mma(Y2[0], ml, b[0], b[1]);
-    mma(Y2[1], ml, b[2], b[3]);
+    mma(Y[0], mh, b0[0], b0[1]); mma(Y[1], mh, b0[2], b0[3]);
+    mma(Y[2], mh, b1[0], b1[1]); mma(Y[3], mh, b1[2], b1[3]);
+    mma(Y[0], ml, b0[0], b0[1]); mma(Y[1], ml, b0[2], b0[3]);
+    mma(Y[2], ml, b1[0], b1[1]); mma(Y[3], ml, b1[2], b1[3]);
   }
+  asm volatile("bar.sync %0, 64;" ::"r"(1 + RG) : "memory");     // both warps are done with the C rows
 #pragma unroll
-  for (int i = 0; i < 2; ++i)
+  for (int i = 0; i < 2; ++i) {                                  // [half that wrote][2][lane]
+    const float* o = Y[(HALF ? 0 : 2) + i];
+    xch[(HALF * 2 + i) * 32 + lane] = make_float4(o[0], o[1], o[2], o[3]);
+  }
+  asm volatile("bar.sync %0, 64;" ::"r"(1 + RG) : "memory");
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const float4 o = xch[((1 - HALF) * 2 + i) * 32 + lane];
+    const float* q = Y[HALF * 2 + i];
+    const float r[4] = {q[0] + o.x, q[1] + o.y, q[2] + o.z, q[3] + o.w};
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const int t = e ? th : tl, c = half * 16 + i * 8 + t4 * 2;
+      const int t = e ? th : tl, c = HALF * 16 + i * 8 + t4 * 2;
       if (t < m && c < nv) {
         const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(xt + t * VP + c));
-        *reinterpret_cast<float2*>(y + t * ldy + c) = make_float2(fmaf(Dh, x.x, Y[i][2 * e] + Y2[i][2 * e]), fmaf(Dh, x.y, Y[i][2 * e + 1] + Y2[i][2 * e + 1]));
+        *reinterpret_cast<float2*>(y + t * ldy + c) = make_float2(fmaf(Dh, x.x, r[2 * e]), fmaf(Dh, x.y, r[2 * e + 1]));
       }
     }
+  }
 }
 
 template <int NP>
@@ -472,12 +486,12 @@ __global__ void __launch_bounds__(kST, NP <= 128 ? 2 : 1) ssd_scan_kernel(const 
         S[m][j][e] = k < N && c < nv ? Sg[(int64_t)k * a.dv + c] : 0.f;
       }
   state_out();
-  const int rg = warp & 3, half = warp >> 2;                     // token tile and column half of this warp's read-outs
+  const int half = warp >> 2, rg = half ? 3 - (warp & 3) : warp & 3;      // token tile; long and short ones share a scheduler
   for (int ch = 0; ch < chunks; ++ch) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                             // tiles, decays and state of this chunk are in place
     if (ch + 1 < chunks) load(ch + 1);
-    const bf16* ct = tiles + (ch & 1) * L::TILE;
+    bf16* ct = tiles + (ch & 1) * L::TILE;
     const bf16* bt = ct + Q * P;
     const bf16* xt = bt + Q * P;
     const float* av = sa + (ch & 1) * Q;
@@ -501,11 +515,15 @@ __global__ void __launch_bounds__(kST, NP <= 128 ? 2 : 1) ssd_scan_kernel(const 
       *reinterpret_cast<uint4*>(xw + Q * VP + t * VP + c) = make_uint4(rm[0], rm[1], rm[2], rm[3]);
     }
     if (rg * 16 < m) {
+      float4* xch = L::XOWN ? reinterpret_cast<float4*>(sdt + 2 * Q) + rg * 128 : reinterpret_cast<float4*>(ct + rg * 16 * P);
       float* y = s.y + (int64_t)(row0 + ch * Q) * a.lda + (int64_t)h * a.dv + v0;
-      if (rg == 0) read_out<NP, 0>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
-      else if (rg == 1) read_out<NP, 1>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
-      else if (rg == 2) read_out<NP, 2>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
-      else read_out<NP, 3>(ct, bt, xt, st, av, dtv, half, lane, m, nv, Dh, y, a.lda);
+#define CB_READ(R)                                                                                   \
+  if (rg == R) {                                                                                     \
+    if (half) read_out<NP, R, 1>(ct, xch, bt, xt, st, av, dtv, lane, m, nv, Dh, y, a.lda);                \
+    else read_out<NP, R, 0>(ct, xch, bt, xt, st, av, dtv, lane, m, nv, Dh, y, a.lda);                     \
+  }
+      CB_READ(0) CB_READ(1) CB_READ(2) CB_READ(3)
+#undef CB_READ
     }
     __syncthreads();                                             // weighted values in place, the old state has been read
     const float ge = ex2(aq);

@@ -30,7 +30,8 @@ class _Layer:
     kind: str
     mixer: object
     gain1: torch.Tensor
-    dwa: torch.Tensor                           # weights of the embedding output and of the results so far
+    dwa: torch.Tensor                           # weights of the embedding output and of the results, rows of later layers behind
+    plan: dict                                  # which planes the average still has to read, what it prepares
     gain2: torch.Tensor | None = None
     w_up: torch.Tensor | None = None
     w_down: torch.Tensor | None = None
@@ -53,6 +54,8 @@ class SukisunModel(RowModel):
             return sd.pop(name) if free_source else sd[name]
 
         f32 = lambda name: take(name).to(dev, torch.float32).contiguous()
+        n = len(c.layers)
+        dwa = torch.zeros(n, n + 1, dtype=torch.float32, device=dev)       # row i: planes 0 .. i + 1
         for i, spec in enumerate(c.layers):
             p = f"l{i}."
             mw = {k[len(p) + 4:]: take(k) for k in [k for k in sd if k.startswith(p + "mix.")]}
@@ -63,7 +66,8 @@ class SukisunModel(RowModel):
                     src._lent = mixer._lent = True
             else:
                 mixer = Mamba2(spec.mixer, mw, W, self.eps, self.num_slots, dtype, dev)
-            L = _Layer(spec.kind, mixer, f32(p + "norm1"), f32(p + "dwa"))
+            dwa[i, :i + 2] = take(p + "dwa").to(dev)
+            L = _Layer(spec.kind, mixer, f32(p + "norm1"), dwa[i:], X.depth_plan(i, n))
             if spec.ff is not None:
                 I, W8 = pad8(spec.ff), pad8(W)
                 L.gain2 = f32(p + "norm2")
@@ -95,7 +99,7 @@ class SukisunModel(RowModel):
                 X.depth_step(x, plane, h, gain=L.gain2, eps=self.eps, **pend)
                 inter = X.linear_xielu(L.w_up, h, self.buf("inter", T, L.w_up.shape[0]), *L.act)
                 pend = dict(y=self.linear(L.w_down, inter, self.buf("y", T, L.w_down.shape[0])))
-            pend["weights"] = L.dwa
+            pend.update(weights=L.dwa, **L.plan)
             if self.layer_hook is not None:
                 X.depth_step(x, plane, None, **pend)
                 pend, plane = {}, plane + 1
@@ -104,4 +108,4 @@ class SukisunModel(RowModel):
 
     def _out_rows(self, state, rows, n, h) -> None:
         x, plane, pend = state
-        X.depth_step(x, plane, h, gain=self.final_gain, rows=rows, store=False, eps=self.eps, **pend)
+        X.depth_step(x, plane, h, gain=self.final_gain, rows=rows, store=False, eps=self.eps, **pend)     # nothing left to prepare

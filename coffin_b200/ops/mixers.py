@@ -137,18 +137,31 @@ def depth_embed(embed: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, scal
     return x
 
 
+DEPTH_BLOCK = 8
+
+
+def depth_plan(layer: int, layers: int) -> dict[str, int]:
+    """``first`` / ``prep`` of a layer's end when the averages are taken in blocks of ``DEPTH_BLOCK`` layers."""
+    start = layer // DEPTH_BLOCK * DEPTH_BLOCK               # the planes 0 .. start were summed up before the block
+    prep = min(DEPTH_BLOCK, layers - 1 - layer) if (layer + 1) % DEPTH_BLOCK == 0 else 0
+    return {"first": start + 1 if start and not prep else 0, "prep": prep}
+
+
 def depth_step(x: torch.Tensor, plane: int, h: torch.Tensor | None, *, gain: torch.Tensor | None = None, y: torch.Tensor | None = None,
-               weights: torch.Tensor | None = None, rows: torch.Tensor | None = None, store: bool = True, eps: float = 1e-5,
-               center: bool = True) -> torch.Tensor | None:
+               weights: torch.Tensor | None = None, first: int = 0, prep: int = 0, rows: torch.Tensor | None = None, store: bool = True,
+               eps: float = 1e-5, center: bool = True) -> torch.Tensor | None:
     """Boundary between two sublayers: plane ``plane`` of ``x [T, planes, W]`` += ``y``; with ``weights`` (a layer's end) the
-    weighted sum of planes ``0 .. plane`` becomes plane ``plane + 1``; then ``h = norm(result) * gain``, layer norm
+    weighted sum of planes ``0 .. plane`` becomes plane ``plane + 1``.  Row 0 of ``weights`` is this layer's; ``prep``: the sums of
+    that many following layers (the next rows) over the same planes are left where their averages will go; ``first``: planes
+    below it have been summed up that way already (``depth_plan``).  Then ``h = norm(result) * gain``, layer norm
     (``center``) or RMS norm.  ``rows`` picks the rows behind the rows of ``h`` (with ``store=False``)."""
     T, planes, W = x.shape
     n = rows.numel() if rows is not None else (h.shape[0] if h is not None else T)
     t = h if h is not None else y
-    assert weights is None or (weights.numel() == plane + 1 and (not store or plane + 2 <= planes))
-    call("depth_step", x, x.stride(0), plane, y, y.stride(0) if y is not None else 0, weights, gain, h, h.stride(0) if h is not None else 0,
-         rows, n, W, float(eps), int(center), int(store), _is_f32(t) if t is not None else 0)
+    assert weights is None or (weights.stride(-1) == 1 and weights.shape[-1] > plane and (not store or plane + 2 + prep <= planes))
+    assert not prep or (weights.dim() == 2 and weights.shape[0] > prep)
+    call("depth_step", x, x.stride(0), plane, y, y.stride(0) if y is not None else 0, weights, weights.stride(0) if weights is not None else 0, first, prep,
+         gain, h, h.stride(0) if h is not None else 0, rows, n, W, float(eps), int(center), int(store), _is_f32(t) if t is not None else 0)
     K._count()
     return h
 

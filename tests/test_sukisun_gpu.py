@@ -71,6 +71,28 @@ def test_depth_step(T, W, planes, dtype):
     assert rel(x[:, p], new[:, p] + y.double()) < 1e-6
 
 
+@pytest.mark.parametrize("T,W", [(1, 64), (1, 2048), (3, 50), (100, 256)])
+def test_depth_averages_in_blocks(T, W):
+    """Layer by layer through 21 layers: partial sums prepared at the block ends and completed inside the blocks."""
+    from coffin_b200.ops import mixers as X
+    n = 21
+    dwa, gain = randn(1, n, n + 1).cuda(), torch.ones(W, device="cuda")
+    x, ref = torch.full((T, n + 2, W), float("nan"), device="cuda"), []
+    e = randn(2, T, W).cuda()
+    x[:, 0], x[:, 1] = e, e
+    h = torch.zeros(T, W, device="cuda")
+    ref, cur = [e.double()], e.double()
+    for i in range(n):
+        y = randn(10 + i, T, W).cuda()
+        plan = X.depth_plan(i, n)
+        assert plan["first"] in (0, i // X.DEPTH_BLOCK * X.DEPTH_BLOCK + 1) and (plan["prep"] > 0) == (i in (7, 15))
+        X.depth_step(x, i + 1, h, gain=gain, y=y, weights=dwa[i:], **plan)
+        ref.append(cur + y.double())
+        cur = P.depth_average(dwa[i, :i + 2].double(), ref)
+        assert rel(x[:, i + 2], cur) < 3e-6 and rel(x[:, i + 1], ref[-1]) < 3e-6 and rel(h, P.layer_norm(cur, gain.double(), 1e-5)) < 3e-6, i
+        cur = x[:, i + 2].double()
+
+
 def test_depth_embed_scales_and_starts_the_first_layer():
     from coffin_b200.ops import mixers as X
     E = randn(5, 30, 44).bfloat16().cuda()
@@ -397,6 +419,8 @@ CONFIGS = {
     "sizes_differ": S.config([S.mamba(2, 64, 128, 1, 4, 2), S.latent(8, 64, 64, 64, 256, 96, 0.08), S.latent(3, 16, 8, 24, 48, 40), S.mamba(6, 8, 24, 3, 3, 2),
                               S.latent(18, 32, 64, 32, 256, 64, 0.1, kv_from=1), S.latent(2, 40, 8, 16, 48, 40, kv_from=2)], width=128, ff=200, vocab=128,
                              scale=11.0),
+    "deep": S.config([S.latent(2, 8, 4, 8, 24, 16)] + [S.mamba(2, 8, 8, 1, 2, 1), S.latent(2, 8, 4, 8, 24, 16, kv_from=0)] * 9, width=32, vocab=60, ff=24,
+                     no_mlp=range(1, 18, 2)),
 }
 
 

@@ -73,7 +73,7 @@ template <int V> __device__ __forceinline__ void st_f32(float* p, const float* d
 
 // PREP: the sums for the next block of layers as well
 template <typename TA, int V, bool PREP>
-__global__ void __launch_bounds__(PREP ? kT : kWide, PREP ? 3 : 1) depth_step_kernel(const DepthArgs a) {
+__global__ void __launch_bounds__(PREP ? kT : kWide, PREP ? 3 : 2) depth_step_kernel(const DepthArgs a) {
   extern __shared__ float v_s[];       // this CTA's columns of the (averaged) residual, then the weights
   __shared__ float red[32];
   __shared__ float cl[2];

@@ -288,8 +288,9 @@ class AttnMaps:
     """Attention layer constants plus its pages ``kpool [slots, G * maps, dim]``, ``vpool [slots, G, vdim]``."""
 
     def __init__(self, *, H: int, G: int, maps: int, dim: int, vdim: int, k_col: int, v_col: int, scale: float, cap: float | None,
-                 temp: tuple[float, int] | None, kpool: torch.Tensor, vpool: torch.Tensor) -> None:
-        if vdim > MAX_VDIM or maps not in (1, 2):
+                 temp: tuple[float, int] | None, kpool: torch.Tensor, vpool: torch.Tensor, finish: bool = True) -> None:
+        """``finish``: the heads will be finished by ``finish``, which bounds the value size."""
+        if (finish and vdim > MAX_VDIM) or maps not in (1, 2):
             raise ValueError(f"attention with {maps} maps and values of {vdim} is outside the kernels' range")
         a = self.a = _AttnStruct()
         size = _lib.call_nostream("attn_maps_args_size")
@@ -416,7 +417,7 @@ class LatentAttn:
         a.norm_q, a.norm_c, a.pool, a.ldk = _ptr(norm_q), _ptr(norm_c), _ptr(pool), pool.stride(0)
         # the plain kernel and the merge of key splits see one key / value head whose values are the head of the key row
         self._plain = AttnMaps(H=H, G=1, maps=1, dim=self.ldk, vdim=cp, k_col=0, v_col=0, scale=scale, cap=None, temp=None, kpool=pool,
-                               vpool=pool)
+                               vpool=pool, finish=False)
         self.tc = pool.dtype == torch.bfloat16 and bool(_lib.call_nostream("latent_decode_ok", self.ldk, cp))
 
     def rows(self, proj, cq, tables, positions, row_seg, cs) -> None:

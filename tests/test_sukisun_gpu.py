@@ -171,7 +171,7 @@ def test_per_head_products(T, H, N, Kd):
             assert (y.view(T, H, N + 3)[..., N:] == 5).all()
 
 
-@pytest.mark.parametrize("H,cp,rp,nsplit", [(4, 16, 16, 1), (6, 96, 32, 3), (16, 128, 16, 2), (17, 80, 16, 5), (32, 512, 64, 7), (40, 256, 32, 2), (5, 272, 16, 64)])
+@pytest.mark.parametrize("H,cp,rp,nsplit", [(4, 16, 16, 1), (7, 112, 32, 3), (16, 128, 16, 2), (17, 80, 16, 5), (32, 512, 64, 7), (40, 256, 32, 2), (5, 272, 16, 64)])
 def test_absorbed_decode_kernel(H, cp, rp, nsplit):
     """Rows of unequal length against scattered pages; one key of every row stands out for one head."""
     from coffin_b200.ops import mixers as X
@@ -216,13 +216,14 @@ def test_gated_norm(groups, n):
 
 # ------------------------------------------------------------------ mixers alone
 MIX = {
-    "mamba": S.mamba(), "mamba_one_group": S.mamba(4, 48, 48, 1, 3, 1), "mamba_groups": S.mamba(6, 16, 16, 6, 2, 6), "mamba_one_tap": S.mamba(2, 8, 24, 1, 1, 2),
+    "mamba": S.mamba(), "mamba_one_group": S.mamba(5, 40, 56, 1, 3, 1), "mamba_groups": S.mamba(6, 16, 16, 6, 2, 6), "mamba_one_tap": S.mamba(2, 8, 24, 1, 1, 2),
     "mamba_64": S.mamba(3, 64, 64, 1, 4, 3), "mamba_128": S.mamba(2, 64, 128, 1, 4, 1), "mamba_256": S.mamba(2, 40, 256, 2, 4, 1),
     "mamba_odd": S.mamba(3, 7, 10, 1, 5, 3), "mamba_wide": S.mamba(1, 136, 72, 1, 6, 1),
     "latent": S.latent(), "latent_one_head": S.latent(1, 8, 4, 8, 16, 8), "latent_many": S.latent(20, 16, 8, 16, 48, 24), "latent_32": S.latent(32, 32, 32, 32, 64, 64),
     "latent_wide": S.latent(3, 128, 64, 128, 512, 192, 192 ** -0.5), "latent_odd": S.latent(3, 11, 6, 13, 45, 19), "latent_big_values": S.latent(2, 48, 16, 200, 136, 40),
     "latent_part": S.latent(4, 16, 24, 24, 64, 32, rot_dims=10), "latent_far_base": S.latent(4, 8, 32, 16, 40, 32, base=5e5), "latent_256": S.latent(2, 192, 64, 256, 256, 64),
-    "latent_long_head": S.latent(2, 288, 16, 48, 64, 40, 0.05),
+    "latent_long_head": S.latent(2, 288, 16, 48, 64, 40, 0.05), "latent_large_rank": S.latent(2, 16, 8, 24, 600, 40),
+    "mamba_large_state": S.mamba(2, 16, 320, 1, 4, 1), "mamba_long_conv": S.mamba(2, 16, 16, 2, 20, 1),
 }
 
 

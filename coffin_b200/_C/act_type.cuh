@@ -44,5 +44,8 @@ __device__ __forceinline__ float xielu_s(float z, float a, float b) {
 __device__ __forceinline__ float xielu_x(float z, float a, float b) {
   return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (expm1f(fminf(z, 0.f)) - z));
 }
+__device__ __forceinline__ float relu2(float z) { z = fmaxf(z, 0.f); return z * z; }
+// epilogue activations of the products: 1 xIELU with its coefficients, 2 squared relu
+__device__ __forceinline__ float epi_act(int act, float z, float a, float b) { return act == 2 ? relu2(z) : xielu_s(z, a, b); }
 __device__ __forceinline__ float sigmoid_s(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 __device__ __forceinline__ float silu_s(float x) { return x * sigmoid_s(x); }

@@ -5,19 +5,76 @@
 
 namespace {
 
+// Keys (turned) and values (mixed) of a row into its page; with `turn_q` its queries are turned in place.
 template <typename TP, typename TA>
-__global__ void __launch_bounds__(256) maps_append_kernel(const AttnMapsArgs a) {
+__global__ void __launch_bounds__(256) maps_append_kernel(const AttnMapsArgs a, int turn_q) {
   griddep_launch();
   griddep_wait();
   const int row = blockIdx.x, seg = a.row_seg ? a.row_seg[row] : row, pos = a.positions[row];
   if (pos < 0) return;
   const int64_t slot = (int64_t)a.tables[(int64_t)seg * a.ldbt + pos / kPage] * kPage + pos % kPage;
-  const TP* p = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
+  TP* p = reinterpret_cast<TP*>(const_cast<void*>(a.proj)) + (int64_t)row * a.ldp;
   const int nk = a.G * a.maps * a.dim, nv = a.G * a.vdim;
   TA* kp = reinterpret_cast<TA*>(a.kpool) + slot * pool_ldk(a);
   TA* vp = reinterpret_cast<TA*>(a.vpool) + slot * pool_ldv(a);
-  for (int c = threadIdx.x; c < nk; c += 256) act_store(kp + c, act_load(p + a.k_col + c));
-  for (int c = threadIdx.x; c < nv; c += 256) act_store(vp + c, act_load(p + a.v_col + c));
+  const float2* cs = a.cs + (int64_t)row * a.rot_half;
+  const TP* w = a.v0 ? reinterpret_cast<const TP*>(a.v0) + (int64_t)row * a.ldv0 : nullptr;
+  for (int c = threadIdx.x; c < nk; c += 256) act_store(kp + c, turned(p + a.k_col, c, c % a.dim, cs, a.rot_half));
+  for (int c = threadIdx.x; c < nv; c += 256) act_store(vp + c, mixed(act_load(p + a.v_col + c), w ? act_load(w + c) : 0.f, a));
+  if (turn_q && a.rot_half) {
+    const int H = a.H * a.maps;
+    for (int e = threadIdx.x; e < H * a.rot_half; e += 256) {
+      const int i = e % a.rot_half;
+      TP* q = p + (e / a.rot_half) * a.dim + 2 * i;
+      const float2 t = cs[i];
+      const float u = act_load(q), v = act_load(q + 1);
+      act_store(q, u * t.x - v * t.y);
+      act_store(q + 1, v * t.x + u * t.y);
+    }
+  }
+}
+
+// The same for bf16 rows and pages whose heads are whole 16-byte pieces.
+__global__ void __launch_bounds__(256) maps_append8_kernel(const AttnMapsArgs a, int turn_q) {
+  griddep_launch();
+  griddep_wait();
+  const int row = blockIdx.x, seg = a.row_seg ? a.row_seg[row] : row, pos = a.positions[row];
+  if (pos < 0) return;
+  const int64_t slot = (int64_t)a.tables[(int64_t)seg * a.ldbt + pos / kPage] * kPage + pos % kPage;
+  bf16* p = reinterpret_cast<bf16*>(const_cast<void*>(a.proj)) + (int64_t)row * a.ldp;
+  bf16* kp = reinterpret_cast<bf16*>(a.kpool) + slot * pool_ldk(a);
+  bf16* vp = reinterpret_cast<bf16*>(a.vpool) + slot * pool_ldv(a);
+  const float2* cs = a.cs + (int64_t)row * a.rot_half;
+  const bf16* w = a.v0 ? reinterpret_cast<const bf16*>(a.v0) + (int64_t)row * a.ldv0 : nullptr;
+  const int nk = a.G * a.maps * a.dim / 8, nv = a.G * a.vdim / 8, nq = turn_q && a.rot_half ? a.H * a.maps * a.dim / 8 : 0;
+  for (int e = threadIdx.x; e < nk + nq + nv; e += 256) {
+    float f[8];
+    if (e < nk + nq) {
+      const int c = (e < nk ? e : e - nk) * 8, i0 = c % a.dim / 2;
+      bf16* src = p + (e < nk ? a.k_col : 0) + c;
+      bf16x8_to_float(*reinterpret_cast<const uint4*>(src), f);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (i0 + i < a.rot_half) {
+          const float2 t = cs[i0 + i];
+          const float u = f[2 * i], v = f[2 * i + 1];
+          f[2 * i] = u * t.x - v * t.y;
+          f[2 * i + 1] = v * t.x + u * t.y;
+        }
+      }
+      *reinterpret_cast<uint4*>(e < nk ? kp + c : src) = float_to_bf16x8(f);
+    } else {
+      const int c = (e - nk - nq) * 8;
+      bf16x8_to_float(*reinterpret_cast<const uint4*>(p + a.v_col + c), f);
+      if (w) {
+        float g[8];
+        bf16x8_to_float(*reinterpret_cast<const uint4*>(w + c), g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = mixed(f[i], g[i], a);
+      }
+      *reinterpret_cast<uint4*>(vp + c) = float_to_bf16x8(f);
+    }
+  }
 }
 
 // One CTA per (query row, head, map): 128 keys at a time, scores by thread, running softmax, values by column.
@@ -47,7 +104,7 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
   const TA* V = reinterpret_cast<const TA*>(a.vpool) + (int64_t)g * a.vdim;
   const int* bt = a.tables + (int64_t)seg * a.ldbt;
   float m = -INFINITY, l = 0.f;
-  for (int k0 = 0; k0 <= pos; k0 += kRT) {
+  for (int k0 = first_key(a, pos); k0 <= pos; k0 += kRT) {
     const int n = min(kRT, pos + 1 - k0), j = k0 + tid;
     float s = -INFINITY;
     if (tid < n) {
@@ -78,14 +135,20 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
   for (int s = tid; s < a.nsplit; s += kRT) { pm[2 * s] = s ? -INFINITY : m; pm[2 * s + 1] = s ? 0.f : l; }
 }
 
-// One warp per (row, head): merge the key splits of every map, o = a_0 - lambda a_1 (two maps), RMS norm over the
-// head's values without weight (two maps), times post_scale, times sigmoid(gate).
+// One warp per (row, head): merge the key splits of every map (and its sink), o = a_0 - lambda a_1 (two maps), RMS norm
+// over the head's values without weight (two maps), times post_scale, times sigmoid(gate) per head and per element.
+struct ElemGate { const void* p; int64_t ld; int f32; };        // pre-activations [rows, H * vdim]
+__device__ __forceinline__ float elem_gate(const ElemGate& g, int64_t row, int c) {
+  return sigmoid_x(g.f32 ? reinterpret_cast<const float*>(g.p)[row * g.ld + c]
+                         : __bfloat162float(reinterpret_cast<const bf16*>(g.p)[row * g.ld + c]));
+}
 constexpr int kVMax = 16;      // values per lane: vdim <= 512; at most 64 splits (4 in the warp form)
 template <typename TA>
 __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                           const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
                                                           int64_t lda, const int* __restrict__ positions, int rows, int H,
-                                                          int maps, int vdim, int nsplit, float lambda, float post_scale, float eps) {
+                                                          int maps, int vdim, int nsplit, float lambda, float post_scale, float eps,
+                                                          const float* __restrict__ sink, const ElemGate eg) {
   griddep_launch();
   griddep_wait();
   const int64_t w = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -98,7 +161,7 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
   float o[kVMax];
 #pragma unroll
   for (int i = 0; i < kVMax; ++i) o[i] = 0.f;
-  if (nsplit == 1 && v4 && maps == 2) {                // prompts: everything a lane needs in one round of loads
+  if (nsplit == 1 && v4 && maps == 2 && !sink) {                // prompts: everything a lane needs in one round of loads
     const int64_t vh = (row * H + h) * 2;
     const float d0 = part_ml[vh * 2 + 1], d1 = part_ml[vh * 2 + 3];
     const float* po = part_o + vh * vdim;
@@ -123,10 +186,13 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
     float M = -INFINITY;
     if (lane < nsplit) M = ml[2 * lane];
     M = warp_max(M);
+    const float sk = sink ? sink[h * maps + mp] : -INFINITY;
+    M = fmaxf(M, sk);
     // splits are filled from the front: each lane weighs its own, the sums walk the filled ones
     float fac = 0.f, den = 0.f;
     if (lane < nsplit && ml[2 * lane] != -INFINITY) { fac = expf(ml[2 * lane] - M); den = fac * ml[2 * lane + 1]; }
     den = warp_sum(den);
+    if (sink) den += expf(sk - M);
     fac *= (mp == 0 ? 1.f : -lambda) / den;
     const int used = __popc(__ballot_sync(0xffffffffu, lane < nsplit && ml[2 * lane] != -INFINITY));
     for (int s = 0; s < used; ++s) {
@@ -158,6 +224,10 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
 #pragma unroll
   for (int i = 0; i < kVMax / 4; ++i) {
     const int v = 4 * (lane + 32 * i);
+    if (eg.p)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (v + e < vdim) o[4 * i + e] *= elem_gate(eg, row, h * vdim + v + e);
     if (v + 3 < vdim && v4 && lda % 4 == 0) {
       act_store4(out + v, make_float4(o[4 * i] * r, o[4 * i + 1] * r, o[4 * i + 2] * r, o[4 * i + 3] * r));
     } else {
@@ -174,7 +244,8 @@ template <typename TA>
 __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                                const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
                                                                int64_t lda, const int* __restrict__ positions, int H, int maps,
-                                                               int vdim, int nsplit, float lambda, float post_scale, float eps) {
+                                                               int vdim, int nsplit, float lambda, float post_scale, float eps,
+                                                               const float* __restrict__ sink, const ElemGate eg) {
   extern __shared__ float sm[];                        // [warps][vdim]
   __shared__ float red[32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -194,11 +265,11 @@ __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __re
 #pragma unroll
     for (int k = 0; k < 2; ++k)
       v[k] = lane + 32 * k < nsplit ? *reinterpret_cast<const float2*>(ml + 2 * (lane + 32 * k)) : make_float2(-INFINITY, 0.f);
-    const float M = warp_max(fmaxf(v[0].x, v[1].x));
+    const float sk = sink ? sink[h * maps + mp] : -INFINITY, M = fmaxf(sk, warp_max(fmaxf(v[0].x, v[1].x)));
     float fac[2];
 #pragma unroll
     for (int k = 0; k < 2; ++k) fac[k] = v[k].x == -INFINITY ? 0.f : expf(v[k].x - M);
-    const float den = warp_sum(fac[0] * v[0].y + fac[1] * v[1].y), c = (mp == 0 ? 1.f : -lambda) / den;
+    const float den = warp_sum(fac[0] * v[0].y + fac[1] * v[1].y) + (sink ? expf(sk - M) : 0.f), c = (mp == 0 ? 1.f : -lambda) / den;
     const int used = __popc(__ballot_sync(0xffffffffu, v[0].x != -INFINITY)) + __popc(__ballot_sync(0xffffffffu, v[1].x != -INFINITY));
 #pragma unroll 4
     for (int s = warp; s < used; s += kWT / 32) {
@@ -228,28 +299,35 @@ __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __re
   if (gates) r *= sigmoid_x(gates[row * ldg + h]);
 #pragma unroll
   for (int k = 0; k < 2; ++k)
-    if (tid + kWT * k < vdim) act_store(act + row * lda + (int64_t)h * vdim + tid + kWT * k, x[k] * r);
+    if (tid + kWT * k < vdim) {
+      const int c = h * vdim + tid + kWT * k;
+      act_store(act + row * lda + c, x[k] * r * (eg.p ? elem_gate(eg, row, c) : 1.f));
+    }
 }
 
 bool maps_args_ok(const AttnMapsArgs& a) {
   return a.proj && a.kpool && a.vpool && a.tables && a.positions && a.H > 0 && a.G > 0 && a.H % a.G == 0 && a.maps >= 1 && a.dim > 0 &&
-         a.vdim > 0;
+         a.vdim > 0 && 2 * a.rot_half <= a.dim && (!a.rot_half || a.cs);
 }
 
 }  // namespace
 
 CB_EXPORT int cb_attn_maps_args_size() { return (int)sizeof(AttnMapsArgs); }
 
-// Keys and values of `rows` projection rows into the pages.
-CB_EXPORT int cb_attn_maps_append(const void* args, int64_t rows, int64_t p_f32, int64_t f32, void* stream) {
+// Keys and values of `rows` projection rows into the pages; turn_q: their queries are turned in place.
+CB_EXPORT int cb_attn_maps_append(const void* args, int64_t rows, int64_t turn_q, int64_t p_f32, int64_t f32, void* stream) {
   if (!args || rows < 1) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (!maps_args_ok(a)) return CB_ERR_ARG;
   cudaStream_t st = (cudaStream_t)stream;
   const dim3 grid((unsigned)rows), block(256);
-  if (f32) return (int)cb_launch(maps_append_kernel<float, float>, grid, block, 0, st, a);
-  if (p_f32) return (int)cb_launch(maps_append_kernel<float, bf16>, grid, block, 0, st, a);
-  return (int)cb_launch(maps_append_kernel<bf16, bf16>, grid, block, 0, st, a);
+  const int tq = (int)turn_q;
+  if (f32) return (int)cb_launch(maps_append_kernel<float, float>, grid, block, 0, st, a, tq);
+  if (p_f32) return (int)cb_launch(maps_append_kernel<float, bf16>, grid, block, 0, st, a, tq);
+  const bool wide = !(a.dim % 8 || a.vdim % 8 || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || pool_ldk(a) % 8 || pool_ldv(a) % 8 ||
+                      a.ldv0 % 8 || (((uintptr_t)a.proj | (uintptr_t)a.v0 | (uintptr_t)a.kpool | (uintptr_t)a.vpool) & 15));
+  if (wide) return (int)cb_launch(maps_append8_kernel, grid, block, 0, st, a, tq);
+  return (int)cb_launch(maps_append_kernel<bf16, bf16>, grid, block, 0, st, a, tq);
 }
 
 // The plain kernel: every row against the pages (its own key included, so append first).
@@ -268,8 +346,11 @@ CB_EXPORT int cb_attn_maps_rows(const void* args, int64_t rows, int64_t p_f32, i
 
 CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const void* gates, int64_t ldg, void* act, int64_t lda,
                                   const void* positions, int64_t rows, int64_t H, int64_t maps, int64_t vdim, int64_t nsplit,
-                                  float lambda, float post_scale, float eps, int64_t f32, void* stream) {
+                                  float lambda, float post_scale, float eps, const void* sink, const void* egate, int64_t lde,
+                                  int64_t e_f32, int64_t f32, void* stream) {
   if (!part_o || !part_ml || !act || !positions || rows < 1 || maps < 1 || maps > 2 || nsplit < 1) return CB_ERR_ARG;
+  const float* sk = (const float*)sink;
+  const ElemGate eg = {egate, lde, (int)e_f32};
   if (vdim > 32 * kVMax || nsplit > 64) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
   if (nsplit > 4) {
@@ -279,17 +360,17 @@ CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const
     if (f32)
       return (int)cb_launch(maps_finish_wide_kernel<float>, wide, dim3(kWT), smem, st, (const float*)part_o, (const float*)part_ml,
                             (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)H, (int)maps, (int)vdim,
-                            (int)nsplit, lambda, post_scale, eps);
+                            (int)nsplit, lambda, post_scale, eps, sk, eg);
     return (int)cb_launch(maps_finish_wide_kernel<bf16>, wide, dim3(kWT), smem, st, (const float*)part_o, (const float*)part_ml,
                           (const float*)gates, ldg, (bf16*)act, lda, (const int*)positions, (int)H, (int)maps, (int)vdim, (int)nsplit,
-                          lambda, post_scale, eps);
+                          lambda, post_scale, eps, sk, eg);
   }
   const dim3 grid((unsigned)((rows * H + 3) / 4)), block(128);
   if (f32)
     return (int)cb_launch(maps_finish_kernel<float>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
                           (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps,
-                          (int)vdim, (int)nsplit, lambda, post_scale, eps);
+                          (int)vdim, (int)nsplit, lambda, post_scale, eps, sk, eg);
   return (int)cb_launch(maps_finish_kernel<bf16>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
                         (const float*)gates, ldg, (bf16*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps, (int)vdim,
-                        (int)nsplit, lambda, post_scale, eps);
+                        (int)nsplit, lambda, post_scale, eps, sk, eg);
 }

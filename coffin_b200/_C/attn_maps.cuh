@@ -4,6 +4,11 @@
 // out head by head as [map 0, map 1, ...] of `dim` each, key heads likewise, values once per key/value head.
 // Scores are scaled, multiplied by a position-dependent query temperature and optionally capped by
 // cap * tanh(score / cap); key and value sizes are independent.
+//
+// Optional parts, each switched on by its field: a sliding window (a query sees itself and the window - 1 tokens before
+// it), a sink per head (an entry of the softmax without key or value), interleaved rotary positions on queries and keys
+// (taken when rows are appended and when a decode query is read), values mixed with another layer's, and an output gate
+// per element.
 #pragma once
 #include "act_type.cuh"
 
@@ -23,7 +28,21 @@ struct AttnMapsArgs {
   // one map, prompt kernels: the finished head (divided by its denominator, times sigmoid(gate)) goes straight to
   // bf16 rows instead of part_o / part_ml (null: no)
   void* act; int64_t lda; const float* gates; int64_t ldg;
+  int window;                            // keys pos - window + 1 .. pos are visible (<= 0: all up to pos)
+  int rot_half;                          // pairs (2 i, 2 i + 1), i < rot_half, of queries and keys turn (0: none)
+  const float* sink;                     // [H * maps] in score units, or null
+  const float2* cs;                      // (cos, sin) [rows, rot_half]
+  const void* v0; int64_t ldv0;          // values of another layer, rows like proj (null: none):
+  float v_own, v_mix;                    //   v = v_own * own + v_mix * v0
+  const void* egate; int64_t lde;        // one map: output gate pre-activations [rows, H * vdim], rows like proj (null: none)
 };
+
+// first key that the query at `pos` sees
+__host__ __device__ __forceinline__ int first_key(const AttnMapsArgs& a, int pos) {
+  return a.window > 0 && pos >= a.window ? pos - a.window + 1 : 0;
+}
+// finite stand-in for "no key seen yet": exponentials of differences with it are 0 or 1, never NaN
+constexpr float kNoKey = -1e30f;
 
 constexpr int kPage = 64;
 __host__ __device__ __forceinline__ int64_t pool_ldk(const AttnMapsArgs& a) { return a.ldk ? a.ldk : (int64_t)a.G * a.maps * a.dim; }
@@ -31,6 +50,18 @@ __host__ __device__ __forceinline__ int64_t pool_ldv(const AttnMapsArgs& a) { re
 
 __device__ __forceinline__ float query_temp(const AttnMapsArgs& a, int pos) {
   return a.temp_every > 0 ? 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1)) : 1.f;
+}
+// entry c of a projected row (entry `in_head` of its head) after the turn
+template <typename T>
+__device__ __forceinline__ float turned(const T* p, int c, int in_head, const float2* cs, int half) {
+  const float x = act_load(p + c);
+  if (in_head >> 1 >= half) return x;
+  const float2 t = cs[in_head >> 1];
+  const float y = act_load(p + (in_head & 1 ? c - 1 : c + 1));
+  return in_head & 1 ? x * t.x + y * t.y : x * t.x - y * t.y;
+}
+__device__ __forceinline__ float mixed(float own, float other, const AttnMapsArgs& a) {
+  return a.v0 ? a.v_own * own + a.v_mix * other : own;
 }
 // tanh through one exponential: |error| ~ 1e-7
 __device__ __forceinline__ float cap_score(float s, float cap, float inv_cap) {

@@ -75,7 +75,7 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
     const bool ok = r < rows && c < a.dim;
     cp16(qs + r * LK + c, ok ? Q + (int64_t)r * a.ldp + c : Q, ok);
   }
-  const int last = pos0 + t0 + rows - 1, pages = last / kPage + 1;
+  const int last = pos0 + t0 + rows - 1, pages = last / kPage + 1, page0 = first_key(a, pos0 + t0) / kPage;
   auto load = [&](int pg) {
     const int64_t base = (int64_t)bt[pg] * kPage;
     bf16* kd = ks + (pg & 1) * kBN * LK;
@@ -92,13 +92,13 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  load(0);
+  load(page0);
   float o[NV][4];
 #pragma unroll
   for (int i = 0; i < NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float mx[2] = {-INFINITY, -INFINITY}, den[2] = {0.f, 0.f};
+  float mx[2] = {kNoKey, kNoKey}, den[2] = {0.f, 0.f};       // finite: with a window a page may hold no key of a row
   const int rlo = warp * 16 + g4;                                // tile rows of this lane: rlo, rlo + 8
-  const int plo = pos0 + t0 + rlo, phi = plo + 8;
+  const int plo = pos0 + t0 + rlo, phi = plo + 8, klo = first_key(a, plo), khi = first_key(a, phi);   // positions, first keys
   const float inv_cap = CAP ? 1.f / a.cap : 0.f;
   float f[2];
 #pragma unroll
@@ -108,8 +108,8 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
   }
   const float cap2 = a.cap * kLog2e;
   uint32_t qf[QREG ? NK : 1][4];
-  const int warp_last = pos0 + t0 + warp * 16 + 15;
-  for (int pg = 0; pg < pages; ++pg) {
+  const int warp_last = pos0 + t0 + warp * 16 + 15, warp_first = first_key(a, pos0 + t0 + warp * 16), warp_full = first_key(a, warp_last);
+  for (int pg = page0; pg < pages; ++pg) {
     if (pg + 1 < pages) {
       load(pg + 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -117,11 +117,11 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    if (QREG && pg == 0) {
+    if (QREG && pg == page0) {
 #pragma unroll
       for (int k = 0; k < NK; ++k) ldsm4(qf[QREG ? k : 0], qs + (warp * 16 + (lane & 15)) * LK + k * 16 + (lane >> 4) * 8);
     }
-    if (pg * kPage <= warp_last) {
+    if (pg * kPage <= warp_last && pg * kPage + kPage > warp_first) {
       const bf16* kt = ks + (pg & 1) * kBN * LK;
       const bf16* vt = vs + (pg & 1) * kBN * LV;
       float s[8][4];
@@ -140,7 +140,8 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
           mma(s[2 * j + 1], qa, b[2], b[3]);
         }
       }
-      const bool edge = pg * kPage + kPage - 1 > pos0 + t0 + warp * 16;    // some key of the page is after some row
+      // some key of the page is after some row, or before some row's window
+      const bool edge = pg * kPage + kPage - 1 > pos0 + t0 + warp * 16 || pg * kPage < warp_full;
       float nm[2] = {mx[0], mx[1]};
 #pragma unroll
       for (int i = 0; i < 8; ++i)
@@ -148,7 +149,10 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
         for (int e = 0; e < 4; ++e) {
           float x = s[i][e] * f[e >> 1];
           if (CAP) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);        // log2(e) * cap * tanh(score / cap)
-          if (edge && pg * kPage + i * 8 + t4 * 2 + (e & 1) > (e >> 1 ? phi : plo)) x = -INFINITY;
+          if (edge) {
+            const int key = pg * kPage + i * 8 + t4 * 2 + (e & 1);
+            if (key > (e >> 1 ? phi : plo) || key < (e >> 1 ? khi : klo)) x = -INFINITY;
+          }
           s[i][e] = x;
           nm[e >> 1] = fmaxf(nm[e >> 1], x);
         }
@@ -156,7 +160,6 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
       for (int i = 0; i < 2; ++i) {
         nm[i] = fmaxf(nm[i], __shfl_xor_sync(0xffffffffu, nm[i], 1));
         nm[i] = fmaxf(nm[i], __shfl_xor_sync(0xffffffffu, nm[i], 2));
-        // a tile's first page always holds a visible key (key 0), so nm is finite from then on
         const float w = ex2(mx[i] - nm[i]);
         if (nm[i] > mx[i]) {
 #pragma unroll
@@ -198,12 +201,21 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
     if (r >= rows) continue;
     if (a.act) {                                                 // one map: the head is finished here
       const int64_t row = row0 + t0 + r;
+      if (a.sink) den[i] += ex2(a.sink[h] * kLog2e - mx[i]);
       const float s = (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / den[i];
       bf16* out = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * a.vdim;
+      const bf16* eg = a.egate ? reinterpret_cast<const bf16*>(a.egate) + row * a.lde + (int64_t)h * a.vdim : nullptr;
 #pragma unroll
       for (int v = 0; v < NV; ++v) {
         const int c = v * 8 + t4 * 2;
-        if (c < a.vdim) *reinterpret_cast<uint32_t*>(out + c) = pack_bf162(o[v][2 * i] * s, o[v][2 * i + 1] * s);
+        if (c >= a.vdim) continue;
+        float x = o[v][2 * i] * s, y = o[v][2 * i + 1] * s;
+        if (eg) {
+          const uint32_t g = *reinterpret_cast<const uint32_t*>(eg + c);
+          x *= sigmoid_x(__uint_as_float(g << 16));
+          y *= sigmoid_x(__uint_as_float(g & 0xffff0000u));
+        }
+        *reinterpret_cast<uint32_t*>(out + c) = pack_bf162(x, y);
       }
       continue;
     }
@@ -264,8 +276,8 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
   const int pos = a.positions[row], seg = a.row_seg ? a.row_seg[row] : row;
   if (pos < 0) return;
   const int64_t vh0 = (int64_t)row * a.H * MAPS + (int64_t)(g * R + r0) * MAPS;
-  const int pages = pos / kPage + 1, per = (pages + a.nsplit - 1) / a.nsplit;
-  const int pg0 = split * per, pg1 = min(pages, pg0 + per);
+  const int lo = first_key(a, pos), page0 = lo / kPage, pages = pos / kPage + 1, per = (pages - page0 + a.nsplit - 1) / a.nsplit;
+  const int pg0 = page0 + split * per, pg1 = min(pages, pg0 + per);
   if (pg0 >= pages) {
     if (tid < nq) a.part_ml[((vh0 + tid) * a.nsplit + split) * 2] = -INFINITY;
     return;
@@ -275,6 +287,8 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
   bf16* K = reinterpret_cast<bf16*>(a.kpool) + (int64_t)g * MAPS * a.dim;
   bf16* V = reinterpret_cast<bf16*>(a.vpool) + (int64_t)g * a.vdim;
   const TP* pr = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp;
+  const float2* cs = a.cs + (int64_t)row * a.rot_half;
+  const TP* v0 = a.v0 ? reinterpret_cast<const TP*>(a.v0) + (int64_t)row * a.ldv0 : nullptr;
   auto load = [&](int pg) {
     const int64_t base = (int64_t)bt[pg] * kPage;
     const int n = pos + 1 - pg * kPage;                // keys of the page that exist
@@ -298,7 +312,7 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
   for (int e = tid; e < MAPS * 8 * LK; e += kDT) {
     const int m = e / (8 * LK), i = (e / LK) % 8, c = e % LK;
     const bool ok = i < nh && c < a.dim;
-    qs[e] = ok ? __float2bfloat16(act_load(pr + ((int64_t)(g * R + r0 + i) * MAPS + m) * a.dim + c)) : __float2bfloat16(0.f);
+    qs[e] = ok ? __float2bfloat16(turned(pr, ((g * R + r0 + i) * MAPS + m) * a.dim + c, c, cs, a.rot_half)) : __float2bfloat16(0.f);
   }
   for (int e = tid; e < 16 * (kPage + 8); e += kDT) pa[e] = __float2bfloat16(0.f);
   float o[NPW][2][4];
@@ -323,12 +337,13 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
       const int r = pos % kPage;
       const int64_t slot = (int64_t)bt[pg] * kPage + r;
       for (int c = tid; c < MAPS * a.dim; c += kDT) {
-        const bf16 x = __float2bfloat16(act_load(pr + a.k_col + (int64_t)g * MAPS * a.dim + c));
+        const bf16 x = __float2bfloat16(turned(pr + a.k_col, g * MAPS * a.dim + c, c % a.dim, cs, a.rot_half));
         kt[((c / a.dim) * kPage + r) * LK + c % a.dim] = x;
         K[slot * ldk + c] = x;
       }
       for (int c = tid; c < a.vdim; c += kDT) {
-        const bf16 x = __float2bfloat16(act_load(pr + a.v_col + (int64_t)g * a.vdim + c));
+        const int64_t vc = (int64_t)g * a.vdim + c;
+        const bf16 x = __float2bfloat16(mixed(act_load(pr + a.v_col + vc), v0 ? act_load(v0 + vc) : 0.f, a));
         vt[r * LV + c] = x;
         V[slot * ldv + c] = x;
       }
@@ -355,14 +370,14 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
           float x = (s[e] + s2[e]) * f;
           if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
           const int key = warp * 8 + t4 * 2 + e;
-          ps[(g4 * MAPS + m) * kPage + key] = pg * kPage + key <= pos ? x : -INFINITY;
+          ps[(g4 * MAPS + m) * kPage + key] = pg * kPage + key <= pos && pg * kPage + key >= lo ? x : -INFINITY;
         }
       }
     }
     __syncthreads();
     if (warp < nq) {
       const float2 x = *reinterpret_cast<const float2*>(ps + warp * kPage + 2 * lane);
-      const float mn = fmaxf(m_run, warp_max(fmaxf(x.x, x.y)));  // finite: the first key of a walked page is visible
+      const float mn = fmaxf(m_run, warp_max(fmaxf(x.x, x.y)));  // finite: a walked page holds a visible key
       float e0 = ex2(x.x - mn), e1 = ex2(x.y - mn);
       const float w = ex2(m_run - mn);
       l_run = l_run * w + warp_sum(e0 + e1);
@@ -445,7 +460,7 @@ CB_EXPORT int cb_attn_maps_flash(const void* args, int64_t segs, int64_t max_row
   if (!args || segs < 1 || segs > 65535 || max_rows < 1) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G) return CB_ERR_ARG;
-  if (a.act ? a.maps != 1 || a.lda % 2 : !a.part_o || !a.part_ml) return CB_ERR_ARG;
+  if (a.act ? a.maps != 1 || a.lda % 2 || a.lde % 2 : !a.part_o || !a.part_ml) return CB_ERR_ARG;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   const int tiles = (int)((max_rows + kBM - 1) / kBM);
   cudaStream_t st = (cudaStream_t)stream;
@@ -460,7 +475,7 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   if (!args || rows < 1 || rows > 65535) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
-      a.nsplit < 1 || a.nsplit > 64)
+      a.nsplit < 1 || a.nsplit > 64 || 2 * a.rot_half > a.dim || (a.rot_half && !a.cs))
     return CB_ERR_ARG;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;

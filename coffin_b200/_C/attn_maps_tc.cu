@@ -77,7 +77,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   const int seg0 = a.seg_row[seg], n = a.seg_row[seg + 1] - seg0, pos0 = a.seg_pos[seg];
   const int row0 = qt * kBQ;
   if (row0 >= n) return;                              // the whole CTA, before anything is allocated
-  const int n_tiles = (pos0 + min(n, row0 + kBQ) - 1) / kBKV + 1;
+  const int page0 = first_key(a, pos0 + row0) / kBKV;             // pages before it are outside every row's window
+  const int n_tiles = (pos0 + min(n, row0 + kBQ) - 1) / kBKV + 1 - page0;
 
   if (threadIdx.x == 0) {
     mbar_init(&q_full, 8);
@@ -112,7 +113,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       for (int j = 0; j < n_tiles && !*abort_flag; ++j) {
         const int s = j % STAGES;
         const uint32_t ph = (j / STAGES) & 1;
-        const int slot0 = bt[j] * kBKV;
+        const int slot0 = bt[page0 + j] * kBKV;
         if (!wait_bar(&k_free[s], ph ^ 1, abort_flag)) { atomicCAS(status, 0, 81); abort_s = 1; break; }
         mbar_expect_tx(&k_full[s], K_BYTES);
         for (int c = 0; c < NK; ++c) tma_load_2d(Ks + s * K_BYTES + c * KC, &tmK, &k_full[s], kmap * DK + c * 64, slot0);
@@ -190,6 +191,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     // score -> log2 units; with a cap first to the exponent of exp(2 score / cap)
     const float f = a.scale * query_temp(a, min(pos, pos0 + n - 1)) * (MODE == PLAIN ? kLog2e : 2.f * kLog2e / a.cap);
     const float cap2 = a.cap * kLog2e;
+    const int key_lo = first_key(a, pos), full_lo = first_key(a, pos0 + row0 + kBQ - 1);
     float m_ref = MODE == CAP_FIXED ? cap2 : -INFINITY, l = 0.f;
     bool ok = true;
     uint32_t xph = 0;
@@ -203,14 +205,14 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[sb]);
-      const int key0 = j * kBKV + hf * 32;
-      const bool edge = j * kBKV + kBKV - 1 > pos0 + row0;       // the page touches the diagonal
+      const int page = (page0 + j) * kBKV, key0 = page + hf * 32;
+      const bool edge = page + kBKV - 1 > pos0 + row0 || page < full_lo;     // the page touches the diagonal or a window's start
       if (MODE == CAP_FIXED) {
         // 2^(log2e (cap tanh - cap)) = 2^(-2 cap log2e / (exp(2 s / cap) + 1))
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
           float p = ex2(-2.f * cap2 * rcp(ex2(__uint_as_float(sv[c]) * f) + 1.f));
-          if (edge && key0 + c > pos) p = 0.f;
+          if (edge && (key0 + c > pos || key0 + c < key_lo)) p = 0.f;
           sv[c] = __float_as_uint(p);
         }
       } else {
@@ -219,7 +221,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         for (int c = 0; c < 32; ++c) {
           float x = __uint_as_float(sv[c]) * f;
           if (MODE == CAP) x = cap2 - 2.f * cap2 * rcp(ex2(x) + 1.f);
-          if (edge && key0 + c > pos) x = -INFINITY;
+          if (edge && (key0 + c > pos || key0 + c < key_lo)) x = -INFINITY;
           sv[c] = __float_as_uint(x);
           mx = fmaxf(mx, x);
         }
@@ -227,9 +229,9 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         mbar_arrive(&pair_bar[q]);
         if (!wait_bar(&pair_bar[q], xph, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 92); abort_s = 1; } ok = false; break; }
         xph ^= 1;
-        mx = fmaxf(xch[sb][0][r], xch[sb][1][r]);
+        mx = fmaxf(kNoKey, fmaxf(xch[sb][0][r], xch[sb][1][r]));   // finite: with a window a page may hold no key of a row
         if (j == 0) {
-          m_ref = mx;                                  // key 0 is visible to every row: finite
+          m_ref = mx;
         } else if (__any_sync(0xffffffffu, mx > m_ref + 8.f)) {
           // every product that wrote O has to be complete before its rows are rescaled
           if (!wait_bar(&p_free[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag)) {
@@ -296,7 +298,9 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     if (ok && a.act) {                                 // one map: the head is finished here
       tc_fence_after();
       const int64_t row = seg0 + t;
+      if (a.sink) l += ex2(a.sink[h] * kLog2e - m_ref);
       const float s = t < n ? (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / l : 0.f;
+      const bf16* eg = a.egate ? reinterpret_cast<const bf16*>(a.egate) + row * a.lde + (int64_t)h * DV : nullptr;
       bf16* op = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * DV;
 #pragma unroll 1
       for (int c0 = hf * (DV / 2); c0 < (hf + 1) * (DV / 2); c0 += 32) {
@@ -309,6 +313,12 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
             float x[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[8 * v + e]) * s;
+            if (eg) {
+              float g[8];
+              bf16x8_to_float(*reinterpret_cast<const uint4*>(eg + c0 + v * 8), g);
+#pragma unroll
+              for (int e = 0; e < 8; ++e) x[e] *= sigmoid_x(g[e]);
+            }
             *reinterpret_cast<uint4*>(op + c0 + v * 8) = float_to_bf16x8(x);
           }
         }
@@ -379,7 +389,8 @@ CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_
   if (!args || segs < 1 || segs > 65535 || max_rows < 1 || !status) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G || a.maps < 1) return CB_ERR_ARG;
-  if (a.act ? a.maps != 1 || a.lda % 8 || ((uintptr_t)a.act & 15) : !a.part_o || !a.part_ml) return CB_ERR_ARG;
+  if (a.act ? a.maps != 1 || a.lda % 8 || ((uintptr_t)a.act & 15) || a.lde % 8 || ((uintptr_t)a.egate & 15) : !a.part_o || !a.part_ml)
+    return CB_ERR_ARG;
   if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || a.ldp % 8 || a.ldk % 8 || a.ldv % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
   CUtensorMap tmK, tmV;
   const uint64_t kw = (uint64_t)a.G * a.maps * a.dim, vw = (uint64_t)a.G * a.vdim;

@@ -46,7 +46,7 @@ struct GemmArgs {
   int splits; float* ws; unsigned* tickets;
   int c_f32 = 0;                   // C is fp32 instead of bf16 (gate pre-activations, logits)
   float* C2 = nullptr; int64_t ldc2 = 0; int n_main = 0;   // columns from n_main on leave as fp32 in C2 (null: none)
-  int act = 0; float act_a = 0.f, act_b = 0.f;   // 1: xIELU epilogue with these coefficients
+  int act = 0; float act_a = 0.f, act_b = 0.f;   // epilogue activation (epi_act), 0: none
 };
 struct TileCoord { int m0, row_end, n0, brow; };
 template <int BN>
@@ -238,8 +238,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
               f.z *= rsr * a.col_scale[gcol + 2]; f.w *= rsr * a.col_scale[gcol + 3];
             }
             if (a.act) {
-              f.x = xielu_s(f.x, a.act_a, a.act_b); f.y = xielu_s(f.y, a.act_a, a.act_b);
-              f.z = xielu_s(f.z, a.act_a, a.act_b); f.w = xielu_s(f.w, a.act_a, a.act_b);
+              f.x = epi_act(a.act, f.x, a.act_a, a.act_b); f.y = epi_act(a.act, f.y, a.act_a, a.act_b);
+              f.z = epi_act(a.act, f.z, a.act_a, a.act_b); f.w = epi_act(a.act, f.w, a.act_a, a.act_b);
             }
             if (a.residual) {
               const uint2 rr = *reinterpret_cast<const uint2*>(a.residual + (int64_t)grow * a.ldr + gcol);
@@ -287,7 +287,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             for (int i = 0; i < 8; ++i) {
               if (I8) f[i] = (float)(int)r[v * 8 + i] * rs * cscale[col0 + v * 8 + i];
               else f[i] = __uint_as_float(r[v * 8 + i]);
-              if (a.act) f[i] = xielu_s(f[i], a.act_a, a.act_b);
+              if (a.act) f[i] = epi_act(a.act, f[i], a.act_a, a.act_b);
             }
             if (rp) {
               float g[8];
@@ -598,11 +598,12 @@ CB_EXPORT int cb_gemm_i8(const void* A, int64_t lda, const void* W, int64_t ldw,
 // Grouped (expert-major) product for routed-MoE prefill: rows of A sorted by expert, W a stack
 // [E, N, K]; C[r, :] = A[r, :] x W[expert(r)]^T for the rows the tile list covers.  The list
 // (g_count m-tiles of at most 128 rows, never crossing an expert boundary) is produced on the device
-// by cb_moe_dispatch, so no count travels to the host; max_tiles bounds it and sizes the grid.
+// by cb_moe_dispatch, so no count travels to the host; max_tiles bounds it and sizes the grid.  act 2: squared relu
+// in the epilogue (0: none).
 // Replaces the reference's expert-major grouped GEMMs (kernels/w8a8_tcu.cu:962, moe_grouped_i8.cu:1283).
 CB_EXPORT int cb_gemm_bf16_grouped(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                                    int64_t rows, int64_t E, int64_t N, int64_t K, const void* g_count,
-                                   const void* g_row0, const void* g_rows, const void* g_expert, int64_t max_tiles,
+                                   const void* g_row0, const void* g_rows, const void* g_expert, int64_t max_tiles, int64_t act,
                                    void* status, void* stream) {
   if (rows < 1 || N < 1 || K < 1 || E < 1 || max_tiles < 1) return CB_ERR_SHAPE;
   if (K % 8 || N % 8 || ldc % 8 || !status || !g_count || !g_row0 || !g_rows || !g_expert) return CB_ERR_SHAPE;
@@ -620,6 +621,7 @@ CB_EXPORT int cb_gemm_bf16_grouped(const void* A, int64_t lda, const void* W, in
   a.pf = nullptr; a.pf_seq = 0;
   a.g_count = (const int*)g_count; a.g_row0 = (const int*)g_row0; a.g_rows = (const int*)g_rows; a.g_expert = (const int*)g_expert;
   a.splits = 1; a.ws = nullptr; a.tickets = nullptr;
+  a.act = (int)act;
   cudaStream_t st = (cudaStream_t)stream;
   if (bn == 256) return launch_gemm<256, 4, false>(tmA, tmB, a, sms, st);
   if (bn == 160) return launch_gemm<160, 5, false>(tmA, tmB, a, sms, st);

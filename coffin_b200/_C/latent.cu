@@ -71,17 +71,45 @@ struct LatentArgs {
   const float2* cs; int half;            // angles [rows, half]
   int q_rank, kv_rank, rot, cp;
   float eps;
+  // queries without a latent (q_rank 0): the projection rows hold H heads of hq columns whose rotated part starts at column
+  // r_off; it is turned in place for the rows before `split` and into qa [rows - split, H, ldk] at column cp from there on
+  int H, split; int64_t hq, r_off; void* qa; int64_t ldqa;
 };
 
 constexpr int kPT = 256, kPV = 8;        // values a thread keeps in registers
 template <typename TP, typename TA>
 __global__ void __launch_bounds__(kPT) latent_rows_kernel(const LatentArgs a) {
   __shared__ float red[32];
-  const int row = blockIdx.x, part = blockIdx.y;                 // part 0: query latent, 1: c and the rotated part
+  const int row = blockIdx.x, part = blockIdx.y;                 // part 0: query latent or heads, 1: c and the rotated part
   griddep_launch();
   griddep_wait();
   const int pos = a.positions[row];
   if (pos < 0) return;
+  if (!part && !a.q_rank) {
+    TP* q = reinterpret_cast<TP*>(const_cast<void*>(a.proj)) + (int64_t)row * a.ldp + a.r_off;
+    TA* qa = reinterpret_cast<TA*>(a.qa) + (int64_t)(row - a.split) * a.ldqa + a.cp;
+    const int np = (a.rot + 1) / 2;
+    for (int e = threadIdx.x; e < a.H * np; e += kPT) {
+      const int h = e / np, i = e % np;
+      const bool two = 2 * i + 1 < a.rot;
+      TP* s = q + h * a.hq + 2 * i;
+      float u = act_load(s), v = two ? act_load(s + 1) : 0.f;
+      if (i < a.half) {
+        const float2 cs = a.cs[(int64_t)row * a.half + i];
+        const float x = u * cs.x - v * cs.y;
+        v = v * cs.x + u * cs.y;
+        u = x;
+      }
+      if (row < a.split) {
+        act_store(s, u);
+        if (two) act_store(s + 1, v);
+      } else {
+        act_store(qa + h * a.ldk + 2 * i, u);
+        if (two) act_store(qa + h * a.ldk + 2 * i + 1, v);
+      }
+    }
+    return;
+  }
   const TP* p = reinterpret_cast<const TP*>(a.proj) + (int64_t)row * a.ldp + (part ? a.c_col : 0);
   const int n = part ? a.kv_rank : a.q_rank;
   const float* w = part ? a.norm_c : a.norm_q;
@@ -149,15 +177,15 @@ __global__ void __launch_bounds__(256) rope_heads_kernel(const TS* __restrict__ 
 }
 
 // ---- page rows, gathered -----------------------------------------------------------------------
-// dst rows [base[s] + j] = page row of token j of segment s, in 16-byte pieces; pages[s] whole pages
+// dst rows [base[s] + j] = page row of token j of segment s, counted from its page first[s] on, in 16-byte pieces
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ pool, int64_t ld16, const int* __restrict__ tables,
                                                             int64_t ldbt, const int* __restrict__ base, const int* __restrict__ lens,
-                                                            uint4* __restrict__ dst) {
+                                                            const int* __restrict__ first, uint4* __restrict__ dst) {
   griddep_launch();
   griddep_wait();
   const int pg = blockIdx.x, s = blockIdx.y, left = lens[s] - pg * kPage;
   if (left <= 0) return;
-  const uint4* src = pool + (int64_t)tables[(int64_t)s * ldbt + pg] * kPage * ld16;
+  const uint4* src = pool + (int64_t)tables[(int64_t)s * ldbt + first[s] + pg] * kPage * ld16;
   uint4* d = dst + ((int64_t)base[s] + pg * kPage) * ld16;
   const int n = (int)(kPage * ld16), ok = (int)(min(left, kPage) * ld16);
   for (int e = threadIdx.x; e < n; e += 256) d[e] = e < ok ? src[e] : make_uint4(0, 0, 0, 0);
@@ -266,7 +294,7 @@ struct LatentDecodeArgs {
   const void* pool; int64_t ldk;         // page rows
   const int* tables; int64_t ldbt; const int* row_seg; const int* positions;
   float* part_o; float* part_ml;         // [rows, H, nsplit, cp], [.., 2]
-  int H, cp, nsplit;
+  int H, cp, nsplit, window;             // window <= 0: none
   float scale;
 };
 constexpr int kDT = 512, kPS = kPage + 4;
@@ -287,8 +315,9 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
   const int pos = a.positions[row], seg = a.row_seg ? a.row_seg[row] : row;
   if (pos < 0) return;
   const int64_t vh0 = (int64_t)row * a.H + h0;
-  const int pages = pos / kPage + 1, per = (pages + a.nsplit - 1) / a.nsplit;
-  const int pg0 = split * per, pg1 = min(pages, pg0 + per);
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, page0 = lo / kPage;     // first visible key
+  const int pages = pos / kPage + 1, per = (pages - page0 + a.nsplit - 1) / a.nsplit;
+  const int pg0 = page0 + split * per, pg1 = min(pages, pg0 + per);
   if (pg0 >= pages) {
     if (tid < nh) a.part_ml[((vh0 + tid) * a.nsplit + split) * 2] = -INFINITY;
     return;
@@ -378,9 +407,9 @@ __global__ void __launch_bounds__(kDT, 1) latent_decode_kernel(const LatentDecod
         const float2 p = *reinterpret_cast<const float2*>(ps + (c * NH + hd) * kPS + 2 * lane);
         x.x += p.x; x.y += p.y;
       }
-      x.x = key <= pos ? x.x * f : -INFINITY;
-      x.y = key + 1 <= pos ? x.y * f : -INFINITY;
-      const float mn = fmaxf(m_run[i], warp_max(fmaxf(x.x, x.y)));     // finite: the first key of a walked page is visible
+      x.x = key <= pos && key >= lo ? x.x * f : -INFINITY;
+      x.y = key + 1 <= pos && key + 1 >= lo ? x.y * f : -INFINITY;
+      const float mn = fmaxf(m_run[i], warp_max(fmaxf(x.x, x.y)));     // finite: a walked page holds a visible key
       float e0 = ex2(x.x - mn), e1 = ex2(x.y - mn);
       const float w = ex2(m_run[i] - mn);
       l_run[i] = l_run[i] * w + e0 + e1;               // this lane's share
@@ -515,12 +544,15 @@ CB_EXPORT int cb_rope_rows(const void* positions, const void* turns, void* cs, i
                         (const int*)positions, (const double*)turns, (float2*)cs, (int)rows, (int)half);
 }
 
-// `rows` projection rows: cq = rmsnorm(query latent); with own != 0 also rmsnorm(c) and the rotated part into the pages.
+// `rows` projection rows: cq = rmsnorm(query latent), or the rotated query parts turned (q_rank 0); with own != 0 also
+// rmsnorm(c) and the rotated part into the pages.
 // p_f32: projection rows are fp32; f32: latents and pages are fp32 instead of bf16.
 CB_EXPORT int cb_latent_rows(const void* args, int64_t rows, int64_t own, int64_t p_f32, int64_t f32, void* stream) {
   if (!args || rows < 1) return CB_ERR_ARG;
   const LatentArgs& a = *(const LatentArgs*)args;
-  if (!a.proj || !a.norm_q || !a.cq || !a.positions || a.q_rank < 1) return CB_ERR_ARG;
+  if (!a.proj || !a.positions || a.q_rank < 0 || (a.q_rank && (!a.norm_q || !a.cq))) return CB_ERR_ARG;
+  if (!a.q_rank && (a.H < 1 || a.split < 0 || (a.split < rows && !a.qa) || (p_f32 && !f32) || 2 * a.half > a.rot || (a.half && !a.cs)))
+    return CB_ERR_ARG;
   if (own && (!a.pool || !a.norm_c || !a.tables || a.kv_rank < 1 || a.kv_rank > a.cp || a.cp + a.rot > a.ldk || (a.half && !a.cs) || 2 * a.half > a.rot))
     return CB_ERR_ARG;
   const dim3 grid((unsigned)rows, own ? 2u : 1u), block(kPT);
@@ -543,13 +575,14 @@ CB_EXPORT int cb_rope_heads(const void* src, int64_t lds, int64_t hs, void* dst,
                         (const float2*)cs, (int)half, (int)rot, (int)H, (int)rows);
 }
 
-// Page rows of `segs` sequences side by side: segment s fills rows base[s] .. base[s] + whole pages of lens[s] tokens.
+// Page rows of `segs` sequences side by side: segment s fills rows base[s] .. base[s] + whole pages of lens[s] tokens, from
+// page first[s] of its table on.
 CB_EXPORT int cb_latent_gather(const void* pool, int64_t row_bytes, const void* tables, int64_t ldbt, const void* base, const void* lens,
-                               void* dst, int64_t segs, int64_t max_pages, void* stream) {
-  if (!pool || !tables || !base || !lens || !dst || segs < 1 || segs > 65535 || max_pages < 1) return CB_ERR_ARG;
+                               const void* first, void* dst, int64_t segs, int64_t max_pages, void* stream) {
+  if (!pool || !tables || !base || !lens || !first || !dst || segs < 1 || segs > 65535 || max_pages < 1) return CB_ERR_ARG;
   if (row_bytes % 16) return CB_ERR_SHAPE;
   return (int)cb_launch(latent_gather_kernel, dim3((unsigned)max_pages, (unsigned)segs), dim3(256), 0, (cudaStream_t)stream,
-                        (const uint4*)pool, row_bytes / 16, (const int*)tables, ldbt, (const int*)base, (const int*)lens, (uint4*)dst);
+                        (const uint4*)pool, row_bytes / 16, (const int*)tables, ldbt, (const int*)base, (const int*)lens, (const int*)first, (uint4*)dst);
 }
 
 // y[t, h, :N] = w[h] x[t, h, :K] (* sigmoid(gate[t, h])), w [H, N, K]; bf16 (K % 8 == 0, 16-byte rows) or fp32.
@@ -577,10 +610,11 @@ CB_EXPORT int cb_latent_decode_ok(int64_t ldk, int64_t cp) {
 }
 
 // Absorbed attention of `rows` queries [rows, H, ldk] against the pages (their own rows appended before): key splits into
-// part_o [rows, H, nsplit, cp] / part_ml.  tiles: groups of 16 heads a CTA serves (1 or 2).
+// part_o [rows, H, nsplit, cp] / part_ml.  tiles: groups of 16 heads a CTA serves (1 or 2); window: tokens a query sees,
+// itself included (<= 0: all up to it).
 CB_EXPORT int cb_latent_decode(const void* q, int64_t ldq, const void* pool, int64_t ldk, const void* tables, int64_t ldbt,
                                const void* row_seg, const void* positions, void* part_o, void* part_ml, int64_t rows, int64_t H, int64_t cp,
-                               int64_t nsplit, int64_t tiles, float scale, void* stream) {
+                               int64_t nsplit, int64_t tiles, int64_t window, float scale, void* stream) {
   if (tiles < 1 || tiles > 2) return CB_ERR_ARG;
   if (!q || !pool || !tables || !positions || !part_o || !part_ml || rows < 1 || rows > 65535 || H < 1 || nsplit < 1 || nsplit > 64)
     return CB_ERR_ARG;
@@ -588,7 +622,7 @@ CB_EXPORT int cb_latent_decode(const void* q, int64_t ldq, const void* pool, int
   LatentDecodeArgs a;
   a.q = q; a.ldq = ldq; a.pool = pool; a.ldk = ldk; a.tables = (const int*)tables; a.ldbt = ldbt; a.row_seg = (const int*)row_seg;
   a.positions = (const int*)positions; a.part_o = (float*)part_o; a.part_ml = (float*)part_ml; a.H = (int)H; a.cp = (int)cp;
-  a.nsplit = (int)nsplit; a.scale = scale;
+  a.nsplit = (int)nsplit; a.window = (int)window; a.scale = scale;
   cudaStream_t st = (cudaStream_t)stream;
   const int r = (int)rows;
   if (tiles == 1) return cp <= 256 ? launch_decode<1, 1>(a, r, st) : launch_decode<1, 2>(a, r, st);

@@ -107,7 +107,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const bf16* __restrict
 __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restrict__ idx, int S, int top_k, int E,
                                                             int* __restrict__ pos, int* __restrict__ src_tok,
                                                             int* g_count, int* g_row0, int* g_rows, int* g_expert,
-                                                            int max_tiles) {
+                                                            int max_tiles, int tile) {
   // Shared memory: per-warp histograms [32][E] (a warp's atomics only meet its own lanes), then the
   // per-expert totals, row offsets and tile offsets.  One CTA: the whole dispatch of a 2048-token chunk
   // (16384 slots) is ~10 us of shared-memory work; several CTAs would need a grid-wide prefix.
@@ -139,12 +139,12 @@ __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restric
     cnt[e] = run;
   }
   __syncthreads();
-  // exclusive prefixes over experts: rows and 128-row tiles (one warp, E <= 1024)
+  // exclusive prefixes over experts: rows and tiles (one warp, E <= 1024)
   if (warp == 0) {
     int carry_r = 0, carry_t = 0;
     for (int e0 = 0; e0 < E; e0 += 32) {
       const int e = e0 + lane;
-      const int n = e < E ? cnt[e] : 0, nt = (n + 127) >> 7;
+      const int n = e < E ? cnt[e] : 0, nt = (n + tile - 1) / tile;
       int pr = n, pt = nt;
 #pragma unroll
       for (int d = 1; d < 32; d <<= 1) {
@@ -166,10 +166,10 @@ __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restric
   for (int e = tid; e < E; e += 1024) {
     const int n = cnt[e], r0 = off[e];
     int nt = toff[e];
-    for (int i = 0; i < n; i += 128, ++nt) {
+    for (int i = 0; i < n; i += tile, ++nt) {
       if (nt < max_tiles) {
         g_row0[nt] = r0 + i;
-        g_rows[nt] = min(128, n - i);
+        g_rows[nt] = min(tile, n - i);
         g_expert[nt] = e;
       }
     }
@@ -226,14 +226,14 @@ CB_EXPORT int cb_moe_combine_pos(const void* y, const void* w, const void* pos, 
 // experts, scatter (53 us -> with one shared histogram and a serial prefix the CTA spent its time in barriers).
 //   pos[s]      row of slot s in the expert-sorted order, -1 for a slot whose expert is not local
 //   src_tok[r]  token whose activation row goes to sorted row r (0 for the unused rows at the end)
-//   tile list   m-tiles of at most 128 rows that never cross an expert boundary (g_count of them)
+//   tile list   m-tiles of at most `tile` rows that never cross an expert boundary (g_count of them)
 // Rows of one expert are adjacent but in no fixed order among themselves: every output row depends
 // on its own input row only, so the result does not depend on that order.
 // Replaces the reference's moe_dispatch (kernels/moe_dispatch.cu:101, count -> prefix -> scatter).
 CB_EXPORT int cb_moe_dispatch(const void* idx, int64_t S, int64_t top_k, int64_t E, void* pos, void* src_tok,
-                              void* g_count, void* g_row0, void* g_rows, void* g_expert, int64_t max_tiles,
+                              void* g_count, void* g_row0, void* g_rows, void* g_expert, int64_t max_tiles, int64_t tile,
                               void* stream) {
-  if (S < 1 || E < 1 || E > 1024 || top_k < 1 || max_tiles < 1) return CB_ERR_SHAPE;
+  if (S < 1 || E < 1 || E > 1024 || top_k < 1 || max_tiles < 1 || tile < 1) return CB_ERR_SHAPE;
   const size_t smem = (size_t)(32 * E + 3 * E + 2) * sizeof(int);
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(moe_dispatch_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -241,5 +241,5 @@ CB_EXPORT int cb_moe_dispatch(const void* idx, int64_t S, int64_t top_k, int64_t
   }
   return (int)cb_launch(moe_dispatch_kernel, dim3(1), dim3(1024), smem, (cudaStream_t)stream,
                         (const int*)idx, (int)S, (int)top_k, (int)E, (int*)pos, (int*)src_tok, (int*)g_count,
-                        (int*)g_row0, (int*)g_rows, (int*)g_expert, (int)max_tiles);
+                        (int*)g_row0, (int*)g_rows, (int*)g_expert, (int)max_tiles, (int)tile);
 }

@@ -202,6 +202,9 @@ def preset(name: str) -> ModelConfig:
     if "sukisun" in name:
         from .models.sukisun.config import preset_sukisun
         return preset_sukisun(name)
+    if "fasolorn" in name:
+        from .models.fasolorn.config import preset_fasolorn
+        return preset_fasolorn(name)
     if name == "tiny-moe":
         return ModelConfig(name="tiny-moe", num_experts=8, num_experts_per_tok=2,
                            moe_intermediate_size=128, shared_expert_intermediate_size=128,
@@ -253,4 +256,7 @@ def load_config(model_dir: str | Path):
     if str(raw.get("architecture", "")).lower() == "sukisun":
         from .models.sukisun.config import SukisunConfig
         return SukisunConfig.from_hf(raw, name=Path(model_dir).name)
+    if str(raw.get("architecture", "")).lower() == "fasolorn":
+        from .models.fasolorn.config import FasolornConfig
+        return FasolornConfig.from_hf(raw, name=Path(model_dir).name)
     return ModelConfig.from_hf(raw, name=Path(model_dir).name)

@@ -97,6 +97,16 @@ def _ensure_builtin() -> None:
 
     register("sukisun", sukisun)
 
+    def fasolorn(cfg, sd, **kw):
+        from .fasolorn.model import FasolornModel
+        if any(kw.pop(k + "_world", 1) > 1 for k in ("tp", "pp", "ep")):
+            raise NotImplementedError("the Fasolorn family runs on one GPU")
+        for k in ("tp_rank", "pp_rank", "ep_rank"):
+            kw.pop(k, None)
+        return FasolornModel(cfg, sd, **kw)
+
+    register("fasolorn", fasolorn)
+
 
 #: kernel sources a family needs; families without an entry use the whole library
 _KERNELS: dict[str, tuple[str, ...]] = {
@@ -104,10 +114,12 @@ _KERNELS: dict[str, tuple[str, ...]] = {
                  "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
     "sukisun": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "depth.cu", "linrec.cu", "ssd.cu",
                 "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
+    "fasolorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "residual.cu", "routed.cu", "moe.cu",
+                 "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
 }
 
 #: families that also run in 32-bit (``dtype=torch.float32``)
-FLOAT32 = ("zufilorn", "sukisun")
+FLOAT32 = ("zufilorn", "sukisun", "fasolorn")
 
 
 def kernel_sources(arch: str) -> tuple[str, ...] | None:

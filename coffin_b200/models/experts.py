@@ -1,0 +1,63 @@
+"""Routed feed-forward of the row-batch families: squared-relu experts, a corrected choice, identity experts, a shared expert.
+
+The shared expert rides with the routed ones: cut into parts of an expert's width (exact, the activation works on single
+columns), its parts are stored behind the experts and every token holds a slot for each with weight one.  So a step is
+router product, routing, one product for all ups and one for all downs; the weighted sum of the slots happens in the
+residual boundary that follows.
+
+Up to ``UNIT_ROWS`` rows (and in 32-bit mode) an expert's rows go in units of 8 through a GEMV that streams every chosen
+expert once; more rows are sorted by expert for the grouped tcgen05 GEMM.
+"""
+from __future__ import annotations
+
+import torch
+
+from ..ops import kernels as K
+from ..ops import routed as R
+from .rowmodel import RowBatch, pad8, padded
+
+
+class RoutedExperts:
+    def __init__(self, W: dict[str, torch.Tensor], *, experts: int, identity: int, top: int, scale: float, ff: int, shared: int, width: int,
+                 dtype, dev) -> None:
+        """``W``: ``e<i>.up`` / ``e<i>.down``, ``router``, ``correction`` and, with ``shared`` > 0, ``shared.up`` / ``shared.down``."""
+        parts = -(-shared // ff)
+        self.r = R.Router(experts, identity, top, scale, parts)
+        I, W8 = pad8(ff), pad8(width)
+        self.up = torch.zeros(experts + parts, I, W8, dtype=dtype, device=dev)
+        self.down = torch.zeros(experts + parts, W8, I, dtype=dtype, device=dev)
+        for e in range(experts):
+            self.up[e, :ff, :width], self.down[e, :width, :ff] = W[f"e{e}.up"].to(dev, dtype), W[f"e{e}.down"].to(dev, dtype)
+        for p in range(parts):
+            a, b = p * ff, min(shared, (p + 1) * ff)
+            self.up[experts + p, :b - a, :width] = W["shared.up"][a:b].to(dev, dtype)
+            self.down[experts + p, :width, :b - a] = W["shared.down"][:, a:b].to(dev, dtype)
+        self.router = padded(W["router"], pad8(experts + identity), W8, dtype, dev)
+        self.correction = W["correction"].to(dev, torch.float32).contiguous()
+
+    def weights(self) -> list[torch.Tensor]:
+        """What a step of one token streams."""
+        n = self.r.slots
+        return [self.router, self.up[:n], self.down[:n]]
+
+    def run(self, model, b: RowBatch, h: torch.Tensor) -> dict:
+        """Keywords of the ``residual_step`` that merges the result."""
+        r, T, I, W8 = self.r, b.T, self.up.shape[1], self.up.shape[2]
+        S = T * r.slots
+        logits = model.linear(self.router, h, model.buf("route_z", T, self.router.shape[0], torch.float32))
+        idx, w = model.buf("route_i", T, r.slots, torch.int32), model.buf("route_w", T, r.slots, torch.float32)
+        idw = model.buf("route_id", T, 1, torch.float32)
+        units = T <= R.UNIT_ROWS
+        if units:
+            disp = R.route_units(r, logits, self.correction, b.positions, idx, w, idw, model.buf("route_u", 1, R.meta_size(r, T), torch.int32)[0])
+        else:
+            R.route(r, logits, self.correction, b.positions, idx, w, idw)
+            disp = K.moe_dispatch(idx, r.stored, R.UNIT if model.f32 else 128)
+        inter, y = model.buf("route_h", S, I), model.buf("route_y", S, W8)
+        if units or model.f32:
+            R.unit_linear(self.up, h, inter, disp, rows=T, gather=True, relu2=True)
+            R.unit_linear(self.down, inter, y, disp, rows=T, gather=False)
+        else:
+            K.gemm_grouped(h.index_select(0, disp["src_tok"]), self.up, disp, out=inter, relu2=True)
+            K.gemm_grouped(inter, self.down, disp, out=y)
+        return {"experts": (y, disp["pos"], w, idw if r.identity else None, h)}

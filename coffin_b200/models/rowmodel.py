@@ -37,24 +37,30 @@ class RowBatch:
     max_rows: int = 1               # longest segment
     max_len: int = 0                # largest position + 1 (0: unknown, inside a graph)
     pre_lens: tuple = ()            # tokens of every leading segment's sequence so far, its own rows included
+    pre_pos: tuple = ()             # position of every leading segment's first row
     cache: dict = dataclasses.field(default_factory=dict)     # what mixers of one forward share
 
-    def expansion(self):
-        """Whole-page rows of the leading segments side by side: ``(first row, length, tables of consecutive blocks)`` per
-        segment on the device, the total number of rows and the most pages of a segment."""
-        e = self.cache.get("expansion")
+    def expansion(self, window: int = 0) -> dict:
+        """Whole-page rows of the leading segments side by side, from the first page that a query of the segment sees through
+        ``window`` (0: all).  Per segment on the device: ``base`` (first row), ``lens``, ``skip`` (pages left out), ``pos`` (the
+        segment's first position counted from the first row), ``tables`` of consecutive blocks; ``rows``: all rows, ``pages``: the
+        most of a segment."""
+        e = self.cache.get(("expansion", window))
         if e is None:
-            pages = [(n + K.BLOCK - 1) // K.BLOCK for n in self.pre_lens]
+            skip = [max(0, p - window + 1) // K.BLOCK if window else 0 for p in self.pre_pos]
+            lens = [n - s * K.BLOCK for n, s in zip(self.pre_lens, skip)]
+            pages = [(n + K.BLOCK - 1) // K.BLOCK for n in lens]
             first = [sum(pages[:i]) for i in range(len(pages))]
-            host = torch.zeros(len(pages), 2 + max(pages), dtype=torch.int32)
-            for i, (p, f, n) in enumerate(zip(pages, first, self.pre_lens)):
-                host[i, 0], host[i, 1] = f * K.BLOCK, n
-                host[i, 2:2 + p] = torch.arange(f, f + p, dtype=torch.int32)
+            n, most = len(pages), max(pages)
+            host = torch.zeros(4 * n + n * most, dtype=torch.int32)
+            for i, (p, f) in enumerate(zip(pages, first)):
+                host[i], host[n + i], host[2 * n + i], host[3 * n + i] = f * K.BLOCK, lens[i], skip[i], self.pre_pos[i] - skip[i] * K.BLOCK
+                host[4 * n + i * most:4 * n + i * most + p] = torch.arange(f, f + p, dtype=torch.int32)
             if self.positions.is_cuda:
                 host = host.pin_memory()
             dev = host.to(self.positions.device, non_blocking=True)
-            base_len = dev[:, :2].t().contiguous()
-            e = self.cache["expansion"] = (base_len[0], base_len[1], dev[:, 2:], sum(pages) * K.BLOCK, max(pages))
+            e = self.cache[("expansion", window)] = {"base": dev[:n], "lens": dev[n:2 * n], "skip": dev[2 * n:3 * n], "pos": dev[3 * n:4 * n],
+                                                     "tables": dev[4 * n:].view(n, most), "rows": sum(pages) * K.BLOCK, "pages": most}
         return e
 
 
@@ -240,18 +246,46 @@ class RowModel:
             return X.gemm_f32out(x, W, out)
         return K.gemm(x, W, out=out)
 
-    def project(self, P, h: torch.Tensor, b: RowBatch) -> tuple[torch.Tensor, torch.Tensor]:
+    def project(self, P, h: torch.Tensor, b: RowBatch, name: str = "proj") -> tuple[torch.Tensor, torch.Tensor]:
         """``(main, gates)`` of an input projection, one product: fp32 for few rows (and in 32-bit mode), else the main columns
-        in the activation type and the gate columns fp32."""
+        in the activation type and the gate columns fp32.  ``name``: workspace of the rows, for rows that outlive the layer."""
         T = b.T
         if self.f32 or T <= 8:
-            y = self.buf("proj32", T, P.n, torch.float32)
+            y = self.buf(name + "32", T, P.n, torch.float32)
             self.linear(P.w, h, y)
             return y[:, :P.n_main], y[:, P.n_main:]
-        main = self.buf("proj", T, P.n_main)
+        main = self.buf(name, T, P.n_main)
+        if P.n == P.n_main:
+            return self.linear(P.w, h, main), main[:, P.n_main:]
         gates = self.buf("gates", T, P.gate.shape[0], torch.float32)
         X.gemm_mixed(h, P.w, main, gates)
         return main, gates
+
+    def feed_forward(self, L, h: torch.Tensor, T: int) -> torch.Tensor:
+        """``w_down (silu(gate) * up)`` of a layer with ``w_gu`` (gate rows, then up rows) and ``w_down``."""
+        I = L.w_down.shape[1]
+        inter = self.buf("inter", T, I)
+        y = self.buf("y", T, L.w_down.shape[0])
+        if self.f32:
+            X.swiglu_f32(X.gemm_f32(h, L.w_gu, self.buf("gu", T, 2 * I)), inter)
+        elif T <= 8 and T * h.shape[1] * 2 <= 160 * 1024:
+            K.gemv(L.w_gu, h, inter, swiglu=True)
+        elif K.PAIR_GEMM and T >= K.PAIR_MIN_ROWS and I >= 128:
+            K.gemm_swiglu(h, L.w_gu, out=inter)
+        else:
+            K.swiglu(K.gemm(h, L.w_gu, out=self.buf("gu", T, 2 * I)), out=inter)
+        return self.linear(L.w_down, inter, y)
+
+    def angles(self, b: RowBatch, base: float, dims: int, turns: torch.Tensor) -> torch.Tensor:
+        """(cos, sin) of the batch's rows, shared by the layers of one rotation."""
+        key = ("rope", base, dims)
+        cs = b.cache.get(key)
+        if cs is None:
+            cs = self.buf(f"rope{base}/{dims}", b.T, max(2, dims), torch.float32)
+            if dims:
+                X.rope_rows(b.positions, turns, cs)
+            b.cache[key] = cs
+        return cs
 
     # ------------------------------------------------------------------ mixer cores
     def recur(self, core: X.Linrec, b: RowBatch, proj, gates, og, act, dec) -> None:
@@ -324,6 +358,7 @@ class RowModel:
                      positions=dev[:T], row_seg=dev[T:2 * T], seg_row=dev[o:o + n_seg + 1], seg_pos=dev[o + n_seg + 1:o + 2 * n_seg + 1],
                      seg_slot=dev[o + 2 * n_seg + 1:o + 3 * n_seg + 1], tables=dev[o + 3 * n_seg + 1:].view(n_seg, pages),
                      pre_lens=tuple(int(items[i][1]) + len(toks[i]) for i in order[:n_pre]),
+                     pre_pos=tuple(int(items[i][1]) for i in order[:n_pre]),
                      max_rows=max(len(t) for t in toks), max_len=max(int(it[1]) + len(t) for it, t in zip(items, toks)))
         return b, order, first
 

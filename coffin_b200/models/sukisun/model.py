@@ -20,9 +20,10 @@ import torch.nn.functional as F
 
 from ...ops import kernels as K
 from ...ops import mixers as X
+from ..latent import LatentAttention
 from ..rowmodel import RowBatch, RowModel, pad8, padded
 from .config import LATENT, SukisunConfig
-from .mixers import LatentAttention, Mamba2
+from .mixers import Mamba2
 
 
 @dataclasses.dataclass

@@ -81,20 +81,6 @@ class ZufilornModel(RowModel):
         self.head = padded(take("head"), pad8(c.vocab_size), pad8(W), dtype, dev)
 
     # ------------------------------------------------------------------ sublayers
-    def feed_forward(self, L: _Layer, h: torch.Tensor, T: int) -> torch.Tensor:
-        I = L.w_down.shape[1]
-        inter = self.buf("inter", T, I)
-        y = self.buf("y", T, L.w_down.shape[0])
-        if self.f32:
-            X.swiglu_f32(X.gemm_f32(h, L.w_gu, self.buf("gu", T, 2 * I)), inter)
-        elif T <= 8 and T * h.shape[1] * 2 <= 160 * 1024:
-            K.gemv(L.w_gu, h, inter, swiglu=True)
-        elif K.PAIR_GEMM and T >= K.PAIR_MIN_ROWS and I >= 128:
-            K.gemm_swiglu(h, L.w_gu, out=inter)
-        else:
-            K.swiglu(K.gemm(h, L.w_gu, out=self.buf("gu", T, 2 * I)), out=inter)
-        return self.linear(L.w_down, inter, y)
-
     def attend(self, core: X.AttnMaps, b: RowBatch, proj, gates, act, *, lam: float, post_scale: float) -> None:
         vh, T, P = core.H * core.maps, b.T, b.pre_rows
         fin = dict(lam=lam, post_scale=post_scale, eps=self.eps)

@@ -393,36 +393,36 @@ def w4_dequant(Wq: torch.Tensor, wscale: torch.Tensor, out: torch.Tensor | None 
     return out
 
 
-def moe_dispatch(idx: torch.Tensor, n_experts: int) -> dict:
+def moe_dispatch(idx: torch.Tensor, n_experts: int, tile: int = 128) -> dict:
     """Expert-major order of the routed slots ``idx [T, k]`` (local expert id, or < 0 for a slot of
     another rank), computed on the device: ``pos [T*k]`` (sorted row of a slot, -1 = none),
     ``src_tok [T*k]`` (token feeding sorted row r) and the m-tile list consumed by
-    :func:`gemm_grouped`.  No count is read back to the host."""
+    :func:`gemm_grouped` (tiles of at most ``tile`` rows of one expert).  No count is read back to the host."""
     T, k = idx.shape
     S = T * k
     dev = idx.device
-    max_tiles = (S + 127) // 128 + n_experts
+    max_tiles = (S + tile - 1) // tile + n_experts
     meta = torch.empty(1 + 3 * max_tiles, dtype=torch.int32, device=dev)
     d = {"pos": torch.empty(S, dtype=torch.int32, device=dev),
          "src_tok": torch.empty(S, dtype=torch.int32, device=dev),
          "count": meta[:1], "row0": meta[1:1 + max_tiles], "rows": meta[1 + max_tiles:1 + 2 * max_tiles],
          "expert": meta[1 + 2 * max_tiles:], "max_tiles": max_tiles, "meta": meta}
     call("moe_dispatch", idx, S, k, n_experts, d["pos"], d["src_tok"], d["count"], d["row0"], d["rows"], d["expert"],
-         max_tiles)
+         max_tiles, tile)
     _count()
     return d
 
 
-def gemm_grouped(A: torch.Tensor, W: torch.Tensor, disp: dict, out: torch.Tensor | None = None) -> torch.Tensor:
+def gemm_grouped(A: torch.Tensor, W: torch.Tensor, disp: dict, out: torch.Tensor | None = None, relu2: bool = False) -> torch.Tensor:
     """``out[r] = A[r] @ W[expert(r)].T`` for expert-sorted rows ``A [S, K]`` and a weight stack
     ``W [E, N, K]`` (bf16), tiles taken from ``disp`` (:func:`moe_dispatch`).  Rows outside the tile
-    list (slots of other ranks) are left untouched."""
+    list (slots of other ranks) are left untouched.  ``relu2``: squared relu in the epilogue."""
     S, Kd = A.shape
     E, N, _ = W.shape
     if out is None:
         out = torch.empty(S, N, dtype=torch.bfloat16, device=A.device)
     call("gemm_bf16_grouped", A, A.stride(0), W, W.stride(1), out, out.stride(0), S, E, N, Kd, disp["count"],
-         disp["row0"], disp["rows"], disp["expert"], disp["max_tiles"], status_word(A.device))
+         disp["row0"], disp["rows"], disp["expert"], disp["max_tiles"], 2 if relu2 else 0, status_word(A.device))
     _count()
     return out
 

@@ -8,10 +8,11 @@ base) is an argument, so a model family picks what it needs:
 * ``depth_embed`` / ``depth_step``: a residual that becomes a weighted sum of all layer results after every layer;
 * ``Linrec``: recurrences with a matrix state - the per-channel gated delta rule, the mLSTM matrix memory and the
   state space with scalar decays (Mamba-2); ``gated_norm``: its output gate and grouped RMS norm;
-* ``AttnMaps``: paged attention with several score maps per head over the same values, capped scores and a
-  position-dependent query temperature;
+* ``AttnMaps``: paged attention with several score maps per head over the same values, capped scores, a
+  position-dependent query temperature, a sliding window, sinks, rotary positions, mixed values and gates per element;
 * ``LatentAttn``: attention over cached low-rank latents with a rotated key part shared by all heads; ``rope_rows`` /
   ``rope_heads``: rotary angles of a batch and interleaved rotation of head parts;
+* ``residual_embed`` / ``residual_step``: a plain fp32 residual whose boundaries also merge expert rows;
 * ``gemm_f32out`` / ``gemm_f32``: projections whose result (or everything) stays fp32; ``linear_xielu``: a projection
   with xIELU in its epilogue.
 """
@@ -123,6 +124,32 @@ def streams_step(x: torch.Tensor, h: torch.Tensor | None, *, gain: torch.Tensor 
     t = h if h is not None else y
     call("streams_step", x, y, y.stride(0) if y is not None else 0, mix, write, read, gain, h, h.stride(0) if h is not None else 0,
          rows, n, S, W, float(eps), int(store), _is_f32(t))
+    K._count()
+    return h
+
+
+# ------------------------------------------------------------------ plain residual
+def residual_embed(embed: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, scale: float) -> torch.Tensor:
+    """``x [T, W]`` (fp32) = ``embed[token] * scale``."""
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and embed.is_contiguous() and tokens.dtype == torch.int64
+    call("residual_embed", embed, tokens, x, T, W, embed.shape[0], float(scale), _is_f32(embed))
+    K._count()
+    return x
+
+
+def residual_step(x: torch.Tensor, h: torch.Tensor | None, *, gain: torch.Tensor | None = None, y: torch.Tensor | None = None,
+                  experts: tuple | None = None, rows: torch.Tensor | None = None, store: bool = True, eps: float = 1e-5) -> torch.Tensor | None:
+    """Boundary between two sublayers: ``x [T, W] += y``, or with ``experts = (ys, pos, w, idw, hin)`` the weighted expert rows
+    ``sum_j w[t, j] ys[pos[t, j]] + idw[t] hin[t]``; then ``h = rmsnorm(x) * gain``.  ``rows`` picks the residual rows behind the rows
+    of ``h`` (with ``store=False``)."""
+    T, W = x.shape
+    n = rows.numel() if rows is not None else (h.shape[0] if h is not None else T)
+    ys, pos, w, idw, hin = experts if experts is not None else (None,) * 5
+    t = next((v for v in (h, y, ys) if v is not None), None)
+    ld = lambda v: v.stride(0) if v is not None else 0
+    call("residual_step", x, y, ld(y), ys, ld(ys), pos, w, w.shape[1] if w is not None else 0, idw, hin, ld(hin), gain, h, ld(h), rows, n, W,
+         float(eps), int(store), _is_f32(t) if t is not None else 0)
     K._count()
     return h
 
@@ -278,18 +305,28 @@ class _AttnStruct(ctypes.Structure):
     _fields_ = [("proj", _P), ("ldp", _I64), ("k_col", _I64), ("v_col", _I64), ("kpool", _P), ("vpool", _P), ("tables", _P),
                 ("ldbt", _I64), ("row_seg", _P), ("positions", _P), ("seg_row", _P), ("seg_pos", _P), ("part_o", _P), ("part_ml", _P),
                 ("H", _I32), ("G", _I32), ("maps", _I32), ("dim", _I32), ("vdim", _I32), ("nsplit", _I32), ("scale", _F), ("cap", _F),
-                ("temp_coef", _F), ("temp_every", _I32), ("ldk", _I64), ("ldv", _I64), ("act", _P), ("lda", _I64), ("gates", _P), ("ldg", _I64)]
+                ("temp_coef", _F), ("temp_every", _I32), ("ldk", _I64), ("ldv", _I64), ("act", _P), ("lda", _I64), ("gates", _P), ("ldg", _I64),
+                ("window", _I32), ("rot_half", _I32), ("sink", _P), ("cs", _P), ("v0", _P), ("ldv0", _I64), ("v_own", _F), ("v_mix", _F),
+                ("egate", _P), ("lde", _I64)]
 
 
 MAX_VDIM = 512
+
+
+def window_pages(window: int) -> int:
+    """Most pages that hold keys of one query."""
+    return (window + K.BLOCK - 2) // K.BLOCK + 1 if window > 0 else 1 << 30
 
 
 class AttnMaps:
     """Attention layer constants plus its pages ``kpool [slots, G * maps, dim]``, ``vpool [slots, G, vdim]``."""
 
     def __init__(self, *, H: int, G: int, maps: int, dim: int, vdim: int, k_col: int, v_col: int, scale: float, cap: float | None,
-                 temp: tuple[float, int] | None, kpool: torch.Tensor, vpool: torch.Tensor, finish: bool = True) -> None:
-        """``finish``: the heads will be finished by ``finish``, which bounds the value size."""
+                 temp: tuple[float, int] | None, kpool: torch.Tensor, vpool: torch.Tensor, finish: bool = True, window: int = 0,
+                 rot_dims: int = 0, sink: torch.Tensor | None = None) -> None:
+        """``finish``: the heads will be finished by ``finish``, which bounds the value size.  ``window``: tokens a query sees,
+        itself included (0: all).  ``rot_dims``: leading columns of queries and keys that turn, in neighbouring pairs, by the
+        angles of ``rows_of``.  ``sink`` (fp32 ``[H * maps]``): a score without key or value in every softmax."""
         if (finish and vdim > MAX_VDIM) or maps not in (1, 2):
             raise ValueError(f"attention with {maps} maps and values of {vdim} is outside the kernels' range")
         a = self.a = _AttnStruct()
@@ -300,6 +337,8 @@ class AttnMaps:
         a.scale, a.cap = float(scale), float(cap or 0.0)
         self.set_pools(kpool, vpool)
         self._tcgen05 = bool(_lib.call_nostream("attn_maps_flash_tc_ok", dim, vdim))
+        a.window, a.rot_half, a.sink = int(window), rot_dims // 2, _ptr(sink)
+        self.window, self.sink, self._egate = int(window), sink, None
         if temp is not None:
             a.temp_coef, a.temp_every = float(temp[0]), int(temp[1])
 
@@ -315,9 +354,20 @@ class AttnMaps:
         a.positions, a.row_seg, a.part_o, a.part_ml, a.nsplit = positions.data_ptr(), _ptr(row_seg), _ptr(part_o), _ptr(part_ml), nsplit
         a.seg_row, a.seg_pos = _ptr(seg_row), _ptr(seg_pos)
 
-    def append(self, proj, tables, positions, row_seg=None) -> None:
+    def rows_of(self, cs: torch.Tensor | None = None, egate: torch.Tensor | None = None, values: torch.Tensor | None = None,
+                lam: float = 0.0) -> None:
+        """What the rows of the next calls carry beside their projection: angles ``cs [rows, rot_dims]``, output gate
+        pre-activations ``egate [rows, H * vdim]`` (one map), and ``values [rows, G * vdim]`` of another layer, of which
+        ``lam`` is mixed into their own (both typed like the projection)."""
+        a = self.a
+        a.cs, a.egate, a.lde = _ptr(cs), _ptr(egate), egate.stride(0) if egate is not None else 0
+        a.v0, a.ldv0, a.v_own, a.v_mix = _ptr(values), values.stride(0) if values is not None else 0, 1.0 - lam, lam
+        self._egate = egate
+
+    def append(self, proj, tables, positions, row_seg=None, turn_queries: bool = False) -> None:
+        """Keys (turned) and values (mixed) into the pages; ``turn_queries``: the rows' queries are turned in place."""
         self._fill(proj, tables, positions, row_seg)
-        call("attn_maps_append", ctypes.byref(self.a), positions.numel(), _is_f32(proj), _is_f32(self.kpool))
+        call("attn_maps_append", ctypes.byref(self.a), positions.numel(), int(turn_queries), _is_f32(proj), _is_f32(self.kpool))
         K._count()
 
     def rows(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int = 1) -> None:
@@ -348,7 +398,7 @@ class AttnMaps:
     def decode_splits(self, rows: int) -> int:
         R = self.H // self.G
         hpc = min(R, 8 // self.maps)
-        return max(1, min(64, 148 // max(1, self.G * -(-R // hpc) * rows)))
+        return max(1, min(64, window_pages(self.window), 148 // max(1, self.G * -(-R // hpc) * rows)))
 
     def decode(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
         """Single tokens (their keys and values are appended by the kernel): ``nsplit`` key splits per row."""
@@ -358,9 +408,12 @@ class AttnMaps:
 
     def finish(self, part_o, part_ml, gates, act, positions, *, nsplit: int = 1, lam: float = 0.0, post_scale: float = 1.0,
                eps: float = 1e-5) -> None:
-        """Merge splits, ``o = a_0 - lam a_1`` + RMS norm (two maps), ``* post_scale * sigmoid(gate)`` per head."""
+        """Merge splits and sinks, ``o = a_0 - lam a_1`` + RMS norm (two maps), ``* post_scale * sigmoid(gate)`` per head, then per
+        element (``rows_of``)."""
+        eg = self._egate
         call("attn_maps_finish", part_o, part_ml, gates, gates.stride(0) if gates is not None else 0, act, act.stride(0), positions,
-             positions.numel(), self.H, self.maps, self.vdim, nsplit, float(lam), float(post_scale), float(eps), _is_f32(act))
+             positions.numel(), self.H, self.maps, self.vdim, nsplit, float(lam), float(post_scale), float(eps), self.sink,
+             eg, eg.stride(0) if eg is not None else 0, _is_f32(eg) if eg is not None else 0, _is_f32(act))
         K._count()
 
 
@@ -390,7 +443,8 @@ def rope_heads(src: torch.Tensor, hs: int, dst: torch.Tensor, hd: int, cs: torch
 class _LatentStruct(ctypes.Structure):
     _fields_ = [("proj", _P), ("ldp", _I64), ("c_col", _I64), ("r_col", _I64), ("norm_q", _P), ("norm_c", _P), ("cq", _P), ("ldq", _I64),
                 ("pool", _P), ("ldk", _I64), ("tables", _P), ("ldbt", _I64), ("row_seg", _P), ("positions", _P), ("cs", _P), ("half", _I32),
-                ("q_rank", _I32), ("kv_rank", _I32), ("rot", _I32), ("cp", _I32), ("eps", _F)]
+                ("q_rank", _I32), ("kv_rank", _I32), ("rot", _I32), ("cp", _I32), ("eps", _F), ("H", _I32), ("split", _I32), ("hq", _I64),
+                ("r_off", _I64), ("qa", _P), ("ldqa", _I64)]
 
 
 def head_linear(w: torch.Tensor, x: torch.Tensor, hx: int, y: torch.Tensor, hy: int, gate: torch.Tensor | None = None) -> torch.Tensor:
@@ -404,10 +458,12 @@ def head_linear(w: torch.Tensor, x: torch.Tensor, hx: int, y: torch.Tensor, hy: 
 
 class LatentAttn:
     """Latent attention of one layer: pages ``pool [slots, ldk]`` hold ``[c | rotated key part]`` (the part at column ``cp``),
-    its own or those of the layer it borrows them from."""
+    its own or those of the layer it borrows them from.  ``q_rank`` 0: the projection rows hold the queries themselves, heads of
+    ``hq`` columns whose rotated part starts at ``r_off``.  ``window``: tokens a query sees, itself included (0: all)."""
 
     def __init__(self, *, H: int, q_rank: int, kv_rank: int, rot: int, rot_dims: int, cp: int, scale: float, eps: float, pool: torch.Tensor,
-                 norm_q: torch.Tensor, norm_c: torch.Tensor | None, c_col: int = 0, r_col: int = 0) -> None:
+                 norm_q: torch.Tensor | None, norm_c: torch.Tensor | None, c_col: int = 0, r_col: int = 0, hq: int = 0, r_off: int = 0,
+                 window: int = 0) -> None:
         a = self.a = _LatentStruct()
         size = _lib.call_nostream("latent_args_size")
         assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
@@ -415,22 +471,26 @@ class LatentAttn:
         self._keep = (norm_q, norm_c)
         a.q_rank, a.kv_rank, a.rot, a.cp, a.eps, a.half, a.c_col, a.r_col = q_rank, kv_rank, rot, cp, float(eps), rot_dims // 2, c_col, r_col
         a.norm_q, a.norm_c, a.pool, a.ldk = _ptr(norm_q), _ptr(norm_c), _ptr(pool), pool.stride(0)
+        a.H, a.hq, a.r_off, self.window = H, hq, r_off, int(window)
         # the plain kernel and the merge of key splits see one key / value head whose values are the head of the key row
         self._plain = AttnMaps(H=H, G=1, maps=1, dim=self.ldk, vdim=cp, k_col=0, v_col=0, scale=scale, cap=None, temp=None, kpool=pool,
-                               vpool=pool, finish=False)
+                               vpool=pool, finish=False, window=window)
         self.tc = pool.dtype == torch.bfloat16 and bool(_lib.call_nostream("latent_decode_ok", self.ldk, cp))
 
-    def rows(self, proj, cq, tables, positions, row_seg, cs) -> None:
-        """Norm the query latents into ``cq``; an owner also norms, rotates and appends what it caches."""
+    def rows(self, proj, cq, tables, positions, row_seg, cs, *, split: int = 0, qa: torch.Tensor | None = None) -> None:
+        """Norm the query latents into ``cq``; without them turn the rotated query parts, in place for the rows before ``split`` and
+        into the absorbed queries ``qa`` of the others.  An owner also norms, rotates and appends what it caches."""
         a = self.a
-        a.proj, a.ldp, a.cq, a.ldq = proj.data_ptr(), proj.stride(0), cq.data_ptr(), cq.stride(0)
+        a.proj, a.ldp, a.cq, a.ldq = proj.data_ptr(), proj.stride(0), _ptr(cq), cq.stride(0) if cq is not None else 0
+        a.split, a.qa, a.ldqa = split, _ptr(qa), qa.stride(0) if qa is not None else 0
         a.tables, a.ldbt, a.row_seg, a.positions, a.cs = tables.data_ptr(), tables.stride(0), _ptr(row_seg), positions.data_ptr(), _ptr(cs)
-        call("latent_rows", ctypes.byref(a), positions.numel(), int(self.own), _is_f32(proj), _is_f32(cq))
+        call("latent_rows", ctypes.byref(a), positions.numel(), int(self.own), _is_f32(proj), _is_f32(self.pool))
         K._count()
 
-    def gather(self, tables, base, lens, out, *, segs: int, max_pages: int) -> None:
-        """Page rows of ``segs`` sequences side by side in ``out`` (segment ``s`` from row ``base[s]``)."""
-        call("latent_gather", self.pool, self.pool.stride(0) * self.pool.element_size(), tables, tables.stride(0), base, lens, out, segs, max_pages)
+    def gather(self, tables, base, lens, first, out, *, segs: int, max_pages: int) -> None:
+        """Page rows of ``segs`` sequences side by side in ``out`` (segment ``s`` from row ``base[s]``, its pages from ``first[s]`` on)."""
+        call("latent_gather", self.pool, self.pool.stride(0) * self.pool.element_size(), tables, tables.stride(0), base, lens, first, out, segs,
+             max_pages)
         K._count()
 
     def _tiles(self, rows: int) -> int:
@@ -439,13 +499,13 @@ class LatentAttn:
 
     def decode_splits(self, rows: int) -> int:
         groups = -(-self.H // (16 * self._tiles(rows)))
-        return max(1, min(64, 148 // max(1, groups * rows)))
+        return max(1, min(64, window_pages(self.window), 148 // max(1, groups * rows)))
 
     def absorbed(self, q, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
         """Queries ``q [rows, H * ldk]`` against the pages: key splits for ``merge`` (one split without the tensor-core kernel)."""
         if self.tc:
             call("latent_decode", q, q.stride(0), self.pool, self.pool.stride(0), tables, tables.stride(0), row_seg, positions, part_o, part_ml,
-                 positions.numel(), self.H, self.cp, nsplit, self._tiles(positions.numel()), self.scale)
+                 positions.numel(), self.H, self.cp, nsplit, self._tiles(positions.numel()), self.window, self.scale)
             K._count()
         else:
             self._plain.rows(q, tables, positions, row_seg, part_o, part_ml, nsplit)

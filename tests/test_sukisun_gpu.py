@@ -300,7 +300,7 @@ def test_prompt_attention_kernels_agree(sizes):
 
 
 def test_absorbed_and_expanded_forms_agree(monkeypatch):
-    from coffin_b200.models.sukisun import mixers as M
+    from coffin_b200.models import latent as M
     layer = S.latent(4, 32, 16, 48, 96, 64, scale=0.5)
     a, ref = mixer_pair(layer, BF16, 150, [70, 80])
     monkeypatch.setattr(M, "ABSORB_ROWS", 10 ** 9)

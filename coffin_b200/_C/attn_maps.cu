@@ -353,7 +353,8 @@ CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const
   const ElemGate eg = {egate, lde, (int)e_f32};
   if (vdim > 32 * kVMax || nsplit > 64) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
-  if (nsplit > 4) {
+  // a CTA per head, where there are many splits to walk or few heads to fill the machine with
+  if (nsplit > 4 || (nsplit > 1 && maps == 1 && rows * H <= 512)) {
     if (rows > 65535) return CB_ERR_SHAPE;
     const size_t smem = sizeof(float) * (size_t)(kWT / 32) * vdim;
     const dim3 wide((unsigned)H, (unsigned)rows);

@@ -257,8 +257,9 @@ int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
 // weighted sums are mma products with the query vectors as rows: eight of the sixteen rows are enough, so the second
 // product takes the bf16 heads of the weights in rows 0-7 and their remainders in rows 8-15.
 constexpr int kDT = 256;
+constexpr int decode_ctas(int dk, int dv, int maps) { return maps == 1 && dk <= 128 && dv <= 128 ? 2 : 1; }    // per SM
 template <int DK, int DV, int MAPS, typename TP>
-__global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
+__global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
   constexpr int LK = DK + 8, LV = DV + 8, KPAGE = MAPS * kPage * LK, VPAGE = kPage * LV, NP = DV / 16, NPW = (NP + 7) / 8;
   extern __shared__ __align__(128) unsigned char smem[];
   bf16* ks = reinterpret_cast<bf16*>(smem);            // [2][MAPS][kPage][LK]
@@ -407,6 +408,26 @@ __global__ void __launch_bounds__(kDT, 1) maps_decode_kernel(const AttnMapsArgs 
     }
     __syncthreads();
   }
+  if (MAPS == 1 && a.act) {                            // the only split: the heads are finished here
+    if (warp < nq && lane == 0) w_s[warp] = 1.f / (l_run + (a.sink ? ex2(a.sink[g * R + r0 + warp] * kLog2e - m_run) : 0.f));
+    __syncthreads();
+    if (g4 >= nq) return;
+    const float inv = w_s[g4];
+    const int hc = (g * R + r0 + g4) * a.vdim;
+    bf16* out = reinterpret_cast<bf16*>(a.act) + (int64_t)row * a.lda + hc;
+    const TP* eg = a.egate ? reinterpret_cast<const TP*>(a.egate) + (int64_t)row * a.lde + hc : nullptr;
+#pragma unroll
+    for (int i = 0; i < NPW; ++i)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int c = (warp + 8 * i) * 16 + j * 8 + t4 * 2;
+        if (warp + 8 * i >= NP || c >= a.vdim) continue;
+        float x = (o[i][j][0] + o[i][j][2]) * inv, y = (o[i][j][1] + o[i][j][3]) * inv;
+        if (eg) { x *= sigmoid_x(act_load(eg + c)); y *= sigmoid_x(act_load(eg + c + 1)); }
+        *reinterpret_cast<uint32_t*>(out + c) = pack_bf162(x, y);
+      }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < NPW; ++i)
 #pragma unroll
@@ -470,11 +491,13 @@ CB_EXPORT int cb_attn_maps_flash(const void* args, int64_t segs, int64_t max_row
   return flash_dv<256>(a, tiles, (int)segs, st);
 }
 
-// Decode attention of `rows` single tokens (appends their keys and values): splits of every row into part_o / part_ml.
+// Decode attention of `rows` single tokens (appends their keys and values): splits of every row into part_o / part_ml, or with
+// one split of one map the finished heads into act.
 CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32, void* stream) {
   if (!args || rows < 1 || rows > 65535) return CB_ERR_ARG;
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
-  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || !a.part_o || !a.part_ml || a.H < 1 || a.G < 1 || a.H % a.G ||
+  if (a.act ? a.maps != 1 || a.nsplit != 1 || a.lda % 2 : !a.part_o || !a.part_ml) return CB_ERR_ARG;
+  if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || a.H < 1 || a.G < 1 || a.H % a.G ||
       a.nsplit < 1 || a.nsplit > 64 || 2 * a.rot_half > a.dim || (a.rot_half && !a.cs))
     return CB_ERR_ARG;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;

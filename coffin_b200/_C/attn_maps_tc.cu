@@ -47,22 +47,26 @@ __device__ __forceinline__ float rcp(float x) {
   return y;
 }
 
+// Buffers of scores and of weights.  Heads up to 128 keep one of each: two CTAs then fit an SM and cover each other's waits (a
+// tile's scores are computed while the softmax of the tile before it, already in registers, goes on).
+constexpr int buffers(int dk, int dv) { return dk <= 128 && dv <= 128 ? 1 : 2; }
 template <int DK, int DV, int MODE, int STAGES>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kThreads, 3 - buffers(DK, DV))
 maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnMapsArgs a, int* status) {
   constexpr int NK = DK / 64, NV = DV / 64;           // 64-element (128-byte) chunks
   constexpr int K_BYTES = kBKV * DK * 2, V_BYTES = kBKV * DV * 2, P_BYTES = kBQ * kBKV * 2;
   constexpr int KC = kBKV * 128;                      // bytes of one chunk block of a page
-  constexpr uint32_t TMEM_COLS = 2 * kBKV + DV + DK / 2 <= 256 ? 256 : 512;
-  static_assert(2 * kBKV + DV + DK / 2 <= 512, "tensor memory");
+  constexpr int NB = buffers(DK, DV);
+  constexpr uint32_t TMEM_COLS = NB * kBKV + DV + DK / 2 <= 256 ? 256 : 512;
+  static_assert(NB * kBKV + DV + DK / 2 <= 512 && (NB == 2 || TMEM_COLS == 256), "tensor memory");
   constexpr uint32_t IDESC_S = umma_idesc(kBQ, kBKV, 1, 1);
   constexpr uint32_t IDESC_O = umma_idesc(kBQ, DV, 1, 1) | (1u << 16);     // B operand MN-major
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* Ks = base;                           // [STAGES][K_BYTES]
   unsigned char* Vs = Ks + STAGES * K_BYTES;          // [STAGES][V_BYTES]
-  unsigned char* Ps = Vs + STAGES * V_BYTES;          // [2][head | remainder]
-  __shared__ uint64_t q_full, k_full[STAGES], v_full[STAGES], k_free[STAGES], v_free[STAGES], s_full[2], s_free[2], p_full[2], p_free[2],
+  unsigned char* Ps = Vs + STAGES * V_BYTES;          // [NB][head | remainder]
+  __shared__ uint64_t q_full, k_full[STAGES], v_full[STAGES], k_free[STAGES], v_free[STAGES], s_full[NB], s_free[NB], p_full[NB], p_free[NB],
       o_full, pair_bar[4];
   __shared__ float xch[2][2][kBQ];                    // [tile parity][column half][row]: maxima of half rows
   __shared__ uint32_t tmem_base_s;
@@ -86,7 +90,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     for (int i = 0; i < STAGES; ++i) {
       mbar_init(&k_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&k_free[i], 1); mbar_init(&v_free[i], 1);
     }
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < NB; ++i) {
       mbar_init(&s_full[i], 1); mbar_init(&s_free[i], 8); mbar_init(&p_full[i], 8); mbar_init(&p_free[i], 1);
     }
     for (int i = 0; i < 4; ++i) mbar_init(&pair_bar[i], 64);
@@ -103,7 +107,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = tmem_base_s;
-  const uint32_t tmem_o = tmem_base + 2 * kBKV;       // S0 | S1 | O | Q
+  const uint32_t tmem_o = tmem_base + NB * kBKV;      // S [NB] | O | Q
   const uint32_t tmem_q = tmem_o + DV;
 
   if (warp == 0) {
@@ -129,9 +133,9 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       if (!ok) { atomicCAS(status, 0, 83); abort_s = 1; }
       tc_fence_after();
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int s = j % STAGES, sb = j & 1;
+        const int s = j % STAGES, sb = j % NB;
         if (!wait_bar(&k_full[s], (j / STAGES) & 1, abort_flag)) { atomicCAS(status, 0, 84); abort_s = 1; break; }
-        if (!wait_bar(&s_free[sb], ((j >> 1) & 1) ^ 1, abort_flag)) { atomicCAS(status, 0, 85); abort_s = 1; break; }
+        if (!wait_bar(&s_free[sb], ((j / NB) & 1) ^ 1, abort_flag)) { atomicCAS(status, 0, 85); abort_s = 1; break; }
         tc_fence_after();
 #pragma unroll
         for (int c = 0; c < NK; ++c) {
@@ -149,8 +153,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     if (lane == 0) {
       bool ok = true;
       for (int j = 0; j < n_tiles; ++j) {
-        const int s = j % STAGES, sb = j & 1;
-        if (!wait_bar(&p_full[sb], (j >> 1) & 1, abort_flag)) { atomicCAS(status, 0, 86); abort_s = 1; ok = false; break; }
+        const int s = j % STAGES, sb = j % NB;
+        if (!wait_bar(&p_full[sb], (j / NB) & 1, abort_flag)) { atomicCAS(status, 0, 86); abort_s = 1; ok = false; break; }
         if (!wait_bar(&v_full[s], (j / STAGES) & 1, abort_flag)) { atomicCAS(status, 0, 87); abort_s = 1; ok = false; break; }
         tc_fence_after();
         const uint64_t pd = umma_desc_sw128(Ps + sb * 2 * P_BYTES), rd = umma_desc_sw128(Ps + sb * 2 * P_BYTES + P_BYTES);
@@ -196,8 +200,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
     bool ok = true;
     uint32_t xph = 0;
     for (int j = 0; j < n_tiles; ++j) {
-      const int sb = j & 1;
-      if (!wait_bar(&s_full[sb], (j >> 1) & 1, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 88); abort_s = 1; } ok = false; break; }
+      const int sb = j % NB, xb = j & 1;
+      if (!wait_bar(&s_full[sb], (j / NB) & 1, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 88); abort_s = 1; } ok = false; break; }
       tc_fence_after();
       uint32_t sv[32];
       tmem_ld32(tmem_base + lane_base + sb * kBKV + hf * 32, sv);
@@ -210,31 +214,36 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       if (MODE == CAP_FIXED) {
         // 2^(log2e (cap tanh - cap)) = 2^(-2 cap log2e / (exp(2 s / cap) + 1))
 #pragma unroll
-        for (int c = 0; c < 32; ++c) {
-          float p = ex2(-2.f * cap2 * rcp(ex2(__uint_as_float(sv[c]) * f) + 1.f));
-          if (edge && (key0 + c > pos || key0 + c < key_lo)) p = 0.f;
-          sv[c] = __float_as_uint(p);
+        for (int c = 0; c < 32; ++c) sv[c] = __float_as_uint(ex2(-2.f * cap2 * rcp(ex2(__uint_as_float(sv[c]) * f) + 1.f)));
+        if (edge) {
+#pragma unroll
+          for (int c = 0; c < 32; ++c)
+            if (key0 + c > pos || key0 + c < key_lo) sv[c] = 0u;
         }
       } else {
-        float mx = -INFINITY;
+        if (MODE == CAP) {
 #pragma unroll
-        for (int c = 0; c < 32; ++c) {
-          float x = __uint_as_float(sv[c]) * f;
-          if (MODE == CAP) x = cap2 - 2.f * cap2 * rcp(ex2(x) + 1.f);
-          if (edge && (key0 + c > pos || key0 + c < key_lo)) x = -INFINITY;
-          sv[c] = __float_as_uint(x);
-          mx = fmaxf(mx, x);
+          for (int c = 0; c < 32; ++c) sv[c] = __float_as_uint(cap2 - 2.f * cap2 * rcp(ex2(__uint_as_float(sv[c]) * f) + 1.f));
         }
-        xch[sb][hf][r] = mx;
+        if (edge) {
+#pragma unroll
+          for (int c = 0; c < 32; ++c)
+            if (key0 + c > pos || key0 + c < key_lo) sv[c] = 0xff800000u;        // -inf
+        }
+        float mx = __uint_as_float(sv[0]);
+#pragma unroll
+        for (int c = 1; c < 32; ++c) mx = fmaxf(mx, __uint_as_float(sv[c]));
+        if (MODE == PLAIN) mx *= f;                    // f > 0: the largest score is the largest product
+        xch[xb][hf][r] = mx;
         mbar_arrive(&pair_bar[q]);
         if (!wait_bar(&pair_bar[q], xph, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 92); abort_s = 1; } ok = false; break; }
         xph ^= 1;
-        mx = fmaxf(kNoKey, fmaxf(xch[sb][0][r], xch[sb][1][r]));   // finite: with a window a page may hold no key of a row
+        mx = fmaxf(kNoKey, fmaxf(xch[xb][0][r], xch[xb][1][r]));   // finite: with a window a page may hold no key of a row
         if (j == 0) {
           m_ref = mx;
         } else if (__any_sync(0xffffffffu, mx > m_ref + 8.f)) {
           // every product that wrote O has to be complete before its rows are rescaled
-          if (!wait_bar(&p_free[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag)) {
+          if (!wait_bar(&p_free[(j - 1) % NB], ((j - 1) / NB) & 1, abort_flag)) {
             if (lane == 0) { atomicCAS(status, 0, 89); abort_s = 1; }
             ok = false;
             break;
@@ -256,7 +265,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
           tc_fence_before();
         }
 #pragma unroll
-        for (int c = 0; c < 32; ++c) sv[c] = __float_as_uint(ex2(__uint_as_float(sv[c]) - m_ref));
+        for (int c = 0; c < 32; ++c)
+          sv[c] = __float_as_uint(ex2(MODE == PLAIN ? fmaf(__uint_as_float(sv[c]), f, -m_ref) : __uint_as_float(sv[c]) - m_ref));
       }
       // head and remainder of the weights
       uint32_t ph[16], pr[16];
@@ -271,7 +281,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         pr[c] = pack_bf162(x, y);
       }
       l += l0 + l1;
-      if (j >= 2 && !wait_bar(&p_free[sb], ((j - 2) >> 1) & 1, abort_flag)) {   // the product of tile j - 2 has read this buffer
+      if (j >= NB && !wait_bar(&p_free[sb], ((j - NB) / NB) & 1, abort_flag)) {   // the product before has read this buffer
         if (lane == 0) { atomicCAS(status, 0, 90); abort_s = 1; }
         ok = false;
         break;
@@ -360,8 +370,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 
 template <int DK, int DV, int MODE>
 int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
-  constexpr int STAGES = DK + DV > 384 ? 2 : 3;
-  const size_t smem = (size_t)STAGES * kBKV * (DK + DV) * 2 + 4 * (size_t)kBQ * kBKV * 2 + 1024;
+  constexpr int NB = buffers(DK, DV), STAGES = DK + DV > (NB == 1 ? 192 : 384) ? 2 : 3;
+  const size_t smem = (size_t)STAGES * kBKV * (DK + DV) * 2 + 2 * NB * (size_t)kBQ * kBKV * 2 + 1024;
   auto kern = maps_tc_kernel<DK, DV, MODE, STAGES>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
@@ -391,7 +401,7 @@ CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G || a.maps < 1) return CB_ERR_ARG;
   if (a.act ? a.maps != 1 || a.lda % 8 || ((uintptr_t)a.act & 15) || a.lde % 8 || ((uintptr_t)a.egate & 15) : !a.part_o || !a.part_ml)
     return CB_ERR_ARG;
-  if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || a.ldp % 8 || a.ldk % 8 || a.ldv % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
+  if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || !(a.scale > 0.f) || a.ldp % 8 || a.ldk % 8 || a.ldv % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
   CUtensorMap tmK, tmV;
   const uint64_t kw = (uint64_t)a.G * a.maps * a.dim, vw = (uint64_t)a.G * a.vdim;
   int rc = cb_make_tmap_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kpool, (uint64_t)slots, kw, (uint64_t)pool_ldk(a), kBKV, 64);

@@ -41,10 +41,6 @@ struct MmaArgs {
   // its RMSNorm (gain tail_gain) in tail_out - what a separate pull kernel would do one launch later
   const bf16* tail_res_in; const float* tail_gain; bf16* tail_res_out; bf16* tail_out; float tail_eps;
   int act = 0; float act_a = 0.f, act_b = 0.f;         // epilogue activation (epi_act), 0: none
-  // expert units: grid row u multiplies rows [g_row0[u], + g_rows[u]) of y by expert g_expert[u]'s weights; row r of x is
-  // src[r] (null: r).  M is the most rows of a unit.
-  const int* g_count = nullptr; const int* g_row0 = nullptr; const int* g_rows = nullptr; const int* g_expert = nullptr;
-  const int* src = nullptr;
   TpComm tp;
 };
 
@@ -92,21 +88,6 @@ __global__ void __launch_bounds__(kT, 3) gemv_mma_kernel(const MmaArgs a_in) {
     a.x += (int64_t)(a.slot_xrow ? a.slot_xrow[slot] : slot) * a.K;
     a.y = OUT_F32 ? (void*)(reinterpret_cast<float*>(a.y) + (int64_t)slot * a.ldy)
                   : (void*)(reinterpret_cast<bf16*>(a.y) + (int64_t)slot * a.ldy);
-  }
-  const int* src = nullptr;
-  if (a.g_count) {
-    asm volatile("griddepcontrol.wait;" ::: "memory");
-    const int u = blockIdx.y;
-    if (u >= *a.g_count) {
-      cbtrace::stamp(0);
-      cbtrace::stamp(1);
-      return;
-    }
-    const int64_t r0 = a.g_row0[u];
-    a.M = a.g_rows[u];
-    a.W += (int64_t)a.g_expert[u] * a.expert_stride;
-    if (a.src) src = a.src + r0; else a.x += r0 * a.K;
-    a.y = OUT_F32 ? (void*)(reinterpret_cast<float*>(a.y) + r0 * a.ldy) : (void*)(reinterpret_cast<bf16*>(a.y) + r0 * a.ldy);
   }
   const int64_t K = a.K, nchunk = K >> 3;
   const int M = a.M;
@@ -266,14 +247,14 @@ __global__ void __launch_bounds__(kT, 3) gemv_mma_kernel(const MmaArgs a_in) {
     if ((int64_t)M * lc > 4 * nT) {
       for (int64_t i = tid; i < (int64_t)M * lc; i += nT) {
         const int64_t m = i / lc, c = xs_c0 + i % lc;
-        if (c < nchunk) cp_async16(xs + i * 8, a.x + ((src ? src[m] : m) * nchunk + c) * 8);
+        if (c < nchunk) cp_async16(xs + i * 8, a.x + (m * nchunk + c) * 8);
       }
       cp_async_commit();
       cp_async_wait_all_();
     } else {
       for (int64_t i = tid; i < (int64_t)M * lc; i += nT) {
         const int64_t m = i / lc, c = xs_c0 + i % lc;
-        if (c < nchunk) *reinterpret_cast<uint4*>(xs + i * 8) = *reinterpret_cast<const uint4*>(a.x + ((src ? src[m] : m) * nchunk + c) * 8);
+        if (c < nchunk) *reinterpret_cast<uint4*>(xs + i * 8) = *reinterpret_cast<const uint4*>(a.x + (m * nchunk + c) * 8);
       }
     }
   }
@@ -489,7 +470,7 @@ int launch_mma(MmaArgs a, cudaStream_t st, int n_slots = 1) {
   a.rounds = 1;
   if (nblk <= cta_slots(1)) {
     const int64_t smax = npair / 4 > 0 ? npair / 4 : 1;         // at least 4 k-step pairs per warp
-    const int kc_cap = (a.slot_expert || a.g_count || nblk > kMaxSplitUnits) ? 1 : g_mma_kcta_max;
+    const int kc_cap = (a.slot_expert || nblk > kMaxSplitUnits) ? 1 : g_mma_kcta_max;
     // prefer deep staging; give it up (2 -> 1 -> 0 batches) when shared memory would cost residency
     int64_t best = -1;
     int best_ks = 1, best_kcta = 1, best_stage = 0;
@@ -531,7 +512,7 @@ int launch_mma(MmaArgs a, cudaStream_t st, int n_slots = 1) {
     cudaGetSymbolAddress((void**)&a.ws, g_split_ws);
     cudaGetSymbolAddress((void**)&a.tickets, g_split_tickets);
   }
-  a.pf_rounds = a.slot_expert || a.g_count ? 0 : (a.rounds < g_mma_pf_rounds ? a.rounds : g_mma_pf_rounds);
+  a.pf_rounds = a.slot_expert ? 0 : (a.rounds < g_mma_pf_rounds ? a.rounds : g_mma_pf_rounds);
   a.xs_ld = slice_ld(ks, kcta);
   size_t smem = (((size_t)a.M * a.xs_ld * 2 + 15) & ~(size_t)15);
   if (ks > 1) smem += (size_t)a.rounds * warps * PB * 128 * sizeof(float);
@@ -651,24 +632,4 @@ CB_EXPORT int cb_moe_gemv(const void* W, const void* x, void* y, int64_t n_slots
   cudaStream_t st = (cudaStream_t)stream;
   if (mode & 1) return launch_mma<true, false, false>(a, st, (int)n_slots);
   return launch_mma<false, false, false>(a, st, (int)n_slots);
-}
-
-// The same product over a unit list (cb_routed_units; cb_moe_dispatch with a tile of at most 8 rows): up to max_rows <= 8 rows
-// of an expert share one pass over its weights.  Row r of y is W[expert(r)] x[src[r]] (src null: x[r]); act 2: squared relu.
-CB_EXPORT int cb_moe_gemv_units(const void* W, const void* x, void* y, int64_t max_units, int64_t max_rows, int64_t N, int64_t K,
-                                int64_t ldy, int64_t act, const void* g_count, const void* g_row0, const void* g_rows,
-                                const void* g_expert, const void* src, int64_t expert_stride, void* stream) {
-  if (!W || !x || !y || !g_count || !g_row0 || !g_rows || !g_expert) return CB_ERR_ARG;
-  if (K % 8 || N < 1 || max_units < 1 || max_units > 65535 || max_rows < 1 || max_rows > 8) return CB_ERR_SHAPE;
-  MmaArgs a;
-  a.W = (const bf16*)W; a.x = (const bf16*)x; a.y = y; a.N = N; a.K = K; a.ldy = ldy; a.up_off = N;
-  a.res_in = nullptr; a.add = nullptr; a.gain = nullptr; a.res_out = nullptr; a.eps = 0.f; a.M = (int)max_rows; a.ksplit = 1;
-  a.rounds = 1; a.pull_site = -1; a.push_site = -1;
-  a.tail_res_in = nullptr; a.tail_gain = nullptr; a.tail_res_out = nullptr; a.tail_out = nullptr; a.tail_eps = 0.f;
-  a.slot_expert = nullptr; a.slot_xrow = nullptr; a.expert_stride = expert_stride;
-  a.act = (int)act;
-  a.g_count = (const int*)g_count; a.g_row0 = (const int*)g_row0; a.g_rows = (const int*)g_rows; a.g_expert = (const int*)g_expert;
-  a.src = (const int*)src;
-  memset(&a.tp, 0, sizeof(a.tp));
-  return launch_mma<false, false, false>(a, (cudaStream_t)stream, (int)max_units);
 }

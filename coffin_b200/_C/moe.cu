@@ -123,6 +123,7 @@ __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restric
   __syncthreads();
   // every warp owns a contiguous range of slots (so that the second pass sees the same slots)
   const int per = (S + 31) / 32, s0 = warp * per, s1 = min(S, s0 + per);
+#pragma unroll 8
   for (int s = s0 + lane; s < s1; s += 32) {
     const int e = idx[s];
     if (e >= 0 && e < E) atomicAdd(&wh[warp * E + e], 1);
@@ -176,6 +177,7 @@ __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restric
   }
   for (int r = off[E] + tid; r < S; r += 1024) src_tok[r] = 0;
   // scatter: slot -> sorted row = first row of the expert + rows of earlier warps + this warp's cursor
+#pragma unroll 8
   for (int s = s0 + lane; s < s1; s += 32) {
     const int e = idx[s];
     if (e >= 0 && e < E) {

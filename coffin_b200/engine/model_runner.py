@@ -29,6 +29,7 @@ class ModelRunner:
         self.cfg = cfg
         self.device = getattr(model, "device", torch.device("cpu"))
         self.block_size = bm.pool.block_size
+        self.stateless = bool(getattr(model, "stateless", False))       # a sequence's pages are all it leaves behind
         self._rng: dict[int, random.Random] = {}
         self.n_prefill_tokens = 0
         self.n_decode_steps = 0
@@ -52,13 +53,14 @@ class ModelRunner:
         matches (KV blocks by reference, delta-net state restored from the snapshot)."""
         seq.blocks = self.bm.new_table()
         toks = seq.all_tokens
-        blocks, n, state = self.bm.match_prefix(toks, seq.mm)
+        blocks, n, state = self.bm.match_prefix(toks, seq.mm, require_states=not self.stateless)
         if debug.PC_TRACE:
             print(f"[pctrace] seq={seq.seq_id} prompt={len(toks)} matched={n} blocks={len(blocks) if n else 0} "
                   f"snapshot={'yes' if state is not None else 'no'}", flush=True)
         if n:
             seq.blocks.adopt(blocks, n)
-            self.model.restore_state(seq.slot, state)
+            if not self.stateless:
+                self.model.restore_state(seq.slot, state)
             seq.num_computed = n
             seq.cached_tokens = n
             self.n_cached_tokens += n
@@ -72,10 +74,10 @@ class ModelRunner:
     def _chunk_end(self, seq: Sequence, n: int) -> int:
         """End of the next chunk: at most ``n`` tokens, cut at the next snapshot boundary and at
         the last block boundary before the sampling position (so that the longest reusable
-        prefix of this prompt gets a state snapshot)."""
+        prefix of this prompt gets a state snapshot).  Where pages are all the state, nothing is cut."""
         start, total = seq.num_computed, seq.num_tokens
         end = min(total, start + n, start + self.cfg.chunk)
-        if self.bm.prefix_cache:
+        if self.bm.prefix_cache and not self.stateless:
             iv = max(self.block_size, self.cfg.snapshot_interval // self.block_size * self.block_size)
             nxt = (start // iv + 1) * iv
             tail = (total - 1) // self.block_size * self.block_size
@@ -120,7 +122,7 @@ class ModelRunner:
         self.n_prefill_tokens += T
         if last:
             seq.pending_logits = logits
-        if self.bm.prefix_cache and end % self.block_size == 0 and not last:
+        if self.bm.prefix_cache and not self.stateless and end % self.block_size == 0 and not last:
             iv = max(self.block_size, self.cfg.snapshot_interval // self.block_size * self.block_size)
             tail = (seq.num_tokens - 1) // self.block_size * self.block_size
             if end % iv == 0 or end == tail:
@@ -175,7 +177,7 @@ class ModelRunner:
 
     def finish_prefill(self, seq: Sequence) -> None:
         """Publish the computed prompt blocks (and their snapshots) to the prefix cache."""
-        if self.bm.prefix_cache and seq.snap_marks:
+        if self.bm.prefix_cache and (seq.snap_marks or self.stateless):
             self.bm.insert(seq.all_tokens[:seq.num_computed], seq.blocks.table, seq.snap_marks, seq.mm)
         seq.snap_marks = {}
 

@@ -114,8 +114,8 @@ _KERNELS: dict[str, tuple[str, ...]] = {
                  "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
     "sukisun": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "depth.cu", "linrec.cu", "ssd.cu",
                 "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
-    "fasolorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "residual.cu", "routed.cu", "moe.cu",
-                 "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
+    "fasolorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "residual.cu", "routed.cu", "gemv_units.cu",
+                 "moe.cu", "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
 }
 
 #: families that also run in 32-bit (``dtype=torch.float32``)

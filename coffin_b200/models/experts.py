@@ -44,19 +44,25 @@ class RoutedExperts:
         """Keywords of the ``residual_step`` that merges the result."""
         r, T, I, W8 = self.r, b.T, self.up.shape[1], self.up.shape[2]
         S = T * r.slots
-        logits = model.linear(self.router, h, model.buf("route_z", T, self.router.shape[0], torch.float32))
+        logits = model.buf("route_z", T, self.router.shape[0], torch.float32)
+        product = None
+        if T <= 8 and not model.f32:    # few rows: the product is the routing kernel's own
+            product = (self.router, h, model.buf("route_ticket", 1, 1, torch.int32))
+        else:
+            model.linear(self.router, h, logits)
         idx, w = model.buf("route_i", T, r.slots, torch.int32), model.buf("route_w", T, r.slots, torch.float32)
         idw = model.buf("route_id", T, 1, torch.float32)
         units = T <= R.UNIT_ROWS
         if units:
-            disp = R.route_units(r, logits, self.correction, b.positions, idx, w, idw, model.buf("route_u", 1, R.meta_size(r, T), torch.int32)[0])
+            disp = R.route_units(r, logits, self.correction, b.positions, idx, w, idw, model.buf("route_u", 1, R.meta_size(r, T), torch.int32)[0],
+                                 product)
         else:
             R.route(r, logits, self.correction, b.positions, idx, w, idw)
             disp = K.moe_dispatch(idx, r.stored, R.UNIT if model.f32 else 128)
         inter, y = model.buf("route_h", S, I), model.buf("route_y", S, W8)
         if units or model.f32:
             R.unit_linear(self.up, h, inter, disp, rows=T, gather=True, relu2=True)
-            R.unit_linear(self.down, inter, y, disp, rows=T, gather=False)
+            R.unit_linear(self.down, inter, y, disp, rows=T, gather=False, follows=True)
         else:
             K.gemm_grouped(h.index_select(0, disp["src_tok"]), self.up, disp, out=inter, relu2=True)
             K.gemm_grouped(inter, self.down, disp, out=y)

@@ -210,7 +210,7 @@ class FasolornConfig:
             for e in range(f.experts):
                 lin(f"{p}mlp.e{e}.up", f.ff, W), lin(f"{p}mlp.e{e}.down", W, f.ff)
             lin(p + "mlp.router", f.experts + f.identity, W)
-            plan.append((p + "mlp.correction", (f.experts + f.identity,), "lam"))
+            plan.append((p + "mlp.correction", (f.experts + f.identity,), "route"))
             if f.shared:
                 lin(p + "mlp.shared.up", f.shared, W), lin(p + "mlp.shared.down", W, f.shared)
         plan.append(("final.norm", (W,), "norm1"))

@@ -64,7 +64,10 @@ class WindowAttention(Mixer):
         if r0 < T:                      # the kernel turns the queries, and appends the rows' own keys and values
             pr, ps, rs = rows(r0, T)
             ns = core.decode_splits(T - r0)
-            po, pm = parts(T - r0, ns)
-            core.decode(pr, b.tables, ps, rs, po, pm, ns)
-            core.finish(po, pm, None, act[r0:], ps, nsplit=ns)
+            if ns == 1:
+                core.decode(pr, b.tables, ps, rs, None, None, 1, act=act[r0:])
+            else:
+                po, pm = parts(T - r0, ns)
+                core.decode(pr, b.tables, ps, rs, po, pm, ns)
+                core.finish(po, pm, None, act[r0:], ps, nsplit=ns)
         return act

@@ -194,6 +194,11 @@ class RowModel:
         return self.embed.index_select(0, tokens)
 
     # ------------------------------------------------------------------ sequence state
+    @property
+    def stateless(self) -> bool:
+        """Whether a sequence leaves nothing behind but pages: any cached page prefix can be reused without a snapshot."""
+        return not any(L.mixer.state for L in self.layers)
+
     def zero_state(self, slot: int) -> None:
         for L in self.layers:
             for t in L.mixer.state.values():

@@ -336,7 +336,7 @@ class AttnMaps:
         a.H, a.G, a.maps, a.dim, a.vdim, a.k_col, a.v_col = H, G, maps, dim, vdim, k_col, v_col
         a.scale, a.cap = float(scale), float(cap or 0.0)
         self.set_pools(kpool, vpool)
-        self._tcgen05 = bool(_lib.call_nostream("attn_maps_flash_tc_ok", dim, vdim))
+        self._tcgen05 = scale > 0 and bool(_lib.call_nostream("attn_maps_flash_tc_ok", dim, vdim))
         a.window, a.rot_half, a.sink = int(window), rot_dims // 2, _ptr(sink)
         self.window, self.sink, self._egate = int(window), sink, None
         if temp is not None:
@@ -398,11 +398,14 @@ class AttnMaps:
     def decode_splits(self, rows: int) -> int:
         R = self.H // self.G
         hpc = min(R, 8 // self.maps)
-        return max(1, min(64, window_pages(self.window), 148 // max(1, self.G * -(-R // hpc) * rows)))
+        resident = 296 if self.maps == 1 and max(self.dim, self.vdim) <= 128 else 148        # CTAs on the machine at once
+        return max(1, min(64, window_pages(self.window), resident // max(1, self.G * -(-R // hpc) * rows)))
 
-    def decode(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int) -> None:
-        """Single tokens (their keys and values are appended by the kernel): ``nsplit`` key splits per row."""
+    def decode(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int, act=None) -> None:
+        """Single tokens (their keys and values are appended by the kernel): ``nsplit`` key splits per row.  With one map and one
+        split ``act`` takes the finished heads and there are no parts."""
         self._fill(proj, tables, positions, row_seg, part_o, part_ml, nsplit)
+        self.a.act, self.a.lda, self.a.gates = _ptr(act), act.stride(0) if act is not None else 0, None
         call("attn_maps_decode", ctypes.byref(self.a), positions.numel(), _is_f32(proj))
         K._count()
 

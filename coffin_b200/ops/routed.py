@@ -51,15 +51,17 @@ def max_units(r: Router, T: int) -> int:
     return min(S, r.stored + S // UNIT)
 
 
-def route_units(r: Router, logits, correction, positions, idx, w, idw, meta) -> dict:
+def route_units(r: Router, logits, correction, positions, idx, w, idw, meta, product: tuple | None = None) -> dict:
     """``route`` for at most ``UNIT_ROWS`` rows, with the expert-sorted order and its units (layout of ``moe_dispatch``'s result) in
-    ``meta`` (int32)."""
+    ``meta`` (int32).  ``product = (router weight, h, ticket)`` (at most 8 bf16 rows; the ticket a zeroed int32): the same launch
+    computes the logits first."""
     T = logits.shape[0]
     S, n = T * r.slots, max_units(r, T)
     d = {"pos": meta[:S], "src_tok": meta[S:2 * S], "count": meta[2 * S:2 * S + 1], "row0": meta[2 * S + 1:2 * S + 1 + n],
          "rows": meta[2 * S + 1 + n:2 * S + 1 + 2 * n], "expert": meta[2 * S + 1 + 2 * n:2 * S + 1 + 3 * n], "max_tiles": n}
     call("routed_units", *_head(r, logits, correction, positions), idx, w, idw, d["pos"], d["src_tok"], d["count"], d["row0"], d["rows"],
-         d["expert"], n)
+         d["expert"], n, *((product[0], product[1], product[1].stride(0), product[1].shape[1], product[2]) if product is not None
+                           else (None, None, 0, 0, None)))
     K._count()
     return d
 
@@ -68,16 +70,18 @@ def meta_size(r: Router, T: int) -> int:
     return 2 * T * r.slots + 1 + 3 * max_units(r, T)
 
 
-def unit_linear(W: torch.Tensor, x: torch.Tensor, out: torch.Tensor, disp: dict, *, rows: int, gather: bool, relu2: bool = False) -> torch.Tensor:
-    """``out[r] = W[expert(r)] @ x[src(r) if gather else r]`` for the sorted rows of a unit list (at most ``rows`` of them per unit)."""
+def unit_linear(W: torch.Tensor, x: torch.Tensor, out: torch.Tensor, disp: dict, *, rows: int, gather: bool, relu2: bool = False,
+                follows: bool = False) -> torch.Tensor:
+    """``out[r] = W[expert(r)] @ x[src(r) if gather else r]`` for the sorted rows of a unit list (at most ``rows`` of them per unit).
+    ``follows``: the launch before this one is ``unit_linear`` over the same list."""
     E, N, Kd = W.shape
-    assert x.is_contiguous() and x.shape[1] == Kd and W.is_contiguous()
+    assert x.stride(1) == 1 and x.shape[1] == Kd and W.is_contiguous()
     src = disp["src_tok"] if gather else None
+    lists = (disp["count"], disp["row0"], disp["rows"], disp["expert"], src)
     if out.dtype == torch.float32:
-        call("routed_linear_f32", W, W.stride(0), x, x.stride(0), out, out.stride(0), N, Kd, disp["count"], disp["row0"], disp["rows"],
-             disp["expert"], src, disp["max_tiles"], int(relu2))
+        call("routed_linear_f32", W, W.stride(0), x, x.stride(0), out, out.stride(0), N, Kd, *lists, disp["max_tiles"], int(relu2))
     else:
-        call("moe_gemv_units", W, x, out, disp["max_tiles"], min(rows, UNIT), N, Kd, out.stride(0), 2 if relu2 else 0, disp["count"],
-             disp["row0"], disp["rows"], disp["expert"], src, W.stride(0))
+        call("gemv_units", W, W.stride(0), x, x.stride(0), out, out.stride(0), disp["max_tiles"], min(rows, UNIT), N, Kd, 2 if relu2 else 0,
+             *lists, int(follows))
     K._count()
     return out

@@ -115,6 +115,8 @@ def _draw(shape, kind: str, gen: torch.Generator, device, dtype, std: float) -> 
         return w.to(dtype)
     if kind == "gate_b":        # input / forget gate biases of a matrix memory
         return torch.randn(shape, generator=gen, device=device, dtype=torch.float32).to(dtype)
+    if kind == "route":         # correction of a router's scores, which are about one over their number
+        return (0.2 / shape[0] * torch.randn(shape, generator=gen, device=device)).to(dtype)
     if kind == "share":         # of a mixture of two
         return torch.rand(shape, generator=gen, device=device, dtype=torch.float32).to(dtype)
     if kind == "lam":

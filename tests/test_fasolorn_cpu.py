@@ -144,6 +144,46 @@ def test_engine_steps_mix_prompts_and_decode_rows(mixed, blocks):
     assert bool([b for b in twin.batches if max(b) > 1 and min(b) == 1]) == mixed and eng.bm.pool.used_blocks == 0
 
 
+class PagedTwin(Twin):
+    """The twin of a model whose pages are all the state: what a sequence was fed is read back through its block table."""
+    stateless = True
+
+    def __init__(self, *a, **kw):
+        super().__init__(*a, **kw)
+        self.pages = [[None] * 64 for _ in range(self.num_blocks)]
+
+    def forward_batch(self, items, want):
+        for toks, pos0, slot, table in items:
+            self.fed[slot] = [self.pages[table[i // 64]][i % 64] for i in range(pos0)]
+            for i, t in enumerate(toks.tolist() if isinstance(toks, torch.Tensor) else toks):
+                self.pages[table[(pos0 + i) // 64]][(pos0 + i) % 64] = t
+        return super().forward_batch(items, want)
+
+    def copy_block(self, src, dst):
+        self.pages[dst] = list(self.pages[src])
+
+    def snapshot_state(self, slot):
+        raise AssertionError("nothing to take a snapshot of")
+
+    restore_state = snapshot_state
+
+
+def test_any_cached_page_prefix_is_reused_without_snapshots():
+    W = S.weights(SMALL, 4)
+    twin = PagedTwin(SMALL, W, slots=2, blocks=24, forward=P.forward)
+    eng = LLMEngine(twin, EngineConfig(max_seq=256, max_num_seqs=2, chunk=100, prefill_quantum=100, mixed_batch=True))
+    base = [(5 * k) % 40 for k in range(180)]
+    prompts = [base, base[:70] + [1, 2, 3], base[:150] + [9] * 20, base[:64] + [4]]
+    params = SamplingParams(max_tokens=4, ignore_eos=True)
+    cached = 0
+    for p, n in zip(prompts, (0, 64, 128, 64)):
+        s, = eng.generate([p], params)
+        assert s.output == plain_greedy(SMALL, W, p, 4)
+        assert eng.runner.n_cached_tokens - cached == n
+        cached = eng.runner.n_cached_tokens
+    assert any(100 in b for b in twin.batches)                     # no chunk was cut for a snapshot's sake
+
+
 def test_trace_replay_batches_admission_and_release():
     W = S.weights(SMALL, 3)
     twin = Twin(SMALL, W, slots=4, blocks=pool_blocks(192), forward=P.forward)

@@ -614,9 +614,12 @@ def test_greedy_generation_through_the_engine(mixed):
     prompts = [toks(n, cfg["vocab"], 90 + n) for n in (70, 9, 40, 130, 3)]
     params = SamplingParams(max_tokens=8, ignore_eos=True)
     seqs = eng.generate(prompts, params)
-    prompts.append(prompts[3][:128] + [7])                     # shares a cached prefix: pages by reference
-    seqs += eng.generate(prompts[-1:], params)
-    assert (eng.runner.n_mixed_steps > 0) == mixed and eng.runner.n_cached_tokens > 0
+    for n, reused in ((128, 128), (90, 64)):                   # cached prefixes: pages by reference, at any page
+        before = eng.runner.n_cached_tokens
+        prompts.append(prompts[3][:n] + [7])
+        seqs += eng.generate(prompts[-1:], params)
+        assert eng.runner.n_cached_tokens - before == reused
+    assert (eng.runner.n_mixed_steps > 0) == mixed and m.stateless
     for s, p in zip(seqs, prompts):
         assert s.output == plain_greedy(cfg, W, p, 8)
 

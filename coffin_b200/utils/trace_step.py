@@ -179,7 +179,8 @@ def main() -> None:
         return
     M = m.bucket_for(args.rows)
     bt = list(range(m.max_blocks_per_seq))
-    m.set_rows(M, [int(first[0])] * args.rows, [args.prompt] * args.rows, list(range(args.rows)), [bt] * args.rows)
+    tokens = [(int(first[0]) + 4099 * r) % cfg.vocab_size for r in range(args.rows)]       # rows that choose experts of their own
+    m.set_rows(M, tokens, [args.prompt] * args.rows, list(range(args.rows)), [bt] * args.rows)
     for _ in range(3):
         m.decode(M, graph=True)
     rows, step_us, prev_us = trace_decode(m, M)

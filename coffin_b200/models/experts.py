@@ -1,6 +1,6 @@
 """Routed feed-forward of the row-batch families: squared-relu experts, a corrected choice, identity experts, a shared expert.
 
-The shared expert rides with the routed ones: cut into parts of an expert's width (exact, the activation works on single
+The shared expert rides with the routed ones: cut into parts of about an expert's width (exact, the activation works on single
 columns), its parts are stored behind the experts and every token holds a slot for each with weight one.  So a step is
 router product, routing, one product for all ups and one for all downs; the weighted sum of the slots happens in the
 residual boundary that follows.
@@ -17,19 +17,24 @@ from ..ops import routed as R
 from .rowmodel import RowBatch, pad8, padded
 
 
+#: most parts of a shared expert; one far wider than its experts gets wider parts, and the experts zero columns
+MAX_PARTS = 16
+
+
 class RoutedExperts:
     def __init__(self, W: dict[str, torch.Tensor], *, experts: int, identity: int, top: int, scale: float, ff: int, shared: int, width: int,
                  dtype, dev) -> None:
         """``W``: ``e<i>.up`` / ``e<i>.down``, ``router``, ``correction`` and, with ``shared`` > 0, ``shared.up`` / ``shared.down``."""
-        parts = -(-shared // ff)
+        parts = min(-(-shared // ff), MAX_PARTS)
+        step = max(ff, -(-shared // parts)) if parts else ff
         self.r = R.Router(experts, identity, top, scale, parts)
-        I, W8 = pad8(ff), pad8(width)
+        I, W8 = pad8(step), pad8(width)
         self.up = torch.zeros(experts + parts, I, W8, dtype=dtype, device=dev)
         self.down = torch.zeros(experts + parts, W8, I, dtype=dtype, device=dev)
         for e in range(experts):
             self.up[e, :ff, :width], self.down[e, :width, :ff] = W[f"e{e}.up"].to(dev, dtype), W[f"e{e}.down"].to(dev, dtype)
         for p in range(parts):
-            a, b = p * ff, min(shared, (p + 1) * ff)
+            a, b = p * step, min(shared, (p + 1) * step)
             self.up[experts + p, :b - a, :width] = W["shared.up"][a:b].to(dev, dtype)
             self.down[experts + p, :width, :b - a] = W["shared.down"][:, a:b].to(dev, dtype)
         self.router = padded(W["router"], pad8(experts + identity), W8, dtype, dev)

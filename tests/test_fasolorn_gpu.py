@@ -208,7 +208,7 @@ def test_unit_products(N, Kd, T, top):
 
 
 MOE = {"all": S.moe(), "no_identity": S.moe(5, 0, 2), "no_shared": S.moe(6, 2, 2, 24, 0), "one_of_many": S.moe(30, 4, 1, 16, 16), "all_of_them": S.moe(3, 2, 5, 32, 100),
-       "narrow_shared": S.moe(4, 1, 2, 48, 8), "mostly_identity": S.moe(2, 9, 3, 16, 24), "large": S.moe(6, 2, 2, 264, 520), "odd": S.moe(5, 1, 2, 13, 29, 0.3)}
+       "narrow_shared": S.moe(4, 1, 2, 48, 8), "mostly_identity": S.moe(2, 9, 3, 16, 24), "large": S.moe(6, 2, 2, 264, 520), "odd": S.moe(5, 1, 2, 13, 29, 0.3), "wide_shared": S.moe(9, 2, 3, 8, 333)}
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])

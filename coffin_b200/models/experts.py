@@ -25,8 +25,8 @@ class RoutedExperts:
     def __init__(self, W: dict[str, torch.Tensor], *, experts: int, identity: int, top: int, scale: float, ff: int, shared: int, width: int,
                  dtype, dev) -> None:
         """``W``: ``e<i>.up`` / ``e<i>.down``, ``router``, ``correction`` and, with ``shared`` > 0, ``shared.up`` / ``shared.down``."""
-        parts = min(-(-shared // ff), MAX_PARTS)
-        step = max(ff, -(-shared // parts)) if parts else ff
+        step = max(ff, -(-shared // MAX_PARTS))                   # columns of a part
+        parts = -(-shared // step)
         self.r = R.Router(experts, identity, top, scale, parts)
         I, W8 = pad8(step), pad8(width)
         self.up = torch.zeros(experts + parts, I, W8, dtype=dtype, device=dev)

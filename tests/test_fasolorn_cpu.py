@@ -82,11 +82,11 @@ def test_reordered_rows_turn_like_halves():
 
 def test_shared_expert_in_parts_is_the_whole():
     from coffin_b200.models.experts import RoutedExperts
-    for ff, shared in ((40, 56), (24, 24), (16, 70), (32, 8), (24, 0), (4, 300)):
+    for ff, shared in ((40, 56), (24, 24), (16, 70), (32, 8), (24, 0), (4, 300), (1, 20), (1, 16), (2, 33)):
         mlp = S.moe(3, 1, 2, ff, shared)
         W = {k[7:]: v for k, v in S.weights(S.config([S.latent()], [mlp])).items() if k.startswith("l0.mlp.")}
         r = RoutedExperts(W, experts=3, identity=1, top=2, scale=1.5, ff=ff, shared=shared, width=72, dtype=torch.float32, dev="cpu")
-        assert r.r.always == min(16, -(-shared // ff)) and r.r.slots == 2 + r.r.always
+        assert r.r.always == -(-shared // max(ff, -(-shared // 16))) and r.r.slots == 2 + r.r.always <= 18
         h = torch.randn(5, 72)
         got = sum((torch.relu(h @ r.up[3 + p].T) ** 2 @ r.down[3 + p].T for p in range(r.r.always)), torch.zeros(5, 72))
         ref = P.squared_relu(h, W["shared.up"].float(), W["shared.down"].float()) if shared else torch.zeros(5, 72)

@@ -77,6 +77,97 @@ __global__ void __launch_bounds__(256) maps_append8_kernel(const AttnMapsArgs a,
   }
 }
 
+// The extended form: heads are normed, then turned; values may turn; keys that are their own values stay as projected, with their
+// factor beside them.  `lanes` (a power of two) threads per head, V columns per access.
+template <typename T, int V>
+__device__ __forceinline__ void load_cols(const T* p, int n, float* f) {
+  if (V == 8) {
+    bf16x8_to_float(*reinterpret_cast<const uint4*>(p), f);
+  } else {
+    f[0] = act_load(p);
+    f[1] = n > 1 ? act_load(p + 1) : 0.f;
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_cols(T* p, int n, const float* f) {
+  if (V == 8) {
+    *reinterpret_cast<uint4*>(p) = float_to_bf16x8(f);
+  } else {
+    act_store(p, f[0]);
+    if (n > 1) act_store(p + 1, f[1]);
+  }
+}
+template <typename TP, typename TA, int V>
+__global__ void __launch_bounds__(256) maps_prep_kernel(const AttnMapsArgs a, int turn_q, int lanes) {
+  griddep_launch();
+  griddep_wait();
+  const int row = blockIdx.x, seg = a.row_seg ? a.row_seg[row] : row, pos = a.positions[row];
+  if (pos < 0) return;
+  const int64_t block = a.tables[(int64_t)seg * a.ldbt + pos / kPage], slot = block * kPage + pos % kPage;
+  TP* p = reinterpret_cast<TP*>(const_cast<void*>(a.proj)) + (int64_t)row * a.ldp;
+  TA* kp = reinterpret_cast<TA*>(a.kpool) + slot * pool_ldk(a);
+  TA* vp = reinterpret_cast<TA*>(a.vpool) + slot * pool_ldv(a);
+  const float2* cs = a.cs + (int64_t)row * a.rot_half;
+  const float2* vcs = a.vcs ? a.vcs + (int64_t)row * (a.vdim / 2) : nullptr;
+  const TP* w = a.v0 ? reinterpret_cast<const TP*>(a.v0) + (int64_t)row * a.ldv0 : nullptr;
+  const int nk = a.G * a.maps, nq = turn_q ? a.H * a.maps : 0, nv = a.kr ? 0 : a.G, total = nk + nq + nv;
+  const int per = 256 / lanes, l = threadIdx.x % lanes;
+  for (int u0 = 0; u0 < total; u0 += per) {
+    const int u = u0 + threadIdx.x / lanes;
+    const bool ok = u < total, key = u < nk, val = u >= nk + nq;
+    const int n = val ? a.vdim : a.dim;
+    TP* src = p + (key ? a.k_col + (int64_t)u * n : (val ? a.v_col + (int64_t)(u - nk - nq) * n : (int64_t)(u - nk) * n));
+    float f[V], rstd = 1.f;
+    if (a.norm) {
+      float ss = 0.f;
+      if (ok && !val)
+        for (int c = l * V; c < n; c += lanes * V) {
+          load_cols<TP, V>(src + c, n - c, f);
+#pragma unroll
+          for (int i = 0; i < V; ++i) ss = fmaf(f[i], f[i], ss);
+        }
+      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      rstd = 1.f / sqrtf(ss / (float)n + a.eps);
+    }
+    if (!ok) continue;                                           // the last pass
+    if (key && a.kr && l == 0) a.kr[factor_at(a, block, u / a.maps) + pos % kPage] = rstd;
+    const bool as_is = key && a.kr;
+    const float* nw = val || as_is ? nullptr : (key ? a.kn : a.qn);
+    const float2* turn = val ? vcs : (as_is ? nullptr : cs);
+    const int half = val ? (vcs ? a.vdim / 2 : 0) : (as_is ? 0 : a.rot_half);
+    const float r = val || as_is ? 1.f : rstd;
+    for (int c = l * V; c < n; c += lanes * V) {
+      load_cols<TP, V>(src + c, n - c, f);
+      if (val && w) {
+        float g[V];
+        load_cols<TP, V>(w + (src - p - a.v_col) + c, n - c, g);
+#pragma unroll
+        for (int i = 0; i < V; ++i) f[i] = mixed(f[i], g[i], a);
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] *= nw && c + i < n ? r * nw[c + i] : r;
+#pragma unroll
+      for (int i = 0; i < V; i += 2)
+        if ((c + i) >> 1 < half) {
+          const float2 t = turn[(c + i) >> 1];
+          const float x = f[i], y = f[i + 1];
+          f[i] = x * t.x - y * t.y;
+          f[i + 1] = y * t.x + x * t.y;
+        }
+      if (key) store_cols<TA, V>(kp + (int64_t)u * n + c, n - c, f);
+      else if (val) store_cols<TA, V>(vp + (int64_t)(u - nk - nq) * n + c, n - c, f);
+      else store_cols<TP, V>(src + c, n - c, f);
+    }
+  }
+}
+template <typename TP, typename TA, int V>
+int launch_prep(const AttnMapsArgs& a, int rows, int turn_q, cudaStream_t st) {
+  const int most = ((a.kr || a.dim > a.vdim ? a.dim : a.vdim) + V - 1) / V;
+  int lanes = 1;
+  while (lanes < 32 && lanes < most) lanes *= 2;
+  return (int)cb_launch(maps_prep_kernel<TP, TA, V>, dim3((unsigned)rows), dim3(256), 0, st, a, turn_q, lanes);
+}
+
 // One CTA per (query row, head, map): 128 keys at a time, scores by thread, running softmax, values by column.
 constexpr int kRT = 128;
 template <typename TP, typename TA>
@@ -99,10 +190,11 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
   for (int c = tid; c < a.dim; c += kRT) q[c] = act_round<TA>(act_load(qr + c)) * f;
   for (int c = tid; c < a.vdim; c += kRT) o[c] = 0.f;
   __syncthreads();
-  const int64_t ldk = pool_ldk(a), ldv = pool_ldv(a);
+  const int64_t ldk = pool_ldk(a), ldv = a.kr ? ldk : pool_ldv(a);
   const TA* K = reinterpret_cast<const TA*>(a.kpool) + (int64_t)(g * a.maps + map) * a.dim;
-  const TA* V = reinterpret_cast<const TA*>(a.vpool) + (int64_t)g * a.vdim;
+  const TA* V = a.kr ? K : reinterpret_cast<const TA*>(a.vpool) + (int64_t)g * a.vdim;
   const int* bt = a.tables + (int64_t)seg * a.ldbt;
+  const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r1 ? a.r2[h] : 0.f;
   float m = -INFINITY, l = 0.f;
   for (int k0 = first_key(a, pos); k0 <= pos; k0 += kRT) {
     const int n = min(kRT, pos + 1 - k0), j = k0 + tid;
@@ -111,7 +203,9 @@ __global__ void __launch_bounds__(kRT) maps_row_kernel(const AttnMapsArgs a) {
       const TA* kr = K + ((int64_t)bt[j / kPage] * kPage + j % kPage) * ldk;
       float d = 0.f;
       for (int c = 0; c < a.dim; ++c) d = fmaf(q[c], act_load(kr + c), d);
+      if (a.kr) d *= a.kr[factor_at(a, bt[j / kPage], g) + j % kPage];
       s = a.cap > 0.f ? a.cap * tanhf(d * inv_cap) : d;
+      if (a.r1) s -= r1 * log1pf(r2 * (float)(pos - j));
     }
     const float mn = fmaxf(m, block_max(s, red));
     const float p = tid < n ? expf(s - mn) : 0.f, w = expf(m - mn);
@@ -148,7 +242,7 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
                                                           const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
                                                           int64_t lda, const int* __restrict__ positions, int rows, int H,
                                                           int maps, int vdim, int nsplit, float lambda, float post_scale, float eps,
-                                                          const float* __restrict__ sink, const ElemGate eg) {
+                                                          const float* __restrict__ sink, const ElemGate eg, const float2* __restrict__ vcs) {
   griddep_launch();
   griddep_wait();
   const int64_t w = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -224,6 +318,10 @@ __global__ void __launch_bounds__(128) maps_finish_kernel(const float* __restric
 #pragma unroll
   for (int i = 0; i < kVMax / 4; ++i) {
     const int v = 4 * (lane + 32 * i);
+    if (vcs)
+#pragma unroll
+      for (int e = 0; e < 4; e += 2)
+        if (v + e + 1 < vdim) turn_back(o[4 * i + e], o[4 * i + e + 1], vcs[row * (vdim / 2) + (v + e) / 2]);
     if (eg.p)
 #pragma unroll
       for (int e = 0; e < 4; ++e)
@@ -245,7 +343,7 @@ __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __re
                                                                const float* __restrict__ gates, int64_t ldg, TA* __restrict__ act,
                                                                int64_t lda, const int* __restrict__ positions, int H, int maps,
                                                                int vdim, int nsplit, float lambda, float post_scale, float eps,
-                                                               const float* __restrict__ sink, const ElemGate eg) {
+                                                               const float* __restrict__ sink, const ElemGate eg, const float2* __restrict__ vcs) {
   extern __shared__ float sm[];                        // [warps][vdim]
   __shared__ float red[32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -293,6 +391,13 @@ __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __re
 #pragma unroll
       for (int w = 0; w < kWT / 32; ++w) x[k] += sm[w * vdim + c];
     ss = fmaf(x[k], x[k], ss);
+    if (vcs) {                                                   // the other entry of a pair is the neighbouring thread's
+      const float y = __shfl_xor_sync(0xffffffffu, x[k], 1);
+      if ((c | 1) < vdim) {
+        const float2 t = vcs[row * (vdim / 2) + c / 2];
+        x[k] = c & 1 ? x[k] * t.x - y * t.y : x[k] * t.x + y * t.y;
+      }
+    }
   }
   float r = post_scale;
   if (maps > 1) r *= 1.f / sqrtf(block_sum(ss, red) / (float)vdim + eps);
@@ -307,7 +412,7 @@ __global__ void __launch_bounds__(kWT) maps_finish_wide_kernel(const float* __re
 
 bool maps_args_ok(const AttnMapsArgs& a) {
   return a.proj && a.kpool && a.vpool && a.tables && a.positions && a.H > 0 && a.G > 0 && a.H % a.G == 0 && a.maps >= 1 && a.dim > 0 &&
-         a.vdim > 0 && 2 * a.rot_half <= a.dim && (!a.rot_half || a.cs);
+         a.vdim > 0 && 2 * a.rot_half <= a.dim && (!a.rot_half || a.cs) && !a.r1 == !a.r2 && (!a.kr || (a.maps == 1 && a.dim == a.vdim && !a.vcs));
 }
 
 }  // namespace
@@ -322,6 +427,14 @@ CB_EXPORT int cb_attn_maps_append(const void* args, int64_t rows, int64_t turn_q
   cudaStream_t st = (cudaStream_t)stream;
   const dim3 grid((unsigned)rows), block(256);
   const int tq = (int)turn_q;
+  if (extended(a)) {
+    if (f32) return launch_prep<float, float, 2>(a, (int)rows, tq, st);
+    if (p_f32) return launch_prep<float, bf16, 2>(a, (int)rows, tq, st);
+    const bool odd = a.dim % 8 || a.vdim % 8 || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || pool_ldk(a) % 8 || pool_ldv(a) % 8 || a.ldv0 % 8 ||
+                     (((uintptr_t)a.proj | (uintptr_t)a.v0 | (uintptr_t)a.kpool | (uintptr_t)a.vpool) & 15);
+    if (odd) return launch_prep<bf16, bf16, 2>(a, (int)rows, tq, st);
+    return launch_prep<bf16, bf16, 8>(a, (int)rows, tq, st);
+  }
   if (f32) return (int)cb_launch(maps_append_kernel<float, float>, grid, block, 0, st, a, tq);
   if (p_f32) return (int)cb_launch(maps_append_kernel<float, bf16>, grid, block, 0, st, a, tq);
   const bool wide = !(a.dim % 8 || a.vdim % 8 || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || pool_ldk(a) % 8 || pool_ldv(a) % 8 ||
@@ -347,10 +460,12 @@ CB_EXPORT int cb_attn_maps_rows(const void* args, int64_t rows, int64_t p_f32, i
 CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const void* gates, int64_t ldg, void* act, int64_t lda,
                                   const void* positions, int64_t rows, int64_t H, int64_t maps, int64_t vdim, int64_t nsplit,
                                   float lambda, float post_scale, float eps, const void* sink, const void* egate, int64_t lde,
-                                  int64_t e_f32, int64_t f32, void* stream) {
+                                  int64_t e_f32, const void* turns, int64_t f32, void* stream) {
   if (!part_o || !part_ml || !act || !positions || rows < 1 || maps < 1 || maps > 2 || nsplit < 1) return CB_ERR_ARG;
   const float* sk = (const float*)sink;
   const ElemGate eg = {egate, lde, (int)e_f32};
+  const float2* vcs = (const float2*)turns;
+  if (vcs && (maps != 1 || vdim % 2)) return CB_ERR_SHAPE;
   if (vdim > 32 * kVMax || nsplit > 64) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
   // a CTA per head, where there are many splits to walk or few heads to fill the machine with
@@ -361,17 +476,17 @@ CB_EXPORT int cb_attn_maps_finish(const void* part_o, const void* part_ml, const
     if (f32)
       return (int)cb_launch(maps_finish_wide_kernel<float>, wide, dim3(kWT), smem, st, (const float*)part_o, (const float*)part_ml,
                             (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)H, (int)maps, (int)vdim,
-                            (int)nsplit, lambda, post_scale, eps, sk, eg);
+                            (int)nsplit, lambda, post_scale, eps, sk, eg, vcs);
     return (int)cb_launch(maps_finish_wide_kernel<bf16>, wide, dim3(kWT), smem, st, (const float*)part_o, (const float*)part_ml,
                           (const float*)gates, ldg, (bf16*)act, lda, (const int*)positions, (int)H, (int)maps, (int)vdim, (int)nsplit,
-                          lambda, post_scale, eps, sk, eg);
+                          lambda, post_scale, eps, sk, eg, vcs);
   }
   const dim3 grid((unsigned)((rows * H + 3) / 4)), block(128);
   if (f32)
     return (int)cb_launch(maps_finish_kernel<float>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
                           (const float*)gates, ldg, (float*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps,
-                          (int)vdim, (int)nsplit, lambda, post_scale, eps, sk, eg);
+                          (int)vdim, (int)nsplit, lambda, post_scale, eps, sk, eg, vcs);
   return (int)cb_launch(maps_finish_kernel<bf16>, grid, block, 0, st, (const float*)part_o, (const float*)part_ml,
                         (const float*)gates, ldg, (bf16*)act, lda, (const int*)positions, (int)rows, (int)H, (int)maps, (int)vdim,
-                        (int)nsplit, lambda, post_scale, eps, sk, eg);
+                        (int)nsplit, lambda, post_scale, eps, sk, eg, vcs);
 }

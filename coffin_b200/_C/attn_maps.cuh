@@ -8,7 +8,10 @@
 // Optional parts, each switched on by its field: a sliding window (a query sees itself and the window - 1 tokens before
 // it), a sink per head (an entry of the softmax without key or value), interleaved rotary positions on queries and keys
 // (taken when rows are appended and when a decode query is read), values mixed with another layer's, and an output gate
-// per element.
+// per element.  Further: chunks (a query sees the tokens of its own chunk), an RMS norm of queries and keys per head ahead of the
+// turn, values cached turned by their position with heads turned back by the query's, a score penalty that grows with the
+// logarithm of the distance, and keys that are their own values: the pages hold keys as projected, read once for both
+// products, and one factor per key stands for its norm.
 #pragma once
 #include "act_type.cuh"
 
@@ -35,12 +38,23 @@ struct AttnMapsArgs {
   const void* v0; int64_t ldv0;          // values of another layer, rows like proj (null: none):
   float v_own, v_mix;                    //   v = v_own * own + v_mix * v0
   const void* egate; int64_t lde;        // one map: output gate pre-activations [rows, H * vdim], rows like proj (null: none)
+  int chunk;                             // > 0: keys of the query's own chunk of this many tokens, counted from position 0
+  int norm; float eps;                   // norm: queries and keys are divided by their root mean square per head, then
+  const float* qn; const float* kn;      //   weighted [dim] (null: not)
+  const float2* vcs;                     // (cos, sin) [rows, vdim / 2]: values are cached turned, heads turned back (null: no)
+  float* kr;                             // one map: factors [blocks, G, 64] of the scores of the keys, which are cached as
+                                         //   projected and are the values too (vpool is not used) (null: no)
+  const float* r1; const float* r2;      // [H]: score -= r1 ln(1 + r2 distance) (null: no)
+  float oscale;                          // one map: factor of the finished head
 };
 
 // first key that the query at `pos` sees
 __host__ __device__ __forceinline__ int first_key(const AttnMapsArgs& a, int pos) {
-  return a.window > 0 && pos >= a.window ? pos - a.window + 1 : 0;
+  const int w = a.window > 0 && pos >= a.window ? pos - a.window + 1 : 0;
+  return a.chunk > 0 ? max(w, pos - pos % a.chunk) : w;
 }
+// norm, value turns, key factors and distance penalties: what the plain forms of append and decode leave out
+__host__ __device__ __forceinline__ bool extended(const AttnMapsArgs& a) { return a.norm || a.vcs || a.kr || a.r1; }
 // finite stand-in for "no key seen yet": exponentials of differences with it are 0 or 1, never NaN
 constexpr float kNoKey = -1e30f;
 
@@ -62,6 +76,19 @@ __device__ __forceinline__ float turned(const T* p, int c, int in_head, const fl
 }
 __device__ __forceinline__ float mixed(float own, float other, const AttnMapsArgs& a) {
   return a.v0 ? a.v_own * own + a.v_mix * other : own;
+}
+// factor slot of key `key` of a block, key/value head g
+__device__ __forceinline__ int64_t factor_at(const AttnMapsArgs& a, int64_t block, int g) { return (block * a.G + g) * kPage; }
+// entries (2 m, 2 m + 1) of a finished head, turned back by the query's angle
+__device__ __forceinline__ void turn_back(float& x, float& y, const float2 t) {
+  const float u = x;
+  x = u * t.x + y * t.y;
+  y = y * t.x - u * t.y;
+}
+__device__ __forceinline__ float lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 // tanh through one exponential: |error| ~ 1e-7
 __device__ __forceinline__ float cap_score(float s, float cap, float inv_cap) {

@@ -44,17 +44,24 @@ __device__ __forceinline__ uint32_t split_head(float& x, float& y) {
 constexpr int kBM = 128, kBN = 64, kFT = 256;
 constexpr float kLog2e = 1.4426950408889634f;
 
-template <int DK, int DV>
-constexpr size_t flash_smem() { return sizeof(bf16) * ((size_t)kBM * (DK + 8) + 2 * (size_t)kBN * (DK + 8 + DV + 8)); }
+// Modes: scores as they are, capped scores, keys that are their own values (one staged page serves both products).
+enum FlashMode : int { PLAIN = 0, CAPPED = 1, SHARED = 2 };
+template <int DK, int DV, int MODE>
+constexpr size_t flash_smem() {
+  return sizeof(bf16) * ((size_t)kBM * (DK + 8) + 2 * (size_t)kBN * (DK + 8 + (MODE == SHARED ? 0 : DV + 8))) + (MODE == SHARED ? 2 * kBN * 4 : 0);
+}
 
-template <int DK, int DV, bool CAP>
+template <int DK, int DV, int MODE>
 __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a) {
+  constexpr bool CAP = MODE == CAPPED, KV = MODE == SHARED;
+  static_assert(!KV || DK == DV, "values are the keys");
   constexpr int LK = DK + 8, LV = DV + 8, NK = DK / 16, NV = DV / 8;
   constexpr bool QREG = DK <= 128;
   extern __shared__ __align__(128) unsigned char smem[];
   bf16* qs = reinterpret_cast<bf16*>(smem);            // [kBM][LK]
   bf16* ks = qs + kBM * LK;                            // [2][kBN][LK]
-  bf16* vs = ks + 2 * kBN * LK;                        // [2][kBN][LV]
+  bf16* vs = KV ? ks : ks + 2 * kBN * LK;              // [2][kBN][LV]
+  float* fs = reinterpret_cast<float*>(ks + 2 * kBN * LK);       // [2][kBN] factors of the keys (SHARED)
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
   const int vh = blockIdx.y, seg = blockIdx.z;
   griddep_launch();
@@ -85,10 +92,14 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
       const bool ok = c < a.dim && pg * kPage + r <= last;
       cp16(kd + r * LK + c, ok ? K + (base + r) * ldk + c : K, ok);
     }
-    for (int e = tid; e < kBN * (DV / 8); e += kFT) {
-      const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
-      const bool ok = c < a.vdim && pg * kPage + r <= last;
-      cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
+    if (KV) {
+      if (tid < kBN / 4) cp16(fs + (pg & 1) * kBN + tid * 4, a.kr + factor_at(a, bt[pg], g) + tid * 4, true);
+    } else {
+      for (int e = tid; e < kBN * (DV / 8); e += kFT) {
+        const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+        const bool ok = c < a.vdim && pg * kPage + r <= last;
+        cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -106,6 +117,7 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
     f[i] = a.scale * query_temp(a, i ? phi : plo);
     f[i] *= CAP ? 2.f * kLog2e * inv_cap : kLog2e;               // CAP: exponent of exp(2 s / cap); else log2 units
   }
+  const float r1 = KV && a.r1 ? a.r1[h] : 0.f, r2 = KV && a.r1 ? a.r2[h] : 0.f;
   const float cap2 = a.cap * kLog2e;
   uint32_t qf[QREG ? NK : 1][4];
   const int warp_last = pos0 + t0 + warp * 16 + 15, warp_first = first_key(a, pos0 + t0 + warp * 16), warp_full = first_key(a, warp_last);
@@ -148,6 +160,11 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           float x = s[i][e] * f[e >> 1];
+          if (KV) {
+            const int key = i * 8 + t4 * 2 + (e & 1);
+            x *= fs[(pg & 1) * kBN + key];
+            if (a.r1) x = fmaf(-r1, lg2(fmaf(r2, (float)((e >> 1 ? phi : plo) - pg * kPage - key), 1.f)), x);      // NaN past the diagonal: masked below
+          }
           if (CAP) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);        // log2(e) * cap * tanh(score / cap)
           if (edge) {
             const int key = pg * kPage + i * 8 + t4 * 2 + (e & 1);
@@ -202,7 +219,8 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
     if (a.act) {                                                 // one map: the head is finished here
       const int64_t row = row0 + t0 + r;
       if (a.sink) den[i] += ex2(a.sink[h] * kLog2e - mx[i]);
-      const float s = (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / den[i];
+      const float s = a.oscale * (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / den[i];
+      const float2* vcs = a.vcs ? a.vcs + row * (a.vdim / 2) : nullptr;
       bf16* out = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * a.vdim;
       const bf16* eg = a.egate ? reinterpret_cast<const bf16*>(a.egate) + row * a.lde + (int64_t)h * a.vdim : nullptr;
 #pragma unroll
@@ -210,6 +228,7 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
         const int c = v * 8 + t4 * 2;
         if (c >= a.vdim) continue;
         float x = o[v][2 * i] * s, y = o[v][2 * i + 1] * s;
+        if (vcs) turn_back(x, y, vcs[c / 2]);
         if (eg) {
           const uint32_t g = *reinterpret_cast<const uint32_t*>(eg + c);
           x *= sigmoid_x(__uint_as_float(g << 16));
@@ -234,10 +253,10 @@ __global__ void __launch_bounds__(kFT, 1) maps_flash_kernel(const AttnMapsArgs a
   }
 }
 
-template <int DK, int DV, bool CAP>
+template <int DK, int DV, int MODE>
 int flash_launch(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
-  auto kern = maps_flash_kernel<DK, DV, CAP>;
-  constexpr size_t smem = flash_smem<DK, DV>();
+  auto kern = maps_flash_kernel<DK, DV, MODE>;
+  constexpr size_t smem = flash_smem<DK, DV, MODE>();
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   return (int)cb_launch(kern, dim3((unsigned)tiles, (unsigned)(a.H * a.maps), (unsigned)segs), dim3(kFT), smem, st, a);
@@ -245,8 +264,9 @@ int flash_launch(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
 template <int DK>
 int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
   const bool cap = a.cap > 0.f;
+  if (a.kr) return cap ? CB_ERR_SHAPE : flash_launch<DK, DK, SHARED>(a, tiles, segs, st);
 #define CB_DV(N) \
-  if (a.vdim <= N) return cap ? flash_launch<DK, N, true>(a, tiles, segs, st) : flash_launch<DK, N, false>(a, tiles, segs, st)
+  if (a.vdim <= N) return cap ? flash_launch<DK, N, CAPPED>(a, tiles, segs, st) : flash_launch<DK, N, PLAIN>(a, tiles, segs, st)
   CB_DV(32); CB_DV(64); CB_DV(128); CB_DV(256);
 #undef CB_DV
   return CB_ERR_SHAPE;
@@ -258,16 +278,27 @@ int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
 // product takes the bf16 heads of the weights in rows 0-7 and their remainders in rows 8-15.
 constexpr int kDT = 256;
 constexpr int decode_ctas(int dk, int dv, int maps) { return maps == 1 && dk <= 128 && dv <= 128 ? 2 : 1; }    // per SM
-template <int DK, int DV, int MAPS, typename TP>
+// Forms: as described, with norms, turned values and distance penalties (one map), and the same with keys that are their own values.
+enum DecodeForm : int { BASIC = 0, NORMED = 1, KEYS_ONLY = 2 };
+template <int DK, int DV, int MAPS, int FORM>
+constexpr size_t decode_smem() {
+  return sizeof(bf16) * (2 * (size_t)kPage * (MAPS * (DK + 8) + (FORM == KEYS_ONLY ? 0 : DV + 8)) + MAPS * 8 * (DK + 8) + 16 * (kPage + 8)) +
+         sizeof(float) * (8 * kPage + (FORM == KEYS_ONLY ? 2 * kPage : 0));
+}
+template <int DK, int DV, int MAPS, typename TP, int FORM>
 __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
+  constexpr bool KV = FORM == KEYS_ONLY;
+  static_assert(FORM == BASIC || MAPS == 1, "one map");
+  static_assert(!KV || DK == DV, "values are the keys");
   constexpr int LK = DK + 8, LV = DV + 8, KPAGE = MAPS * kPage * LK, VPAGE = kPage * LV, NP = DV / 16, NPW = (NP + 7) / 8;
   extern __shared__ __align__(128) unsigned char smem[];
   bf16* ks = reinterpret_cast<bf16*>(smem);            // [2][MAPS][kPage][LK]
-  bf16* vs = ks + 2 * KPAGE;                           // [2][kPage][LV]
-  bf16* qs = vs + 2 * VPAGE;                           // [MAPS][8][LK]
+  bf16* vs = KV ? ks : ks + 2 * KPAGE;                 // [2][kPage][LV]
+  bf16* qs = KV ? ks + 2 * KPAGE : vs + 2 * VPAGE;     // [MAPS][8][LK]
   bf16* pa = qs + MAPS * 8 * LK;                       // [16][kPage + 8]: heads, remainders
   float* ps = reinterpret_cast<float*>(pa + 16 * (kPage + 8));   // [8][kPage] scores
-  __shared__ float w_s[8];
+  float* fs = ps + 8 * kPage;                          // [2][kPage] factors of the keys (KEYS_ONLY)
+  __shared__ float w_s[8], own_s;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
   const int split = blockIdx.x, row = blockIdx.z;
   const int R = a.H / a.G, cpg = (R + hpc - 1) / hpc, g = blockIdx.y / cpg, r0 = (blockIdx.y % cpg) * hpc, nh = min(hpc, R - r0);
@@ -300,21 +331,59 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
       const bool ok = r < n && c < a.dim;
       cp16(kd + (m * kPage + r) * LK + c, ok ? K + (base + r) * ldk + m * a.dim + c : K, ok);
     }
-    for (int e = tid; e < kPage * (DV / 8); e += kDT) {
-      const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
-      const bool ok = r < n && c < a.vdim;
-      cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
+    if (KV) {
+      if (tid < kPage / 4) cp16(fs + (pg & 1) * kPage + tid * 4, a.kr + factor_at(a, bt[pg], g) + tid * 4, true);
+    } else {
+      for (int e = tid; e < kPage * (DV / 8); e += kDT) {
+        const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
+        const bool ok = r < n && c < a.vdim;
+        cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   load(pg0);
   const bool cap = a.cap > 0.f;
   const float f = a.scale * query_temp(a, pos) * (cap ? 2.f * kLog2e / a.cap : kLog2e), cap2 = a.cap * kLog2e;
-  for (int e = tid; e < MAPS * 8 * LK; e += kDT) {
-    const int m = e / (8 * LK), i = (e / LK) % 8, c = e % LK;
-    const bool ok = i < nh && c < a.dim;
-    qs[e] = ok ? __float2bfloat16(turned(pr, ((g * R + r0 + i) * MAPS + m) * a.dim + c, c, cs, a.rot_half)) : __float2bfloat16(0.f);
+  if (FORM == BASIC) {
+    for (int e = tid; e < MAPS * 8 * LK; e += kDT) {
+      const int m = e / (8 * LK), i = (e / LK) % 8, c = e % LK;
+      const bool ok = i < nh && c < a.dim;
+      qs[e] = ok ? __float2bfloat16(turned(pr, ((g * R + r0 + i) * MAPS + m) * a.dim + c, c, cs, a.rot_half)) : __float2bfloat16(0.f);
+    }
+  } else {
+    // a warp per query vector, a pair of columns per lane and step; then the norm of the token's own key by the last warp
+    auto inverse_rms = [&](const TP* x) {
+      float ss = 0.f;
+      for (int c = lane * 2; c < a.dim; c += 64) {
+        const float u = act_load(x + c), v = act_load(x + c + 1);
+        ss = fmaf(u, u, fmaf(v, v, ss));
+      }
+      return a.norm ? 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps) : 1.f;
+    };
+    const TP* q = pr + (int64_t)(g * R + r0 + warp) * a.dim;
+    const float rq = warp < nh ? inverse_rms(q) : 0.f;
+    for (int c = lane * 2; c < LK; c += 64) {
+      float x = 0.f, y = 0.f;
+      if (warp < nh && c < a.dim) {
+        x = act_load(q + c) * rq;
+        y = act_load(q + c + 1) * rq;
+        if (a.qn) { x *= a.qn[c]; y *= a.qn[c + 1]; }
+        if (c >> 1 < a.rot_half) {
+          const float2 t = cs[c >> 1];
+          const float u = x;
+          x = u * t.x - y * t.y;
+          y = y * t.x + u * t.y;
+        }
+      }
+      *reinterpret_cast<uint32_t*>(qs + warp * LK + c) = pack_bf162(x, y);
+    }
+    if (warp == kDT / 32 - 1 && pg1 == pages) {
+      const float rk = inverse_rms(pr + a.k_col + (int64_t)g * a.dim);
+      if (lane == 0) own_s = rk;
+    }
   }
+  const float r1 = FORM != BASIC && a.r1 && g4 < nh ? a.r1[g * R + r0 + g4] : 0.f, r2 = FORM != BASIC && a.r1 && g4 < nh ? a.r2[g * R + r0 + g4] : 0.f;
   for (int e = tid; e < 16 * (kPage + 8); e += kDT) pa[e] = __float2bfloat16(0.f);
   float o[NPW][2][4];
 #pragma unroll
@@ -337,16 +406,53 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
       // the same values)
       const int r = pos % kPage;
       const int64_t slot = (int64_t)bt[pg] * kPage + r;
-      for (int c = tid; c < MAPS * a.dim; c += kDT) {
-        const bf16 x = __float2bfloat16(turned(pr + a.k_col, g * MAPS * a.dim + c, c % a.dim, cs, a.rot_half));
-        kt[((c / a.dim) * kPage + r) * LK + c % a.dim] = x;
-        K[slot * ldk + c] = x;
-      }
-      for (int c = tid; c < a.vdim; c += kDT) {
-        const int64_t vc = (int64_t)g * a.vdim + c;
-        const bf16 x = __float2bfloat16(mixed(act_load(pr + a.v_col + vc), v0 ? act_load(v0 + vc) : 0.f, a));
-        vt[r * LV + c] = x;
-        V[slot * ldv + c] = x;
+      if (FORM == BASIC) {
+        for (int c = tid; c < MAPS * a.dim; c += kDT) {
+          const bf16 x = __float2bfloat16(turned(pr + a.k_col, g * MAPS * a.dim + c, c % a.dim, cs, a.rot_half));
+          kt[((c / a.dim) * kPage + r) * LK + c % a.dim] = x;
+          K[slot * ldk + c] = x;
+        }
+        for (int c = tid; c < a.vdim; c += kDT) {
+          const int64_t vc = (int64_t)g * a.vdim + c;
+          const bf16 x = __float2bfloat16(mixed(act_load(pr + a.v_col + vc), v0 ? act_load(v0 + vc) : 0.f, a));
+          vt[r * LV + c] = x;
+          V[slot * ldv + c] = x;
+        }
+      } else {
+        const TP* k = pr + a.k_col + (int64_t)g * a.dim;
+        const float rk = KV ? 1.f : own_s;
+        for (int c = tid * 2; c < a.dim; c += 2 * kDT) {
+          float x = act_load(k + c) * rk, y = act_load(k + c + 1) * rk;
+          if (!KV && a.kn) { x *= a.kn[c]; y *= a.kn[c + 1]; }
+          if (!KV && c >> 1 < a.rot_half) {
+            const float2 t = cs[c >> 1];
+            const float u = x;
+            x = u * t.x - y * t.y;
+            y = y * t.x + u * t.y;
+          }
+          const uint32_t xy = pack_bf162(x, y);
+          *reinterpret_cast<uint32_t*>(kt + r * LK + c) = xy;
+          *reinterpret_cast<uint32_t*>(K + slot * ldk + c) = xy;
+        }
+        if (KV) {
+          if (tid == 0) fs[(pg & 1) * kPage + r] = a.kr[factor_at(a, bt[pg], g) + r] = own_s;
+        } else {
+          const float2* vcs = a.vcs + (int64_t)row * (a.vdim / 2);
+          for (int c = (kDT - 1 - tid) * 2; c < a.vdim; c += 2 * kDT) {      // first the threads that had no key columns
+            const int64_t vc = (int64_t)g * a.vdim + c;
+            float x = mixed(act_load(pr + a.v_col + vc), v0 ? act_load(v0 + vc) : 0.f, a);
+            float y = mixed(act_load(pr + a.v_col + vc + 1), v0 ? act_load(v0 + vc + 1) : 0.f, a);
+            if (a.vcs) {
+              const float2 t = vcs[c >> 1];
+              const float u = x;
+              x = u * t.x - y * t.y;
+              y = y * t.x + u * t.y;
+            }
+            const uint32_t xy = pack_bf162(x, y);
+            *reinterpret_cast<uint32_t*>(vt + r * LV + c) = xy;
+            *reinterpret_cast<uint32_t*>(V + slot * ldv + c) = xy;
+          }
+        }
       }
       __syncthreads();
     }
@@ -369,8 +475,10 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           float x = (s[e] + s2[e]) * f;
-          if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
           const int key = warp * 8 + t4 * 2 + e;
+          if (KV) x *= fs[(pg & 1) * kPage + key];
+          if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
+          if (FORM != BASIC && a.r1) x = fmaf(-r1, lg2(fmaf(r2, (float)(pos - pg * kPage - key), 1.f)), x);
           ps[(g4 * MAPS + m) * kPage + key] = pg * kPage + key <= pos && pg * kPage + key >= lo ? x : -INFINITY;
         }
       }
@@ -409,12 +517,13 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
     __syncthreads();
   }
   if (MAPS == 1 && a.act) {                            // the only split: the heads are finished here
-    if (warp < nq && lane == 0) w_s[warp] = 1.f / (l_run + (a.sink ? ex2(a.sink[g * R + r0 + warp] * kLog2e - m_run) : 0.f));
+    if (warp < nq && lane == 0) w_s[warp] = a.oscale / (l_run + (a.sink ? ex2(a.sink[g * R + r0 + warp] * kLog2e - m_run) : 0.f));
     __syncthreads();
     if (g4 >= nq) return;
     const float inv = w_s[g4];
     const int hc = (g * R + r0 + g4) * a.vdim;
     bf16* out = reinterpret_cast<bf16*>(a.act) + (int64_t)row * a.lda + hc;
+    const float2* vcs = FORM == NORMED && a.vcs ? a.vcs + (int64_t)row * (a.vdim / 2) : nullptr;
     const TP* eg = a.egate ? reinterpret_cast<const TP*>(a.egate) + (int64_t)row * a.lde + hc : nullptr;
 #pragma unroll
     for (int i = 0; i < NPW; ++i)
@@ -423,6 +532,7 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
         const int c = (warp + 8 * i) * 16 + j * 8 + t4 * 2;
         if (warp + 8 * i >= NP || c >= a.vdim) continue;
         float x = (o[i][j][0] + o[i][j][2]) * inv, y = (o[i][j][1] + o[i][j][3]) * inv;
+        if (vcs) turn_back(x, y, vcs[c >> 1]);
         if (eg) { x *= sigmoid_x(act_load(eg + c)); y *= sigmoid_x(act_load(eg + c + 1)); }
         *reinterpret_cast<uint32_t*>(out + c) = pack_bf162(x, y);
       }
@@ -444,18 +554,28 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
   }
 }
 
-template <int DK, int DV, int MAPS, typename TP>
-int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
-  constexpr size_t smem = sizeof(bf16) * (2 * (size_t)kPage * (MAPS * (DK + 8) + DV + 8) + MAPS * 8 * (DK + 8) + 16 * (kPage + 8)) +
-                          sizeof(float) * 8 * kPage;
-  auto kern = maps_decode_kernel<DK, DV, MAPS, TP>;
+template <int DK, int DV, int MAPS, typename TP, int FORM>
+int decode_form(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  constexpr size_t smem = decode_smem<DK, DV, MAPS, FORM>();
+  auto kern = maps_decode_kernel<DK, DV, MAPS, TP, FORM>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const int R = a.H / a.G;
   return (int)cb_launch(kern, dim3((unsigned)a.nsplit, (unsigned)(a.G * ((R + hpc - 1) / hpc)), (unsigned)rows), dim3(kDT), smem, st, a, hpc);
 }
+template <int DK, int DV, int MAPS, typename TP>
+int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  if constexpr (MAPS == 1) {
+    if (extended(a)) return decode_form<DK, DV, 1, TP, NORMED>(a, hpc, rows, st);
+  }
+  return decode_form<DK, DV, MAPS, TP, BASIC>(a, hpc, rows, st);
+}
 template <int DK, int MAPS, typename TP>
 int decode_dv(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
+  if constexpr (MAPS == 1) {
+    constexpr int D = DK < 64 ? 64 : DK;
+    if (a.kr) return decode_form<D, D, 1, TP, KEYS_ONLY>(a, hpc, rows, st);
+  }
   if (a.vdim <= 64) return decode_launch<DK, 64, MAPS, TP>(a, hpc, rows, st);
   if (a.vdim <= 128) return decode_launch<DK, 128, MAPS, TP>(a, hpc, rows, st);
   return decode_launch<DK, 256, MAPS, TP>(a, hpc, rows, st);
@@ -482,6 +602,7 @@ CB_EXPORT int cb_attn_maps_flash(const void* args, int64_t segs, int64_t max_row
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G) return CB_ERR_ARG;
   if (a.act ? a.maps != 1 || a.lda % 2 || a.lde % 2 : !a.part_o || !a.part_ml) return CB_ERR_ARG;
+  if ((a.r1 && !a.kr) || (a.kr && (a.maps != 1 || a.dim != a.vdim || a.vcs || a.sink || a.egate))) return CB_ERR_SHAPE;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   const int tiles = (int)((max_rows + kBM - 1) / kBM);
   cudaStream_t st = (cudaStream_t)stream;
@@ -498,8 +619,9 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   const AttnMapsArgs& a = *(const AttnMapsArgs*)args;
   if (a.act ? a.maps != 1 || a.nsplit != 1 || a.lda % 2 : !a.part_o || !a.part_ml) return CB_ERR_ARG;
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || a.H < 1 || a.G < 1 || a.H % a.G ||
-      a.nsplit < 1 || a.nsplit > 64 || 2 * a.rot_half > a.dim || (a.rot_half && !a.cs))
+      a.nsplit < 1 || a.nsplit > 64 || 2 * a.rot_half > a.dim || (a.rot_half && !a.cs) || !a.r1 != !a.r2)
     return CB_ERR_ARG;
+  if (extended(a) && (a.maps != 1 || (a.kr && (a.dim != a.vdim || a.vcs)))) return CB_ERR_SHAPE;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
   const int R = a.H / a.G;

@@ -8,6 +8,9 @@
 // product, P = bf16 head + bf16 remainder, two products per page; the result leaves as unnormalised fp32 sums with
 // (reference maximum, denominator), which maps_finish_kernel combines across the maps.
 //
+// SHARED: the keys are their own values.  One ring of pages serves both products (K-major for the scores, MN-major for the
+// sums), released by the second; a key's factor comes with its page, and the penalty r1 ln(1 + r2 distance) is taken off.
+//
 // With a cap the scores are bounded, so the reference maximum is the cap itself (when 2^-2cap is far from underflow):
 // no row maximum, no exchange between the halves of a row, no rescale.  Otherwise the reference is raised lazily as in
 // attn_tc.cu.  Waits are bounded by 2 s and report through the status word; TMEM is freed on every path.
@@ -19,7 +22,7 @@ using namespace sm100;
 
 constexpr int kBQ = 128, kBKV = 64, kThreads = 352;
 constexpr float kLog2e = 1.4426950408889634f;
-enum Mode : int { PLAIN = 0, CAP = 1, CAP_FIXED = 2 };
+enum Mode : int { PLAIN = 0, CAP = 1, CAP_FIXED = 2, SHARED = 3 };
 
 __device__ __forceinline__ uint64_t now_ns() {
   uint64_t t;
@@ -53,8 +56,10 @@ constexpr int buffers(int dk, int dv) { return dk <= 128 && dv <= 128 ? 1 : 2; }
 template <int DK, int DV, int MODE, int STAGES>
 __global__ void __launch_bounds__(kThreads, 3 - buffers(DK, DV))
 maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnMapsArgs a, int* status) {
+  constexpr bool KV = MODE == SHARED;
+  static_assert(!KV || DK == DV, "values are the keys");
   constexpr int NK = DK / 64, NV = DV / 64;           // 64-element (128-byte) chunks
-  constexpr int K_BYTES = kBKV * DK * 2, V_BYTES = kBKV * DV * 2, P_BYTES = kBQ * kBKV * 2;
+  constexpr int K_BYTES = kBKV * DK * 2, V_BYTES = KV ? 0 : kBKV * DV * 2, P_BYTES = kBQ * kBKV * 2;
   constexpr int KC = kBKV * 128;                      // bytes of one chunk block of a page
   constexpr int NB = buffers(DK, DV);
   constexpr uint32_t TMEM_COLS = NB * kBKV + DV + DK / 2 <= 256 ? 256 : 512;
@@ -68,6 +73,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
   unsigned char* Ps = Vs + STAGES * V_BYTES;          // [NB][head | remainder]
   __shared__ uint64_t q_full, k_full[STAGES], v_full[STAGES], k_free[STAGES], v_free[STAGES], s_full[NB], s_free[NB], p_full[NB], p_free[NB],
       o_full, pair_bar[4];
+  __shared__ __align__(16) float factor_s[KV ? STAGES : 1][kBKV];
   __shared__ float xch[2][2][kBQ];                    // [tile parity][column half][row]: maxima of half rows
   __shared__ uint32_t tmem_base_s;
   __shared__ int abort_s;
@@ -119,8 +125,12 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         const uint32_t ph = (j / STAGES) & 1;
         const int slot0 = bt[page0 + j] * kBKV;
         if (!wait_bar(&k_free[s], ph ^ 1, abort_flag)) { atomicCAS(status, 0, 81); abort_s = 1; break; }
-        mbar_expect_tx(&k_full[s], K_BYTES);
+        mbar_expect_tx(&k_full[s], K_BYTES + (KV ? kBKV * 4 : 0));
         for (int c = 0; c < NK; ++c) tma_load_2d(Ks + s * K_BYTES + c * KC, &tmK, &k_full[s], kmap * DK + c * 64, slot0);
+        if (KV) {
+          bulk_load(factor_s[s], a.kr + factor_at(a, bt[page0 + j], kh), kBKV * 4, &k_full[s]);
+          continue;
+        }
         if (!wait_bar(&v_free[s], ph ^ 1, abort_flag)) { atomicCAS(status, 0, 82); abort_s = 1; break; }
         mbar_expect_tx(&v_full[s], V_BYTES);
         for (int c = 0; c < NV; ++c) tma_load_2d(Vs + s * V_BYTES + c * KC, &tmV, &v_full[s], kh * DV + c * 64, slot0);
@@ -144,7 +154,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
           for (int k = 0; k < 4; ++k)
             umma_f16_ta(tmem_base + sb * kBKV, tmem_q + c * 32 + k * 8, kd + 2 * k, IDESC_S, (c | k) != 0);
         }
-        umma_commit(&k_free[s]);
+        if (!KV) umma_commit(&k_free[s]);
         umma_commit(&s_full[sb]);
       }
     }
@@ -155,16 +165,16 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       for (int j = 0; j < n_tiles; ++j) {
         const int s = j % STAGES, sb = j % NB;
         if (!wait_bar(&p_full[sb], (j / NB) & 1, abort_flag)) { atomicCAS(status, 0, 86); abort_s = 1; ok = false; break; }
-        if (!wait_bar(&v_full[s], (j / STAGES) & 1, abort_flag)) { atomicCAS(status, 0, 87); abort_s = 1; ok = false; break; }
+        if (!wait_bar(KV ? &k_full[s] : &v_full[s], (j / STAGES) & 1, abort_flag)) { atomicCAS(status, 0, 87); abort_s = 1; ok = false; break; }
         tc_fence_after();
         const uint64_t pd = umma_desc_sw128(Ps + sb * 2 * P_BYTES), rd = umma_desc_sw128(Ps + sb * 2 * P_BYTES + P_BYTES);
-        const uint64_t vd = umma_desc_mn_sw128(Vs + s * V_BYTES, KC);
+        const uint64_t vd = umma_desc_mn_sw128(KV ? Ks + s * K_BYTES : Vs + s * V_BYTES, KC);
 #pragma unroll
         for (int k = 0; k < 4; ++k)      // 16 keys per instruction: +32 bytes along P's rows, +16 rows of V
           umma_f16(tmem_o, pd + 2 * k, vd + (uint64_t)(k * 16 * 128 >> 4), IDESC_O, (j | k) != 0);
 #pragma unroll
         for (int k = 0; k < 4; ++k) umma_f16(tmem_o, rd + 2 * k, vd + (uint64_t)(k * 16 * 128 >> 4), IDESC_O, 1);
-        umma_commit(&v_free[s]);
+        umma_commit(KV ? &k_free[s] : &v_free[s]);
         umma_commit(&p_free[sb]);
       }
       if (ok) umma_commit(&o_full);
@@ -193,7 +203,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       if (lane == 0) mbar_arrive(&q_full);
     }
     // score -> log2 units; with a cap first to the exponent of exp(2 score / cap)
-    const float f = a.scale * query_temp(a, min(pos, pos0 + n - 1)) * (MODE == PLAIN ? kLog2e : 2.f * kLog2e / a.cap);
+    const float f = a.scale * query_temp(a, min(pos, pos0 + n - 1)) * (MODE == PLAIN || KV ? kLog2e : 2.f * kLog2e / a.cap);
+    const float r1 = KV && a.r1 ? a.r1[h] : 0.f, r2 = KV && a.r1 ? a.r2[h] : 0.f;
     const float cap2 = a.cap * kLog2e;
     const int key_lo = first_key(a, pos), full_lo = first_key(a, pos0 + row0 + kBQ - 1);
     float m_ref = MODE == CAP_FIXED ? cap2 : -INFINITY, l = 0.f;
@@ -224,6 +235,23 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
         if (MODE == CAP) {
 #pragma unroll
           for (int c = 0; c < 32; ++c) sv[c] = __float_as_uint(cap2 - 2.f * cap2 * rcp(ex2(__uint_as_float(sv[c]) * f) + 1.f));
+        }
+        if (KV) {
+          // the factors of this page have landed: its scores were computed behind the same barrier
+          if (!wait_bar(&k_full[j % STAGES], (j / STAGES) & 1, abort_flag)) { if (lane == 0) { atomicCAS(status, 0, 94); abort_s = 1; } ok = false; break; }
+          const float4* kf = reinterpret_cast<const float4*>(factor_s[j % STAGES] + hf * 32);
+          const float far = fmaf(r2, (float)(pos - key0), 1.f);
+#pragma unroll
+          for (int c4 = 0; c4 < 8; ++c4) {
+            const float4 k4 = kf[c4];
+            const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              float x = __uint_as_float(sv[c4 * 4 + e]) * f * kk[e];
+              if (a.r1) x = fmaf(-r1, lg2(fmaf(-r2, (float)(c4 * 4 + e), far)), x);      // NaN past the diagonal: masked below
+              sv[c4 * 4 + e] = __float_as_uint(x);
+            }
+          }
         }
         if (edge) {
 #pragma unroll
@@ -309,7 +337,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       tc_fence_after();
       const int64_t row = seg0 + t;
       if (a.sink) l += ex2(a.sink[h] * kLog2e - m_ref);
-      const float s = t < n ? (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / l : 0.f;
+      const float s = t < n ? a.oscale * (a.gates ? sigmoid_x(a.gates[row * a.ldg + h]) : 1.f) / l : 0.f;
+      const float2* vcs = !KV && a.vcs ? a.vcs + row * (DV / 2) : nullptr;
       const bf16* eg = a.egate ? reinterpret_cast<const bf16*>(a.egate) + row * a.lde + (int64_t)h * DV : nullptr;
       bf16* op = reinterpret_cast<bf16*>(a.act) + row * a.lda + (int64_t)h * DV;
 #pragma unroll 1
@@ -323,6 +352,14 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
             float x[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[8 * v + e]) * s;
+            if (vcs) {
+#pragma unroll
+              for (int e = 0; e < 8; e += 4) {
+                const float4 t2 = *reinterpret_cast<const float4*>(vcs + (c0 + v * 8 + e) / 2);
+                turn_back(x[e], x[e + 1], make_float2(t2.x, t2.y));
+                turn_back(x[e + 2], x[e + 3], make_float2(t2.z, t2.w));
+              }
+            }
             if (eg) {
               float g[8];
               bf16x8_to_float(*reinterpret_cast<const uint4*>(eg + c0 + v * 8), g);
@@ -370,8 +407,8 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 
 template <int DK, int DV, int MODE>
 int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
-  constexpr int NB = buffers(DK, DV), STAGES = DK + DV > (NB == 1 ? 192 : 384) ? 2 : 3;
-  const size_t smem = (size_t)STAGES * kBKV * (DK + DV) * 2 + 2 * NB * (size_t)kBQ * kBKV * 2 + 1024;
+  constexpr int NB = buffers(DK, DV), COLS = MODE == SHARED ? DK : DK + DV, STAGES = COLS > (NB == 1 ? 192 : 384) ? 2 : 3;
+  const size_t smem = (size_t)STAGES * kBKV * COLS * 2 + 2 * NB * (size_t)kBQ * kBKV * 2 + 1024;
   auto kern = maps_tc_kernel<DK, DV, MODE, STAGES>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
@@ -380,6 +417,9 @@ int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs
 }
 template <int DK, int DV>
 int mode_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
+  if constexpr (DK == DV) {
+    if (a.kr) return launch_tc<DK, DV, SHARED>(tmK, tmK, a, tiles, segs, status, st);
+  }
   if (!(a.cap > 0.f)) return launch_tc<DK, DV, PLAIN>(tmK, tmV, a, tiles, segs, status, st);
   // 2^(-2 cap log2e) well inside the range of fp32 and of a bf16 remainder 2^-16 below it
   if (a.cap <= 30.f) return launch_tc<DK, DV, CAP_FIXED>(tmK, tmV, a, tiles, segs, status, st);
@@ -390,7 +430,7 @@ int mode_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& 
 
 // Whether cb_attn_maps_flash_tc takes these head sizes.
 CB_EXPORT int cb_attn_maps_flash_tc_ok(int64_t dim, int64_t vdim) {
-  return (dim == 64 || dim == 128 || dim == 192 || dim == 256) && (vdim == 64 || vdim == 128 || vdim == 256);
+  return (dim == 64 || dim == 128 || dim == 192 || dim == 256) && (vdim == 64 || vdim == 128 || vdim == 256 || (vdim == 192 && dim == 192));
 }
 
 // Prompt attention of `segs` segments of at most `max_rows` rows on tcgen05; arguments as for cb_attn_maps_flash.
@@ -401,19 +441,21 @@ CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.seg_row || !a.seg_pos || a.H < 1 || a.G < 1 || a.H % a.G || a.maps < 1) return CB_ERR_ARG;
   if (a.act ? a.maps != 1 || a.lda % 8 || ((uintptr_t)a.act & 15) || a.lde % 8 || ((uintptr_t)a.egate & 15) : !a.part_o || !a.part_ml)
     return CB_ERR_ARG;
+  if ((a.r1 && !a.kr) || (a.kr && (a.maps != 1 || a.dim != a.vdim || a.vcs || a.sink || a.egate || a.cap > 0.f || !a.act))) return CB_ERR_SHAPE;
+  if (a.vcs && (((uintptr_t)a.vcs & 15) || !a.act)) return CB_ERR_ARG;
   if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || !(a.scale > 0.f) || a.ldp % 8 || a.ldk % 8 || a.ldv % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
   CUtensorMap tmK, tmV;
   const uint64_t kw = (uint64_t)a.G * a.maps * a.dim, vw = (uint64_t)a.G * a.vdim;
   int rc = cb_make_tmap_2d(&tmK, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kpool, (uint64_t)slots, kw, (uint64_t)pool_ldk(a), kBKV, 64);
   if (rc) return rc;
-  rc = cb_make_tmap_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.vpool, (uint64_t)slots, vw, (uint64_t)pool_ldv(a), kBKV, 64);
+  rc = a.kr ? 0 : cb_make_tmap_2d(&tmV, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.vpool, (uint64_t)slots, vw, (uint64_t)pool_ldv(a), kBKV, 64);
   if (rc) return rc;
   const int tiles = (int)((max_rows + kBQ - 1) / kBQ);
   int* st_word = (int*)status;
   cudaStream_t st = (cudaStream_t)stream;
 #define CB_TC(K, V) \
   if (a.dim == K && a.vdim == V) return mode_tc<K, V>(tmK, tmV, a, tiles, (int)segs, st_word, st)
-  CB_TC(64, 64); CB_TC(64, 128); CB_TC(64, 256); CB_TC(128, 64); CB_TC(128, 128); CB_TC(128, 256); CB_TC(192, 64); CB_TC(192, 128); CB_TC(192, 256); CB_TC(256, 64); CB_TC(256, 128);
+  CB_TC(64, 64); CB_TC(64, 128); CB_TC(64, 256); CB_TC(128, 64); CB_TC(128, 128); CB_TC(128, 256); CB_TC(192, 64); CB_TC(192, 128); CB_TC(192, 192); CB_TC(192, 256); CB_TC(256, 64); CB_TC(256, 128);
   CB_TC(256, 256);
 #undef CB_TC
   return CB_ERR_SHAPE;

@@ -25,7 +25,7 @@ FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--use_fast_math", "-Xcompiler", "-fP
 # Sources whose arithmetic is specified in 32-bit (recurrent states, decays, capped scores, the fp32 stream sums):
 # compiled without the approximate forms of exp / tanh / log / division that --use_fast_math substitutes.
 PRECISE = {"streams.cu", "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu", "gemm_f32.cu",
-           "depth.cu", "latent.cu", "ssd.cu", "residual.cu", "routed.cu"}
+           "depth.cu", "latent.cu", "rope.cu", "ssd.cu", "residual.cu", "routed.cu"}
 
 
 def flags(src: Path) -> list[str]:

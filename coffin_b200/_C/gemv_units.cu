@@ -27,13 +27,16 @@ __device__ __forceinline__ void mma(float* c, uint32_t a0, uint32_t a1, uint32_t
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
+// GATED: an expert has N gate rows, then N up rows; a block is 8 outputs, its gate rows are fragments g, its up rows g + 8.
+template <bool GATED>
 __global__ void __launch_bounds__(kT, 3) gemv_units_kernel(const UnitArgs a) {
+  constexpr int kOut = GATED ? 8 : 16;                           // outputs of a block
   extern __shared__ __align__(16) unsigned char smem[];
   float* part = reinterpret_cast<float*>(smem);                  // [2][kWarps][kPart]
   bf16* xs = reinterpret_cast<bf16*>(part + 2 * kWarps * kPart); // [max_rows][K + kPad]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int nchunk = a.K >> 3, npair = (nchunk + 3) >> 2, per = (npair + kWarps - 1) / kWarps;
-  const int p0 = warp * per, p1 = min(npair, p0 + per), nblk = (a.N + 15) >> 4, ldxs = a.K + kPad;
+  const int p0 = warp * per, p1 = min(npair, p0 + per), nblk = (a.N + kOut - 1) / kOut, ldxs = a.K + kPad;
   if (!a.early) griddep_wait();
   griddep_launch();
   const int64_t total = (int64_t)__ldcg(a.count) * nblk;
@@ -43,8 +46,8 @@ __global__ void __launch_bounds__(kT, 3) gemv_units_kernel(const UnitArgs a) {
   // rows of block `blk` that this lane loads, of expert e
   auto block = [&](int e, int blk, const bf16** lo_, const bf16** hi_) {
     const bf16* w = a.W + (int64_t)e * a.stride;
-    *lo_ = w + (int64_t)min(blk * 16 + g, a.N - 1) * a.K;
-    *hi_ = w + (int64_t)min(blk * 16 + g + 8, a.N - 1) * a.K;
+    *lo_ = w + (int64_t)min(blk * kOut + g, a.N - 1) * a.K;
+    *hi_ = w + (int64_t)(GATED ? a.N + min(blk * kOut + g, a.N - 1) : min(blk * kOut + g + 8, a.N - 1)) * a.K;
   };
   auto load = [&](const bf16* l, const bf16* h, int p) {
 #pragma unroll
@@ -87,7 +90,7 @@ __global__ void __launch_bounds__(kT, 3) gemv_units_kernel(const UnitArgs a) {
         mma(acc, wl[u].z, wh[u].z, wl[u].w, wh[u].w, v.z, v.w);
       }
     }
-    const int n0 = blk * 16, rr = r0, MM = M;
+    const int n0 = blk * kOut, rr = r0, MM = M;
     if (it + 1 < hi) {
       if (++blk == nblk) {
         blk = 0;
@@ -100,14 +103,19 @@ __global__ void __launch_bounds__(kT, 3) gemv_units_kernel(const UnitArgs a) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) mine[(2 * t + (i & 1)) * kMS + g + (i >> 1) * 8] = acc[i];
     __syncthreads();
-    if (tid < 128) {
-      const int m = tid >> 4, r = tid & 15;
+    if (tid < 8 * kOut) {
+      const int m = tid / kOut, r = tid % kOut;
       if (m < MM && n0 + r < a.N) {
         const float* q = part + (it & 1) * kWarps * kPart + m * kMS + r;
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) v += q[w * kPart];
-        if (a.act) v = epi_act(a.act, v, 0.f, 0.f);
+        if (GATED) {
+          float up = 0.f;
+#pragma unroll
+          for (int w = 0; w < kWarps; ++w) up += q[w * kPart + 8];
+          v = silu_s(v) * up;
+        } else if (a.act) v = epi_act(a.act, v, 0.f, 0.f);
         a.y[(int64_t)(rr + m) * a.ldy + n0 + r] = __float2bfloat16(v);
       }
     }
@@ -117,7 +125,7 @@ __global__ void __launch_bounds__(kT, 3) gemv_units_kernel(const UnitArgs a) {
 }  // namespace
 
 // y[r] = act(W[expert(r)] x[src[r]]) (src null: x[r]) for the sorted rows of the unit list; units hold at most max_rows <= 8 rows.
-// act 2: squared relu (0: none).  early: the kernel before this one is the same product over the same list (see above).
+// act 2: squared relu (0: none); 3: silu(gate) * up, W holds N gate rows, then N up rows of every expert.  early: the kernel before this one is the same product over the same list (see above).
 CB_EXPORT int cb_gemv_units(const void* W, int64_t stride, const void* x, int64_t ldx, void* y, int64_t ldy, int64_t max_units,
                             int64_t max_rows, int64_t N, int64_t K, int64_t act, const void* count, const void* row0, const void* rows,
                             const void* expert, const void* src, int64_t early, void* stream) {
@@ -127,14 +135,15 @@ CB_EXPORT int cb_gemv_units(const void* W, int64_t stride, const void* x, int64_
   UnitArgs a;
   a.W = (const bf16*)W; a.stride = stride; a.x = (const bf16*)x; a.ldx = ldx; a.y = (bf16*)y; a.ldy = ldy;
   a.count = (const int*)count; a.row0 = (const int*)row0; a.rows = (const int*)rows; a.expert = (const int*)expert; a.src = (const int*)src;
-  a.N = (int)N; a.K = (int)K; a.act = (int)act; a.early = (int)early; a.max_rows = (int)max_rows;
+  a.N = (int)N; a.K = (int)K; a.act = act == 3 ? 0 : (int)act; a.early = (int)early; a.max_rows = (int)max_rows;
   const size_t smem = sizeof(float) * 2 * kWarps * kPart + sizeof(bf16) * (size_t)max_rows * (K + kPad);
   if (smem > 220 * 1024) return CB_ERR_SHAPE;
-  cudaError_t e = cudaFuncSetAttribute(gemv_units_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  auto kern = act == 3 ? gemv_units_kernel<true> : gemv_units_kernel<false>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   int64_t per_sm = (int64_t)(224 * 1024 / (smem + 1024));
   per_sm = per_sm < 1 ? 1 : (per_sm > 3 ? 3 : per_sm);
-  const int64_t items = max_units * ((N + 15) / 16), grid = items < 148 * per_sm ? items : 148 * per_sm;
+  const int64_t per_block = act == 3 ? 8 : 16, items = max_units * ((N + per_block - 1) / per_block), grid = items < 148 * per_sm ? items : 148 * per_sm;
   int64_t carve = (per_sm * (int64_t)(smem + 1024) * 100 + 228 * 1024 - 1) / (228 * 1024);
-  return (int)cb_launch_carve((int)(carve > 100 ? 100 : carve), gemv_units_kernel, dim3((unsigned)grid), dim3(kT), smem, (cudaStream_t)stream, a);
+  return (int)cb_launch_carve((int)(carve > 100 ? 100 : carve), kern, dim3((unsigned)grid), dim3(kT), smem, (cudaStream_t)stream, a);
 }

@@ -5,7 +5,7 @@
 //              One key / value head for all query heads: decoding, and portions of few tokens.
 //   expanded : keys and values of every head are multiplied out of the pages' rows (one GEMM whose weight carries
 //              identity rows for the shared part) and the prompt kernels of attn_maps_flash.cu / attn_maps_tc.cu run on them.
-// Here: the angles of a batch, the norm / rotate / append kernel, the gather of page rows, the per-head products of the
+// Here: the norm / rotate / append kernel, the gather of page rows, the per-head products of the
 // absorbed form (tensor cores; plain form for 32-bit) and its split-key decode kernel.  Norms, angles, scores and softmax
 // are fp32; the attention weights enter the second product as bf16 head + remainder.
 #include "act_type.cuh"
@@ -42,20 +42,6 @@ __device__ __forceinline__ uint32_t split_head(float& x, float& y) {
   x -= __uint_as_float(h << 16);
   y -= __uint_as_float(h & 0xffff0000u);
   return h;
-}
-
-// ---- angles ------------------------------------------------------------------------------------
-// cs[row, i] = (cos, sin) of position * freq_i, freq in turns (fp64: the turn count is reduced exactly, whatever the position)
-__global__ void __launch_bounds__(256) rope_rows_kernel(const int* __restrict__ positions, const double* __restrict__ turns,
-                                                        float2* __restrict__ cs, int rows, int half) {
-  griddep_launch();
-  griddep_wait();
-  const int e = blockIdx.x * 256 + threadIdx.x;
-  if (e >= rows * half) return;
-  const double t = (double)max(positions[e / half], 0) * turns[e % half];
-  float s, c;
-  sincospif(2.f * (float)(t - rint(t)), &s, &c);
-  cs[e] = make_float2(c, s);
 }
 
 // ---- norm, rotate, append ----------------------------------------------------------------------
@@ -148,32 +134,6 @@ __global__ void __launch_bounds__(kPT) latent_rows_kernel(const LatentArgs a) {
       if (2 * i + 1 < a.rot) act_store(out + a.cp + 2 * i + 1, v);
     }
   }
-}
-
-// rotated query parts: src [rows, heads] at column off of each head -> dst (the same place, or the absorbed query)
-template <typename TS, typename TA>
-__global__ void __launch_bounds__(256) rope_heads_kernel(const TS* __restrict__ src, int64_t lds, int64_t hs, TA* __restrict__ dst,
-                                                         int64_t ldd, int64_t hd, const float2* __restrict__ cs, int half, int rot, int H,
-                                                         int rows) {
-  griddep_launch();
-  griddep_wait();
-  const int np = (rot + 1) / 2;
-  const int64_t e = (int64_t)blockIdx.x * 256 + threadIdx.x;
-  if (e >= (int64_t)rows * H * np) return;
-  const int i = (int)(e % np), h = (int)(e / np % H);
-  const int64_t row = e / np / H;
-  const TS* s = src + row * lds + h * hs + 2 * i;
-  TA* d = dst + row * ldd + h * hd + 2 * i;
-  const bool two = 2 * i + 1 < rot;
-  float u = act_load(s), v = two ? act_load(s + 1) : 0.f;
-  if (i < half) {
-    const float2 c = cs[row * half + i];
-    const float x = u * c.x - v * c.y;
-    v = v * c.x + u * c.y;
-    u = x;
-  }
-  act_store(d, u);
-  if (two) act_store(d + 1, v);
 }
 
 // ---- page rows, gathered -----------------------------------------------------------------------
@@ -537,13 +497,6 @@ int launch_heads(const HeadArgs& a, cudaStream_t st) {
 
 CB_EXPORT int cb_latent_args_size() { return (int)sizeof(LatentArgs); }
 
-// (cos, sin) of position * turns[i] turns, for `rows` rows: cs [rows, half, 2] fp32; turns fp64 [half].
-CB_EXPORT int cb_rope_rows(const void* positions, const void* turns, void* cs, int64_t rows, int64_t half, void* stream) {
-  if (!positions || !turns || !cs || rows < 1 || half < 1 || rows * half > (int64_t)1 << 30) return CB_ERR_ARG;
-  return (int)cb_launch(rope_rows_kernel, dim3((unsigned)((rows * half + 255) / 256)), dim3(256), 0, (cudaStream_t)stream,
-                        (const int*)positions, (const double*)turns, (float2*)cs, (int)rows, (int)half);
-}
-
 // `rows` projection rows: cq = rmsnorm(query latent), or the rotated query parts turned (q_rank 0); with own != 0 also
 // rmsnorm(c) and the rotated part into the pages.
 // p_f32: projection rows are fp32; f32: latents and pages are fp32 instead of bf16.
@@ -560,19 +513,6 @@ CB_EXPORT int cb_latent_rows(const void* args, int64_t rows, int64_t own, int64_
   if (f32) return (int)cb_launch(latent_rows_kernel<float, float>, grid, block, 0, st, a);
   if (p_f32) return (int)cb_launch(latent_rows_kernel<float, bf16>, grid, block, 0, st, a);
   return (int)cb_launch(latent_rows_kernel<bf16, bf16>, grid, block, 0, st, a);
-}
-
-// Rotated parts of `H` heads: dst[t, h] = rotate(src[t, h]) (row strides lds / ldd, head strides hs / hd); may be in place.
-CB_EXPORT int cb_rope_heads(const void* src, int64_t lds, int64_t hs, void* dst, int64_t ldd, int64_t hd, const void* cs, int64_t half,
-                            int64_t rot, int64_t H, int64_t rows, int64_t f32, void* stream) {
-  if (!src || !dst || rows < 1 || H < 1 || rot < 1 || 2 * half > rot || (half && !cs)) return CB_ERR_ARG;
-  const dim3 grid((unsigned)((rows * H * ((rot + 1) / 2) + 255) / 256)), block(256);
-  cudaStream_t st = (cudaStream_t)stream;
-  if (f32)
-    return (int)cb_launch(rope_heads_kernel<float, float>, grid, block, 0, st, (const float*)src, lds, hs, (float*)dst, ldd, hd,
-                          (const float2*)cs, (int)half, (int)rot, (int)H, (int)rows);
-  return (int)cb_launch(rope_heads_kernel<bf16, bf16>, grid, block, 0, st, (const bf16*)src, lds, hs, (bf16*)dst, ldd, hd,
-                        (const float2*)cs, (int)half, (int)rot, (int)H, (int)rows);
 }
 
 // Page rows of `segs` sequences side by side: segment s fills rows base[s] .. base[s] + whole pages of lens[s] tokens, from

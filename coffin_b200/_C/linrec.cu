@@ -8,6 +8,9 @@
 //              S <- exp(f + m' - m) S + exp(i - m) k v^T;  n likewise with k;
 //              o = S^T q / (max(|n.q|, exp(-m)) + 1e-6)
 //            o is RMS-normed per head, weighted and multiplied by a sigmoid gate.
+//   gated  : the forget gate f of a key channel (sigmoid above a lower bound) also decides what is written,
+//              S <- f * S + (1 - f) v^T;  o = S^T silu(q)
+//            o is RMS-normed per head and weighted.
 //
 // One cluster of CTAs per (head, sequence): every CTA owns `jc` value columns of the head's state in registers
 // (the columns of S never interact), computes the head's q / k / decays itself, and only the RMS norm over the
@@ -111,7 +114,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
   const int dk = a.dk, dv = a.dv, jc = a.jc;
   float* sq = sm;                                      // [dk]
   float* sk = sq + dk;                                 // [dk]
-  float* sg = sk + dk;                                 // [dk] decays (delta) / n (mLSTM)
+  float* sg = sk + dk;                                 // [dk] decays (delta, gated) / n (mLSTM)
   float* sv = sg + dk;                                 // [jc]
   float* su = sv + jc;                                 // [jc]
   float* so = su + jc;                                 // [jc]
@@ -138,6 +141,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
   };
   float p_dt = 0.f, p_ea = 0.f, p_bi = 0.f, p_bf = 0.f;
   if (KIND == LINREC_MLSTM) { p_bi = a.gate_b[h]; p_bf = a.gate_b[a.H + h]; }
+  if (KIND == LINREC_GATED && tid < dk) { p_bf = a.gate_b[(int64_t)h * dk + tid]; p_bi = a.lower[(int64_t)h * dk + tid]; }
   if (KIND == LINREC_DELTA) {
 #pragma unroll
     for (int u = 0; u < 2; ++u)
@@ -189,10 +193,16 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     // what channel `tid` needs from this row, requested together
     float x_a = 0.f, x_b = 0.f, x_v = 0.f, x_og = 0.f;
     const int64_t vch = (int64_t)h * dv + j0 + tid;
-    const float gate0 = a.gates[row * a.ldg + h], gate1 = KIND == LINREC_MLSTM ? a.gates[row * a.ldg + a.H + h] : 0.f;
+    const float gate0 = KIND == LINREC_GATED ? 0.f : a.gates[row * a.ldg + h], gate1 = KIND == LINREC_MLSTM ? a.gates[row * a.ldg + a.H + h] : 0.f;
     if (KIND == LINREC_DELTA) {
       if (tid < dk && a.dec) x_a = a.dec[row * a.ldd + (int64_t)h * dk + tid];
       if (tid < ncol && a.og) x_og = act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + vch);
+    } else if (KIND == LINREC_GATED) {
+      if (tid < dk) {
+        x_a = act_load(pr + (int64_t)h * dk + tid);
+        x_b = a.gates[row * a.ldg + (int64_t)h * dk + tid];
+      }
+      if (tid < ncol) x_v = act_load(pr + a.v_col + vch);
     } else {
       if (tid < dk) {
         x_a = act_load(pr + (int64_t)h * dk + tid);
@@ -267,6 +277,14 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
         const float x = !LOW || a.og ? (c == tid ? x_og : act_load(reinterpret_cast<const TA*>(a.og) + row * a.ldo + ch)) : (low_g ? sog[c] : row_dot(g2 + ch * a.rg, lg, a.rg));
         sog[c] = sigmoid_s(x);
       }
+    } else if (KIND == LINREC_GATED) {
+      for (int c = tid; c < dk; c += kT) {
+        const int64_t ch = (int64_t)h * dk + c;
+        const bool own = c == tid;
+        sq[c] = silu_x(own ? x_a : act_load(pr + ch));
+        sg[c] = forget((own ? x_b : a.gates[row * a.ldg + ch]) + (own ? p_bf : a.gate_b[ch]), own ? p_bi : a.lower[ch], sk + c);
+      }
+      for (int c = tid; c < ncol; c += kT) sv[c] = c == tid ? x_v : act_load(pr + a.v_col + (int64_t)h * dv + j0 + c);
     } else {
       const float rs = 1.f / sqrtf((float)dk);
       const float zi = gate0 + p_bi, zf = gate1 + p_bf;
@@ -297,7 +315,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     __syncthreads();
     // ---- state pass: partial sums of the read-outs over this thread's rows
     float pa[4] = {}, pb[4] = {};
-    if (KIND == LINREC_MLSTM) {
+    if (KIND != LINREC_DELTA) {
       float v4[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) v4[e] = q4 * 4 + e < ncol ? sv[q4 * 4 + e] : 0.f;
@@ -305,10 +323,10 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
       for (int i = 0; i < RMAX; ++i) {
         const int r = rg + i * RG;
         if (i < nr) {
-          const float k = sk[r], q = sq[r];
+          const float k = sk[r], q = sq[r], g = KIND == LINREC_GATED ? sg[r] : aa;
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            S[i][e] = fmaf(aa, S[i][e], k * v4[e]);
+            S[i][e] = fmaf(g, S[i][e], k * v4[e]);
             pb[e] = fmaf(S[i][e], q, pb[e]);
           }
         }
@@ -384,7 +402,7 @@ __global__ void __launch_bounds__(kT, RMAX <= 4 && !LOW ? 3 : (RMAX <= 16 ? 2 : 
     }
     const float rstd = 1.f / sqrtf(ss / (float)dv + a.eps);
     TA* out = reinterpret_cast<TA*>(a.act) + row * a.lda + (int64_t)h * dv + j0;
-    for (int c = tid; c < ncol; c += kT) act_store(out + c, so[c] * rstd * (c == tid ? p_nw : nw[c]) * sog[c]);
+    for (int c = tid; c < ncol; c += kT) act_store(out + c, so[c] * rstd * (c == tid ? p_nw : nw[c]) * (KIND == LINREC_GATED ? 1.f : sog[c]));
     __syncthreads();
   }
   // ---- state back
@@ -519,6 +537,11 @@ CB_EXPORT int cb_linrec_step(const void* args, int64_t kind, int64_t segs, int64
     if (!a.n || !a.m || !a.og || !(a.cap > 0.f)) return CB_ERR_ARG;
     if (f32) return dispatch_step<LINREC_MLSTM, float, float>(a, (int)segs, st);
     return p_f32 ? dispatch_step<LINREC_MLSTM, float, bf16>(a, (int)segs, st) : dispatch_step<LINREC_MLSTM, bf16, bf16>(a, (int)segs, st);
+  }
+  if (kind == LINREC_GATED) {
+    if (!a.gate_b || !a.lower || !a.norm_w || a.G != a.H) return CB_ERR_ARG;
+    if (f32) return dispatch_step<LINREC_GATED, float, float>(a, (int)segs, st);
+    return p_f32 ? dispatch_step<LINREC_GATED, float, bf16>(a, (int)segs, st) : dispatch_step<LINREC_GATED, bf16, bf16>(a, (int)segs, st);
   }
   return CB_ERR_ARG;
 }

@@ -8,6 +8,7 @@
 //            T = (I + diag(beta) A)^-1 diag(beta),  A_ts = sum_c k_t k_s G_t / G_s  (s < t)
 //   mLSTM :  u = v and the same with scalar decays under the running maximum; its normaliser n is one more value
 //            column, v = 1.
+//   gated :  u = v, k = 1 - f, decays per channel, no normaliser.
 //
 // `prep` (one CTA per chunk and head) computes those factors in fp32; `scan` (two warps per 16 value columns) walks
 // the chunks with S^T in accumulator registers.  The 32-bit quantities enter the products as a bf16 head plus a bf16
@@ -31,7 +32,7 @@ struct ChunkArgs {
 };
 
 // operand block, bf16 units, row pitch P = DK + 8:  X head [NX][P] | X remainder | K^ head [16][P] | K^ remainder |
-// T head [16][24] | T remainder | B head | B remainder | G fp32 [DK].   NX = 32 (k~ then q~) for delta, 16 (q~) for mLSTM.
+// T head [16][24] | T remainder | B head | B remainder | G fp32 [DK].   NX = 32 (k~ then q~) for delta, else 16 (q~).
 template <int KIND, int DK> struct Image {
   static constexpr int P = DK + 8, NX = KIND == LINREC_DELTA ? 32 : 16;
   static constexpr int xh = 0, xl = xh + NX * P, kh = xl + NX * P, kl = kh + C * P, th = kl + C * P, tl = th + C * 24, bh = tl + C * 24,
@@ -365,6 +366,88 @@ __global__ void __launch_bounds__(64) chunk_prep_mlstm_kernel(const ChunkArgs ca
   }
 }
 
+// ---- prep: gated --------------------------------------------------------------------------------
+// Decays below 2^-60 a token are cut off there: the state is an average of values, so what they would leave is far below its
+// rounding, and cumulative logarithms stay short enough to subtract.
+template <int DK>
+__global__ void __launch_bounds__(kPT, 7) chunk_prep_gated_kernel(const ChunkArgs ca) {
+  using I = Image<LINREC_GATED, DK>;
+  constexpr int LD = DK + 4;
+  const LinrecArgs& a = ca.r;
+  extern __shared__ __align__(16) float sm[];
+  float* sq = sm;                    // [C][LD]
+  float* sk = sq + C * LD;
+  float* sL = sk + C * LD;           // cumulative log2 decays, inclusive
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.y, seg = blockIdx.z;
+  griddep_launch();
+  griddep_wait();
+  const int row0 = a.seg_row[seg], n = a.seg_row[seg + 1] - row0, slot = a.seg_slot[seg];
+  const int c0 = blockIdx.x * C;
+  if (c0 >= n || slot < 0) return;
+  const int m = min(C, n - c0);
+  const bf16* proj = reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + c0) * a.ldp + (int64_t)h * a.dk;
+  const float* gates = a.gates + (int64_t)(row0 + c0) * a.ldg + (int64_t)h * a.dk;
+  bf16* im = reinterpret_cast<bf16*>(ca.image + (block_index(row0, seg, blockIdx.x) * a.H + h) * I::bytes);
+  // a channel per thread; channels beyond dk and tokens beyond the segment are neutral and empty
+  for (int c = tid; c < DK; c += kPT) {
+    const bool ok = c < a.dk;
+    const float low = ok ? a.lower[(int64_t)h * a.dk + c] : 0.f, bias = ok ? a.gate_b[(int64_t)h * a.dk + c] : 0.f;
+    float z[C], q[C], L = 0.f;
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      z[t] = ok && t < m ? gates[(int64_t)t * a.ldg + c] : 0.f;
+      q[t] = ok && t < m ? __bfloat162float(proj[(int64_t)t * a.ldp + c]) : 0.f;
+    }
+#pragma unroll
+    for (int t = 0; t < C; ++t) {
+      float in = 0.f;
+      if (ok && t < m) L += fmaxf(log2f(forget(z[t] + bias, low, &in)), -60.f);
+      sq[t * LD + c] = silu_s(q[t]);
+      sk[t * LD + c] = in;
+      sL[t * LD + c] = L;
+    }
+    reinterpret_cast<float*>(im + I::g)[c] = ex2(L);
+  }
+  __syncthreads();
+  for (int e = tid; e < C * (DK / 2); e += kPT) {
+    const int t = e / (DK / 2), c = (e % (DK / 2)) * 2, i = t * LD + c, l = (C - 1) * LD + c;
+    put2(im + I::xh + t * I::P + c, im + I::xl + t * I::P + c, sq[i] * ex2(sL[i]), sq[i + 1] * ex2(sL[i + 1]));
+    put2(im + I::kh + t * I::P + c, im + I::kl + t * I::P + c, sk[i] * ex2(sL[l] - sL[i]), sk[i + 1] * ex2(sL[l + 1] - sL[i + 1]));
+  }
+  // pairwise products: a warp takes tokens t = warp, 7 - warp, 8 + warp, 15 - warp (equal numbers of pairs)
+#pragma unroll 1
+  for (int i = 0; i < 4; ++i) {
+    const int t = i == 0 ? warp : (i == 1 ? 7 - warp : (i == 2 ? 8 + warp : 15 - warp));
+    float qt[DK / 32], Lt[DK / 32];
+#pragma unroll
+    for (int j = 0; j < DK / 32; ++j) { qt[j] = sq[t * LD + lane + 32 * j]; Lt[j] = sL[t * LD + lane + 32 * j]; }
+#pragma unroll 1
+    for (int s = 0; s <= t; s += 4) {                            // four tokens s share the reduction tree; those after t are discarded
+      float p[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int j = 0; j < DK / 32; ++j) {
+          const int at = (s + u) * LD + lane + 32 * j;
+          p[u] = fmaf(qt[j], sk[at] * ex2(fminf(Lt[j] - sL[at], 0.f)), p[u]);
+        }
+      const bool hi = lane & 16, hq = lane & 8;                  // halves of the warp keep tokens 0, 1 / 2, 3, quarters one of them
+      float x = hi ? p[2] : p[0], y = hi ? p[3] : p[1];
+      x += __shfl_xor_sync(0xffffffffu, hi ? p[0] : p[2], 16);
+      y += __shfl_xor_sync(0xffffffffu, hi ? p[1] : p[3], 16);
+      float k = hq ? y : x;
+      k += __shfl_xor_sync(0xffffffffu, hq ? x : y, 8);
+      k += __shfl_xor_sync(0xffffffffu, k, 4);
+      k += __shfl_xor_sync(0xffffffffu, k, 2);
+      k += __shfl_xor_sync(0xffffffffu, k, 1);
+      const int su = s + (hi ? 2 : 0) + (hq ? 1 : 0);
+      if ((lane & 7) == 0 && su <= t) put1(im + I::bh + t * 24 + su, im + I::bl + t * 24 + su, k);
+    }
+    if (lane > t && lane < C) put1(im + I::bh + t * 24 + lane, im + I::bl + t * 24 + lane, 0.f);
+  }
+}
+
 // ---- scan ---------------------------------------------------------------------------------------
 // A CTA owns 32 value columns of a head: two column groups of 16, each shared by two warps that hold half of the key
 // channels.  The halves' partial read-outs meet in shared memory once per chunk; both then know u and update their half
@@ -587,7 +670,7 @@ __global__ void __launch_bounds__(128) chunk_finish_kernel(const ChunkArgs ca, i
   const int64_t row = w / a.H;
   const int h = (int)(w % a.H);
   const float* o = ca.o + row * ca.ldo_ + (int64_t)h * a.dv;
-  const bf16* og = reinterpret_cast<const bf16*>(a.og) + row * a.ldo + (int64_t)h * a.dv;
+  const bf16* og = KIND == LINREC_GATED ? nullptr : reinterpret_cast<const bf16*>(a.og) + row * a.ldo + (int64_t)h * a.dv;
   const float* nw = a.norm_w + (KIND == LINREC_MLSTM ? (int64_t)h * a.dv : 0);
   float inv = 1.f;
   if (KIND == LINREC_MLSTM) inv = 1.f / (fmaxf(fabsf(ca.nq[row * a.H + h]), expf(-ca.gm[row * a.H + h])) + 1e-6f);
@@ -606,7 +689,12 @@ __global__ void __launch_bounds__(128) chunk_finish_kernel(const ChunkArgs ca, i
   for (int i = 0; i < kVMax / 4; ++i) {
     const int c = 4 * (lane + 32 * i);
     if (c < a.dv) {
-      const float4 gt = act_load4(og + c), w4 = *reinterpret_cast<const float4*>(nw + c);
+      const float4 w4 = *reinterpret_cast<const float4*>(nw + c);
+      if (KIND == LINREC_GATED) {
+        act_store4(out + c, make_float4(x[i].x * r * w4.x, x[i].y * r * w4.y, x[i].z * r * w4.z, x[i].w * r * w4.w));
+        continue;
+      }
+      const float4 gt = act_load4(og + c);
       act_store4(out + c, make_float4(x[i].x * r * w4.x * sigmoid_s(gt.x), x[i].y * r * w4.y * sigmoid_s(gt.y),
                                       x[i].z * r * w4.z * sigmoid_s(gt.z), x[i].w * r * w4.w * sigmoid_s(gt.w)));
     }
@@ -631,6 +719,12 @@ int run_chunks(const ChunkArgs& ca, int max_rows, int rows, cudaStream_t st) {
   }
     if (a.taps == 4) CB_PREP(4) else CB_PREP(0)
 #undef CB_PREP
+    if (e != cudaSuccess) return (int)e;
+  } else if (KIND == LINREC_GATED) {
+    const size_t smem = sizeof(float) * 3 * C * (DK + 4);
+    auto kern = chunk_prep_gated_kernel<DK>;
+    if (smem > 40 * 1024 && (e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) != cudaSuccess) return (int)e;
+    e = cb_launch(kern, dim3((unsigned)chunks, (unsigned)a.H, (unsigned)ca.segs), dim3(kPT), smem, st, ca);
     if (e != cudaSuccess) return (int)e;
   } else {
     e = cb_launch(chunk_gates_mlstm_kernel, dim3((unsigned)a.H, (unsigned)ca.segs), dim3(kGT), 0, st, ca);
@@ -678,10 +772,12 @@ CB_EXPORT int cb_linrec_chunk(const void* args, int64_t kind, int64_t segs, int6
   ChunkArgs ca;
   ca.r = *(const LinrecArgs*)args;
   const LinrecArgs& a = ca.r;
-  if (!a.proj || !a.gates || !a.act || !a.og || !a.seg_row || !a.seg_pos || !a.seg_slot || !a.S || a.H < 1 || a.G < 1 || a.H % a.G)
+  if (!a.proj || !a.gates || !a.act || (!a.og && kind != LINREC_GATED) || !a.seg_row || !a.seg_pos || !a.seg_slot || !a.S || a.H < 1 || a.G < 1 || a.H % a.G)
     return CB_ERR_ARG;
   if (!cb_linrec_chunk_ok(a.dk, a.dv) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || a.lda % 4 || a.ldo % 4) return CB_ERR_SHAPE;
-  if (kind == LINREC_DELTA ? (!a.dec || !a.ring || a.taps < 1 || a.taps > a.ring_mask + 1) : (!a.n || !a.m || !(a.cap > 0.f))) return CB_ERR_ARG;
+  if (kind == LINREC_DELTA && (!a.dec || !a.ring || a.taps < 1 || a.taps > a.ring_mask + 1)) return CB_ERR_ARG;
+  if (kind == LINREC_MLSTM && (!a.n || !a.m || !(a.cap > 0.f))) return CB_ERR_ARG;
+  if (kind == LINREC_GATED && (!a.gate_b || !a.lower || !a.norm_w || a.G != a.H)) return CB_ERR_ARG;
   if (scratch_bytes < cb_linrec_chunk_scratch(kind, rows, segs, a.H, a.dk, a.dv)) return CB_ERR_ARG;
   unsigned char* p = (unsigned char*)scratch;
   ca.image = p; p += al((rows / C + segs + 2) * a.H * image_bytes(kind, a.dk));
@@ -702,6 +798,7 @@ CB_EXPORT int cb_linrec_chunk(const void* args, int64_t kind, int64_t segs, int6
   }
   if (kind == LINREC_DELTA) { CB_RUN(LINREC_DELTA) }
   if (kind == LINREC_MLSTM) { CB_RUN(LINREC_MLSTM) }
+  if (kind == LINREC_GATED) { CB_RUN(LINREC_GATED) }
 #undef CB_RUN
   return CB_ERR_ARG;
 }

@@ -2,7 +2,8 @@
 //
 // The boundary adds what the sublayer left - a dense row, or the weighted expert rows of a routed feed-forward found
 // through their sorted positions plus a multiple of the sublayer's own input (experts that return their input) - and
-// leaves the RMS-normalised row for the next projection.  A row crosses HBM once per sublayer and its sum is never rounded.
+// leaves the RMS-normalised row for the next projection.  What is added may be RMS-normed with a gain of its own first (a norm
+// behind every sublayer), and the token's embedding may be added with it (layers that run again).  A row crosses HBM once per sublayer and its sum is never rounded.
 // Residuals of several streams and depth averages are streams.cu's and depth.cu's.
 #include "act_type.cuh"
 
@@ -19,6 +20,8 @@ struct ResidualArgs {
   const void* hin; int64_t ldhin;        // that input (may be the rows h is written to)
   const float* gain; void* h; int64_t ldh;
   const int* rows;                       // residual row behind output row i (null: i)
+  const float* post;                     // gain of the norm over what is added, or null
+  const void* embed; const int64_t* tokens; int64_t vocab;   // table and tokens of the rows, or null
   int W; float eps; int store;
 };
 
@@ -36,7 +39,7 @@ template <typename TA> struct Vec<TA, 1> {
 };
 
 // V columns per access, up to IT accesses per thread; the row stays in registers between the sum and the norm.
-template <typename TA, int V, int IT>
+template <typename TA, int V, int IT, bool POST>
 __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualArgs a) {
   __shared__ float red[32];
   __shared__ int pos_s[kMaxSlots];
@@ -55,7 +58,12 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualArgs 
   const TA* hin = reinterpret_cast<const TA*>(a.hin) + r * a.ldhin;
   const TA* ys = reinterpret_cast<const TA*>(a.ys);
   const float idw = a.idw ? a.idw[r] : 0.f;
-  float u[IT][V], ss = 0.f;
+  const TA* er = nullptr;
+  if (POST && a.embed) {
+    const int64_t tok = a.tokens[r];
+    er = reinterpret_cast<const TA*>(a.embed) + (tok < 0 ? 0 : (tok >= a.vocab ? a.vocab - 1 : tok)) * a.W;
+  }
+  float u[IT][V], add[POST ? IT : 1][V], ss = 0.f, sa = 0.f;
 #pragma unroll
   for (int t = 0; t < IT; ++t) {
     const int i = (tid + t * NT) * V;
@@ -63,7 +71,8 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualArgs 
     for (int v = 0; v < V; ++v) u[t][v] = 0.f;
     if (i >= a.W) continue;
     Vec<float, V>::load(xr + i, u[t]);
-    float s[V], f[V];
+    float* s = add[POST ? t : 0];
+    float f[V];
 #pragma unroll
     for (int v = 0; v < V; ++v) s[v] = 0.f;
     if (y) Vec<TA, V>::load(y + i, s);
@@ -81,6 +90,11 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualArgs 
 #pragma unroll
       for (int v = 0; v < V; ++v) s[v] = fmaf(idw, f[v], s[v]);
     }
+    if (POST) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) sa = fmaf(s[v], s[v], sa);
+      continue;
+    }
     if (y || ys) {
 #pragma unroll
       for (int v = 0; v < V; ++v) u[t][v] += s[v];
@@ -88,6 +102,28 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualArgs 
     }
 #pragma unroll
     for (int v = 0; v < V; ++v) ss = fmaf(u[t][v], u[t][v], ss);
+  }
+  if (POST) {
+    const float ra = a.post ? 1.f / sqrtf(block_sum(sa, red) / (float)a.W + a.eps) : 1.f;
+#pragma unroll
+    for (int t = 0; t < IT; ++t) {
+      const int i = (tid + t * NT) * V;
+      if (i >= a.W) continue;
+      float g[V];
+#pragma unroll
+      for (int v = 0; v < V; ++v) g[v] = 1.f;
+      if (a.post) Vec<float, V>::load(a.post + i, g);
+#pragma unroll
+      for (int v = 0; v < V; ++v) u[t][v] = fmaf(add[t][v], g[v] * ra, u[t][v]);
+      if (er) {
+        Vec<TA, V>::load(er + i, g);
+#pragma unroll
+        for (int v = 0; v < V; ++v) u[t][v] += g[v];
+      }
+      if (a.store) Vec<float, V>::store(xr + i, u[t]);
+#pragma unroll
+      for (int v = 0; v < V; ++v) ss = fmaf(u[t][v], u[t][v], ss);
+    }
   }
   if (!a.h) return;
   const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)a.W + a.eps);
@@ -115,38 +151,44 @@ __global__ void __launch_bounds__(256) residual_embed_kernel(const TA* __restric
   for (int i = threadIdx.x; i < W; i += 256) x[r * W + i] = act_load(embed + tok * W + i) * scale;
 }
 
-template <typename TA>
+template <typename TA, bool POST>
 int step_launch(const ResidualArgs& a, int64_t n, cudaStream_t st) {
   const bool v4 = a.W % 4 == 0 && a.ldh % 4 == 0 && a.ldy % 4 == 0 && a.ldys % 4 == 0 && a.ldhin % 4 == 0;
   const int per = v4 ? (a.W + 3) / 4 : a.W;
   const int nt = per >= 1024 ? 1024 : (per + 31) / 32 * 32;
   const dim3 grid((unsigned)n), block((unsigned)nt);
   if (v4) {
-    if (per <= nt) return (int)cb_launch(residual_step_kernel<TA, 4, 1>, grid, block, 0, st, a);
-    if (per <= 2 * nt) return (int)cb_launch(residual_step_kernel<TA, 4, 2>, grid, block, 0, st, a);
-    if (per <= 4 * nt) return (int)cb_launch(residual_step_kernel<TA, 4, 4>, grid, block, 0, st, a);
+    if (per <= nt) return (int)cb_launch(residual_step_kernel<TA, 4, 1, POST>, grid, block, 0, st, a);
+    if (per <= 2 * nt) return (int)cb_launch(residual_step_kernel<TA, 4, 2, POST>, grid, block, 0, st, a);
+    if (per <= 4 * nt) return (int)cb_launch(residual_step_kernel<TA, 4, 4, POST>, grid, block, 0, st, a);
     return CB_ERR_SHAPE;
   }
-  if (per <= 4 * nt) return (int)cb_launch(residual_step_kernel<TA, 1, 4>, grid, block, 0, st, a);
-  if (per <= 16 * nt) return (int)cb_launch(residual_step_kernel<TA, 1, 16>, grid, block, 0, st, a);
+  if (per <= 4 * nt) return (int)cb_launch(residual_step_kernel<TA, 1, 4, POST>, grid, block, 0, st, a);
+  if (per <= 16 * nt) return (int)cb_launch(residual_step_kernel<TA, 1, 16, POST>, grid, block, 0, st, a);
   return CB_ERR_SHAPE;
 }
 
 }  // namespace
 
 // One sublayer boundary over `n` rows of x [.., W]: x += y (y null: nothing) + sum_j w[r, j] ys[pos[r, j]] (ys null: nothing)
-// + idw[r] hin[r] (idw null: nothing); then h = rmsnorm(x) * gain (h null: no norm).  rows (int32 [n], optional): residual
+// + idw[r] hin[r] (idw null: nothing), the sum of the added terms RMS-normed and multiplied by post first (post null: not), and
+// embed[token[r]] (embed null: nothing); then h = rmsnorm(x) * gain (h null: no norm).  rows (int32 [n], optional): residual
 // row behind output row i (with store 0: x is left as it is).  f32: activations are fp32 instead of bf16.  W <= 16384.
 CB_EXPORT int cb_residual_step(void* x, const void* y, int64_t ldy, const void* ys, int64_t ldys, const void* pos, const void* w, int64_t k,
                                const void* idw, const void* hin, int64_t ldhin, const void* gain, void* h, int64_t ldh, const void* rows,
-                               int64_t n, int64_t W, float eps, int64_t store, int64_t f32, void* stream) {
+                               int64_t n, int64_t W, float eps, int64_t store, const void* post, const void* embed, const void* tokens,
+                               int64_t vocab, int64_t f32, void* stream) {
   if (!x || n < 1 || W < 1 || (h && !gain) || (rows && store)) return CB_ERR_ARG;
+  if ((post && !y && !ys) || (embed && (!tokens || vocab < 1))) return CB_ERR_ARG;
   if ((ys && (!pos || !w || k < 1 || k > kMaxSlots)) || (idw && !hin)) return CB_ERR_ARG;
   ResidualArgs a;
   a.x = (float*)x; a.y = y; a.ldy = ldy; a.ys = ys; a.ldys = ldys; a.pos = (const int*)pos; a.w = (const float*)w; a.k = (int)k;
   a.idw = (const float*)idw; a.hin = hin; a.ldhin = ldhin; a.gain = (const float*)gain; a.h = h; a.ldh = ldh; a.rows = (const int*)rows;
   a.W = (int)W; a.eps = eps; a.store = (int)store;
-  return f32 ? step_launch<float>(a, n, (cudaStream_t)stream) : step_launch<bf16>(a, n, (cudaStream_t)stream);
+  a.post = (const float*)post; a.embed = embed; a.tokens = (const int64_t*)tokens; a.vocab = vocab;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (post || embed) return f32 ? step_launch<float, true>(a, n, st) : step_launch<bf16, true>(a, n, st);
+  return f32 ? step_launch<float, false>(a, n, st) : step_launch<bf16, false>(a, n, st);
 }
 
 // x[t] = embed[token[t]] * scale

@@ -3,7 +3,8 @@
 //
 // The router's logits cover `experts` stored experts and, behind them, `identity` ones without weights.  Scores are their
 // softmax; the `top` largest of score + correction are chosen; a chosen output weighs score / (sum of the chosen scores +
-// 1e-20) * scale.  A token's slots are its `top` choices and then `always` further stored experts (the parts of a shared
+// 1e-20) * scale.  With by_logit the correction is part of the logits: the largest of logit + correction are chosen, and weigh
+// their softmax over the chosen ones, times scale.  A token's slots are its `top` choices and then `always` further stored experts (the parts of a shared
 // expert) with weight one.  A slot that chose an identity expert holds no expert (-1); its weight goes to idw, a multiple
 // of the token's input.  All of it is fp32.
 //
@@ -23,6 +24,7 @@ struct RouteArgs {
   int T, experts, identity, top, always;
   float scale;
   int* idx; float* w; float* idw;        // [T, top + always], [T, top + always], [T]
+  int by_logit;
 };
 
 // unsigned integers in the order of the floats
@@ -43,6 +45,10 @@ __device__ __forceinline__ int route_row(const RouteArgs& a, const float* row, i
     const int e = lane + 32 * i;
     s[i] = e < n ? row[e] : -INFINITY;
     c[i] = e < n ? __float_as_uint(a.corr[e]) : 0u;
+    if (a.by_logit && e < n) {
+      s[i] += __uint_as_float(c[i]);
+      c[i] = order_key(s[i]);
+    }
   }
 #pragma unroll
   for (int i = 0; i < PER; ++i) mx = fmaxf(mx, s[i]);
@@ -56,7 +62,7 @@ __device__ __forceinline__ int route_row(const RouteArgs& a, const float* row, i
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     s[i] *= inv;
-    c[i] = lane + 32 * i < n ? order_key(s[i] + __uint_as_float(c[i])) : 0u;      // 0: below every number
+    if (!a.by_logit) c[i] = lane + 32 * i < n ? order_key(s[i] + __uint_as_float(c[i])) : 0u;      // 0: below every number
   }
   float my = 0.f, chosen = 0.f;
   int mine = -1;
@@ -230,12 +236,13 @@ __global__ void __launch_bounds__(32 * kOut * kSlices) routed_step_kernel(const 
   route_units<PER>(a, u, sm, true);
 }
 
-// y[r] = act(W[expert] x[r or src[r]]) over units of up to 8 rows, true fp32: a warp per output column.
+// y[r] = act(W[expert] x[r or src[r]]) over units of up to 8 rows, true fp32: a warp per output column.  act 2: squared relu;
+// 3: silu(gate) * up, an expert's N gate rows before its N up rows.
 __global__ void __launch_bounds__(256) routed_linear_f32_kernel(const float* __restrict__ W, int64_t stride, const float* __restrict__ x,
                                                                 int64_t ldx, float* __restrict__ y, int64_t ldy, int N, int K,
                                                                 const int* __restrict__ count, const int* __restrict__ row0,
                                                                 const int* __restrict__ rows, const int* __restrict__ expert,
-                                                                const int* __restrict__ src, int relu2) {
+                                                                const int* __restrict__ src, int act) {
   griddep_launch();
   griddep_wait();
   const int n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -248,14 +255,21 @@ __global__ void __launch_bounds__(256) routed_linear_f32_kernel(const float* __r
       float s = 0.f;
       for (int k = lane; k < K; k += 32) s = fmaf(w[k], xr[k], s);
       s = warp_sum(s);
-      if (relu2) { s = fmaxf(s, 0.f); s *= s; }
+      if (act == 2) { s = fmaxf(s, 0.f); s *= s; }
+      if (act == 3) {
+        const float* wu = w + (int64_t)N * K;
+        float u = 0.f;
+        for (int k = lane; k < K; k += 32) u = fmaf(wu[k], xr[k], u);
+        s = silu_x(s) * warp_sum(u);
+      }
       if (lane == 0) y[(int64_t)(r0 + i) * ldy + n] = s;
     }
   }
 }
 
 int route_args(RouteArgs* a, const void* logits, int64_t ldl, const void* corr, const void* positions, int64_t T, int64_t experts,
-               int64_t identity, int64_t top, int64_t always, float scale, void* idx, void* w, void* idw) {
+               int64_t identity, int64_t top, int64_t always, float scale, int64_t by_logit, void* idx, void* w, void* idw) {
+  a->by_logit = (int)by_logit;
   if (!logits || !corr || !idx || !w || !idw || T < 1 || experts < 1 || identity < 0 || always < 0) return CB_ERR_ARG;
   if (experts + identity > kMaxOut || top < 1 || top > kMaxTop || top > experts + identity || always > kMaxTop) return CB_ERR_SHAPE;
   a->logits = (const float*)logits; a->ldl = ldl; a->corr = (const float*)corr; a->positions = (const int*)positions;
@@ -287,9 +301,10 @@ int launch_units(const RouteArgs& a, const UnitList& u, const RouterProduct* p, 
 
 // Slots of `T` rows: idx / w [T, top + always] (idx -1: no stored expert), idw [T].
 CB_EXPORT int cb_routed_topk(const void* logits, int64_t ldl, const void* corr, const void* positions, int64_t T, int64_t experts,
-                             int64_t identity, int64_t top, int64_t always, float scale, void* idx, void* w, void* idw, void* stream) {
+                             int64_t identity, int64_t top, int64_t always, float scale, int64_t by_logit, void* idx, void* w, void* idw,
+                             void* stream) {
   RouteArgs a;
-  const int rc = route_args(&a, logits, ldl, corr, positions, T, experts, identity, top, always, scale, idx, w, idw);
+  const int rc = route_args(&a, logits, ldl, corr, positions, T, experts, identity, top, always, scale, by_logit, idx, w, idw);
   if (rc) return rc;
 #define CB_TOPK(N) (int)cb_launch(routed_topk_kernel<N>, dim3((unsigned)((T + 3) / 4)), dim3(128), 0, (cudaStream_t)stream, a)
   CB_PER(CB_TOPK);
@@ -299,11 +314,11 @@ CB_EXPORT int cb_routed_topk(const void* logits, int64_t ldl, const void* corr, 
 // The same for T <= 64 rows, with the sorted order (pos [T * slots], src [T * slots]) and the units of up to 8 rows of an expert.
 // router / h / ticket given (T <= 8, bf16): logits = router h^T first, by the same launch; ticket: a zeroed counter.
 CB_EXPORT int cb_routed_units(const void* logits, int64_t ldl, const void* corr, const void* positions, int64_t T, int64_t experts,
-                              int64_t identity, int64_t top, int64_t always, float scale, void* idx, void* w, void* idw, void* pos,
+                              int64_t identity, int64_t top, int64_t always, float scale, int64_t by_logit, void* idx, void* w, void* idw, void* pos,
                               void* src, void* count, void* row0, void* rows, void* expert, int64_t max_units, const void* router,
                               const void* h, int64_t ldh, int64_t K, void* ticket, void* stream) {
   RouteArgs a;
-  const int rc = route_args(&a, logits, ldl, corr, positions, T, experts, identity, top, always, scale, idx, w, idw);
+  const int rc = route_args(&a, logits, ldl, corr, positions, T, experts, identity, top, always, scale, by_logit, idx, w, idw);
   if (rc) return rc;
   if (T > kMaxRows || units_smem(a, router ? 8 : 0) > 44 * 1024) return CB_ERR_SHAPE;
   if (!pos || !src || !count || !row0 || !rows || !expert || max_units < 1) return CB_ERR_ARG;
@@ -316,13 +331,13 @@ CB_EXPORT int cb_routed_units(const void* logits, int64_t ldl, const void* corr,
 #undef CB_UNITS
 }
 
-// fp32 expert product over a unit list (any number of units): y[r] = W[expert] x[src[r]] (src null: x[r]), squared relu with relu2.
+// fp32 expert product over a unit list (any number of units): y[r] = act(W[expert] x[src[r]]) (src null: x[r]); act as cb_gemv_units.
 CB_EXPORT int cb_routed_linear_f32(const void* W, int64_t stride, const void* x, int64_t ldx, void* y, int64_t ldy, int64_t N, int64_t K,
                                    const void* count, const void* row0, const void* rows, const void* expert, const void* src,
-                                   int64_t max_units, int64_t relu2, void* stream) {
+                                   int64_t max_units, int64_t act, void* stream) {
   if (!W || !x || !y || !count || !row0 || !rows || !expert || N < 1 || K < 1 || max_units < 1) return CB_ERR_ARG;
   const dim3 grid((unsigned)((N + 7) / 8), (unsigned)(max_units < 4096 ? max_units : 4096));
   return (int)cb_launch(routed_linear_f32_kernel, grid, dim3(256), 0, (cudaStream_t)stream, (const float*)W, stride, (const float*)x, ldx,
                         (float*)y, ldy, (int)N, (int)K, (const int*)count, (const int*)row0, (const int*)rows, (const int*)expert,
-                        (const int*)src, (int)relu2);
+                        (const int*)src, (int)act);
 }

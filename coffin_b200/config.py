@@ -205,6 +205,9 @@ def preset(name: str) -> ModelConfig:
     if "fasolorn" in name:
         from .models.fasolorn.config import preset_fasolorn
         return preset_fasolorn(name)
+    if "nodutar" in name:
+        from .models.nodutar.config import preset_nodutar
+        return preset_nodutar(name)
     if name == "tiny-moe":
         return ModelConfig(name="tiny-moe", num_experts=8, num_experts_per_tok=2,
                            moe_intermediate_size=128, shared_expert_intermediate_size=128,
@@ -259,4 +262,7 @@ def load_config(model_dir: str | Path):
     if str(raw.get("architecture", "")).lower() == "fasolorn":
         from .models.fasolorn.config import FasolornConfig
         return FasolornConfig.from_hf(raw, name=Path(model_dir).name)
+    if str(raw.get("architecture", "")).lower() == "nodutar":
+        from .models.nodutar.config import NodutarConfig
+        return NodutarConfig.from_hf(raw, name=Path(model_dir).name)
     return ModelConfig.from_hf(raw, name=Path(model_dir).name)

@@ -77,35 +77,23 @@ def _ensure_builtin() -> None:
     for n in ("qwen4_exp", "qwen4exp"):
         register(n, qwen4)
 
-    def zufilorn(cfg, sd, **kw):
-        from .zufilorn.model import ZufilornModel
+    for n, cls in _ROW_FAMILIES.items():
+        register(n, _row_family(n, cls))
+
+
+#: families on ``models.rowmodel`` and their classes
+_ROW_FAMILIES = {"zufilorn": "ZufilornModel", "sukisun": "SukisunModel", "fasolorn": "FasolornModel", "nodutar": "NodutarModel"}
+
+
+def _row_family(name: str, cls: str) -> Callable:
+    def make(cfg, sd, **kw):
+        import importlib
         if any(kw.pop(k + "_world", 1) > 1 for k in ("tp", "pp", "ep")):
-            raise NotImplementedError("the Zufilorn family runs on one GPU")
+            raise NotImplementedError(f"the {name.capitalize()} family runs on one GPU")
         for k in ("tp_rank", "pp_rank", "ep_rank"):
             kw.pop(k, None)
-        return ZufilornModel(cfg, sd, **kw)
-
-    register("zufilorn", zufilorn)
-
-    def sukisun(cfg, sd, **kw):
-        from .sukisun.model import SukisunModel
-        if any(kw.pop(k + "_world", 1) > 1 for k in ("tp", "pp", "ep")):
-            raise NotImplementedError("the Sukisun family runs on one GPU")
-        for k in ("tp_rank", "pp_rank", "ep_rank"):
-            kw.pop(k, None)
-        return SukisunModel(cfg, sd, **kw)
-
-    register("sukisun", sukisun)
-
-    def fasolorn(cfg, sd, **kw):
-        from .fasolorn.model import FasolornModel
-        if any(kw.pop(k + "_world", 1) > 1 for k in ("tp", "pp", "ep")):
-            raise NotImplementedError("the Fasolorn family runs on one GPU")
-        for k in ("tp_rank", "pp_rank", "ep_rank"):
-            kw.pop(k, None)
-        return FasolornModel(cfg, sd, **kw)
-
-    register("fasolorn", fasolorn)
+        return getattr(importlib.import_module(f".{name}.model", __package__), cls)(cfg, sd, **kw)
+    return make
 
 
 #: kernel sources a family needs; families without an entry use the whole library
@@ -113,13 +101,15 @@ _KERNELS: dict[str, tuple[str, ...]] = {
     "zufilorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "streams.cu",
                  "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
     "sukisun": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "depth.cu", "linrec.cu", "ssd.cu",
-                "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
+                "latent.cu", "rope.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
     "fasolorn": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "residual.cu", "routed.cu", "gemv_units.cu",
-                 "moe.cu", "latent.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
+                 "moe.cu", "latent.cu", "rope.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
+    "nodutar": ("elementwise.cu", "gemm_tc.cu", "gemm_tc2.cu", "gemv_mma.cu", "gemm_f32.cu", "residual.cu", "routed.cu", "gemv_units.cu",
+                "moe.cu", "rope.cu", "linrec.cu", "linrec_chunk.cu", "attn_maps.cu", "attn_maps_flash.cu", "attn_maps_tc.cu"),
 }
 
 #: families that also run in 32-bit (``dtype=torch.float32``)
-FLOAT32 = ("zufilorn", "sukisun", "fasolorn")
+FLOAT32 = tuple(_ROW_FAMILIES)
 
 
 def kernel_sources(arch: str) -> tuple[str, ...] | None:

@@ -1,4 +1,5 @@
-"""Routed feed-forward of the row-batch families: squared-relu experts, a corrected choice, identity experts, a shared expert.
+"""Routed feed-forward of the row-batch families: squared-relu or gated silu experts, a choice by corrected scores or by logits,
+identity experts, a shared expert.
 
 The shared expert rides with the routed ones: cut into parts of about an expert's width (exact, the activation works on single
 columns), its parts are stored behind the experts and every token holds a slot for each with weight one.  So a step is
@@ -22,23 +23,31 @@ MAX_PARTS = 16
 
 
 class RoutedExperts:
-    def __init__(self, W: dict[str, torch.Tensor], *, experts: int, identity: int, top: int, scale: float, ff: int, shared: int, width: int,
-                 dtype, dev) -> None:
-        """``W``: ``e<i>.up`` / ``e<i>.down``, ``router``, ``correction`` and, with ``shared`` > 0, ``shared.up`` / ``shared.down``."""
+    def __init__(self, W: dict[str, torch.Tensor], *, experts: int, identity: int = 0, top: int, scale: float = 1.0, ff: int, shared: int = 0,
+                 width: int, dtype, dev, gated: bool = False, by_logit: bool = False, correction: str = "correction") -> None:
+        """``W``: ``e<i>.up`` / ``e<i>.down`` (``gated``: and ``e<i>.gate``, the activation is ``silu(gate) * up`` instead of the squared
+        relu of up), ``router``, its ``correction`` under that name and, with ``shared`` > 0, ``shared.up`` / ``shared.down``
+        (/ ``shared.gate``).  ``by_logit``: as ``ops.routed.Router``."""
         step = max(ff, -(-shared // MAX_PARTS))                   # columns of a part
         parts = -(-shared // step)
-        self.r = R.Router(experts, identity, top, scale, parts)
+        self.r = R.Router(experts, identity, top, scale, parts, by_logit)
+        self.gated = gated
         I, W8 = pad8(step), pad8(width)
-        self.up = torch.zeros(experts + parts, I, W8, dtype=dtype, device=dev)
+        # gate rows of an expert come before its up rows
+        self.up = torch.zeros(experts + parts, 2 * I if gated else I, W8, dtype=dtype, device=dev)
+        first = (("gate", 0), ("up", I)) if gated else (("up", 0),)
         self.down = torch.zeros(experts + parts, W8, I, dtype=dtype, device=dev)
         for e in range(experts):
-            self.up[e, :ff, :width], self.down[e, :width, :ff] = W[f"e{e}.up"].to(dev, dtype), W[f"e{e}.down"].to(dev, dtype)
+            for n, o in first:
+                self.up[e, o:o + ff, :width] = W[f"e{e}.{n}"].to(dev, dtype)
+            self.down[e, :width, :ff] = W[f"e{e}.down"].to(dev, dtype)
         for p in range(parts):
             a, b = p * step, min(shared, (p + 1) * step)
-            self.up[experts + p, :b - a, :width] = W["shared.up"][a:b].to(dev, dtype)
+            for n, o in first:
+                self.up[experts + p, o:o + b - a, :width] = W[f"shared.{n}"][a:b].to(dev, dtype)
             self.down[experts + p, :width, :b - a] = W["shared.down"][:, a:b].to(dev, dtype)
         self.router = padded(W["router"], pad8(experts + identity), W8, dtype, dev)
-        self.correction = W["correction"].to(dev, torch.float32).contiguous()
+        self.correction = W[correction].to(dev, torch.float32).contiguous()
 
     def weights(self) -> list[torch.Tensor]:
         """What a step of one token streams."""
@@ -47,7 +56,8 @@ class RoutedExperts:
 
     def run(self, model, b: RowBatch, h: torch.Tensor) -> dict:
         """Keywords of the ``residual_step`` that merges the result."""
-        r, T, I, W8 = self.r, b.T, self.up.shape[1], self.up.shape[2]
+        r, T, I, W8 = self.r, b.T, self.down.shape[2], self.up.shape[2]
+        relu2, swiglu = not self.gated, self.gated
         S = T * r.slots
         logits = model.buf("route_z", T, self.router.shape[0], torch.float32)
         product = None
@@ -66,9 +76,13 @@ class RoutedExperts:
             disp = K.moe_dispatch(idx, r.stored, R.UNIT if model.f32 else 128)
         inter, y = model.buf("route_h", S, I), model.buf("route_y", S, W8)
         if units or model.f32:
-            R.unit_linear(self.up, h, inter, disp, rows=T, gather=True, relu2=True)
+            R.unit_linear(self.up, h, inter, disp, rows=T, gather=True, relu2=relu2, swiglu=swiglu)
             R.unit_linear(self.down, inter, y, disp, rows=T, gather=False, follows=True)
         else:
-            K.gemm_grouped(h.index_select(0, disp["src_tok"]), self.up, disp, out=inter, relu2=True)
+            rows = h.index_select(0, disp["src_tok"])
+            if swiglu:
+                K.swiglu(K.gemm_grouped(rows, self.up, disp, out=model.buf("route_gu", S, 2 * I)), out=inter)
+            else:
+                K.gemm_grouped(rows, self.up, disp, out=inter, relu2=True)
             K.gemm_grouped(inter, self.down, disp, out=y)
         return {"experts": (y, disp["pos"], w, idw if r.identity else None, h)}

@@ -6,13 +6,15 @@ base) is an argument, so a model family picks what it needs:
 
 * ``streams_embed`` / ``streams_step``: a residual of several fp32 streams with static read / write / mixing weights;
 * ``depth_embed`` / ``depth_step``: a residual that becomes a weighted sum of all layer results after every layer;
-* ``Linrec``: recurrences with a matrix state - the per-channel gated delta rule, the mLSTM matrix memory and the
-  state space with scalar decays (Mamba-2); ``gated_norm``: its output gate and grouped RMS norm;
+* ``Linrec``: recurrences with a matrix state - the per-channel gated delta rule, the mLSTM matrix memory, forget gates that
+  also write (HGRN2) and the state space with scalar decays (Mamba-2); ``gated_norm``: its output gate and grouped RMS norm;
 * ``AttnMaps``: paged attention with several score maps per head over the same values, capped scores, a
-  position-dependent query temperature, a sliding window, sinks, rotary positions, mixed values and gates per element;
+  position-dependent query temperature, a sliding window or chunks, sinks, rotary positions (of values too), norms of queries
+  and keys, penalties by the logarithm of the distance, keys that are their own values, mixed values and gates per element;
 * ``LatentAttn``: attention over cached low-rank latents with a rotated key part shared by all heads; ``rope_rows`` /
   ``rope_heads``: rotary angles of a batch and interleaved rotation of head parts;
-* ``residual_embed`` / ``residual_step``: a plain fp32 residual whose boundaries also merge expert rows;
+* ``residual_embed`` / ``residual_step``: a plain fp32 residual whose boundaries also merge expert rows, norm what they add
+  and repeat the embedding;
 * ``gemm_f32out`` / ``gemm_f32``: projections whose result (or everything) stays fp32; ``linear_xielu``: a projection
   with xIELU in its epilogue.
 """
@@ -26,7 +28,7 @@ from . import _lib
 from . import kernels as K
 from ._lib import call
 
-DELTA, MLSTM, SSD = 0, 1, 2
+DELTA, MLSTM, SSD, GATED = 0, 1, 2, 3
 RING = 16             # shallowest convolution ring
 _P, _I64, _I32, _F = ctypes.c_void_p, ctypes.c_int64, ctypes.c_int, ctypes.c_float
 
@@ -139,17 +141,21 @@ def residual_embed(embed: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, s
 
 
 def residual_step(x: torch.Tensor, h: torch.Tensor | None, *, gain: torch.Tensor | None = None, y: torch.Tensor | None = None,
-                  experts: tuple | None = None, rows: torch.Tensor | None = None, store: bool = True, eps: float = 1e-5) -> torch.Tensor | None:
+                  experts: tuple | None = None, post: torch.Tensor | None = None, again: tuple | None = None, rows: torch.Tensor | None = None,
+                  store: bool = True, eps: float = 1e-5) -> torch.Tensor | None:
     """Boundary between two sublayers: ``x [T, W] += y``, or with ``experts = (ys, pos, w, idw, hin)`` the weighted expert rows
-    ``sum_j w[t, j] ys[pos[t, j]] + idw[t] hin[t]``; then ``h = rmsnorm(x) * gain``.  ``rows`` picks the residual rows behind the rows
-    of ``h`` (with ``store=False``)."""
+    ``sum_j w[t, j] ys[pos[t, j]] + idw[t] hin[t]``; with ``post`` what is added is ``rmsnorm(that) * post``; with
+    ``again = (table, tokens)`` the embeddings are added too; then ``h = rmsnorm(x) * gain``.  ``rows`` picks the residual rows
+    behind the rows of ``h`` (with ``store=False``)."""
     T, W = x.shape
     n = rows.numel() if rows is not None else (h.shape[0] if h is not None else T)
     ys, pos, w, idw, hin = experts if experts is not None else (None,) * 5
-    t = next((v for v in (h, y, ys) if v is not None), None)
+    table, tokens = again if again is not None else (None, None)
+    t = next((v for v in (h, y, ys, table) if v is not None), None)
+    assert table is None or (table.is_contiguous() and table.shape[1] == W and table.dtype == t.dtype and tokens.dtype == torch.int64)
     ld = lambda v: v.stride(0) if v is not None else 0
     call("residual_step", x, y, ld(y), ys, ld(ys), pos, w, w.shape[1] if w is not None else 0, idw, hin, ld(hin), gain, h, ld(h), rows, n, W,
-         float(eps), int(store), _is_f32(t) if t is not None else 0)
+         float(eps), int(store), post, table, tokens, table.shape[0] if table is not None else 0, _is_f32(t) if t is not None else 0)
     K._count()
     return h
 
@@ -200,7 +206,7 @@ class _LinrecStruct(ctypes.Structure):
                 ("A_log", _P), ("dt_bias", _P), ("a2", _P), ("ra", _I64), ("a1_col", _I64), ("g2", _P), ("rg", _I64), ("g1_col", _I64),
                 ("norm_w", _P), ("gate_b", _P), ("S", _P), ("n", _P), ("m", _P), ("ring", _P), ("ring_mask", _I32), ("ring_w", _I64),
                 ("H", _I32), ("G", _I32), ("dk", _I32), ("dv", _I32), ("jc", _I32), ("k_col", _I64), ("v_col", _I64),
-                ("eps", _F), ("cap", _F), ("conv_b", _P), ("D", _P)]
+                ("eps", _F), ("cap", _F), ("conv_b", _P), ("D", _P), ("lower", _P)]
 
 
 def linrec_supported(H: int, dk: int, dv: int) -> bool:
@@ -212,20 +218,21 @@ class Linrec:
 
     ``state``: ``S [slots, H, dk, dv]`` and, by kind, ``ring [slots, depth, width]`` (delta: the last raw projection
     rows, indexed by position modulo depth) or ``n [slots, H, dk]`` and ``m [slots, H]`` (mLSTM), all zero at the
-    start of a sequence.  State space: keys, queries and values are B, C and x, the ring is the delta's, and the rows
+    start of a sequence.  Gated: the gate columns are the forget gates' pre-activations of all channels, ``gate_b`` their bias,
+    ``lower`` their lower bounds; there are no keys and no output gate.  State space: keys, queries and values are B, C and x, the ring is the delta's, and the rows
     that leave are fp32 and unnormed (``gated_norm`` follows)."""
 
     def __init__(self, kind: int, *, H: int, G: int, dk: int, dv: int, k_col: int, v_col: int, eps: float, state: dict,
                  norm_w: torch.Tensor | None = None, conv_w: torch.Tensor | None = None, A_log=None, dt_bias=None, a2=None,
-                 a1_col: int = 0, g2=None, g1_col: int = 0, gate_b=None, cap: float = 0.0, conv_b=None, D=None) -> None:
+                 a1_col: int = 0, g2=None, g1_col: int = 0, gate_b=None, cap: float = 0.0, conv_b=None, D=None, lower=None) -> None:
         if kind != SSD and not linrec_supported(H, dk, dv):
             raise ValueError(f"recurrent head of {dk} x {dv} is outside the kernel's range")
         a = self.a = _LinrecStruct()
         size = _lib.call_nostream("linrec_args_size")
         assert ctypes.sizeof(a) == size, f"argument layout: {ctypes.sizeof(a)} here, {size} in the library"
         self.kind, self.state, self.conv_w = kind, state, conv_w
-        self._keep = (norm_w, conv_w, A_log, dt_bias, a2, g2, gate_b, conv_b, D, *state.values())
-        a.conv_b, a.D = _ptr(conv_b), _ptr(D)
+        self._keep = (norm_w, conv_w, A_log, dt_bias, a2, g2, gate_b, conv_b, D, lower, *state.values())
+        a.conv_b, a.D, a.lower = _ptr(conv_b), _ptr(D), _ptr(lower)
         a.H, a.G, a.dk, a.dv, a.k_col, a.v_col, a.eps, a.cap = H, G, dk, dv, k_col, v_col, float(eps), float(cap)
         a.norm_w, a.conv_w, a.A_log, a.dt_bias, a.gate_b = _ptr(norm_w), _ptr(conv_w), _ptr(A_log), _ptr(dt_bias), _ptr(gate_b)
         a.taps = conv_w.shape[1] if conv_w is not None else 0
@@ -307,7 +314,8 @@ class _AttnStruct(ctypes.Structure):
                 ("H", _I32), ("G", _I32), ("maps", _I32), ("dim", _I32), ("vdim", _I32), ("nsplit", _I32), ("scale", _F), ("cap", _F),
                 ("temp_coef", _F), ("temp_every", _I32), ("ldk", _I64), ("ldv", _I64), ("act", _P), ("lda", _I64), ("gates", _P), ("ldg", _I64),
                 ("window", _I32), ("rot_half", _I32), ("sink", _P), ("cs", _P), ("v0", _P), ("ldv0", _I64), ("v_own", _F), ("v_mix", _F),
-                ("egate", _P), ("lde", _I64)]
+                ("egate", _P), ("lde", _I64), ("chunk", _I32), ("norm", _I32), ("eps", _F), ("qn", _P), ("kn", _P), ("vcs", _P), ("kr", _P), ("r1", _P),
+                ("r2", _P), ("oscale", _F)]
 
 
 MAX_VDIM = 512
@@ -323,10 +331,15 @@ class AttnMaps:
 
     def __init__(self, *, H: int, G: int, maps: int, dim: int, vdim: int, k_col: int, v_col: int, scale: float, cap: float | None,
                  temp: tuple[float, int] | None, kpool: torch.Tensor, vpool: torch.Tensor, finish: bool = True, window: int = 0,
-                 rot_dims: int = 0, sink: torch.Tensor | None = None) -> None:
+                 rot_dims: int = 0, sink: torch.Tensor | None = None, chunk: int = 0, norm: tuple | None = None,
+                 factors: torch.Tensor | None = None, distance: tuple | None = None, out_scale: float = 1.0) -> None:
         """``finish``: the heads will be finished by ``finish``, which bounds the value size.  ``window``: tokens a query sees,
         itself included (0: all).  ``rot_dims``: leading columns of queries and keys that turn, in neighbouring pairs, by the
-        angles of ``rows_of``.  ``sink`` (fp32 ``[H * maps]``): a score without key or value in every softmax."""
+        angles of ``rows_of``.  ``sink`` (fp32 ``[H * maps]``): a score without key or value in every softmax.  ``chunk``: a query
+        sees the tokens of its own chunk of this size.  ``norm = (eps, q weight, k weight)``: queries and keys are RMS-normed per
+        head before they turn (weights fp32 ``[dim]`` or None).  ``factors`` (fp32, a page's ``[G, 64]`` together): keys are cached as
+        projected and are the values, ``vpool`` is not used, and a key's factor takes its norm's place.  ``distance = (r1, r2)``
+        (fp32 ``[H]``): scores lose ``r1 ln(1 + r2 distance)``.  ``out_scale``: factor of the finished heads."""
         if (finish and vdim > MAX_VDIM) or maps not in (1, 2):
             raise ValueError(f"attention with {maps} maps and values of {vdim} is outside the kernels' range")
         a = self.a = _AttnStruct()
@@ -341,6 +354,14 @@ class AttnMaps:
         self.window, self.sink, self._egate = int(window), sink, None
         if temp is not None:
             a.temp_coef, a.temp_every = float(temp[0]), int(temp[1])
+        qn, kn = (norm[1], norm[2]) if norm is not None else (None, None)
+        r1, r2 = distance if distance is not None else (None, None)
+        a.chunk, a.norm, a.eps, a.qn, a.kn = int(chunk), int(norm is not None), float(norm[0]) if norm is not None else 0.0, _ptr(qn), _ptr(kn)
+        a.kr, a.r1, a.r2, a.oscale = _ptr(factors), _ptr(r1), _ptr(r2), float(out_scale)
+        self.chunk, self._vcs, self.out_scale, self._keep = int(chunk), None, float(out_scale), (qn, kn, r1, r2, factors)
+        self.keys_only = factors is not None
+        if self.keys_only and (maps != 1 or dim != vdim):
+            raise ValueError("keys that are their own values: one map, one size")
 
     def set_pools(self, kpool: torch.Tensor, vpool: torch.Tensor) -> None:
         """Rows of keys and values; they may be column ranges of wider rows."""
@@ -355,11 +376,13 @@ class AttnMaps:
         a.seg_row, a.seg_pos = _ptr(seg_row), _ptr(seg_pos)
 
     def rows_of(self, cs: torch.Tensor | None = None, egate: torch.Tensor | None = None, values: torch.Tensor | None = None,
-                lam: float = 0.0) -> None:
+                lam: float = 0.0, turns: torch.Tensor | None = None) -> None:
         """What the rows of the next calls carry beside their projection: angles ``cs [rows, rot_dims]``, output gate
         pre-activations ``egate [rows, H * vdim]`` (one map), and ``values [rows, G * vdim]`` of another layer, of which
-        ``lam`` is mixed into their own (both typed like the projection)."""
+        ``lam`` is mixed into their own (both typed like the projection).  ``turns [rows, vdim]``: angles by which values are turned
+        when they are cached and heads are turned back."""
         a = self.a
+        a.vcs, self._vcs = _ptr(turns), turns
         a.cs, a.egate, a.lde = _ptr(cs), _ptr(egate), egate.stride(0) if egate is not None else 0
         a.v0, a.ldv0, a.v_own, a.v_mix = _ptr(values), values.stride(0) if values is not None else 0, 1.0 - lam, lam
         self._egate = egate
@@ -399,7 +422,7 @@ class AttnMaps:
         R = self.H // self.G
         hpc = min(R, 8 // self.maps)
         resident = 296 if self.maps == 1 and max(self.dim, self.vdim) <= 128 else 148        # CTAs on the machine at once
-        return max(1, min(64, window_pages(self.window), resident // max(1, self.G * -(-R // hpc) * rows)))
+        return max(1, min(64, window_pages(self.window), window_pages(self.chunk), resident // max(1, self.G * -(-R // hpc) * rows)))
 
     def decode(self, proj, tables, positions, row_seg, part_o, part_ml, nsplit: int, act=None) -> None:
         """Single tokens (their keys and values are appended by the kernel): ``nsplit`` key splits per row.  With one map and one
@@ -415,8 +438,8 @@ class AttnMaps:
         element (``rows_of``)."""
         eg = self._egate
         call("attn_maps_finish", part_o, part_ml, gates, gates.stride(0) if gates is not None else 0, act, act.stride(0), positions,
-             positions.numel(), self.H, self.maps, self.vdim, nsplit, float(lam), float(post_scale), float(eps), self.sink,
-             eg, eg.stride(0) if eg is not None else 0, _is_f32(eg) if eg is not None else 0, _is_f32(act))
+             positions.numel(), self.H, self.maps, self.vdim, nsplit, float(lam), post_scale * self.out_scale, float(eps), self.sink,
+             eg, eg.stride(0) if eg is not None else 0, _is_f32(eg) if eg is not None else 0, self._vcs, _is_f32(act))
         K._count()
 
 

@@ -18,12 +18,14 @@ UNIT, UNIT_ROWS = 8, 64
 @dataclasses.dataclass(frozen=True)
 class Router:
     """``experts`` stored experts, then ``identity`` outputs that return the input; the ``top`` largest of score + correction are
-    chosen and weigh score / (their sum + 1e-20) * ``scale``; ``always`` more stored experts take every token with weight one."""
+    chosen and weigh score / (their sum + 1e-20) * ``scale``; ``always`` more stored experts take every token with weight one.
+    ``by_logit``: the ``top`` largest of logit + correction are chosen and weigh their softmax over the chosen ones, times ``scale``."""
     experts: int
     identity: int
     top: int
     scale: float
     always: int = 0
+    by_logit: bool = False
 
     @property
     def slots(self) -> int:
@@ -36,7 +38,7 @@ class Router:
 
 def _head(r: Router, logits: torch.Tensor, correction: torch.Tensor, positions: torch.Tensor | None) -> tuple:
     assert logits.dtype == correction.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= r.experts + r.identity
-    return logits, logits.stride(0), correction, positions, logits.shape[0], r.experts, r.identity, r.top, r.always, float(r.scale)
+    return logits, logits.stride(0), correction, positions, logits.shape[0], r.experts, r.identity, r.top, r.always, float(r.scale), int(r.by_logit)
 
 
 def route(r: Router, logits, correction, positions, idx, w, idw) -> None:
@@ -71,17 +73,20 @@ def meta_size(r: Router, T: int) -> int:
 
 
 def unit_linear(W: torch.Tensor, x: torch.Tensor, out: torch.Tensor, disp: dict, *, rows: int, gather: bool, relu2: bool = False,
-                follows: bool = False) -> torch.Tensor:
+                swiglu: bool = False, follows: bool = False) -> torch.Tensor:
     """``out[r] = W[expert(r)] @ x[src(r) if gather else r]`` for the sorted rows of a unit list (at most ``rows`` of them per unit).
-    ``follows``: the launch before this one is ``unit_linear`` over the same list."""
+    ``swiglu``: ``W`` holds gate rows, then as many up rows, and ``silu(gate) * up`` leaves.  ``follows``: the launch before this
+    one is ``unit_linear`` over the same list."""
     E, N, Kd = W.shape
+    act = 3 if swiglu else (2 if relu2 else 0)
+    N = N // 2 if swiglu else N
     assert x.stride(1) == 1 and x.shape[1] == Kd and W.is_contiguous()
     src = disp["src_tok"] if gather else None
     lists = (disp["count"], disp["row0"], disp["rows"], disp["expert"], src)
     if out.dtype == torch.float32:
-        call("routed_linear_f32", W, W.stride(0), x, x.stride(0), out, out.stride(0), N, Kd, *lists, disp["max_tiles"], int(relu2))
+        call("routed_linear_f32", W, W.stride(0), x, x.stride(0), out, out.stride(0), N, Kd, *lists, disp["max_tiles"], act)
     else:
-        call("gemv_units", W, W.stride(0), x, x.stride(0), out, out.stride(0), disp["max_tiles"], min(rows, UNIT), N, Kd, 2 if relu2 else 0,
+        call("gemv_units", W, W.stride(0), x, x.stride(0), out, out.stride(0), disp["max_tiles"], min(rows, UNIT), N, Kd, act,
              *lists, int(follows))
     K._count()
     return out

@@ -14,7 +14,7 @@ from pathlib import Path
 import torch
 
 KEEP_PREFIXES = ("model.language_model.", "mtp.", "lm_head.", "model.visual.")
-# flat naming (Zufilorn, Sukisun, Fasolorn): tables, ``l<layer>.<...>``, final norm and head at the top level
+# flat naming (Zufilorn, Sukisun, Fasolorn, Nodutar): tables, ``l<layer>.<...>``, final norm and head at the top level
 FLAT_KEYS = re.compile(r"(embed|pos|head|final\.norm|l(\d+)\..+)")
 
 

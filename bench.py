@@ -117,7 +117,8 @@ def main() -> None:
     ap.add_argument("--mma-kcta", type=int, default=0, help="tuning: max CTAs sharing one 16-row GEMV block (1 = off)")
     ap.add_argument("--mma-prefetch", type=int, default=-1, help="tuning: GEMV sweep rounds prefetched into L2 before the dependency wait")
     ap.add_argument("--gemv-impl", default="", help="tuning: mma | scalar")
-    ap.add_argument("--beside", default="", choices=["", "zufilorn-1b", "zufilorn-4b", "sukisun-1b", "sukisun-4b", "fasolorn-4b", "fasolorn-35b-a3b"],
+    ap.add_argument("--beside", default="", choices=["", "zufilorn-1b", "zufilorn-4b", "sukisun-1b", "sukisun-4b", "fasolorn-4b", "fasolorn-35b-a3b", "nodutar-35b-a3b",
+                                                        "nodutar-3b"],
                     help="instead of the headline workload: this model and the Qwen3.5 hybrid of the same width, layers, vocabulary and "
                          "feed-forwards, prefill and decode throughput at a few sizes")
     ap.add_argument("--layers", type=int, default=0, help="Qwen4-exp: cut the geometry to its first N layers")
@@ -425,7 +426,7 @@ def bench_qwen4(args, cfg, W: int) -> None:
 
 
 def bench_beside(args, W: int) -> None:
-    """Throughput of a Zufilorn, Sukisun or Fasolorn shape beside the Qwen3.5 hybrid of equal size (both random-init bf16): prefill of one
+    """Throughput of a Zufilorn, Sukisun, Fasolorn or Nodutar shape beside the Qwen3.5 hybrid of equal size (both random-init bf16): prefill of one
     prompt and CUDA-graph decode of 1, 8 and 32 sequences, device-timed with events over ``--steps`` repetitions after
     ``--warmup`` untimed ones.  One JSON line."""
     import dataclasses
@@ -435,8 +436,11 @@ def bench_beside(args, W: int) -> None:
     from coffin_b200.ops import kernels as K
     torch.cuda.set_device(0)
     new = preset(args.beside)
-    old = preset("qwen35-35b-a3b" if args.beside.endswith("-a3b") else "qwen35-4b")
-    if not args.beside.endswith(("-4b", "-a3b")):              # the same proportions at this width
+    old = preset("qwen35-35b-a3b" if args.beside.endswith("-a3b") or args.beside == "nodutar-3b" else "qwen35-4b")
+    if args.beside == "nodutar-3b":                            # half the width, depth and experts
+        old = dataclasses.replace(old, name="qwen35 3b, routed", hidden_size=1024, num_hidden_layers=20, layer_types=_pattern(20), num_attention_heads=8,
+                                  num_key_value_heads=1, linear_num_key_heads=8, linear_num_value_heads=16, num_experts=128)
+    elif not args.beside.endswith(("-4b", "-a3b")):              # the same proportions at this width
         f = 2560 // new.hidden_size
         old = dataclasses.replace(old, name=f"qwen35 at width {new.hidden_size}", vocab_size=new.vocab_size, hidden_size=new.hidden_size,
                                   num_hidden_layers=new.num_hidden_layers, layer_types=_pattern(new.num_hidden_layers),

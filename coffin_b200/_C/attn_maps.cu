@@ -78,7 +78,8 @@ __global__ void __launch_bounds__(256) maps_append8_kernel(const AttnMapsArgs a,
 }
 
 // The extended form: heads are normed, then turned; values may turn; keys that are their own values stay as projected, with their
-// factor beside them.  `lanes` (a power of two) threads per head, V columns per access.
+// factor beside them.  2^sh threads per head; V columns per access (8: bf16, a head is one access of its threads and stays in
+// registers).
 template <typename T, int V>
 __device__ __forceinline__ void load_cols(const T* p, int n, float* f) {
   if (V == 8) {
@@ -97,75 +98,107 @@ __device__ __forceinline__ void store_cols(T* p, int n, const float* f) {
     if (n > 1) act_store(p + 1, f[1]);
   }
 }
+// w[c ..] (n columns left) times r
+template <int V>
+__device__ __forceinline__ void weigh(float* f, const float* w, int n, float r) {
+  if (V == 8) {
+    const float4 a = *reinterpret_cast<const float4*>(w), b = *reinterpret_cast<const float4*>(w + 4);
+    const float g[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] *= r * g[i];
+  } else {
+    f[0] *= r * w[0];
+    if (n > 1) f[1] *= r * w[1];
+  }
+}
+template <int V>
+__device__ __forceinline__ void turn_cols(float* f, const float2* t, int pairs) {
+  if (V == 8 && pairs >= 4 && !((uintptr_t)t & 15)) {
+    const float4 a = *reinterpret_cast<const float4*>(t), b = *reinterpret_cast<const float4*>(t + 2);
+    const float c[4] = {a.x, a.z, b.x, b.z}, s[4] = {a.y, a.w, b.y, b.w};
+#pragma unroll
+    for (int i = 0; i < V / 2; ++i) {
+      const float x = f[2 * i], y = f[2 * i + 1];
+      f[2 * i] = x * c[i & 3] - y * s[i & 3];
+      f[2 * i + 1] = y * c[i & 3] + x * s[i & 3];
+    }
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < V / 2; ++i)
+    if (i < pairs) {
+      const float2 c = t[i];
+      const float x = f[2 * i], y = f[2 * i + 1];
+      f[2 * i] = x * c.x - y * c.y;
+      f[2 * i + 1] = y * c.x + x * c.y;
+    }
+}
 template <typename TP, typename TA, int V>
-__global__ void __launch_bounds__(256) maps_prep_kernel(const AttnMapsArgs a, int turn_q, int lanes) {
+__global__ void __launch_bounds__(512) maps_prep_kernel(const AttnMapsArgs a, int turn_q, int sh) {
   griddep_launch();
   griddep_wait();
   const int row = blockIdx.x, seg = a.row_seg ? a.row_seg[row] : row, pos = a.positions[row];
   if (pos < 0) return;
   const int64_t block = a.tables[(int64_t)seg * a.ldbt + pos / kPage], slot = block * kPage + pos % kPage;
   TP* p = reinterpret_cast<TP*>(const_cast<void*>(a.proj)) + (int64_t)row * a.ldp;
-  TA* kp = reinterpret_cast<TA*>(a.kpool) + slot * pool_ldk(a);
-  TA* vp = reinterpret_cast<TA*>(a.vpool) + slot * pool_ldv(a);
-  const float2* cs = a.cs + (int64_t)row * a.rot_half;
-  const float2* vcs = a.vcs ? a.vcs + (int64_t)row * (a.vdim / 2) : nullptr;
-  const TP* w = a.v0 ? reinterpret_cast<const TP*>(a.v0) + (int64_t)row * a.ldv0 : nullptr;
   const int nk = a.G * a.maps, nq = turn_q ? a.H * a.maps : 0, nv = a.kr ? 0 : a.G, total = nk + nq + nv;
-  const int per = 256 / lanes, l = threadIdx.x % lanes;
+  const int per = blockDim.x >> sh, l = threadIdx.x & ((1 << sh) - 1), stride = V << sh;
   for (int u0 = 0; u0 < total; u0 += per) {
-    const int u = u0 + threadIdx.x / lanes;
+    const int u = u0 + (threadIdx.x >> sh);
     const bool ok = u < total, key = u < nk, val = u >= nk + nq;
-    const int n = val ? a.vdim : a.dim;
-    TP* src = p + (key ? a.k_col + (int64_t)u * n : (val ? a.v_col + (int64_t)(u - nk - nq) * n : (int64_t)(u - nk) * n));
+    const int n = val ? a.vdim : a.dim, hd = key ? u : (val ? u - nk - nq : u - nk);      // columns of the head, its number
+    TP* src = p + (key ? a.k_col : (val ? a.v_col : 0)) + hd * n;
     float f[V], rstd = 1.f;
+    if (V == 8 && ok && l * V < n) load_cols<TP, V>(src + l * V, n, f);        // this thread's only columns
     if (a.norm) {
       float ss = 0.f;
       if (ok && !val)
-        for (int c = l * V; c < n; c += lanes * V) {
-          load_cols<TP, V>(src + c, n - c, f);
+        for (int c = l * V; c < n; c += stride) {
+          if (V != 8) load_cols<TP, V>(src + c, n - c, f);
 #pragma unroll
           for (int i = 0; i < V; ++i) ss = fmaf(f[i], f[i], ss);
         }
-      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      for (int o = 1 << sh >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
       rstd = 1.f / sqrtf(ss / (float)n + a.eps);
     }
     if (!ok) continue;                                           // the last pass
-    if (key && a.kr && l == 0) a.kr[factor_at(a, block, u / a.maps) + pos % kPage] = rstd;
     const bool as_is = key && a.kr;
-    const float* nw = val || as_is ? nullptr : (key ? a.kn : a.qn);
-    const float2* turn = val ? vcs : (as_is ? nullptr : cs);
-    const int half = val ? (vcs ? a.vdim / 2 : 0) : (as_is ? 0 : a.rot_half);
-    const float r = val || as_is ? 1.f : rstd;
-    for (int c = l * V; c < n; c += lanes * V) {
-      load_cols<TP, V>(src + c, n - c, f);
-      if (val && w) {
+    if (as_is && l == 0) a.kr[factor_at(a, block, hd) + pos % kPage] = rstd;
+    const float* nw = val ? nullptr : (key ? a.kn : a.qn);
+    const float2* turn = val ? a.vcs + (int64_t)row * (a.vdim / 2) : a.cs + (int64_t)row * a.rot_half;
+    const int half = val ? (a.vcs ? a.vdim / 2 : 0) : a.rot_half;
+    for (int c = l * V; c < n; c += stride) {
+      if (V != 8) load_cols<TP, V>(src + c, n - c, f);
+      if (val && a.v0) {
         float g[V];
-        load_cols<TP, V>(w + (src - p - a.v_col) + c, n - c, g);
+        load_cols<TP, V>(reinterpret_cast<const TP*>(a.v0) + (int64_t)row * a.ldv0 + hd * n + c, n - c, g);
 #pragma unroll
         for (int i = 0; i < V; ++i) f[i] = mixed(f[i], g[i], a);
       }
+      if (!as_is) {
+        if (nw) {
+          weigh<V>(f, nw + c, n - c, rstd);
+        } else if (!val) {
 #pragma unroll
-      for (int i = 0; i < V; ++i) f[i] *= nw && c + i < n ? r * nw[c + i] : r;
-#pragma unroll
-      for (int i = 0; i < V; i += 2)
-        if ((c + i) >> 1 < half) {
-          const float2 t = turn[(c + i) >> 1];
-          const float x = f[i], y = f[i + 1];
-          f[i] = x * t.x - y * t.y;
-          f[i + 1] = y * t.x + x * t.y;
+          for (int i = 0; i < V; ++i) f[i] *= rstd;
         }
-      if (key) store_cols<TA, V>(kp + (int64_t)u * n + c, n - c, f);
-      else if (val) store_cols<TA, V>(vp + (int64_t)(u - nk - nq) * n + c, n - c, f);
+        turn_cols<V>(f, turn + c / 2, half - c / 2);
+      }
+      if (key) store_cols<TA, V>(reinterpret_cast<TA*>(a.kpool) + slot * pool_ldk(a) + hd * n + c, n - c, f);
+      else if (val) store_cols<TA, V>(reinterpret_cast<TA*>(a.vpool) + slot * pool_ldv(a) + hd * n + c, n - c, f);
       else store_cols<TP, V>(src + c, n - c, f);
     }
   }
 }
 template <typename TP, typename TA, int V>
 int launch_prep(const AttnMapsArgs& a, int rows, int turn_q, cudaStream_t st) {
-  const int most = ((a.kr || a.dim > a.vdim ? a.dim : a.vdim) + V - 1) / V;
-  int lanes = 1;
-  while (lanes < 32 && lanes < most) lanes *= 2;
-  return (int)cb_launch(maps_prep_kernel<TP, TA, V>, dim3((unsigned)rows), dim3(256), 0, st, a, turn_q, lanes);
+  const int most = ((a.kr || a.dim > a.vdim ? a.dim : a.vdim) + V - 1) / V, total = (turn_q ? a.H + a.G : a.G) * a.maps + (a.kr ? 0 : a.G);
+  int sh = 0;
+  while (sh < 5 && 1 << sh < most) ++sh;
+  const int passes = ((total << sh) + 511) / 512, per = (total + passes - 1) / passes;     // as few threads as the passes need
+  int threads = ((per << sh) + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  return (int)cb_launch(maps_prep_kernel<TP, TA, V>, dim3((unsigned)rows), dim3((unsigned)threads), 0, st, a, turn_q, sh);
 }
 
 // One CTA per (query row, head, map): 128 keys at a time, scores by thread, running softmax, values by column.
@@ -430,7 +463,7 @@ CB_EXPORT int cb_attn_maps_append(const void* args, int64_t rows, int64_t turn_q
   if (extended(a)) {
     if (f32) return launch_prep<float, float, 2>(a, (int)rows, tq, st);
     if (p_f32) return launch_prep<float, bf16, 2>(a, (int)rows, tq, st);
-    const bool odd = a.dim % 8 || a.vdim % 8 || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || pool_ldk(a) % 8 || pool_ldv(a) % 8 || a.ldv0 % 8 ||
+    const bool odd = a.dim % 8 || a.vdim % 8 || a.dim > 256 || a.vdim > 256 || (((uintptr_t)a.qn | (uintptr_t)a.kn) & 15) || a.ldp % 8 || a.k_col % 8 || a.v_col % 8 || pool_ldk(a) % 8 || pool_ldv(a) % 8 || a.ldv0 % 8 ||
                      (((uintptr_t)a.proj | (uintptr_t)a.v0 | (uintptr_t)a.kpool | (uintptr_t)a.vpool) & 15);
     if (odd) return launch_prep<bf16, bf16, 2>(a, (int)rows, tq, st);
     return launch_prep<bf16, bf16, 8>(a, (int)rows, tq, st);

@@ -11,7 +11,9 @@
 //   gated :  u = v, k = 1 - f, decays per channel, no normaliser.
 //
 // `prep` (one CTA per chunk and head) computes those factors in fp32; `scan` (two warps per 16 value columns) walks
-// the chunks with S^T in accumulator registers.  The 32-bit quantities enter the products as a bf16 head plus a bf16
+// the chunks with S^T in accumulator registers.  A gated state is linear in its start, so where heads are few its scan is cut into
+// blocks of chunks that run side by side: `states` leaves what every block adds and how much of its start it keeps, and a
+// block of the scan folds the blocks before it first.  The 32-bit quantities enter the products as a bf16 head plus a bf16
 // remainder (three products, 16 mantissa bits), the sums and the state are fp32; `finish` applies the head norm and
 // the output gate.  A segment may start and end anywhere: its last chunk is padded with neutral tokens.
 #include "linrec.cuh"
@@ -29,7 +31,11 @@ struct ChunkArgs {
   float* gi; float* gf; float* gm; float* gb;   // mLSTM, [rows, H]: input log gate, forget log gate, m after / before the token
   float* nq;                 // mLSTM: n . q [rows, H]
   int segs;
+  // gated, blocks of `per` chunks (0: not cut): [entries, H, slices * kST, NT] float4 - the segment's first state, then what the
+  // blocks leave from nothing (the first from that state) - and the products of the blocks' decays [entries, H, DK]
+  float4* part; float* keep; int per;
 };
+__host__ __device__ __forceinline__ int64_t entry_index(int row0, int seg, int per) { return (int64_t)(row0 / (16 * per)) + 2 * seg; }
 
 // operand block, bf16 units, row pitch P = DK + 8:  X head [NX][P] | X remainder | K^ head [16][P] | K^ remainder |
 // T head [16][24] | T remainder | B head | B remainder | G fp32 [DK].   NX = 32 (k~ then q~) for delta, else 16 (q~).
@@ -453,37 +459,146 @@ __global__ void __launch_bounds__(kPT, 7) chunk_prep_gated_kernel(const ChunkArg
 // channels.  The halves' partial read-outs meet in shared memory once per chunk; both then know u and update their half
 // of the state.
 constexpr int kST = 128;
+// bf16 values of a chunk, staged as [token][32 columns] with pitch kVP: the fragments (columns x tokens) of column group cg
+constexpr int kVP = 40;
+__device__ __forceinline__ void value_frags(uint32_t* u, const bf16* vs, int cg, int lane) {
+  ldsm4t(u, vs + ((lane & 7) + ((lane >> 4) << 3)) * kVP + cg * 16 + ((lane >> 3) & 1) * 8);
+}
+// Gated: what a block of chunks leaves (all but the last of a segment), the same rows and columns per thread as in the scan.
+template <int DK, int STAGES>
+__global__ void __launch_bounds__(kST) chunk_states_kernel(const ChunkArgs ca, int slices) {
+  using I = Image<LINREC_GATED, DK>;
+  constexpr int P = I::P, NT = DK / 16, KB = 2 * C * P * 2;      // bytes of K^ head and remainder
+  constexpr int VB = C * kVP * 2, SB = KB + DK * 4 + VB;
+  const LinrecArgs& a = ca.r;
+  extern __shared__ __align__(16) unsigned char smem[];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, cg = warp >> 1, half = warp & 1, g4 = lane >> 2, t4 = lane & 3;
+  const int h = blockIdx.y, seg = blockIdx.z, kc = half * (DK / 2), slice = blockIdx.x % slices, blk = blockIdx.x / slices;
+  griddep_launch();
+  griddep_wait();
+  const int row0 = a.seg_row[seg], n = a.seg_row[seg + 1] - row0, slot = a.seg_slot[seg];
+  const int chunks = (n + C - 1) / C, c_lo = blk * ca.per, c_hi = c_lo + ca.per;
+  if (slot < 0 || n < 1 || c_hi >= chunks) return;               // the last block's state is the scan's
+  const int va = (slice * 2 + cg) * 16 + g4, vb = va + 8;
+  const int64_t entry = entry_index(row0, seg, ca.per) + blk;
+  float4* out = ca.part + ((entry * a.H + h) * slices + slice) * (kST * NT) + tid;
+  const int64_t ostep = (int64_t)a.H * slices * (kST * NT);      // next entry
+  const unsigned char* img = ca.image + (block_index(row0, seg, c_lo) * a.H + h) * I::bytes + tid * 16;
+  const size_t istep = (size_t)a.H * I::bytes;
+  const uint32_t sb = (uint32_t)__cvta_generic_to_shared(smem) + tid * 16;
+  const int vt = tid / 4, vc = slice * 32 + (tid % 4) * 8;       // token and first column this thread copies
+  const bool vok = vc < a.dv;
+  const bf16* vsrc = vok ? reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + c_lo * C + vt) * a.ldp + a.v_col + (int64_t)h * a.dv + vc
+                         : reinterpret_cast<const bf16*>(a.proj);
+  const int64_t vstep = vok ? C * a.ldp : 0;
+  const int vbytes = vok ? 16 : 0;
+  const uint32_t vdst = (uint32_t)__cvta_generic_to_shared(smem) + KB + DK * 4 + vt * kVP * 2 + (tid % 4) * 16;
+  auto load = [&](int ch, int stage) {                           // chunk of the block; every chunk of it is whole
+    const unsigned char* src = img + (size_t)ch * istep;
+    const uint32_t dst = sb + stage * SB;
+    constexpr int full = KB / 16 / kST, rest = KB / 16 % kST;
+#pragma unroll
+    for (int i = 0; i < full; ++i)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * kST * 16), "l"(src + I::kh * 2 + i * kST * 16) : "memory");
+    if (tid < rest)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + full * kST * 16), "l"(src + I::kh * 2 + full * kST * 16) : "memory");
+    if (tid < DK / 4) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + KB), "l"(src + I::g * 2) : "memory");
+    if (vt < C)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vdst + stage * SB), "l"(vsrc + ch * vstep), "r"(vbytes) : "memory");
+  };
+#pragma unroll
+  for (int s = 0; s < STAGES - 1; ++s) {
+    if (s < ca.per) load(s, s);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  float S[NT][4], keep[NT][2];
+  const bool keeps = slice == 0 && cg == 0;                      // the decays are the same for every column
+  const float* Sg = a.S + ((int64_t)slot * a.H + h) * a.dk * a.dv;
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    keep[i][0] = keep[i][1] = 1.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = kc + i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
+      S[i][e] = blk == 0 && c < a.dk && v < a.dv ? Sg[(int64_t)c * a.dv + v] : 0.f;
+    }
+    if (blk == 0) out[i * kST] = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+  }
+  int stage = 0;
+  for (int ch = 0; ch < ca.per; ++ch) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+    __syncthreads();
+    if (ch + STAGES - 1 < ca.per) load(ch + STAGES - 1, stage == 0 ? STAGES - 1 : stage - 1);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const unsigned char* st = smem + stage * SB;
+    const bf16* kh = reinterpret_cast<const bf16*>(st) + (lane & 15) * P + kc + (lane >> 4) * 8;
+    const float* G = reinterpret_cast<const float*>(st + KB) + kc + t4 * 2;
+    stage = stage + 1 == STAGES ? 0 : stage + 1;
+    uint32_t u[4];
+    value_frags(u, reinterpret_cast<const bf16*>(st + KB + DK * 4), cg, lane);
+#pragma unroll
+    for (int k = 0; k < NT / 2; ++k) {
+      uint32_t bh[4], bl[4];
+      ldsm4t(bh, kh + k * 16);
+      ldsm4t(bl, kh + C * P + k * 16);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float2 gg = *reinterpret_cast<const float2*>(G + (2 * k + i) * 8);
+        float* s = S[2 * k + i];
+        s[0] *= gg.x; s[1] *= gg.y; s[2] *= gg.x; s[3] *= gg.y;
+        if (keeps) { keep[2 * k + i][0] *= gg.x; keep[2 * k + i][1] *= gg.y; }
+        mma(s, u, bh[2 * i], bh[2 * i + 1]);
+        mma(s, u, bl[2 * i], bl[2 * i + 1]);
+      }
+    }
+  }
+  out += ostep;
+#pragma unroll
+  for (int i = 0; i < NT; ++i) out[i * kST] = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+  if (keeps && g4 == 0) {
+    float* kp = ca.keep + ((entry + 1) * a.H + h) * DK + kc + t4 * 2;
+#pragma unroll
+    for (int i = 0; i < NT; ++i) *reinterpret_cast<float2*>(kp + i * 8) = make_float2(keep[i][0], keep[i][1]);
+  }
+}
+
 template <int KIND, int DK, int STAGES>
-__global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
+__global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca, int slices) {
   using I = Image<KIND, DK>;
   constexpr int P = I::P, NT = DK / 16, NR = I::NX / 8;         // NT: n-tiles (8 channels) of this warp's half
   const LinrecArgs& a = ca.r;
   extern __shared__ __align__(16) unsigned char smem[];
   __shared__ float xch[4][NR * 4][32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, cg = warp >> 1, half = warp & 1, g4 = lane >> 2, t4 = lane & 3;
+  constexpr bool GAT = KIND == LINREC_GATED;
   const int h = blockIdx.y, seg = blockIdx.z, kc = half * (DK / 2);      // first channel of the half
+  const int slice = GAT ? (int)blockIdx.x % slices : (int)blockIdx.x, blk = GAT ? (int)blockIdx.x / slices : 0;
   griddep_launch();
   griddep_wait();
   const int row0 = a.seg_row[seg], n = a.seg_row[seg + 1] - row0, slot = a.seg_slot[seg];
   if (slot < 0 || n < 1) return;
-  const int chunks = (n + C - 1) / C;
+  const int all = (n + C - 1) / C, per = GAT && ca.per ? ca.per : all, first = blk * per, chunks = min(all, first + per) - first;
+  if (GAT && chunks < 1) return;
+  const bool cut = GAT && per < all, last = !cut || first + per >= all;
   // mLSTM: the slice after the value columns carries the normaliser as one column whose value is 1
   const bool nrm = KIND == LINREC_MLSTM && blockIdx.x == gridDim.x - 1;
-  const int v0 = nrm ? 0 : ((int)blockIdx.x * 2 + cg) * 16;
+  const int v0 = nrm ? 0 : (slice * 2 + cg) * 16;
   const int vlim = nrm ? (cg == 0 ? 1 : 0) : a.dv;               // columns that exist
   const int va = v0 + g4, vb = va + 8;
   const bool oka = va < vlim, okb = vb < vlim;
   const int64_t sstride = nrm ? 1 : a.dv;
   float* Sg = nrm ? a.n + ((int64_t)slot * a.H + h) * a.dk : a.S + ((int64_t)slot * a.H + h) * a.dk * a.dv;
   float S[NT][4];
+  if (!cut) {
 #pragma unroll
-  for (int i = 0; i < NT; ++i)
+    for (int i = 0; i < NT; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int c = kc + i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
-      S[i][e] = c < a.dk && v < vlim ? Sg[(int64_t)c * sstride + v] : 0.f;
-    }
-  const unsigned char* img = ca.image + (block_index(row0, seg, 0) * a.H + h) * I::bytes + tid * 16;
+      for (int e = 0; e < 4; ++e) {
+        const int c = kc + i * 8 + t4 * 2 + (e & 1), v = e >> 1 ? vb : va;
+        S[i][e] = c < a.dk && v < vlim ? Sg[(int64_t)c * sstride + v] : 0.f;
+      }
+  }
+  const unsigned char* img = ca.image + (block_index(row0, seg, first) * a.H + h) * I::bytes + tid * 16;
   const size_t istep = (size_t)a.H * I::bytes;
   const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(smem) + tid * 16;
   auto load = [&](int ch, int stage) {
@@ -497,27 +612,49 @@ __global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + full * kST * 16), "l"(src + full * kST * 16) : "memory");
   };
   // values of a chunk go through the same ring: [token][32 columns], pitch chosen against bank conflicts
-  constexpr int VE = KIND == LINREC_DELTA ? 4 : 2, VP = KIND == LINREC_DELTA ? 36 : 40, VB = C * VP * VE, VPER = 32 * VE / 16;   // 16-byte pieces a row
+  constexpr int VE = KIND == LINREC_DELTA ? 4 : 2, VP = KIND == LINREC_DELTA ? 36 : kVP, VB = C * VP * VE, VPER = 32 * VE / 16;   // 16-byte pieces a row
   const int64_t ldv = KIND == LINREC_DELTA ? (int64_t)a.H * a.dv : a.ldp;
-  const int vt = tid / VPER, vc = (int)blockIdx.x * 32 + (tid % VPER) * (16 / VE);          // token and first column this thread copies
+  const int vt = tid / VPER, vc = slice * 32 + (tid % VPER) * (16 / VE);          // token and first column this thread copies
   const char* vsrc = KIND == LINREC_DELTA
                          ? reinterpret_cast<const char*>(ca.v + (int64_t)(row0 + vt) * ldv + (int64_t)h * a.dv + vc)
-                         : reinterpret_cast<const char*>(reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + vt) * ldv + a.v_col +
+                         : reinterpret_cast<const char*>(reinterpret_cast<const bf16*>(a.proj) + (int64_t)(row0 + first * C + vt) * ldv + a.v_col +
                                                          (int64_t)h * a.dv + vc);
   const uint32_t vdst = (uint32_t)__cvta_generic_to_shared(smem) + STAGES * (uint32_t)I::bytes + vt * VP * VE + (tid % VPER) * 16;
   auto load_v = [&](int ch, int stage) {
     if (nrm || vt >= C) return;
-    const bool ok = ch * C + vt < n && vc < a.dv;                // 16-byte pieces never straddle dv (a multiple of 8)
+    const bool ok = (first + ch) * C + vt < n && vc < a.dv;                // 16-byte pieces never straddle dv (a multiple of 8)
     const char* src = ok ? vsrc + (int64_t)ch * C * ldv * VE : reinterpret_cast<const char*>(a.proj);
     const int bytes = ok ? 16 : 0;
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vdst + stage * VB), "l"(src), "r"(bytes) : "memory");
   };
-  float* op = nrm ? ca.nq + (int64_t)(row0 + half * 8 + t4 * 2) * a.H + h : ca.o + (int64_t)(row0 + half * 8 + t4 * 2) * ca.ldo_ + (int64_t)h * a.dv + va;
+  float* op = nrm ? ca.nq + (int64_t)(row0 + half * 8 + t4 * 2) * a.H + h : ca.o + (int64_t)(row0 + first * C + half * 8 + t4 * 2) * ca.ldo_ + (int64_t)h * a.dv + va;
   const int64_t ostep = nrm ? a.H : ca.ldo_;
 #pragma unroll
   for (int s = 0; s < STAGES - 1; ++s) {
     if (s < chunks) { load(s, s); load_v(s, s); }
     asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  if (cut) {                                                     // the state at the block's start, from the blocks before it
+    const int64_t e0 = entry_index(row0, seg, per), pstep = (int64_t)a.H * slices * (kST * NT);
+    const float4* pp = ca.part + ((e0 * a.H + h) * slices + slice) * (kST * NT) + tid + (blk ? pstep : 0);
+    const float* kp = ca.keep + ((e0 + 1) * a.H + h) * DK + kc + t4 * 2;
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const float4 f = pp[i * kST];
+      S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
+    }
+#pragma unroll 1
+    for (int j = 1; j < blk; ++j) {
+      pp += pstep;
+      kp += (int64_t)a.H * DK;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const float4 f = pp[i * kST];
+        const float2 g = *reinterpret_cast<const float2*>(kp + i * 8);
+        S[i][0] = fmaf(g.x, S[i][0], f.x); S[i][1] = fmaf(g.y, S[i][1], f.y);
+        S[i][2] = fmaf(g.x, S[i][2], f.z); S[i][3] = fmaf(g.y, S[i][3], f.w);
+      }
+    }
   }
   int stage = 0;
   for (int ch = 0; ch < chunks; ++ch) {
@@ -530,8 +667,11 @@ __global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
     float v[2][4];                                               // [token tile][row lo / hi, token 2t, 2t + 1]
-    {
-      const unsigned char* vs = smem + STAGES * I::bytes + stage * VB;
+    uint32_t vf[4];                                              // the same packed (gated)
+    const unsigned char* vs = smem + STAGES * I::bytes + stage * VB;
+    if (GAT) {
+      value_frags(vf, reinterpret_cast<const bf16*>(vs), cg, lane);
+    } else {
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -608,7 +748,7 @@ __global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
     } else {
 #pragma unroll
       for (int q = 0; q < 4; ++q) {                              // values are bf16: no remainder
-        uh[q] = pack_bf162(v[q >> 1][(q & 1) * 2], v[q >> 1][(q & 1) * 2 + 1]);
+        uh[q] = GAT ? vf[q] : pack_bf162(v[q >> 1][(q & 1) * 2], v[q >> 1][(q & 1) * 2 + 1]);
         ul[q] = 0;
       }
     }
@@ -641,13 +781,14 @@ __global__ void __launch_bounds__(kST) chunk_scan_kernel(const ChunkArgs ca) {
       mma(O, uh, b0, b1);
       mma(O2, uh, l0, l1);
       if (KIND == LINREC_DELTA) mma(O2, ul, b0, b1);
-      const int left = n - ch * C - half * 8 - t4 * 2;
+      const int left = n - (first + ch) * C - half * 8 - t4 * 2;
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if ((e & 1) < left && (e >> 1 ? okb : oka)) op[(e & 1) * ostep + (e >> 1) * 8] = O[e] + O2[e];
       op += C * ostep;
     }
   }
+  if (!last) return;
 #pragma unroll
   for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -701,6 +842,7 @@ __global__ void __launch_bounds__(128) chunk_finish_kernel(const ChunkArgs ca, i
   }
 }
 
+constexpr int kMinBlock = 8;           // chunks of a block of the gated scan, at least
 template <int KIND, int DK>
 int run_chunks(const ChunkArgs& ca, int max_rows, int rows, cudaStream_t st) {
   using I = Image<KIND, DK>;
@@ -733,13 +875,30 @@ int run_chunks(const ChunkArgs& ca, int max_rows, int rows, cudaStream_t st) {
     e = cb_launch(chunk_prep_mlstm_kernel<DK>, dim3((unsigned)chunks, (unsigned)a.H, (unsigned)ca.segs), dim3(64), smem, st, ca);
     if (e != cudaSuccess) return (int)e;
   }
-  constexpr int STAGES = DK <= 128 ? 4 : 3;
+  constexpr int STAGES = KIND == LINREC_GATED ? 3 : (DK <= 128 ? 4 : 3);
   auto scan = chunk_scan_kernel<KIND, DK, STAGES>;
-  const size_t smem = STAGES * (I::bytes + C * (KIND == LINREC_DELTA ? 36 * 4 : 40 * 2));
+  const size_t smem = STAGES * (I::bytes + C * (KIND == LINREC_DELTA ? 36 * 4 : kVP * 2));
   e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const int slices = (a.dv + 31) / 32 + (KIND == LINREC_MLSTM ? 1 : 0);
-  e = cb_launch(scan, dim3((unsigned)slices, (unsigned)a.H, (unsigned)ca.segs), dim3(kST), smem, st, ca);
+  int blocks = 1;
+  ChunkArgs cb = ca;
+  if constexpr (KIND == LINREC_GATED) {
+    const int resident = 148 * (DK <= 128 ? 3 : 1), base = slices * a.H * ca.segs;
+    const int want = resident / base < chunks / kMinBlock ? resident / base : chunks / kMinBlock;
+    if (want > 1) {
+      cb.per = (chunks + want - 1) / want;
+      blocks = (chunks + cb.per - 1) / cb.per;
+      constexpr int SS = 4;
+      auto states = chunk_states_kernel<DK, SS>;
+      const size_t sm = SS * (2 * C * I::P * 2 + DK * 4 + C * kVP * 2);
+      e = cudaFuncSetAttribute(states, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+      if (e != cudaSuccess) return (int)e;
+      if (blocks > 1) e = cb_launch(states, dim3((unsigned)(slices * (blocks - 1)), (unsigned)a.H, (unsigned)ca.segs), dim3(kST), sm, st, cb, slices);
+      if (e != cudaSuccess) return (int)e;
+    }
+  }
+  e = cb_launch(scan, dim3((unsigned)(slices * blocks), (unsigned)a.H, (unsigned)ca.segs), dim3(kST), smem, st, cb, slices);
   if (e != cudaSuccess) return (int)e;
   return (int)cb_launch(chunk_finish_kernel<KIND>, dim3((unsigned)(((int64_t)rows * a.H + 3) / 4)), dim3(128), 0, st, ca, rows);
 }
@@ -752,6 +911,14 @@ int64_t image_bytes(int64_t kind, int64_t dk) {
   return d == 32 ? Image<LINREC_MLSTM, 32>::bytes : (d == 64 ? Image<LINREC_MLSTM, 64>::bytes : (d == 128 ? Image<LINREC_MLSTM, 128>::bytes : Image<LINREC_MLSTM, 256>::bytes));
 }
 int64_t al(int64_t x) { return (x + 255) & ~(int64_t)255; }
+// entries of the gated scan's blocks, whatever their size
+int64_t part_entries(int64_t rows, int64_t segs) { return rows / (C * kMinBlock) + 2 * segs + 2; }
+int64_t part_bytes(int64_t kind, int64_t rows, int64_t segs, int64_t H, int64_t dk, int64_t dv) {
+  return kind == LINREC_GATED ? al(part_entries(rows, segs) * H * ((dv + 31) / 32) * 32 * padded_dk(dk) * 4) : 0;
+}
+int64_t keep_bytes(int64_t kind, int64_t rows, int64_t segs, int64_t H, int64_t dk) {
+  return kind == LINREC_GATED ? al(part_entries(rows, segs) * H * padded_dk(dk) * 4) : 0;
+}
 
 }  // namespace
 
@@ -761,7 +928,8 @@ CB_EXPORT int cb_linrec_chunk_ok(int64_t dk, int64_t dv) { return dk % 8 == 0 &&
 // Scratch bytes of a call over `rows` rows in `segs` segments.
 CB_EXPORT int64_t cb_linrec_chunk_scratch(int64_t kind, int64_t rows, int64_t segs, int64_t H, int64_t dk, int64_t dv) {
   const int64_t blocks = rows / C + segs + 2;
-  return al(blocks * H * image_bytes(kind, dk)) + 2 * al(rows * H * dv * 4) + 5 * al(rows * H * 4);
+  return al(blocks * H * image_bytes(kind, dk)) + 2 * al(rows * H * dv * 4) + 5 * al(rows * H * 4) +
+         part_bytes(kind, rows, segs, H, dk, dv) + keep_bytes(kind, rows, segs, H, dk);
 }
 
 // `segs` segments of the recurrence `kind`, rows [0, rows) of the projection; bf16 projection rows and activations,
@@ -786,6 +954,9 @@ CB_EXPORT int cb_linrec_chunk(const void* args, int64_t kind, int64_t segs, int6
   ca.ldo_ = (int64_t)a.H * a.dv;
   float** g[5] = {&ca.gi, &ca.gf, &ca.gm, &ca.gb, &ca.nq};
   for (int i = 0; i < 5; ++i) { *g[i] = (float*)p; p += al(rows * a.H * 4); }
+  ca.part = (float4*)p; p += part_bytes(kind, rows, segs, a.H, a.dk, a.dv);
+  ca.keep = (float*)p;
+  ca.per = 0;
   ca.segs = (int)segs;
   cudaStream_t st = (cudaStream_t)stream;
   const int d = padded_dk(a.dk);

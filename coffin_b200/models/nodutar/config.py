@@ -231,7 +231,7 @@ def preset_nodutar(name: str) -> NodutarConfig:
         f = 1 if name == "nodutar-35b-a3b" else 2
         W, runs, experts = 2048 // f, 40 // f, 256 // f
         ff = RoutedFF(512, experts, 9)
-        par = LayerSpec(PARALLEL, ParallelMixer(ChunkAttention(16 // f, 4 // f, 128, 128, 128 ** -0.5, 500000.0, 64, 1024), GatedState(16 // f, 128, 128),
+        par = LayerSpec(PARALLEL, ParallelMixer(ChunkAttention(16 // f, 4 // f, 128, 128, 128 ** -0.5, 500000.0, 64, 1280), GatedState(16 // f, 128, 128),
                                                 1.0, 1.0), ff)
         att = LayerSpec(ATTENTION, DistanceMixer(32 // f, 4 // f, 128, 128 ** -0.5), ff)
         layers = tuple(att if i % 4 == 3 else par for i in range(runs - 4))

@@ -423,6 +423,34 @@ def test_a_token_is_remembered_across_portions(dtype):
         assert rel(plain_mixer(layer, W, gone)[-1], ref[-1]) > 10 * TOL[BF16]
 
 
+@pytest.mark.parametrize("mem", [(2, 32, 24), (1, 128, 64), (3, 200, 40), (1, 16, 72)])
+def test_long_portions_of_unequal_length_scan_in_blocks(mem):
+    """One forward over portions from two tokens to hundreds, some continuing a state; memories that outlast a block of the scan."""
+    layer = right_only(*mem)
+    W, n = S.weights(S.config([layer], [None], width=64, eps=EPS), 7), mem[0] * mem[1]
+    W["l0.mix.right.f.b"] = torch.linspace(2, 8, n).bfloat16()
+    m = build(S.config([layer], [None], width=64, eps=EPS), W, BF16, blocks=60, max_seq=1300)
+    hs = [randn(30 + i, t, 64).bfloat16() for i, t in enumerate((900, 2, 300, 129))]
+    for i in range(4):
+        m.zero_state(i)
+    mix, tabs = m.layers[0].mixer, [table(900, 1), table(2, 20), table(300, 22), table(129, 30)]
+    at, got = [0] * 4, [[] for _ in range(4)]
+    for cuts in ((0, 2, 0, 129), (640, 0, 17, 0), (260, 0, 283, 0)):
+        live = [i for i in range(4) if cuts[i]]
+        b, _, first = m.make_batch([([0] * cuts[i], at[i], i, tabs[i]) for i in live])
+        hb = m.buf("h", b.T, 64)
+        for k, i in enumerate(live):
+            hb[first[k]:first[k] + cuts[i]].copy_(hs[i][at[i]:at[i] + cuts[i]])
+        y = m.linear(mix.w_out, mix.run(m, b, hb), m.buf("y", b.T, 64)).float().clone()
+        for k, i in enumerate(live):
+            got[i].append(y[first[k]:first[k] + cuts[i]])
+            at[i] += cuts[i]
+    m.check_status()
+    for g, h in zip(got, hs):
+        ref, g = plain_mixer(layer, W, h), torch.cat(g)
+        assert rel(g, ref) < TOL[BF16] and max(rel(g[i:i + 16], ref[i:i + 16]) for i in range(0, len(h), 16)) < 2 * TOL[BF16]
+
+
 # ------------------------------------------------------------------ whole models
 CONFIGS = {
     "all": S.ALL,

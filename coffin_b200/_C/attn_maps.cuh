@@ -46,7 +46,11 @@ struct AttnMapsArgs {
                                          //   projected and are the values too (vpool is not used) (null: no)
   const float* r1; const float* r2;      // [H]: score -= r1 ln(1 + r2 distance) (null: no)
   float oscale;                          // one map: factor of the finished head
+  float bound;                           // > 0: no score is larger, and no row's largest below -bound (norms bound them; at most
+                                         //   kMaxBound): the reference of every softmax instead of a running maximum
 };
+// 2^(-2 bound log2 e) stays well inside the range of fp32, and of a bf16 remainder 2^-9 below it
+constexpr float kMaxBound = 34.f;
 
 // first key that the query at `pos` sees
 __host__ __device__ __forceinline__ int first_key(const AttnMapsArgs& a, int pos) {

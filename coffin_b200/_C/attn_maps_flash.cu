@@ -279,26 +279,33 @@ int flash_dv(const AttnMapsArgs& a, int tiles, int segs, cudaStream_t st) {
 constexpr int kDT = 256;
 constexpr int decode_ctas(int dk, int dv, int maps) { return maps == 1 && dk <= 128 && dv <= 128 ? 2 : 1; }    // per SM
 // Forms: as described, with norms, turned values and distance penalties (one map), and the same with keys that are their own values.
-enum DecodeForm : int { BASIC = 0, NORMED = 1, KEYS_ONLY = 2 };
+// _FIXED: bounded scores (AttnMapsArgs.bound); a warp exponentiates its own scores, no maximum crosses the block.
+enum DecodeForm : int { BASIC = 0, NORMED = 1, KEYS_ONLY = 2, NORMED_FIXED = 3, KEYS_FIXED = 4 };
+constexpr bool keys_only(int form) { return form == KEYS_ONLY || form == KEYS_FIXED; }
+constexpr bool fixed_ref(int form) { return form == NORMED_FIXED || form == KEYS_FIXED; }
+// staged pages: keys alone leave room for more
+constexpr int decode_ring(int form, int dk, int dv) { return keys_only(form) ? 4 : (fixed_ref(form) && dk + dv <= 256 ? 3 : 2); }
 template <int DK, int DV, int MAPS, int FORM>
 constexpr size_t decode_smem() {
-  return sizeof(bf16) * (2 * (size_t)kPage * (MAPS * (DK + 8) + (FORM == KEYS_ONLY ? 0 : DV + 8)) + MAPS * 8 * (DK + 8) + 16 * (kPage + 8)) +
-         sizeof(float) * (8 * kPage + (FORM == KEYS_ONLY ? 2 * kPage : 0));
+  return sizeof(bf16) * (decode_ring(FORM, DK, DV) * (size_t)kPage * (MAPS * (DK + 8) + (keys_only(FORM) ? 0 : DV + 8)) + MAPS * 8 * (DK + 8) +
+                         (fixed_ref(FORM) ? 2 : 1) * 16 * (kPage + 8)) +
+         sizeof(float) * ((fixed_ref(FORM) ? 0 : 8 * kPage) + (keys_only(FORM) ? decode_ring(FORM, DK, DV) * kPage : 0));
 }
 template <int DK, int DV, int MAPS, typename TP, int FORM>
 __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_kernel(const AttnMapsArgs a, int hpc) {
-  constexpr bool KV = FORM == KEYS_ONLY;
+  constexpr bool KV = keys_only(FORM), FIX = fixed_ref(FORM);
   static_assert(FORM == BASIC || MAPS == 1, "one map");
   static_assert(!KV || DK == DV, "values are the keys");
   constexpr int LK = DK + 8, LV = DV + 8, KPAGE = MAPS * kPage * LK, VPAGE = kPage * LV, NP = DV / 16, NPW = (NP + 7) / 8;
+  constexpr int ST = decode_ring(FORM, DK, DV), PA = 16 * (kPage + 8);
   extern __shared__ __align__(128) unsigned char smem[];
-  bf16* ks = reinterpret_cast<bf16*>(smem);            // [2][MAPS][kPage][LK]
-  bf16* vs = KV ? ks : ks + 2 * KPAGE;                 // [2][kPage][LV]
-  bf16* qs = KV ? ks + 2 * KPAGE : vs + 2 * VPAGE;     // [MAPS][8][LK]
-  bf16* pa = qs + MAPS * 8 * LK;                       // [16][kPage + 8]: heads, remainders
-  float* ps = reinterpret_cast<float*>(pa + 16 * (kPage + 8));   // [8][kPage] scores
-  float* fs = ps + 8 * kPage;                          // [2][kPage] factors of the keys (KEYS_ONLY)
-  __shared__ float w_s[8], own_s;
+  bf16* ks = reinterpret_cast<bf16*>(smem);            // [ST][MAPS][kPage][LK]
+  bf16* vs = KV ? ks : ks + ST * KPAGE;                // [ST][kPage][LV]
+  bf16* qs = KV ? ks + ST * KPAGE : vs + ST * VPAGE;   // [MAPS][8][LK]
+  bf16* pa = qs + MAPS * 8 * LK;                       // [16][kPage + 8]: heads, remainders (FIXED: two of them)
+  float* ps = reinterpret_cast<float*>(pa + (FIX ? 2 : 1) * PA);   // [8][kPage] scores (not FIXED)
+  float* fs = ps + (FIX ? 0 : 8 * kPage);              // [ST][kPage] factors of the keys (KEYS_ONLY)
+  __shared__ float w_s[8], own_s, l_s[FIX ? kDT / 32 : 1][8];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3;
   const int split = blockIdx.x, row = blockIdx.z;
   const int R = a.H / a.G, cpg = (R + hpc - 1) / hpc, g = blockIdx.y / cpg, r0 = (blockIdx.y % cpg) * hpc, nh = min(hpc, R - r0);
@@ -324,15 +331,15 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
   auto load = [&](int pg) {
     const int64_t base = (int64_t)bt[pg] * kPage;
     const int n = pos + 1 - pg * kPage;                // keys of the page that exist
-    bf16* kd = ks + (pg & 1) * KPAGE;
-    bf16* vd = vs + (pg & 1) * VPAGE;
+    bf16* kd = ks + (pg % ST) * KPAGE;
+    bf16* vd = vs + (pg % ST) * VPAGE;
     for (int e = tid; e < MAPS * kPage * (DK / 8); e += kDT) {
       const int r = e / (MAPS * DK / 8), m = (e / (DK / 8)) % MAPS, c = (e % (DK / 8)) * 8;
       const bool ok = r < n && c < a.dim;
       cp16(kd + (m * kPage + r) * LK + c, ok ? K + (base + r) * ldk + m * a.dim + c : K, ok);
     }
     if (KV) {
-      if (tid < kPage / 4) cp16(fs + (pg & 1) * kPage + tid * 4, a.kr + factor_at(a, bt[pg], g) + tid * 4, true);
+      if (tid < kPage / 4) cp16(fs + (pg % ST) * kPage + tid * 4, a.kr + factor_at(a, bt[pg], g) + tid * 4, true);
     } else {
       for (int e = tid; e < kPage * (DV / 8); e += kDT) {
         const int r = e / (DV / 8), c = (e % (DV / 8)) * 8;
@@ -340,9 +347,12 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
         cp16(vd + r * LV + c, ok ? V + (base + r) * ldv + c : V, ok);
       }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  load(pg0);
+#pragma unroll
+  for (int i = 0; i < ST - 1; ++i) {
+    if (pg0 + i < pg1) load(pg0 + i);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
   const bool cap = a.cap > 0.f;
   const float f = a.scale * query_temp(a, pos) * (cap ? 2.f * kLog2e / a.cap : kLog2e), cap2 = a.cap * kLog2e;
   if (FORM == BASIC) {
@@ -384,23 +394,28 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
     }
   }
   const float r1 = FORM != BASIC && a.r1 && g4 < nh ? a.r1[g * R + r0 + g4] : 0.f, r2 = FORM != BASIC && a.r1 && g4 < nh ? a.r2[g * R + r0 + g4] : 0.f;
-  for (int e = tid; e < 16 * (kPage + 8); e += kDT) pa[e] = __float2bfloat16(0.f);
+  for (int e = tid; e < (FIX ? 2 : 1) * PA; e += kDT) pa[e] = __float2bfloat16(0.f);
   float o[NPW][2][4];
 #pragma unroll
   for (int i = 0; i < NPW; ++i)
 #pragma unroll
     for (int j = 0; j < 2; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
-  float m_run = -INFINITY, l_run = 0.f;                // of vector `warp`
+  const float ref = FIX ? a.bound * kLog2e : 0.f;
+  float m_run = FIX ? ref : -INFINITY, l_run = 0.f;    // of vector `warp` (FIXED: this lane's part of vector g4)
   for (int pg = pg0; pg < pg1; ++pg) {
-    if (pg + 1 < pg1) {
-      load(pg + 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    if (FIX) {                                         // one barrier ends the page before and starts this one
+      asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
+      __syncthreads();
+      if (pg + ST - 1 < pg1) load(pg + ST - 1);
+      asm volatile("cp.async.commit_group;" ::: "memory");
     } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      if (pg + ST - 1 < pg1) load(pg + ST - 1);
+      asm volatile("cp.async.commit_group;" ::: "memory");
+      asm volatile("cp.async.wait_group %0;" ::"n"(ST - 1) : "memory");
+      __syncthreads();
     }
-    __syncthreads();
-    bf16* kt = ks + (pg & 1) * KPAGE;
-    bf16* vt = vs + (pg & 1) * VPAGE;
+    bf16* kt = ks + (pg % ST) * KPAGE;
+    bf16* vt = vs + (pg % ST) * VPAGE;
     if (pg == pages - 1) {
       // the token's own key and value: into the staged page, and into the pool (CTAs of other heads of the group store
       // the same values)
@@ -435,7 +450,7 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
           *reinterpret_cast<uint32_t*>(K + slot * ldk + c) = xy;
         }
         if (KV) {
-          if (tid == 0) fs[(pg & 1) * kPage + r] = a.kr[factor_at(a, bt[pg], g) + r] = own_s;
+          if (tid == 0) fs[(pg % ST) * kPage + r] = a.kr[factor_at(a, bt[pg], g) + r] = own_s;
         } else {
           const float2* vcs = a.vcs + (int64_t)row * (a.vdim / 2);
           for (int c = (kDT - 1 - tid) * 2; c < a.vdim; c += 2 * kDT) {      // first the threads that had no key columns
@@ -471,12 +486,29 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
         mma(s, a0, b[0], b[1]);
         mma(s2, a1, b[2], b[3]);
       }
-      if (g4 < nh) {
+      if (FIX) {
+        float p[2];
+        const int key = warp * 8 + t4 * 2, left = pos - pg * kPage - key;      // distance of the first key
+        float2 kf = make_float2(1.f, 1.f);
+        if (KV) kf = *reinterpret_cast<const float2*>(fs + (pg % ST) * kPage + key);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float x = fmaf((s[e] + s2[e]) * f, e ? kf.y : kf.x, -ref);
+          if (a.r1) x = fmaf(-r1, lg2(fmaf(r2, (float)(left - e), 1.f)), x);
+          p[e] = left - e >= 0 && pg * kPage + key + e >= lo ? ex2(x) : 0.f;
+        }
+        if (g4 < nh) {
+          l_run += p[0] + p[1];
+          bf16* pw = pa + (pg & 1) * PA + g4 * (kPage + 8) + key;
+          *reinterpret_cast<uint32_t*>(pw) = split_head(p[0], p[1]);
+          *reinterpret_cast<uint32_t*>(pw + 8 * (kPage + 8)) = pack_bf162(p[0], p[1]);
+        }
+      } else if (g4 < nh) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           float x = (s[e] + s2[e]) * f;
           const int key = warp * 8 + t4 * 2 + e;
-          if (KV) x *= fs[(pg & 1) * kPage + key];
+          if (KV) x *= fs[(pg % ST) * kPage + key];
           if (cap) x = cap2 - __fdividef(2.f * cap2, ex2(x) + 1.f);
           if (FORM != BASIC && a.r1) x = fmaf(-r1, lg2(fmaf(r2, (float)(pos - pg * kPage - key), 1.f)), x);
           ps[(g4 * MAPS + m) * kPage + key] = pg * kPage + key <= pos && pg * kPage + key >= lo ? x : -INFINITY;
@@ -484,7 +516,7 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
       }
     }
     __syncthreads();
-    if (warp < nq) {
+    if (!FIX && warp < nq) {
       const float2 x = *reinterpret_cast<const float2*>(ps + warp * kPage + 2 * lane);
       const float mn = fmaxf(m_run, warp_max(fmaxf(x.x, x.y)));  // finite: a walked page holds a visible key
       float e0 = ex2(x.x - mn), e1 = ex2(x.y - mn);
@@ -495,17 +527,19 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
       *reinterpret_cast<uint32_t*>(pa + (8 + warp) * (kPage + 8) + 2 * lane) = pack_bf162(e0, e1);
       if (lane == 0) w_s[warp] = w;
     }
-    __syncthreads();
-    const float w = g4 < nq ? w_s[g4] : 0.f;
+    if (!FIX) __syncthreads();
+    const float w = FIX ? 1.f : (g4 < nq ? w_s[g4] : 0.f);
     uint32_t pf[4][4];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) ldsm4(pf[k], pa + (lane & 15) * (kPage + 8) + k * 16 + (lane >> 4) * 8);
+    for (int k = 0; k < 4; ++k) ldsm4(pf[k], pa + (FIX ? (pg & 1) * PA : 0) + (lane & 15) * (kPage + 8) + k * 16 + (lane >> 4) * 8);
 #pragma unroll
     for (int i = 0; i < NPW; ++i) {
       const int cp = warp + 8 * i;
       if (cp >= NP) break;
+      if (!FIX) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) { o[i][j][0] *= w; o[i][j][1] *= w; o[i][j][2] *= w; o[i][j][3] *= w; }
+        for (int j = 0; j < 2; ++j) { o[i][j][0] *= w; o[i][j][1] *= w; o[i][j][2] *= w; o[i][j][3] *= w; }
+      }
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         uint32_t b[4];
@@ -514,7 +548,16 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
         mma(o[i][1], pf[k], b[2], b[3]);
       }
     }
+    if (!FIX) __syncthreads();
+  }
+  if (FIX) {                                           // denominators: lanes of a vector, then warps; vector `warp` ends up in l_run
+    l_run += __shfl_xor_sync(0xffffffffu, l_run, 1);
+    l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
+    if (t4 == 0) l_s[warp][g4] = l_run;
     __syncthreads();
+    l_run = 0.f;
+#pragma unroll
+    for (int i = 0; i < kDT / 32; ++i) l_run += l_s[i][warp];
   }
   if (MAPS == 1 && a.act) {                            // the only split: the heads are finished here
     if (warp < nq && lane == 0) w_s[warp] = a.oscale / (l_run + (a.sink ? ex2(a.sink[g * R + r0 + warp] * kLog2e - m_run) : 0.f));
@@ -523,7 +566,7 @@ __global__ void __launch_bounds__(kDT, decode_ctas(DK, DV, MAPS)) maps_decode_ke
     const float inv = w_s[g4];
     const int hc = (g * R + r0 + g4) * a.vdim;
     bf16* out = reinterpret_cast<bf16*>(a.act) + (int64_t)row * a.lda + hc;
-    const float2* vcs = FORM == NORMED && a.vcs ? a.vcs + (int64_t)row * (a.vdim / 2) : nullptr;
+    const float2* vcs = FORM != BASIC && !KV && a.vcs ? a.vcs + (int64_t)row * (a.vdim / 2) : nullptr;
     const TP* eg = a.egate ? reinterpret_cast<const TP*>(a.egate) + (int64_t)row * a.lde + hc : nullptr;
 #pragma unroll
     for (int i = 0; i < NPW; ++i)
@@ -566,6 +609,7 @@ int decode_form(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
 template <int DK, int DV, int MAPS, typename TP>
 int decode_launch(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
   if constexpr (MAPS == 1) {
+    if (extended(a) && a.bound > 0.f) return decode_form<DK, DV, 1, TP, NORMED_FIXED>(a, hpc, rows, st);
     if (extended(a)) return decode_form<DK, DV, 1, TP, NORMED>(a, hpc, rows, st);
   }
   return decode_form<DK, DV, MAPS, TP, BASIC>(a, hpc, rows, st);
@@ -574,6 +618,7 @@ template <int DK, int MAPS, typename TP>
 int decode_dv(const AttnMapsArgs& a, int hpc, int rows, cudaStream_t st) {
   if constexpr (MAPS == 1) {
     constexpr int D = DK < 64 ? 64 : DK;
+    if (a.kr && a.bound > 0.f) return decode_form<D, D, 1, TP, KEYS_FIXED>(a, hpc, rows, st);
     if (a.kr) return decode_form<D, D, 1, TP, KEYS_ONLY>(a, hpc, rows, st);
   }
   if (a.vdim <= 64) return decode_launch<DK, 64, MAPS, TP>(a, hpc, rows, st);
@@ -621,6 +666,7 @@ CB_EXPORT int cb_attn_maps_decode(const void* args, int64_t rows, int64_t p_f32,
   if (!a.proj || !a.kpool || !a.vpool || !a.tables || !a.positions || a.H < 1 || a.G < 1 || a.H % a.G ||
       a.nsplit < 1 || a.nsplit > 64 || 2 * a.rot_half > a.dim || (a.rot_half && !a.cs) || !a.r1 != !a.r2)
     return CB_ERR_ARG;
+  if (a.bound > kMaxBound || (a.bound > 0.f && a.cap > 0.f)) return CB_ERR_ARG;
   if (extended(a) && (a.maps != 1 || (a.kr && (a.dim != a.vdim || a.vcs)))) return CB_ERR_SHAPE;
   if (!cb_attn_maps_tc_ok(a.G, a.maps, a.dim, a.vdim) || a.ldk % 8 || a.ldv % 8) return CB_ERR_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;

@@ -12,7 +12,8 @@
 // sums), released by the second; a key's factor comes with its page, and the penalty r1 ln(1 + r2 distance) is taken off.
 //
 // With a cap the scores are bounded, so the reference maximum is the cap itself (when 2^-2cap is far from underflow):
-// no row maximum, no exchange between the halves of a row, no rescale.  Otherwise the reference is raised lazily as in
+// no row maximum, no exchange between the halves of a row, no rescale.  The same where norms of queries and keys bound the
+// scores (FIXED, SHARED_FIXED: a distance penalty is never negative, and a token's own key has none).  Otherwise the reference is raised lazily as in
 // attn_tc.cu.  Waits are bounded by 2 s and report through the status word; TMEM is freed on every path.
 #include "attn_maps.cuh"
 #include "sm100.cuh"
@@ -22,7 +23,7 @@ using namespace sm100;
 
 constexpr int kBQ = 128, kBKV = 64, kThreads = 352;
 constexpr float kLog2e = 1.4426950408889634f;
-enum Mode : int { PLAIN = 0, CAP = 1, CAP_FIXED = 2, SHARED = 3 };
+enum Mode : int { PLAIN = 0, CAP = 1, CAP_FIXED = 2, SHARED = 3, FIXED = 4, SHARED_FIXED = 5 };
 
 __device__ __forceinline__ uint64_t now_ns() {
   uint64_t t;
@@ -56,7 +57,7 @@ constexpr int buffers(int dk, int dv) { return dk <= 128 && dv <= 128 ? 1 : 2; }
 template <int DK, int DV, int MODE, int STAGES>
 __global__ void __launch_bounds__(kThreads, 3 - buffers(DK, DV))
 maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const AttnMapsArgs a, int* status) {
-  constexpr bool KV = MODE == SHARED;
+  constexpr bool KV = MODE == SHARED || MODE == SHARED_FIXED, FIX = MODE == FIXED || MODE == SHARED_FIXED;
   static_assert(!KV || DK == DV, "values are the keys");
   constexpr int NK = DK / 64, NV = DV / 64;           // 64-element (128-byte) chunks
   constexpr int K_BYTES = kBKV * DK * 2, V_BYTES = KV ? 0 : kBKV * DV * 2, P_BYTES = kBQ * kBKV * 2;
@@ -203,11 +204,11 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
       if (lane == 0) mbar_arrive(&q_full);
     }
     // score -> log2 units; with a cap first to the exponent of exp(2 score / cap)
-    const float f = a.scale * query_temp(a, min(pos, pos0 + n - 1)) * (MODE == PLAIN || KV ? kLog2e : 2.f * kLog2e / a.cap);
+    const float f = a.scale * query_temp(a, min(pos, pos0 + n - 1)) * (MODE == PLAIN || KV || FIX ? kLog2e : 2.f * kLog2e / a.cap);
     const float r1 = KV && a.r1 ? a.r1[h] : 0.f, r2 = KV && a.r1 ? a.r2[h] : 0.f;
     const float cap2 = a.cap * kLog2e;
     const int key_lo = first_key(a, pos), full_lo = first_key(a, pos0 + row0 + kBQ - 1);
-    float m_ref = MODE == CAP_FIXED ? cap2 : -INFINITY, l = 0.f;
+    float m_ref = MODE == CAP_FIXED ? cap2 : (FIX ? a.bound * kLog2e : -INFINITY), l = 0.f;
     bool ok = true;
     uint32_t xph = 0;
     for (int j = 0; j < n_tiles; ++j) {
@@ -247,12 +248,21 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
             const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              float x = __uint_as_float(sv[c4 * 4 + e]) * f * kk[e];
+              float x = MODE == SHARED_FIXED ? fmaf(__uint_as_float(sv[c4 * 4 + e]) * f, kk[e], -m_ref) : __uint_as_float(sv[c4 * 4 + e]) * f * kk[e];
               if (a.r1) x = fmaf(-r1, lg2(fmaf(-r2, (float)(c4 * 4 + e), far)), x);      // NaN past the diagonal: masked below
               sv[c4 * 4 + e] = __float_as_uint(x);
             }
           }
         }
+        if (FIX) {
+#pragma unroll
+          for (int c = 0; c < 32; ++c) sv[c] = __float_as_uint(ex2(KV ? __uint_as_float(sv[c]) : fmaf(__uint_as_float(sv[c]), f, -m_ref)));
+          if (edge) {
+#pragma unroll
+            for (int c = 0; c < 32; ++c)
+              if (key0 + c > pos || key0 + c < key_lo) sv[c] = 0u;
+          }
+        } else {
         if (edge) {
 #pragma unroll
           for (int c = 0; c < 32; ++c)
@@ -295,6 +305,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 #pragma unroll
         for (int c = 0; c < 32; ++c)
           sv[c] = __float_as_uint(ex2(MODE == PLAIN ? fmaf(__uint_as_float(sv[c]), f, -m_ref) : __uint_as_float(sv[c]) - m_ref));
+        }
       }
       // head and remainder of the weights
       uint32_t ph[16], pr[16];
@@ -407,7 +418,7 @@ maps_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ 
 
 template <int DK, int DV, int MODE>
 int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
-  constexpr int NB = buffers(DK, DV), COLS = MODE == SHARED ? DK : DK + DV, STAGES = COLS > (NB == 1 ? 192 : 384) ? 2 : 3;
+  constexpr int NB = buffers(DK, DV), COLS = MODE == SHARED || MODE == SHARED_FIXED ? DK : DK + DV, STAGES = COLS > (NB == 1 ? 192 : 384) ? 2 : 3;
   const size_t smem = (size_t)STAGES * kBKV * COLS * 2 + 2 * NB * (size_t)kBQ * kBKV * 2 + 1024;
   auto kern = maps_tc_kernel<DK, DV, MODE, STAGES>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -418,8 +429,10 @@ int launch_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs
 template <int DK, int DV>
 int mode_tc(const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnMapsArgs& a, int tiles, int segs, int* status, cudaStream_t st) {
   if constexpr (DK == DV) {
+    if (a.kr && a.bound > 0.f) return launch_tc<DK, DV, SHARED_FIXED>(tmK, tmK, a, tiles, segs, status, st);
     if (a.kr) return launch_tc<DK, DV, SHARED>(tmK, tmK, a, tiles, segs, status, st);
   }
+  if (!(a.cap > 0.f) && a.bound > 0.f) return launch_tc<DK, DV, FIXED>(tmK, tmV, a, tiles, segs, status, st);
   if (!(a.cap > 0.f)) return launch_tc<DK, DV, PLAIN>(tmK, tmV, a, tiles, segs, status, st);
   // 2^(-2 cap log2e) well inside the range of fp32 and of a bf16 remainder 2^-16 below it
   if (a.cap <= 30.f) return launch_tc<DK, DV, CAP_FIXED>(tmK, tmV, a, tiles, segs, status, st);
@@ -442,7 +455,7 @@ CB_EXPORT int cb_attn_maps_flash_tc(const void* args, int64_t segs, int64_t max_
   if (a.act ? a.maps != 1 || a.lda % 8 || ((uintptr_t)a.act & 15) || a.lde % 8 || ((uintptr_t)a.egate & 15) : !a.part_o || !a.part_ml)
     return CB_ERR_ARG;
   if ((a.r1 && !a.kr) || (a.kr && (a.maps != 1 || a.dim != a.vdim || a.vcs || a.sink || a.egate || a.cap > 0.f || !a.act))) return CB_ERR_SHAPE;
-  if (a.vcs && (((uintptr_t)a.vcs & 15) || !a.act)) return CB_ERR_ARG;
+  if ((a.vcs && (((uintptr_t)a.vcs & 15) || !a.act)) || a.bound > kMaxBound) return CB_ERR_ARG;
   if (!cb_attn_maps_flash_tc_ok(a.dim, a.vdim) || !(a.scale > 0.f) || a.ldp % 8 || a.ldk % 8 || a.ldv % 8 || ((uintptr_t)a.proj & 15)) return CB_ERR_SHAPE;
   CUtensorMap tmK, tmV;
   const uint64_t kw = (uint64_t)a.G * a.maps * a.dim, vw = (uint64_t)a.G * a.vdim;

@@ -315,7 +315,11 @@ class _AttnStruct(ctypes.Structure):
                 ("temp_coef", _F), ("temp_every", _I32), ("ldk", _I64), ("ldv", _I64), ("act", _P), ("lda", _I64), ("gates", _P), ("ldg", _I64),
                 ("window", _I32), ("rot_half", _I32), ("sink", _P), ("cs", _P), ("v0", _P), ("ldv0", _I64), ("v_own", _F), ("v_mix", _F),
                 ("egate", _P), ("lde", _I64), ("chunk", _I32), ("norm", _I32), ("eps", _F), ("qn", _P), ("kn", _P), ("vcs", _P), ("kr", _P), ("r1", _P),
-                ("r2", _P), ("oscale", _F)]
+                ("r2", _P), ("oscale", _F), ("bound", _F)]
+
+
+#: largest bound of scores that serves as the reference of a softmax: weights down to exp(-2 bound) stay normal numbers
+MAX_BOUND = 34.0
 
 
 MAX_VDIM = 512
@@ -358,10 +362,21 @@ class AttnMaps:
         r1, r2 = distance if distance is not None else (None, None)
         a.chunk, a.norm, a.eps, a.qn, a.kn = int(chunk), int(norm is not None), float(norm[0]) if norm is not None else 0.0, _ptr(qn), _ptr(kn)
         a.kr, a.r1, a.r2, a.oscale = _ptr(factors), _ptr(r1), _ptr(r2), float(out_scale)
+        a.bound = self.bound = self._bound(scale, dim, norm, distance) if cap is None else 0.0
         self.chunk, self._vcs, self.out_scale, self._keep = int(chunk), None, float(out_scale), (qn, kn, r1, r2, factors)
         self.keys_only = factors is not None
         if self.keys_only and (maps != 1 or dim != vdim):
             raise ValueError("keys that are their own values: one map, one size")
+
+    @staticmethod
+    def _bound(scale: float, dim: int, norm: tuple | None, distance: tuple | None) -> float:
+        """What no score exceeds (a normed head's length is at most the root of its size, times its largest weight), or 0 if nothing
+        useful is known.  A margin covers the rounding of queries and keys; penalties have to take off, never add."""
+        if norm is None or (distance is not None and not bool(((distance[0] >= 0) & (distance[1] >= 0)).all())):
+            return 0.0
+        most = lambda w: float(w.abs().max()) if w is not None else 1.0
+        b = 1.02 * abs(scale) * dim * most(norm[1]) * most(norm[2])
+        return b if 0.0 < b <= MAX_BOUND else 0.0
 
     def set_pools(self, kpool: torch.Tensor, vpool: torch.Tensor) -> None:
         """Rows of keys and values; they may be column ranges of wider rows."""

@@ -111,6 +111,20 @@ def test_runs_of_a_layer_share_weights_but_not_pages_or_state(monkeypatch):
     assert made[5]["factors"] is d.pools[1] is not c.pools[1] and not c.state
 
 
+def test_bound_of_scores():
+    from coffin_b200.ops.mixers import MAX_BOUND, AttnMaps
+    one, two, r = torch.ones(16), torch.full((16,), -2.0), torch.tensor([0.5, 0.0])
+    assert AttnMaps._bound(0.25, 16, None, None) == 0 and AttnMaps._bound(0.25, 16, (1e-6, None, None), None) == pytest.approx(4.08)
+    assert AttnMaps._bound(-0.25, 16, (1e-6, two, one), (r, r)) == pytest.approx(8.16)
+    assert AttnMaps._bound(0.25, 16, (1e-6, None, None), (r, -r)) == 0 and AttnMaps._bound(MAX_BOUND / 16, 16, (1e-6, None, None), None) == 0
+
+
+def test_splits_cover_the_pages_of_a_chunk():
+    from coffin_b200.ops.mixers import window_pages
+    for size in (1, 2, 63, 64, 65, 66, 128, 130, 1000):
+        assert max(p // 64 - p // size * size // 64 + 1 for p in range(5 * size * 64)[:20000]) <= window_pages(size)
+
+
 def test_plain_model_ignores_what_comes_later_and_other_chunks():
     W = S.weights(S.ALL, 1)
     ids = [(7 * k) % 96 for k in range(12)]

@@ -239,7 +239,9 @@ def test_mixer_in_portions(name, dtype, cuts):
 
 @pytest.mark.parametrize("layer", [left_only(4, 2, 64, 64, 100, 32, scale=0.6), left_only(2, 1, 128, 256, 129, 128, scale=0.4), left_only(2, 2, 64, 128, 64, 8, scale=0.6),
                                    left_only(4, 1, 256, 64, 300, 64, scale=0.3), left_only(2, 1, 192, 192, 96, 64, scale=0.3), S.attention(4, 2, 64, 0.8), S.attention(2, 1, 128, 0.6),
-                                   S.attention(2, 1, 192, 0.4), S.attention(2, 2, 256, 0.3)])
+                                   S.attention(2, 1, 192, 0.4), S.attention(2, 2, 256, 0.3), left_only(4, 2, 64, 64, 100, 32, scale=0.1), left_only(4, 2, 128, 128, 200, 64, scale=0.06),
+                                   left_only(2, 1, 256, 128, 0, 64, scale=0.03), left_only(2, 2, 192, 192, 70, 64, scale=0.03), S.attention(4, 2, 64, 0.5), S.attention(2, 1, 128, 0.25),
+                                   S.attention(2, 1, 192, 0.15), S.attention(2, 2, 256, 0.12)])
 def test_prompt_attention_kernels_agree(layer):
     """tcgen05, mma.sync and the plain equations on prompts and long portions; peaky scores, so that the reference maximum is
     raised again and again, and chunks that leave whole pages of a tile to some of its rows."""
@@ -268,10 +270,27 @@ def test_key_splits(kind, nsplit, monkeypatch):
         assert rel(got[190:], ref[190:]) < TOL[BF16], chunk
 
 
-def test_splits_cover_the_pages_of_a_chunk():
-    from coffin_b200.ops.mixers import window_pages
-    for size in (1, 2, 63, 64, 65, 66, 128, 130, 1000):
-        assert max(p // 64 - p // size * size // 64 + 1 for p in range(5 * size * 64)[:20000]) <= window_pages(size)
+@pytest.mark.parametrize("layer", [left_only(6, 2, 64, 64, 150, 32, scale=0.1), left_only(3, 1, 32, 256, 0, 8, scale=0.2), left_only(4, 2, 256, 64, 90, 8, scale=0.03), S.attention(4, 2, 24),
+                                   S.attention(12, 1, 64, 0.4), S.attention(2, 1, 256, 0.1)])
+def test_bounded_scores_need_no_running_maximum(layer, monkeypatch):
+    """The same results with the bound as the softmax's reference and with running maxima, on prompts, portions and decode steps of
+    one and of several splits; scores at the bound itself and far below it."""
+    from coffin_b200.ops import mixers as X
+    W = S.weights(S.config([layer], [None], width=64), 3)
+    pre = "l0.mix.left." if layer["type"] == "parallel" else "l0.mix."
+    for n in ("q", "k"):                                           # one direction dominates: scores near plus and minus the bound
+        W[pre + n] = (W[pre + n].float() * 0.3 + 2.0 * torch.randn(W[pre + n].shape[0], 1) * torch.eye(64)[:1]).bfloat16()
+    h = randn(4, 230, 64)
+    h[:, 0] *= 3
+    h = h.bfloat16()
+    for cuts in ([230], [140, 1, 2], [1]):
+        for ns in (1, 3):
+            monkeypatch.setattr(X.AttnMaps, "decode_splits", lambda self, rows: ns)
+            a, ref = mixer_pair(layer, BF16, 230, cuts, h=h, W=W)
+            with monkeypatch.context() as mp:
+                mp.setattr(X.AttnMaps, "_bound", staticmethod(lambda *x: 0.0))
+                b, _ = mixer_pair(layer, BF16, 230, cuts, h=h, W=W)
+            assert rel(a, ref) < 2 * TOL[BF16] and rel(b, ref) < 2 * TOL[BF16] and rel(a, b) < 6e-3, (cuts, ns, rel(a, ref), rel(a, b))
 
 
 def standout(kind, chunk=0):

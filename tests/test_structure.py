@@ -114,7 +114,8 @@ def test_layering_lower_layers_do_not_import_upward():
 
 def test_every_preset_resolves_and_validates():
     from coffin_b200.config import preset
-    for name in ("tiny", "qwen35-4b", "qwen35-27b", "qwen35-35b-a3b", "tiny-qwen4", "qwen4exp-a", "tiny-fasolorn", "fasolorn-4b", "fasolorn-35b-a3b"):
+    for name in ("tiny", "qwen35-4b", "qwen35-27b", "qwen35-35b-a3b", "tiny-qwen4", "qwen4exp-a", "tiny-fasolorn", "fasolorn-4b", "fasolorn-35b-a3b",
+                 "tiny-nodutar", "nodutar-35b-a3b", "nodutar-3b"):
         cfg = preset(name)
         assert cfg.num_hidden_layers == len(cfg.layer_types)
         if hasattr(cfg, "validate"):
